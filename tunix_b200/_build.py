@@ -27,6 +27,8 @@ NVCC_FLAGS = [
     "--use_fast_math", "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden",
     "--expt-relaxed-constexpr",
 ]
+# kernels that also serve the 32-bit mode of a model (see csrc/precise.cuh) keep full-precision math functions
+PRECISE_SOURCES = {"stack.cu", "recurrent.cu", "window_attention.cu"}
 CXX_FLAGS = ["-O3", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread"]
 
 
@@ -57,7 +59,7 @@ def build_cuda(force: bool = False, verbose: bool = False) -> Path:
     sources = sorted(CSRC.glob("*.cu"))
     headers = sorted(CSRC.glob("*.cuh"))
     stamp = BUILD_DIR / "cuda.stamp"
-    digest = _digest(sources + headers, " ".join(NVCC_FLAGS))
+    digest = _digest(sources + headers, " ".join(NVCC_FLAGS + sorted(PRECISE_SOURCES)))
     if not force and CUDA_LIB.exists() and stamp.exists() and stamp.read_text() == digest:
         return CUDA_LIB
     BUILD_DIR.mkdir(parents=True, exist_ok=True)
@@ -67,10 +69,11 @@ def build_cuda(force: bool = False, verbose: bool = False) -> Path:
     def compile_one(src: Path) -> Path:
         obj = BUILD_DIR / (src.stem + ".o")
         ostamp = BUILD_DIR / (src.stem + ".stamp")
-        d = _digest([src], hdr_digest)
+        flags = [f for f in NVCC_FLAGS if f != "--use_fast_math" or src.name not in PRECISE_SOURCES]
+        d = _digest([src], hdr_digest + " ".join(flags))
         if not force and obj.exists() and ostamp.exists() and ostamp.read_text() == d:
             return obj
-        cmd = [nvcc, *NVCC_FLAGS, "-I", str(CSRC), "-c", str(src), "-o", str(obj)]
+        cmd = [nvcc, *flags, "-I", str(CSRC), "-c", str(src), "-o", str(obj)]
         if verbose:
             cmd.insert(1, "-Xptxas")
             cmd.insert(2, "-v")

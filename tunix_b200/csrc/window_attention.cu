@@ -1,0 +1,163 @@
+// Sliding-window attention over a paged cache with kept first tokens and a learned distance bias, for ragged batches.
+//
+//   qk_norm_write : after the fused projection of a step: RMS norm of q and of k over the WHOLE projection (all heads at
+//                   once), q to a compact buffer, k and v rows to their pages (value rows may be wider or narrower than
+//                   key rows).
+//   window_attn   : any head sizes, bf16 or float: one warp per (token, query head), lanes over keys for the scores and
+//                   over value columns for the output, online softmax in fp32. Position i sees j <= i with
+//                   i - j < window or j < keep. Models whose heads fit the tensor-core kernels (attention_fwd.cu,
+//                   decode.cu) use those instead.
+//
+// This file is compiled without fast-math: the same kernels serve the 32-bit mode.
+#include "precise.cuh"
+
+using namespace tb;
+
+namespace {
+
+struct Paged {
+  const int* table;
+  int max_pages, page_size;
+};
+
+__device__ __forceinline__ long long page_row(const Paged& pg, const int* pt, int p) {
+  return (long long)pt[p / pg.page_size] * pg.page_size + p % pg.page_size;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+qk_norm_write_kernel(const T* __restrict__ proj, long long ldp, int q_off, int k_off, int v_off, const T* __restrict__ qw,
+                     const T* __restrict__ kw, float eps, Ragged rb, Paged pg, int NQ, int NK, int NV, T* __restrict__ q,
+                     T* __restrict__ kp, T* __restrict__ vp) {
+  __shared__ float red[33];
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x, tid = threadIdx.x;
+  const int e = rb.ent[t], p0 = rb.pos0[e];
+  const T* row = proj + (long long)t * ldp;
+  if (p0 < 0) {
+    for (int c = tid; c < NQ; c += blockDim.x) q[(long long)t * NQ + c] = from_f<T>(0.f);
+    return;
+  }
+  float sq = 0.f, sk = 0.f;
+  for (int c = tid; c < NQ; c += blockDim.x) { const float v = to_f(row[q_off + c]); sq += v * v; }
+  for (int c = tid; c < NK; c += blockDim.x) { const float v = to_f(row[k_off + c]); sk += v * v; }
+  sq = block_sum(sq, red);
+  sk = block_sum(sk, red);
+  const float rq = 1.f / sqrtf(sq / (float)NQ + eps), rk = 1.f / sqrtf(sk / (float)NK + eps);
+  const int p = p0 + t - rb.cu[e];
+  const long long pr = page_row(pg, pg.table + (long long)rb.slot[e] * pg.max_pages, p);
+  for (int c = tid; c < NQ; c += blockDim.x) q[(long long)t * NQ + c] = from_f<T>(to_f(row[q_off + c]) * rq * to_f(qw[c]));
+  for (int c = tid; c < NK; c += blockDim.x) kp[pr * NK + c] = from_f<T>(to_f(row[k_off + c]) * rk * to_f(kw[c]));
+  for (int c = tid; c < NV; c += blockDim.x) vp[pr * NV + c] = row[v_off + c];
+}
+
+constexpr int VREG = 16;        // value columns per lane: value heads up to 512 wide
+
+template <typename T>
+__global__ void __launch_bounds__(128)
+window_attn_kernel(const T* __restrict__ q, const T* __restrict__ kp, const T* __restrict__ vp, Ragged rb, Paged pg, int H,
+                   int G, int dq, int dv, float scale, const float* __restrict__ bias, int far, int window, int keep,
+                   T* __restrict__ out) {
+  extern __shared__ float qs_all[];               // [4][dq]
+  pdl_trigger();
+  pdl_wait();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long wid = (long long)blockIdx.x * 4 + warp;
+  if (wid >= (long long)rb.n * H) return;
+  const int t = (int)(wid / H), h = (int)(wid - (long long)t * H), g = h / (H / G);
+  const int e = rb.ent[t], p0 = rb.pos0[e];
+  T* o = out + ((long long)t * H + h) * dv;
+  if (p0 < 0) {
+    for (int c = lane; c < dv; c += 32) o[c] = from_f<T>(0.f);
+    return;
+  }
+  float* qs = qs_all + warp * dq;
+  for (int d = lane; d < dq; d += 32) qs[d] = to_f(q[((long long)t * H + h) * dq + d]) * scale;
+  __syncwarp();
+  const int i = p0 + t - rb.cu[e];
+  const int lo = window > 0 ? max(0, i - window + 1) : 0;
+  const int kept = min(keep, lo);                 // keys 0 .. kept-1 lie before the window
+  const int cnt = kept + i - lo + 1;
+  const int* pt = pg.table + (long long)rb.slot[e] * pg.max_pages;
+  float m = -INFINITY, l = 0.f;
+  float acc[VREG];
+#pragma unroll
+  for (int r = 0; r < VREG; ++r) acc[r] = 0.f;
+  for (int b = 0; b < cnt; b += 32) {
+    const int x = b + lane;
+    float s = -INFINITY;
+    long long row = 0;
+    if (x < cnt) {
+      const int j = x < kept ? x : lo + x - kept;
+      row = page_row(pg, pt, j);
+      const T* k = kp + (row * G + g) * dq;
+      float dot = 0.f;
+      for (int d = 0; d < dq; ++d) dot += qs[d] * to_f(k[d]);
+      s = dot + bias[(long long)min(i - j, far) * H + h];
+    }
+    const float mn = fmaxf(m, warp_max(s));
+    const float p = expf(s - mn), c = expf(m - mn);
+    l = l * c + warp_sum(p);
+    m = mn;
+#pragma unroll
+    for (int r = 0; r < VREG; ++r) acc[r] *= c;
+    const int lim = min(32, cnt - b);
+    for (int y = 0; y < lim; ++y) {
+      const float py = __shfl_sync(0xffffffffu, p, y);
+      const long long ry = __shfl_sync(0xffffffffu, row, y);
+      const T* v = vp + (ry * G + g) * dv;
+#pragma unroll
+      for (int r = 0; r < VREG; ++r) {
+        const int cc = r * 32 + lane;
+        if (cc < dv) acc[r] += py * to_f(v[cc]);
+      }
+    }
+  }
+  const float inv = 1.f / l;
+#pragma unroll
+  for (int r = 0; r < VREG; ++r) {
+    const int cc = r * 32 + lane;
+    if (cc < dv) o[cc] = from_f<T>(acc[r] * inv);
+  }
+}
+
+}  // namespace
+
+#define RAGGED Ragged rb{cu, slot, pos0, ent, E, n}
+#define PAGED Paged pg{table, max_pages, page_size}
+
+// NQ = H * dq, NK = G * dq, NV = G * dv columns of proj [n, ldp]; pools [pages, page_size, NK] and [.., NV]; q [n, NQ].
+TB_API int tb_qk_norm_write(int dtype, const void* proj, long long ldp, int q_off, int k_off, int v_off, const void* qw,
+                            const void* kw, float eps, const int* cu, const int* slot, const int* pos0, const int* ent, int E,
+                            int n, const int* table, int max_pages, int page_size, int NQ, int NK, int NV, void* q, void* kp,
+                            void* vp, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  RAGGED;
+  PAGED;
+#define RUN(T)                                                                                                               \
+  return launch_pdl(qk_norm_write_kernel<T>, dim3(n), dim3(256), 0, stream, (const T*)proj, ldp, q_off, k_off, v_off,        \
+                    (const T*)qw, (const T*)kw, eps, rb, pg, NQ, NK, NV, (T*)q, (T*)kp, (T*)vp) == cudaSuccess ? 0 : -5
+  if (dtype == 0) RUN(__nv_bfloat16);
+  RUN(float);
+#undef RUN
+}
+
+// bias fp32 [far + 1, H]: what is added to the score of a key at distance min(i - j, far). window <= 0: no window.
+TB_API int tb_window_attn(int dtype, const void* q, const void* kp, const void* vp, const int* cu, const int* slot,
+                          const int* pos0, const int* ent, int E, int n, const int* table, int max_pages, int page_size, int H,
+                          int G, int dq, int dv, float scale, const float* bias, int far, int window, int keep, void* out,
+                          cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (G <= 0 || H % G || dv > VREG * 32 || dq > 3000) return -2;
+  RAGGED;
+  PAGED;
+  const long long warps = (long long)n * H;
+  const dim3 grid((unsigned)((warps + 3) / 4));
+#define RUN(T)                                                                                                              \
+  return launch_pdl(window_attn_kernel<T>, grid, dim3(128), (size_t)4 * dq * 4, stream, (const T*)q, (const T*)kp,           \
+                    (const T*)vp, rb, pg, H, G, dq, dv, scale, bias, far, window, keep, (T*)out) == cudaSuccess ? 0 : -5
+  if (dtype == 0) RUN(__nv_bfloat16);
+  RUN(float);
+#undef RUN
+}

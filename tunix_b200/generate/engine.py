@@ -15,6 +15,11 @@ slot and pages at the next check point and the next waiting request is prefilled
            the step counter and the page table from device memory, so the whole step is captured once in a
            CUDA graph and replayed; the host looks at the slots' done flags only every `check_every` steps.
 Outputs match `Sampler` (`SamplerOutput` with ragged tokens, optional per-token log-probs).
+
+Layer-stack models (`models/stack.py`) run through `models.stack_exec.StackExecutor` instead: one step function over
+ragged batches (prompt portions and decoded tokens side by side) that reads and writes the same page pool plus, for
+recurrent layers, fp32 states per slot (`SlotStates`). Admission, sampling, the captured decode step, pre-emption and the
+server are the same code. `StepSession` drives that step function by hand, token lists in and logits out.
 """
 from __future__ import annotations
 
@@ -32,6 +37,20 @@ from .base_sampler import BaseSampler, SamplerOutput
 from .sampler import next_power_of_2, pad_prompts_left
 
 
+class SlotStates:
+    """Recurrent state of every layer pass: fp32 tensors with one row per slot. A kernel that runs a sequence's first
+    token starts from zero whatever the slot held before, so a slot needs no clearing when its owner changes."""
+
+    def __init__(self, shapes: Sequence[dict], max_seqs: int, device):
+        self.tensors = [{k: torch.zeros((max_seqs, *s), dtype=torch.float32, device=device) for k, s in d.items()} for d in shapes]
+
+    def __getitem__(self, layer_pass: int) -> dict:
+        return self.tensors[layer_pass]
+
+    def nbytes_per_slot(self) -> int:
+        return sum(t[0].numel() * 4 for d in self.tensors for t in d.values())
+
+
 class PagePool:
     """Device page pools for every layer plus the host-side bookkeeping.
 
@@ -45,10 +64,15 @@ class PagePool:
                  prefix_caching: bool = True, kv_heads: Optional[int] = None):
         from ..experimental.generate import kv_cache_manager as kvm
         self.page_size, self.num_pages, self.max_pages = page_size, num_pages, max_pages_per_seq
-        row = (kv_heads or cfg.num_kv_heads) * cfg.head_dim       # a tensor-parallel rank keeps its own kv heads only
+        if hasattr(cfg, "kv_rows"):                # layer-stack models: rows and states per layer pass
+            rows, self.state = cfg.kv_rows(), SlotStates(cfg.state_shapes(), max_seqs, device)
+        else:
+            row = (kv_heads or cfg.num_kv_heads) * cfg.head_dim   # a tensor-parallel rank keeps its own kv heads only
+            rows, self.state = [(row, row)] * cfg.num_layers, None
         # zero-initialised: rows of a page that were never written must hold finite values
-        self.k = [torch.zeros(num_pages, page_size, row, dtype=dtype, device=device) for _ in range(cfg.num_layers)]
-        self.v = [torch.zeros(num_pages, page_size, row, dtype=dtype, device=device) for _ in range(cfg.num_layers)]
+        pages = lambda n: torch.zeros(num_pages, page_size, n, dtype=dtype, device=device)  # noqa: E731
+        self.k = [None if r is None else pages(r[0]) for r in rows]
+        self.v = [None if r is None else pages(r[1]) for r in rows]
         self.table_host = np.full((max_seqs, max_pages_per_seq), -1, np.int32)
         self.table = torch.full((max_seqs, max_pages_per_seq), -1, dtype=torch.int32, device=device)
         self.Error = kvm.PagePoolError
@@ -120,7 +144,9 @@ class PagedEngine(BaseSampler):
         self.cache_size = cache_config.cache_size
         self.device = next(transformer.parameters()).device
         self.dtype = next(transformer.parameters()).dtype
-        if self.device.type != "cuda" or self.dtype != torch.bfloat16:
+        # layer-stack models bring their own step function; they also run in 32-bit
+        self.exec = transformer.executor() if hasattr(transformer, "executor") else None
+        if self.device.type != "cuda" or (self.dtype != torch.bfloat16 and not (self.exec and self.dtype == torch.float32)):
             raise ValueError("PagedEngine runs bf16 models on CUDA; use Sampler elsewhere")
         if self.cfg.is_moe and getattr(transformer.layers[0].mlp, "ep", None) is not None:
             raise NotImplementedError("expert-parallel MoE decode goes through Sampler")
@@ -152,8 +178,9 @@ class PagedEngine(BaseSampler):
         # smaller pool makes requests wait for pages and, when running sequences outgrow it, sends the youngest one
         # back to the queue
         self.num_pages = num_pages
-        self.prefix_caching = prefix_caching
+        self.prefix_caching = prefix_caching and self.exec is None     # a recurrent state has no pages to share
         self.prefill_chunk = prefill_chunk      # > 0: prompts are prefilled in pieces of at most this many tokens
+        self.step_tokens = 16384                # layer-stack models: most tokens of one prefill step
         self.preemptions = 0
         self.forbidden: Optional[torch.Tensor] = None
         self.pool: Optional[PagePool] = None
@@ -228,6 +255,10 @@ class PagedEngine(BaseSampler):
         return joint
 
     def _fuse_all(self):
+        if self.exec is not None:
+            self.exec.refresh()
+            self.exec.pk = self._pk
+            return
         self._wqkv, self._wgu = [], []
         for layer in self._model.layers:
             at = layer.self_attn
@@ -246,8 +277,8 @@ class PagedEngine(BaseSampler):
         if not self.pack_weights:
             self._packed = None
             return
-        srcs = []
-        for i, layer in enumerate(self._model.layers):
+        srcs = self.exec.pack_sources() if self.exec is not None else []
+        for i, layer in enumerate(self._model.layers if self.exec is None else ()):
             at, mlp = layer.self_attn, layer.mlp
             dense = not self.cfg.is_moe
             srcs.append({"qkv": self._wqkv[i], "o": at.o_proj.weight.data if self._plain(at.o_proj) else None,
@@ -393,8 +424,38 @@ class PagedEngine(BaseSampler):
             x = self._mlp_and_norms(layer, i, x, a)
         return self._model.norm(x[:, -1])
 
+    def _prefill_ragged(self, work):
+        """Prompts [(slot, token ids)] of a layer-stack model, from position 0, in steps of at most `step_tokens` tokens
+        (portions of at most `prefill_chunk`). Returns the hidden state of every prompt's last token [len(work), D]."""
+        from ..ops.ragged import RaggedBatch
+        chunk = self.prefill_chunk if self.prefill_chunk and self.prefill_chunk > 0 else self.step_tokens
+        chunk = min(chunk, self.step_tokens)
+        done, out = [0] * len(work), None
+        while any(d < len(t) for d, (_, t) in zip(done, work)):
+            room, step, ends, at = self.step_tokens, [], [], 0
+            for i, (slot, toks) in enumerate(work):
+                take = min(chunk, room, len(toks) - done[i])
+                if take <= 0:
+                    continue
+                step.append((slot, done[i], toks[done[i]:done[i] + take]))
+                done[i] += take
+                room -= take
+                at += take
+                if done[i] == len(toks):
+                    ends.append((i, at - 1))
+            h = self.exec.forward(RaggedBatch.build(step, self.device), self.pool)
+            if out is None:
+                out = torch.empty((len(work), h.shape[1]), dtype=h.dtype, device=h.device)
+            if ends:
+                ix = torch.tensor(ends, dtype=torch.int64).to(self.device)
+                out[ix[:, 0]] = h[ix[:, 1]]
+        return out
+
     def _decode_step(self, st) -> None:
         """One token for every sequence of the wave. `st` holds the static device buffers."""
+        if self.exec is not None:
+            self._sample_into(self.exec.forward(st["batch"], self.pool), st)
+            return
         cfg, pool = self.cfg, self.pool
         B = st["tokens"].shape[0]
         N, KH, H = self.n_heads, self.n_kv, cfg.head_dim
@@ -432,6 +493,8 @@ class PagedEngine(BaseSampler):
         self._sample_into(hlast, st)
 
     def _logits(self, hlast, out=None):
+        if self.exec is not None:
+            return self.exec.logits(hlast, out)
         ph = self._pk(len(self._model.layers), "head")
         if ph is not None:
             logits = K.gemm_packed(hlast, ph, out=out, out_dtype=torch.float32)
@@ -517,7 +580,7 @@ class PagedEngine(BaseSampler):
         N, H, V = self.n_heads, self.cfg.head_dim, self.cfg.vocab_size
         i64 = dict(dtype=torch.int64, device=dev)
         i32 = dict(dtype=torch.int32, device=dev)
-        return {
+        st = {
             "tokens": torch.zeros(B, **i64),
             "positions": torch.full((B,), -1, **i32),             # -1 / 0: an empty slot
             "seq_lens": torch.zeros(B, **i32),
@@ -538,6 +601,10 @@ class PagedEngine(BaseSampler):
             "params": {"temperature": temperature, "top_p": top_p, "top_k": top_k, "seed": seed},
             "split": split,
         }
+        if self.exec is not None:
+            from ..ops.ragged import RaggedBatch
+            st["batch"] = RaggedBatch.decode_slots(st["tokens"], st["slots"], st["positions"])
+        return st
 
     def _run(self, toks_np, lens_np, max_steps, eos_ids, pad_id, temperature, top_p, top_k, seed):
         """All requests of one call through the continuous-batching loop. toks_np [n, P] left-padded prompts,
@@ -729,6 +796,11 @@ class PagedEngine(BaseSampler):
         ps = self.pool.page_size
         cached = [0] * g if cached is None else list(cached)
         lens_l = [int(x) for x in lens_np]
+        if self.exec is not None:
+            P = toks_np.shape[1]
+            hlast = self._prefill_ragged([(s, toks_np[i, P - lens_l[i]:].tolist()) for i, s in enumerate(slots_list)])
+            self._first_tokens(st, hlast, slots_list, lens_l, pad_id, limits)
+            return
         use = [min(c, (ln - 1) // ps * ps) for c, ln in zip(cached, lens_l)]       # tokens taken from the pages
         newlen = [ln - u for ln, u in zip(lens_l, use)]
         Pn = max(newlen)
@@ -740,7 +812,6 @@ class PagedEngine(BaseSampler):
         nl = torch.as_tensor(newlen, device=dev)
         prev = torch.as_tensor(use, dtype=torch.int32, device=dev)
         wfrom = torch.as_tensor(cached, dtype=torch.int32, device=dev)
-        lens = torch.as_tensor(lens_l, device=dev)
         seg = (torch.arange(Pn, device=dev)[None] >= (Pn - nl)[:, None]).to(torch.int32)
         positions = (torch.clamp(torch.cumsum(seg, -1) - 1, min=0) + prev[:, None]).to(torch.int32)
         slots = torch.as_tensor(slots_list, dtype=torch.int32, device=dev)
@@ -752,11 +823,17 @@ class PagedEngine(BaseSampler):
             use_prev = before if (c0 > 0 or any(use)) else None
             hlast = self._prefill(toks[:, c0:c1].contiguous(), positions[:, c0:c1].contiguous(),
                                   seg[:, c0:c1].contiguous(), slots, use_prev, wfrom)
+        self._first_tokens(st, hlast, slots_list, lens_l, pad_id, limits)
+
+    def _first_tokens(self, st, hlast, slots_list, lens_l, pad_id, limits) -> None:
+        """Sample every admitted prompt's first token from its last hidden state and set the slot state."""
+        dev, g = self.device, len(slots_list)
         logits = self._logits(hlast)
         nxt = torch.zeros(g, dtype=torch.int64, device=dev)
         nlp = torch.zeros(g, device=dev)
         self._sample(logits, st, nxt, nlp)
-        ix = slots.to(torch.int64)
+        lens = torch.as_tensor(lens_l, device=dev)
+        ix = torch.as_tensor(slots_list, dtype=torch.int64, device=dev)
         lim = torch.as_tensor(limits, dtype=torch.int64, device=dev)
         st["out_tokens"][ix] = pad_id
         st["out_tokens"][ix, 0] = nxt
@@ -775,6 +852,9 @@ class PagedEngine(BaseSampler):
         one step; the state the warm-up and the capture touched is put back."""
         keys = ("tokens", "positions", "seq_lens", "done", "out_tokens", "out_lp", "out_pos", "step")
         snap = {k: st[k].clone() for k in keys}
+        if self.exec is not None:          # a recurrent state must not advance twice: warm up with every slot idle
+            st["positions"].fill_(-1)
+            st["seq_lens"].zero_()
         self._decode_step(st)
         for k, v in snap.items():
             st[k].copy_(v)
@@ -786,6 +866,61 @@ class PagedEngine(BaseSampler):
         for k, v in snap.items():
             st[k].copy_(v)
         return graph
+
+
+class StepSession:
+    """Drives a layer-stack model's step function by hand over an engine's page pool and slot states: the caller says
+    which tokens of which requests run together and which logits it wants; nothing is sampled. A request is admitted at
+    its first step, keeps its slot and pages until it is ended, and may sit out any number of steps in between."""
+
+    def __init__(self, engine: PagedEngine):
+        if engine.exec is None:
+            raise NotImplementedError("steps are driven by hand for layer-stack models only")
+        self.engine = engine
+        engine._fuse_all()
+        engine._packed_on = False
+        engine.pool = None
+        engine.reinitialize_cache()
+        self._free = list(range(engine.max_running))[::-1]
+        self._live: dict = {}               # request id -> [slot, tokens so far]
+
+    @torch.no_grad()
+    def step(self, entries, end=()):
+        """entries: [(request id, token ids, wanted places among them)]. Returns fp32 logits [wanted, vocab] in order."""
+        from ..ops.ragged import RaggedBatch
+        eng, work, rows, at = self.engine, [], [], 0
+        pool = eng.pool
+        for rid, tokens, want in entries:
+            if not tokens:
+                continue
+            req = self._live.get(rid)
+            if req is None:
+                if not self._free:
+                    raise RuntimeError(f"request {rid!r}: all {eng.max_running} slots are in use")
+                req = self._live[rid] = [self._free.pop(), 0]
+                pool.open(req[0], list(tokens), 0)
+            else:
+                pool.grow(req[0], req[1] + len(tokens))
+            if req[1] + len(tokens) > pool.max_pages * pool.page_size:
+                raise ValueError(f"request {rid!r} does not fit the page table ({pool.max_pages} pages)")
+            work.append((req[0], req[1], tokens))
+            rows += [at + int(w) for w in want]
+            req[1] += len(tokens)
+            at += len(tokens)
+        logits = torch.empty((0, eng.cfg.vocab_size), dtype=torch.float32, device=eng.device)
+        if work:
+            pool.sync_table()
+            h = eng.exec.forward(RaggedBatch.build(work, eng.device), pool)
+            if rows:
+                logits = eng._logits(h[torch.tensor(rows, dtype=torch.int64, device=eng.device)])
+        for rid in end:
+            self.end(rid)
+        return logits
+
+    def end(self, rid) -> None:
+        slot, _ = self._live.pop(rid)
+        self.engine.pool.release(slot)
+        self._free.append(slot)
 
 
 class EngineServer:

@@ -14,7 +14,8 @@ import torch
 from . import naming
 from .config import ModelConfig, get_config
 from .safetensors_loader import load_safetensors_into
-from .transformer import Transformer, create_model
+from .stack import describes_layer_stack
+from .transformer import create_model
 
 
 class ModelSource(enum.Enum):
@@ -42,13 +43,16 @@ class AutoModel:
                         model_path: Optional[str] = None, model_download_path: Optional[str] = None,
                         device=None, dtype: Optional[torch.dtype] = None, load_dtype: Optional[torch.dtype] = None,
                         remat_config: Optional[str] = None, use_flash_attention: Optional[bool] = None,
-                        seed: int = 0, **config_overrides):
-        """Returns (model, model_path)."""
+                        seed: int = 0, config: Optional[ModelConfig] = None, **config_overrides):
+        """Returns (model, model_path). `config`: use this configuration instead of resolving `model_id`."""
+        path = model_path or (model_id if os.path.isdir(model_id) else None)
         try:
-            cfg: ModelConfig = naming.config_for(model_id)
+            if config is None and path is not None and describes_layer_stack(path):
+                from .hf_config import config_from_hf
+                config, model_path = config_from_hf(path), path     # such a directory never means a preset
+            cfg: ModelConfig = config if config is not None else naming.config_for(model_id)
         except (KeyError, ValueError):
             # no preset of that name: a checkpoint directory describes itself through its config.json
-            path = model_path or (model_id if os.path.isdir(model_id) else None)
             if path is None or not os.path.exists(os.path.join(path, "config.json")):
                 raise
             from .hf_config import config_from_hf
@@ -71,6 +75,6 @@ class AutoModel:
             model_path = download_model(model_id, model_source, model_download_path)
         if not os.path.exists(model_path):
             raise FileNotFoundError(model_path)
-        model = Transformer(cfg, device=device)
+        model = create_model(cfg, device=device, init=False)
         load_safetensors_into(model, model_path, dtype=load_dtype)
         return model, model_path

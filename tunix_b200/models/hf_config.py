@@ -46,6 +46,9 @@ def config_from_hf(src: Union[str, dict], dtype: Optional[torch.dtype] = None, *
             c = json.load(f)
     else:
         c = dict(src)
+    from .stack import config_from_stack_json, is_stack_json
+    if is_stack_json(c):                                    # layer-stack designs describe themselves layer by layer
+        return config_from_stack_json(src, dtype, **overrides)
     outer = c
     if isinstance(c.get("text_config"), dict):
         c = dict(c["text_config"])

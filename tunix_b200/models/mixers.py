@@ -1,0 +1,203 @@
+"""Sequence mixers of layer-stack models (`models/stack.py`): what a layer does along the sequence axis, each with its
+sizes and constants in a spec, its parameters in a module and its per-sequence cache or state in a layout.
+
+  RGLRUMixer              Griffin's recurrent block: short causal convolution, block-diagonal gates, real-gated linear
+                          recurrent unit, gelu-gated output
+  BiasedWindowAttention   grouped-query attention without rotation: RMS norm over the whole query / key projection,
+                          learned bias per (distance bucket, head), sliding window with kept first tokens, sigmoid
+                          output gate
+  MatrixMemory            mLSTM: matrix memory with exponential input gate, capped gate pre-activations, per-head norm
+                          and sigmoid output gate
+  ParallelMixer           two mixers on the same input, half the sum of their normed outputs
+
+A spec's `kv_rows()` names the paged cache rows a pass through the layer needs (key columns, value columns), or None;
+`state_shapes()` the fp32 state it keeps per sequence slot. The kernels are launched by `models/stack_exec.py`.
+"""
+from __future__ import annotations
+
+import math
+from dataclasses import dataclass
+from typing import Optional
+
+import torch
+import torch.nn as nn
+
+from .transformer import Linear, RMSNorm
+
+MEMORY_SLICE = 32       # value columns a CTA of the matrix-memory kernels owns (csrc/recurrent.cu: MV)
+
+
+# ---------------------------------------------------------------------------------------------------- specs
+@dataclass(frozen=True)
+class RGLRUSpec:
+    width: int
+    blocks: int
+    conv: int                    # taps of the causal convolution
+
+    def kv_rows(self):
+        return None
+
+    def state_shapes(self) -> dict:
+        return {"s": (self.width,), "ring": (self.conv, self.width)}
+
+
+@dataclass(frozen=True)
+class WindowAttentionSpec:
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    bias_max: int                # distance from which on every key falls into the last bucket
+    window: int                  # 0 = unlimited
+    keep_first: int = 0          # leading tokens of the sequence that stay visible
+    buckets: int = 32            # rows of the bias table
+
+    def kv_rows(self):
+        return (self.kv_heads * self.dim, self.kv_heads * self.vdim)
+
+    def state_shapes(self) -> dict:
+        return {}
+
+
+@dataclass(frozen=True)
+class MatrixMemorySpec:
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+
+    def kv_rows(self):
+        return None
+
+    def state_shapes(self) -> dict:
+        slices = -(-self.vdim // MEMORY_SLICE)
+        return {"S": (self.heads, self.dim, self.vdim), "n": (self.heads, slices, self.dim), "m": (self.heads, slices)}
+
+
+@dataclass(frozen=True)
+class ParallelSpec:
+    left: WindowAttentionSpec
+    right: MatrixMemorySpec
+
+    def kv_rows(self):
+        return self.left.kv_rows()
+
+    def state_shapes(self) -> dict:
+        return self.right.state_shapes()
+
+
+# ------------------------------------------------------------------------------------------------- bias table
+def distance_buckets(rows: int, bias_max: int, device=None) -> torch.Tensor:
+    """Bucket of every distance 0 .. bias_max: the lower half of the rows holds one distance each, the upper half
+    grows logarithmically and ends at `bias_max`; larger distances share the last row with it."""
+    half = rows // 2
+    n = torch.arange(bias_max + 1, dtype=torch.float64, device=device)
+    if half < 1 or bias_max <= half:
+        return torch.clamp(n, max=rows - 1).long()
+    log_pos = torch.log(torch.clamp(n, min=1) / half) / math.log(bias_max / half) * (rows - half)
+    # a ratio that is an integer in exact arithmetic must not fall below it by rounding
+    upper = torch.clamp(half + torch.floor(log_pos + 1e-12), max=rows - 1)
+    return torch.where(n < half, n, upper).long()
+
+
+# --------------------------------------------------------------------------------------------------- modules
+def _param(*shape, dtype, device, fill: float = 0.0):
+    return nn.Parameter(torch.full(shape, fill, dtype=dtype, device=device))
+
+
+class RGLRUMixer(nn.Module):
+    def __init__(self, spec: RGLRUSpec, width: int, eps: float, dtype, device=None):
+        super().__init__()
+        if spec.width % spec.blocks:
+            raise ValueError(f"{spec.width} channels do not split into {spec.blocks} blocks")
+        self.spec = spec
+        W, bs = spec.width, spec.width // spec.blocks
+        self.y_proj = Linear(width, W, True, dtype, device)
+        self.x_proj = Linear(width, W, True, dtype, device)
+        self.conv_weight = _param(W, spec.conv, dtype=dtype, device=device)
+        self.conv_bias = _param(W, dtype=dtype, device=device)
+        self.ra_weight = _param(spec.blocks, bs, bs, dtype=dtype, device=device)
+        self.ra_bias = _param(spec.blocks, bs, dtype=dtype, device=device)
+        self.ri_weight = _param(spec.blocks, bs, bs, dtype=dtype, device=device)
+        self.ri_bias = _param(spec.blocks, bs, dtype=dtype, device=device)
+        self.lam = _param(W, dtype=dtype, device=device, fill=-4.0)
+        self.o_proj = Linear(W, width, False, dtype, device)
+
+    def init_special(self) -> None:
+        self.conv_weight.zero_()
+        self.conv_weight[:, -1] = 1.0
+        self.ra_bias.zero_()
+        self.ri_bias.zero_()
+
+    def fused_groups(self) -> list:
+        return [[self.y_proj, self.x_proj]]
+
+
+class BiasedWindowAttention(nn.Module):
+    def __init__(self, spec: WindowAttentionSpec, width: int, eps: float, dtype, device=None):
+        super().__init__()
+        if spec.heads % spec.kv_heads:
+            raise ValueError(f"{spec.heads} query heads over {spec.kv_heads} key / value heads")
+        self.spec, self.eps = spec, eps
+        H, G = spec.heads, spec.kv_heads
+        self.q_proj = Linear(width, H * spec.dim, False, dtype, device)
+        self.k_proj = Linear(width, G * spec.dim, False, dtype, device)
+        self.v_proj = Linear(width, G * spec.vdim, False, dtype, device)
+        self.g_proj = Linear(width, H * spec.vdim, False, dtype, device)
+        self.o_proj = Linear(H * spec.vdim, width, False, dtype, device)
+        self.q_norm = RMSNorm(H * spec.dim, eps, False, dtype, device)
+        self.k_norm = RMSNorm(G * spec.dim, eps, False, dtype, device)
+        self.rel = _param(spec.buckets, H, dtype=dtype, device=device)
+
+    def bias_table(self) -> torch.Tensor:
+        """fp32 [far + 1, heads]: what is added to the score of a key at distance min(i - j, far)."""
+        idx = distance_buckets(self.rel.shape[0], self.spec.bias_max, self.rel.device)
+        return self.rel.detach().float()[idx].contiguous()
+
+    def init_special(self) -> None:
+        pass
+
+
+class MatrixMemory(nn.Module):
+    def __init__(self, spec: MatrixMemorySpec, width: int, eps: float, dtype, device=None):
+        super().__init__()
+        self.spec, self.eps = spec, eps
+        H = spec.heads
+        self.q_proj = Linear(width, H * spec.dim, False, dtype, device)
+        self.k_proj = Linear(width, H * spec.dim, False, dtype, device)
+        self.v_proj = Linear(width, H * spec.vdim, False, dtype, device)
+        self.g_proj = Linear(width, H * spec.vdim, False, dtype, device)
+        self.i_proj = Linear(width, H, True, dtype, device)
+        self.f_proj = Linear(width, H, True, dtype, device)
+        self.o_proj = Linear(H * spec.vdim, width, False, dtype, device)
+        self.norm = RMSNorm(H * spec.vdim, eps, False, dtype, device)
+
+    def init_special(self) -> None:
+        self.f_proj.bias.fill_(3.0)
+
+
+class ParallelMixer(nn.Module):
+    def __init__(self, spec: ParallelSpec, width: int, eps: float, dtype, device=None):
+        super().__init__()
+        self.spec = spec
+        self.left = BiasedWindowAttention(spec.left, width, eps, dtype, device)
+        self.right = MatrixMemory(spec.right, width, eps, dtype, device)
+        self.left_norm = RMSNorm(width, eps, False, dtype, device)
+        self.right_norm = RMSNorm(width, eps, False, dtype, device)
+
+    def init_special(self) -> None:
+        self.left.init_special()
+        self.right.init_special()
+
+    def fused_groups(self) -> list:
+        lf, rt = self.left, self.right
+        return [[lf.q_proj, lf.k_proj, lf.v_proj, lf.g_proj, rt.q_proj, rt.k_proj, rt.v_proj, rt.g_proj],
+                [rt.i_proj, rt.f_proj]]
+
+
+MIXERS = {RGLRUSpec: RGLRUMixer, ParallelSpec: ParallelMixer}
+
+
+def create_mixer(spec, width: int, eps: float, dtype, device: Optional[torch.device] = None) -> nn.Module:
+    return MIXERS[type(spec)](spec, width, eps, dtype, device)

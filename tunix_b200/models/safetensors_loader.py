@@ -52,12 +52,34 @@ _KEY_MAPS = {
         (r"model\.layers\.(\d+)\.experts\.gate_up_proj", r"layers.\1.moe.gate_proj|layers.\1.moe.up_proj"),
         (r"model\.layers\.(\d+)\.experts\.down_proj", r"layers.\1.moe.down_proj"),
     ],
+    # Layer-stack checkpoints (models/stack.py) number their layers l0, l1, ...
+    "roluzen": [
+        (r"embed", "embed_tokens"),
+        (r"head", "lm_head"),
+        (r"final\.norm", "norm.weight"),
+        (r"l(\d+)\.norm1", r"layers.\1.input_layernorm.weight"),
+        (r"l(\d+)\.norm2", r"layers.\1.post_attention_layernorm.weight"),
+        (r"l(\d+)\.hc(1|2)\.(in|out)", r"layers.\1.hc\2.weight_\3"),
+        (r"l(\d+)\.hc(1|2)\.mix", r"layers.\1.hc\2.mix"),
+        (r"l(\d+)\.mlp\.(gate|up|down)", r"layers.\1.mlp.\2_proj.weight"),
+        (r"l(\d+)\.mix\.(left|right)\.out", r"layers.\1.mixer.\2_norm.weight"),
+        (r"l(\d+)\.mix\.left\.(q|k)\.norm", r"layers.\1.mixer.left.\2_norm.weight"),
+        (r"l(\d+)\.mix\.left\.rel", r"layers.\1.mixer.left.rel"),
+        (r"l(\d+)\.mix\.right\.norm", r"layers.\1.mixer.right.norm.weight"),
+        (r"l(\d+)\.mix\.right\.(i|f)\.b", r"layers.\1.mixer.right.\2_proj.bias"),
+        (r"l(\d+)\.mix\.(left|right)\.(q|k|v|g|o|i|f)", r"layers.\1.mixer.\2.\3_proj.weight"),
+        (r"l(\d+)\.mix\.(y|x)\.b", r"layers.\1.mixer.\2_proj.bias"),
+        (r"l(\d+)\.mix\.(y|x|o)", r"layers.\1.mixer.\2_proj.weight"),
+        (r"l(\d+)\.mix\.(conv|ra|ri)\.b", r"layers.\1.mixer.\2_bias"),
+        (r"l(\d+)\.mix\.(conv|ra|ri)", r"layers.\1.mixer.\2_weight"),
+        (r"l(\d+)\.mix\.lam", r"layers.\1.mixer.lam"),
+    ],
 }
 
 
 def key_map_for(cfg) -> list:
-    if cfg.family == "gemma4":
-        return _KEY_MAPS["gemma4"]
+    if cfg.family in ("gemma4", "roluzen"):
+        return _KEY_MAPS[cfg.family]
     return _KEY_MAPS["gemma_post_norms" if cfg.post_norms else "default"]
 
 
@@ -73,6 +95,8 @@ def map_key(hf_key: str, table: list) -> Optional[str]:
 
 def inverse_map_key(our_key: str, cfg) -> str:
     """Our parameter name -> HF key (used by the saver)."""
+    if cfg.family == "roluzen":
+        return _inverse_stack_key(our_key)
     if our_key == "embed_tokens":
         return "model.embed_tokens.weight"
     if our_key == "lm_head":
@@ -86,6 +110,46 @@ def inverse_map_key(our_key: str, cfg) -> str:
         k = k.replace(".post_ffw_norm.", ".post_feedforward_layernorm.")
     k = k.replace(".mlp.router.weight", ".mlp.gate.weight")
     return k
+
+
+# parameter name -> checkpoint name of layer-stack models, the inverse of _KEY_MAPS["roluzen"]
+_STACK_INVERSE = [
+    (r"embed_tokens", "embed"), (r"lm_head", "head"), (r"norm\.weight", "final.norm"),
+    (r"layers\.(\d+)\.input_layernorm\.weight", r"l\1.norm1"),
+    (r"layers\.(\d+)\.post_attention_layernorm\.weight", r"l\1.norm2"),
+    (r"layers\.(\d+)\.(hc\d)\.weight_(in|out)", r"l\1.\2.\3"),
+    (r"layers\.(\d+)\.(hc\d)\.mix", r"l\1.\2.mix"),
+    (r"layers\.(\d+)\.mlp\.(gate|up|down)_proj\.weight", r"l\1.mlp.\2"),
+    (r"layers\.(\d+)\.mixer\.(left|right)_norm\.weight", r"l\1.mix.\2.out"),
+    (r"layers\.(\d+)\.mixer\.left\.(q|k)_norm\.weight", r"l\1.mix.left.\2.norm"),
+    (r"layers\.(\d+)\.mixer\.left\.rel", r"l\1.mix.left.rel"),
+    (r"layers\.(\d+)\.mixer\.right\.norm\.weight", r"l\1.mix.right.norm"),
+    (r"layers\.(\d+)\.mixer\.right\.(i|f)_proj\.bias", r"l\1.mix.right.\2.b"),
+    (r"layers\.(\d+)\.mixer\.(left|right)\.(\w)_proj\.weight", r"l\1.mix.\2.\3"),
+    (r"layers\.(\d+)\.mixer\.(y|x)_proj\.bias", r"l\1.mix.\2.b"),
+    (r"layers\.(\d+)\.mixer\.(y|x|o)_proj\.weight", r"l\1.mix.\2"),
+    (r"layers\.(\d+)\.mixer\.(conv|ra|ri)_bias", r"l\1.mix.\2.b"),
+    (r"layers\.(\d+)\.mixer\.(conv|ra|ri)_weight", r"l\1.mix.\2"),
+    (r"layers\.(\d+)\.mixer\.lam", r"l\1.mix.lam"),
+]
+
+
+def _inverse_stack_key(our_key: str) -> str:
+    for pat, repl in _STACK_INVERSE:
+        m = re.fullmatch(pat, our_key)
+        if m:
+            return m.expand(repl)
+    raise KeyError(f"no checkpoint name for parameter {our_key!r}")
+
+
+def tensor_shapes(path: str) -> dict:
+    """name -> shape of every tensor in the safetensors files under `path` (headers only, no data is read)."""
+    out = {}
+    for f in ([path] if os.path.isfile(path) else sorted(glob.glob(os.path.join(path, "*.safetensors")))):
+        with open(f, "rb") as fh:
+            header = json.loads(fh.read(int.from_bytes(fh.read(8), "little")))
+        out.update({k: tuple(v["shape"]) for k, v in header.items() if k != "__metadata__"})
+    return out
 
 
 def load_safetensors_into(model, path: str, dtype: Optional[torch.dtype] = None, strict: bool = True,

@@ -1,0 +1,266 @@
+"""Layer-stack models: decoders whose layers are listed one by one, each with its own mixer (`models/mixers.py`) and
+feed-forward, a range of layers that may run several times with the same weights, and parallel residual streams joined by
+hyper-connections. Roluzen is the first design of this kind.
+
+The residual streams are fp32. A sublayer q of a layer reads u = sum_s in[s] x_s, computes y = f(norm(u)) and leaves
+x_t = sum_s mix[s, t] x_s + out[t] y on every stream; the model's output is the norm of the streams' sum.
+
+The model holds parameters; `models/stack_exec.py` runs it on ragged batches over the paged cache and the slot states of
+`generate/engine.py`. `forward` scores whole sequences through that same path on a temporary cache (no gradients).
+"""
+from __future__ import annotations
+
+import json
+import os
+from dataclasses import dataclass, field
+from typing import Optional, Union
+
+import torch
+import torch.nn as nn
+
+from ..ops import functional as F
+from .config import ModelConfig
+from .mixers import MatrixMemorySpec, ParallelSpec, RGLRUSpec, WindowAttentionSpec, create_mixer
+from .transformer import MLP, RMSNorm
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    mixer: object                       # one of the specs of models/mixers.py
+    ff: Optional[int]                   # width of the gated feed-forward; None = the layer has none
+
+
+@dataclass
+class StackConfig(ModelConfig):
+    layer_specs: tuple = field(default_factory=tuple)
+    loop: Optional[tuple] = None        # (start, stop, times): these layers run `times` times in a row
+    streams: int = 0                    # residual streams with hyper-connections; 0 = one plain residual
+
+    def __post_init__(self):
+        if not self.layer_specs:
+            raise ValueError("a layer-stack model needs its layers")
+        self.num_layers = len(self.layer_specs)
+        ffs = [s.ff for s in self.layer_specs if s.ff is not None]
+        self.hidden_dim = max(ffs) if ffs else 0
+        att = [s.mixer.left for s in self.layer_specs if isinstance(s.mixer, ParallelSpec)]
+        if att:                         # what generic callers size caches and reports by: the first attention layer
+            self.num_heads, self.num_kv_heads, self.head_dim = att[0].heads, att[0].kv_heads, att[0].dim
+        if self.loop is not None:
+            a, b, times = self.loop
+            if not (0 <= a <= b <= self.num_layers and times >= 0):
+                raise ValueError(f"loop {self.loop} does not fit {self.num_layers} layers")
+
+    def runs(self) -> list:
+        """Layer index of every pass, in order. Each pass has its own cache and state."""
+        n = self.num_layers
+        if self.loop is None:
+            return list(range(n))
+        a, b, times = self.loop
+        return list(range(a)) + list(range(a, b)) * times + list(range(b, n))
+
+    # ---- what the engine's cache manager allocates, per pass
+    def kv_rows(self) -> list:
+        return [self.layer_specs[i].mixer.kv_rows() for i in self.runs()]
+
+    def state_shapes(self) -> list:
+        return [self.layer_specs[i].mixer.state_shapes() for i in self.runs()]
+
+    def num_params(self) -> int:
+        return sum(p.numel() for p in StackModel(self, device=torch.device("meta")).parameters())
+
+    # ---- presets (random weights: no checkpoint of this design is published)
+    @classmethod
+    def roluzen_tiny(cls) -> "StackConfig":
+        att = WindowAttentionSpec(heads=4, kv_heads=2, dim=32, vdim=32, scale=32 ** -0.5, bias_max=64, window=24, keep_first=2,
+                                  buckets=12)
+        par = LayerSpec(ParallelSpec(att, MatrixMemorySpec(heads=2, dim=24, vdim=40, gate_cap=12.0)), 192)
+        rec = LayerSpec(RGLRUSpec(width=160, blocks=5, conv=4), 192)
+        return cls(family="roluzen", vocab_size=384, embed_dim=128, layer_specs=(rec, par, rec), loop=(1, 3, 2), streams=3)
+
+    @classmethod
+    def _roluzen(cls, D, ff, heads, kv, dim, mh, mdk, mdv, W, blocks, n, loop, window=1024, vocab=151936):
+        att = WindowAttentionSpec(heads=heads, kv_heads=kv, dim=dim, vdim=dim, scale=dim ** -0.5, bias_max=4 * window,
+                                  window=window, keep_first=4, buckets=32)
+        par = LayerSpec(ParallelSpec(att, MatrixMemorySpec(heads=mh, dim=mdk, vdim=mdv, gate_cap=15.0)), ff)
+        rec = LayerSpec(RGLRUSpec(width=W, blocks=blocks, conv=4), ff)
+        specs = tuple(par if i % 3 == 0 else rec for i in range(n))
+        return cls(family="roluzen", vocab_size=vocab, embed_dim=D, layer_specs=specs, loop=loop, streams=2)
+
+    @classmethod
+    def roluzen_2b(cls) -> "StackConfig":
+        return cls._roluzen(2048, 6144, 16, 8, 128, 8, 128, 256, 2048, 16, 18, (0, 3, 2))
+
+    @classmethod
+    def roluzen_8b(cls) -> "StackConfig":
+        return cls._roluzen(4096, 12288, 32, 8, 128, 8, 256, 512, 4096, 16, 24, (0, 3, 2))
+
+
+# ------------------------------------------------------------------------------------------ config.json reader
+def _parallel_spec(m: dict, shapes, prefix: str) -> ParallelSpec:
+    lf, rt = m["left"], m["right"]
+    mask = lf.get("mask") or {}
+    rel = (shapes or {}).get(prefix + "left.rel")
+    left = WindowAttentionSpec(heads=int(lf["heads"]), kv_heads=int(lf["kv_heads"]), dim=int(lf["dim"]), vdim=int(lf["vdim"]),
+                               scale=float(lf["scale"]), bias_max=int(lf["bias_max"]), window=int(mask.get("size") or 0),
+                               keep_first=int(mask.get("keep_first") or 0), buckets=int(rel[0]) if rel else 32)
+    return ParallelSpec(left, MatrixMemorySpec(heads=int(rt["heads"]), dim=int(rt["dim"]), vdim=int(rt["vdim"]),
+                                               gate_cap=float(rt["gate_cap"])))
+
+
+def _rglru_spec(m: dict, shapes, prefix: str) -> RGLRUSpec:
+    return RGLRUSpec(width=int(m["width"]), blocks=int(m["blocks"]), conv=int(m["conv"]))
+
+
+MIXER_READERS = {"rglru": _rglru_spec, "parallel": _parallel_spec}
+ARCHITECTURES = {"Roluzen": "roluzen"}
+
+
+def is_stack_json(c: dict) -> bool:
+    return c.get("architecture") in ARCHITECTURES
+
+
+def describes_layer_stack(path: str) -> bool:
+    """Whether the checkpoint directory `path` holds a layer-stack model's config.json."""
+    try:
+        with open(os.path.join(path, "config.json"), encoding="utf-8") as f:
+            return is_stack_json(json.load(f))
+    except (OSError, ValueError):
+        return False
+
+
+def config_from_stack_json(src: Union[str, dict], dtype: Optional[torch.dtype] = None, shapes: Optional[dict] = None,
+                           **overrides) -> StackConfig:
+    """`src`: a checkpoint directory, a config.json path or the parsed dict. Sizes that only a tensor's shape tells (rows
+    of the bias tables) come from the safetensors headers of the directory, or from `shapes` (name -> shape)."""
+    c = src
+    if isinstance(src, str):
+        path = os.path.join(src, "config.json") if os.path.isdir(src) else src
+        with open(path, encoding="utf-8") as f:
+            c = json.load(f)
+        if shapes is None:
+            from .safetensors_loader import tensor_shapes
+            shapes = tensor_shapes(os.path.dirname(path))
+    specs = []
+    for i, layer in enumerate(c["layers"]):
+        if layer["type"] not in MIXER_READERS:
+            raise ValueError(f"layer {i}: no mixer {layer['type']!r} in this framework")
+        mlp = layer.get("mlp")
+        if mlp is not None and mlp.get("kind") != "dense":
+            raise ValueError(f"layer {i}: no feed-forward {mlp.get('kind')!r} in this framework")
+        specs.append(LayerSpec(MIXER_READERS[layer["type"]](layer["mixer"], shapes, f"l{i}.mix."),
+                               None if mlp is None else int(mlp["ff"])))
+    lp = c.get("loop")
+    kw = dict(family=ARCHITECTURES[c["architecture"]], vocab_size=int(c["vocab"]), embed_dim=int(c["width"]),
+              norm_eps=float(c["norm"]["eps"]), layer_specs=tuple(specs),
+              loop=None if not lp else (int(lp["start"]), int(lp["stop"]), int(lp["times"])),
+              streams=int(c.get("streams") or 0), dtype=dtype or torch.bfloat16)
+    kw.update(overrides)
+    return StackConfig(**kw)
+
+
+# --------------------------------------------------------------------------------------------------- the model
+class HyperConnection(nn.Module):
+    """How a sublayer reads and writes the residual streams: `weight_in` [S], `weight_out` [S], `mix` [S from, S to]."""
+
+    def __init__(self, streams: int, dtype, device=None):
+        super().__init__()
+        S = streams
+        self.weight_in = nn.Parameter(torch.full((S,), 1.0 / S, dtype=dtype, device=device))
+        self.weight_out = nn.Parameter(torch.ones(S, dtype=dtype, device=device))
+        self.mix = nn.Parameter(torch.eye(S, dtype=dtype, device=device))
+
+
+class StackLayer(nn.Module):
+    def __init__(self, cfg: StackConfig, spec: LayerSpec, device=None):
+        super().__init__()
+        D, dt, eps = cfg.embed_dim, cfg.dtype, cfg.norm_eps
+        self.spec = spec
+        self.input_layernorm = RMSNorm(D, eps, False, dt, device)
+        self.mixer = create_mixer(spec.mixer, D, eps, dt, device)
+        self.hc1 = HyperConnection(cfg.streams, dt, device) if cfg.streams else None
+        self.post_attention_layernorm = self.mlp = self.hc2 = None
+        if spec.ff is not None:
+            self.post_attention_layernorm = RMSNorm(D, eps, False, dt, device)
+            # the generic gated MLP reads only these sizes
+            self.mlp = MLP(ModelConfig(embed_dim=D, hidden_dim=spec.ff, activation=cfg.activation, dtype=dt), device)
+            self.hc2 = HyperConnection(cfg.streams, dt, device) if cfg.streams else None
+
+
+class StackModel(nn.Module):
+    def __init__(self, cfg: StackConfig, device=None):
+        super().__init__()
+        self.config = cfg
+        dt = cfg.dtype
+        self.embed_tokens = nn.Parameter(torch.empty(cfg.vocab_size, cfg.embed_dim, dtype=dt, device=device))
+        self.layers = nn.ModuleList([StackLayer(cfg, s, device) for s in cfg.layer_specs])
+        self.norm = RMSNorm(cfg.embed_dim, cfg.norm_eps, False, dt, device)
+        self.lm_head = nn.Parameter(torch.empty(cfg.vocab_size, cfg.embed_dim, dtype=dt, device=device))
+        self.tp = None
+        self._exec = None
+
+    @torch.no_grad()
+    def init_weights(self, seed: int = 0, std: float = 0.02) -> "StackModel":
+        gen = torch.Generator(device=self.embed_tokens.device).manual_seed(seed)
+        for name, p in self.named_parameters():
+            if name.endswith((".mix", "_bias")):
+                continue
+            if p.dim() >= 2:
+                p.normal_(0.0, std, generator=gen)
+            elif name.endswith("bias"):
+                p.zero_()
+        for layer in self.layers:
+            layer.mixer.init_special()
+        return self
+
+    def head_weight(self) -> torch.Tensor:
+        return self.lm_head
+
+    def compute_final_logits(self, hidden):
+        return F.lm_head_logits(hidden, self.head_weight(), softcap=self.config.final_logit_softcap)
+
+    def token_logprobs(self, hidden, targets, *, temperature: float = 1.0, want_entropy: bool = False, chunk: Optional[int] = None):
+        return F.lm_head_logprobs(hidden, self.head_weight(), targets, softcap=self.config.final_logit_softcap,
+                                  temperature=temperature, want_entropy=want_entropy, chunk=chunk or self.config.logprob_chunk)
+
+    @property
+    def num_params(self) -> int:
+        return sum(p.numel() for p in self.parameters())
+
+    def executor(self):
+        from .stack_exec import StackExecutor
+        if self._exec is None:
+            self._exec = StackExecutor(self)
+        return self._exec
+
+    @torch.no_grad()
+    def forward(self, input_tokens, positions=None, cache=None, attention_mask=None, segment_ids=None, skip_lm_head: bool = False,
+                output_hidden_states: bool = False, **unused):
+        """Whole sequences [B, T] (rows may be padded: segment id 0; one segment per row) -> (logits or hidden states, None).
+        Forward only; sampling goes through `generate.engine.PagedEngine`, which keeps the cache and the states."""
+        if cache is not None or attention_mask is not None:
+            raise NotImplementedError("layer-stack models keep their cache and state in PagedEngine: sample through it")
+        from ..generate.engine import PagePool
+        from ..ops.ragged import RaggedBatch
+        B, T = input_tokens.shape
+        dev = self.embed_tokens.device
+        keep = torch.ones(B, T, dtype=torch.bool) if segment_ids is None else (segment_ids.cpu() > 0)
+        if segment_ids is not None and int(segment_ids.max()) > 1:
+            raise NotImplementedError("packed rows (several segments) are not scored by layer-stack models")
+        toks = input_tokens.cpu()
+        rows = [toks[b][keep[b]].tolist() for b in range(B)]
+        pages = [-(-max(len(r), 1) // 64) for r in rows]
+        pool = PagePool(self.config, sum(pages), 64, B, max(pages), dev, self.config.dtype, prefix_caching=False)
+        work = []
+        for b, r in enumerate(rows):
+            pool.open(b, r, 0)
+            if r:
+                work.append((b, 0, r))
+        pool.sync_table()
+        ex = self.executor()
+        ex.refresh()
+        h = ex.forward(RaggedBatch.build(work, dev), pool)
+        hidden = torch.zeros(B, T, h.shape[-1], dtype=h.dtype, device=dev)
+        hidden[keep.to(dev)] = h
+        return (hidden if skip_lm_head or output_hidden_states else self.compute_final_logits(hidden)), None
+
+

@@ -1,0 +1,195 @@
+"""Runs a `models.stack.StackModel` on ragged batches: prompts, portions of prompts and decoded tokens of any mix go
+through the same function, reading and writing the engine's paged cache and slot states.
+
+Between two sublayers one kernel closes the one before (hyper-connection write) and opens the one after (hyper-connection
+read and norm). Projections that share an input run as one GEMM over weights joined in memory. bf16 models run on the
+package's tcgen05 GEMMs, with fp32 accumulation; 32-bit models use library GEMMs in full precision (no TF32)."""
+from __future__ import annotations
+
+from typing import Callable, Optional
+
+import torch
+
+from ..ops import kernels as K
+from ..ops import stack_kernels as SK
+from ..ops.ragged import RaggedBatch
+from .mixers import ParallelMixer, RGLRUMixer
+
+
+def joint_weight(mods):
+    """One [sum(out_i), in] tensor over the weights of `mods` (moved there once; the modules keep views), and the joint
+    bias or None. Adapters and quantised bases are not supported on these models."""
+    if any(m.quant is not None or (m.lora_a is not None and m.lora_enabled) for m in mods):
+        raise NotImplementedError("layer-stack models run without adapters or quantised weights")
+    ws = [m.weight for m in mods]
+    rows, base = sum(w.shape[0] for w in ws), ws[0].data
+    off, adjacent = base.storage_offset(), True
+    for w in ws:
+        if w.untyped_storage().data_ptr() != base.untyped_storage().data_ptr() or w.storage_offset() != off or not w.is_contiguous():
+            adjacent = False
+            break
+        off += w.numel()
+    if adjacent:
+        joint = base.as_strided((rows, base.shape[1]), (base.shape[1], 1), base.storage_offset())
+    else:
+        joint = torch.cat([w.data for w in ws], 0)
+        r = 0
+        for w in ws:
+            w.data = joint[r:r + w.shape[0]]
+            r += w.shape[0]
+    bias = torch.cat([m.bias.data for m in mods]) if mods[0].bias is not None else None
+    return joint, bias
+
+
+def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None,
+           packed=None) -> torch.Tensor:
+    """x @ w^T (+ bias), fp32 accumulation, output in `out_dtype` (default: x's)."""
+    out_dtype = out_dtype or x.dtype
+    if x.dtype == torch.bfloat16:
+        if packed is not None:
+            return K.gemm_packed(x, packed, bias=bias, out_dtype=out_dtype)
+        if x.shape[1] % 8 == 0:
+            return K.gemm(x, w, bias=bias, out_dtype=out_dtype)
+    prev = torch.backends.cuda.matmul.allow_tf32
+    torch.backends.cuda.matmul.allow_tf32 = False
+    try:
+        if x.dtype != out_dtype:
+            x, w, bias = x.to(out_dtype), w.to(out_dtype), None if bias is None else bias.to(out_dtype)
+        return torch.nn.functional.linear(x, w, bias)
+    finally:
+        torch.backends.cuda.matmul.allow_tf32 = prev
+
+
+class StackExecutor:
+    def __init__(self, model):
+        self.model = model
+        self.cfg = model.config
+        self.runs = self.cfg.runs()
+        self.dtype = model.embed_tokens.dtype
+        self.pk: Callable = lambda i, name: None        # packed decode weights, set by the engine
+        self._one = None
+        self.w: list = []
+        self.refresh()
+
+    # ------------------------------------------------------------------------------------------------ weights
+    @torch.no_grad()
+    def refresh(self) -> None:
+        """(Re)build everything derived from the parameters. Buffers keep their addresses, so that a captured decode
+        graph stays valid after an in-place weight update."""
+        fresh = []
+        for layer in self.model.layers:
+            d = {}
+            for name, mods in zip(("proj", "gates"), layer.mixer.fused_groups()):
+                d[name], d[name + "_bias"] = joint_weight(mods)
+            if isinstance(layer.mixer, ParallelMixer):
+                d["bias"] = layer.mixer.left.bias_table()
+                d["gates_bias"] = None                   # added by the recurrence in fp32
+            if layer.mlp is not None:
+                d["gu"], _ = joint_weight([layer.mlp.gate_proj, layer.mlp.up_proj])
+            fresh.append(d)
+        for new, old in zip(fresh, self.w):
+            for k, v in old.items():
+                if v is not None and v.shape == new[k].shape:
+                    if v.data_ptr() != new[k].data_ptr():
+                        v.copy_(new[k])
+                    new[k] = v
+        self.w = fresh
+
+    def pack_sources(self) -> list:
+        """Per layer, the weights the engine may keep in packed form for decoding (`PagedEngine._pack_all`)."""
+        out = []
+        for layer, d in zip(self.model.layers, self.w):
+            src = {"proj": d["proj"]}
+            if layer.mlp is not None:
+                src.update(gu=d["gu"], down=layer.mlp.down_proj.weight.data)
+            out.append(src)
+        return out
+
+    def _hc(self, hc):
+        if hc is not None:
+            return hc.weight_in, hc.weight_out, hc.mix
+        if self._one is None:
+            self._one = torch.ones(1, dtype=self.dtype, device=self.model.embed_tokens.device)
+        return self._one, self._one, self._one
+
+    # ------------------------------------------------------------------------------------------------ sublayers
+    def _rglru(self, i, m: RGLRUMixer, h, rb: RaggedBatch, pool, r):
+        d = self.w[i]
+        proj = linear(h, d["proj"], d["proj_bias"], packed=self.pk(i, "proj") if rb.decode else None)
+        o = SK.rglru(proj, m.spec.width, 0, m, rb, pool.state[r])
+        return (linear(o, m.o_proj.weight), None, None, None)
+
+    def _parallel(self, i, m: ParallelMixer, h, rb: RaggedBatch, pool, r):
+        d, lf, rt = self.w[i], m.left, m.right
+        a, s = lf.spec, rt.spec
+        proj = linear(h, d["proj"], packed=self.pk(i, "proj") if rb.decode else None)
+        gates = linear(h, d["gates"], out_dtype=torch.float32)
+        off, cols = [], 0
+        for width in (a.heads * a.dim, a.kv_heads * a.dim, a.kv_heads * a.vdim, a.heads * a.vdim, s.heads * s.dim, s.heads * s.dim,
+                      s.heads * s.vdim, s.heads * s.vdim):
+            off.append(cols)
+            cols += width
+        q = SK.qk_norm_write(proj, off[0], off[1], off[2], lf.q_norm.weight, lf.k_norm.weight, lf.eps, rb, pool.table,
+                             pool.page_size, pool.k[r], pool.v[r], a.heads * a.dim)
+        att = SK.window_attn(q, pool.k[r], pool.v[r], rb, pool.table, pool.page_size, a, d["bias"])
+        o = SK.mlstm(proj, off[4], off[5], off[6], gates, rt.i_proj.bias, rt.f_proj.bias, s.gate_cap, rb, s.heads, s.dim, s.vdim,
+                     pool.state[r])
+        a1, a2 = SK.gate_outputs(att, o, proj, off[3], off[7], rt.norm.weight, rt.eps, s.heads, s.vdim)
+        return (linear(a1, lf.o_proj.weight), linear(a2, rt.o_proj.weight), m.left_norm.weight, m.right_norm.weight)
+
+    def _mlp(self, i, mlp, h, rb: RaggedBatch):
+        gu_w = self.w[i]["gu"]
+        F = gu_w.shape[0] // 2
+        pgu = self.pk(i, "gu") if rb.decode else None
+        if pgu is not None and pgu.glu:
+            act = K.gemm_packed(h, pgu, glu=K.GLU_SILU)
+        else:
+            gu = linear(h, gu_w, packed=pgu)
+            act = K.glu_fwd(gu[:, :F], gu[:, F:], K.GLU_SILU) if gu.dtype == torch.bfloat16 and F % 8 == 0 else SK.silu_mul(gu)
+        return linear(act, mlp.down_proj.weight, packed=self.pk(i, "down") if rb.decode else None)
+
+    # ------------------------------------------------------------------------------------------------ the stack
+    @torch.no_grad()
+    def forward(self, rb: RaggedBatch, pool, layer_sums: Optional[list] = None) -> torch.Tensor:
+        """Final normed hidden rows [n, D] of the batch's tokens. `pool`: the engine's PagePool (cache, page table, states).
+        `layer_sums` (a list) receives the sum of the streams after every layer pass."""
+        cfg, model = self.cfg, self.model
+        eps, n = cfg.norm_eps, rb.n
+        x = torch.empty((n, max(cfg.streams, 1), cfg.embed_dim), dtype=torch.float32, device=rb.tokens.device)
+        close = dict(tokens=rb.tokens, embed=model.embed_tokens)       # what the next stream_step closes
+
+        def pending(out, hc):
+            y, y2, wy, wy2 = out
+            _, w_out, mix = self._hc(hc)
+            return dict(y=y, y2=y2, wy=wy, wy2=wy2, mix=mix, w_out=w_out)
+
+        ended = False                                                  # the pending sublayer ends a layer pass
+        def step(w_in, norm_w):
+            nonlocal ended
+            total = None
+            if layer_sums is not None and ended:
+                total = torch.empty((n, cfg.embed_dim), dtype=torch.float32, device=x.device)
+                layer_sums.append(total)
+            ended = False
+            return SK.stream_step(x, eps, w_in=w_in, norm_w=norm_w, sum_out=total, **close)
+
+        for r, i in enumerate(self.runs):
+            layer = model.layers[i]
+            h = step(self._hc(layer.hc1)[0], layer.input_layernorm.weight)
+            mix = self._rglru if isinstance(layer.mixer, RGLRUMixer) else self._parallel
+            close = pending(mix(i, layer.mixer, h, rb, pool, r), layer.hc1)
+            if layer.mlp is not None:
+                h = step(self._hc(layer.hc2)[0], layer.post_attention_layernorm.weight)
+                close = pending((self._mlp(i, layer.mlp, h, rb), None, None, None), layer.hc2)
+            ended = True
+        return step(None, model.norm.weight)
+
+    def logits(self, hidden: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """fp32 logits of normed hidden rows."""
+        packed = self.pk(len(self.model.layers), "head")
+        if hidden.dtype == torch.bfloat16 and packed is not None:
+            return K.gemm_packed(hidden, packed, out=out, out_dtype=torch.float32)
+        if hidden.dtype == torch.bfloat16 and hidden.shape[1] % 8 == 0:
+            return K.gemm(hidden, self.model.head_weight(), out=out, out_dtype=torch.float32)
+        z = linear(hidden, self.model.head_weight(), out_dtype=torch.float32)
+        return z if out is None else out.copy_(z)

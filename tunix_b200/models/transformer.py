@@ -511,6 +511,9 @@ def create_model(cfg: ModelConfig, device=None, seed: int = 0, init: bool = True
     if cfg.family == "gemma4":
         from .gemma4 import Gemma4Transformer
         model = Gemma4Transformer(cfg, device=device)
+    elif hasattr(cfg, "layer_specs"):
+        from .stack import StackModel
+        model = StackModel(cfg, device=device)
     else:
         model = Transformer(cfg, device=device)
     if init:
