@@ -15,6 +15,9 @@ template <>
 __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
 
 __device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+// e^z for z <= 0 that is raised to high powers by a recurrence: near 1 the error of expf (up to one unit in the last place,
+// always to the same side for a slowly varying z) would add up over a thousand steps, so the sum is rounded once.
+__device__ __forceinline__ float decay_exp(float z) { return z > -0.6f ? 1.f + expm1f(z) : expf(z); }
 // log(1 + e^z), without overflow
 __device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float log_sigmoid(float z) { return -softplus(-z); }

@@ -85,7 +85,7 @@ rglru_gates_kernel(const T* __restrict__ u, const T* __restrict__ ra, const T* _
     if (t >= nt) continue;
     const float la = -8.f * sigmoid(sr[j]) * sp;
     const long long o = (long long)(t0 + t) * W + ch;
-    A[o] = expf(la);
+    A[o] = decay_exp(la);
     B[o] = sqrtf(-expm1f(2.f * la)) * sigmoid(si[j]) * us[t * bs + col];
   }
 }
@@ -170,7 +170,7 @@ mlstm_seq_kernel(const T* __restrict__ proj, long long ldp, int q_off, int k_off
     const float ig = cap * tanhf((gates[(long long)t * 2 * heads + hd] + bi) / cap);
     const float fg = log_sigmoid(cap * tanhf((gates[(long long)t * 2 * heads + heads + hd] + bf) / cap));
     const float mn = fmaxf(fg + m, ig);
-    const float da = expf(fg + m - mn), db = expf(ig - mn);
+    const float da = decay_exp(fg + m - mn), db = expf(ig - mn);
     m = mn;
     __syncthreads();
     float nq = 0.f;
