@@ -39,6 +39,12 @@ struct AttnArgs {
   long long ldo;
   float* lse;                // [B, N, Tq]
   int* status;
+  // paged form: the query tiles of a ragged batch, keys and values in the pages of their sequences
+  const int *cu, *slot, *pos0, *tile_t0, *tile_ent, *table;
+  int max_pages, page_size;
+  int keep;                  // with a window: the first `keep` tokens of a sequence stay visible
+  const float* bias;         // [N, far + 1] added to the score of a key at distance min(distance, far), or null
+  int far;
 };
 
 template <int H>
@@ -58,7 +64,7 @@ struct FwdCfg {
   static constexpr int TMEM_COLS = (128 + H) <= 256 ? 256 : 512;
 };
 
-template <int H>
+template <int H, bool PAGED>
 __global__ void __launch_bounds__(160, 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                 const __grid_constant__ CUtensorMap tmV, const AttnArgs a) {
@@ -78,15 +84,36 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   const int qt = gridDim.x - 1 - blockIdx.x;  // heavy (late) causal tiles first
   const int n = blockIdx.y, b = blockIdx.z;
   const int kvh = n / (a.N / a.KH);
-  const int q0 = qt * BQ;
+  // the tile's first row in Q and O, its valid rows, the position of its first query, the keys of its sequence
+  int row0, nrows, i0, Tk;
+  const int* pages = nullptr;
+  if (PAGED) {
+    const int e = a.tile_ent[qt];
+    row0 = a.tile_t0[qt];
+    nrows = min(BQ, a.cu[e + 1] - row0);
+    i0 = a.pos0[e] + row0 - a.cu[e];
+    Tk = i0 + nrows;
+    pages = a.table + (long long)a.slot[e] * a.max_pages;
+  } else {
+    row0 = b * a.Tq + qt * BQ;
+    nrows = a.Tq - qt * BQ;
+    i0 = qt * BQ + a.q_off;
+    Tk = a.Tk;
+  }
 
-  // key-block range of this query tile
-  int kv_end = a.Tk;
-  if (a.causal) kv_end = min(a.Tk, q0 + BQ + a.q_off);
+  // key-block range of this query tile; blocks of kept first tokens come before those of the window
+  int kv_end = Tk;
+  if (a.causal) kv_end = min(Tk, i0 + BQ);
   int kv_start = 0;
-  if (a.window > 0) kv_start = max(0, q0 + a.q_off - a.window + 1);
+  if (a.window > 0) kv_start = max(0, i0 - a.window + 1);
   const int jb0 = kv_start / BKV;
-  const int nblk = kv_end > jb0 * BKV ? (kv_end - jb0 * BKV + BKV - 1) / BKV : 0;
+  const int n_sink = PAGED ? min((min(a.keep, Tk) + BKV - 1) / BKV, jb0) : 0;
+  const int nblk = n_sink + (kv_end > jb0 * BKV ? (kv_end - jb0 * BKV + BKV - 1) / BKV : 0);
+  auto block_key = [&](int j) { return (j < n_sink ? j : jb0 + j - n_sink) * BKV; };      // first key of block j
+  auto block_row = [&](int j) {                                                           // its row in the K / V maps
+    const int k = block_key(j);
+    return PAGED ? pages[k / a.page_size] * a.page_size + k % a.page_size : b * Tk + k;
+  };
 
   if (threadIdx.x == 0) {
     mbar_init(barQ, 1);
@@ -116,17 +143,18 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       const uint32_t idesc_o = make_idesc_bf16(BQ, H, 0, 1);
       auto load_k = [&](int j) {
         mbar_expect_tx(barK, C_::KV_BYTES);
+        const int row = block_row(j);
 #pragma unroll
         for (int c = 0; c < C_::HS; ++c)
-          tma_load_2d(sK + c * (BKV * 128), &tmK, barK, kvh * H + 64 * c, b * a.Tk + (jb0 + j) * BKV);
+          tma_load_2d(sK + c * (BKV * 128), &tmK, barK, kvh * H + 64 * c, row);
       };
       auto load_v = [&](int j) {
         const uint32_t bar = barV0 + 8 * (j & 1);
         mbar_expect_tx(bar, C_::KV_BYTES);
+        const int row = block_row(j);
 #pragma unroll
         for (int c = 0; c < C_::HS; ++c)
-          tma_load_2d(sV + (j & 1) * C_::KV_BYTES + c * (BKV * 128), &tmV, bar, kvh * H + 64 * c,
-                      b * a.Tk + (jb0 + j) * BKV);
+          tma_load_2d(sV + (j & 1) * C_::KV_BYTES + c * (BKV * 128), &tmV, bar, kvh * H + 64 * c, row);
       };
       auto issue_s = [&](int j) {
         const uint32_t d = tmem + C_::TMEM_S + (j & 1) * BKV;
@@ -142,7 +170,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       mbar_expect_tx(barQ, C_::Q_BYTES);
 #pragma unroll
       for (int c = 0; c < C_::HS; ++c)
-        tma_load_2d(sQ + c * (BQ * 128), &tmQ, barQ, n * H + 64 * c, b * a.Tq + q0);
+        tma_load_2d(sQ + c * (BQ * 128), &tmQ, barQ, n * H + 64 * c, row0);
       load_k(0);
       load_v(0);
       ok = ok && mbar_wait_bounded(barQ, 0, abort_flag, a.status, ST_TIMEOUT_PRODUCER);
@@ -179,9 +207,10 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   } else {
     // ---------------------------------------------------------- softmax warps
     const int r = threadIdx.x;             // row inside the tile == TMEM lane
-    const int qi = q0 + r;                 // query index in the sequence
-    const bool row_valid = qi < a.Tq;
-    const int qpos = qi + a.q_off;
+    const int qi = qt * BQ + r;            // query index in the sequence (not PAGED)
+    const bool row_valid = r < nrows;
+    const int qpos = i0 + r;
+    const float* bias = PAGED && a.bias ? a.bias + (long long)n * (a.far + 1) : nullptr;
     const uint32_t lane_addr = (uint32_t)(warp * 32) << 16;
     const int my_seg = (a.seg_q && row_valid) ? a.seg_q[(long long)b * a.Tq + qi] : 0;
     const float sc2 = a.scale * LOG2E;
@@ -199,15 +228,32 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
 #pragma unroll
         for (int i = 0; i < 32; ++i) { sraw[i] = t0[i]; sraw[32 + i] = t1[i]; }
       }
-      const int k0 = (jb0 + j) * BKV;
+      const int k0 = block_key(j);
       float z[64];
       float mx = -INFINITY;
       const int* segk = a.seg_k ? a.seg_k + (long long)b * a.Tk + k0 : nullptr;
       // most key blocks of a causal tile lie fully below the diagonal: skip the per-element mask there
-      const bool need_mask = (k0 + BKV > a.Tk) || (segk != nullptr) ||
-                             (a.causal && (k0 + BKV - 1 > q0 + a.q_off)) ||
-                             (a.window > 0 && (k0 <= q0 + BQ - 1 + a.q_off - a.window));
-      if (!need_mask && a.softcap <= 0.f) {
+      const bool need_mask = (k0 + BKV > Tk) || (segk != nullptr) || (a.causal && (k0 + BKV - 1 > i0)) ||
+                             (a.window > 0 && (k0 <= i0 + BQ - 1 - a.window));
+      if (PAGED) {
+        if (bias) {
+#pragma unroll
+          for (int i = 0; i < 64; ++i)
+            z[i] = fmaf(__uint_as_float(sraw[i]), sc2, __ldg(bias + min(max(qpos - k0 - i, 0), a.far)) * LOG2E);
+        } else {
+#pragma unroll
+          for (int i = 0; i < 64; ++i) z[i] = __uint_as_float(sraw[i]) * sc2;
+        }
+        if (need_mask) {
+#pragma unroll
+          for (int i = 0; i < 64; ++i) {
+            const int kp = k0 + i;
+            if (kp > qpos || (a.window > 0 && kp <= qpos - a.window && kp >= a.keep)) z[i] = -INFINITY;
+          }
+        }
+#pragma unroll
+        for (int i = 0; i < 64; ++i) mx = fmaxf(mx, z[i]);
+      } else if (!need_mask && a.softcap <= 0.f) {
 #pragma unroll
         for (int i = 0; i < 64; ++i) {
           z[i] = __uint_as_float(sraw[i]) * sc2;
@@ -284,7 +330,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       ok = mbar_wait_bounded(barPV, (nblk - 1) & 1, abort_flag, a.status, ST_TIMEOUT_EPILOGUE);
     tc_fence_after();
     const float inv_l = (l > 0.f) ? 1.f / l : 0.f;
-    __nv_bfloat16* orow = a.O + ((long long)b * a.Tq + qi) * a.ldo + (long long)n * H;
+    __nv_bfloat16* orow = a.O + (long long)(row0 + r) * a.ldo + (long long)n * H;
 #pragma unroll 1
     for (int c = 0; c < H / 32; ++c) {
       uint32_t o[32];
@@ -307,7 +353,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         }
       }
     }
-    if (row_valid && a.lse)
+    if (!PAGED && row_valid && a.lse)
       a.lse[((long long)b * a.N + n) * a.Tq + qi] = (l > 0.f) ? (m_used / LOG2E + logf(l)) : INFINITY;
   }
 
@@ -332,10 +378,10 @@ int launch_fwd(const void* q, const void* k, const void* v, const AttnArgs& a, l
   if (tb_make_tmap_2d_bf16(&tv, v, (uint64_t)a.B * a.Tk, (uint64_t)a.KH * H, ldv, BKV, 64, 1)) return -3;
   static DeviceOnce once;
   if (once.first() &&
-      cudaFuncSetAttribute(attn_fwd_kernel<H>, cudaFuncAttributeMaxDynamicSharedMemorySize, C_::SMEM_BYTES) != cudaSuccess)
+      cudaFuncSetAttribute(attn_fwd_kernel<H, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, C_::SMEM_BYTES) != cudaSuccess)
     return -5;
   dim3 grid((a.Tq + BQ - 1) / BQ, a.N, a.B);
-  attn_fwd_kernel<H><<<grid, 160, C_::SMEM_BYTES, stream>>>(tq, tk, tv, a);
+  attn_fwd_kernel<H, false><<<grid, 160, C_::SMEM_BYTES, stream>>>(tq, tk, tv, a);
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
 }
 
@@ -760,6 +806,46 @@ TB_API int tb_attn_fwd(const void* q, const void* k, const void* v, void* o, flo
     case 64: return launch_fwd<64>(q, k, v, a, ldq, ldk, ldv, stream);
     case 128: return launch_fwd<128>(q, k, v, a, ldq, ldk, ldv, stream);
     case 256: return launch_fwd<256>(q, k, v, a, ldq, ldk, ldv, stream);
+    default: return -2;
+  }
+}
+
+template <int H>
+static int launch_fwd_paged(const void* q, const void* k, const void* v, const AttnArgs& a, long long rows, long long pool_rows,
+                            int tiles, cudaStream_t stream) {
+  using C_ = FwdCfg<H>;
+  CUtensorMap tq, tk, tv;
+  const uint64_t qc = (uint64_t)a.N * H, kc = (uint64_t)a.KH * H;
+  if (tb_make_tmap_2d_bf16(&tq, q, (uint64_t)rows, qc, qc, BQ, 64, 1) || tb_make_tmap_2d_bf16(&tk, k, (uint64_t)pool_rows, kc, kc, BKV, 64, 1) ||
+      tb_make_tmap_2d_bf16(&tv, v, (uint64_t)pool_rows, kc, kc, BKV, 64, 1))
+    return -3;
+  static DeviceOnce once;
+  if (once.first() &&
+      cudaFuncSetAttribute(attn_fwd_kernel<H, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, C_::SMEM_BYTES) != cudaSuccess)
+    return -5;
+  attn_fwd_kernel<H, true><<<dim3(tiles, a.N), 160, C_::SMEM_BYTES, stream>>>(tq, tk, tv, a);
+  return cudaGetLastError() == cudaSuccess ? 0 : -5;
+}
+
+// Causal attention of the query tiles (at most 128 rows of one entry each) of a ragged batch over paged keys and values:
+// q / out [n, N * H]; pools [pool_rows, KH * H] with page_size a multiple of 64; a key block of 64 tokens lies in one page
+// and is fetched by TMA through the page table. window <= 0: no window. The unused tail of a page must hold finite values.
+TB_API int tb_attn_fwd_paged(const void* q, const void* k_pool, const void* v_pool, void* out, int n, long long pool_rows, int N,
+                             int KH, int H, float scale, int window, int keep, const float* bias, int far, const int* cu,
+                             const int* slot, const int* pos0, const int* tile_t0, const int* tile_ent, int tiles,
+                             const int* table, int max_pages, int page_size, int* status, cudaStream_t stream) {
+  if (n <= 0 || tiles <= 0) return 0;
+  if (KH <= 0 || N % KH || page_size % BKV || N > 65535) return -2;
+  AttnArgs a = {};
+  a.N = N; a.KH = KH; a.scale = scale; a.causal = 1; a.window = window > 0 ? window : 0;
+  a.keep = a.window > 0 ? keep : 0; a.bias = bias; a.far = far;
+  a.O = reinterpret_cast<__nv_bfloat16*>(out); a.ldo = (long long)N * H; a.status = status;
+  a.cu = cu; a.slot = slot; a.pos0 = pos0; a.tile_t0 = tile_t0; a.tile_ent = tile_ent; a.table = table;
+  a.max_pages = max_pages; a.page_size = page_size;
+  switch (H) {
+    case 64: return launch_fwd_paged<64>(q, k_pool, v_pool, a, n, pool_rows, tiles, stream);
+    case 128: return launch_fwd_paged<128>(q, k_pool, v_pool, a, n, pool_rows, tiles, stream);
+    case 256: return launch_fwd_paged<256>(q, k_pool, v_pool, a, n, pool_rows, tiles, stream);
     default: return -2;
   }
 }

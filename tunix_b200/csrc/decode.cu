@@ -10,13 +10,15 @@
 //                    context split). The query heads of a kv head are the rows of a 16-row mma.sync tile, K / V
 //                    stream through a double-buffered cp.async stage and are read with ldmatrix; running
 //                    max / sum per query head, partial results of the splits merged by `paged_decode_combine`.
-//                    Sliding window and logit soft-cap supported. Memory-bound by construction: every K / V
+//                    Sliding window (optionally with kept first tokens), a bias per (distance, head) added to the
+//                    scores, and logit soft-cap supported; with a window only the tiles that hold visible keys are
+//                    walked and split over CTAs. Memory-bound by construction: every K / V
 //                    byte of the sequence is read exactly once per kv head.
 //
 // The reference keeps only host-side page-table logic (tunix/experimental/generate/*) and runs decode on a
 // dense cache through XLA (tunix/generate/sampler.py:732-793); these kernels are the device side of the
 // in-framework engine that replaces its vLLM / SGLang integrations.
-#include "common.cuh"
+#include "mma.cuh"
 
 using namespace tb;
 
@@ -107,28 +109,8 @@ qkv_post_kernel(__nv_bfloat16* __restrict__ qkv, long long ld, const int* __rest
   }
 }
 
-// ---- tensor-core fragments (warp-level mma.sync: with at most 16 query rows per kv head there is no 64/128-row
+// ---- tensor-core fragments (warp-level mma.sync of mma.cuh: with at most 16 query rows per kv head there is no 64/128-row
 // tile to give to tcgen05, and the kernel is bound by the K/V stream, not by math) --------------------------------
-__device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm_x4_t(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void mma_16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, int src_bytes) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(src_bytes) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-
 constexpr int TILE_KEYS = 64;   // keys staged per pipeline stage; 16 per warp
 
 // byte offset of 16-byte chunk c of row r in a [rows, H] bf16 tile whose 128-byte groups are XOR-swizzled by row
@@ -145,6 +127,18 @@ __device__ __forceinline__ uint32_t tile_off(int r, int c) {
   return swz<H>(r, c);
 }
 
+// The key tiles a single query at position len - 1 walks: the tiles that hold kept first tokens, then those of the window.
+struct KeyTiles {
+  int w_lo, first, n_sink, total;
+  __device__ __forceinline__ KeyTiles(int len, int window, int keep) {
+    w_lo = window > 0 ? max(0, len - window) : 0;
+    first = w_lo / TILE_KEYS;
+    n_sink = min((min(keep, len) + TILE_KEYS - 1) / TILE_KEYS, first);
+    total = n_sink + (len + TILE_KEYS - 1) / TILE_KEYS - first;
+  }
+  __device__ __forceinline__ int start(int tile) const { return (tile < n_sink ? tile : first + tile - n_sink) * TILE_KEYS; }
+};
+
 // One CTA per (sequence, kv head, context split): the G (<= 16) query heads of the kv head are the 16 rows of the
 // A operand, a warp owns 16 keys of each 64-key stage, S = Q K^T and O += P V run on mma.sync and read K / V with
 // ldmatrix; every K / V byte is read once. Staging: with pages of a multiple of 64 tokens a tile lies in one page
@@ -158,7 +152,8 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_consta
                     const __nv_bfloat16* __restrict__ k_pool, const __nv_bfloat16* __restrict__ v_pool,
                     const int* __restrict__ page_table, int max_pages, int page_size,
                     const int* __restrict__ seq_ids, const int* __restrict__ seq_lens, int KH, int G, float scale,
-                    float softcap, int window, int num_splits, int split_tokens,
+                    float softcap, int window, int keep, const float* __restrict__ bias, int far,   // bias [N, far + 1] or null
+                    int num_splits, int split_tokens,
                     float* __restrict__ part_acc,                                               // [B, N, splits, H]
                     float* __restrict__ part_ml,                                                // [B, N, splits, 2]
                     __nv_bfloat16* __restrict__ out, long long ldo,   // written directly when there is one split
@@ -177,15 +172,16 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_consta
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int N = KH * G;
   const int len = seq_lens[b];
-  int lo = split * split_tokens;
-  if (lo >= len) {                // past the end of this sequence: the combine kernel never reads this split
+  const KeyTiles kt(len, window, keep);
+  const int tile0 = split * (split_tokens / TILE_KEYS);
+  const int n_tiles = min(kt.total - tile0, split_tokens / TILE_KEYS);
+  if (len <= 0 || n_tiles <= 0) { // past the end of this sequence: the combine kernel never reads this split
     if (num_splits == 1)          // (an empty slot with a single split: its output row is zero)
       for (int idx = threadIdx.x; idx < G * H; idx += 128)
         out[(long long)b * ldo + (long long)(kh * G) * H + idx] = __float2bfloat16(0.f);
     return;
   }
-  const int hi = min(len, lo + split_tokens);
-  if (window > 0) lo = max(lo, len - window);
+  auto visible = [&](int t) { return t < len && (t >= kt.w_lo || t < keep); };
   const int* pt = page_table + (long long)seq_ids[b] * max_pages;
   const long long row_elems = (long long)KH * H;
   const uint32_t smem_base = smem_u32(smem);
@@ -199,9 +195,6 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_consta
     *reinterpret_cast<uint4*>(q_s + swz<H>(r, c)) = u;
   }
 
-  const int t_first = split * split_tokens + ((max(lo - split * split_tokens, 0)) / TILE_KEYS) * TILE_KEYS;
-  const int n_tiles = hi > t_first ? (hi - t_first + TILE_KEYS - 1) / TILE_KEYS : 0;
-
   if (TMA) {
     if (tid == 0) {
       for (int i = 0; i < STAGES; ++i) mbar_init(smem_u32(&full_bars[i]), 1);
@@ -212,7 +205,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_consta
   }
   // one thread, one tile: the tile's 64 tokens lie in one page
   auto issue_tma = [&](int tile, int buf) {
-    const int t0 = t_first + tile * TILE_KEYS;
+    const int t0 = kt.start(tile0 + tile);
     const int row = pt[t0 / page_size] * page_size + t0 % page_size;
     const uint32_t kb = smem_base + buf * 2 * TILE_BYTES, vb = kb + TILE_BYTES;
     const uint32_t bar = smem_u32(&full_bars[buf]);
@@ -224,12 +217,12 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_consta
     }
   };
   auto issue = [&](int tile, int buf) {
-    const int t0 = t_first + tile * TILE_KEYS;
+    const int t0 = kt.start(tile0 + tile);
     const uint32_t kb = smem_base + buf * 2 * TILE_BYTES, vb = kb + TILE_BYTES;
     for (int idx = tid; idx < TILE_KEYS * CPR; idx += 128) {
       const int r = idx / CPR, c = idx - r * CPR;
       const int t = t0 + r;
-      const bool ok = t >= lo && t < hi;
+      const bool ok = visible(t);
       long long off = 0;
       if (ok) {
         const int page = pt[t / page_size];
@@ -271,8 +264,8 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_consta
     }
     const uint32_t kb = smem_base + buf * 2 * TILE_BYTES, vb = kb + TILE_BYTES;
     const int kr0 = warp * 16;
-    const int tw = t_first + tile * TILE_KEYS + kr0;      // first key of this warp's slice
-    if (tw < hi) {
+    const int tw = kt.start(tile0 + tile) + kr0;          // first key of this warp's slice
+    if (tw < len) {
       float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
 #pragma unroll
       for (int ks = 0; ks < H / 16; ++ks) {
@@ -290,7 +283,11 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_consta
           const int t = tw + nb * 8 + 2 * (lane & 3) + (j & 1);
           float v = s[nb][j] * scale;
           if (softcap > 0.f) v = softcap * tanhf(v / softcap);
-          if (t < lo || t >= hi) v = -INFINITY;
+          if (bias != nullptr && t < len) {
+            const int row = (lane >> 2) + (j >> 1) * 8;
+            if (row < G) v += __ldg(bias + (long long)(kh * G + row) * (far + 1) + min(len - 1 - t, far));
+          }
+          if (!visible(t)) v = -INFINITY;
           s[nb][j] = v;
           if (j < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
         }
@@ -383,12 +380,13 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_consta
 // out[b, n, :] = sum_s acc_s * exp(m_s - M) / sum_s l_s * exp(m_s - M)
 __global__ void paged_decode_combine_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
                                             const int* __restrict__ seq_lens, int N, int H, int num_splits, int split_tokens,
-                                            int window, __nv_bfloat16* __restrict__ out, long long ldo) {
+                                            int window, int keep, __nv_bfloat16* __restrict__ out, long long ldo) {
   pdl_trigger();
   pdl_wait();
   const int b = blockIdx.x, n = blockIdx.y;
   const int len = seq_lens[b];
-  const int used = min(num_splits, (len + split_tokens - 1) / split_tokens);
+  const int tps = split_tokens / TILE_KEYS;
+  const int used = len > 0 ? min(num_splits, (KeyTiles(len, window, keep).total + tps - 1) / tps) : 0;
   const long long base = ((long long)b * N + n) * num_splits;
   float M = -INFINITY;
   for (int s = 0; s < used; ++s) M = fmaxf(M, part_ml[(base + s) * 2]);
@@ -412,8 +410,8 @@ template <int H, bool TMA, int STAGES>
 int launch_decode_v(int G, dim3 grid, cudaStream_t stream, const CUtensorMap& tmK, const CUtensorMap& tmV,
                     const __nv_bfloat16* q, long long ldq, const __nv_bfloat16* kp, const __nv_bfloat16* vp, const int* pt,
                     int max_pages, int page_size, const int* seq_ids, const int* seq_lens, int KH, float scale, float softcap,
-                    int window, int splits, int split_tokens, float* pa, float* pml, __nv_bfloat16* out, long long ldo,
-                    int* status) {
+                    int window, int keep, const float* bias, int far, int splits, int split_tokens, float* pa, float* pml,
+                    __nv_bfloat16* out, long long ldo, int* status) {
   constexpr int TILE2 = 2 * TILE_KEYS * H * 2;                       // one stage: a K tile and a V tile
   constexpr int SMEM = STAGES * TILE2 + (TMA ? 1024 : 0);
   static DeviceOnce once;
@@ -423,7 +421,7 @@ int launch_decode_v(int G, dim3 grid, cudaStream_t stream, const CUtensorMap& tm
   // a split of one 64-key tile needs one stage only: more CTAs fit on an SM
   const int smem = split_tokens > TILE_KEYS ? SMEM : TILE2 + (TMA ? 1024 : 0);
   return launch_pdl(paged_decode_kernel<H, TMA, STAGES>, grid, dim3(128), smem, stream, tmK, tmV, q, ldq, kp, vp, pt, max_pages,
-                    page_size, seq_ids, seq_lens, KH, G, scale, softcap, window, splits, split_tokens, pa, pml, out, ldo,
+                    page_size, seq_ids, seq_lens, KH, G, scale, softcap, window, keep, bias, far, splits, split_tokens, pa, pml, out, ldo,
                     status) == cudaSuccess ? 0 : -5;
 }
 
@@ -432,7 +430,8 @@ template <int H>
 int launch_decode(int G, dim3 grid, cudaStream_t stream, const __nv_bfloat16* q, long long ldq,
                   const __nv_bfloat16* kp, const __nv_bfloat16* vp, long long pool_rows, const int* pt, int max_pages,
                   int page_size, const int* seq_ids, const int* seq_lens, int KH, float scale, float softcap, int window,
-                  int splits, int split_tokens, float* pa, float* pml, __nv_bfloat16* out, long long ldo, int* status) {
+                  int keep, const float* bias, int far, int splits, int split_tokens, float* pa, float* pml, __nv_bfloat16* out,
+                  long long ldo, int* status) {
   static const bool no_tma = getenv("TUNIX_B200_DECODE_NO_TMA") != nullptr;
   static const char* stages_env = getenv("TUNIX_B200_DECODE_STAGES");
   CUtensorMap tmK, tmV;
@@ -442,7 +441,7 @@ int launch_decode(int G, dim3 grid, cudaStream_t stream, const __nv_bfloat16* q,
                    tb_make_tmap_2d_bf16(&tmK, kp, (uint64_t)pool_rows, (uint64_t)KH * H, (uint64_t)KH * H, TILE_KEYS, 64, 1) == 0 &&
                    tb_make_tmap_2d_bf16(&tmV, vp, (uint64_t)pool_rows, (uint64_t)KH * H, (uint64_t)KH * H, TILE_KEYS, 64, 1) == 0;
 #define LD(T, S) launch_decode_v<H, T, S>(G, grid, stream, tmK, tmV, q, ldq, kp, vp, pt, max_pages, page_size, seq_ids, seq_lens, \
-                                         KH, scale, softcap, window, splits, split_tokens, pa, pml, out, ldo, status)
+                                         KH, scale, softcap, window, keep, bias, far, splits, split_tokens, pa, pml, out, ldo, status)
   if (!tma) return LD(false, 2);
   // measured at head dim 128 (8 kv heads, 256 sequences x 768 tokens): 2 / 3 / 4 stages take 157 / 161 / 194 us,
   // cp.async staging 190 us: three CTAs per SM with two stages each beat deeper rings on fewer CTAs
@@ -497,34 +496,40 @@ TB_API int tb_qkv_post(void* qkv, long long ld, const int* seq_ids, const int* p
 // workspace: part_acc fp32 [B*N*splits*H], part_ml fp32 [B*N*splits*2] with splits = ceil(max_ctx / split_tokens);
 // split_tokens = context tokens per CTA, a multiple of 64 in [64, 2048] (0 = 256). CTAs of splits that lie past the
 // end of their sequence return at once. pool_rows = num_pages * page_size (rows of the pools, for the tensor maps;
-// 0 = no TMA staging). status: word that a bounded mbarrier wait writes its code to.
+// 0 = no TMA staging). window > 0: keys at distance < window, and the sequence's first `keep` tokens. bias fp32
+// [N, far + 1] (null = none) is added to the scaled score of a key at distance min(distance, far). status: word that a bounded mbarrier wait writes its code to.
 TB_API int tb_paged_decode(const void* q, long long ldq, const void* k_pool, const void* v_pool,
                            const int* page_table, int max_pages, int page_size, const int* seq_ids,
                            const int* seq_lens, int B, int N, int KH, int H, int max_ctx, float scale, float softcap,
-                           int window, int split_tokens, long long pool_rows, float* part_acc, float* part_ml, void* out,
-                           long long ldo, int* status, cudaStream_t stream) {
+                           int window, int keep, const float* bias, int far, int split_tokens, long long pool_rows,
+                           float* part_acc, float* part_ml, void* out, long long ldo, int* status, cudaStream_t stream) {
   if (B <= 0) return 0;
   if (KH <= 0 || N % KH || (ldq % 8)) return -2;
   const int G = N / KH;
   if (G > MAX_G) return -2;
   if (split_tokens <= 0) split_tokens = 256;
   if (split_tokens % TILE_KEYS || split_tokens > MAX_SPLIT_TOKENS) return -2;
-  const int splits = (max_ctx + split_tokens - 1) / split_tokens;
+  int max_tiles = (max_ctx + TILE_KEYS - 1) / TILE_KEYS;
+  if (window > 0) {
+    const int vis = (keep + TILE_KEYS - 1) / TILE_KEYS + (window + TILE_KEYS - 1) / TILE_KEYS + 1;
+    if (vis < max_tiles) max_tiles = vis;
+  }
+  const int splits = (max_tiles + split_tokens / TILE_KEYS - 1) / (split_tokens / TILE_KEYS);
   dim3 grid(B, KH, splits);
   int rc;
   auto qq = (const __nv_bfloat16*)q;
   auto kp = (const __nv_bfloat16*)k_pool;
   auto vp = (const __nv_bfloat16*)v_pool;
   switch (H) {
-    case 64: rc = launch_decode<64>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
-    case 128: rc = launch_decode<128>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
-    case 256: rc = launch_decode<256>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
+    case 64: rc = launch_decode<64>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, keep, bias, far, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
+    case 128: rc = launch_decode<128>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, keep, bias, far, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
+    case 256: rc = launch_decode<256>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, keep, bias, far, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
     default: return -2;
   }
   if (rc) return rc;
   if (splits == 1) return 0;
   return launch_pdl(paged_decode_combine_kernel, dim3(B, N), dim3(128), 0, stream, (const float*)part_acc,
-                    (const float*)part_ml, seq_lens, N, H, splits, split_tokens, window, (__nv_bfloat16*)out, ldo) == cudaSuccess ? 0 : -5;
+                    (const float*)part_ml, seq_lens, N, H, splits, split_tokens, window, keep, (__nv_bfloat16*)out, ldo) == cudaSuccess ? 0 : -5;
 }
 
 // ------------------------------------------------------------------ per-step bookkeeping of the decode loop

@@ -12,6 +12,7 @@
 //              of a head need not meet.
 //
 // This file is compiled without fast-math: the same kernels serve the 32-bit mode.
+#include "mma.cuh"
 #include "precise.cuh"
 
 using namespace tb;
@@ -117,6 +118,299 @@ __global__ void rglru_scan_kernel(const float* __restrict__ A, const float* __re
     ring[(sl * K + (p0 + t - t0) % K) * W + c] = to_f(proj[(long long)t * ldp + x_off + c]);
 }
 
+// ---- bf16, prompt portions: the gates on tensor cores, the recurrence cut into tiles of LT tokens
+// A tile is LT consecutive tokens of one entry (tile_t0 / tile_ent from the host). The gate kernel leaves, per token and
+// channel, the tile-local recurrence h (from zero) and the running product p of the decays; a small kernel chains the
+// tiles' last rows; the last kernel adds p * carry and applies the output gate. Nothing waits on another block.
+constexpr int LT = 64;          // tokens per tile
+constexpr int LC = 64;          // channels per CTA of the gate kernel
+constexpr int LTPC = 4;         // consecutive tiles per CTA: the weights stay in shared memory
+
+struct Tiles {
+  const int* t0;      // [tiles] first token of the tile
+  const int* ent;     // [tiles] its entry
+  int count;
+};
+
+// u [n, W] -> H, P fp32 [n, W], and the tiles' last rows in LH, LP fp32 [tiles, W]
+__global__ void __launch_bounds__(256)
+rglru_tile_kernel(const __nv_bfloat16* __restrict__ u, const __nv_bfloat16* __restrict__ ra,
+                  const __nv_bfloat16* __restrict__ ba, const __nv_bfloat16* __restrict__ ri,
+                  const __nv_bfloat16* __restrict__ bi, const __nv_bfloat16* __restrict__ lam, Ragged rb, Tiles tl, int W,
+                  int bs, float* __restrict__ H, float* __restrict__ P, float* __restrict__ LH, float* __restrict__ LP) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  const int kp = (bs + 15) & ~15;                       // contraction length, zero-padded
+  const int pitch = kp * 2 + 16;                        // bytes per row
+  uint8_t* Us = smem;                                   // [LT] rows of u
+  uint8_t* Ws = smem + LT * pitch;                      // [2 * LC] rows: LC of ra, LC of ri
+  float* As = reinterpret_cast<float*>(Ws + 2 * LC * pitch);   // [LT][LC + 1]
+  float* Bs = As + LT * (LC + 1);
+  __shared__ float segA[4][LC], segB[4][LC];
+  pdl_trigger();
+  pdl_wait();
+  const int per_blk = (bs + LC - 1) / LC;
+  const int blk = blockIdx.x / per_blk, o0 = (blockIdx.x - blk * per_blk) * LC;    // channels o0.. of block blk
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, li = lane >> 3, lr = lane & 7;
+  const int chunks = kp / 8;
+  const uint32_t us = smem_u32(Us), ws = smem_u32(Ws);
+  for (int i = tid; i < 2 * LC * chunks; i += 256) {
+    const int r = i / chunks, c = i - r * chunks;
+    const int o = o0 + (r & (LC - 1));
+    const bool ok = o < bs && c * 8 < bs;
+    const __nv_bfloat16* src = (r < LC ? ra : ri) + ((long long)blk * bs + (ok ? o : 0)) * bs + (ok ? c * 8 : 0);
+    cp_async16(ws + r * pitch + c * 16, src, ok ? 16 : 0);
+  }
+  cp_async_commit();
+  for (int k = 0; k < LTPC; ++k) {
+    const int tile = blockIdx.y * LTPC + k;
+    if (tile >= tl.count) break;
+    const int e = tl.ent[tile], t0 = tl.t0[tile];
+    const int nt = min(LT, rb.cu[e + 1] - t0);
+    for (int i = tid; i < LT * chunks; i += 256) {
+      const int r = i / chunks, c = i - r * chunks;
+      const bool ok = r < nt && c * 8 < bs;
+      cp_async16(us + r * pitch + c * 16, u + (ok ? (long long)(t0 + r) * W + (long long)blk * bs + c * 8 : 0), ok ? 16 : 0);
+    }
+    cp_async_commit();
+    cp_async_wait<0>();
+    __syncthreads();
+    // warps: 4 rows of 16 tokens x 2 halves of 32 channels; both gates of a channel in the same thread
+    const int m0 = (warp & 3) * 16, n0 = (warp >> 2) * 32;
+    float r[4][4], g[4][4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+#pragma unroll
+      for (int q = 0; q < 4; ++q) r[j][q] = g[j][q] = 0.f;
+    for (int ks = 0; ks < kp / 16; ++ks) {
+      uint32_t a[4], w0[4], w1[4];
+      ldsm_x4(a, us + (m0 + (li & 1) * 8 + lr) * pitch + (ks * 2 + (li >> 1)) * 16);
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int row = n0 + h * 16 + (li >> 1) * 8 + lr;
+        ldsm_x4(w0, ws + row * pitch + (ks * 2 + (li & 1)) * 16);
+        ldsm_x4(w1, ws + (LC + row) * pitch + (ks * 2 + (li & 1)) * 16);
+        mma_16816(r[2 * h], a, w0[0], w0[1]);
+        mma_16816(r[2 * h + 1], a, w0[2], w0[3]);
+        mma_16816(g[2 * h], a, w1[0], w1[1]);
+        mma_16816(g[2 * h + 1], a, w1[2], w1[3]);
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        const int c = n0 + j * 8 + 2 * (lane & 3) + (q & 1), t = m0 + (lane >> 2) + (q >> 1) * 8;
+        const int o = o0 + c;
+        float av = 1.f, bv = 0.f;
+        if (t < nt && o < bs) {
+          const int ch = blk * bs + o;
+          const float la = -8.f * sigmoid(r[j][q] + to_f(ba[ch])) * softplus(to_f(lam[ch]));
+          const float uv = to_f(*reinterpret_cast<const __nv_bfloat16*>(Us + t * pitch + o * 2));
+          av = decay_exp(la);
+          bv = sqrtf(-expm1f(2.f * la)) * sigmoid(g[j][q] + to_f(bi[ch])) * uv;
+        }
+        As[t * (LC + 1) + c] = av;
+        Bs[t * (LC + 1) + c] = bv;
+      }
+    __syncthreads();
+    // recurrence inside the tile: 4 segments of 16 tokens per channel, then the segments in order
+    const int c = tid & (LC - 1), sg = tid >> 6;
+    float pa = 1.f, hb = 0.f;
+#pragma unroll
+    for (int t = 0; t < LT / 4; ++t) {
+      const int x = (sg * (LT / 4) + t) * (LC + 1) + c;
+      const float av = As[x];
+      hb = av * hb + Bs[x];
+      pa *= av;
+      As[x] = pa;
+      Bs[x] = hb;
+    }
+    segA[sg][c] = pa;
+    segB[sg][c] = hb;
+    __syncthreads();
+    float cp = 1.f, ch = 0.f;
+    for (int j = 0; j < sg; ++j) { ch = segA[j][c] * ch + segB[j][c]; cp *= segA[j][c]; }
+    if (o0 + c < bs) {
+      const long long col = (long long)blk * bs + o0 + c;
+#pragma unroll
+      for (int t = 0; t < LT / 4; ++t) {
+        const int tt = sg * (LT / 4) + t;
+        if (tt >= nt) break;
+        const float p = As[tt * (LC + 1) + c], h = Bs[tt * (LC + 1) + c] + p * ch;
+        H[(long long)(t0 + tt) * W + col] = h;
+        P[(long long)(t0 + tt) * W + col] = p * cp;
+        if (tt == nt - 1) {
+          LH[(long long)tile * W + col] = h;
+          LP[(long long)tile * W + col] = p * cp;
+        }
+      }
+    }
+    __syncthreads();
+  }
+}
+
+// One thread per (entry, channel): LH becomes the state before each tile; the entry's new state and ring rows.
+// first_tile[e]: the entry's first tile.
+__global__ void rglru_chain_kernel(float* __restrict__ LH, const float* __restrict__ LP, const __nv_bfloat16* __restrict__ proj,
+                                   long long ldp, int x_off, Ragged rb, const int* __restrict__ first_tile, int W, int K,
+                                   float* __restrict__ state, float* __restrict__ ring) {
+  pdl_trigger();
+  pdl_wait();
+  const int c = blockIdx.x * blockDim.x + threadIdx.x, e = blockIdx.y;
+  if (c >= W) return;
+  const int p0 = rb.pos0[e], t0 = rb.cu[e], t1 = rb.cu[e + 1];
+  if (p0 < 0 || t1 <= t0) return;
+  const long long sl = rb.slot[e];
+  float s = p0 > 0 ? state[sl * W + c] : 0.f;
+  const int a = first_tile[e], b = a + (t1 - t0 + LT - 1) / LT;
+  for (int x = a; x < b; x += 8) {
+    float h[8], p[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+      if (x + j < b) { h[j] = LH[(long long)(x + j) * W + c]; p[j] = LP[(long long)(x + j) * W + c]; }
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+      if (x + j < b) {
+        LH[(long long)(x + j) * W + c] = s;
+        s = p[j] * s + h[j];
+      }
+  }
+  state[sl * W + c] = s;
+  for (int t = max(t0, t1 - K); t < t1; ++t)
+    ring[(sl * K + (p0 + t - t0) % K) * W + c] = to_f(proj[(long long)t * ldp + x_off + c]);
+}
+
+// out = (H + P * state before the tile) * gelu(y); 4 channels per thread
+__global__ void __launch_bounds__(256)
+rglru_out_kernel(const float* __restrict__ H, const float* __restrict__ P, const float* __restrict__ carry,
+                 const __nv_bfloat16* __restrict__ proj, long long ldp, int y_off, Ragged rb, const int* __restrict__ first_tile,
+                 int W, __nv_bfloat16* __restrict__ out) {
+  pdl_trigger();
+  pdl_wait();
+  const int per = W / 4;
+  const long long total = (long long)rb.n * per;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const int t = (int)(i / per), c = (int)(i - (long long)t * per) * 4;
+    const int e = rb.ent[t];
+    const int tile = first_tile[e] + (t - rb.cu[e]) / LT;
+    const float4 h = *reinterpret_cast<const float4*>(H + (long long)t * W + c);
+    const float4 p = *reinterpret_cast<const float4*>(P + (long long)t * W + c);
+    const float4 s = *reinterpret_cast<const float4*>(carry + (long long)tile * W + c);
+    const uint2 y = *reinterpret_cast<const uint2*>(proj + (long long)t * ldp + y_off + c);
+    uint2 o;
+    o.x = pack_bf16((h.x + p.x * s.x) * gelu_tanh(bf16_lo(y.x)), (h.y + p.y * s.y) * gelu_tanh(bf16_hi(y.x)));
+    o.y = pack_bf16((h.z + p.z * s.z) * gelu_tanh(bf16_lo(y.y)), (h.w + p.w * s.w) * gelu_tanh(bf16_hi(y.y)));
+    *reinterpret_cast<uint2*>(out + (long long)t * W + c) = o;
+  }
+}
+
+// 4 channels per thread form of rglru_conv_kernel
+__global__ void __launch_bounds__(256)
+rglru_conv4_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int x_off, const __nv_bfloat16* __restrict__ w,
+                   const __nv_bfloat16* __restrict__ bias, const float* __restrict__ ring, Ragged rb, int W, int K,
+                   __nv_bfloat16* __restrict__ u) {
+  pdl_trigger();
+  pdl_wait();
+  const int per = W / 4;
+  const long long total = (long long)rb.n * per;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const int t = (int)(i / per), c = (int)(i - (long long)t * per) * 4;
+    const int e = rb.ent[t], p0 = rb.pos0[e], first = rb.cu[e], p = p0 + t - first;
+    float acc[4];
+#pragma unroll
+    for (int q = 0; q < 4; ++q) acc[q] = to_f(bias[c + q]);
+    for (int j = 0; j < K && j <= p; ++j) {
+      const int s = t - j;
+      float v[4];
+      if (s >= first) {
+        const uint2 x = *reinterpret_cast<const uint2*>(proj + (long long)s * ldp + x_off + c);
+        v[0] = bf16_lo(x.x); v[1] = bf16_hi(x.x); v[2] = bf16_lo(x.y); v[3] = bf16_hi(x.y);
+      } else {
+        const float4 x = *reinterpret_cast<const float4*>(ring + ((long long)rb.slot[e] * K + (p - j) % K) * W + c);
+        v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
+      }
+#pragma unroll
+      for (int q = 0; q < 4; ++q) acc[q] += to_f(w[(long long)(c + q) * K + K - 1 - j]) * v[q];
+    }
+    uint2 o;
+    o.x = pack_bf16(acc[0], acc[1]);
+    o.y = pack_bf16(acc[2], acc[3]);
+    *reinterpret_cast<uint2*>(u + (long long)t * W + c) = o;
+  }
+}
+
+// ---- bf16, one token per entry: convolution, gates, recurrence and output gate in one launch. CTA: 16 entries x DC output
+// channels of one block; every CTA computes the convolution of its whole block (the ring row written is never read).
+constexpr int DC = 32;
+__global__ void __launch_bounds__(128)
+rglru_step_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int x_off, int y_off,
+                  const __nv_bfloat16* __restrict__ cw, const __nv_bfloat16* __restrict__ cb,
+                  const __nv_bfloat16* __restrict__ ra, const __nv_bfloat16* __restrict__ ba,
+                  const __nv_bfloat16* __restrict__ ri, const __nv_bfloat16* __restrict__ bi,
+                  const __nv_bfloat16* __restrict__ lam, Ragged rb, int W, int bs, int K, float* __restrict__ state,
+                  float* __restrict__ ring, __nv_bfloat16* __restrict__ out) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  const int kp = (bs + 15) & ~15, pitch = kp * 2 + 16, chunks = kp / 8;
+  uint8_t* Us = smem;                                   // [16] rows of u
+  uint8_t* Ws = smem + 16 * pitch;                      // [2 * DC] rows
+  const uint32_t us = smem_u32(Us), ws = smem_u32(Ws);
+  const int per_blk = (bs + DC - 1) / DC;
+  const int blk = blockIdx.x / per_blk, o0 = (blockIdx.x - blk * per_blk) * DC, e0 = blockIdx.y * 16;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, li = lane >> 3, lr = lane & 7;
+  // weights do not depend on the kernels before
+  for (int i = tid; i < 2 * DC * chunks; i += 128) {
+    const int r = i / chunks, c = i - r * chunks, o = o0 + (r & (DC - 1));
+    const bool ok = o < bs && c * 8 < bs;
+    cp_async16(ws + r * pitch + c * 16, (r < DC ? ra : ri) + ((long long)blk * bs + (ok ? o : 0)) * bs + (ok ? c * 8 : 0), ok ? 16 : 0);
+  }
+  cp_async_commit();
+  pdl_trigger();
+  pdl_wait();
+  for (int i = tid; i < 16 * kp; i += 128) {
+    const int r = i / kp, c = i - r * kp, e = e0 + r;
+    float acc = 0.f;
+    if (e < rb.E && c < bs) {
+      const int p = rb.pos0[e];
+      if (p >= 0) {
+        const int ch = blk * bs + c;
+        const long long rows = (long long)rb.slot[e] * K;
+        const float x = to_f(proj[(long long)e * ldp + x_off + ch]);
+        acc = to_f(cb[ch]) + to_f(cw[(long long)ch * K + K - 1]) * x;
+        for (int j = 1; j < K && j <= p; ++j) acc += to_f(cw[(long long)ch * K + K - 1 - j]) * ring[(rows + (p - j) % K) * W + ch];
+        if (c >= o0 && c < o0 + DC) ring[(rows + p % K) * W + ch] = x;
+      }
+    }
+    *reinterpret_cast<__nv_bfloat16*>(Us + r * pitch + c * 2) = __float2bfloat16(acc);
+  }
+  cp_async_wait<0>();
+  __syncthreads();
+  float r[4] = {0.f, 0.f, 0.f, 0.f}, g[4] = {0.f, 0.f, 0.f, 0.f};
+  for (int ks = 0; ks < kp / 16; ++ks) {
+    uint32_t a[4], w[4];
+    ldsm_x4(a, us + ((li & 1) * 8 + lr) * pitch + (ks * 2 + (li >> 1)) * 16);
+    // matrices 0, 1: this warp's 8 channels of ra; 2, 3: of ri
+    ldsm_x4(w, ws + ((li >> 1) * DC + warp * 8 + lr) * pitch + (ks * 2 + (li & 1)) * 16);
+    mma_16816(r, a, w[0], w[1]);
+    mma_16816(g, a, w[2], w[3]);
+  }
+#pragma unroll
+  for (int q = 0; q < 4; ++q) {
+    const int o = o0 + warp * 8 + 2 * (lane & 3) + (q & 1), row = (lane >> 2) + (q >> 1) * 8, e = e0 + row;
+    if (o >= bs || e >= rb.E) continue;
+    const int ch = blk * bs + o, p = rb.pos0[e];
+    float res = 0.f;
+    if (p >= 0) {
+      const float la = -8.f * sigmoid(r[q] + to_f(ba[ch])) * softplus(to_f(lam[ch]));
+      const float uv = to_f(*reinterpret_cast<const __nv_bfloat16*>(Us + row * pitch + o * 2));
+      float* st = state + (long long)rb.slot[e] * W + ch;
+      const float s = (p > 0 ? decay_exp(la) * *st : 0.f) + sqrtf(-expm1f(2.f * la)) * sigmoid(g[q] + to_f(bi[ch])) * uv;
+      *st = s;
+      res = s * gelu_tanh(to_f(proj[(long long)e * ldp + y_off + ch]));
+    }
+    out[(long long)e * W + ch] = __float2bfloat16(res);
+  }
+}
+
 // ------------------------------------------------------------------------------------------------ mLSTM
 constexpr int MV = 32;          // value columns per CTA (a slice)
 constexpr int MTHREADS = 256;
@@ -204,27 +498,469 @@ mlstm_seq_kernel(const T* __restrict__ proj, long long ldp, int q_off, int k_off
   if (tid == 0) *Mh = m;
 }
 
+// ---- one token per entry: the state slice streams through registers, nothing is staged
+template <typename T>
+__global__ void __launch_bounds__(MTHREADS)
+mlstm_step_kernel(const T* __restrict__ proj, long long ldp, int q_off, int k_off, int v_off, const float* __restrict__ gates,
+                  const T* __restrict__ ib, const T* __restrict__ fb, float cap, Ragged rb, int heads, int dk, int dv,
+                  float* __restrict__ Sg, float* __restrict__ Ng, float* __restrict__ Mg, float* __restrict__ out) {
+  extern __shared__ float sm[];
+  float* qs = sm;                      // [dk]
+  float* ks = qs + dk;                 // [dk]
+  __shared__ float part[MTHREADS / 32][MV];
+  __shared__ float red[33];
+  pdl_trigger();
+  pdl_wait();
+  const int e = blockIdx.z, hd = blockIdx.y, sl = blockIdx.x, slices = gridDim.x;
+  const int p0 = rb.pos0[e];
+  const int c0 = sl * MV, nc = min(MV, dv - c0);
+  const int tid = threadIdx.x, col = tid & 31, rg = tid >> 5;
+  float* o = out + ((long long)e * heads + hd) * dv + c0;
+  if (p0 < 0) {
+    if (tid < nc) o[tid] = 0.f;
+    return;
+  }
+  const bool old = p0 > 0;
+  const long long slot = rb.slot[e];
+  float* Sh = Sg + (slot * heads + hd) * (long long)dk * dv + c0;
+  float* Nh = Ng + ((slot * heads + hd) * slices + sl) * (long long)dk;
+  float* Mh = Mg + (slot * heads + hd) * slices + sl;
+  const T* row = proj + (long long)e * ldp;
+  const float m = old ? *Mh : 0.f;
+  const float ig = cap * tanhf((gates[(long long)e * 2 * heads + hd] + to_f(ib[hd])) / cap);
+  const float fg = log_sigmoid(cap * tanhf((gates[(long long)e * 2 * heads + heads + hd] + to_f(fb[hd])) / cap));
+  const float mn = fmaxf(fg + m, ig);
+  const float da = decay_exp(fg + m - mn), db = expf(ig - mn);
+  const float qscale = 1.f / sqrtf((float)dk);
+  float nq = 0.f;
+  for (int d = tid; d < dk; d += MTHREADS) {
+    const float q = to_f(row[q_off + hd * dk + d]) * qscale, k = to_f(row[k_off + hd * dk + d]);
+    qs[d] = q;
+    ks[d] = k;
+    const float nn = da * (old ? Nh[d] : 0.f) + db * k;
+    Nh[d] = nn;
+    nq += nn * q;
+  }
+  nq = block_sum(nq, red);             // also: every thread has read m, and qs / ks are complete
+  if (tid == 0) *Mh = mn;
+  float acc = 0.f;
+  if (col < nc) {
+    const float bv = db * to_f(row[v_off + hd * dv + c0 + col]);
+    constexpr int U = 8;
+    for (int d0 = rg; d0 < dk; d0 += U * (MTHREADS / 32)) {
+      float s[U];
+#pragma unroll
+      for (int j = 0; j < U; ++j) {
+        const int d = d0 + j * (MTHREADS / 32);
+        s[j] = (old && d < dk) ? Sh[(long long)d * dv + col] : 0.f;
+      }
+#pragma unroll
+      for (int j = 0; j < U; ++j) {
+        const int d = d0 + j * (MTHREADS / 32);
+        if (d < dk) {
+          const float v = da * s[j] + bv * ks[d];
+          Sh[(long long)d * dv + col] = v;
+          acc += v * qs[d];
+        }
+      }
+    }
+  }
+  part[rg][col] = acc;
+  __syncthreads();
+  if (tid < nc) {
+    float v = 0.f;
+#pragma unroll
+    for (int j = 0; j < MTHREADS / 32; ++j) v += part[j][tid];
+    o[tid] = v / (fmaxf(fabsf(nq), expf(-mn)) + 1e-6f);
+  }
+}
+
+// ---- bf16, prompt portions: chunks of ML tokens on tensor cores
+// With F the running sum of f inside a chunk, g_s = i_s - F_s and M_t = max(m_prev, max_{s <= t} g_s), the recurrence above
+// unrolls to  m_t = F_t + M_t,
+//   o_t ~ e^(m_prev - M_t) q_t S + sum_{s <= t} e^(g_s - M_t) (q_t . k_s) v_s,   S' = e^(m_prev - M_L) S + sum_s e^(g_s - M_L) k_s v_s^T.
+// n and its products ride along as one more value column that holds ones. q, k, v are bf16 and exact; every fp32 factor (the
+// weights, the state, the scaled values) enters the tensor cores as a bf16 pair hi + lo. S stays in fp32 accumulators.
+constexpr int ML = 64;
+constexpr int MN = MV + 8;              // value columns with the ones column (index MV), padded to 8
+constexpr int MVP = MN * 2;             // row pitch in bytes of [.., MN] bf16 tiles: 80, an odd multiple of 16
+constexpr int MPP = ML * 2 + 16;        // row pitch of the [ML, ML] weight tiles
+
+struct MlstmSmem {
+  int pitch, q, k, v, wv, p, s, gate, total;            // byte offsets; q, k, v are double buffered
+};
+__host__ __device__ inline MlstmSmem mlstm_smem(int dk) {
+  MlstmSmem L;
+  const int kp = (dk + 15) & ~15;
+  L.pitch = kp * 2 + 16;
+  L.q = 0;
+  L.k = L.q + 2 * ML * L.pitch;
+  L.v = L.k + 2 * ML * L.pitch;
+  L.wv = L.v + 2 * ML * MVP;
+  L.p = L.wv + 2 * ML * MVP;
+  L.s = L.p + 2 * ML * MPP;
+  L.gate = L.s + 2 * kp * MVP;
+  L.total = L.gate + 6 * ML * 4;
+  return L;
+}
+
+template <int MT>       // 16-row tiles of S per warp: dk <= 128 * MT
+__global__ void __launch_bounds__(256, 1)
+mlstm_chunk_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int q_off, int k_off, int v_off,
+                   const float* __restrict__ gates, const __nv_bfloat16* __restrict__ ib, const __nv_bfloat16* __restrict__ fb,
+                   float cap, Ragged rb, int heads, int dk, int dv, float* __restrict__ Sg, float* __restrict__ Ng,
+                   float* __restrict__ Mg, float* __restrict__ out) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  const MlstmSmem L = mlstm_smem(dk);
+  const uint32_t sb = smem_u32(smem);
+  float* G = reinterpret_cast<float*>(smem + L.gate);   // g_s
+  float* Mx = G + ML;                                   // M_t
+  float* Ct = Mx + ML;                                  // e^(m_prev - M_t)
+  float* Wt = Ct + ML;                                  // e^(g_s - M_L)
+  float* Em = Wt + ML;                                  // e^(-m_t)
+  float* Den = Em + ML;
+  __shared__ float s_m, s_decay;
+  pdl_trigger();
+  pdl_wait();
+  const int e = blockIdx.z, hd = blockIdx.y, sl = blockIdx.x, slices = gridDim.x;
+  const int p0 = rb.pos0[e], t0 = rb.cu[e], len = rb.cu[e + 1] - t0;
+  if (p0 < 0 || len <= 0) return;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, li = lane >> 3, lr = lane & 7;
+  const int kp = (dk + 15) & ~15, kchunks = kp / 8, mtiles = kp / 16;
+  const int c0 = sl * MV, nc = min(MV, dv - c0);
+  const long long slot = rb.slot[e];
+  float* Sh = Sg + (slot * heads + hd) * (long long)dk * dv + c0;
+  float* Nh = Ng + ((slot * heads + hd) * slices + sl) * (long long)dk;
+  float* Mh = Mg + (slot * heads + hd) * slices + sl;
+  const float bi = to_f(ib[hd]), bf = to_f(fb[hd]);
+  const float qscale = 1.f / sqrtf((float)dk);
+
+  auto load = [&](int ch, int buf) {
+    const int rows = min(ML, len - ch * ML);
+    const __nv_bfloat16* base = proj + (long long)(t0 + ch * ML) * ldp;
+    for (int i = tid; i < ML * kchunks; i += 256) {
+      const int r = i / kchunks, c = i - r * kchunks;
+      const bool ok = r < rows && c * 8 < dk;
+      const long long src = ok ? (long long)r * ldp + hd * dk + c * 8 : 0;
+      const uint32_t d = (buf * ML + r) * L.pitch + c * 16;
+      cp_async16(sb + L.q + d, base + q_off + src, ok ? 16 : 0);
+      cp_async16(sb + L.k + d, base + k_off + src, ok ? 16 : 0);
+    }
+    for (int i = tid; i < ML * (MV / 8); i += 256) {
+      const int r = i / (MV / 8), c = i - r * (MV / 8);
+      const bool ok = r < rows && c * 8 < nc;
+      cp_async16(sb + L.v + (buf * ML + r) * MVP + c * 16, base + v_off + (ok ? (long long)r * ldp + hd * dv + c0 + c * 8 : 0),
+                 ok ? 16 : 0);
+    }
+    cp_async_commit();
+  };
+
+  // the ones column (and its padding) of both value buffers
+  for (int i = tid; i < 2 * ML; i += 256) {
+    uint4 u = make_uint4(0x3f80u, 0u, 0u, 0u);          // bf16 1.0 in the first of 8 columns
+    *reinterpret_cast<uint4*>(smem + L.v + i * MVP + MV * 2) = u;
+  }
+  load(0, 0);
+
+  // state -> accumulators: warp w owns the 16-row tiles w, w + 8, ...
+  float S[MT][5][4];
+#pragma unroll
+  for (int a = 0; a < MT; ++a)
+#pragma unroll
+    for (int j = 0; j < 5; ++j)
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        const int d = (warp + a * 8) * 16 + (lane >> 2) + (q >> 1) * 8, c = j * 8 + 2 * (lane & 3) + (q & 1);
+        float v = 0.f;
+        if (p0 > 0 && d < dk) {
+          if (c < nc) v = Sh[(long long)d * dv + c];
+          else if (c == MV) v = Nh[d];
+        }
+        S[a][j][q] = v;
+      }
+  auto store_s = [&]() {                // hi + lo of the state, the B operand of Q S
+#pragma unroll
+    for (int a = 0; a < MT; ++a) {
+      if (warp + a * 8 >= mtiles) continue;
+#pragma unroll
+      for (int j = 0; j < 5; ++j)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          const int d = (warp + a * 8) * 16 + (lane >> 2) + h * 8;
+          const uint32_t off = d * MVP + (j * 8 + 2 * (lane & 3)) * 2;
+          __nv_bfloat16 h0, l0, h1, l1;
+          split_bf16(S[a][j][2 * h], h0, l0);
+          split_bf16(S[a][j][2 * h + 1], h1, l1);
+          *reinterpret_cast<__nv_bfloat162*>(smem + L.s + off) = __halves2bfloat162(h0, h1);
+          *reinterpret_cast<__nv_bfloat162*>(smem + L.s + kp * MVP + off) = __halves2bfloat162(l0, l1);
+        }
+    }
+  };
+  store_s();
+  float m_prev = p0 > 0 ? *Mh : 0.f;
+  const int n_ch = (len + ML - 1) / ML;
+  const int wm = (warp & 3) * 16, wn = warp >> 2;       // 16 tokens; half of the keys (P) or of the value columns (O)
+  for (int ch = 0; ch < n_ch; ++ch) {
+    const int buf = ch & 1, rows = min(ML, len - ch * ML);
+    cp_async_wait<0>();
+    __syncthreads();                    // the tiles are in; the other buffer and S of the last chunk are settled
+    if (ch + 1 < n_ch) load(ch + 1, buf ^ 1);
+    const uint32_t qb = sb + L.q + buf * ML * L.pitch, kb = sb + L.k + buf * ML * L.pitch, vb = sb + L.v + buf * ML * MVP;
+    if (warp == 0) {
+      // gates of the chunk, two tokens per lane
+      float f[2], ii[2];
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        const int t = 2 * lane + j;
+        f[j] = 0.f;
+        ii[j] = -INFINITY;
+        if (t < rows) {
+          const float* gr = gates + (long long)(t0 + ch * ML + t) * 2 * heads + hd;
+          ii[j] = cap * tanhf((gr[0] + bi) / cap);
+          f[j] = log_sigmoid(cap * tanhf((gr[heads] + bf) / cap));
+        }
+      }
+      float run = f[0] + f[1];
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const float x = __shfl_up_sync(0xffffffffu, run, o);
+        if (lane >= o) run += x;
+      }
+      const float F1 = run, F0 = run - f[1];
+      const float g0 = ii[0] - F0, g1 = ii[1] - F1;
+      float mx = fmaxf(g0, g1);
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const float x = __shfl_up_sync(0xffffffffu, mx, o);
+        if (lane >= o) mx = fmaxf(mx, x);
+      }
+      float before = __shfl_up_sync(0xffffffffu, mx, 1);
+      if (lane == 0) before = -INFINITY;
+      const float M0 = fmaxf(m_prev, fmaxf(before, g0)), M1 = fmaxf(m_prev, mx);
+      const float ML_ = __shfl_sync(0xffffffffu, M1, 31), FL = __shfl_sync(0xffffffffu, F1, 31);
+      const int t = 2 * lane;
+      G[t] = g0; G[t + 1] = g1;
+      Mx[t] = M0; Mx[t + 1] = M1;
+      Ct[t] = expf(m_prev - M0); Ct[t + 1] = expf(m_prev - M1);
+      Wt[t] = expf(g0 - ML_); Wt[t + 1] = expf(g1 - ML_);
+      Em[t] = expf(-(F0 + M0)); Em[t + 1] = expf(-(F1 + M1));
+      if (lane == 0) { s_m = FL + ML_; s_decay = expf(m_prev - ML_); }
+    }
+    // P = Q K^T (this warp: 16 tokens x 32 keys; key tiles past the diagonal are skipped)
+    float P[4][4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) P[j][0] = P[j][1] = P[j][2] = P[j][3] = 0.f;
+    const int kn = wn * 32;
+    if (kn <= wm + 15) {
+      for (int ks = 0; ks < mtiles; ++ks) {
+        uint32_t a[4], b[4];
+        ldsm_x4(a, qb + (wm + (li & 1) * 8 + lr) * L.pitch + (ks * 2 + (li >> 1)) * 16);
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          ldsm_x4(b, kb + (kn + h * 16 + (li >> 1) * 8 + lr) * L.pitch + (ks * 2 + (li & 1)) * 16);
+          mma_16816(P[2 * h], a, b[0], b[1]);
+          mma_16816(P[2 * h + 1], a, b[2], b[3]);
+        }
+      }
+    }
+    __syncthreads();                    // gates are in shared memory
+    m_prev = s_m;
+    const float decay = s_decay;
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int t = wm + (lane >> 2) + h * 8, s = kn + j * 8 + 2 * (lane & 3);
+        const float M = Mx[t];
+        const float w0 = s <= t ? P[j][2 * h] * qscale * expf(G[s] - M) : 0.f;
+        const float w1 = s + 1 <= t ? P[j][2 * h + 1] * qscale * expf(G[s + 1] - M) : 0.f;
+        __nv_bfloat16 h0, l0, h1, l1;
+        split_bf16(w0, h0, l0);
+        split_bf16(w1, h1, l1);
+        *reinterpret_cast<__nv_bfloat162*>(smem + L.p + t * MPP + s * 2) = __halves2bfloat162(h0, h1);
+        *reinterpret_cast<__nv_bfloat162*>(smem + L.p + ML * MPP + t * MPP + s * 2) = __halves2bfloat162(l0, l1);
+      }
+    for (int i = tid; i < ML * (MN / 2); i += 256) {    // w_s v_s, hi and lo
+      const int r = i / (MN / 2), c = (i - r * (MN / 2)) * 2;
+      const uint32_t v2 = *reinterpret_cast<const uint32_t*>(smem + L.v + (buf * ML + r) * MVP + c * 2);
+      const float w = Wt[r];
+      __nv_bfloat16 h0, l0, h1, l1;
+      split_bf16(w * bf16_lo(v2), h0, l0);
+      split_bf16(w * bf16_hi(v2), h1, l1);
+      *reinterpret_cast<__nv_bfloat162*>(smem + L.wv + r * MVP + c * 2) = __halves2bfloat162(h0, h1);
+      *reinterpret_cast<__nv_bfloat162*>(smem + L.wv + ML * MVP + r * MVP + c * 2) = __halves2bfloat162(l0, l1);
+    }
+    __syncthreads();
+    // O = diag(c) Q S + P V; column tiles 0..2 (first half) or 3, 4 (second half; tile 4 carries the ones column)
+    float O[3][4];
+#pragma unroll
+    for (int j = 0; j < 3; ++j) O[j][0] = O[j][1] = O[j][2] = O[j][3] = 0.f;
+    const uint32_t row16 = (li & 1) * 8 + lr;           // row inside a 16-row B tile
+    for (int ks = 0; ks < mtiles; ++ks) {
+      uint32_t a[4], b[4], b2[2];
+      ldsm_x4(a, qb + (wm + (li & 1) * 8 + lr) * L.pitch + (ks * 2 + (li >> 1)) * 16);
+#pragma unroll
+      for (int part = 0; part < 2; ++part) {
+        const uint32_t base = sb + L.s + part * kp * MVP + (ks * 16 + row16) * MVP;
+        ldsm_x4_t(b, base + (wn * 3 + (li >> 1)) * 16);
+        mma_16816(O[0], a, b[0], b[1]);
+        mma_16816(O[1], a, b[2], b[3]);
+        if (wn == 0) {
+          ldsm_x2_t(b2, base + 2 * 16);
+          mma_16816(O[2], a, b2[0], b2[1]);
+        }
+      }
+    }
+    {
+      const float ca = Ct[wm + (lane >> 2)] * qscale, cb = Ct[wm + (lane >> 2) + 8] * qscale;
+#pragma unroll
+      for (int j = 0; j < 3; ++j) { O[j][0] *= ca; O[j][1] *= ca; O[j][2] *= cb; O[j][3] *= cb; }
+    }
+#pragma unroll
+    for (int ks = 0; ks < ML / 16; ++ks) {
+      if (ks * 16 > wm + 15) continue;                  // weights past the diagonal are zero
+      uint32_t b[4], b2[2];
+      const uint32_t base = vb + (ks * 16 + row16) * MVP;
+      ldsm_x4_t(b, base + (wn * 3 + (li >> 1)) * 16);
+      if (wn == 0) ldsm_x2_t(b2, base + 2 * 16);
+#pragma unroll
+      for (int part = 0; part < 2; ++part) {
+        uint32_t a[4];
+        ldsm_x4(a, sb + L.p + part * ML * MPP + (wm + (li & 1) * 8 + lr) * MPP + (ks * 2 + (li >> 1)) * 16);
+        mma_16816(O[0], a, b[0], b[1]);
+        mma_16816(O[1], a, b[2], b[3]);
+        if (wn == 0) mma_16816(O[2], a, b2[0], b2[1]);
+      }
+    }
+    if (wn == 1 && (lane & 3) == 0) {                   // column MV: n . q
+      const int ta = wm + (lane >> 2), tb_ = ta + 8;
+      Den[ta] = 1.f / (fmaxf(fabsf(O[1][0]), Em[ta]) + 1e-6f);
+      Den[tb_] = 1.f / (fmaxf(fabsf(O[1][2]), Em[tb_]) + 1e-6f);
+    }
+    // S = decay S + K^T (w V)
+#pragma unroll
+    for (int a = 0; a < MT; ++a) {
+      const int mt = warp + a * 8;
+      if (mt >= mtiles) continue;
+#pragma unroll
+      for (int j = 0; j < 5; ++j)
+#pragma unroll
+        for (int q = 0; q < 4; ++q) S[a][j][q] *= decay;
+#pragma unroll
+      for (int ks = 0; ks < ML / 16; ++ks) {
+        uint32_t ak[4];
+        ldsm_x4_t(ak, kb + (ks * 16 + (li >> 1) * 8 + lr) * L.pitch + (mt * 2 + (li & 1)) * 16);
+#pragma unroll
+        for (int part = 0; part < 2; ++part) {
+          uint32_t b[4], b2[2];
+          const uint32_t base = sb + L.wv + part * ML * MVP + (ks * 16 + row16) * MVP;
+          ldsm_x4_t(b, base + (li >> 1) * 16);
+          mma_16816(S[a][0], ak, b[0], b[1]);
+          mma_16816(S[a][1], ak, b[2], b[3]);
+          ldsm_x4_t(b, base + (2 + (li >> 1)) * 16);
+          mma_16816(S[a][2], ak, b[0], b[1]);
+          mma_16816(S[a][3], ak, b[2], b[3]);
+          ldsm_x2_t(b2, base + 4 * 16);
+          mma_16816(S[a][4], ak, b2[0], b2[1]);
+        }
+      }
+    }
+    __syncthreads();                    // Den is complete; nobody reads the old S any more
+    store_s();
+#pragma unroll
+    for (int j = 0; j < 3; ++j) {
+      const int tile = wn * 3 + j;
+      if (tile > 3) continue;
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int t = wm + (lane >> 2) + h * 8, c = tile * 8 + 2 * (lane & 3);
+        if (t < rows && c < nc) {
+          const float dn = Den[t];
+          float* o = out + ((long long)(t0 + ch * ML + t) * heads + hd) * dv + c0 + c;
+          o[0] = O[j][2 * h] * dn;
+          if (c + 1 < nc) o[1] = O[j][2 * h + 1] * dn;
+        }
+      }
+    }
+  }
+#pragma unroll
+  for (int a = 0; a < MT; ++a)
+#pragma unroll
+    for (int j = 0; j < 5; ++j)
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        const int d = (warp + a * 8) * 16 + (lane >> 2) + (q >> 1) * 8, c = j * 8 + 2 * (lane & 3) + (q & 1);
+        if (d < dk) {
+          if (c < nc) Sh[(long long)d * dv + c] = S[a][j][q];
+          else if (c == MV) Nh[d] = S[a][j][q];
+        }
+      }
+  if (tid == 0) *Mh = m_prev;
+}
+
 }  // namespace
 
 #define RAGGED Ragged rb{cu, slot, pos0, ent, E, n}
 
 // x and y are columns x_off.. and y_off.. of proj [n, ldp]. u / A / B: workspaces [n, W] (T, fp32, fp32).
-// state fp32 [slots, W], ring fp32 [slots, K, W]; out T [n, W].
+// state fp32 [slots, W], ring fp32 [slots, K, W]; out T [n, W]. `one`: every entry is one token.
+// bf16 portions also take tile lists (LT tokens a tile): tile_t0 / tile_ent [tiles], first_tile [E], and workspaces
+// LH / LP fp32 [tiles, W]; with tiles == 0 the plain kernels run.
 TB_API int tb_rglru(int dtype, const void* proj, long long ldp, int x_off, int y_off, const void* conv_w, const void* conv_b,
                     const void* ra, const void* rab, const void* ri, const void* rib, const void* lam, const int* cu,
                     const int* slot, const int* pos0, const int* ent, int E, int n, int W, int K, int blocks, float* state,
-                    float* ring, void* u, float* A, float* B, void* out, cudaStream_t stream) {
+                    float* ring, void* u, float* A, float* B, void* out, int one, const int* tile_t0, const int* tile_ent,
+                    const int* first_tile, int tiles, float* LH, float* LP, cudaStream_t stream) {
   if (n <= 0 || E <= 0) return 0;
-  if (blocks <= 0 || W % blocks || K < 1 || n > 65535 * GT) return -2;
-  const int bs = W / blocks;
+  if (blocks <= 0 || W % blocks || K < 1 || E > 65535) return -2;
+  const int bs = W / blocks, kp = (bs + 15) & ~15, pitch = kp * 2 + 16;
   RAGGED;
+  typedef __nv_bfloat16 bf;
+  if (dtype == 0 && bs % 8 == 0 && x_off % 4 == 0 && y_off % 4 == 0 && ldp % 4 == 0) {
+    if (one) {
+      const size_t smem = (size_t)(16 + 2 * DC) * pitch;
+      if (smem <= 200 * 1024) {
+        static DeviceOnce once;
+        if (once.first() && cudaFuncSetAttribute(rglru_step_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess)
+          return -5;
+        const dim3 grid(blocks * ((bs + DC - 1) / DC), (E + 15) / 16);
+        return launch_pdl(rglru_step_kernel, grid, dim3(128), smem, stream, (const bf*)proj, ldp, x_off, y_off, (const bf*)conv_w,
+                          (const bf*)conv_b, (const bf*)ra, (const bf*)rab, (const bf*)ri, (const bf*)rib, (const bf*)lam, rb, W,
+                          bs, K, state, ring, (bf*)out) == cudaSuccess ? 0 : -5;
+      }
+    } else if (tiles > 0) {
+      const size_t smem = (size_t)(LT + 2 * LC) * pitch + 2 * LT * (LC + 1) * 4;
+      if (smem <= 220 * 1024) {
+        static DeviceOnce once;
+        if (once.first() && cudaFuncSetAttribute(rglru_tile_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024) != cudaSuccess)
+          return -5;
+        Tiles tl{tile_t0, tile_ent, tiles};
+        const long long want = ((long long)n * (W / 4) + 255) / 256;
+        const dim3 flat((unsigned)(want < 148 * 16 ? want : 148 * 16));
+        const dim3 gtile(blocks * ((bs + LC - 1) / LC), (tiles + LTPC - 1) / LTPC);
+        if (gtile.y > 65535) return -2;
+        cudaError_t err = launch_pdl(rglru_conv4_kernel, flat, dim3(256), 0, stream, (const bf*)proj, ldp, x_off, (const bf*)conv_w,
+                                     (const bf*)conv_b, (const float*)ring, rb, W, K, (bf*)u);
+        if (err == cudaSuccess)
+          err = launch_pdl(rglru_tile_kernel, gtile, dim3(256), smem, stream, (const bf*)u, (const bf*)ra, (const bf*)rab,
+                           (const bf*)ri, (const bf*)rib, (const bf*)lam, rb, tl, W, bs, A, B, LH, LP);
+        if (err == cudaSuccess)
+          err = launch_pdl(rglru_chain_kernel, dim3((W + 63) / 64, E), dim3(64), 0, stream, LH, (const float*)LP, (const bf*)proj,
+                           ldp, x_off, rb, first_tile, W, K, state, ring);
+        if (err == cudaSuccess)
+          err = launch_pdl(rglru_out_kernel, flat, dim3(256), 0, stream, (const float*)A, (const float*)B, (const float*)LH,
+                           (const bf*)proj, ldp, y_off, rb, first_tile, W, (bf*)out);
+        return err == cudaSuccess ? 0 : -5;
+      }
+    }
+  }
   const dim3 gconv((W + 127) / 128, n), ggate((bs + GC - 1) / GC, blocks, (n + GT - 1) / GT), gscan((W + 63) / 64, E);
-  if (n > 65535 || ggate.z > 65535 || E > 65535) return -2;
+  if (n > 65535 || blocks > 65535) return -2;
   const size_t smem = (size_t)GT * bs * 4;
+  if (smem > 200 * 1024) return -2;
 #define RUN(T)                                                                                                              \
   {                                                                                                                         \
     static DeviceOnce once;                                                                                                 \
-    if (smem > 200 * 1024) return -2;                                                                                       \
     if (once.first() && cudaFuncSetAttribute(rglru_gates_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize,            \
                                              200 * 1024) != cudaSuccess) return -5;                                         \
     cudaError_t err = launch_pdl(rglru_conv_kernel<T>, gconv, dim3(128), 0, stream, (const T*)proj, ldp, x_off,             \
@@ -245,25 +981,45 @@ TB_API int tb_mlstm_slices(int dv) { return (dv + MV - 1) / MV; }
 
 // q, k, v: columns of proj [n, ldp]; gates fp32 [n, 2 * heads] = (W_i h, W_f h) without bias.
 // S fp32 [slots, heads, dk, dv], N fp32 [slots, heads, slices, dk], M fp32 [slots, heads, slices]; out fp32 [n, heads, dv].
-TB_API int tb_mlstm_seq(int dtype, const void* proj, long long ldp, int q_off, int k_off, int v_off, const float* gates,
-                        const void* ib, const void* fb, float cap, const int* cu, const int* slot, const int* pos0,
-                        const int* ent, int E, int n, int heads, int dk, int dv, float* S, float* N, float* M, float* out,
-                        cudaStream_t stream) {
+// `one`: every entry is one token. `chunked`: bf16 portions take the tensor-core form where the sizes allow.
+TB_API int tb_mlstm(int dtype, const void* proj, long long ldp, int q_off, int k_off, int v_off, const float* gates,
+                    const void* ib, const void* fb, float cap, const int* cu, const int* slot, const int* pos0,
+                    const int* ent, int E, int n, int heads, int dk, int dv, float* S, float* N, float* M, float* out, int one,
+                    int chunked, cudaStream_t stream) {
   if (n <= 0 || E <= 0) return 0;
   if (E > 65535 || heads > 65535) return -2;
   RAGGED;
+  const dim3 grid(tb_mlstm_slices(dv), heads, E);
+#define ARGS(T) (const T*)proj, ldp, q_off, k_off, v_off, gates, (const T*)ib, (const T*)fb, cap, rb, heads, dk, dv, S, N, M, out
+  if (one) {
+    const size_t smem = (size_t)2 * dk * 4;
+    if (smem > 48 * 1024) return -2;
+    cudaError_t err = dtype == 0 ? launch_pdl(mlstm_step_kernel<__nv_bfloat16>, grid, dim3(MTHREADS), smem, stream, ARGS(__nv_bfloat16))
+                                 : launch_pdl(mlstm_step_kernel<float>, grid, dim3(MTHREADS), smem, stream, ARGS(float));
+    return err == cudaSuccess ? 0 : -5;
+  }
+  if (dtype == 0 && chunked && dk <= 256 && dk % 8 == 0 && dv % 8 == 0 && q_off % 8 == 0 && k_off % 8 == 0 && v_off % 8 == 0 &&
+      ldp % 8 == 0 && (reinterpret_cast<uintptr_t>(proj) & 15) == 0) {
+    const size_t smem = mlstm_smem(dk).total;
+    static DeviceOnce once;
+    if (once.first() &&
+        (cudaFuncSetAttribute(mlstm_chunk_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 225 * 1024) != cudaSuccess ||
+         cudaFuncSetAttribute(mlstm_chunk_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 225 * 1024) != cudaSuccess))
+      return -5;
+    cudaError_t err = dk <= 128 ? launch_pdl(mlstm_chunk_kernel<1>, grid, dim3(256), smem, stream, ARGS(__nv_bfloat16))
+                                : launch_pdl(mlstm_chunk_kernel<2>, grid, dim3(256), smem, stream, ARGS(__nv_bfloat16));
+    return err == cudaSuccess ? 0 : -5;
+  }
   const size_t smem = ((size_t)dk * (MV + 3) + MV * 9) * 4;
   if (smem > 200 * 1024) return -2;
-  const dim3 grid(tb_mlstm_slices(dv), heads, E);
 #define RUN(T)                                                                                                              \
   {                                                                                                                         \
     static DeviceOnce once;                                                                                                 \
     if (once.first() && cudaFuncSetAttribute(mlstm_seq_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize,              \
                                              200 * 1024) != cudaSuccess) return -5;                                         \
-    cudaError_t err = launch_pdl(mlstm_seq_kernel<T>, grid, dim3(MTHREADS), smem, stream, (const T*)proj, ldp, q_off, k_off, \
-                                 v_off, gates, (const T*)ib, (const T*)fb, cap, rb, heads, dk, dv, S, N, M, out);            \
-    return err == cudaSuccess ? 0 : -5;                                                                                     \
+    return launch_pdl(mlstm_seq_kernel<T>, grid, dim3(MTHREADS), smem, stream, ARGS(T)) == cudaSuccess ? 0 : -5;            \
   }
   if (dtype == 0) RUN(__nv_bfloat16) else RUN(float)
 #undef RUN
+#undef ARGS
 }

@@ -94,7 +94,7 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ kp, const T* _
       const T* k = kp + (row * G + g) * dq;
       float dot = 0.f;
       for (int d = 0; d < dq; ++d) dot += qs[d] * to_f(k[d]);
-      s = dot + bias[(long long)min(i - j, far) * H + h];
+      s = dot + bias[(long long)h * (far + 1) + min(i - j, far)];
     }
     const float mn = fmaxf(m, warp_max(s));
     const float p = expf(s - mn), c = expf(m - mn);
@@ -143,7 +143,7 @@ TB_API int tb_qk_norm_write(int dtype, const void* proj, long long ldp, int q_of
 #undef RUN
 }
 
-// bias fp32 [far + 1, H]: what is added to the score of a key at distance min(i - j, far). window <= 0: no window.
+// bias fp32 [H, far + 1]: what is added to the score of a key at distance min(i - j, far). window <= 0: no window.
 TB_API int tb_window_attn(int dtype, const void* q, const void* kp, const void* vp, const int* cu, const int* slot,
                           const int* pos0, const int* ent, int E, int n, const int* table, int max_pages, int page_size, int H,
                           int G, int dq, int dv, float scale, const float* bias, int far, int window, int keep, void* out,

@@ -151,9 +151,9 @@ class BiasedWindowAttention(nn.Module):
         self.rel = _param(spec.buckets, H, dtype=dtype, device=device)
 
     def bias_table(self) -> torch.Tensor:
-        """fp32 [far + 1, heads]: what is added to the score of a key at distance min(i - j, far)."""
+        """fp32 [heads, far + 1]: what is added to the score of a key at distance min(i - j, far)."""
         idx = distance_buckets(self.rel.shape[0], self.spec.bias_max, self.rel.device)
-        return self.rel.detach().float()[idx].contiguous()
+        return self.rel.detach().float()[idx].t().contiguous()
 
     def init_special(self) -> None:
         pass

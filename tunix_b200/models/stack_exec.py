@@ -67,6 +67,7 @@ class StackExecutor:
         self.runs = self.cfg.runs()
         self.dtype = model.embed_tokens.dtype
         self.pk: Callable = lambda i, name: None        # packed decode weights, set by the engine
+        self.plain = False          # bf16 through the simple kernels of the 32-bit path (a cross-check, slow)
         self._one = None
         self.w: list = []
         self.refresh()
@@ -116,7 +117,7 @@ class StackExecutor:
     def _rglru(self, i, m: RGLRUMixer, h, rb: RaggedBatch, pool, r):
         d = self.w[i]
         proj = linear(h, d["proj"], d["proj_bias"], packed=self.pk(i, "proj") if rb.decode else None)
-        o = SK.rglru(proj, m.spec.width, 0, m, rb, pool.state[r])
+        o = SK.rglru(proj, m.spec.width, 0, m, rb, pool.state[r], self.plain)
         return (linear(o, m.o_proj.weight), None, None, None)
 
     def _parallel(self, i, m: ParallelMixer, h, rb: RaggedBatch, pool, r):
@@ -131,11 +132,27 @@ class StackExecutor:
             cols += width
         q = SK.qk_norm_write(proj, off[0], off[1], off[2], lf.q_norm.weight, lf.k_norm.weight, lf.eps, rb, pool.table,
                              pool.page_size, pool.k[r], pool.v[r], a.heads * a.dim)
-        att = SK.window_attn(q, pool.k[r], pool.v[r], rb, pool.table, pool.page_size, a, d["bias"])
+        att = self._attend(q, a, d["bias"], rb, pool, r)
         o = SK.mlstm(proj, off[4], off[5], off[6], gates, rt.i_proj.bias, rt.f_proj.bias, s.gate_cap, rb, s.heads, s.dim, s.vdim,
-                     pool.state[r])
+                     pool.state[r], self.plain)
         a1, a2 = SK.gate_outputs(att, o, proj, off[3], off[7], rt.norm.weight, rt.eps, s.heads, s.vdim)
         return (linear(a1, lf.o_proj.weight), linear(a2, rt.o_proj.weight), m.left_norm.weight, m.right_norm.weight)
+
+    def _attend(self, q, a, bias, rb: RaggedBatch, pool, r):
+        """Tensor-core kernels where the heads fit them (the framework's paged decode and flash attention, extended by the
+        bias and the kept tokens); otherwise, and in 32-bit, the general kernel."""
+        fits = q.dtype == torch.bfloat16 and a.dim == a.vdim and a.dim in (64, 128, 256) and not self.plain
+        kw = dict(scale=a.scale, window=a.window, keep_first=a.keep_first, bias=bias)
+        if fits and rb.decode and a.heads // a.kv_heads <= 16:
+            max_ctx = pool.table.shape[1] * pool.page_size
+            split = K.decode_split_tokens(rb.n, a.kv_heads, min(max_ctx, a.window + a.keep_first + 128) if a.window else max_ctx)
+            return K.paged_decode(q.view(rb.n, a.heads, a.dim), pool.k[r], pool.v[r], pool.table, rb.slot, self._lens,
+                                  num_kv_heads=a.kv_heads, page_size=pool.page_size, max_ctx=max_ctx, split_tokens=split,
+                                  **kw).view(rb.n, -1)
+        if fits and not rb.decode and pool.page_size % 64 == 0:
+            return K.attn_fwd_paged(q, pool.k[r], pool.v[r], rb, pool.table, pool.page_size, num_heads=a.heads,
+                                    num_kv_heads=a.kv_heads, head_dim=a.dim, **kw)
+        return SK.window_attn(q, pool.k[r], pool.v[r], rb, pool.table, pool.page_size, a, bias)
 
     def _mlp(self, i, mlp, h, rb: RaggedBatch):
         gu_w = self.w[i]["gu"]
@@ -163,6 +180,8 @@ class StackExecutor:
             _, w_out, mix = self._hc(hc)
             return dict(y=y, y2=y2, wy=wy, wy2=wy2, mix=mix, w_out=w_out)
 
+        if rb.decode:
+            self._lens = rb.pos0 + 1                                   # keys each query sees (0: idle slot)
         ended = False                                                  # the pending sublayer ends a layer pass
         def step(w_in, norm_w):
             nonlocal ended

@@ -8,6 +8,8 @@ from typing import Optional, Sequence
 
 import torch
 
+TILE = 64       # tokens per tile of the tiled recurrences (csrc/recurrent.cu: LT)
+
 
 @dataclass
 class RaggedBatch:
@@ -17,6 +19,7 @@ class RaggedBatch:
     pos0: torch.Tensor              # int32 [E] position of its first token (< 0: idle slot)
     ent: torch.Tensor               # int32 [n] entry of every token
     lens: Optional[Sequence[int]]   # host copy of the entries' lengths (None: every entry is one token)
+    _tiles: Optional[dict] = None
 
     @property
     def n(self) -> int:
@@ -53,6 +56,24 @@ class RaggedBatch:
         B = tokens.shape[0]
         ar = torch.arange(B + 1, dtype=torch.int32, device=tokens.device)
         return cls(tokens, ar, slots, positions, ar[:B], None)
+
+    def tiles(self, size: int = TILE) -> tuple:
+        """(first token, entry) of every tile of at most `size` tokens of one entry, the first tile of every entry, and the
+        number of tiles. Built once per batch and size: every layer uses the same lists."""
+        if self._tiles is None:
+            self._tiles = {}
+        if size not in self._tiles:
+            t0, ent, first, at = [], [], [], 0
+            for e, L in enumerate(self.lens if self.lens is not None else [1] * self.entries):
+                first.append(len(t0))
+                for o in range(0, L, size):
+                    t0.append(at + o)
+                    ent.append(e)
+                at += L
+            k = len(t0)
+            dev = torch.tensor(t0 + ent + first, dtype=torch.int32).to(self.tokens.device)
+            self._tiles[size] = (dev[:k], dev[k:2 * k], dev[2 * k:], k)
+        return self._tiles[size]
 
     def args(self) -> tuple:
         return (self.cu.data_ptr(), self.slot.data_ptr(), self.pos0.data_ptr(), self.ent.data_ptr(), self.entries, self.n)

@@ -16,9 +16,10 @@ _lib.register_cuda_sigs({
     "tb_stream_step": [_I, _P, _I, _I, _I, _F, _P, _P, _P, _P, _P, _P, _P, _P, _I, _P, _P, _P, _P, _P],
     "tb_silu_mul": [_I, _P, _P, _LL, _I, _P],
     "tb_gate_outputs": [_I, _P, _P, _P, _LL, _I, _I, _P, _F, _I, _I, _I, _I, _P, _P, _P],
-    "tb_rglru": [_I, _P, _LL, _I, _I, _P, _P, _P, _P, _P, _P, _P, *_RB, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P],
+    "tb_rglru": [_I, _P, _LL, _I, _I, _P, _P, _P, _P, _P, _P, _P, *_RB, _I, _I, _I, _P, _P, _P, _P, _P, _P, _I, _P, _P,
+                 _P, _I, _P, _P, _P],
     "tb_mlstm_slices": [_I],
-    "tb_mlstm_seq": [_I, _P, _LL, _I, _I, _I, _P, _P, _P, _F, *_RB, _I, _I, _I, _P, _P, _P, _P, _P],
+    "tb_mlstm": [_I, _P, _LL, _I, _I, _I, _P, _P, _P, _F, *_RB, _I, _I, _I, _P, _P, _P, _P, _I, _I, _P],
     "tb_qk_norm_write": [_I, _P, _LL, _I, _I, _I, _P, _P, _F, *_RB, _P, _I, _I, _I, _I, _I, _P, _P, _P, _P],
     "tb_window_attn": [_I, _P, _P, _P, *_RB, _P, _I, _I, _I, _I, _I, _I, _F, _P, _I, _I, _I, _P, _P],
 })
@@ -72,36 +73,41 @@ def gate_outputs(attn, o, proj, g1_off: int, g2_off: int, norm_w, eps: float, he
     return a1, a2
 
 
-def rglru(proj, x_off: int, y_off: int, m, rb: RaggedBatch, state: dict) -> torch.Tensor:
-    """Convolution, gates, recurrence and output gate of `models.mixers.RGLRUMixer` m on its projections; [n, W]."""
+def rglru(proj, x_off: int, y_off: int, m, rb: RaggedBatch, state: dict, plain: bool = False) -> torch.Tensor:
+    """Convolution, gates, recurrence and output gate of `models.mixers.RGLRUMixer` m on its projections; [n, W].
+    `plain`: the simple kernels of the 32-bit path, also for bf16."""
     n, sp = proj.shape[0], m.spec
     W = sp.width
     dev = proj.device
-    u = torch.empty((n, W), dtype=proj.dtype, device=dev)
-    A = torch.empty((n, W), dtype=torch.float32, device=dev)
-    Bv = torch.empty_like(A)
-    out = torch.empty_like(u)
+    one = rb.decode and not plain and proj.dtype == torch.bfloat16
+    tiles = (None, None, None, 0) if plain or one or proj.dtype != torch.bfloat16 else rb.tiles()
+    out = torch.empty((n, W), dtype=proj.dtype, device=dev)
+    u = torch.empty_like(out)
+    ws = torch.empty((2 * n + 2 * tiles[3], W), dtype=torch.float32, device=dev)
+    A, Bv, LH, LP = ws[:n], ws[n:2 * n], ws[2 * n:2 * n + tiles[3]], ws[2 * n + tiles[3]:]
     rc = _lib.cuda().tb_rglru(_dt(proj), proj.data_ptr(), proj.stride(0), x_off, y_off, m.conv_weight.data_ptr(),
                               m.conv_bias.data_ptr(), m.ra_weight.data_ptr(), m.ra_bias.data_ptr(), m.ri_weight.data_ptr(),
                               m.ri_bias.data_ptr(), m.lam.data_ptr(), *rb.args(), W, sp.conv, sp.blocks, state["s"].data_ptr(),
-                              state["ring"].data_ptr(), u.data_ptr(), A.data_ptr(), Bv.data_ptr(), out.data_ptr(),
+                              state["ring"].data_ptr(), u.data_ptr(), A.data_ptr(), Bv.data_ptr(), out.data_ptr(), int(one),
+                              _lib.ptr(tiles[0]), _lib.ptr(tiles[1]), _lib.ptr(tiles[2]), tiles[3], LH.data_ptr(), LP.data_ptr(),
                               _lib.stream_ptr())
     _lib.check(rc, "tb_rglru")
-    _count(3)
+    _count(1 if one else 4)
     return out
 
 
 def mlstm(proj, q_off: int, k_off: int, v_off: int, gates, i_bias, f_bias, cap: float, rb: RaggedBatch, heads: int, dk: int,
-          dv: int, state: dict) -> torch.Tensor:
-    """Matrix memory over a ragged batch; gates fp32 [n, 2 heads]. Returns o fp32 [n, heads, dv]."""
+          dv: int, state: dict, plain: bool = False) -> torch.Tensor:
+    """Matrix memory over a ragged batch; gates fp32 [n, 2 heads]. Returns o fp32 [n, heads, dv]. `plain`: the token by
+    token kernel of the 32-bit path, also for bf16."""
     n = proj.shape[0]
     assert gates.dtype == torch.float32 and gates.is_contiguous() and gates.shape == (n, 2 * heads)
     out = torch.empty((n, heads, dv), dtype=torch.float32, device=proj.device)
-    rc = _lib.cuda().tb_mlstm_seq(_dt(proj), proj.data_ptr(), proj.stride(0), q_off, k_off, v_off, gates.data_ptr(),
-                                  i_bias.data_ptr(), f_bias.data_ptr(), float(cap), *rb.args(), heads, dk, dv,
-                                  state["S"].data_ptr(), state["n"].data_ptr(), state["m"].data_ptr(), out.data_ptr(),
-                                  _lib.stream_ptr())
-    _lib.check(rc, "tb_mlstm_seq")
+    rc = _lib.cuda().tb_mlstm(_dt(proj), proj.data_ptr(), proj.stride(0), q_off, k_off, v_off, gates.data_ptr(),
+                              i_bias.data_ptr(), f_bias.data_ptr(), float(cap), *rb.args(), heads, dk, dv,
+                              state["S"].data_ptr(), state["n"].data_ptr(), state["m"].data_ptr(), out.data_ptr(),
+                              int(rb.decode and not plain), int(not plain), _lib.stream_ptr())
+    _lib.check(rc, "tb_mlstm")
     _count()
     return out
 
@@ -121,12 +127,12 @@ def qk_norm_write(proj, q_off: int, k_off: int, v_off: int, q_w, k_w, eps: float
 
 
 def window_attn(q, k_pool, v_pool, rb: RaggedBatch, table, page_size: int, sp, bias) -> torch.Tensor:
-    """`sp`: models.mixers.WindowAttentionSpec; bias fp32 [far + 1, heads]. Returns [n, heads * vdim]."""
+    """`sp`: models.mixers.WindowAttentionSpec; bias fp32 [heads, far + 1]. Returns [n, heads * vdim]."""
     n = q.shape[0]
     out = torch.empty((n, sp.heads * sp.vdim), dtype=q.dtype, device=q.device)
     rc = _lib.cuda().tb_window_attn(_dt(q), q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(), *rb.args(), table.data_ptr(),
                                     table.shape[1], page_size, sp.heads, sp.kv_heads, sp.dim, sp.vdim, float(sp.scale),
-                                    bias.data_ptr(), bias.shape[0] - 1, sp.window, sp.keep_first, out.data_ptr(),
+                                    bias.data_ptr(), bias.shape[1] - 1, sp.window, sp.keep_first, out.data_ptr(),
                                     _lib.stream_ptr())
     _lib.check(rc, "tb_window_attn")
     _count()
