@@ -123,8 +123,8 @@ __global__ void rglru_scan_kernel(const float* __restrict__ A, const float* __re
 // channel, the tile-local recurrence h (from zero) and the running product p of the decays; a small kernel chains the
 // tiles' last rows; the last kernel adds p * carry and applies the output gate. Nothing waits on another block.
 constexpr int LT = 64;          // tokens per tile
-constexpr int LC = 64;          // channels per CTA of the gate kernel
-constexpr int LTPC = 4;         // consecutive tiles per CTA: the weights stay in shared memory
+constexpr int LC = 32;          // channels per CTA of the gate kernel
+constexpr int LTPC = 8;         // consecutive tiles per CTA: the weights stay in shared memory
 
 struct Tiles {
   const int* t0;      // [tiles] first token of the tile
@@ -133,7 +133,7 @@ struct Tiles {
 };
 
 // u [n, W] -> H, P fp32 [n, W], and the tiles' last rows in LH, LP fp32 [tiles, W]
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 2)
 rglru_tile_kernel(const __nv_bfloat16* __restrict__ u, const __nv_bfloat16* __restrict__ ra,
                   const __nv_bfloat16* __restrict__ ba, const __nv_bfloat16* __restrict__ ri,
                   const __nv_bfloat16* __restrict__ bi, const __nv_bfloat16* __restrict__ lam, Ragged rb, Tiles tl, int W,
@@ -145,7 +145,9 @@ rglru_tile_kernel(const __nv_bfloat16* __restrict__ u, const __nv_bfloat16* __re
   uint8_t* Ws = smem + LT * pitch;                      // [2 * LC] rows: LC of ra, LC of ri
   float* As = reinterpret_cast<float*>(Ws + 2 * LC * pitch);   // [LT][LC + 1]
   float* Bs = As + LT * (LC + 1);
-  __shared__ float segA[4][LC], segB[4][LC];
+  constexpr int SEGS = 256 / LC, SEG = LT / SEGS;              // segments of a tile in the scan, tokens per segment
+  __shared__ float segA[SEGS][LC], segB[SEGS][LC];
+  __shared__ float s_sp[LC], s_ba[LC], s_bi[LC];
   pdl_trigger();
   pdl_wait();
   const int per_blk = (bs + LC - 1) / LC;
@@ -161,6 +163,12 @@ rglru_tile_kernel(const __nv_bfloat16* __restrict__ u, const __nv_bfloat16* __re
     cp_async16(ws + r * pitch + c * 16, src, ok ? 16 : 0);
   }
   cp_async_commit();
+  if (tid < LC && o0 + tid < bs) {
+    const int ch = blk * bs + o0 + tid;
+    s_sp[tid] = -8.f * softplus(to_f(lam[ch]));
+    s_ba[tid] = to_f(ba[ch]);
+    s_bi[tid] = to_f(bi[ch]);
+  }
   for (int k = 0; k < LTPC; ++k) {
     const int tile = blockIdx.y * LTPC + k;
     if (tile >= tl.count) break;
@@ -174,74 +182,71 @@ rglru_tile_kernel(const __nv_bfloat16* __restrict__ u, const __nv_bfloat16* __re
     cp_async_commit();
     cp_async_wait<0>();
     __syncthreads();
-    // warps: 4 rows of 16 tokens x 2 halves of 32 channels; both gates of a channel in the same thread
-    const int m0 = (warp & 3) * 16, n0 = (warp >> 2) * 32;
-    float r[4][4], g[4][4];
+    // warps: 4 rows of 16 tokens x 2 halves of 16 channels; both gates of a channel in the same thread
+    const int m0 = (warp & 3) * 16, n0 = (warp >> 2) * 16;
+    float r[2][4], g[2][4];
 #pragma unroll
-    for (int j = 0; j < 4; ++j)
+    for (int j = 0; j < 2; ++j)
 #pragma unroll
       for (int q = 0; q < 4; ++q) r[j][q] = g[j][q] = 0.f;
+    const uint32_t ua = us + (m0 + (li & 1) * 8 + lr) * pitch + (li >> 1) * 16;
+    const uint32_t wa = ws + (n0 + (li >> 1) * 8 + lr) * pitch + (li & 1) * 16;
+#pragma unroll 4
     for (int ks = 0; ks < kp / 16; ++ks) {
       uint32_t a[4], w0[4], w1[4];
-      ldsm_x4(a, us + (m0 + (li & 1) * 8 + lr) * pitch + (ks * 2 + (li >> 1)) * 16);
-#pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        const int row = n0 + h * 16 + (li >> 1) * 8 + lr;
-        ldsm_x4(w0, ws + row * pitch + (ks * 2 + (li & 1)) * 16);
-        ldsm_x4(w1, ws + (LC + row) * pitch + (ks * 2 + (li & 1)) * 16);
-        mma_16816(r[2 * h], a, w0[0], w0[1]);
-        mma_16816(r[2 * h + 1], a, w0[2], w0[3]);
-        mma_16816(g[2 * h], a, w1[0], w1[1]);
-        mma_16816(g[2 * h + 1], a, w1[2], w1[3]);
-      }
+      ldsm_x4(a, ua + ks * 32);
+      ldsm_x4(w0, wa + ks * 32);
+      ldsm_x4(w1, wa + LC * pitch + ks * 32);
+      mma_16816(r[0], a, w0[0], w0[1]);
+      mma_16816(r[1], a, w0[2], w0[3]);
+      mma_16816(g[0], a, w1[0], w1[1]);
+      mma_16816(g[1], a, w1[2], w1[3]);
     }
 #pragma unroll
-    for (int j = 0; j < 4; ++j)
+    for (int j = 0; j < 2; ++j)
 #pragma unroll
       for (int q = 0; q < 4; ++q) {
         const int c = n0 + j * 8 + 2 * (lane & 3) + (q & 1), t = m0 + (lane >> 2) + (q >> 1) * 8;
         const int o = o0 + c;
         float av = 1.f, bv = 0.f;
         if (t < nt && o < bs) {
-          const int ch = blk * bs + o;
-          const float la = -8.f * sigmoid(r[j][q] + to_f(ba[ch])) * softplus(to_f(lam[ch]));
+          const float em = quick_expm1(quick_sigmoid(r[j][q] + s_ba[c]) * s_sp[c]);      // a - 1
           const float uv = to_f(*reinterpret_cast<const __nv_bfloat16*>(Us + t * pitch + o * 2));
-          av = decay_exp(la);
-          bv = sqrtf(-expm1f(2.f * la)) * sigmoid(g[j][q] + to_f(bi[ch])) * uv;
+          av = 1.f + em;
+          bv = sqrtf(-em * (2.f + em)) * quick_sigmoid(g[j][q] + s_bi[c]) * uv;
         }
         As[t * (LC + 1) + c] = av;
         Bs[t * (LC + 1) + c] = bv;
       }
     __syncthreads();
-    // recurrence inside the tile: 4 segments of 16 tokens per channel, then the segments in order
-    const int c = tid & (LC - 1), sg = tid >> 6;
-    float pa = 1.f, hb = 0.f;
+    // recurrence inside the tile: SEGS segments per channel, then the segments in order
+    const int c = tid & (LC - 1), sg = tid / LC;
+    float pa[SEG], hb[SEG];
 #pragma unroll
-    for (int t = 0; t < LT / 4; ++t) {
-      const int x = (sg * (LT / 4) + t) * (LC + 1) + c;
+    for (int t = 0; t < SEG; ++t) {
+      const int x = (sg * SEG + t) * (LC + 1) + c;
       const float av = As[x];
-      hb = av * hb + Bs[x];
-      pa *= av;
-      As[x] = pa;
-      Bs[x] = hb;
+      hb[t] = t ? av * hb[t - 1] + Bs[x] : Bs[x];
+      pa[t] = t ? pa[t - 1] * av : av;
     }
-    segA[sg][c] = pa;
-    segB[sg][c] = hb;
+    segA[sg][c] = pa[SEG - 1];
+    segB[sg][c] = hb[SEG - 1];
     __syncthreads();
-    float cp = 1.f, ch = 0.f;
-    for (int j = 0; j < sg; ++j) { ch = segA[j][c] * ch + segB[j][c]; cp *= segA[j][c]; }
+    float cp = 1.f, chn = 0.f;
+    for (int j = 0; j < sg; ++j) { chn = segA[j][c] * chn + segB[j][c]; cp *= segA[j][c]; }
     if (o0 + c < bs) {
       const long long col = (long long)blk * bs + o0 + c;
 #pragma unroll
-      for (int t = 0; t < LT / 4; ++t) {
-        const int tt = sg * (LT / 4) + t;
-        if (tt >= nt) break;
-        const float p = As[tt * (LC + 1) + c], h = Bs[tt * (LC + 1) + c] + p * ch;
-        H[(long long)(t0 + tt) * W + col] = h;
-        P[(long long)(t0 + tt) * W + col] = p * cp;
-        if (tt == nt - 1) {
-          LH[(long long)tile * W + col] = h;
-          LP[(long long)tile * W + col] = p * cp;
+      for (int t = 0; t < SEG; ++t) {
+        const int tt = sg * SEG + t;
+        if (tt < nt) {
+          const float h = hb[t] + pa[t] * chn, p = pa[t] * cp;
+          H[(long long)(t0 + tt) * W + col] = h;
+          P[(long long)(t0 + tt) * W + col] = p;
+          if (tt == nt - 1) {
+            LH[(long long)tile * W + col] = h;
+            LP[(long long)tile * W + col] = p;
+          }
         }
       }
     }
@@ -298,51 +303,63 @@ rglru_out_kernel(const float* __restrict__ H, const float* __restrict__ P, const
     const float4 s = *reinterpret_cast<const float4*>(carry + (long long)tile * W + c);
     const uint2 y = *reinterpret_cast<const uint2*>(proj + (long long)t * ldp + y_off + c);
     uint2 o;
-    o.x = pack_bf16((h.x + p.x * s.x) * gelu_tanh(bf16_lo(y.x)), (h.y + p.y * s.y) * gelu_tanh(bf16_hi(y.x)));
-    o.y = pack_bf16((h.z + p.z * s.z) * gelu_tanh(bf16_lo(y.y)), (h.w + p.w * s.w) * gelu_tanh(bf16_hi(y.y)));
+    o.x = pack_bf16((h.x + p.x * s.x) * quick_gelu_tanh(bf16_lo(y.x)), (h.y + p.y * s.y) * quick_gelu_tanh(bf16_hi(y.x)));
+    o.y = pack_bf16((h.z + p.z * s.z) * quick_gelu_tanh(bf16_lo(y.y)), (h.w + p.w * s.w) * quick_gelu_tanh(bf16_hi(y.y)));
     *reinterpret_cast<uint2*>(out + (long long)t * W + c) = o;
   }
 }
 
-// 4 channels per thread form of rglru_conv_kernel
-__global__ void __launch_bounds__(256)
-rglru_conv4_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int x_off, const __nv_bfloat16* __restrict__ w,
-                   const __nv_bfloat16* __restrict__ bias, const float* __restrict__ ring, Ragged rb, int W, int K,
-                   __nv_bfloat16* __restrict__ u) {
+// rglru_conv_kernel for whole tiles: a thread takes 4 channels of CT consecutive tokens and keeps the KT taps and the
+// past inputs in registers.
+constexpr int CT = 16;
+template <int KT>
+__global__ void __launch_bounds__(128)
+rglru_conv_tile_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int x_off, const __nv_bfloat16* __restrict__ w,
+                       const __nv_bfloat16* __restrict__ bias, const float* __restrict__ ring, Ragged rb, Tiles tl, int W,
+                       __nv_bfloat16* __restrict__ u) {
   pdl_trigger();
   pdl_wait();
-  const int per = W / 4;
-  const long long total = (long long)rb.n * per;
-  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
-    const int t = (int)(i / per), c = (int)(i - (long long)t * per) * 4;
-    const int e = rb.ent[t], p0 = rb.pos0[e], first = rb.cu[e], p = p0 + t - first;
-    float acc[4];
+  const int c = (blockIdx.x * 128 + threadIdx.x) * 4;
+  const int tile = blockIdx.y, e = tl.ent[tile];
+  const int first = rb.cu[e], p0 = rb.pos0[e];
+  const int t0 = tl.t0[tile] + blockIdx.z * CT, t1 = min(min(t0 + CT, tl.t0[tile] + LT), rb.cu[e + 1]);
+  if (c >= W || t0 >= t1) return;
+  float taps[KT][4], past[KT][4], b4[4];                // past[j]: the input j tokens back
 #pragma unroll
-    for (int q = 0; q < 4; ++q) acc[q] = to_f(bias[c + q]);
-    for (int j = 0; j < K && j <= p; ++j) {
-      const int s = t - j;
-      float v[4];
-      if (s >= first) {
-        const uint2 x = *reinterpret_cast<const uint2*>(proj + (long long)s * ldp + x_off + c);
-        v[0] = bf16_lo(x.x); v[1] = bf16_hi(x.x); v[2] = bf16_lo(x.y); v[3] = bf16_hi(x.y);
-      } else {
-        const float4 x = *reinterpret_cast<const float4*>(ring + ((long long)rb.slot[e] * K + (p - j) % K) * W + c);
-        v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
-      }
+  for (int q = 0; q < 4; ++q) {
+    b4[q] = to_f(bias[c + q]);
 #pragma unroll
-      for (int q = 0; q < 4; ++q) acc[q] += to_f(w[(long long)(c + q) * K + K - 1 - j]) * v[q];
+    for (int j = 0; j < KT; ++j) taps[j][q] = to_f(w[(long long)(c + q) * KT + KT - 1 - j]);
+  }
+#pragma unroll
+  for (int j = 1; j < KT; ++j) {
+    const int t = t0 - j, p = p0 + t - first;
+#pragma unroll
+    for (int q = 0; q < 4; ++q) past[j][q] = 0.f;
+    if (t >= first) load_v<4>(proj + (long long)t * ldp + x_off + c, past[j]);
+    else if (p >= 0) load_v<4>(ring + ((long long)rb.slot[e] * KT + p % KT) * W + c, past[j]);
+  }
+  for (int t = t0; t < t1; ++t) {
+    load_v<4>(proj + (long long)t * ldp + x_off + c, past[0]);
+    float o[4];
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      o[q] = b4[q];
+#pragma unroll
+      for (int j = 0; j < KT; ++j) o[q] += taps[j][q] * past[j][q];
     }
-    uint2 o;
-    o.x = pack_bf16(acc[0], acc[1]);
-    o.y = pack_bf16(acc[2], acc[3]);
-    *reinterpret_cast<uint2*>(u + (long long)t * W + c) = o;
+    store_v<4>(u + (long long)t * W + c, o);
+#pragma unroll
+    for (int j = KT - 1; j > 0; --j)
+#pragma unroll
+      for (int q = 0; q < 4; ++q) past[j][q] = past[j - 1][q];
   }
 }
 
 // ---- bf16, one token per entry: convolution, gates, recurrence and output gate in one launch. CTA: 16 entries x DC output
 // channels of one block; every CTA computes the convolution of its whole block (the ring row written is never read).
 constexpr int DC = 32;
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(256)
 rglru_step_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int x_off, int y_off,
                   const __nv_bfloat16* __restrict__ cw, const __nv_bfloat16* __restrict__ cb,
                   const __nv_bfloat16* __restrict__ ra, const __nv_bfloat16* __restrict__ ba,
@@ -358,7 +375,7 @@ rglru_step_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int x_o
   const int blk = blockIdx.x / per_blk, o0 = (blockIdx.x - blk * per_blk) * DC, e0 = blockIdx.y * 16;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, li = lane >> 3, lr = lane & 7;
   // weights do not depend on the kernels before
-  for (int i = tid; i < 2 * DC * chunks; i += 128) {
+  for (int i = tid; i < 2 * DC * chunks; i += 256) {
     const int r = i / chunks, c = i - r * chunks, o = o0 + (r & (DC - 1));
     const bool ok = o < bs && c * 8 < bs;
     cp_async16(ws + r * pitch + c * 16, (r < DC ? ra : ri) + ((long long)blk * bs + (ok ? o : 0)) * bs + (ok ? c * 8 : 0), ok ? 16 : 0);
@@ -366,46 +383,67 @@ rglru_step_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int x_o
   cp_async_commit();
   pdl_trigger();
   pdl_wait();
-  for (int i = tid; i < 16 * kp; i += 128) {
-    const int r = i / kp, c = i - r * kp, e = e0 + r;
-    float acc = 0.f;
-    if (e < rb.E && c < bs) {
-      const int p = rb.pos0[e];
-      if (p >= 0) {
-        const int ch = blk * bs + c;
-        const long long rows = (long long)rb.slot[e] * K;
-        const float x = to_f(proj[(long long)e * ldp + x_off + ch]);
-        acc = to_f(cb[ch]) + to_f(cw[(long long)ch * K + K - 1]) * x;
-        for (int j = 1; j < K && j <= p; ++j) acc += to_f(cw[(long long)ch * K + K - 1 - j]) * ring[(rows + (p - j) % K) * W + ch];
-        if (c >= o0 && c < o0 + DC) ring[(rows + p % K) * W + ch] = x;
+  const int quads = kp / 4;
+  for (int i = tid; i < 16 * quads; i += 256) {
+    const int r = i / quads, c = (i - r * quads) * 4, e = e0 + r;
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    const int p = e < rb.E && c < bs ? rb.pos0[e] : -1;
+    if (p >= 0) {
+      const int ch = blk * bs + c;
+      const long long rows = (long long)rb.slot[e] * K;
+      float x[4], b4[4];
+      load_v<4>(proj + (long long)e * ldp + x_off + ch, x);
+      load_v<4>(cb + ch, b4);
+#pragma unroll
+      for (int q = 0; q < 4; ++q) acc[q] = b4[q] + to_f(cw[(long long)(ch + q) * K + K - 1]) * x[q];
+#pragma unroll 4
+      for (int j = 1; j < K; ++j) {
+        if (j > p) break;
+        float v[4];
+        load_v<4>(ring + (rows + (p - j) % K) * W + ch, v);
+#pragma unroll
+        for (int q = 0; q < 4; ++q) acc[q] += to_f(cw[(long long)(ch + q) * K + K - 1 - j]) * v[q];
       }
+      if (c >= o0 && c < o0 + DC) store_v<4>(ring + (rows + p % K) * W + ch, x);
     }
-    *reinterpret_cast<__nv_bfloat16*>(Us + r * pitch + c * 2) = __float2bfloat16(acc);
+    store_v<4>(reinterpret_cast<__nv_bfloat16*>(Us + r * pitch) + c, acc);
   }
   cp_async_wait<0>();
   __syncthreads();
+  // 8 warps: 4 groups of 8 channels x 2 halves of the contraction, summed through shared memory
   float r[4] = {0.f, 0.f, 0.f, 0.f}, g[4] = {0.f, 0.f, 0.f, 0.f};
-  for (int ks = 0; ks < kp / 16; ++ks) {
+  __shared__ float half_sum[4][32][8];
+  const int cg = warp & 3, kh = warp >> 2, nks = kp / 16, kmid = (nks + 1) / 2;
+#pragma unroll 4
+  for (int ks = kh ? kmid : 0; ks < (kh ? nks : kmid); ++ks) {
     uint32_t a[4], w[4];
     ldsm_x4(a, us + ((li & 1) * 8 + lr) * pitch + (ks * 2 + (li >> 1)) * 16);
     // matrices 0, 1: this warp's 8 channels of ra; 2, 3: of ri
-    ldsm_x4(w, ws + ((li >> 1) * DC + warp * 8 + lr) * pitch + (ks * 2 + (li & 1)) * 16);
+    ldsm_x4(w, ws + ((li >> 1) * DC + cg * 8 + lr) * pitch + (ks * 2 + (li & 1)) * 16);
     mma_16816(r, a, w[0], w[1]);
     mma_16816(g, a, w[2], w[3]);
   }
+  if (kh) {
+#pragma unroll
+    for (int q = 0; q < 4; ++q) { half_sum[cg][lane][q] = r[q]; half_sum[cg][lane][4 + q] = g[q]; }
+  }
+  __syncthreads();
+  if (kh) return;
+#pragma unroll
+  for (int q = 0; q < 4; ++q) { r[q] += half_sum[cg][lane][q]; g[q] += half_sum[cg][lane][4 + q]; }
 #pragma unroll
   for (int q = 0; q < 4; ++q) {
-    const int o = o0 + warp * 8 + 2 * (lane & 3) + (q & 1), row = (lane >> 2) + (q >> 1) * 8, e = e0 + row;
+    const int o = o0 + cg * 8 + 2 * (lane & 3) + (q & 1), row = (lane >> 2) + (q >> 1) * 8, e = e0 + row;
     if (o >= bs || e >= rb.E) continue;
     const int ch = blk * bs + o, p = rb.pos0[e];
     float res = 0.f;
     if (p >= 0) {
-      const float la = -8.f * sigmoid(r[q] + to_f(ba[ch])) * softplus(to_f(lam[ch]));
+      const float em = quick_expm1(-8.f * quick_sigmoid(r[q] + to_f(ba[ch])) * softplus(to_f(lam[ch])));   // a - 1
       const float uv = to_f(*reinterpret_cast<const __nv_bfloat16*>(Us + row * pitch + o * 2));
       float* st = state + (long long)rb.slot[e] * W + ch;
-      const float s = (p > 0 ? decay_exp(la) * *st : 0.f) + sqrtf(-expm1f(2.f * la)) * sigmoid(g[q] + to_f(bi[ch])) * uv;
+      const float s = (p > 0 ? (1.f + em) * *st : 0.f) + sqrtf(-em * (2.f + em)) * quick_sigmoid(g[q] + to_f(bi[ch])) * uv;
       *st = s;
-      res = s * gelu_tanh(to_f(proj[(long long)e * ldp + y_off + ch]));
+      res = s * quick_gelu_tanh(to_f(proj[(long long)e * ldp + y_off + ch]));
     }
     out[(long long)e * W + ch] = __float2bfloat16(res);
   }
@@ -579,33 +617,34 @@ mlstm_step_kernel(const T* __restrict__ proj, long long ldp, int q_off, int k_of
 // With F the running sum of f inside a chunk, g_s = i_s - F_s and M_t = max(m_prev, max_{s <= t} g_s), the recurrence above
 // unrolls to  m_t = F_t + M_t,
 //   o_t ~ e^(m_prev - M_t) q_t S + sum_{s <= t} e^(g_s - M_t) (q_t . k_s) v_s,   S' = e^(m_prev - M_L) S + sum_s e^(g_s - M_L) k_s v_s^T.
-// n and its products ride along as one more value column that holds ones. q, k, v are bf16 and exact; every fp32 factor (the
-// weights, the state, the scaled values) enters the tensor cores as a bf16 pair hi + lo. S stays in fp32 accumulators.
+// n rides along as one more column of S, fed by a value column of ones. What enters the recurrence keeps 32-bit accuracy: S
+// and n stay in fp32 accumulators, the scaled values go to the tensor cores as bf16 pairs hi + lo, k is bf16 and exact. The
+// read-out q S takes S rounded to bf16 (n as a pair, since the denominator may cancel); row sums of the weights are fp32.
 constexpr int ML = 64;
 constexpr int MN = MV + 8;              // value columns with the ones column (index MV), padded to 8
 constexpr int MVP = MN * 2;             // row pitch in bytes of [.., MN] bf16 tiles: 80, an odd multiple of 16
 constexpr int MPP = ML * 2 + 16;        // row pitch of the [ML, ML] weight tiles
 
 struct MlstmSmem {
-  int pitch, q, k, v, wv, p, s, gate, total;            // byte offsets; q, k, v are double buffered
+  int pitch, q, k, v, wv, p, s, gate, total;            // byte offsets
 };
 __host__ __device__ inline MlstmSmem mlstm_smem(int dk) {
   MlstmSmem L;
   const int kp = (dk + 15) & ~15;
   L.pitch = kp * 2 + 16;
   L.q = 0;
-  L.k = L.q + 2 * ML * L.pitch;
-  L.v = L.k + 2 * ML * L.pitch;
-  L.wv = L.v + 2 * ML * MVP;
+  L.k = L.q + ML * L.pitch;
+  L.v = L.k + ML * L.pitch;
+  L.wv = L.v + ML * MVP;
   L.p = L.wv + 2 * ML * MVP;
-  L.s = L.p + 2 * ML * MPP;
-  L.gate = L.s + 2 * kp * MVP;
-  L.total = L.gate + 6 * ML * 4;
+  L.s = L.p + ML * MPP;
+  L.gate = L.s + kp * MVP;
+  L.total = L.gate + 8 * ML * 4;
   return L;
 }
 
 template <int MT>       // 16-row tiles of S per warp: dk <= 128 * MT
-__global__ void __launch_bounds__(256, 1)
+__global__ void __launch_bounds__(256, 2)
 mlstm_chunk_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int q_off, int k_off, int v_off,
                    const float* __restrict__ gates, const __nv_bfloat16* __restrict__ ib, const __nv_bfloat16* __restrict__ fb,
                    float cap, Ragged rb, int heads, int dk, int dv, float* __restrict__ Sg, float* __restrict__ Ng,
@@ -619,6 +658,7 @@ mlstm_chunk_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int q_
   float* Wt = Ct + ML;                                  // e^(g_s - M_L)
   float* Em = Wt + ML;                                  // e^(-m_t)
   float* Den = Em + ML;
+  float* Sum = Den + ML;                                // [2][ML] row sums of the weights, per half of the keys
   __shared__ float s_m, s_decay;
   pdl_trigger();
   pdl_wait();
@@ -635,32 +675,29 @@ mlstm_chunk_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int q_
   const float bi = to_f(ib[hd]), bf = to_f(fb[hd]);
   const float qscale = 1.f / sqrtf((float)dk);
 
-  auto load = [&](int ch, int buf) {
+  auto load = [&](int ch) {
     const int rows = min(ML, len - ch * ML);
     const __nv_bfloat16* base = proj + (long long)(t0 + ch * ML) * ldp;
     for (int i = tid; i < ML * kchunks; i += 256) {
       const int r = i / kchunks, c = i - r * kchunks;
       const bool ok = r < rows && c * 8 < dk;
       const long long src = ok ? (long long)r * ldp + hd * dk + c * 8 : 0;
-      const uint32_t d = (buf * ML + r) * L.pitch + c * 16;
+      const uint32_t d = r * L.pitch + c * 16;
       cp_async16(sb + L.q + d, base + q_off + src, ok ? 16 : 0);
       cp_async16(sb + L.k + d, base + k_off + src, ok ? 16 : 0);
     }
     for (int i = tid; i < ML * (MV / 8); i += 256) {
       const int r = i / (MV / 8), c = i - r * (MV / 8);
       const bool ok = r < rows && c * 8 < nc;
-      cp_async16(sb + L.v + (buf * ML + r) * MVP + c * 16, base + v_off + (ok ? (long long)r * ldp + hd * dv + c0 + c * 8 : 0),
-                 ok ? 16 : 0);
+      cp_async16(sb + L.v + r * MVP + c * 16, base + v_off + (ok ? (long long)r * ldp + hd * dv + c0 + c * 8 : 0), ok ? 16 : 0);
     }
     cp_async_commit();
   };
 
-  // the ones column (and its padding) of both value buffers
-  for (int i = tid; i < 2 * ML; i += 256) {
-    uint4 u = make_uint4(0x3f80u, 0u, 0u, 0u);          // bf16 1.0 in the first of 8 columns
-    *reinterpret_cast<uint4*>(smem + L.v + i * MVP + MV * 2) = u;
-  }
-  load(0, 0);
+  // the ones column (and its padding)
+  for (int i = tid; i < ML; i += 256)
+    *reinterpret_cast<uint4*>(smem + L.v + i * MVP + MV * 2) = make_uint4(0x3f80u, 0u, 0u, 0u);   // 1.0 in the first of 8 columns
+  load(0);
 
   // state -> accumulators: warp w owns the 16-row tiles w, w + 8, ...
   float S[MT][5][4];
@@ -678,22 +715,21 @@ mlstm_chunk_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int q_
         }
         S[a][j][q] = v;
       }
-  auto store_s = [&]() {                // hi + lo of the state, the B operand of Q S
+  // S as the B operand of Q S: bf16, and in the last column tile n as hi (column MV) and lo (column MV + 1)
+  auto store_s = [&]() {
 #pragma unroll
     for (int a = 0; a < MT; ++a) {
       if (warp + a * 8 >= mtiles) continue;
 #pragma unroll
-      for (int j = 0; j < 5; ++j)
+      for (int h = 0; h < 2; ++h) {
+        const int d = (warp + a * 8) * 16 + (lane >> 2) + h * 8;
 #pragma unroll
-        for (int h = 0; h < 2; ++h) {
-          const int d = (warp + a * 8) * 16 + (lane >> 2) + h * 8;
-          const uint32_t off = d * MVP + (j * 8 + 2 * (lane & 3)) * 2;
-          __nv_bfloat16 h0, l0, h1, l1;
-          split_bf16(S[a][j][2 * h], h0, l0);
-          split_bf16(S[a][j][2 * h + 1], h1, l1);
-          *reinterpret_cast<__nv_bfloat162*>(smem + L.s + off) = __halves2bfloat162(h0, h1);
-          *reinterpret_cast<__nv_bfloat162*>(smem + L.s + kp * MVP + off) = __halves2bfloat162(l0, l1);
-        }
+        for (int j = 0; j < 4; ++j)
+          *reinterpret_cast<uint32_t*>(smem + L.s + d * MVP + (j * 8 + 2 * (lane & 3)) * 2) = pack_bf16(S[a][j][2 * h], S[a][j][2 * h + 1]);
+        __nv_bfloat16 hi, lo;
+        split_bf16((lane & 3) == 0 ? S[a][4][2 * h] : 0.f, hi, lo);
+        *reinterpret_cast<__nv_bfloat162*>(smem + L.s + d * MVP + (MV + 2 * (lane & 3)) * 2) = __halves2bfloat162(hi, lo);
+      }
     }
   };
   store_s();
@@ -701,11 +737,10 @@ mlstm_chunk_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int q_
   const int n_ch = (len + ML - 1) / ML;
   const int wm = (warp & 3) * 16, wn = warp >> 2;       // 16 tokens; half of the keys (P) or of the value columns (O)
   for (int ch = 0; ch < n_ch; ++ch) {
-    const int buf = ch & 1, rows = min(ML, len - ch * ML);
+    const int rows = min(ML, len - ch * ML);
     cp_async_wait<0>();
-    __syncthreads();                    // the tiles are in; the other buffer and S of the last chunk are settled
-    if (ch + 1 < n_ch) load(ch + 1, buf ^ 1);
-    const uint32_t qb = sb + L.q + buf * ML * L.pitch, kb = sb + L.k + buf * ML * L.pitch, vb = sb + L.v + buf * ML * MVP;
+    __syncthreads();                    // the tiles are in, S of the last chunk is stored
+    const uint32_t qb = sb + L.q, kb = sb + L.k, vb = sb + L.v;
     if (warp == 0) {
       // gates of the chunk, two tokens per lane
       float f[2], ii[2];
@@ -752,6 +787,7 @@ mlstm_chunk_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int q_
     for (int j = 0; j < 4; ++j) P[j][0] = P[j][1] = P[j][2] = P[j][3] = 0.f;
     const int kn = wn * 32;
     if (kn <= wm + 15) {
+#pragma unroll 4
       for (int ks = 0; ks < mtiles; ++ks) {
         uint32_t a[4], b[4];
         ldsm_x4(a, qb + (wm + (li & 1) * 8 + lr) * L.pitch + (ks * 2 + (li >> 1)) * 16);
@@ -767,22 +803,25 @@ mlstm_chunk_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int q_
     m_prev = s_m;
     const float decay = s_decay;
 #pragma unroll
-    for (int j = 0; j < 4; ++j)
+    for (int h = 0; h < 2; ++h) {
+      const int t = wm + (lane >> 2) + h * 8;
+      const float M = Mx[t];
+      float sum = 0.f;
 #pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        const int t = wm + (lane >> 2) + h * 8, s = kn + j * 8 + 2 * (lane & 3);
-        const float M = Mx[t];
-        const float w0 = s <= t ? P[j][2 * h] * qscale * expf(G[s] - M) : 0.f;
-        const float w1 = s + 1 <= t ? P[j][2 * h + 1] * qscale * expf(G[s + 1] - M) : 0.f;
-        __nv_bfloat16 h0, l0, h1, l1;
-        split_bf16(w0, h0, l0);
-        split_bf16(w1, h1, l1);
-        *reinterpret_cast<__nv_bfloat162*>(smem + L.p + t * MPP + s * 2) = __halves2bfloat162(h0, h1);
-        *reinterpret_cast<__nv_bfloat162*>(smem + L.p + ML * MPP + t * MPP + s * 2) = __halves2bfloat162(l0, l1);
+      for (int j = 0; j < 4; ++j) {
+        const int s = kn + j * 8 + 2 * (lane & 3);
+        const float w0 = s <= t ? P[j][2 * h] * qscale * __expf(G[s] - M) : 0.f;
+        const float w1 = s + 1 <= t ? P[j][2 * h + 1] * qscale * __expf(G[s + 1] - M) : 0.f;
+        sum += w0 + w1;
+        *reinterpret_cast<uint32_t*>(smem + L.p + t * MPP + s * 2) = pack_bf16(w0, w1);
       }
+      sum += __shfl_xor_sync(0xffffffffu, sum, 1);
+      sum += __shfl_xor_sync(0xffffffffu, sum, 2);
+      if ((lane & 3) == 0) Sum[wn * ML + t] = sum;
+    }
     for (int i = tid; i < ML * (MN / 2); i += 256) {    // w_s v_s, hi and lo
       const int r = i / (MN / 2), c = (i - r * (MN / 2)) * 2;
-      const uint32_t v2 = *reinterpret_cast<const uint32_t*>(smem + L.v + (buf * ML + r) * MVP + c * 2);
+      const uint32_t v2 = *reinterpret_cast<const uint32_t*>(smem + L.v + r * MVP + c * 2);
       const float w = Wt[r];
       __nv_bfloat16 h0, l0, h1, l1;
       split_bf16(w * bf16_lo(v2), h0, l0);
@@ -791,24 +830,22 @@ mlstm_chunk_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int q_
       *reinterpret_cast<__nv_bfloat162*>(smem + L.wv + ML * MVP + r * MVP + c * 2) = __halves2bfloat162(l0, l1);
     }
     __syncthreads();
-    // O = diag(c) Q S + P V; column tiles 0..2 (first half) or 3, 4 (second half; tile 4 carries the ones column)
+    // O = diag(c) Q S + P V; column tiles 0, 1 and the pair of n (first half of the warps) or 2, 3 (second half)
     float O[3][4];
 #pragma unroll
     for (int j = 0; j < 3; ++j) O[j][0] = O[j][1] = O[j][2] = O[j][3] = 0.f;
     const uint32_t row16 = (li & 1) * 8 + lr;           // row inside a 16-row B tile
+#pragma unroll 4
     for (int ks = 0; ks < mtiles; ++ks) {
       uint32_t a[4], b[4], b2[2];
       ldsm_x4(a, qb + (wm + (li & 1) * 8 + lr) * L.pitch + (ks * 2 + (li >> 1)) * 16);
-#pragma unroll
-      for (int part = 0; part < 2; ++part) {
-        const uint32_t base = sb + L.s + part * kp * MVP + (ks * 16 + row16) * MVP;
-        ldsm_x4_t(b, base + (wn * 3 + (li >> 1)) * 16);
-        mma_16816(O[0], a, b[0], b[1]);
-        mma_16816(O[1], a, b[2], b[3]);
-        if (wn == 0) {
-          ldsm_x2_t(b2, base + 2 * 16);
-          mma_16816(O[2], a, b2[0], b2[1]);
-        }
+      const uint32_t base = sb + L.s + (ks * 16 + row16) * MVP;
+      ldsm_x4_t(b, base + (wn * 2 + (li >> 1)) * 16);
+      mma_16816(O[0], a, b[0], b[1]);
+      mma_16816(O[1], a, b[2], b[3]);
+      if (wn == 0) {
+        ldsm_x2_t(b2, base + 4 * 16);
+        mma_16816(O[2], a, b2[0], b2[1]);
       }
     }
     {
@@ -819,23 +856,19 @@ mlstm_chunk_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int q_
 #pragma unroll
     for (int ks = 0; ks < ML / 16; ++ks) {
       if (ks * 16 > wm + 15) continue;                  // weights past the diagonal are zero
-      uint32_t b[4], b2[2];
-      const uint32_t base = vb + (ks * 16 + row16) * MVP;
-      ldsm_x4_t(b, base + (wn * 3 + (li >> 1)) * 16);
-      if (wn == 0) ldsm_x2_t(b2, base + 2 * 16);
-#pragma unroll
-      for (int part = 0; part < 2; ++part) {
-        uint32_t a[4];
-        ldsm_x4(a, sb + L.p + part * ML * MPP + (wm + (li & 1) * 8 + lr) * MPP + (ks * 2 + (li >> 1)) * 16);
-        mma_16816(O[0], a, b[0], b[1]);
-        mma_16816(O[1], a, b[2], b[3]);
-        if (wn == 0) mma_16816(O[2], a, b2[0], b2[1]);
-      }
+      uint32_t a[4], b[4];
+      ldsm_x4_t(b, vb + (ks * 16 + row16) * MVP + (wn * 2 + (li >> 1)) * 16);
+      ldsm_x4(a, sb + L.p + (wm + (li & 1) * 8 + lr) * MPP + (ks * 2 + (li >> 1)) * 16);
+      mma_16816(O[0], a, b[0], b[1]);
+      mma_16816(O[1], a, b[2], b[3]);
     }
-    if (wn == 1 && (lane & 3) == 0) {                   // column MV: n . q
-      const int ta = wm + (lane >> 2), tb_ = ta + 8;
-      Den[ta] = 1.f / (fmaxf(fabsf(O[1][0]), Em[ta]) + 1e-6f);
-      Den[tb_] = 1.f / (fmaxf(fabsf(O[1][2]), Em[tb_]) + 1e-6f);
+    if (wn == 0 && (lane & 3) == 0) {                   // n . q
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int t = wm + (lane >> 2) + h * 8;
+        const float nq = O[2][2 * h] + O[2][2 * h + 1] + Sum[t] + Sum[ML + t];
+        Den[t] = 1.f / (fmaxf(fabsf(nq), Em[t]) + 1e-6f);
+      }
     }
     // S = decay S + K^T (w V)
 #pragma unroll
@@ -865,20 +898,19 @@ mlstm_chunk_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int q_
         }
       }
     }
-    __syncthreads();                    // Den is complete; nobody reads the old S any more
+    __syncthreads();                    // Den is complete; nobody reads the tiles or the old S any more
+    if (ch + 1 < n_ch) load(ch + 1);
     store_s();
 #pragma unroll
-    for (int j = 0; j < 3; ++j) {
-      const int tile = wn * 3 + j;
-      if (tile > 3) continue;
+    for (int j = 0; j < 2; ++j) {
+      const int tile = wn * 2 + j;
 #pragma unroll
       for (int h = 0; h < 2; ++h) {
         const int t = wm + (lane >> 2) + h * 8, c = tile * 8 + 2 * (lane & 3);
         if (t < rows && c < nc) {
           const float dn = Den[t];
-          float* o = out + ((long long)(t0 + ch * ML + t) * heads + hd) * dv + c0 + c;
-          o[0] = O[j][2 * h] * dn;
-          if (c + 1 < nc) o[1] = O[j][2 * h + 1] * dn;
+          *reinterpret_cast<float2*>(out + ((long long)(t0 + ch * ML + t) * heads + hd) * dv + c0 + c) =
+              make_float2(O[j][2 * h] * dn, O[j][2 * h + 1] * dn);      // dv and c are even
         }
       }
     }
@@ -924,7 +956,7 @@ TB_API int tb_rglru(int dtype, const void* proj, long long ldp, int x_off, int y
         if (once.first() && cudaFuncSetAttribute(rglru_step_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess)
           return -5;
         const dim3 grid(blocks * ((bs + DC - 1) / DC), (E + 15) / 16);
-        return launch_pdl(rglru_step_kernel, grid, dim3(128), smem, stream, (const bf*)proj, ldp, x_off, y_off, (const bf*)conv_w,
+        return launch_pdl(rglru_step_kernel, grid, dim3(256), smem, stream, (const bf*)proj, ldp, x_off, y_off, (const bf*)conv_w,
                           (const bf*)conv_b, (const bf*)ra, (const bf*)rab, (const bf*)ri, (const bf*)rib, (const bf*)lam, rb, W,
                           bs, K, state, ring, (bf*)out) == cudaSuccess ? 0 : -5;
       }
@@ -939,8 +971,21 @@ TB_API int tb_rglru(int dtype, const void* proj, long long ldp, int x_off, int y
         const dim3 flat((unsigned)(want < 148 * 16 ? want : 148 * 16));
         const dim3 gtile(blocks * ((bs + LC - 1) / LC), (tiles + LTPC - 1) / LTPC);
         if (gtile.y > 65535) return -2;
-        cudaError_t err = launch_pdl(rglru_conv4_kernel, flat, dim3(256), 0, stream, (const bf*)proj, ldp, x_off, (const bf*)conv_w,
-                                     (const bf*)conv_b, (const float*)ring, rb, W, K, (bf*)u);
+        if (tiles > 65535) return -2;
+        cudaError_t err;
+#define CONV(KT)                                                                                                              \
+  case KT:                                                                                                                    \
+    err = launch_pdl(rglru_conv_tile_kernel<KT>, dim3((W / 4 + 127) / 128, tiles, LT / CT), dim3(128), 0, stream,              \
+                     (const bf*)proj, ldp, x_off, (const bf*)conv_w, (const bf*)conv_b, (const float*)ring, rb, tl, W, (bf*)u); \
+    break;
+        switch (K) {
+          CONV(1) CONV(2) CONV(3) CONV(4) CONV(5) CONV(6) CONV(7) CONV(8)
+          default:
+            if (n > 65535) return -2;
+            err = launch_pdl(rglru_conv_kernel<bf>, dim3((W + 127) / 128, n), dim3(128), 0, stream, (const bf*)proj, ldp, x_off,
+                             (const bf*)conv_w, (const bf*)conv_b, (const float*)ring, rb, W, K, (bf*)u);
+        }
+#undef CONV
         if (err == cudaSuccess)
           err = launch_pdl(rglru_tile_kernel, gtile, dim3(256), smem, stream, (const bf*)u, (const bf*)ra, (const bf*)rab,
                            (const bf*)ri, (const bf*)rib, (const bf*)lam, rb, tl, W, bs, A, B, LH, LP);

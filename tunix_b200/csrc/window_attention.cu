@@ -24,10 +24,10 @@ __device__ __forceinline__ long long page_row(const Paged& pg, const int* pt, in
   return (long long)pt[p / pg.page_size] * pg.page_size + p % pg.page_size;
 }
 
-template <typename T>
+template <typename T, int V>
 __global__ void __launch_bounds__(256)
 qk_norm_write_kernel(const T* __restrict__ proj, long long ldp, int q_off, int k_off, int v_off, const T* __restrict__ qw,
-                     const T* __restrict__ kw, float eps, Ragged rb, Paged pg, int NQ, int NK, int NV, T* __restrict__ q,
+                     const T* __restrict__ kw, float eps, Ragged rb, Paged pg, int NQ, int NK, int NVv, T* __restrict__ q,
                      T* __restrict__ kp, T* __restrict__ vp) {
   __shared__ float red[33];
   pdl_trigger();
@@ -40,16 +40,39 @@ qk_norm_write_kernel(const T* __restrict__ proj, long long ldp, int q_off, int k
     return;
   }
   float sq = 0.f, sk = 0.f;
-  for (int c = tid; c < NQ; c += blockDim.x) { const float v = to_f(row[q_off + c]); sq += v * v; }
-  for (int c = tid; c < NK; c += blockDim.x) { const float v = to_f(row[k_off + c]); sk += v * v; }
-  sq = block_sum(sq, red);
-  sk = block_sum(sk, red);
+  const int step = blockDim.x * V;
+  auto sumsq = [&](int off, int N) {
+    float s = 0.f;
+    for (int c = tid * V; c < N; c += step) {
+      float v[V];
+      load_v<V>(row + off + c, v);
+#pragma unroll
+      for (int i = 0; i < V; ++i) s += v[i] * v[i];
+    }
+    return s;
+  };
+  sq = block_sum(sumsq(q_off, NQ), red);
+  sk = block_sum(sumsq(k_off, NK), red);
   const float rq = 1.f / sqrtf(sq / (float)NQ + eps), rk = 1.f / sqrtf(sk / (float)NK + eps);
   const int p = p0 + t - rb.cu[e];
   const long long pr = page_row(pg, pg.table + (long long)rb.slot[e] * pg.max_pages, p);
-  for (int c = tid; c < NQ; c += blockDim.x) q[(long long)t * NQ + c] = from_f<T>(to_f(row[q_off + c]) * rq * to_f(qw[c]));
-  for (int c = tid; c < NK; c += blockDim.x) kp[pr * NK + c] = from_f<T>(to_f(row[k_off + c]) * rk * to_f(kw[c]));
-  for (int c = tid; c < NV; c += blockDim.x) vp[pr * NV + c] = row[v_off + c];
+  auto norm = [&](int off, int N, float r, const T* w, T* dst) {
+    for (int c = tid * V; c < N; c += step) {
+      float v[V], ww[V];
+      load_v<V>(row + off + c, v);
+      load_v<V>(w + c, ww);
+#pragma unroll
+      for (int i = 0; i < V; ++i) v[i] = v[i] * r * ww[i];
+      store_v<V>(dst + c, v);
+    }
+  };
+  norm(q_off, NQ, rq, qw, q + (long long)t * NQ);
+  norm(k_off, NK, rk, kw, kp + pr * NK);
+  for (int c = tid * V; c < NVv; c += step) {
+    float v[V];
+    load_v<V>(row + v_off + c, v);
+    store_v<V>(vp + pr * NVv + c, v);
+  }
 }
 
 constexpr int VREG = 16;        // value columns per lane: value heads up to 512 wide
@@ -135,12 +158,13 @@ TB_API int tb_qk_norm_write(int dtype, const void* proj, long long ldp, int q_of
   if (n <= 0) return 0;
   RAGGED;
   PAGED;
-#define RUN(T)                                                                                                               \
-  return launch_pdl(qk_norm_write_kernel<T>, dim3(n), dim3(256), 0, stream, (const T*)proj, ldp, q_off, k_off, v_off,        \
-                    (const T*)qw, (const T*)kw, eps, rb, pg, NQ, NK, NV, (T*)q, (T*)kp, (T*)vp) == cudaSuccess ? 0 : -5
-  if (dtype == 0) RUN(__nv_bfloat16);
-  RUN(float);
+  const bool vec = NQ % 8 == 0 && NK % 8 == 0 && NV % 8 == 0 && q_off % 8 == 0 && k_off % 8 == 0 && v_off % 8 == 0 && ldp % 8 == 0;
+#define RUN(T, V)                                                                                                            \
+  launch_pdl(qk_norm_write_kernel<T, V>, dim3(n), dim3(256), 0, stream, (const T*)proj, ldp, q_off, k_off, v_off,            \
+             (const T*)qw, (const T*)kw, eps, rb, pg, NQ, NK, NV, (T*)q, (T*)kp, (T*)vp)
+  const cudaError_t err = dtype == 0 ? (vec ? RUN(__nv_bfloat16, 8) : RUN(__nv_bfloat16, 1)) : RUN(float, 1);
 #undef RUN
+  return err == cudaSuccess ? 0 : -5;
 }
 
 // bias fp32 [H, far + 1]: what is added to the score of a key at distance min(i - j, far). window <= 0: no window.

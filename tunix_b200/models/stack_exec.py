@@ -124,7 +124,10 @@ class StackExecutor:
         d, lf, rt = self.w[i], m.left, m.right
         a, s = lf.spec, rt.spec
         proj = linear(h, d["proj"], packed=self.pk(i, "proj") if rb.decode else None)
-        gates = linear(h, d["gates"], out_dtype=torch.float32)
+        if rb.decode and h.dtype == torch.bfloat16 and h.shape[1] % 8 == 0:
+            gates = SK.few_outputs(h, d["gates"])
+        else:
+            gates = linear(h, d["gates"], out_dtype=torch.float32)
         off, cols = [], 0
         for width in (a.heads * a.dim, a.kv_heads * a.dim, a.kv_heads * a.vdim, a.heads * a.vdim, s.heads * s.dim, s.heads * s.dim,
                       s.heads * s.vdim, s.heads * s.vdim):

@@ -14,6 +14,7 @@ _P, _I, _LL, _F = _lib.P, _lib.I, _lib.LL, _lib.F
 _RB = [_P, _P, _P, _P, _I, _I]
 _lib.register_cuda_sigs({
     "tb_stream_step": [_I, _P, _I, _I, _I, _F, _P, _P, _P, _P, _P, _P, _P, _P, _I, _P, _P, _P, _P, _P],
+    "tb_few_outputs": [_P, _P, _I, _I, _I, _P, _P],
     "tb_silu_mul": [_I, _P, _P, _LL, _I, _P],
     "tb_gate_outputs": [_I, _P, _P, _P, _LL, _I, _I, _P, _F, _I, _I, _I, _I, _P, _P, _P],
     "tb_rglru": [_I, _P, _LL, _I, _I, _P, _P, _P, _P, _P, _P, _P, *_RB, _I, _I, _I, _P, _P, _P, _P, _P, _P, _I, _P, _P,
@@ -58,6 +59,17 @@ def silu_mul(gu: torch.Tensor) -> torch.Tensor:
     _lib.check(rc, "tb_silu_mul")
     _count()
     return h
+
+
+def few_outputs(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """x bf16 [n, K] @ w^T [N, K] -> fp32 [n, N] for a handful of outputs and decode-size n (a GEMM tile would leave one CTA
+    with the whole contraction)."""
+    assert x.dtype == w.dtype == torch.bfloat16 and x.is_contiguous() and w.is_contiguous() and x.shape[1] % 8 == 0
+    out = torch.empty((x.shape[0], w.shape[0]), dtype=torch.float32, device=x.device)
+    rc = _lib.cuda().tb_few_outputs(x.data_ptr(), w.data_ptr(), x.shape[0], x.shape[1], w.shape[0], out.data_ptr(), _lib.stream_ptr())
+    _lib.check(rc, "tb_few_outputs")
+    _count()
+    return out
 
 
 def gate_outputs(attn, o, proj, g1_off: int, g2_off: int, norm_w, eps: float, heads: int, vdim: int):
