@@ -141,10 +141,8 @@ rglru_tile_kernel(const __nv_bfloat16* __restrict__ u, const __nv_bfloat16* __re
   extern __shared__ __align__(16) uint8_t smem[];
   const int kp = (bs + 15) & ~15;                       // contraction length, zero-padded
   const int pitch = kp * 2 + 16;                        // bytes per row
-  uint8_t* Us = smem;                                   // [LT] rows of u
-  uint8_t* Ws = smem + LT * pitch;                      // [2 * LC] rows: LC of ra, LC of ri
-  float* As = reinterpret_cast<float*>(Ws + 2 * LC * pitch);   // [LT][LC + 1]
-  float* Bs = As + LT * (LC + 1);
+  const int ubytes = max(LT * pitch, 2 * LT * (LC + 1) * 4);   // one buffer: a u tile, later the scan's a and b
+  uint8_t* Ws = smem + 2 * ubytes;                      // [2 * LC] rows: LC of ra, LC of ri
   constexpr int SEGS = 256 / LC, SEG = LT / SEGS;              // segments of a tile in the scan, tokens per segment
   __shared__ float segA[SEGS][LC], segB[SEGS][LC];
   __shared__ float s_sp[LC], s_ba[LC], s_bi[LC];
@@ -154,7 +152,18 @@ rglru_tile_kernel(const __nv_bfloat16* __restrict__ u, const __nv_bfloat16* __re
   const int blk = blockIdx.x / per_blk, o0 = (blockIdx.x - blk * per_blk) * LC;    // channels o0.. of block blk
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, li = lane >> 3, lr = lane & 7;
   const int chunks = kp / 8;
-  const uint32_t us = smem_u32(Us), ws = smem_u32(Ws);
+  const uint32_t ws = smem_u32(Ws);
+  const int tile_end = min(tl.count, ((int)blockIdx.y + 1) * LTPC);
+  auto load_u = [&](int tile) {
+    const int t0 = tl.t0[tile], nt = min(LT, rb.cu[tl.ent[tile] + 1] - t0);
+    const uint32_t dst = smem_u32(smem) + (tile & 1) * ubytes;
+    for (int i = tid; i < LT * chunks; i += 256) {
+      const int r = i / chunks, c = i - r * chunks;
+      const bool ok = r < nt && c * 8 < bs;
+      cp_async16(dst + r * pitch + c * 16, u + (ok ? (long long)(t0 + r) * W + (long long)blk * bs + c * 8 : 0), ok ? 16 : 0);
+    }
+    cp_async_commit();
+  };
   for (int i = tid; i < 2 * LC * chunks; i += 256) {
     const int r = i / chunks, c = i - r * chunks;
     const int o = o0 + (r & (LC - 1));
@@ -162,26 +171,23 @@ rglru_tile_kernel(const __nv_bfloat16* __restrict__ u, const __nv_bfloat16* __re
     const __nv_bfloat16* src = (r < LC ? ra : ri) + ((long long)blk * bs + (ok ? o : 0)) * bs + (ok ? c * 8 : 0);
     cp_async16(ws + r * pitch + c * 16, src, ok ? 16 : 0);
   }
-  cp_async_commit();
+  load_u(blockIdx.y * LTPC);                            // one group: the weights and the first tile
   if (tid < LC && o0 + tid < bs) {
     const int ch = blk * bs + o0 + tid;
     s_sp[tid] = -8.f * softplus(to_f(lam[ch]));
     s_ba[tid] = to_f(ba[ch]);
     s_bi[tid] = to_f(bi[ch]);
   }
-  for (int k = 0; k < LTPC; ++k) {
-    const int tile = blockIdx.y * LTPC + k;
-    if (tile >= tl.count) break;
+  for (int tile = blockIdx.y * LTPC; tile < tile_end; ++tile) {
     const int e = tl.ent[tile], t0 = tl.t0[tile];
     const int nt = min(LT, rb.cu[e + 1] - t0);
-    for (int i = tid; i < LT * chunks; i += 256) {
-      const int r = i / chunks, c = i - r * chunks;
-      const bool ok = r < nt && c * 8 < bs;
-      cp_async16(us + r * pitch + c * 16, u + (ok ? (long long)(t0 + r) * W + (long long)blk * bs + c * 8 : 0), ok ? 16 : 0);
-    }
-    cp_async_commit();
+    uint8_t* Us = smem + (tile & 1) * ubytes;
+    const uint32_t us = smem_u32(Us);
+    float* As = reinterpret_cast<float*>(Us);           // [LT][LC + 1], once the tile has been consumed
+    float* Bs = As + LT * (LC + 1);
     cp_async_wait<0>();
-    __syncthreads();
+    __syncthreads();                                    // the tile is in; the other buffer is done with
+    if (tile + 1 < tile_end) load_u(tile + 1);
     // warps: 4 rows of 16 tokens x 2 halves of 16 channels; both gates of a channel in the same thread
     const int m0 = (warp & 3) * 16, n0 = (warp >> 2) * 16;
     float r[2][4], g[2][4];
@@ -202,21 +208,30 @@ rglru_tile_kernel(const __nv_bfloat16* __restrict__ u, const __nv_bfloat16* __re
       mma_16816(g[0], a, w1[0], w1[1]);
       mma_16816(g[1], a, w1[2], w1[3]);
     }
+    float bvs[2][4];
 #pragma unroll
     for (int j = 0; j < 2; ++j)
 #pragma unroll
       for (int q = 0; q < 4; ++q) {
         const int c = n0 + j * 8 + 2 * (lane & 3) + (q & 1), t = m0 + (lane >> 2) + (q >> 1) * 8;
-        const int o = o0 + c;
         float av = 1.f, bv = 0.f;
-        if (t < nt && o < bs) {
+        if (t < nt && o0 + c < bs) {
           const float em = quick_expm1(quick_sigmoid(r[j][q] + s_ba[c]) * s_sp[c]);      // a - 1
-          const float uv = to_f(*reinterpret_cast<const __nv_bfloat16*>(Us + t * pitch + o * 2));
+          const float uv = to_f(*reinterpret_cast<const __nv_bfloat16*>(Us + t * pitch + (o0 + c) * 2));
           av = 1.f + em;
           bv = sqrtf(-em * (2.f + em)) * quick_sigmoid(g[j][q] + s_bi[c]) * uv;
         }
-        As[t * (LC + 1) + c] = av;
-        Bs[t * (LC + 1) + c] = bv;
+        r[j][q] = av;
+        bvs[j][q] = bv;
+      }
+    __syncthreads();                                    // every warp is done with u
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        const int c = n0 + j * 8 + 2 * (lane & 3) + (q & 1), t = m0 + (lane >> 2) + (q >> 1) * 8;
+        As[t * (LC + 1) + c] = r[j][q];
+        Bs[t * (LC + 1) + c] = bvs[j][q];
       }
     __syncthreads();
     // recurrence inside the tile: SEGS segments per channel, then the segments in order
@@ -250,7 +265,6 @@ rglru_tile_kernel(const __nv_bfloat16* __restrict__ u, const __nv_bfloat16* __re
         }
       }
     }
-    __syncthreads();
   }
 }
 
@@ -359,6 +373,7 @@ rglru_conv_tile_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, in
 // ---- bf16, one token per entry: convolution, gates, recurrence and output gate in one launch. CTA: 16 entries x DC output
 // channels of one block; every CTA computes the convolution of its whole block (the ring row written is never read).
 constexpr int DC = 32;
+template <int KT>               // taps, or 0 for any number
 __global__ void __launch_bounds__(256)
 rglru_step_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int x_off, int y_off,
                   const __nv_bfloat16* __restrict__ cw, const __nv_bfloat16* __restrict__ cb,
@@ -383,30 +398,55 @@ rglru_step_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int x_o
   cp_async_commit();
   pdl_trigger();
   pdl_wait();
-  const int quads = kp / 4;
-  for (int i = tid; i < 16 * quads; i += 256) {
-    const int r = i / quads, c = (i - r * quads) * 4, e = e0 + r;
-    float acc[4] = {0.f, 0.f, 0.f, 0.f};
-    const int p = e < rb.E && c < bs ? rb.pos0[e] : -1;
-    if (p >= 0) {
-      const int ch = blk * bs + c;
-      const long long rows = (long long)rb.slot[e] * K;
-      float x[4], b4[4];
-      load_v<4>(proj + (long long)e * ldp + x_off + ch, x);
+  // a thread keeps its 4 channels (one pass per 1024) and walks the entries
+  const int quads = kp / 4, span = min(quads, 256), rstep = 256 / span;
+  for (int cq = tid % span; cq < quads && tid < rstep * span; cq += span) {
+    const int c = cq * 4, ch = blk * bs + c;
+    const bool in = c < bs;
+    float taps[KT > 0 ? KT : 1][4], b4[4];
+    if (in) {
       load_v<4>(cb + ch, b4);
 #pragma unroll
-      for (int q = 0; q < 4; ++q) acc[q] = b4[q] + to_f(cw[(long long)(ch + q) * K + K - 1]) * x[q];
-#pragma unroll 4
-      for (int j = 1; j < K; ++j) {
-        if (j > p) break;
-        float v[4];
-        load_v<4>(ring + (rows + (p - j) % K) * W + ch, v);
+      for (int j = 0; j < KT; ++j)
 #pragma unroll
-        for (int q = 0; q < 4; ++q) acc[q] += to_f(cw[(long long)(ch + q) * K + K - 1 - j]) * v[q];
-      }
-      if (c >= o0 && c < o0 + DC) store_v<4>(ring + (rows + p % K) * W + ch, x);
+        for (int q = 0; q < 4; ++q) taps[j][q] = to_f(cw[(long long)(ch + q) * KT + KT - 1 - j]);
     }
-    store_v<4>(reinterpret_cast<__nv_bfloat16*>(Us + r * pitch) + c, acc);
+#pragma unroll 4
+    for (int r = tid / span; r < 16; r += rstep) {
+      const int e = e0 + r;
+      float acc[4] = {0.f, 0.f, 0.f, 0.f};
+      const int p = in && e < rb.E ? rb.pos0[e] : -1;
+      if (p >= 0) {
+        const long long rows = (long long)rb.slot[e] * K;
+        float x[4];
+        load_v<4>(proj + (long long)e * ldp + x_off + ch, x);
+        if constexpr (KT > 0) {
+          float v[KT][4];
+#pragma unroll
+          for (int j = 1; j < KT; ++j) {
+            v[j][0] = v[j][1] = v[j][2] = v[j][3] = 0.f;
+            if (j <= p) load_v<4>(ring + (rows + (p - j) % KT) * W + ch, v[j]);
+          }
+#pragma unroll
+          for (int q = 0; q < 4; ++q) {
+            acc[q] = b4[q] + taps[0][q] * x[q];
+#pragma unroll
+            for (int j = 1; j < KT; ++j) acc[q] += taps[j][q] * v[j][q];
+          }
+        } else {
+#pragma unroll
+          for (int q = 0; q < 4; ++q) acc[q] = b4[q] + to_f(cw[(long long)(ch + q) * K + K - 1]) * x[q];
+          for (int j = 1; j < K && j <= p; ++j) {
+            float v[4];
+            load_v<4>(ring + (rows + (p - j) % K) * W + ch, v);
+#pragma unroll
+            for (int q = 0; q < 4; ++q) acc[q] += to_f(cw[(long long)(ch + q) * K + K - 1 - j]) * v[q];
+          }
+        }
+        if (c >= o0 && c < o0 + DC) store_v<4>(ring + (rows + p % K) * W + ch, x);
+      }
+      store_v<4>(reinterpret_cast<__nv_bfloat16*>(Us + r * pitch) + c, acc);
+    }
   }
   cp_async_wait<0>();
   __syncthreads();
@@ -952,16 +992,27 @@ TB_API int tb_rglru(int dtype, const void* proj, long long ldp, int x_off, int y
     if (one) {
       const size_t smem = (size_t)(16 + 2 * DC) * pitch;
       if (smem <= 200 * 1024) {
-        static DeviceOnce once;
-        if (once.first() && cudaFuncSetAttribute(rglru_step_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess)
-          return -5;
         const dim3 grid(blocks * ((bs + DC - 1) / DC), (E + 15) / 16);
-        return launch_pdl(rglru_step_kernel, grid, dim3(256), smem, stream, (const bf*)proj, ldp, x_off, y_off, (const bf*)conv_w,
-                          (const bf*)conv_b, (const bf*)ra, (const bf*)rab, (const bf*)ri, (const bf*)rib, (const bf*)lam, rb, W,
-                          bs, K, state, ring, (bf*)out) == cudaSuccess ? 0 : -5;
+#define STEP(KT)                                                                                                              \
+  {                                                                                                                           \
+    static DeviceOnce once;                                                                                                   \
+    if (once.first() && cudaFuncSetAttribute(rglru_step_kernel<KT>, cudaFuncAttributeMaxDynamicSharedMemorySize,              \
+                                             200 * 1024) != cudaSuccess) return -5;                                           \
+    return launch_pdl(rglru_step_kernel<KT>, grid, dim3(256), smem, stream, (const bf*)proj, ldp, x_off, y_off,               \
+                      (const bf*)conv_w, (const bf*)conv_b, (const bf*)ra, (const bf*)rab, (const bf*)ri, (const bf*)rib,     \
+                      (const bf*)lam, rb, W, bs, K, state, ring, (bf*)out) == cudaSuccess ? 0 : -5;                           \
+  }
+        switch (K) {
+          case 2: STEP(2)
+          case 3: STEP(3)
+          case 4: STEP(4)
+          default: STEP(0)
+        }
+#undef STEP
       }
     } else if (tiles > 0) {
-      const size_t smem = (size_t)(LT + 2 * LC) * pitch + 2 * LT * (LC + 1) * 4;
+      const size_t ub = (size_t)(LT * pitch > 2 * LT * (LC + 1) * 4 ? LT * pitch : 2 * LT * (LC + 1) * 4);
+      const size_t smem = 2 * ub + (size_t)2 * LC * pitch;
       if (smem <= 220 * 1024) {
         static DeviceOnce once;
         if (once.first() && cudaFuncSetAttribute(rglru_tile_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024) != cudaSuccess)
