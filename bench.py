@@ -120,7 +120,15 @@ def main() -> int:
                     help="comma list. baseline = the same step on the in-repo baseline (N > 1: NCCL collectives; "
                          "N = 1: stock PyTorch ops instead of this package's kernels) -> vs_baseline; same_mb = "
                          "micro-batch 2 x 4 accumulation steps at every N, the like-for-like scaling point")
-    args = ap.parse_args()
+    ap.add_argument("--workload", default="sft", choices=["sft", "stack_serving"],
+                    help="sft: the headline step; stack_serving: prefill and decode throughput of layer-stack models beside "
+                         "the closest uniform decoder (one GPU, `tunix_b200/generate/bench_stack.py`)")
+    args, rest = ap.parse_known_args()
+    if args.workload == "stack_serving":          # its own options: --models, --prefill-len, --decode-seqs, ...
+        from tunix_b200.generate import bench_stack
+        return bench_stack.main(rest)
+    if rest:
+        ap.error(f"unrecognized arguments: {' '.join(rest)}")
     if args.impl == "reference":
         return reference_arm(args)
 

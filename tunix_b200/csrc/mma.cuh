@@ -29,6 +29,18 @@ __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commi
 template <int N>
 __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
+// Walks the cells (row, column) tid, tid + threads, ... of a row-major grid with `cols` columns: no division per step.
+struct GridWalk {
+  int r, c, dr, dc, cols;
+  __device__ __forceinline__ GridWalk(int tid, int threads, int cols_)
+      : r(tid / cols_), c(tid % cols_), dr(threads / cols_), dc(threads % cols_), cols(cols_) {}
+  __device__ __forceinline__ void next() {
+    c += dc;
+    r += dr;
+    if (c >= cols) { c -= cols; ++r; }
+  }
+};
+
 // v = hi + lo with both parts bf16: a product with hi and one with lo carries 16 bits of v's mantissa
 __device__ __forceinline__ void split_bf16(float v, __nv_bfloat16& hi, __nv_bfloat16& lo) {
   hi = __float2bfloat16(v);

@@ -78,10 +78,24 @@ __device__ __forceinline__ void store_v(__nv_bfloat16* p, const float (&v)[V]) {
 // The same functions for kernels that only bf16 models run: hardware exponential and division (relative error of a few
 // units in the last place), which is far below the rounding of their bf16 inputs and outputs. quick_expm1 keeps its relative
 // accuracy near zero (Taylor series there), as the decays of a recurrence need it.
-__device__ __forceinline__ float quick_sigmoid(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
+__device__ __forceinline__ float quick_exp(float z) {
+  float r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(z * 1.4426950408889634f));
+  return r;
+}
+__device__ __forceinline__ float quick_sigmoid(float z) {
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + quick_exp(-z)));
+  return r;
+}
 __device__ __forceinline__ float quick_expm1(float z) {
   const float t = z * fmaf(z, fmaf(z, fmaf(z, fmaf(z, fmaf(z, fmaf(z, 1.f / 5040.f, 1.f / 720.f), 1.f / 120.f), 1.f / 24.f), 1.f / 6.f), 0.5f), 1.f);
-  return fabsf(z) < 0.3f ? t : __expf(z) - 1.f;
+  return fabsf(z) < 0.3f ? t : quick_exp(z) - 1.f;
+}
+__device__ __forceinline__ float quick_sqrt(float z) {
+  float r;
+  asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(z));
+  return r;
 }
 __device__ __forceinline__ float quick_gelu_tanh(float z) {
   // 0.5 z (1 + tanh(y)) = z sigmoid(2 y)

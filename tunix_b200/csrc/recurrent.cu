@@ -133,13 +133,14 @@ struct Tiles {
 };
 
 // u [n, W] -> H, P fp32 [n, W], and the tiles' last rows in LH, LP fp32 [tiles, W]
+template <int KP>       // block size rounded up to 16, or 0 for a run-time value
 __global__ void __launch_bounds__(256, 2)
 rglru_tile_kernel(const __nv_bfloat16* __restrict__ u, const __nv_bfloat16* __restrict__ ra,
                   const __nv_bfloat16* __restrict__ ba, const __nv_bfloat16* __restrict__ ri,
                   const __nv_bfloat16* __restrict__ bi, const __nv_bfloat16* __restrict__ lam, Ragged rb, Tiles tl, int W,
                   int bs, float* __restrict__ H, float* __restrict__ P, float* __restrict__ LH, float* __restrict__ LP) {
   extern __shared__ __align__(16) uint8_t smem[];
-  const int kp = (bs + 15) & ~15;                       // contraction length, zero-padded
+  const int kp = KP > 0 ? KP : (bs + 15) & ~15;         // contraction length, zero-padded
   const int pitch = kp * 2 + 16;                        // bytes per row
   const int ubytes = max(LT * pitch, 2 * LT * (LC + 1) * 4);   // one buffer: a u tile, later the scan's a and b
   uint8_t* Ws = smem + 2 * ubytes;                      // [2 * LC] rows: LC of ra, LC of ri
@@ -154,13 +155,14 @@ rglru_tile_kernel(const __nv_bfloat16* __restrict__ u, const __nv_bfloat16* __re
   const int chunks = kp / 8;
   const uint32_t ws = smem_u32(Ws);
   const int tile_end = min(tl.count, ((int)blockIdx.y + 1) * LTPC);
+  const GridWalk walk(tid, 256, chunks);
   auto load_u = [&](int tile) {
     const int t0 = tl.t0[tile], nt = min(LT, rb.cu[tl.ent[tile] + 1] - t0);
     const uint32_t dst = smem_u32(smem) + (tile & 1) * ubytes;
-    for (int i = tid; i < LT * chunks; i += 256) {
-      const int r = i / chunks, c = i - r * chunks;
-      const bool ok = r < nt && c * 8 < bs;
-      cp_async16(dst + r * pitch + c * 16, u + (ok ? (long long)(t0 + r) * W + (long long)blk * bs + c * 8 : 0), ok ? 16 : 0);
+    const __nv_bfloat16* src = u + (long long)t0 * W + blk * bs;
+    for (GridWalk g = walk; g.r < LT; g.next()) {
+      const bool ok = g.r < nt && g.c * 8 < bs;
+      cp_async16(dst + g.r * pitch + g.c * 16, ok ? src + (long long)g.r * W + g.c * 8 : u, ok ? 16 : 0);
     }
     cp_async_commit();
   };
@@ -219,7 +221,7 @@ rglru_tile_kernel(const __nv_bfloat16* __restrict__ u, const __nv_bfloat16* __re
           const float em = quick_expm1(quick_sigmoid(r[j][q] + s_ba[c]) * s_sp[c]);      // a - 1
           const float uv = to_f(*reinterpret_cast<const __nv_bfloat16*>(Us + t * pitch + (o0 + c) * 2));
           av = 1.f + em;
-          bv = sqrtf(-em * (2.f + em)) * quick_sigmoid(g[j][q] + s_bi[c]) * uv;
+          bv = quick_sqrt(-em * (2.f + em)) * quick_sigmoid(g[j][q] + s_bi[c]) * uv;
         }
         r[j][q] = av;
         bvs[j][q] = bv;
@@ -250,14 +252,16 @@ rglru_tile_kernel(const __nv_bfloat16* __restrict__ u, const __nv_bfloat16* __re
     float cp = 1.f, chn = 0.f;
     for (int j = 0; j < sg; ++j) { chn = segA[j][c] * chn + segB[j][c]; cp *= segA[j][c]; }
     if (o0 + c < bs) {
-      const long long col = (long long)blk * bs + o0 + c;
+      const int col = blk * bs + o0 + c;
+      const long long first = (long long)(t0 + sg * SEG) * W + col;
+      float *hp = H + first, *pp = P + first;
 #pragma unroll
-      for (int t = 0; t < SEG; ++t) {
+      for (int t = 0; t < SEG; ++t, hp += W, pp += W) {
         const int tt = sg * SEG + t;
         if (tt < nt) {
           const float h = hb[t] + pa[t] * chn, p = pa[t] * cp;
-          H[(long long)(t0 + tt) * W + col] = h;
-          P[(long long)(t0 + tt) * W + col] = p;
+          *hp = h;
+          *pp = p;
           if (tt == nt - 1) {
             LH[(long long)tile * W + col] = h;
             LP[(long long)tile * W + col] = p;
@@ -653,6 +657,19 @@ mlstm_step_kernel(const T* __restrict__ proj, long long ldp, int q_off, int k_of
   }
 }
 
+// gates [n, 2 * heads], in place: pre-activations -> log input gate i and log forget gate f
+template <typename T>
+__global__ void mlstm_gates_kernel(float* __restrict__ gates, const T* __restrict__ ib, const T* __restrict__ fb, float cap,
+                                   int n, int heads) {
+  pdl_trigger();
+  pdl_wait();
+  for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < n * 2 * heads; i += gridDim.x * blockDim.x) {
+    const int h = i % (2 * heads);
+    const float z = cap * tanhf((gates[i] + to_f(h < heads ? ib[h] : fb[h - heads])) / cap);
+    gates[i] = h < heads ? z : log_sigmoid(z);
+  }
+}
+
 // ---- bf16, prompt portions: chunks of ML tokens on tensor cores
 // With F the running sum of f inside a chunk, g_s = i_s - F_s and M_t = max(m_prev, max_{s <= t} g_s), the recurrence above
 // unrolls to  m_t = F_t + M_t,
@@ -668,9 +685,8 @@ constexpr int MPP = ML * 2 + 16;        // row pitch of the [ML, ML] weight tile
 struct MlstmSmem {
   int pitch, q, k, v, wv, p, s, gate, total;            // byte offsets
 };
-__host__ __device__ inline MlstmSmem mlstm_smem(int dk) {
-  MlstmSmem L;
-  const int kp = (dk + 15) & ~15;
+__host__ __device__ constexpr MlstmSmem mlstm_smem(int kp) {
+  MlstmSmem L{};
   L.pitch = kp * 2 + 16;
   L.q = 0;
   L.k = L.q + ML * L.pitch;
@@ -683,14 +699,14 @@ __host__ __device__ inline MlstmSmem mlstm_smem(int dk) {
   return L;
 }
 
-template <int MT>       // 16-row tiles of S per warp: dk <= 128 * MT
+template <int KP>       // key size, zero-padded
 __global__ void __launch_bounds__(256, 2)
 mlstm_chunk_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int q_off, int k_off, int v_off,
-                   const float* __restrict__ gates, const __nv_bfloat16* __restrict__ ib, const __nv_bfloat16* __restrict__ fb,
-                   float cap, Ragged rb, int heads, int dk, int dv, float* __restrict__ Sg, float* __restrict__ Ng,
+                   const float* __restrict__ gates, Ragged rb, int heads, int dk, int dv, float* __restrict__ Sg, float* __restrict__ Ng,
                    float* __restrict__ Mg, float* __restrict__ out) {
   extern __shared__ __align__(16) uint8_t smem[];
-  const MlstmSmem L = mlstm_smem(dk);
+  constexpr MlstmSmem L = mlstm_smem(KP);
+  constexpr int mtiles = KP / 16, MT = (mtiles + 7) / 8;        // 16-row tiles of S, and per warp
   const uint32_t sb = smem_u32(smem);
   float* G = reinterpret_cast<float*>(smem + L.gate);   // g_s
   float* Mx = G + ML;                                   // M_t
@@ -706,25 +722,24 @@ mlstm_chunk_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int q_
   const int p0 = rb.pos0[e], t0 = rb.cu[e], len = rb.cu[e + 1] - t0;
   if (p0 < 0 || len <= 0) return;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, li = lane >> 3, lr = lane & 7;
-  const int kp = (dk + 15) & ~15, kchunks = kp / 8, mtiles = kp / 16;
   const int c0 = sl * MV, nc = min(MV, dv - c0);
   const long long slot = rb.slot[e];
   float* Sh = Sg + (slot * heads + hd) * (long long)dk * dv + c0;
   float* Nh = Ng + ((slot * heads + hd) * slices + sl) * (long long)dk;
   float* Mh = Mg + (slot * heads + hd) * slices + sl;
-  const float bi = to_f(ib[hd]), bf = to_f(fb[hd]);
   const float qscale = 1.f / sqrtf((float)dk);
 
+  const GridWalk walk(tid, 256, KP / 8);
   auto load = [&](int ch) {
     const int rows = min(ML, len - ch * ML);
     const __nv_bfloat16* base = proj + (long long)(t0 + ch * ML) * ldp;
-    for (int i = tid; i < ML * kchunks; i += 256) {
-      const int r = i / kchunks, c = i - r * kchunks;
-      const bool ok = r < rows && c * 8 < dk;
-      const long long src = ok ? (long long)r * ldp + hd * dk + c * 8 : 0;
-      const uint32_t d = r * L.pitch + c * 16;
-      cp_async16(sb + L.q + d, base + q_off + src, ok ? 16 : 0);
-      cp_async16(sb + L.k + d, base + k_off + src, ok ? 16 : 0);
+    const __nv_bfloat16 *qs = base + q_off + hd * dk, *ks = base + k_off + hd * dk;
+    for (GridWalk g = walk; g.r < ML; g.next()) {
+      const bool ok = g.r < rows && g.c * 8 < dk;
+      const long long src = ok ? g.r * ldp + g.c * 8 : 0;
+      const uint32_t d = g.r * L.pitch + g.c * 16;
+      cp_async16(sb + L.q + d, qs + src, ok ? 16 : 0);
+      cp_async16(sb + L.k + d, ks + src, ok ? 16 : 0);
     }
     for (int i = tid; i < ML * (MV / 8); i += 256) {
       const int r = i / (MV / 8), c = i - r * (MV / 8);
@@ -791,8 +806,8 @@ mlstm_chunk_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int q_
         ii[j] = -INFINITY;
         if (t < rows) {
           const float* gr = gates + (long long)(t0 + ch * ML + t) * 2 * heads + hd;
-          ii[j] = cap * tanhf((gr[0] + bi) / cap);
-          f[j] = log_sigmoid(cap * tanhf((gr[heads] + bf) / cap));
+          ii[j] = gr[0];
+          f[j] = gr[heads];
         }
       }
       float run = f[0] + f[1];
@@ -816,9 +831,9 @@ mlstm_chunk_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int q_
       const int t = 2 * lane;
       G[t] = g0; G[t + 1] = g1;
       Mx[t] = M0; Mx[t + 1] = M1;
-      Ct[t] = expf(m_prev - M0); Ct[t + 1] = expf(m_prev - M1);
+      Ct[t] = quick_exp(m_prev - M0); Ct[t + 1] = quick_exp(m_prev - M1);
       Wt[t] = expf(g0 - ML_); Wt[t + 1] = expf(g1 - ML_);
-      Em[t] = expf(-(F0 + M0)); Em[t + 1] = expf(-(F1 + M1));
+      Em[t] = quick_exp(-(F0 + M0)); Em[t + 1] = quick_exp(-(F1 + M1));
       if (lane == 0) { s_m = FL + ML_; s_decay = expf(m_prev - ML_); }
     }
     // P = Q K^T (this warp: 16 tokens x 32 keys; key tiles past the diagonal are skipped)
@@ -850,8 +865,8 @@ mlstm_chunk_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int q_
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int s = kn + j * 8 + 2 * (lane & 3);
-        const float w0 = s <= t ? P[j][2 * h] * qscale * __expf(G[s] - M) : 0.f;
-        const float w1 = s + 1 <= t ? P[j][2 * h + 1] * qscale * __expf(G[s + 1] - M) : 0.f;
+        const float w0 = s <= t ? P[j][2 * h] * qscale * quick_exp(G[s] - M) : 0.f;
+        const float w1 = s + 1 <= t ? P[j][2 * h + 1] * qscale * quick_exp(G[s + 1] - M) : 0.f;
         sum += w0 + w1;
         *reinterpret_cast<uint32_t*>(smem + L.p + t * MPP + s * 2) = pack_bf16(w0, w1);
       }
@@ -1014,9 +1029,6 @@ TB_API int tb_rglru(int dtype, const void* proj, long long ldp, int x_off, int y
       const size_t ub = (size_t)(LT * pitch > 2 * LT * (LC + 1) * 4 ? LT * pitch : 2 * LT * (LC + 1) * 4);
       const size_t smem = 2 * ub + (size_t)2 * LC * pitch;
       if (smem <= 220 * 1024) {
-        static DeviceOnce once;
-        if (once.first() && cudaFuncSetAttribute(rglru_tile_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024) != cudaSuccess)
-          return -5;
         Tiles tl{tile_t0, tile_ent, tiles};
         const long long want = ((long long)n * (W / 4) + 255) / 256;
         const dim3 flat((unsigned)(want < 148 * 16 ? want : 148 * 16));
@@ -1037,9 +1049,17 @@ TB_API int tb_rglru(int dtype, const void* proj, long long ldp, int x_off, int y
                              (const bf*)conv_w, (const bf*)conv_b, (const float*)ring, rb, W, K, (bf*)u);
         }
 #undef CONV
-        if (err == cudaSuccess)
-          err = launch_pdl(rglru_tile_kernel, gtile, dim3(256), smem, stream, (const bf*)u, (const bf*)ra, (const bf*)rab,
-                           (const bf*)ri, (const bf*)rib, (const bf*)lam, rb, tl, W, bs, A, B, LH, LP);
+#define TILE(KP)                                                                                                              \
+  {                                                                                                                           \
+    static DeviceOnce once;                                                                                                   \
+    if (once.first() && cudaFuncSetAttribute(rglru_tile_kernel<KP>, cudaFuncAttributeMaxDynamicSharedMemorySize,              \
+                                             220 * 1024) != cudaSuccess) return -5;                                           \
+    err = launch_pdl(rglru_tile_kernel<KP>, gtile, dim3(256), smem, stream, (const bf*)u, (const bf*)ra, (const bf*)rab,       \
+                     (const bf*)ri, (const bf*)rib, (const bf*)lam, rb, tl, W, bs, A, B, LH, LP);                              \
+  }
+        if (err != cudaSuccess) return -5;
+        if (kp == 64) TILE(64) else if (kp == 128) TILE(128) else if (kp == 256) TILE(256) else TILE(0)
+#undef TILE
         if (err == cudaSuccess)
           err = launch_pdl(rglru_chain_kernel, dim3((W + 63) / 64, E), dim3(64), 0, stream, LH, (const float*)LP, (const bf*)proj,
                            ldp, x_off, rb, first_tile, W, K, state, ring);
@@ -1077,8 +1097,8 @@ TB_API int tb_mlstm_slices(int dv) { return (dv + MV - 1) / MV; }
 
 // q, k, v: columns of proj [n, ldp]; gates fp32 [n, 2 * heads] = (W_i h, W_f h) without bias.
 // S fp32 [slots, heads, dk, dv], N fp32 [slots, heads, slices, dk], M fp32 [slots, heads, slices]; out fp32 [n, heads, dv].
-// `one`: every entry is one token. `chunked`: bf16 portions take the tensor-core form where the sizes allow.
-TB_API int tb_mlstm(int dtype, const void* proj, long long ldp, int q_off, int k_off, int v_off, const float* gates,
+// `one`: every entry is one token. `chunked` (overwrites gates): bf16 portions take the tensor-core form where the sizes allow.
+TB_API int tb_mlstm(int dtype, const void* proj, long long ldp, int q_off, int k_off, int v_off, float* gates,
                     const void* ib, const void* fb, float cap, const int* cu, const int* slot, const int* pos0,
                     const int* ent, int E, int n, int heads, int dk, int dv, float* S, float* N, float* M, float* out, int one,
                     int chunked, cudaStream_t stream) {
@@ -1096,15 +1116,25 @@ TB_API int tb_mlstm(int dtype, const void* proj, long long ldp, int q_off, int k
   }
   if (dtype == 0 && chunked && dk <= 256 && dk % 8 == 0 && dv % 8 == 0 && q_off % 8 == 0 && k_off % 8 == 0 && v_off % 8 == 0 &&
       ldp % 8 == 0 && (reinterpret_cast<uintptr_t>(proj) & 15) == 0) {
-    const size_t smem = mlstm_smem(dk).total;
-    static DeviceOnce once;
-    if (once.first() &&
-        (cudaFuncSetAttribute(mlstm_chunk_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 225 * 1024) != cudaSuccess ||
-         cudaFuncSetAttribute(mlstm_chunk_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 225 * 1024) != cudaSuccess))
-      return -5;
-    cudaError_t err = dk <= 128 ? launch_pdl(mlstm_chunk_kernel<1>, grid, dim3(256), smem, stream, ARGS(__nv_bfloat16))
-                                : launch_pdl(mlstm_chunk_kernel<2>, grid, dim3(256), smem, stream, ARGS(__nv_bfloat16));
-    return err == cudaSuccess ? 0 : -5;
+    if ((long long)n * 2 * heads > (1 << 30)) return -2;
+    const int want = (n * 2 * heads + 255) / 256;
+    cudaError_t err = launch_pdl(mlstm_gates_kernel<__nv_bfloat16>, dim3(want < 148 * 8 ? want : 148 * 8), dim3(256), 0, stream, gates,
+                                 (const __nv_bfloat16*)ib, (const __nv_bfloat16*)fb, cap, n, heads);
+    if (err != cudaSuccess) return -5;
+#define CHUNK(KP)                                                                                                             \
+  {                                                                                                                           \
+    static DeviceOnce once;                                                                                                   \
+    if (once.first() && cudaFuncSetAttribute(mlstm_chunk_kernel<KP>, cudaFuncAttributeMaxDynamicSharedMemorySize,             \
+                                             mlstm_smem(KP).total) != cudaSuccess) return -5;                                 \
+    return launch_pdl(mlstm_chunk_kernel<KP>, grid, dim3(256), mlstm_smem(KP).total, stream, (const __nv_bfloat16*)proj, ldp, \
+                      q_off, k_off, v_off, (const float*)gates, rb, heads, dk, dv, S, N, M, out) == cudaSuccess ? 0 : -5;     \
+  }
+    if (dk <= 32) CHUNK(32)
+    if (dk <= 64) CHUNK(64)
+    if (dk <= 128) CHUNK(128)
+    if (dk <= 192) CHUNK(192)
+    CHUNK(256)
+#undef CHUNK
   }
   const size_t smem = ((size_t)dk * (MV + 3) + MV * 9) * 4;
   if (smem > 200 * 1024) return -2;

@@ -47,7 +47,11 @@ def _time(fn, iters: int, warmup: int = 3, flush: bool = True):
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("kernel", choices=["gemm", "attn_fwd", "attn_bwd", "rmsnorm", "adamw", "logsoftmax", "sample",
-                                       "glu", "moe", "paged_decode", "lm_head", "lm_head_bwd", "lora"])
+                                       "glu", "moe", "paged_decode", "lm_head", "lm_head_bwd", "lora", "stack"])
+    ap.add_argument("--model", default="roluzen_8b", help="stack: preset whose sizes are measured")
+    ap.add_argument("--only", default="", help="stack: comma list of kernels")
+    ap.add_argument("--decode-batch", type=int, default=64, help="stack: sequences of a decode step")
+    ap.add_argument("--decode-ctx", type=int, default=1024, help="stack: their context")
     ap.add_argument("--m", type=int, default=8192)
     ap.add_argument("--n", type=int, default=4096)
     ap.add_argument("--k", type=int, default=4096)
@@ -203,6 +207,11 @@ def main(argv=None) -> int:
         gb = 2.0 * Bn * ctx * KH * H * 2 / ms / 1e6
         out.update(shape=[Bn, ctx, N, KH, H], ms=ms, gbs=gb, frac_of_peak=gb / peak_gb,
                    split_tokens=args.split or K.decode_split_tokens(Bn, KH, args.max_ctx or ctx))
+    elif args.kernel == "stack":
+        from tunix_b200.ops import bench_stack_kernels
+        bench_stack_kernels.run(args, (peak_tf, peak_gb, src), _time)
+        _lib.raise_if_kernel_error()
+        return 0
     elif args.kernel == "moe":
         from tunix_b200.ops import moe
         T, E, k, D, Fd = args.rows, args.experts, args.topk, args.dim, args.ffn

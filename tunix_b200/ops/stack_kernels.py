@@ -110,7 +110,8 @@ def rglru(proj, x_off: int, y_off: int, m, rb: RaggedBatch, state: dict, plain: 
 
 def mlstm(proj, q_off: int, k_off: int, v_off: int, gates, i_bias, f_bias, cap: float, rb: RaggedBatch, heads: int, dk: int,
           dv: int, state: dict, plain: bool = False) -> torch.Tensor:
-    """Matrix memory over a ragged batch; gates fp32 [n, 2 heads]. Returns o fp32 [n, heads, dv]. `plain`: the token by
+    """Matrix memory over a ragged batch; gates fp32 [n, 2 heads] (may be overwritten). Returns o fp32
+    [n, heads, dv]. `plain`: the token by
     token kernel of the 32-bit path, also for bf16."""
     n = proj.shape[0]
     assert gates.dtype == torch.float32 and gates.is_contiguous() and gates.shape == (n, 2 * heads)
