@@ -1,0 +1,174 @@
+"""Layer-stack models without a GPU: configuration reader, weight names, registry, cache layout, ragged batches, the bias
+buckets, and the oracle's own consistency (its closed forms against its recurrences)."""
+import json
+import math
+
+import pytest
+import torch
+
+from tests import roluzen_oracle as O
+from tests import stack_cases as C
+
+
+@pytest.mark.parametrize("name", sorted(C.CASES))
+def test_checkpoint_round_trip(tmp_path, name):
+    from safetensors.torch import load_file
+    from tunix_b200.models.automodel import AutoModel
+    from tunix_b200.models.safetensors_saver import save_lora_merged_model_as_safetensors
+    from tunix_b200.models.stack import StackModel
+    cfg = C.CASES[name]
+    src = C.write(tmp_path / "roluzen-tiny", cfg, C.weights(cfg))      # a directory name that could be taken for a preset
+    model, path = AutoModel.from_pretrained(src, model_source="local")
+    assert isinstance(model, StackModel) and path == src
+    assert model.config.runs() == O.layer_runs(cfg) and model.config.norm_eps == cfg["norm"]["eps"]
+    save_lora_merged_model_as_safetensors(model, str(tmp_path / "out"), source_dir=src)
+    a, b = load_file(src + "/model.safetensors"), load_file(str(tmp_path / "out" / "model.safetensors"))
+    assert a.keys() == b.keys() and all(torch.equal(a[k], b[k]) for k in a)
+    again, _ = AutoModel.from_pretrained("anything", model_source="local", model_path=str(tmp_path / "out"), dtype=torch.float32)
+    assert again.embed_tokens.dtype == torch.float32
+
+
+def test_constants_come_from_config_json(tmp_path):
+    from tunix_b200.models.hf_config import config_from_hf
+    cfg = C.CASES["mixed"]
+    src = C.write(tmp_path / "m", cfg, C.weights(cfg, buckets=14))
+    c = config_from_hf(src)
+    left, right = c.layer_specs[1].mixer.left, c.layer_specs[1].mixer.right
+    want = cfg["layers"][1]["mixer"]
+    assert (left.scale, left.bias_max, left.window, left.keep_first) == (want["left"]["scale"], 40, 20, 3)
+    assert left.buckets == 14                                          # told by the tensor's shape only
+    assert (right.gate_cap, right.dim, right.vdim) == (9.0, 24, 40)
+    assert c.layer_specs[2].ff is None and c.layer_specs[3].mixer.conv == 2 and c.streams == 3 and c.loop == (1, 3, 2)
+    with pytest.raises(ValueError, match="mixer"):
+        config_from_hf(dict(cfg, layers=[dict(cfg["layers"][0], type="other")]))
+    with pytest.raises(ValueError, match="feed-forward"):
+        config_from_hf(dict(cfg, layers=[dict(cfg["layers"][0], mlp={"kind": "sparse", "ff": 8})]))
+
+
+def test_cache_layout_is_per_pass():
+    from tunix_b200.models.hf_config import config_from_hf
+    c = config_from_hf(C.CASES["mixed"])
+    assert c.runs() == [0, 1, 2, 1, 2, 3]
+    assert c.kv_rows() == [None, (32, 48), (32, 48), (32, 48), (32, 48), None]
+    states = c.state_shapes()
+    assert states[0] == {"s": (80,), "ring": (4, 80)} and states[5] == {"s": (80,), "ring": (2, 80)}
+    assert states[1] == {"S": (2, 24, 40), "n": (2, 2, 24), "m": (2, 2)}
+
+
+def test_pool_and_states_on_cpu():
+    from tunix_b200.generate.engine import PagePool
+    from tunix_b200.models.hf_config import config_from_hf
+    c = config_from_hf(C.CASES["mixed"])
+    pool = PagePool(c, 6, 16, 2, 4, "cpu", torch.float32, prefix_caching=False)
+    assert pool.k[0] is None and pool.k[1].shape == (6, 16, 32) and pool.v[1].shape == (6, 16, 48)
+    assert pool.state[1]["S"].shape == (2, 2, 24, 40) and pool.state[1]["S"].dtype == torch.float32
+    assert pool.state.nbytes_per_slot() == 4 * (80 + 320 + 80 + 160 + 4 * (2 * 24 * 40 + 2 * 2 * 24 + 4))
+    pool.open(0, [1] * 20, 0)
+    pool.grow(0, 60)
+    assert len(pool.pages_of(0)) == 4
+    with pytest.raises(pool.Error):
+        pool.open(1, [1] * 60, 0)
+    pool.release(0)
+    pool.open(1, [1] * 60, 0)
+
+
+def test_registry_presets_and_names():
+    from tunix_b200.models import naming, registry
+    from tunix_b200.models.config import get_config
+    from tunix_b200.models.transformer import create_model
+    assert registry.get_family("roluzen").family == "roluzen" and registry.family_of_hf_id("x/Roluzen-2B").family == "roluzen"
+    assert naming.config_for("roluzen-2b") == get_config("roluzen_2b")
+    model = create_model(get_config("roluzen_tiny"), seed=3)
+    assert model.config.runs() == [0, 1, 2, 1, 2]
+    assert torch.equal(model.layers[0].hc1.mix, torch.eye(3)) and model.layers[1].mixer.right.f_proj.bias.eq(3).all()
+    with pytest.raises(ValueError, match="loop"):
+        get_config("roluzen_tiny").replace(loop=(2, 5, 1))
+    with pytest.raises(NotImplementedError):
+        model(torch.zeros(1, 1, dtype=torch.long), cache=[])
+
+
+@pytest.mark.parametrize("rows,far", [(11, 40), (16, 100), (8, 64), (7, 33), (32, 4096), (6, 12)])
+def test_distance_buckets(rows, far):
+    from tunix_b200.models.mixers import distance_buckets
+    got = distance_buckets(rows, far)
+    want = [O.distance_bucket(n, rows, far) for n in range(far + 1)]
+    # where the logarithm is an integer in exact arithmetic the two may round apart; nowhere else
+    for n, (a, b) in enumerate(zip(got.tolist(), want)):
+        if a != b:
+            half = rows // 2
+            x = math.log(n / half) / math.log(far / half) * (rows - half)
+            assert abs(x - round(x)) < 1e-9, n
+    assert got[far] == rows - 1 and O.distance_bucket(10 * far, rows, far) == rows - 1
+
+
+def test_ragged_batch_layout():
+    from tunix_b200.ops.ragged import RaggedBatch
+    rb = RaggedBatch.build([(3, 0, [5, 6, 7]), (1, 9, [8]), (0, 2, [1, 2])], "cpu")
+    assert rb.tokens.tolist() == [5, 6, 7, 8, 1, 2] and rb.cu.tolist() == [0, 3, 4, 6]
+    assert rb.slot.tolist() == [3, 1, 0] and rb.pos0.tolist() == [0, 9, 2] and rb.ent.tolist() == [0, 0, 0, 1, 2, 2]
+    assert not rb.decode
+    t0, ent, first, n = rb.tiles(2)
+    assert t0.tolist() == [0, 2, 3, 4] and ent.tolist() == [0, 0, 1, 2] and first.tolist() == [0, 2, 3] and n == 4
+    assert RaggedBatch.build([(0, 4, [1]), (2, 7, [3])], "cpu").decode
+
+
+def test_joint_weights_share_memory_and_follow_updates():
+    from tunix_b200.models.config import get_config
+    from tunix_b200.models.stack_exec import StackExecutor
+    from tunix_b200.models.transformer import create_model
+    model = create_model(get_config("roluzen_tiny"), seed=0)
+    ex = StackExecutor(model)
+    before = {k: v.data_ptr() for k, v in ex.w[1].items() if v is not None}
+    left = model.layers[1].mixer.left
+    n = left.q_proj.weight.shape[0]
+    assert left.k_proj.weight.data_ptr() == ex.w[1]["proj"][n:].data_ptr()
+    with torch.no_grad():
+        left.k_proj.weight.fill_(2.0)
+        left.rel.fill_(1.5)
+        model.layers[0].mixer.y_proj.bias.fill_(0.25)
+    ex.refresh()
+    assert {k: v.data_ptr() for k, v in ex.w[1].items() if v is not None} == before
+    assert ex.w[1]["proj"][n].eq(2).all() and ex.w[1]["bias"].eq(1.5).all() and ex.w[0]["proj_bias"][0] == 0.25
+    model.layers[1].mixer.left.q_proj.lora_a = torch.nn.Parameter(torch.zeros(1, 1))
+    with pytest.raises(NotImplementedError, match="adapters"):
+        ex.refresh()
+
+
+def test_oracle_memory_against_its_unrolled_sum():
+    """The token-by-token matrix memory of the oracle against the direct sum over all earlier tokens."""
+    torch.manual_seed(0)
+    T, m = 30, {"heads": 2, "dim": 6, "vdim": 5, "gate_cap": 7.0}
+    D = 16
+    w = {n: torch.randn(r, D, dtype=torch.float64) for n, r in (("q", 12), ("k", 12), ("v", 10), ("g", 10), ("i", 2), ("f", 2))}
+    w.update({"i.b": torch.randn(2).double(), "f.b": torch.randn(2).double() + 2, "norm": torch.ones(10).double(),
+              "o": torch.eye(10).double()})
+    h = torch.randn(T, D, dtype=torch.float64)
+    got = O.matrix_memory(w, "", h, m, 1e-6)
+    ig = 7 * torch.tanh((h @ w["i"].T + w["i.b"]) / 7)
+    F = torch.nn.functional.logsigmoid(7 * torch.tanh((h @ w["f"].T + w["f.b"]) / 7)).cumsum(0)
+    q, k, v = (h @ w["q"].T).view(T, 2, 6) / 6 ** 0.5, (h @ w["k"].T).view(T, 2, 6), (h @ w["v"].T).view(T, 2, 5)
+    out = torch.zeros(T, 2, 5, dtype=torch.float64)
+    for t in range(T):
+        for a in range(2):
+            lw = F[t, a] - F[:t + 1, a] + ig[:t + 1, a]
+            top = max(F[t, a].item(), lw.max().item())
+            s = torch.exp(lw - top) * (k[:t + 1, a] @ q[t, a])
+            out[t, a] = s @ v[:t + 1, a] / (max(abs(s.sum().item()), math.exp(-top)) + 1e-6)
+    want = O.rms(out, 1e-6).reshape(T, 10) * torch.sigmoid(h @ w["g"].T)
+    assert torch.allclose(got, want, atol=1e-9)
+
+
+def test_trace_runner_help_names_its_options():
+    import os
+    import subprocess
+    import sys
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    path = os.path.join(root, "bin", "trace_run")
+    assert os.access(path, os.X_OK)
+    out = subprocess.run([sys.executable, path, "--help"], capture_output=True, text=True).stdout
+    assert all(o in out for o in ("--model", "--dtype", "--out", "--max-tokens"))
+
+
+def test_configs_are_json():
+    for cfg in C.CASES.values():
+        assert json.loads(json.dumps(cfg)) == cfg

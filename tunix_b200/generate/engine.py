@@ -897,8 +897,8 @@ class StepSession:
             if req is None:
                 if not self._free:
                     raise RuntimeError(f"request {rid!r}: all {eng.max_running} slots are in use")
+                pool.open(self._free[-1], list(tokens), 0)
                 req = self._live[rid] = [self._free.pop(), 0]
-                pool.open(req[0], list(tokens), 0)
             else:
                 pool.grow(req[0], req[1] + len(tokens))
             if req[1] + len(tokens) > pool.max_pages * pool.page_size:
