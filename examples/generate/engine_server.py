@@ -9,6 +9,7 @@ interrupted:
 
     curl -s 127.0.0.1:8000/v1/completions -d '{"prompt": "hello", "max_tokens": 16}'"""
 import argparse
+import os
 import time
 from concurrent.futures import ThreadPoolExecutor
 
@@ -17,6 +18,7 @@ import torch
 
 from tunix_b200.common.configs import CacheConfig
 from tunix_b200.generate.engine import EngineServer, PagedEngine
+from tunix_b200.models.automodel import AutoModel
 from tunix_b200.models.config import ModelConfig
 from tunix_b200.models.transformer import create_model
 
@@ -41,10 +43,17 @@ class Tok:                      # the engine needs ids for bos / eos / pad and a
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--http", type=int, default=None, help="serve the OpenAI-style routes on this port afterwards")
+    ap.add_argument("--model", default=None, help="a preset with random weights (e.g. roluzen_2b) or a checkpoint directory")
     args = ap.parse_args()
     cfg = ModelConfig(family="qwen3", num_layers=4, vocab_size=4096, embed_dim=1024, hidden_dim=3072, num_heads=8, head_dim=128,
                       num_kv_heads=2, qk_norm=True, dtype=torch.bfloat16, max_position=1024)
-    model = create_model(cfg, device=torch.device("cuda"), seed=0)
+    if args.model is None:
+        model = create_model(cfg, device=torch.device("cuda"), seed=0)
+    else:
+        source = "local" if os.path.isdir(args.model) else "random"
+        model, _ = AutoModel.from_pretrained(args.model, model_source=source, model_path=args.model if source == "local" else None,
+                                             device="cuda", dtype=torch.bfloat16)
+        cfg = model.config
     engine = PagedEngine(model, Tok(), CacheConfig(1024, cfg.num_layers, cfg.num_kv_heads, cfg.head_dim), page_size=64,
                          max_running_requests=32, check_every=8)
     rng = np.random.default_rng(0)
@@ -66,7 +75,7 @@ def main():
         print("after the weight update:", toks.tolist(), [round(float(x), 3) for x in lps])
         if args.http is not None:
             from tunix_b200.generate.openai_server import serve
-            with serve(srv, Tok(), model_name="qwen3-random-init", port=args.http) as http:
+            with serve(srv, Tok(), model_name=args.model or "qwen3-random-init", port=args.http) as http:
                 print("serving on", http.url)
                 try:
                     while True:

@@ -1,0 +1,205 @@
+"""Distance-biased sliding-window attention with kept first tokens over the paged cache, in its three kernels (general, flash
+attention over pages, paged decode): against a dense restatement, with queries whose scores single out one key at an edge."""
+import math
+
+import pytest
+import torch
+
+from tests import roluzen_oracle as O
+from tests.test_stack_kernels_gpu import batch, rand, rel
+
+pytestmark = pytest.mark.gpu
+
+
+def dense(q, k, v, i0, scale, bias, size, keep):
+    """q [T, H, d] at positions i0.., k / v [P, G, *] of the whole sequence, bias [H, far + 1] -> [T, H, dv] in fp64."""
+    q, k, v, bias = (t.double().cpu() for t in (q, k, v, bias))
+    T, H, _ = q.shape
+    P, G, _ = k.shape
+    far = bias.shape[1] - 1
+    out = torch.zeros(T, H, v.shape[2], dtype=torch.float64)
+    for t in range(T):
+        i = i0 + t
+        js = [j for j in range(P) if O.visible(i, j, size or 10 ** 9, keep)]
+        dist = torch.tensor([min(i - j, far) for j in js])
+        for h in range(H):
+            g = h // (H // G)
+            s = k[js, g] @ q[t, h] * scale + bias[h, dist]
+            out[t, h] = torch.softmax(s, -1) @ v[js, g]
+    return out
+
+
+class Cache:
+    """Sequences of unequal length scattered over shuffled pages; what no sequence owns holds large values."""
+
+    def __init__(self, lens, G, dq, dv, dtype, page=64, seed=0, unit=False):
+        g = torch.Generator("cuda").manual_seed(seed)
+        pages = [-(-n // page) for n in lens]
+        total = sum(pages) + 2
+        self.k = torch.full((total, page, G * dq), 50.0, device="cuda", dtype=dtype)
+        self.v = torch.full((total, page, G * dv), 50.0, device="cuda", dtype=dtype)
+        perm = torch.randperm(total, generator=torch.Generator().manual_seed(seed)).tolist()
+        self.table = torch.full((len(lens) + 1, max(pages) + 1), -1, dtype=torch.int32)
+        self.seqs = []
+        for s, n in enumerate(lens):
+            own = [perm.pop() for _ in range(pages[s])]
+            self.table[s, :len(own)] = torch.tensor(own)
+            k = torch.randn(n, G, dq, device="cuda", generator=g)
+            k = (k / k.norm(dim=-1, keepdim=True) if unit else k).to(dtype)
+            v = torch.randn(n, G, dv, device="cuda", generator=g).to(dtype)
+            self.seqs.append((k, v))
+            for j in range(n):
+                self.k[own[j // page], j % page] = k[j].reshape(-1)
+                self.v[own[j // page], j % page] = v[j].reshape(-1)
+        self.table = self.table.cuda()
+        self.page = page
+
+
+def run(kind, cache, rb, q, sp, bias, split=0):
+    from tunix_b200.ops import kernels as K
+    from tunix_b200.ops import stack_kernels as SK
+    n = q.shape[0]
+    if kind == "general":
+        return SK.window_attn(q.reshape(n, -1), cache.k, cache.v, rb, cache.table, cache.page, sp, bias).view(n, sp.heads, sp.vdim)
+    kw = dict(scale=sp.scale, window=sp.window, keep_first=sp.keep_first, bias=bias)
+    if kind == "decode":
+        return K.paged_decode(q, cache.k, cache.v, cache.table, rb.slot, rb.pos0 + 1, num_kv_heads=sp.kv_heads, page_size=cache.page,
+                              max_ctx=cache.table.shape[1] * cache.page, split_tokens=split, **kw)
+    return K.attn_fwd_paged(q.reshape(n, -1).contiguous(), cache.k, cache.v, rb, cache.table, cache.page, num_heads=sp.heads,
+                            num_kv_heads=sp.kv_heads, head_dim=sp.dim, **kw).view(n, sp.heads, sp.vdim)
+
+
+def spec(H, G, dq, dv, window, keep, scale=0.2):
+    from tunix_b200.models.mixers import WindowAttentionSpec
+    return WindowAttentionSpec(heads=H, kv_heads=G, dim=dq, vdim=dv, scale=scale, bias_max=1, window=window, keep_first=keep)
+
+
+GENERAL = [("general", torch.float32, 4, 2, 12, 20), ("general", torch.bfloat16, 3, 1, 17, 9), ("general", torch.float32, 2, 2, 64, 512)]
+FLASH = [("flash", torch.bfloat16, 4, 2, 64, 64), ("flash", torch.bfloat16, 3, 1, 128, 128), ("flash", torch.bfloat16, 2, 2, 256, 256)]
+DECODE = [("decode", torch.bfloat16, 6, 2, 64, 64), ("decode", torch.bfloat16, 16, 1, 128, 128), ("decode", torch.bfloat16, 3, 3, 256, 256)]
+MASKS = [(20, 3), (64, 5), (65, 64), (63, 70), (200, 0), (0, 0), (1, 1), (130, 130)]
+
+
+def tol(dtype):
+    return 2e-6 if dtype == torch.float32 else 1.2e-2
+
+
+@pytest.mark.parametrize("window,keep", MASKS)
+@pytest.mark.parametrize("kind,dtype,H,G,dq,dv", GENERAL + FLASH)
+def test_portions(kind, dtype, H, G, dq, dv, window, keep):
+    """Portions of unequal requests at page and tile edges, down to two tokens, with a wide bias table."""
+    sp = spec(H, G, dq, dv, window, keep)
+    cache = Cache([300, 64, 130, 7], G, dq, dv, dtype)
+    bias = rand(H, 91, std=2.0)
+    parts = [(0, 120, 180), (1, 0, 64), (2, 128, 2), (3, 0, 7)]
+    rb = batch(parts)
+    q = rand(sum(n for _, _, n in parts), H, dq, dtype=dtype)
+    out = run(kind, cache, rb, q, sp, bias)
+    at = 0
+    for s, p, n in parts:
+        k, v = cache.seqs[s]
+        assert rel(out[at:at + n], dense(q[at:at + n], k[:p + n], v[:p + n], p, sp.scale, bias, window, keep)) < tol(dtype), s
+        at += n
+
+
+@pytest.mark.parametrize("window,keep", MASKS)
+@pytest.mark.parametrize("kind,dtype,H,G,dq,dv", GENERAL[:2] + DECODE)
+def test_single_tokens(kind, dtype, H, G, dq, dv, window, keep):
+    """Decoded tokens at positions around page edges, in every split of the context over CTAs; an idle slot gives zeros."""
+    sp = spec(H, G, dq, dv, window, keep)
+    lens = [1, 63, 64, 65, 129, 300, 22]
+    cache = Cache(lens, G, dq, dv, dtype, seed=3)
+    bias = rand(H, 91, std=2.0)
+    rb = batch([(s, n - 1, 1) for s, n in enumerate(lens)] + [(len(lens), 0, 1)])
+    rb.pos0[-1] = -1                                                    # idle
+    q = rand(len(lens) + 1, H, dq, dtype=dtype)
+    want = [dense(q[s:s + 1], k, v, lens[s] - 1, sp.scale, bias, window, keep) for s, (k, v) in enumerate(cache.seqs)]
+    for split in (0, 64, 128, 512):
+        out = run(kind, cache, rb, q, sp, bias, split)
+        for s, w in enumerate(want):
+            assert rel(out[s:s + 1], w) < tol(dtype), (s, split)
+        assert out[-1].abs().max() == 0
+        if kind == "general":
+            break
+
+
+def outstanding(cache, s, positions, targets, H, dq):
+    """Queries at `positions` that score far above everything else with the key at `targets`."""
+    k, _ = cache.seqs[s]
+    G = k.shape[1]
+    q = torch.stack([torch.stack([k[j, h // (H // G)].float() / k[j, h // (H // G)].float().norm() for h in range(H)]) for j in targets])
+    return (q * 300.0).to(k.dtype)
+
+
+EDGES = [(20, 3), (64, 5), (70, 64), (129, 66), (128, 1)]
+
+
+@pytest.mark.parametrize("window,keep", EDGES)
+@pytest.mark.parametrize("kind,dtype,H,G,dq,dv,decoded", [(*c, d) for d, cs in ((False, GENERAL[:2] + FLASH[:2]), (True, GENERAL[:2] + DECODE[:2]))
+                                                          for c in cs])
+def test_one_key_at_an_edge(kind, dtype, H, G, dq, dv, window, keep, decoded):
+    """Every query asks for one key: just inside and just outside the window, the last kept and the first dropped token, the
+    sequence's first token, page edges, itself. Seen, the output is that key's value; unseen, it must be something else."""
+    P = 330
+    sp = spec(H, G, dq, dv, window, keep, scale=0.3)
+    cache = Cache([P], G, dq, dv, dtype, seed=5, unit=True)
+    k, v = cache.seqs[0]
+    bias = torch.zeros(H, 40, device="cuda")
+    pairs = []
+    for i in (63, 64, 127, 128, 191, 200, 255, 256, 320, 329):
+        for j in {i, i - 1, i - window + 1, i - window, 0, keep - 1, keep, 63, 64, 127, 128}:
+            if 0 <= j <= i:
+                pairs.append((i, j))
+    if decoded:
+        got = torch.cat([run(kind, cache, batch([(0, i, 1)]), outstanding(cache, 0, [i], [j], H, dq), sp, bias) for i, j in pairs])
+    else:                                    # one portion that reaches each position; the other rows ask for themselves
+        rows = []
+        for i, j in pairs:
+            lo = max(0, i - 2)
+            q = outstanding(cache, 0, range(lo, i + 1), [*range(lo, i), j], H, dq)
+            rows.append(run(kind, cache, batch([(0, lo, i + 1 - lo)]), q, sp, bias)[-1:])
+        got = torch.cat(rows)
+    for (i, j), o in zip(pairs, got):
+        val = torch.stack([v[j, h // (H // G)] for h in range(H)]).double().cpu()
+        err = ((o.double().cpu() - val).norm() / val.norm()).item()
+        if O.visible(i, j, window, keep):
+            assert err < 0.05, (i, j, err)
+        else:
+            assert err > 0.3, (i, j, err)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("H,G,dq,dv", [(4, 2, 16, 24), (3, 1, 10, 6), (8, 8, 64, 64)])
+def test_query_key_norm_and_page_write(H, G, dq, dv, dtype):
+    """The norm runs over all heads at once; keys and values land in their pages, idle rows nowhere."""
+    from tunix_b200.ops import stack_kernels as SK
+    NQ, NK, NV, eps = H * dq, G * dq, G * dv, 1e-2
+    rb = batch([(1, 62, 4), (0, 0, 3), (2, 5, 1)])
+    rb.pos0[2] = -1
+    n = 8
+    proj = rand(n, 2 + NQ + NK + NV, dtype=dtype, std=0.3)
+    qw, kw = rand(NQ, dtype=dtype, seed=1), rand(NK, dtype=dtype, seed=2)
+    table = torch.tensor([[4, -1], [2, 0], [3, 3]], dtype=torch.int32, device="cuda")
+    kp, vp = torch.zeros(5, 64, NK, device="cuda", dtype=dtype), torch.zeros(5, 64, NV, device="cuda", dtype=dtype)
+    q = SK.qk_norm_write(proj, 2, 2 + NQ, 2 + NQ + NK, qw, kw, eps, rb, table, 64, kp, vp, NQ)
+    d = proj.double()
+    t = 2e-6 if dtype == torch.float32 else 5e-3
+    assert rel(q[:7], O.rms(d[:7, 2:2 + NQ], eps) * qw.double()) < t and q[7].abs().max() == 0
+    kn = O.rms(d[:, 2 + NQ:2 + NQ + NK], eps) * kw.double()
+    where = [(2, 62), (2, 63), (0, 0), (0, 1), (4, 0), (4, 1), (4, 2)]
+    for row, (pg, o) in enumerate(where):
+        assert rel(kp[pg, o], kn[row]) < t and torch.equal(vp[pg, o], proj[row, 2 + NQ + NK:])
+    assert (kp.abs().sum(-1) > 0).sum() == 7 and (vp.abs().sum(-1) > 0).sum() == 7
+
+
+def test_existing_decode_attention_without_bias_is_unchanged_by_the_tile_walk():
+    """Windowed decode without bias or kept tokens, many splits: the walk over visible tiles equals the dense result."""
+    sp = spec(8, 2, 64, 64, 100, 0, scale=1 / math.sqrt(64))
+    cache = Cache([640, 100, 101, 1], 2, 64, 64, torch.bfloat16, seed=9)
+    rb = batch([(s, n - 1, 1) for s, n in enumerate([640, 100, 101, 1])])
+    q = rand(4, 8, 64, dtype=torch.bfloat16)
+    zero = torch.zeros(8, 2, device="cuda")
+    for split in (64, 128, 256):
+        out = run("decode", cache, rb, q, sp, None, split)
+        for s, (k, v) in enumerate(cache.seqs):
+            assert rel(out[s:s + 1], dense(q[s:s + 1], k, v, k.shape[0] - 1, sp.scale, zero, 100, 0)) < 1.2e-2

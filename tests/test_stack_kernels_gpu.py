@@ -1,0 +1,194 @@
+"""The layer-stack kernels one mechanism at a time against tests/roluzen_oracle.py: odd and even sizes, 32-bit and bf16, the
+simple and the tensor-core forms, and inputs in which one key stands out at a window's, a page's or the kept tokens' edge."""
+import math
+
+import pytest
+import torch
+
+from tests import roluzen_oracle as O
+
+pytestmark = pytest.mark.gpu
+DT = [torch.float32, torch.bfloat16]
+
+
+def rel(a, b):
+    a, b = a.double().cpu(), b.double().cpu()
+    return ((a - b).norm() / b.norm()).item()
+
+
+def rand(*shape, dtype=torch.float32, std=1.0, seed=None):
+    g = torch.Generator("cuda").manual_seed(seed if seed is not None else 7 + sum(shape))
+    return (torch.randn(*shape, device="cuda", generator=g) * std).to(dtype)
+
+
+def batch(parts):
+    """[(slot, first position, length)] -> RaggedBatch"""
+    from tunix_b200.ops.ragged import RaggedBatch
+    return RaggedBatch.build([(s, p, [0] * n) for s, p, n in parts], "cuda")
+
+
+# ------------------------------------------------------------------------------------------------ streams
+@pytest.mark.parametrize("dtype", DT)
+@pytest.mark.parametrize("S,D", [(1, 40), (2, 36), (3, 37), (4, 1024), (5, 130), (8, 64)])
+def test_stream_step(S, D, dtype):
+    from tunix_b200.ops import stack_kernels as SK
+    n, eps, tol = 9, 1e-3, 1e-6 if dtype == torch.float32 else 5e-3
+    w = {k: rand(*s, dtype=dtype, seed=i) for i, (k, s) in enumerate({"in": (S,), "out": (S,), "mix": (S, S)}.items())}
+    wd = {k: v.double().cpu() for k, v in w.items()}
+    embed, nw, wy, wy2 = (rand(*s, dtype=dtype, seed=20 + i) for i, s in enumerate([(50, D), (D,), (D,), (D,)]))
+    y, y2 = rand(n, D, dtype=dtype, seed=30), rand(n, D, dtype=dtype, seed=31)
+    toks = torch.tensor([3, 0, 49, 7, 7, 1, 2, 48, 5], device="cuda")
+    d = lambda t: t.double().cpu()  # noqa: E731
+    x = torch.empty(n, S, D, device="cuda")
+    h = SK.stream_step(x, eps, tokens=toks, embed=embed, w_in=w["in"], norm_w=nw)
+    ref = d(embed)[toks.cpu()][:, None].repeat(1, S, 1)
+    assert rel(x, ref) == 0 and rel(h, O.rms(O.hyper_in(wd, "", ref), eps) * d(nw)) < tol
+    total = torch.empty(n, D, device="cuda")
+    h = SK.stream_step(x, eps, y=y, mix=w["mix"], w_out=w["out"], w_in=w["in"], norm_w=nw, sum_out=total)
+    ref = O.hyper_out(wd, "", ref, d(y))
+    assert rel(x, ref) < 1e-6 and rel(total, ref.sum(1)) < 1e-6 and rel(h, O.rms(O.hyper_in(wd, "", ref), eps) * d(nw)) < tol
+    h = SK.stream_step(x, eps, y=y, y2=y2, wy=wy, wy2=wy2, mix=w["mix"], w_out=w["out"], norm_w=nw)      # no w_in: the plain sum
+    ref = O.hyper_out(wd, "", ref, 0.5 * (O.rms(d(y), eps) * d(wy) + O.rms(d(y2), eps) * d(wy2)))
+    assert rel(x, ref) < 1e-6 and rel(h, O.rms(ref.sum(1), eps) * d(nw)) < tol
+
+
+@pytest.mark.parametrize("dtype", DT)
+@pytest.mark.parametrize("F", [8, 31, 500])
+def test_silu_mul(F, dtype):
+    from tunix_b200.ops import stack_kernels as SK
+    gu = rand(17, 2 * F, dtype=dtype, std=3)
+    ref = O.silu(gu[:, :F].double()) * gu[:, F:].double()
+    assert rel(SK.silu_mul(gu), ref) < (1e-6 if dtype == torch.float32 else 5e-3)
+
+
+@pytest.mark.parametrize("dtype", DT)
+@pytest.mark.parametrize("C1,heads,vdim", [(64, 2, 40), (6, 3, 7), (256, 1, 72)])
+def test_gate_outputs(C1, heads, vdim, dtype):
+    from tunix_b200.ops import stack_kernels as SK
+    n, C2, eps = 11, heads * vdim, 1e-2
+    attn, o, proj, w = rand(n, C1, dtype=dtype), rand(n, heads, vdim, std=0.05), rand(n, 5 + C1 + C2 + 3, dtype=dtype, std=2), rand(C2, dtype=dtype)
+    a1, a2 = SK.gate_outputs(attn, o, proj, 5, 5 + C1, w, eps, heads, vdim)
+    tol = 1e-6 if dtype == torch.float32 else 5e-3
+    assert rel(a1, attn.double() * torch.sigmoid(proj[:, 5:5 + C1].double())) < tol
+    ref = O.rms(o.double(), eps).reshape(n, C2) * w.double() * torch.sigmoid(proj[:, 5 + C1:5 + C1 + C2].double())
+    assert rel(a2, ref) < tol
+
+
+@pytest.mark.parametrize("K,N", [(40, 4), (1024, 6), (4096, 16), (256, 70)])
+def test_few_outputs(K, N):
+    from tunix_b200.ops import stack_kernels as SK
+    x, w = rand(5, K, dtype=torch.bfloat16), rand(N, K, dtype=torch.bfloat16, seed=1)
+    assert rel(SK.few_outputs(x, w), x.double() @ w.double().T) < 1e-5
+
+
+# ------------------------------------------------------------------------------------------------ gated recurrence
+def rglru_reference(m, proj, s0, past):
+    """One sequence's portion: proj [T, 2 W] (y | x), state s0 [W], the inputs before it [P, W] (oldest first)."""
+    d = lambda t: t.detach().double().cpu()  # noqa: E731
+    W, nb = m.spec.width, m.spec.blocks
+    P = past.shape[0]
+    x = torch.cat([d(past), d(proj[:, W:])])
+    u = O.causal_conv(x, d(m.conv_weight), d(m.conv_bias))[P:]
+    if m.ra_weight.dtype == torch.bfloat16:
+        u = u.to(torch.bfloat16).double()                  # the convolution's output is an activation
+    ub = u.view(u.shape[0], nb, -1)
+    gate = lambda w, b: torch.sigmoid(torch.einsum("boi,tbi->tbo", d(w), ub) + d(b)).reshape(-1, W)  # noqa: E731
+    a = torch.exp(-8 * gate(m.ra_weight, m.ra_bias) * torch.nn.functional.softplus(d(m.lam)))
+    i = gate(m.ri_weight, m.ri_bias)
+    s, out = d(s0), []
+    for t in range(u.shape[0]):
+        s = a[t] * s + torch.sqrt(1 - a[t] ** 2) * i[t] * u[t]
+        out.append(s)
+    return torch.stack(out) * O.gelu_tanh(d(proj[:, :W])), s
+
+
+@pytest.mark.parametrize("dtype,plain", [(torch.float32, False), (torch.bfloat16, True), (torch.bfloat16, False)])
+@pytest.mark.parametrize("W,blocks,K", [(96, 3, 4), (64, 1, 1), (36, 9, 2), (512, 4, 3), (80, 2, 9), (256, 1, 4)])
+def test_gated_recurrence(W, blocks, K, dtype, plain):
+    """Three sequences of unequal portions, decoded steps after them, then a slot that starts over."""
+    from tunix_b200.models.mixers import RGLRUMixer, RGLRUSpec
+    from tunix_b200.ops import stack_kernels as SK
+    m = RGLRUMixer(RGLRUSpec(W, blocks, K), 8, 1e-6, dtype, "cuda")
+    for i, p in enumerate(m.parameters()):
+        p.data.copy_(rand(*p.shape, dtype=dtype, std=0.4, seed=i))
+    m.lam.data.copy_(rand(W, dtype=dtype, std=3) - 3)
+    state = {"s": rand(4, W, seed=50), "ring": rand(4, K, W, seed=51)}         # left by earlier owners
+    past = {s: torch.zeros(0, W, device="cuda") for s in range(4)}
+    s_ref = {s: torch.zeros(W) for s in range(4)}
+    tol = 2e-6 if dtype == torch.float32 else 4e-3
+    seed = 60
+    for parts in ([(2, 0, 130), (0, 0, 64), (3, 0, 1)], [(0, 64, 2), (3, 1, 65), (2, 130, 63)], [(0, 66, 1), (2, 193, 1), (3, 66, 1)],
+                  [(2, 194, 1), (0, 67, 1), (3, 67, 1)], [(1, 0, 1), (0, 0, 3)]):
+        for s, p, _ in parts:
+            if p == 0:
+                past[s], s_ref[s] = torch.zeros(0, W, device="cuda"), torch.zeros(W)
+        n = sum(k for _, _, k in parts)
+        seed += 1
+        proj = rand(n, 2 * W, dtype=dtype, seed=seed)
+        out = SK.rglru(proj, W, 0, m, batch(parts), state, plain)
+        at = 0
+        for s, p, k in parts:
+            part = proj[at:at + k]
+            want, s_ref[s] = rglru_reference(m, part, s_ref[s], past[s][-(K - 1):] if K > 1 else past[s][:0])
+            assert rel(out[at:at + k], want) < tol, (parts, s)
+            assert rel(state["s"][s], s_ref[s]) < (2e-6 if dtype == torch.float32 else 2e-3)
+            past[s] = torch.cat([past[s], part[:, W:].float()])
+            at += k
+
+
+# ------------------------------------------------------------------------------------------------ matrix memory
+def mlstm_reference(q, k, v, ig, fg, S, n, m):
+    out = []
+    dk = q.shape[-1]
+    for t in range(q.shape[0]):
+        new = torch.maximum(fg[t] + m, ig[t])
+        a, b = torch.exp(fg[t] + m - new), torch.exp(ig[t] - new)
+        S = a[:, None, None] * S + b[:, None, None] * k[t][:, :, None] * v[t][:, None]
+        n = a[:, None] * n + b[:, None] * k[t]
+        m = new
+        qt = q[t] * dk ** -0.5
+        out.append(torch.einsum("hkv,hk->hv", S, qt) / (torch.maximum((n * qt).sum(-1).abs(), torch.exp(-m)) + 1e-6)[:, None])
+    return torch.stack(out), S, n, m
+
+
+@pytest.mark.parametrize("dtype,plain", [(torch.float32, False), (torch.bfloat16, True), (torch.bfloat16, False)])
+@pytest.mark.parametrize("H,dk,dv,cap", [(2, 24, 40, 15.0), (1, 64, 64, 5.0), (3, 8, 8, 9.0), (2, 12, 33, 15.0), (1, 136, 72, 15.0),
+                                         (2, 256, 32, 20.0)])
+def test_matrix_memory(H, dk, dv, cap, dtype, plain):
+    """Portions around the chunk length, decoded steps, a slot that starts over; gates from closed to wide open, so that both
+    branches of the denominator and of the running maximum occur."""
+    from tunix_b200.models.mixers import MatrixMemorySpec
+    from tunix_b200.ops import stack_kernels as SK
+    shapes = MatrixMemorySpec(H, dk, dv, cap).state_shapes()
+    state = {k: rand(4, *s, seed=70 + i) for i, (k, s) in enumerate(shapes.items())}
+    ib, fb = rand(H, dtype=dtype, std=1.0, seed=80), rand(H, dtype=dtype, std=2.0, seed=81) + 3
+    d = lambda t: t.double().cpu()  # noqa: E731
+    zero = lambda: (torch.zeros(H, dk, dv).double(), torch.zeros(H, dk).double(), torch.zeros(H).double())  # noqa: E731
+    refs, seed = {s: zero() for s in range(4)}, 90
+    tol = 3e-4 if dtype == torch.float32 or plain else 2e-2     # a denominator near zero magnifies rounding
+    for parts in ([(3, 0, 64), (1, 0, 131), (0, 0, 1)], [(1, 131, 2), (0, 1, 63), (3, 64, 65)], [(3, 129, 1), (1, 133, 1), (0, 64, 1)],
+                  [(2, 0, 1), (1, 134, 1), (0, 65, 1)], [(2, 1, 2), (1, 0, 5)]):
+        for s, p, _ in parts:
+            if p == 0:
+                refs[s] = zero()
+        n = sum(k for _, _, k in parts)
+        seed += 1
+        off = 8
+        proj = rand(n, off + H * (2 * dk + dv), dtype=dtype, seed=seed)
+        gates = rand(n, 2 * H, std=4.0, seed=seed + 100)
+        ko, vo = off + H * dk, off + 2 * H * dk
+        out = SK.mlstm(proj, off, ko, vo, gates.clone(), ib, fb, cap, batch(parts), H, dk, dv, state, plain)
+        at = 0
+        for s, p, k in parts:
+            sl = slice(at, at + k)
+            q, kk, v = d(proj[sl, off:ko]).view(k, H, dk), d(proj[sl, ko:vo]).view(k, H, dk), d(proj[sl, vo:]).view(k, H, dv)
+            ig = cap * torch.tanh((d(gates[sl, :H]) + d(ib)) / cap)
+            fg = torch.nn.functional.logsigmoid(cap * torch.tanh((d(gates[sl, H:]) + d(fb)) / cap))
+            want, *refs[s] = mlstm_reference(q, kk, v, ig, fg, *refs[s])
+            assert rel(out[sl], want) < tol, (parts, s)
+            S, nn, m = refs[s]
+            assert rel(state["S"][s], S) < 2e-5
+            for x in range(shapes["n"][1]):
+                assert rel(state["n"][s][:, x], nn) < 2e-5
+                assert (state["m"][s][:, x].double().cpu() - m).abs().max() < 1e-4
+            at += k

@@ -1,6 +1,8 @@
 """Rollout on the in-framework sampler (tunix/rl/rollout/vanilla_rollout.py:31-106)."""
 from __future__ import annotations
 
+import math
+
 import numpy as np
 
 from ...common.configs import CacheConfig, RolloutConfig
@@ -20,9 +22,12 @@ def _page_budget(model, cache_size: int, rc: RolloutConfig):
     want = int(rc.max_running_requests) * per_seq
     if dev.type != "cuda" or not rc.hbm_utilization:
         return want
-    page_bytes = cfg.num_layers * 2 * cfg.num_kv_heads * cfg.head_dim * int(rc.page_size) * 2
+    rows = [sum(r) for r in cfg.kv_rows() if r] if hasattr(cfg, "kv_rows") else [2 * cfg.num_kv_heads * cfg.head_dim] * cfg.num_layers
+    page_bytes = sum(rows) * int(rc.page_size) * 2
     free, _ = torch.cuda.mem_get_info(dev)
-    cap = int(free * float(rc.hbm_utilization)) // max(page_bytes, 1)
+    if hasattr(cfg, "state_shapes"):                # recurrent layers keep fp32 states per running sequence as well
+        free -= int(rc.max_running_requests) * sum(4 * math.prod(s) for d in cfg.state_shapes() for s in d.values())
+    cap = max(int(free * float(rc.hbm_utilization)) // max(page_bytes, 1), 0)
     return max(min(want, cap), per_seq)             # never below one full sequence
 
 
