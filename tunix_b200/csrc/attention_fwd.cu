@@ -42,6 +42,7 @@ struct AttnArgs {
   // paged form: the query tiles of a ragged batch, keys and values in the pages of their sequences
   const int *cu, *slot, *pos0, *tile_t0, *tile_ent, *table;
   int max_pages, page_size;
+  int chunk;                 // > 0: keys of the query's own chunk only (chunks of `chunk` positions from the sequence's start)
   int keep;                  // with a window: the first `keep` tokens of a sequence stay visible
   const float* bias;         // [N, far + 1] added to the score of a key at distance min(distance, far), or null
   int far;
@@ -106,6 +107,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   if (a.causal) kv_end = min(Tk, i0 + BQ);
   int kv_start = 0;
   if (a.window > 0) kv_start = max(0, i0 - a.window + 1);
+  if (PAGED && a.chunk > 0) kv_start = max(kv_start, i0 - i0 % a.chunk);
   const int jb0 = kv_start / BKV;
   const int n_sink = PAGED ? min((min(a.keep, Tk) + BKV - 1) / BKV, jb0) : 0;
   const int nblk = n_sink + (kv_end > jb0 * BKV ? (kv_end - jb0 * BKV + BKV - 1) / BKV : 0);
@@ -214,6 +216,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     const uint32_t lane_addr = (uint32_t)(warp * 32) << 16;
     const int my_seg = (a.seg_q && row_valid) ? a.seg_q[(long long)b * a.Tq + qi] : 0;
     const float sc2 = a.scale * LOG2E;
+    const int chunk0 = PAGED && a.chunk > 0 ? qpos - qpos % a.chunk : 0;       // first position of this query's chunk
+    const float inv_cap = a.softcap > 0.f ? 1.f / a.softcap : 0.f;
     float m_used = 0.f, l = 0.f;
     bool ok = true;
     for (int j = 0; j < nblk && ok; ++j) {
@@ -234,9 +238,17 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       const int* segk = a.seg_k ? a.seg_k + (long long)b * a.Tk + k0 : nullptr;
       // most key blocks of a causal tile lie fully below the diagonal: skip the per-element mask there
       const bool need_mask = (k0 + BKV > Tk) || (segk != nullptr) || (a.causal && (k0 + BKV - 1 > i0)) ||
-                             (a.window > 0 && (k0 <= i0 + BQ - 1 - a.window));
+                             (a.window > 0 && (k0 <= i0 + BQ - 1 - a.window)) ||
+                             (PAGED && a.chunk > 0 && k0 < i0 + nrows - 1 - (i0 + nrows - 1) % a.chunk);
       if (PAGED) {
-        if (bias) {
+        if (a.softcap > 0.f) {
+#pragma unroll
+          for (int i = 0; i < 64; ++i) z[i] = cap_score(__uint_as_float(sraw[i]) * a.scale, a.softcap, inv_cap) * LOG2E;
+          if (bias) {
+#pragma unroll
+            for (int i = 0; i < 64; ++i) z[i] += __ldg(bias + min(max(qpos - k0 - i, 0), a.far)) * LOG2E;
+          }
+        } else if (bias) {
 #pragma unroll
           for (int i = 0; i < 64; ++i)
             z[i] = fmaf(__uint_as_float(sraw[i]), sc2, __ldg(bias + min(max(qpos - k0 - i, 0), a.far)) * LOG2E);
@@ -248,7 +260,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
 #pragma unroll
           for (int i = 0; i < 64; ++i) {
             const int kp = k0 + i;
-            if (kp > qpos || (a.window > 0 && kp <= qpos - a.window && kp >= a.keep)) z[i] = -INFINITY;
+            if (kp > qpos || (((a.window > 0 && kp <= qpos - a.window) || kp < chunk0) && kp >= a.keep)) z[i] = -INFINITY;
           }
         }
 #pragma unroll
@@ -264,7 +276,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         for (int i = 0; i < 64; ++i) {
           const int kp = k0 + i;
           float s = __uint_as_float(sraw[i]);
-          if (a.softcap > 0.f) s = a.softcap * tanhf(s * a.scale / a.softcap) * LOG2E;
+          if (a.softcap > 0.f) s = cap_score(s * a.scale, a.softcap, inv_cap) * LOG2E;
           else s *= sc2;
           bool keep = kp < a.Tk;
           if (a.causal) keep = keep && (kp <= qpos);
@@ -829,16 +841,17 @@ static int launch_fwd_paged(const void* q, const void* k, const void* v, const A
 
 // Causal attention of the query tiles (at most 128 rows of one entry each) of a ragged batch over paged keys and values:
 // q / out [n, N * H]; pools [pool_rows, KH * H] with page_size a multiple of 64; a key block of 64 tokens lies in one page
-// and is fetched by TMA through the page table. window <= 0: no window. The unused tail of a page must hold finite values.
+// and is fetched by TMA through the page table. window, chunk <= 0: none; softcap <= 0: none. The unused tail of a page must hold finite values.
 TB_API int tb_attn_fwd_paged(const void* q, const void* k_pool, const void* v_pool, void* out, int n, long long pool_rows, int N,
-                             int KH, int H, float scale, int window, int keep, const float* bias, int far, const int* cu,
+                             int KH, int H, float scale, float softcap, int window, int chunk, int keep, const float* bias, int far, const int* cu,
                              const int* slot, const int* pos0, const int* tile_t0, const int* tile_ent, int tiles,
                              const int* table, int max_pages, int page_size, int* status, cudaStream_t stream) {
   if (n <= 0 || tiles <= 0) return 0;
   if (KH <= 0 || N % KH || page_size % BKV || N > 65535) return -2;
   AttnArgs a = {};
   a.N = N; a.KH = KH; a.scale = scale; a.causal = 1; a.window = window > 0 ? window : 0;
-  a.keep = a.window > 0 ? keep : 0; a.bias = bias; a.far = far;
+  a.softcap = softcap; a.chunk = chunk > 0 ? chunk : 0;
+  a.keep = a.window > 0 || a.chunk > 0 ? keep : 0; a.bias = bias; a.far = far;
   a.O = reinterpret_cast<__nv_bfloat16*>(out); a.ldo = (long long)N * H; a.status = status;
   a.cu = cu; a.slot = slot; a.pos0 = pos0; a.tile_t0 = tile_t0; a.tile_ent = tile_ent; a.table = table;
   a.max_pages = max_pages; a.page_size = page_size;

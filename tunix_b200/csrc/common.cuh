@@ -269,6 +269,11 @@ __device__ __forceinline__ float warp_max(float v) {
   return v;
 }
 // Block-wide sum; `red` must hold 33 floats of shared memory.
+// cap * tanh(s / cap) with an absolute error of a few 1e-7 * cap, whatever math flags the file is compiled with (the hardware
+// tanh is off by 5e-4)
+__device__ __forceinline__ float cap_score(float s, float cap, float inv_cap) {
+  return cap - 2.f * cap / (1.f + __expf(2.f * s * inv_cap));
+}
 __device__ __forceinline__ float block_sum(float v, float* red) {
   int lane = threadIdx.x & 31, w = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;
   v = warp_sum(v);

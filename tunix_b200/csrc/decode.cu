@@ -10,9 +10,9 @@
 //                    context split). The query heads of a kv head are the rows of a 16-row mma.sync tile, K / V
 //                    stream through a double-buffered cp.async stage and are read with ldmatrix; running
 //                    max / sum per query head, partial results of the splits merged by `paged_decode_combine`.
-//                    Sliding window (optionally with kept first tokens), a bias per (distance, head) added to the
-//                    scores, and logit soft-cap supported; with a window only the tiles that hold visible keys are
-//                    walked and split over CTAs. Memory-bound by construction: every K / V
+//                    Sliding window (optionally with kept first tokens), chunks of positions, a bias per (distance, head)
+//                    added to the scores, and logit soft-cap supported; with a window or chunks only the tiles that hold
+//                    visible keys are walked and split over CTAs. Memory-bound by construction: every K / V
 //                    byte of the sequence is read exactly once per kv head.
 //
 // The reference keeps only host-side page-table logic (tunix/experimental/generate/*) and runs decode on a
@@ -130,8 +130,9 @@ __device__ __forceinline__ uint32_t tile_off(int r, int c) {
 // The key tiles a single query at position len - 1 walks: the tiles that hold kept first tokens, then those of the window.
 struct KeyTiles {
   int w_lo, first, n_sink, total;
-  __device__ __forceinline__ KeyTiles(int len, int window, int keep) {
+  __device__ __forceinline__ KeyTiles(int len, int window, int chunk, int keep) {
     w_lo = window > 0 ? max(0, len - window) : 0;
+    if (chunk > 0 && len > 0) w_lo = max(w_lo, len - 1 - (len - 1) % chunk);
     first = w_lo / TILE_KEYS;
     n_sink = min((min(keep, len) + TILE_KEYS - 1) / TILE_KEYS, first);
     total = n_sink + (len + TILE_KEYS - 1) / TILE_KEYS - first;
@@ -152,7 +153,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_consta
                     const __nv_bfloat16* __restrict__ k_pool, const __nv_bfloat16* __restrict__ v_pool,
                     const int* __restrict__ page_table, int max_pages, int page_size,
                     const int* __restrict__ seq_ids, const int* __restrict__ seq_lens, int KH, int G, float scale,
-                    float softcap, int window, int keep, const float* __restrict__ bias, int far,   // bias [N, far + 1] or null
+                    float softcap, int window, int chunk, int keep, const float* __restrict__ bias, int far,   // bias [N, far + 1] or null
                     int num_splits, int split_tokens,
                     float* __restrict__ part_acc,                                               // [B, N, splits, H]
                     float* __restrict__ part_ml,                                                // [B, N, splits, 2]
@@ -172,7 +173,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_consta
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int N = KH * G;
   const int len = seq_lens[b];
-  const KeyTiles kt(len, window, keep);
+  const KeyTiles kt(len, window, chunk, keep);
   const int tile0 = split * (split_tokens / TILE_KEYS);
   const int n_tiles = min(kt.total - tile0, split_tokens / TILE_KEYS);
   if (len <= 0 || n_tiles <= 0) { // past the end of this sequence: the combine kernel never reads this split
@@ -235,6 +236,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_consta
     cp_async_commit();
   };
 
+  const float inv_cap = softcap > 0.f ? 1.f / softcap : 0.f;
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
   float o[H / 8][4];
 #pragma unroll
@@ -282,7 +284,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_consta
         for (int j = 0; j < 4; ++j) {
           const int t = tw + nb * 8 + 2 * (lane & 3) + (j & 1);
           float v = s[nb][j] * scale;
-          if (softcap > 0.f) v = softcap * tanhf(v / softcap);
+          if (softcap > 0.f) v = cap_score(v, softcap, inv_cap);
           if (bias != nullptr && t < len) {
             const int row = (lane >> 2) + (j >> 1) * 8;
             if (row < G) v += __ldg(bias + (long long)(kh * G + row) * (far + 1) + min(len - 1 - t, far));
@@ -380,13 +382,13 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_consta
 // out[b, n, :] = sum_s acc_s * exp(m_s - M) / sum_s l_s * exp(m_s - M)
 __global__ void paged_decode_combine_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
                                             const int* __restrict__ seq_lens, int N, int H, int num_splits, int split_tokens,
-                                            int window, int keep, __nv_bfloat16* __restrict__ out, long long ldo) {
+                                            int window, int chunk, int keep, __nv_bfloat16* __restrict__ out, long long ldo) {
   pdl_trigger();
   pdl_wait();
   const int b = blockIdx.x, n = blockIdx.y;
   const int len = seq_lens[b];
   const int tps = split_tokens / TILE_KEYS;
-  const int used = len > 0 ? min(num_splits, (KeyTiles(len, window, keep).total + tps - 1) / tps) : 0;
+  const int used = len > 0 ? min(num_splits, (KeyTiles(len, window, chunk, keep).total + tps - 1) / tps) : 0;
   const long long base = ((long long)b * N + n) * num_splits;
   float M = -INFINITY;
   for (int s = 0; s < used; ++s) M = fmaxf(M, part_ml[(base + s) * 2]);
@@ -410,7 +412,7 @@ template <int H, bool TMA, int STAGES>
 int launch_decode_v(int G, dim3 grid, cudaStream_t stream, const CUtensorMap& tmK, const CUtensorMap& tmV,
                     const __nv_bfloat16* q, long long ldq, const __nv_bfloat16* kp, const __nv_bfloat16* vp, const int* pt,
                     int max_pages, int page_size, const int* seq_ids, const int* seq_lens, int KH, float scale, float softcap,
-                    int window, int keep, const float* bias, int far, int splits, int split_tokens, float* pa, float* pml,
+                    int window, int chunk, int keep, const float* bias, int far, int splits, int split_tokens, float* pa, float* pml,
                     __nv_bfloat16* out, long long ldo, int* status) {
   constexpr int TILE2 = 2 * TILE_KEYS * H * 2;                       // one stage: a K tile and a V tile
   constexpr int SMEM = STAGES * TILE2 + (TMA ? 1024 : 0);
@@ -421,7 +423,7 @@ int launch_decode_v(int G, dim3 grid, cudaStream_t stream, const CUtensorMap& tm
   // a split of one 64-key tile needs one stage only: more CTAs fit on an SM
   const int smem = split_tokens > TILE_KEYS ? SMEM : TILE2 + (TMA ? 1024 : 0);
   return launch_pdl(paged_decode_kernel<H, TMA, STAGES>, grid, dim3(128), smem, stream, tmK, tmV, q, ldq, kp, vp, pt, max_pages,
-                    page_size, seq_ids, seq_lens, KH, G, scale, softcap, window, keep, bias, far, splits, split_tokens, pa, pml, out, ldo,
+                    page_size, seq_ids, seq_lens, KH, G, scale, softcap, window, chunk, keep, bias, far, splits, split_tokens, pa, pml, out, ldo,
                     status) == cudaSuccess ? 0 : -5;
 }
 
@@ -430,7 +432,7 @@ template <int H>
 int launch_decode(int G, dim3 grid, cudaStream_t stream, const __nv_bfloat16* q, long long ldq,
                   const __nv_bfloat16* kp, const __nv_bfloat16* vp, long long pool_rows, const int* pt, int max_pages,
                   int page_size, const int* seq_ids, const int* seq_lens, int KH, float scale, float softcap, int window,
-                  int keep, const float* bias, int far, int splits, int split_tokens, float* pa, float* pml, __nv_bfloat16* out,
+                  int chunk, int keep, const float* bias, int far, int splits, int split_tokens, float* pa, float* pml, __nv_bfloat16* out,
                   long long ldo, int* status) {
   static const bool no_tma = getenv("TUNIX_B200_DECODE_NO_TMA") != nullptr;
   static const char* stages_env = getenv("TUNIX_B200_DECODE_STAGES");
@@ -441,7 +443,7 @@ int launch_decode(int G, dim3 grid, cudaStream_t stream, const __nv_bfloat16* q,
                    tb_make_tmap_2d_bf16(&tmK, kp, (uint64_t)pool_rows, (uint64_t)KH * H, (uint64_t)KH * H, TILE_KEYS, 64, 1) == 0 &&
                    tb_make_tmap_2d_bf16(&tmV, vp, (uint64_t)pool_rows, (uint64_t)KH * H, (uint64_t)KH * H, TILE_KEYS, 64, 1) == 0;
 #define LD(T, S) launch_decode_v<H, T, S>(G, grid, stream, tmK, tmV, q, ldq, kp, vp, pt, max_pages, page_size, seq_ids, seq_lens, \
-                                         KH, scale, softcap, window, keep, bias, far, splits, split_tokens, pa, pml, out, ldo, status)
+                                         KH, scale, softcap, window, chunk, keep, bias, far, splits, split_tokens, pa, pml, out, ldo, status)
   if (!tma) return LD(false, 2);
   // measured at head dim 128 (8 kv heads, 256 sequences x 768 tokens): 2 / 3 / 4 stages take 157 / 161 / 194 us,
   // cp.async staging 190 us: three CTAs per SM with two stages each beat deeper rings on fewer CTAs
@@ -496,12 +498,12 @@ TB_API int tb_qkv_post(void* qkv, long long ld, const int* seq_ids, const int* p
 // workspace: part_acc fp32 [B*N*splits*H], part_ml fp32 [B*N*splits*2] with splits = ceil(max_ctx / split_tokens);
 // split_tokens = context tokens per CTA, a multiple of 64 in [64, 2048] (0 = 256). CTAs of splits that lie past the
 // end of their sequence return at once. pool_rows = num_pages * page_size (rows of the pools, for the tensor maps;
-// 0 = no TMA staging). window > 0: keys at distance < window, and the sequence's first `keep` tokens. bias fp32
+// 0 = no TMA staging). window > 0: keys at distance < window, chunk > 0: keys of the query's chunk, and the sequence's first `keep` tokens. bias fp32
 // [N, far + 1] (null = none) is added to the scaled score of a key at distance min(distance, far). status: word that a bounded mbarrier wait writes its code to.
 TB_API int tb_paged_decode(const void* q, long long ldq, const void* k_pool, const void* v_pool,
                            const int* page_table, int max_pages, int page_size, const int* seq_ids,
                            const int* seq_lens, int B, int N, int KH, int H, int max_ctx, float scale, float softcap,
-                           int window, int keep, const float* bias, int far, int split_tokens, long long pool_rows,
+                           int window, int chunk, int keep, const float* bias, int far, int split_tokens, long long pool_rows,
                            float* part_acc, float* part_ml, void* out, long long ldo, int* status, cudaStream_t stream) {
   if (B <= 0) return 0;
   if (KH <= 0 || N % KH || (ldq % 8)) return -2;
@@ -510,8 +512,9 @@ TB_API int tb_paged_decode(const void* q, long long ldq, const void* k_pool, con
   if (split_tokens <= 0) split_tokens = 256;
   if (split_tokens % TILE_KEYS || split_tokens > MAX_SPLIT_TOKENS) return -2;
   int max_tiles = (max_ctx + TILE_KEYS - 1) / TILE_KEYS;
-  if (window > 0) {
-    const int vis = (keep + TILE_KEYS - 1) / TILE_KEYS + (window + TILE_KEYS - 1) / TILE_KEYS + 1;
+  const int span = window > 0 && (chunk <= 0 || window < chunk) ? window : chunk;       // most keys besides the kept ones
+  if (span > 0) {
+    const int vis = (keep + TILE_KEYS - 1) / TILE_KEYS + (span + TILE_KEYS - 1) / TILE_KEYS + 1;
     if (vis < max_tiles) max_tiles = vis;
   }
   const int splits = (max_tiles + split_tokens / TILE_KEYS - 1) / (split_tokens / TILE_KEYS);
@@ -521,15 +524,15 @@ TB_API int tb_paged_decode(const void* q, long long ldq, const void* k_pool, con
   auto kp = (const __nv_bfloat16*)k_pool;
   auto vp = (const __nv_bfloat16*)v_pool;
   switch (H) {
-    case 64: rc = launch_decode<64>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, keep, bias, far, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
-    case 128: rc = launch_decode<128>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, keep, bias, far, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
-    case 256: rc = launch_decode<256>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, keep, bias, far, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
+    case 64: rc = launch_decode<64>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, chunk, keep, bias, far, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
+    case 128: rc = launch_decode<128>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, chunk, keep, bias, far, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
+    case 256: rc = launch_decode<256>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, chunk, keep, bias, far, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
     default: return -2;
   }
   if (rc) return rc;
   if (splits == 1) return 0;
   return launch_pdl(paged_decode_combine_kernel, dim3(B, N), dim3(128), 0, stream, (const float*)part_acc,
-                    (const float*)part_ml, seq_lens, N, H, splits, split_tokens, window, keep, (__nv_bfloat16*)out, ldo) == cudaSuccess ? 0 : -5;
+                    (const float*)part_ml, seq_lens, N, H, splits, split_tokens, window, chunk, keep, (__nv_bfloat16*)out, ldo) == cudaSuccess ? 0 : -5;
 }
 
 // ------------------------------------------------------------------ per-step bookkeeping of the decode loop

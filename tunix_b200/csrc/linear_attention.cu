@@ -1,0 +1,657 @@
+// Gated linear attention over ragged batches: a matrix state S [dk, dv] per head whose rows decay by a factor of their own at
+// every token, S <- diag(f) S + k v^T. The state lives in fp32 per slot; a sequence's first token starts from zero.
+//
+// What makes f, k and the read-out differs per mechanism (MODE):
+//   BONUS (RWKV time mixing)  f = exp(-exp(z + c0)); o = (S_before + diag(c1) k v^T)^T q
+//   LOWER (HGRN2)             f = c1 + (1 - c1) sigmoid(z + c0), k = 1 - f, q = silu(q); o = S^T q
+// with z fp32 from a projection and c0, c1 parameters per head and channel. Then every head's o is divided by its root mean
+// square over dv, weighted (one weight for all heads or one per head), and gated by silu if there is a gate.
+//
+//   gla_step  : one token per entry. The state streams through registers once; norm and gate in the same launch.
+//   gla_chunk : portions of prompts, bf16, on tensor cores (below).
+//   gla_seq   : token by token, any sizes, also 32-bit; head_norm after it.
+//
+// This file is compiled without fast-math: the same kernels serve the 32-bit mode.
+#include "mma.cuh"
+#include "precise.cuh"
+
+using namespace tb;
+
+namespace {
+
+typedef __nv_bfloat16 bf;
+enum Mode { BONUS = 0, LOWER = 1 };
+
+struct GlaArgs {
+  const void *q, *k, *v, *gate;       // T [n, ld*], head h at columns h * dk or h * dv; k null with LOWER, gate may be null
+  long long ldq, ldk, ldv, ldg;
+  const float* z;                     // fp32 [n, ldz]
+  long long ldz;
+  const void *c0, *c1;                // T [heads * dk]
+  int heads, dk, dv;
+  Ragged rb;
+  float* S;                           // fp32 [slots, heads, dk, dv]
+  // token shift: the last row of every portion is carried to the next one (gla_chunk, gla_seq; null: nothing to carry)
+  const void* h;                      // T [n, D]
+  float* carry;                       // fp32 [slots, D]
+  int D;
+  // output norm
+  const void* nw;                     // T [dv] or [heads * dv]
+  int per_head;
+  float eps;
+};
+
+template <int MODE>
+__device__ __forceinline__ void gates_exact(float z, float c0, float c1, float& f, float& k) {
+  if (MODE == BONUS) {
+    f = decay_exp(-expf(z + c0));
+  } else {
+    // near 1 the decay is rounded once: 1 - k
+    k = (1.f - c1) * sigmoid(-(z + c0));
+    f = k < 0.5f ? 1.f - k : c1 + (1.f - c1) * sigmoid(z + c0);
+  }
+}
+// log f for bf16 models; bounded, so that sums of it stay finite
+template <int MODE>
+__device__ __forceinline__ float gates_log(float z, float c0, float c1, float& k) {
+  if (MODE == BONUS) return -fminf(quick_exp(z + c0), 1e4f);
+  k = (1.f - c1) * quick_sigmoid(-(z + c0));
+  return k < 0.5f ? log1pf(-k) : logf(fmaxf(c1 + (1.f - c1) * quick_sigmoid(z + c0), 1e-30f));
+}
+
+template <typename T>
+__device__ __forceinline__ float silu(float z) {
+  return z * (sizeof(T) == 2 ? quick_sigmoid(z) : sigmoid(z));
+}
+
+template <typename T>
+__device__ __forceinline__ void carry_rows(const GlaArgs& a, int last, long long slot, int part, int parts) {
+  if (!a.h) return;
+  const T* h = static_cast<const T*>(a.h) + (long long)last * a.D;
+  for (int c = part * blockDim.x + threadIdx.x; c < a.D; c += parts * blockDim.x) a.carry[slot * a.D + c] = to_f(h[c]);
+}
+
+// ------------------------------------------------------------------------------------------------ one token
+constexpr int GT = 256;
+
+template <typename T, int MODE, int V>
+__global__ void __launch_bounds__(GT)
+gla_step_kernel(const GlaArgs a, T* __restrict__ out) {
+  extern __shared__ float sm[];
+  const int dk = a.dk, dv = a.dv, hd = blockIdx.x, e = blockIdx.y, tid = threadIdx.x;
+  float* qs = sm;                      // [dk]
+  float* ks = qs + dk;                 // [dk]
+  float* fs = ks + dk;                 // [dk]
+  float* us = fs + dk;                 // [dk]
+  float* part = us + dk;               // [R][dv]
+  __shared__ float red[33];
+  pdl_trigger();
+  pdl_wait();
+  const int p0 = a.rb.pos0[e];
+  T* o = out + ((long long)e * a.heads + hd) * dv;
+  if (p0 < 0) {
+    for (int c = tid; c < dv; c += GT) o[c] = from_f<T>(0.f);
+    return;
+  }
+  const bool old = p0 > 0;
+  float* S = a.S + ((long long)a.rb.slot[e] * a.heads + hd) * dk * dv;
+  for (int d = tid; d < dk; d += GT) {
+    const int c = hd * dk + d;
+    const float c1 = to_f(static_cast<const T*>(a.c1)[c]);
+    float q = to_f(static_cast<const T*>(a.q)[e * a.ldq + c]), k = 0.f, f;
+    if (MODE == BONUS) k = to_f(static_cast<const T*>(a.k)[e * a.ldk + c]);
+    else q = silu<T>(q);
+    gates_exact<MODE>(a.z[e * a.ldz + c], to_f(static_cast<const T*>(a.c0)[c]), c1, f, k);
+    qs[d] = q;
+    ks[d] = k;
+    fs[d] = f;
+    us[d] = MODE == BONUS ? c1 : 0.f;
+  }
+  __syncthreads();
+  const int C = dv / V, R = GT / C, r = tid / C, col = (tid - r * C) * V;
+  if (r < R) {
+    float v[V], acc[V];
+    load_v<V>(static_cast<const T*>(a.v) + e * a.ldv + hd * dv + col, v);
+#pragma unroll
+    for (int i = 0; i < V; ++i) acc[i] = 0.f;
+    constexpr int U = 4;
+    for (int d0 = r; d0 < dk; d0 += U * R) {
+      float s[U][V];
+#pragma unroll
+      for (int j = 0; j < U; ++j) {
+        const int d = d0 + j * R;
+        if (old && d < dk) {
+          load_v<V>(S + (long long)d * dv + col, s[j]);
+        } else {
+#pragma unroll
+          for (int i = 0; i < V; ++i) s[j][i] = 0.f;
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < U; ++j) {
+        const int d = d0 + j * R;
+        if (d < dk) {
+          const float k = ks[d], f = fs[d], q = qs[d], uk = us[d] * k;
+#pragma unroll
+          for (int i = 0; i < V; ++i) {
+            if (MODE == BONUS) acc[i] += q * (s[j][i] + uk * v[i]);
+            s[j][i] = f * s[j][i] + k * v[i];
+            if (MODE == LOWER) acc[i] += q * s[j][i];
+          }
+          store_v<V>(S + (long long)d * dv + col, s[j]);
+        }
+      }
+    }
+    store_v<V>(part + r * dv + col, acc);
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int c = tid; c < dv; c += GT) {
+    float x = 0.f;
+    for (int j = 0; j < R; ++j) x += part[j * dv + c];
+    part[c] = x;                       // row 0, read by this thread only
+    ss += x * x;
+  }
+  ss = block_sum(ss, red);
+  const float rstd = 1.f / sqrtf(ss / (float)dv + a.eps);
+  for (int c = tid; c < dv; c += GT) {
+    float x = part[c] * rstd * to_f(static_cast<const T*>(a.nw)[a.per_head ? hd * dv + c : c]);
+    if (a.gate) x *= silu<T>(to_f(static_cast<const T*>(a.gate)[e * a.ldg + hd * dv + c]));
+    o[c] = from_f<T>(x);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------ token by token
+constexpr int SV = 32;          // value columns per CTA
+
+template <typename T, int MODE>
+__global__ void __launch_bounds__(GT)
+gla_seq_kernel(const GlaArgs a, float* __restrict__ out) {
+  extern __shared__ float sm[];
+  const int dk = a.dk, dv = a.dv, e = blockIdx.z, hd = blockIdx.y, sl = blockIdx.x;
+  float* S = sm;                       // [dk][SV]
+  float* qs = S + dk * SV;             // [dk]
+  float* ks = qs + dk;
+  float* fs = ks + dk;
+  float* us = fs + dk;
+  float* vs = us + dk;                 // [SV]
+  float* part = vs + SV;               // [8][SV]
+  pdl_trigger();
+  pdl_wait();
+  const int t0 = a.rb.cu[e], t1 = a.rb.cu[e + 1], p0 = a.rb.pos0[e];
+  const int c0 = sl * SV, nc = min(SV, dv - c0), tid = threadIdx.x, col = tid & 31, rg = tid >> 5;
+  if (t0 >= t1) return;
+  if (p0 < 0) {
+    for (int t = t0; t < t1; ++t)
+      if (tid < nc) out[((long long)t * a.heads + hd) * dv + c0 + tid] = 0.f;
+    return;
+  }
+  const long long slot = a.rb.slot[e];
+  float* Sg = a.S + (slot * a.heads + hd) * dk * dv + c0;
+  for (int i = tid; i < dk * SV; i += GT) {
+    const int d = i / SV, c = i - d * SV;
+    S[i] = (p0 > 0 && c < nc) ? Sg[(long long)d * dv + c] : 0.f;
+  }
+  for (int t = t0; t < t1; ++t) {
+    for (int d = tid; d < dk; d += GT) {
+      const int c = hd * dk + d;
+      const float c1 = to_f(static_cast<const T*>(a.c1)[c]);
+      float q = to_f(static_cast<const T*>(a.q)[t * a.ldq + c]), k = 0.f, f;
+      if (MODE == BONUS) k = to_f(static_cast<const T*>(a.k)[t * a.ldk + c]);
+      else q = silu<T>(q);
+      gates_exact<MODE>(a.z[t * a.ldz + c], to_f(static_cast<const T*>(a.c0)[c]), c1, f, k);
+      qs[d] = q;
+      ks[d] = k;
+      fs[d] = f;
+      us[d] = MODE == BONUS ? c1 * k : 0.f;
+    }
+    if (tid < SV) vs[tid] = tid < nc ? to_f(static_cast<const T*>(a.v)[t * a.ldv + hd * dv + c0 + tid]) : 0.f;
+    __syncthreads();
+    float acc = 0.f;
+    const float v = vs[col];
+    for (int d = rg; d < dk; d += GT / 32) {
+      const float s = S[d * SV + col], n = fs[d] * s + ks[d] * v;
+      acc += qs[d] * (MODE == BONUS ? s + us[d] * v : n);
+      S[d * SV + col] = n;
+    }
+    part[rg * SV + col] = acc;
+    __syncthreads();
+    if (tid < nc) {
+      float o = 0.f;
+#pragma unroll
+      for (int j = 0; j < GT / 32; ++j) o += part[j * SV + tid];
+      out[((long long)t * a.heads + hd) * dv + c0 + tid] = o;
+    }
+  }
+  __syncthreads();
+  for (int i = tid; i < dk * SV; i += GT) {
+    const int d = i / SV, c = i - d * SV;
+    if (c < nc) Sg[(long long)d * dv + c] = S[i];
+  }
+  carry_rows<T>(a, t1 - 1, slot, hd * gridDim.x + sl, gridDim.x * gridDim.y);
+}
+
+// o fp32 [n, heads, dv] -> out T [n, heads * dv]: norm per head, weight, gate. One CTA per token, a warp per head.
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+head_norm_kernel(const GlaArgs a, const float* __restrict__ o, T* __restrict__ out) {
+  pdl_trigger();
+  pdl_wait();
+  const long long t = blockIdx.x;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5, dv = a.dv;
+  const T* w = static_cast<const T*>(a.nw);
+  const T* gate = a.gate ? static_cast<const T*>(a.gate) + t * a.ldg : nullptr;
+  for (int hd = warp; hd < a.heads; hd += nw) {
+    const float* x = o + (t * a.heads + hd) * dv;
+    float ss = 0.f;
+    for (int c = lane * V; c < dv; c += 32 * V) {
+      float v[V];
+      load_v<V>(x + c, v);
+#pragma unroll
+      for (int i = 0; i < V; ++i) ss += v[i] * v[i];
+    }
+    const float r = 1.f / sqrtf(warp_sum(ss) / (float)dv + a.eps);
+    for (int c = lane * V; c < dv; c += 32 * V) {
+      float v[V], ww[V], g[V];
+      load_v<V>(x + c, v);
+      load_v<V>(w + (a.per_head ? hd * dv + c : c), ww);
+      if (gate) load_v<V>(gate + hd * dv + c, g);
+#pragma unroll
+      for (int i = 0; i < V; ++i) v[i] *= r * ww[i] * (gate ? silu<T>(g[i]) : 1.f);
+      store_v<V>(out + t * a.heads * dv + hd * dv + c, v);
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------ portions, tensor cores
+// A CTA owns 64 value columns of one head, 16 per warp, and walks its entry in blocks of 16 tokens. With L_t the sum of log f
+// from the block's start through token t and L its end,
+//   o_t = (q_t e^(L_t)) S + sum_{s <= t} (q_t e^(L_t) . k_s e^(-L_s)) v_s,    S' = diag(e^L) S + sum_s (k_s e^(L - L_s)) v_s^T
+// (BONUS reads S before the token: L_(t-1), s < t, and the current token weighs q . (c1 k)).
+// S^T stays in fp32 accumulators [16 values, dk]: their layout is that of the B operand of q S, so the state is packed to bf16
+// for the read-out without leaving registers. The updates k e^(L - L_s) go to the tensor cores as bf16 pairs hi + lo, v is
+// bf16 and exact. Several blocks are prepared at once (TT tokens); every warp prepares one block (half of its channels at
+// dk > 64), so a tile of tokens costs two barriers.
+// e^(-L_s) must stay finite: where some channel decays by more than e^-SAFE within a block, the tile's weights are summed
+// directly, with e^(L_t - L_s) per pair and channel.
+constexpr int DV = 64;
+constexpr float SAFE = 60.f;
+constexpr int VPITCH = DV * 2 + 16;
+constexpr int PPITCH = 48;
+
+struct ChunkSmem {
+  int tt, pitch, q, k, z, v, Q, Ki, Kh, Kl, P, D, dg, ssq, total;
+};
+__host__ __device__ constexpr ChunkSmem chunk_smem(int KP) {
+  ChunkSmem L{};
+  L.tt = 4096 / KP;
+  L.pitch = KP * 2 + 16;
+  L.q = 0;
+  L.k = L.q + L.tt * L.pitch;
+  L.z = L.k + L.tt * L.pitch;
+  L.v = L.z + L.tt * KP * 4;
+  L.Q = L.v + 2 * L.tt * VPITCH;
+  L.Ki = L.Q + L.tt * L.pitch;
+  L.Kh = L.Ki + L.tt * L.pitch;
+  L.Kl = L.Kh + L.tt * L.pitch;
+  L.P = L.Kl + L.tt * L.pitch;
+  L.D = L.P + (L.tt / 16) * 16 * PPITCH;
+  L.dg = L.D + (L.tt / 16) * KP * 4;
+  L.ssq = L.dg + (KP / 64) * L.tt * 4;
+  L.total = L.ssq + 4 * L.tt * 4;
+  return L;
+}
+
+template <int KP, int MODE>
+__global__ void __launch_bounds__(128)
+gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  constexpr ChunkSmem M = chunk_smem(KP);
+  constexpr int TT = M.tt, SUBS = TT / 16, HALVES = KP / 64, KT = KP / 8;
+  const uint32_t sb = smem_u32(smem);
+  float* Dd = reinterpret_cast<float*>(smem + M.D);     // [SUBS][KP] e^L
+  float* Dg = reinterpret_cast<float*>(smem + M.dg);    // [HALVES][TT] q . (c1 k)
+  float* Ssq = reinterpret_cast<float*>(smem + M.ssq);  // [4][TT]
+  const float* Z = reinterpret_cast<const float*>(smem + M.z);
+  pdl_trigger();
+  pdl_wait();
+  const int dk = a.dk, dv = a.dv, e = blockIdx.z, hd = blockIdx.y, sl = blockIdx.x;
+  const int p0 = a.rb.pos0[e], t0 = a.rb.cu[e], len = a.rb.cu[e + 1] - t0;
+  if (p0 < 0 || len <= 0) return;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, li = lane >> 3, lr = lane & 7;
+  const int g = lane >> 2, qd = 2 * (lane & 3);         // row and first column of this lane in an accumulator tile
+  const int c0 = sl * DV, nc = min(DV, dv - c0), v0 = warp * 16;
+  const bool active = v0 < nc;
+  const long long slot = a.rb.slot[e];
+  float* Sg = a.S + (slot * a.heads + hd) * dk * dv + c0;
+
+  const bf* qg = static_cast<const bf*>(a.q) + (long long)t0 * a.ldq + hd * dk;
+  const bf* kg = MODE == BONUS ? static_cast<const bf*>(a.k) + (long long)t0 * a.ldk + hd * dk : nullptr;
+  const bf* vg = static_cast<const bf*>(a.v) + (long long)t0 * a.ldv + hd * dv + c0;
+  const float* zg = a.z + (long long)t0 * a.ldz + hd * dk;
+  auto load = [&](int tile) {
+    const int at = tile * TT, rows = min(TT, len - at);
+    for (int i = tid; i < TT * (KP / 8); i += 128) {
+      const int r = i / (KP / 8), c = i % (KP / 8);
+      const bool ok = r < rows && c * 8 < dk;
+      cp_async16(sb + M.q + r * M.pitch + c * 16, qg + (ok ? (at + r) * a.ldq + c * 8 : 0), ok ? 16 : 0);
+      if (MODE == BONUS) cp_async16(sb + M.k + r * M.pitch + c * 16, kg + (ok ? (at + r) * a.ldk + c * 8 : 0), ok ? 16 : 0);
+    }
+    for (int i = tid; i < TT * (KP / 4); i += 128) {
+      const int r = i / (KP / 4), c = i % (KP / 4);
+      const bool ok = r < rows && c * 4 < dk;
+      cp_async16(sb + M.z + r * (KP * 4) + c * 16, zg + (ok ? (at + r) * a.ldz + c * 4 : 0), ok ? 16 : 0);
+    }
+    const uint32_t vb = sb + M.v + (tile & 1) * TT * VPITCH;
+    for (int i = tid; i < TT * (DV / 8); i += 128) {
+      const int r = i / (DV / 8), c = i % (DV / 8);
+      const bool ok = r < rows && c * 8 < nc;
+      cp_async16(vb + r * VPITCH + c * 16, vg + (ok ? (at + r) * a.ldv + c * 8 : 0), ok ? 16 : 0);
+    }
+    cp_async_commit();
+  };
+  load(0);
+
+  // S^T: tile j holds channels 8 j + qd, + 1 of values v0 + g (elements 0, 1) and v0 + g + 8 (2, 3)
+  float S[KT][4];
+#pragma unroll
+  for (int j = 0; j < KT; ++j)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int d = j * 8 + qd + (i & 1), v = v0 + g + (i >> 1) * 8;
+      S[j][i] = (p0 > 0 && d < dk && v < nc) ? Sg[(long long)d * dv + v] : 0.f;
+    }
+
+  // the block and the two channels this lane prepares
+  const int psub = warp / HALVES, pd = (warp % HALVES) * 64 + 2 * lane;
+  float b0[2], b1[2];
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const bool ok = pd + i < dk;
+    b0[i] = ok ? to_f(static_cast<const bf*>(a.c0)[hd * dk + pd + i]) : 0.f;
+    b1[i] = ok ? to_f(static_cast<const bf*>(a.c1)[hd * dk + pd + i]) : (MODE == LOWER ? 1.f : 0.f);
+  }
+
+  const int tiles = (len + TT - 1) / TT;
+  for (int tile = 0; tile < tiles; ++tile) {
+    const int rows = min(TT, len - tile * TT);
+    cp_async_wait<0>();
+    __syncthreads();                    // the tile is in; nobody reads the last tile's operands any more
+    float L[16][2], kk[16][2];
+    {
+      float run0 = 0.f, run1 = 0.f;
+#pragma unroll
+      for (int t = 0; t < 16; ++t) {
+        const int row = psub * 16 + t;
+        const float2 z = *reinterpret_cast<const float2*>(Z + row * KP + pd);
+        float l0 = gates_log<MODE>(z.x, b0[0], b1[0], kk[t][0]), l1 = gates_log<MODE>(z.y, b0[1], b1[1], kk[t][1]);
+        if (MODE == BONUS) {
+          const uint32_t k2 = *reinterpret_cast<const uint32_t*>(smem + M.k + row * M.pitch + pd * 2);
+          kk[t][0] = bf16_lo(k2);
+          kk[t][1] = bf16_hi(k2);
+        }
+        if (row >= rows) l0 = l1 = kk[t][0] = kk[t][1] = 0.f;
+        run0 += l0;
+        run1 += l1;
+        L[t][0] = run0;
+        L[t][1] = run1;
+      }
+    }
+    const float e0 = L[15][0], e1 = L[15][1];
+    float dg[16];
+#pragma unroll
+    for (int t = 0; t < 16; ++t) {
+      const int row = psub * 16 + t;
+      const uint32_t at = row * M.pitch + pd * 2;
+      const uint32_t q2 = *reinterpret_cast<const uint32_t*>(smem + M.q + at);
+      float q0 = bf16_lo(q2), q1 = bf16_hi(q2);
+      if (MODE == LOWER) { q0 = silu<bf>(q0); q1 = silu<bf>(q1); }
+      else dg[t] = q0 * b1[0] * kk[t][0] + q1 * b1[1] * kk[t][1];
+      float x0, x1;                     // decay from the block's start to the read-out
+      if (MODE == LOWER) { x0 = quick_exp(L[t][0]); x1 = quick_exp(L[t][1]); }
+      else if (t == 0) x0 = x1 = 1.f;
+      else { x0 = quick_exp(L[t > 0 ? t - 1 : 0][0]); x1 = quick_exp(L[t > 0 ? t - 1 : 0][1]); }
+      *reinterpret_cast<uint32_t*>(smem + M.Q + at) = pack_bf16(q0 * x0, q1 * x1);
+      *reinterpret_cast<uint32_t*>(smem + M.Ki + at) = pack_bf16(kk[t][0] * quick_exp(fminf(-L[t][0], SAFE)), kk[t][1] * quick_exp(fminf(-L[t][1], SAFE)));
+      bf h0, h1, l0, l1;
+      split_bf16(kk[t][0] * quick_exp(e0 - L[t][0]), h0, l0);
+      split_bf16(kk[t][1] * quick_exp(e1 - L[t][1]), h1, l1);
+      *reinterpret_cast<__nv_bfloat162*>(smem + M.Kh + at) = __halves2bfloat162(h0, h1);
+      *reinterpret_cast<__nv_bfloat162*>(smem + M.Kl + at) = __halves2bfloat162(l0, l1);
+    }
+    *reinterpret_cast<float2*>(Dd + psub * KP + pd) = make_float2(quick_exp(e0), quick_exp(e1));
+    if (MODE == BONUS) {
+#pragma unroll
+      for (int t = 0; t < 16; ++t) {
+        const float s = warp_sum(dg[t]);
+        if (lane == 0) Dg[(warp % HALVES) * TT + psub * 16 + t] = s;
+      }
+    }
+    const bool direct = __syncthreads_or(fminf(e0, e1) < -SAFE);
+    if (direct) {
+      // L, q and k of the whole tile go to shared memory, then one thread per weight
+#pragma unroll
+      for (int t = 0; t < 16; ++t) {
+        const int row = psub * 16 + t;
+        const uint32_t at = row * M.pitch + pd * 2;
+        *reinterpret_cast<float2*>(smem + M.z + (row * KP + pd) * 4) = make_float2(L[t][0], L[t][1]);
+        *reinterpret_cast<uint32_t*>(smem + M.k + at) = pack_bf16(kk[t][0], kk[t][1]);
+        if (MODE == LOWER) {
+          uint32_t* q2 = reinterpret_cast<uint32_t*>(smem + M.q + at);
+          *q2 = pack_bf16(silu<bf>(bf16_lo(*q2)), silu<bf>(bf16_hi(*q2)));
+        }
+      }
+      __syncthreads();
+      for (int i = tid; i < SUBS * 256; i += 128) {
+        const int sub = i >> 8, t = (i >> 4) & 15, s = i & 15, rt = sub * 16 + t, rs = sub * 16 + s;
+        float p = 0.f;
+        if (MODE == BONUS && s == t) {
+#pragma unroll
+          for (int h = 0; h < HALVES; ++h) p += Dg[h * TT + rt];
+        } else if (s <= t) {
+          const bf* q = reinterpret_cast<const bf*>(smem + M.q + rt * M.pitch);
+          const bf* k = reinterpret_cast<const bf*>(smem + M.k + rs * M.pitch);
+          const float *Lt = Z + (MODE == BONUS ? rt - 1 : rt) * KP, *Ls = Z + rs * KP;
+          for (int d = 0; d < dk; ++d) p += to_f(q[d]) * to_f(k[d]) * quick_exp(Lt[d] - Ls[d]);
+        }
+        *reinterpret_cast<bf*>(smem + M.P + (sub * 16 + t) * PPITCH + s * 2) = __float2bfloat16(p);
+      }
+      __syncthreads();
+    }
+    if (tile + 1 < tiles) load(tile + 1);
+
+    float O[SUBS][2][4];
+    const uint32_t vb = sb + M.v + (tile & 1) * TT * VPITCH;
+    if (active) {
+#pragma unroll
+      for (int sub = 0; sub < SUBS; ++sub) {
+        float P[2][4];
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int i = 0; i < 4; ++i) O[sub][j][i] = P[j][i] = 0.f;
+        const uint32_t r_nt = sub * 16 + (li & 1) * 8 + lr, r_b = sub * 16 + (li >> 1) * 8 + lr;
+#pragma unroll
+        for (int ks = 0; ks < KP / 16; ++ks) {
+          uint32_t q[4], k[4];
+          ldsm_x4(q, sb + M.Q + r_nt * M.pitch + (ks * 2 + (li >> 1)) * 16);
+          ldsm_x4(k, sb + M.Ki + r_b * M.pitch + (ks * 2 + (li & 1)) * 16);
+          mma_16816(P[0], q, k[0], k[1]);
+          mma_16816(P[1], q, k[2], k[3]);
+          mma_16816(O[sub][0], q, pack_bf16(S[2 * ks][0], S[2 * ks][1]), pack_bf16(S[2 * ks + 1][0], S[2 * ks + 1][1]));
+          mma_16816(O[sub][1], q, pack_bf16(S[2 * ks][2], S[2 * ks][3]), pack_bf16(S[2 * ks + 1][2], S[2 * ks + 1][3]));
+        }
+        uint32_t ap[4], bv[4], av[4];
+        if (direct) {
+          ldsm_x4(ap, sb + M.P + r_nt * PPITCH + (li >> 1) * 16);
+        } else {
+#pragma unroll
+          for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+              const int t = g + (i >> 1) * 8, s = j * 8 + qd + (i & 1);
+              if (s > t) P[j][i] = 0.f;
+              if (MODE == BONUS && s == t) {
+                P[j][i] = Dg[sub * 16 + t];
+                if (HALVES == 2) P[j][i] += Dg[TT + sub * 16 + t];
+              }
+            }
+          ap[0] = pack_bf16(P[0][0], P[0][1]);
+          ap[1] = pack_bf16(P[0][2], P[0][3]);
+          ap[2] = pack_bf16(P[1][0], P[1][1]);
+          ap[3] = pack_bf16(P[1][2], P[1][3]);
+        }
+        ldsm_x4_t(bv, vb + r_nt * VPITCH + (v0 / 8 + (li >> 1)) * 16);
+        mma_16816(O[sub][0], ap, bv[0], bv[1]);
+        mma_16816(O[sub][1], ap, bv[2], bv[3]);
+        ldsm_x4_t(av, vb + r_b * VPITCH + (v0 / 8 + (li & 1)) * 16);
+#pragma unroll
+        for (int j = 0; j < KT; j += 2) {
+          const float2 d0 = *reinterpret_cast<const float2*>(Dd + sub * KP + j * 8 + qd);
+          const float2 d1 = *reinterpret_cast<const float2*>(Dd + sub * KP + j * 8 + 8 + qd);
+          S[j][0] *= d0.x; S[j][1] *= d0.y; S[j][2] *= d0.x; S[j][3] *= d0.y;
+          S[j + 1][0] *= d1.x; S[j + 1][1] *= d1.y; S[j + 1][2] *= d1.x; S[j + 1][3] *= d1.y;
+          uint32_t k[4];
+          ldsm_x4_t(k, sb + M.Kh + r_nt * M.pitch + (j + (li >> 1)) * 16);
+          mma_16816(S[j], av, k[0], k[1]);
+          mma_16816(S[j + 1], av, k[2], k[3]);
+          ldsm_x4_t(k, sb + M.Kl + r_nt * M.pitch + (j + (li >> 1)) * 16);
+          mma_16816(S[j], av, k[0], k[1]);
+          mma_16816(S[j + 1], av, k[2], k[3]);
+        }
+      }
+    }
+    // outputs: of a whole head normed and gated here, of a slice in fp32 for head_norm
+    if (out != nullptr) {
+#pragma unroll
+      for (int sub = 0; sub < SUBS; ++sub)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          float s = 0.f;
+          if (active) {
+#pragma unroll
+            for (int j = 0; j < 2; ++j) s += O[sub][j][2 * h] * O[sub][j][2 * h] + O[sub][j][2 * h + 1] * O[sub][j][2 * h + 1];
+          }
+          s += __shfl_xor_sync(0xffffffffu, s, 1);
+          s += __shfl_xor_sync(0xffffffffu, s, 2);
+          if ((lane & 3) == 0) Ssq[warp * TT + sub * 16 + g + h * 8] = s;
+        }
+      __syncthreads();
+    }
+    if (active) {
+#pragma unroll
+      for (int sub = 0; sub < SUBS; ++sub)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          const int r = sub * 16 + g + h * 8;
+          if (r >= rows) continue;
+          const long long t = t0 + tile * TT + r;
+          float rstd = 1.f;
+          if (out != nullptr) rstd = 1.f / sqrtf((Ssq[r] + Ssq[TT + r] + Ssq[2 * TT + r] + Ssq[3 * TT + r]) / (float)dv + a.eps);
+#pragma unroll
+          for (int j = 0; j < 2; ++j) {
+            const int c = c0 + v0 + j * 8 + qd;
+            if (c >= dv) continue;                      // dv is a multiple of 8
+            const float x0 = O[sub][j][2 * h], x1 = O[sub][j][2 * h + 1];
+            if (out == nullptr) {
+              *reinterpret_cast<float2*>(raw + (t * a.heads + hd) * dv + c) = make_float2(x0, x1);
+            } else {
+              const uint32_t w2 = *reinterpret_cast<const uint32_t*>(static_cast<const bf*>(a.nw) + (a.per_head ? hd * dv + c : c));
+              float y0 = x0 * rstd * bf16_lo(w2), y1 = x1 * rstd * bf16_hi(w2);
+              if (a.gate) {
+                const uint32_t g2 = *reinterpret_cast<const uint32_t*>(static_cast<const bf*>(a.gate) + t * a.ldg + hd * dv + c);
+                y0 *= silu<bf>(bf16_lo(g2));
+                y1 *= silu<bf>(bf16_hi(g2));
+              }
+              *reinterpret_cast<uint32_t*>(out + t * a.heads * dv + hd * dv + c) = pack_bf16(y0, y1);
+            }
+          }
+        }
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < KT; ++j)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int d = j * 8 + qd + (i & 1), v = v0 + g + (i >> 1) * 8;
+      if (d < dk && v < nc) Sg[(long long)d * dv + v] = S[j][i];
+    }
+  carry_rows<bf>(a, t0 + len - 1, slot, hd * gridDim.x + sl, gridDim.x * gridDim.y);
+}
+
+template <int KP, int MODE>
+int launch_chunk(const GlaArgs& a, float* raw, bf* out, cudaStream_t stream) {
+  constexpr int smem = chunk_smem(KP).total;
+  static DeviceOnce once;
+  if (once.first() &&
+      cudaFuncSetAttribute(gla_chunk_kernel<KP, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -5;
+  const dim3 grid((a.dv + DV - 1) / DV, a.heads, a.rb.E);
+  return launch_pdl(gla_chunk_kernel<KP, MODE>, grid, dim3(128), smem, stream, a, raw, out) == cudaSuccess ? 0 : -5;
+}
+
+template <typename T, int MODE, int V>
+int launch_step(const GlaArgs& a, T* out, cudaStream_t stream) {
+  const int R = GT / (a.dv / V);
+  const size_t smem = ((size_t)4 * a.dk + (size_t)R * a.dv) * 4;
+  static DeviceOnce once;
+  if (smem > 200 * 1024) return -2;
+  if (once.first() &&
+      cudaFuncSetAttribute(gla_step_kernel<T, MODE, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess) return -5;
+  return launch_pdl(gla_step_kernel<T, MODE, V>, dim3(a.heads, a.rb.E), dim3(GT), smem, stream, a, out) == cudaSuccess ? 0 : -5;
+}
+
+template <typename T, int MODE>
+int run(const GlaArgs& a, float* raw, T* out, int one, int chunked, cudaStream_t stream) {
+  if (one) {
+    const bool vec = a.dv % 4 == 0 && a.ldv % 4 == 0 && a.dk % 4 == 0;
+    if (vec && a.dv <= 4 * GT) return launch_step<T, MODE, 4>(a, out, stream);
+    if (a.dv <= GT) return launch_step<T, MODE, 1>(a, out, stream);
+  }
+  bool normed = false;
+  if constexpr (sizeof(T) == 2) {
+    if (chunked && !one && a.dk <= 128 && a.dk % 8 == 0 && a.dv % 8 == 0 && a.ldq % 8 == 0 && a.ldv % 8 == 0 && a.ldz % 4 == 0 &&
+        (MODE == LOWER || a.ldk % 8 == 0) && a.ldg % 2 == 0) {
+      normed = a.dv <= DV;
+      bf* o = normed ? out : nullptr;
+      const int rc = a.dk <= 64 ? launch_chunk<64, MODE>(a, raw, o, stream) : launch_chunk<128, MODE>(a, raw, o, stream);
+      if (rc) return rc;
+      if (normed) return 0;
+      chunked = 2;
+    }
+  }
+  if (chunked != 2) {
+    const size_t smem = ((size_t)a.dk * (SV + 4) + SV + (GT / 32) * SV) * 4;
+    static DeviceOnce once;
+    if (smem > 220 * 1024) return -2;
+    if (once.first() &&
+        cudaFuncSetAttribute(gla_seq_kernel<T, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024) != cudaSuccess) return -5;
+    const dim3 grid((a.dv + SV - 1) / SV, a.heads, a.rb.E);
+    if (launch_pdl(gla_seq_kernel<T, MODE>, grid, dim3(GT), smem, stream, a, raw) != cudaSuccess) return -5;
+  }
+  const bool vec = a.dv % 4 == 0 && a.ldg % 4 == 0;
+  const dim3 grid(a.rb.n);
+  const cudaError_t err = vec ? launch_pdl(head_norm_kernel<T, 4>, grid, dim3(256), 0, stream, a, (const float*)raw, out)
+                              : launch_pdl(head_norm_kernel<T, 1>, grid, dim3(256), 0, stream, a, (const float*)raw, out);
+  return err == cudaSuccess ? 0 : -5;
+}
+
+}  // namespace
+
+// mode: 0 BONUS, 1 LOWER. q, k [n, heads * dk], v, gate [n, heads * dv] (row strides ld*; k null with LOWER, gate may be null),
+// z fp32 [n, heads * dk] with row stride ldz; c0, c1 T [heads * dk]; S fp32 [slots, heads, dk, dv].
+// h T [n, D] / carry fp32 [slots, D] (or null): last rows of portions kept for the token shift (not with `one`).
+// nw T [dv], or [heads * dv] with per_head; raw fp32 [n, heads * dv] workspace; out T [n, heads * dv].
+// one: every entry is one token. chunked: bf16 portions take the tensor-core form where the sizes allow.
+TB_API int tb_gated_linear(int dtype, int mode, const void* q, long long ldq, const void* k, long long ldk, const void* v,
+                           long long ldv, const void* gate, long long ldg, const float* z, long long ldz, const void* c0,
+                           const void* c1, const int* cu, const int* slot, const int* pos0, const int* ent, int E, int n,
+                           int heads, int dk, int dv, float* S, const void* h, float* carry, int D, const void* nw, int per_head,
+                           float eps, float* raw, void* out, int one, int chunked, cudaStream_t stream) {
+  if (n <= 0 || E <= 0) return 0;
+  if (heads <= 0 || dk <= 0 || dv <= 0 || E > 65535 || heads > 65535 || (mode != BONUS && mode != LOWER) || (mode == BONUS && !k)) return -2;
+  GlaArgs a{q, k, v, gate, ldq, ldk, ldv, ldg, z, ldz, c0, c1, heads, dk, dv, Ragged{cu, slot, pos0, ent, E, n}, S, h, carry, D,
+            nw, per_head, eps};
+  if (dtype == 0)
+    return mode == BONUS ? run<bf, BONUS>(a, raw, (bf*)out, one, chunked, stream) : run<bf, LOWER>(a, raw, (bf*)out, one, chunked, stream);
+  return mode == BONUS ? run<float, BONUS>(a, raw, (float*)out, one, chunked, stream) : run<float, LOWER>(a, raw, (float*)out, one, chunked, stream);
+}

@@ -102,6 +102,13 @@ __device__ __forceinline__ float quick_gelu_tanh(float z) {
   return z * quick_sigmoid(1.5957691216057308f * (z + 0.044715f * z * z * z));
 }
 
+// First visible position of a query at position i: a sliding window of `window` keys and / or chunks of `chunk` positions
+// counted from the start of the sequence (<= 0: none).
+__device__ __forceinline__ int first_visible(int i, int window, int chunk) {
+  const int w = window > 0 ? max(0, i - window + 1) : 0;
+  return chunk > 0 ? max(w, i - i % chunk) : w;
+}
+
 // A ragged batch: entry e holds tokens cu[e] .. cu[e+1]-1 of the flat token list, which continue the sequence in slot
 // slot[e] at position pos0[e] (negative: an idle slot, nothing is read or written for it).
 struct Ragged {

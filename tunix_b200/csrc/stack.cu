@@ -5,8 +5,15 @@
 //   stream_step : one launch between two sublayers. It closes the sublayer before it (streams <- mix^T streams +
 //                 out * y) and opens the one after it (u = in . streams, h = RMS norm(u) * w), so that the streams are
 //                 read and written once per sublayer. y is one tensor, or half the sum of two tensors that are
-//                 RMS-normed first (two mixers side by side). The first launch of a forward pass takes the embedding
-//                 rows instead of streams, the last one has no successor but the final norm.
+//                 RMS-normed first (two mixers side by side), or one tensor that is RMS-normed first (an update with a
+//                 norm of its own). The first launch of a forward pass takes the embedding rows (normed, if the model
+//                 norms them) instead of streams, the last one has no successor but the final norm. Norms may run over
+//                 equal groups of a row. Without a norm the row itself is written in the activation type. In a decode
+//                 step the launch can also mix the new row with the one before it (token shift).
+//   token_shift : the same mixes for portions of prompts.
+//   few_outputs, small_act : products with a handful of outputs, and what is applied to them (tanh; gelu times a row
+//                 that belongs to the token).
+//   xielu       : the activation of feed-forwards without a gate.
 //
 // This file is compiled without fast-math: the same kernels serve the 32-bit mode.
 #include "precise.cuh"
@@ -24,7 +31,7 @@ struct StreamArgs {
   // the sublayer that just ended
   const void* y;              // T [n, D] or null
   const void* y2;             // T [n, D] or null: y and y2 are normed, weighted and averaged
-  const void* wy;             // T [D]
+  const void* wy;             // T [D]; with y2 null: y alone is normed and weighted
   const void* wy2;            // T [D]
   const void* mix;            // T [S, S], row = from, column = to
   const void* out;            // T [S]
@@ -32,18 +39,52 @@ struct StreamArgs {
   const long long* tokens;    // [n] or null
   const void* embed;          // T [V, D]
   int vocab;
+  const void* embed_w;        // T [D] or null: weight of the norm of the embedding rows
+  int groups;                 // equal parts of a row that the norms of embedding and streams are taken over
   // the sublayer that follows
   const void* in;             // T [S]; null = all ones (the sum of the streams)
   const void* w;              // T [D] norm weight
   void* h;                    // T [n, D]
   float* sum_out;             // fp32 [n, D] or null: the sum of the streams
+  // token shift of a batch of single tokens (row = entry): mixes T [n_mix, n, D] instead of h
+  const void* mu;             // T [n_mix, D] or null
+  int n_mix;
+  float* before;              // fp32 [slots, D]: the normed row of the token before, replaced by this one
+  void* mixes;
+  const int *slot, *pos0;
 };
+
+// 1 / rms of every group of the row u [D] in shared memory -> rs [groups]; part [groups + warps] is scratch. Starts and
+// ends with a barrier.
+__device__ __forceinline__ void group_rstd(const float* u, int D, int groups, float eps, float* part, float* rs) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  const int per = (nw + groups - 1) / groups, len = D / groups;
+  __syncthreads();
+  for (int i = warp; i < groups * per; i += nw) {
+    const int g = i / per, p = i - g * per;
+    const int a = g * len + (int)((long long)len * p / per), b = g * len + (int)((long long)len * (p + 1) / per);
+    float s = 0.f;
+    for (int d = a + lane; d < b; d += 32) s += u[d] * u[d];
+    s = warp_sum(s);
+    if (lane == 0) part[i] = s;
+  }
+  __syncthreads();
+  for (int g = threadIdx.x; g < groups; g += blockDim.x) {
+    float s = 0.f;
+    for (int p = 0; p < per; ++p) s += part[g * per + p];
+    rs[g] = 1.f / sqrtf(s / (float)len + eps);
+  }
+  __syncthreads();
+}
 
 // V elements of a row per thread and iteration (4, or 1 for widths that are no multiple of 4)
 template <typename T, int S, int V>
 __global__ void __launch_bounds__(512) stream_step_kernel(const StreamArgs a) {
-  extern __shared__ float u_s[];          // [D]
+  extern __shared__ float u_s[];          // [D], then scratch of the grouped norms
   __shared__ float red[33];
+  float* part = u_s + ((a.D + 3) & ~3);   // [groups + warps]
+  float* rs = part + a.groups + 32;       // [groups]
+  const int glen = a.D / a.groups;
   pdl_trigger();
   pdl_wait();
   const long long row = blockIdx.x;
@@ -60,6 +101,16 @@ __global__ void __launch_bounds__(512) stream_step_kernel(const StreamArgs a) {
   const T* y = a.y ? static_cast<const T*>(a.y) + row * D : nullptr;
   const T* y2 = a.y2 ? static_cast<const T*>(a.y2) + row * D : nullptr;
   float r1 = 1.f, r2 = 0.f;
+  if (a.wy && !y2) {
+    float s1 = 0.f;
+    for (int d = threadIdx.x * V; d < D; d += step) {
+      float v1[V];
+      load_v<V>(y + d, v1);
+#pragma unroll
+      for (int i = 0; i < V; ++i) s1 += v1[i] * v1[i];
+    }
+    r1 = 1.f / sqrtf(block_sum(s1, red) / (float)D + a.eps);
+  }
   if (y2) {
     float s1 = 0.f, s2 = 0.f;
     for (int d = threadIdx.x * V; d < D; d += step) {
@@ -79,6 +130,14 @@ __global__ void __launch_bounds__(512) stream_step_kernel(const StreamArgs a) {
     long long t = a.tokens[row];
     t = t < 0 ? 0 : (t >= a.vocab ? a.vocab - 1 : t);
     emb = static_cast<const T*>(a.embed) + t * D;
+    if (a.embed_w) {
+      for (int d = threadIdx.x * V; d < D; d += step) {
+        float ev[V];
+        load_v<V>(emb + d, ev);
+        store_v<V>(u_s + d, ev);
+      }
+      group_rstd(u_s, D, a.groups, a.eps, part, rs);
+    }
   }
   float ss = 0.f;
   for (int d = threadIdx.x * V; d < D; d += step) {
@@ -86,6 +145,12 @@ __global__ void __launch_bounds__(512) stream_step_kernel(const StreamArgs a) {
     if (emb) {
       float ev[V];
       load_v<V>(emb + d, ev);
+      if (a.embed_w) {
+        float w[V];
+        load_v<V>(static_cast<const T*>(a.embed_w) + d, w);
+#pragma unroll
+        for (int i = 0; i < V; ++i) ev[i] *= rs[(d + i) / glen] * w[i];
+      }
 #pragma unroll
       for (int s = 0; s < S; ++s)
 #pragma unroll
@@ -104,6 +169,11 @@ __global__ void __launch_bounds__(512) stream_step_kernel(const StreamArgs a) {
           load_v<V>(static_cast<const T*>(a.wy2) + d, w2);
 #pragma unroll
           for (int i = 0; i < V; ++i) yv[i] = yv[i] * r1 * w1[i] + v2[i] * r2 * w2[i];
+        } else if (a.wy) {
+          float w1[V];
+          load_v<V>(static_cast<const T*>(a.wy) + d, w1);
+#pragma unroll
+          for (int i = 0; i < V; ++i) yv[i] *= r1 * w1[i];
         }
 #pragma unroll
         for (int t = 0; t < S; ++t)
@@ -134,17 +204,57 @@ __global__ void __launch_bounds__(512) stream_step_kernel(const StreamArgs a) {
     if (a.sum_out) store_v<V>(a.sum_out + row * D + d, tot);
     store_v<V>(u_s + d, u);
   }
-  if (!a.h) return;
-  ss = block_sum(ss, red);
-  const float r = 1.f / sqrtf(ss / (float)D + a.eps);
-  T* h = static_cast<T*>(a.h) + row * D;
+  if (!a.h && !a.mu) return;
+  if (!a.w) {                                            // the row itself
+    T* h = static_cast<T*>(a.h) + row * D;
+    for (int d = threadIdx.x * V; d < D; d += step) {
+      float u[V];
+      load_v<V>(u_s + d, u);
+      store_v<V>(h + d, u);
+    }
+    return;
+  }
+  float r = 1.f;
+  if (a.groups > 1) {
+    group_rstd(u_s, D, a.groups, a.eps, part, rs);
+  } else {
+    r = 1.f / sqrtf(block_sum(ss, red) / (float)D + a.eps);
+  }
+  T* h = a.h ? static_cast<T*>(a.h) + row * D : nullptr;
+  const int p0 = a.mu ? a.pos0[row] : 0;
+  float* before = a.mu ? a.before + (long long)a.slot[row] * D : nullptr;
   for (int d = threadIdx.x * V; d < D; d += step) {      // each thread reads back what it wrote
     float u[V], w[V];
     load_v<V>(u_s + d, u);
     load_v<V>(static_cast<const T*>(a.w) + d, w);
+    if (a.groups > 1) {
+      const int g = d / glen;
+      if (V == 1 || d + V - 1 < (g + 1) * glen) {
+        const float rg = rs[g];
 #pragma unroll
-    for (int i = 0; i < V; ++i) u[i] = u[i] * r * w[i];
-    store_v<V>(h + d, u);
+        for (int i = 0; i < V; ++i) u[i] *= rg * w[i];
+      } else {
+#pragma unroll
+        for (int i = 0; i < V; ++i) u[i] *= rs[(d + i) / glen] * w[i];
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < V; ++i) u[i] = u[i] * r * w[i];
+    }
+    if (h) store_v<V>(h + d, u);
+    if (a.mu) {
+      float b[V], m[V];
+#pragma unroll
+      for (int i = 0; i < V; ++i) { u[i] = to_f(from_f<T>(u[i])); b[i] = 0.f; }
+      if (p0 > 0) load_v<V>(before + d, b);
+      for (int k = 0; k < a.n_mix; ++k) {
+        load_v<V>(static_cast<const T*>(a.mu) + (long long)k * D + d, m);
+#pragma unroll
+        for (int i = 0; i < V; ++i) m[i] = u[i] + (b[i] - u[i]) * m[i];
+        store_v<V>(static_cast<T*>(a.mixes) + ((long long)k * gridDim.x + row) * D + d, m);
+      }
+      if (p0 >= 0) store_v<V>(before + d, u);
+    }
   }
 }
 
@@ -154,8 +264,9 @@ cudaError_t launch_stream_step(const StreamArgs& a, int n, cudaStream_t stream) 
   const int per = vec ? a.D / 4 : a.D;
   int threads = n <= 296 ? 512 : 256;              // few rows: the latency of one row counts
   while (threads > 128 && threads / 2 >= per) threads /= 2;
-  if (vec) return launch_pdl(stream_step_kernel<T, S, 4>, dim3(n), dim3(threads), (size_t)a.D * 4, stream, a);
-  return launch_pdl(stream_step_kernel<T, S, 1>, dim3(n), dim3(threads), (size_t)a.D * 4, stream, a);
+  const size_t smem = (size_t)(((a.D + 3) & ~3) + 2 * a.groups + 32) * 4;
+  if (vec) return launch_pdl(stream_step_kernel<T, S, 4>, dim3(n), dim3(threads), smem, stream, a);
+  return launch_pdl(stream_step_kernel<T, S, 1>, dim3(n), dim3(threads), smem, stream, a);
 }
 
 template <typename T>
@@ -237,10 +348,27 @@ gate_outputs_kernel(const T* __restrict__ attn, const float* __restrict__ o, con
   }
 }
 
-// out[t, o] = sum_k x[t, k] w[o, k] in fp32, for a handful of outputs and few rows (gates of a decode step): one CTA per
-// row, a warp per output.
+// What is applied to a few outputs: 0 nothing, 1 tanh, 2 gelu (tanh form) times a row of the token's own,
+// e[tokens[t], e_off + o].
+template <typename T>
+__device__ __forceinline__ float apply_small(int act, float z, const long long* tokens, int vocab, const T* e, long long lde,
+                                             int e_off, long long t, int o) {
+  if (act == 1) return tanhf(z);
+  if (act == 2) {
+    long long id = tokens[t];
+    id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
+    return gelu_tanh(z) * to_f(e[id * lde + e_off + o]);
+  }
+  return z;
+}
+
+// out[t, o] = act(sum_k x[t, k] w[o, k]) with an fp32 sum, for a handful of outputs and few rows (gates of a decode step):
+// one CTA per row, a warp per output.
+template <typename TO>
 __global__ void __launch_bounds__(512)
-few_outputs_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ w, int K, int N, float* __restrict__ out) {
+few_outputs_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ w, int K, int N, int act,
+                   const long long* __restrict__ tokens, int vocab, const __nv_bfloat16* __restrict__ e, long long lde, int e_off,
+                   TO* __restrict__ out) {
   pdl_trigger();
   pdl_wait();
   const long long t = blockIdx.x;
@@ -256,7 +384,81 @@ few_outputs_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __r
       for (int i = 0; i < 8; ++i) acc += a[i] * b[i];
     }
     acc = warp_sum(acc);
-    if (lane == 0) out[t * N + o] = acc;
+    if (lane == 0) out[t * N + o] = from_f<TO>(apply_small(act, acc, tokens, vocab, e, lde, e_off, t, o));
+  }
+}
+
+// out[t, o] = act(z[t, o])
+template <typename T>
+__global__ void small_act_kernel(const float* __restrict__ z, int N, long long total, int act, const long long* __restrict__ tokens,
+                                 int vocab, const T* __restrict__ e, long long lde, int e_off, T* __restrict__ out) {
+  pdl_trigger();
+  pdl_wait();
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const long long t = i / N;
+    out[i] = from_f<T>(apply_small(act, z[i], tokens, vocab, e, lde, e_off, t, (int)(i - t * N)));
+  }
+}
+
+// xIELU in place: z > 0: softplus(p) z^2 + z / 2; else (1/2 + softplus(q)) (e^z - 1 - z) + z / 2; (p, q) = act
+template <typename T, int V>
+__global__ void __launch_bounds__(256) xielu_kernel(T* __restrict__ x, const T* __restrict__ act, long long total) {
+  pdl_trigger();
+  pdl_wait();
+  const float ap = softplus(to_f(act[0])), an = 0.5f + softplus(to_f(act[1]));
+  for (long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * V; i < total; i += (long long)gridDim.x * blockDim.x * V) {
+    float v[V];
+    load_v<V>(x + i, v);
+#pragma unroll
+    for (int q = 0; q < V; ++q) {
+      const float z = v[q], m = fminf(z, 0.f);
+      const float em = sizeof(T) == 2 ? quick_expm1(m) : expm1f(m);
+      v[q] = (z > 0.f ? ap * z * z : an * (em - z)) + 0.5f * z;
+    }
+    store_v<V>(x + i, v);
+  }
+}
+
+// Token shift of a ragged batch: mixes[m, t] = h[t] + (before - h[t]) mu[m], where before is the row of the sequence's
+// token before (its slot's `carry` at the start of a portion, zero at the start of the sequence). A thread keeps V
+// channels of all mu and walks ST tokens. The carry is only read: whoever runs after this kernel replaces it.
+constexpr int ST = 16;
+template <typename T, int V, int NM>
+__global__ void __launch_bounds__(128)
+token_shift_kernel(const T* __restrict__ h, const T* __restrict__ mu, const float* __restrict__ carry, Ragged rb, int D,
+                   int n_mix, T* __restrict__ mixes) {
+  pdl_trigger();
+  pdl_wait();
+  const int d = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+  if (d >= D) return;
+  const int t0 = blockIdx.y * ST, t1 = min(t0 + ST, rb.n);
+  float m[NM][V], prev[V];
+#pragma unroll
+  for (int k = 0; k < NM; ++k)
+    if (k < n_mix) load_v<V>(mu + (long long)k * D + d, m[k]);
+  if (t0 > 0) load_v<V>(h + (long long)(t0 - 1) * D + d, prev);
+  for (int t = t0; t < t1; ++t) {
+    const int e = rb.ent[t];
+    float u[V];
+    load_v<V>(h + (long long)t * D + d, u);
+    if (t == rb.cu[e]) {
+      if (rb.pos0[e] > 0) {
+        load_v<V>(carry + (long long)rb.slot[e] * D + d, prev);
+      } else {
+#pragma unroll
+        for (int i = 0; i < V; ++i) prev[i] = 0.f;
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < NM; ++k)
+      if (k < n_mix) {
+        float v[V];
+#pragma unroll
+        for (int i = 0; i < V; ++i) v[i] = u[i] + (prev[i] - u[i]) * m[k][i];
+        store_v<V>(mixes + ((long long)k * rb.n + t) * D + d, v);
+      }
+#pragma unroll
+    for (int i = 0; i < V; ++i) prev[i] = u[i];
   }
 }
 
@@ -265,11 +467,57 @@ few_outputs_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __r
 // dtype: 0 = bf16, 1 = float (activations and weights). x fp32 [n, S, D]; see StreamArgs.
 TB_API int tb_stream_step(int dtype, float* x, int n, int S, int D, float eps, const void* y, const void* y2, const void* wy,
                           const void* wy2, const void* mix, const void* out, const long long* tokens, const void* embed,
-                          int vocab, const void* in, const void* w, void* h, float* sum_out, cudaStream_t stream) {
+                          int vocab, const void* embed_w, int groups, const void* in, const void* w, void* h, float* sum_out,
+                          const void* mu, int n_mix, float* before, void* mixes, const int* slot, const int* pos0,
+                          cudaStream_t stream) {
   if (n <= 0) return 0;
-  if (S < 1 || S > MAX_STREAMS || D <= 0 || D > 12000 || (y && tokens) || (y2 && !y)) return -2;
-  StreamArgs a{x, D, eps, y, y2, wy, wy2, mix, out, tokens, embed, vocab, in, w, h, sum_out};
+  if (S < 1 || S > MAX_STREAMS || D <= 0 || D > 11000 || (y && tokens) || (y2 && !y)) return -2;
+  if (groups < 1 || groups > 256 || D % groups || (mu && (!w || !before || !mixes))) return -2;
+  StreamArgs a{x, D, eps, y, y2, wy, wy2, mix, out, tokens, embed, vocab, embed_w, groups, in, w, h, sum_out,
+               mu, n_mix, before, mixes, slot, pos0};
   return dtype == 0 ? dispatch_stream_step<__nv_bfloat16>(a, S, n, stream) : dispatch_stream_step<float>(a, S, n, stream);
+}
+
+// h T [n, D] contiguous, mu T [n_mix, D] with at most 8 mixes, carry fp32 [slots, D] -> mixes T [n_mix, n, D]
+TB_API int tb_token_shift(int dtype, const void* h, const void* mu, int n_mix, const float* carry, const int* cu, const int* slot,
+                          const int* pos0, const int* ent, int E, int n, int D, void* mixes, cudaStream_t stream) {
+  if (n <= 0 || E <= 0) return 0;
+  if (n_mix < 1 || n_mix > 8 || (n + ST - 1) / ST > 65535) return -2;
+  Ragged rb{cu, slot, pos0, ent, E, n};
+  typedef __nv_bfloat16 bf;
+#define TS(T, V, NM)                                                                                                        \
+  launch_pdl(token_shift_kernel<T, V, NM>, dim3((D / V + 127) / 128, (n + ST - 1) / ST), dim3(128), 0, stream, (const T*)h,  \
+             (const T*)mu, carry, rb, D, n_mix, (T*)mixes)
+  cudaError_t err = dtype != 0 ? TS(float, 1, 8) : D % 4 ? TS(bf, 1, 8) : n_mix <= 5 ? TS(bf, 4, 5) : TS(bf, 4, 8);
+#undef TS
+  return err == cudaSuccess ? 0 : -5;
+}
+
+// act T [2]; x T [total] in place
+TB_API int tb_xielu(int dtype, void* x, const void* act, long long total, cudaStream_t stream) {
+  if (total <= 0) return 0;
+  const int V = dtype == 0 && total % 8 == 0 ? 8 : 1;
+  const long long want = (total / V + 255) / 256;
+  const dim3 grid((unsigned)(want < 148 * 16 ? want : 148 * 16));
+  typedef __nv_bfloat16 bf;
+  cudaError_t err = dtype != 0 ? launch_pdl(xielu_kernel<float, 1>, grid, dim3(256), 0, stream, (float*)x, (const float*)act, total)
+                    : V == 8   ? launch_pdl(xielu_kernel<bf, 8>, grid, dim3(256), 0, stream, (bf*)x, (const bf*)act, total)
+                               : launch_pdl(xielu_kernel<bf, 1>, grid, dim3(256), 0, stream, (bf*)x, (const bf*)act, total);
+  return err == cudaSuccess ? 0 : -5;
+}
+
+// z fp32 [n, N] -> out T [n, N]; act as in apply_small, e T [vocab, lde]
+TB_API int tb_small_act(int dtype, const float* z, int n, int N, int act, const long long* tokens, int vocab, const void* e,
+                        long long lde, int e_off, void* out, cudaStream_t stream) {
+  const long long total = (long long)n * N, want = (total + 255) / 256;
+  if (total <= 0) return 0;
+  const dim3 grid((unsigned)(want < 148 * 16 ? want : 148 * 16));
+  cudaError_t err = dtype == 0
+      ? launch_pdl(small_act_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, z, N, total, act, tokens, vocab,
+                   (const __nv_bfloat16*)e, lde, e_off, (__nv_bfloat16*)out)
+      : launch_pdl(small_act_kernel<float>, grid, dim3(256), 0, stream, z, N, total, act, tokens, vocab, (const float*)e, lde,
+                   e_off, (float*)out);
+  return err == cudaSuccess ? 0 : -5;
 }
 
 TB_API int tb_silu_mul(int dtype, const void* gu, void* h, long long rows, int F, cudaStream_t stream) {
@@ -296,11 +544,16 @@ TB_API int tb_gate_outputs(int dtype, const void* attn, const float* o, const vo
   return err == cudaSuccess ? 0 : -5;
 }
 
-// x bf16 [n, K], w bf16 [N, K] (contiguous, K a multiple of 8) -> out fp32 [n, N]
-TB_API int tb_few_outputs(const void* x, const void* w, int n, int K, int N, float* out, cudaStream_t stream) {
+// x bf16 [n, K], w bf16 [N, K] (contiguous, K a multiple of 8) -> out [n, N], fp32 or (out_bf16) bf16; act, e as in apply_small
+TB_API int tb_few_outputs(const void* x, const void* w, int n, int K, int N, int act, const long long* tokens, int vocab,
+                          const void* e, long long lde, int e_off, void* out, int out_bf16, cudaStream_t stream) {
   if (n <= 0 || N <= 0) return 0;
   if (K % 8) return -2;
   const int threads = N >= 16 ? 512 : N >= 8 ? 256 : 128;
-  return launch_pdl(few_outputs_kernel, dim3(n), dim3(threads), 0, stream, (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, K, N,
-                    out) == cudaSuccess ? 0 : -5;
+  typedef __nv_bfloat16 bf;
+#define FO(TO)                                                                                                              \
+  launch_pdl(few_outputs_kernel<TO>, dim3(n), dim3(threads), 0, stream, (const bf*)x, (const bf*)w, K, N, act, tokens, vocab, \
+             (const bf*)e, lde, e_off, (TO*)out)
+  return (out_bf16 ? FO(bf) : FO(float)) == cudaSuccess ? 0 : -5;
+#undef FO
 }

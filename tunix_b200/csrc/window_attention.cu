@@ -1,11 +1,15 @@
-// Sliding-window attention over a paged cache with kept first tokens and a learned distance bias, for ragged batches.
+// Attention over a paged cache for the ragged batches of layer-stack models: sliding windows with kept first tokens or
+// chunks, learned distance bias, score cap, rotary positions.
 //
 //   qk_norm_write : after the fused projection of a step: RMS norm of q and of k over the WHOLE projection (all heads at
 //                   once), q to a compact buffer, k and v rows to their pages (value rows may be wider or narrower than
 //                   key rows).
+//   rope_norm_write : the same place for rotary attention: the first `rd` dimensions of every query and key head turn by
+//                   the angles of the token's position (element i together with i + rd / 2), then each head is divided by
+//                   its root mean square. A layer that reads another layer's cache has queries only.
 //   window_attn   : any head sizes, bf16 or float: one warp per (token, query head), lanes over keys for the scores and
 //                   over value columns for the output, online softmax in fp32. Position i sees j <= i with
-//                   i - j < window or j < keep. Models whose heads fit the tensor-core kernels (attention_fwd.cu,
+//                   (i - j < window and j in i's chunk) or j < keep. Models whose heads fit the tensor-core kernels (attention_fwd.cu,
 //                   decode.cu) use those instead.
 //
 // This file is compiled without fast-math: the same kernels serve the 32-bit mode.
@@ -75,13 +79,69 @@ qk_norm_write_kernel(const T* __restrict__ proj, long long ldp, int q_off, int k
   }
 }
 
+// One warp per (token, head) over the query heads, then key heads, then value heads of a row. cos / sin [positions, rd / 2].
+template <typename T>
+__global__ void __launch_bounds__(256)
+rope_norm_write_kernel(const T* __restrict__ proj, long long ldp, int q_off, int k_off, int v_off, const float* __restrict__ cos_t,
+                       const float* __restrict__ sin_t, int rd, float eps, Ragged rb, Paged pg, int H, int G, int dq, int dv,
+                       T* __restrict__ q, T* __restrict__ kp, T* __restrict__ vp) {
+  pdl_trigger();
+  pdl_wait();
+  const int heads = H + 2 * G;
+  const long long wid = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (wid >= (long long)rb.n * heads) return;
+  const int lane = threadIdx.x & 31;
+  const int t = (int)(wid / heads), hh = (int)(wid - (long long)t * heads);
+  const int e = rb.ent[t], p0 = rb.pos0[e];
+  const T* row = proj + (long long)t * ldp;
+  if (p0 < 0) {
+    if (hh < H)
+      for (int c = lane; c < dq; c += 32) q[((long long)t * H + hh) * dq + c] = from_f<T>(0.f);
+    return;
+  }
+  const int p = p0 + t - rb.cu[e];
+  long long pr = 0;
+  if (hh >= H) pr = page_row(pg, pg.table + (long long)rb.slot[e] * pg.max_pages, p);
+  if (hh >= H + G) {
+    const int g = hh - H - G;
+    for (int c = lane; c < dv; c += 32) vp[(pr * G + g) * dv + c] = row[v_off + g * dv + c];
+    return;
+  }
+  const T* src = row + (hh < H ? q_off + hh * dq : k_off + (hh - H) * dq);
+  T* dst = hh < H ? q + ((long long)t * H + hh) * dq : kp + (pr * G + hh - H) * dq;
+  const int half = rd >> 1;
+  const float *ct = cos_t + (long long)p * half, *st = sin_t + (long long)p * half;
+  // the turned head stays in registers up to 256 dimensions (lane + 32 j), wider ones are turned twice
+  auto turned = [&](int c) {
+    const float x = to_f(src[c]);
+    if (c < half) return x * ct[c] - to_f(src[c + half]) * st[c];
+    if (c < 2 * half) return x * ct[c - half] + to_f(src[c - half]) * st[c - half];
+    return x;
+  };
+  float v[8], ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < 8; ++j) {
+    const int c = lane + 32 * j;
+    v[j] = c < dq ? turned(c) : 0.f;
+    ss += v[j] * v[j];
+  }
+  for (int c = lane + 256; c < dq; c += 32) { const float x = turned(c); ss += x * x; }
+  const float r = 1.f / sqrtf(warp_sum(ss) / (float)dq + eps);
+#pragma unroll
+  for (int j = 0; j < 8; ++j) {
+    const int c = lane + 32 * j;
+    if (c < dq) dst[c] = from_f<T>(v[j] * r);
+  }
+  for (int c = lane + 256; c < dq; c += 32) dst[c] = from_f<T>(turned(c) * r);
+}
+
 constexpr int VREG = 16;        // value columns per lane: value heads up to 512 wide
 
 template <typename T>
 __global__ void __launch_bounds__(128)
 window_attn_kernel(const T* __restrict__ q, const T* __restrict__ kp, const T* __restrict__ vp, Ragged rb, Paged pg, int H,
-                   int G, int dq, int dv, float scale, const float* __restrict__ bias, int far, int window, int keep,
-                   T* __restrict__ out) {
+                   int G, int dq, int dv, float scale, float cap, const float* __restrict__ bias, int far, int window, int chunk,
+                   int keep, T* __restrict__ out) {
   extern __shared__ float qs_all[];               // [4][dq]
   pdl_trigger();
   pdl_wait();
@@ -99,7 +159,7 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ kp, const T* _
   for (int d = lane; d < dq; d += 32) qs[d] = to_f(q[((long long)t * H + h) * dq + d]) * scale;
   __syncwarp();
   const int i = p0 + t - rb.cu[e];
-  const int lo = window > 0 ? max(0, i - window + 1) : 0;
+  const int lo = first_visible(i, window, chunk);
   const int kept = min(keep, lo);                 // keys 0 .. kept-1 lie before the window
   const int cnt = kept + i - lo + 1;
   const int* pt = pg.table + (long long)rb.slot[e] * pg.max_pages;
@@ -117,7 +177,8 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ kp, const T* _
       const T* k = kp + (row * G + g) * dq;
       float dot = 0.f;
       for (int d = 0; d < dq; ++d) dot += qs[d] * to_f(k[d]);
-      s = dot + bias[(long long)h * (far + 1) + min(i - j, far)];
+      s = cap > 0.f ? cap * tanhf(dot / cap) : dot;
+      if (bias) s += bias[(long long)h * (far + 1) + min(i - j, far)];
     }
     const float mn = fmaxf(m, warp_max(s));
     const float p = expf(s - mn), c = expf(m - mn);
@@ -167,11 +228,31 @@ TB_API int tb_qk_norm_write(int dtype, const void* proj, long long ldp, int q_of
   return err == cudaSuccess ? 0 : -5;
 }
 
-// bias fp32 [H, far + 1]: what is added to the score of a key at distance min(i - j, far). window <= 0: no window.
+// q | k | v: columns of proj [n, ldp]; H query heads, G key / value heads (0: queries only), rd rotated dimensions with tables
+// cos / sin fp32 [positions, rd / 2]; q [n, H * dq]; pools [pages, page_size, G * dq] and [.., G * dv].
+TB_API int tb_rope_norm_write(int dtype, const void* proj, long long ldp, int q_off, int k_off, int v_off, const float* cos_t,
+                              const float* sin_t, int rd, float eps, const int* cu, const int* slot, const int* pos0,
+                              const int* ent, int E, int n, const int* table, int max_pages, int page_size, int H, int G, int dq,
+                              int dv, void* q, void* kp, void* vp, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (rd < 0 || rd % 2 || rd > dq) return -2;
+  RAGGED;
+  PAGED;
+  const long long warps = (long long)n * (H + 2 * G);
+  const dim3 grid((unsigned)((warps + 7) / 8));
+#define RUN(T)                                                                                                              \
+  launch_pdl(rope_norm_write_kernel<T>, grid, dim3(256), 0, stream, (const T*)proj, ldp, q_off, k_off, v_off, cos_t, sin_t,  \
+             rd, eps, rb, pg, H, G, dq, dv, (T*)q, (T*)kp, (T*)vp)
+  return (dtype == 0 ? RUN(__nv_bfloat16) : RUN(float)) == cudaSuccess ? 0 : -5;
+#undef RUN
+}
+
+// bias fp32 [H, far + 1] or null: what is added to the score of a key at distance min(i - j, far). window, chunk <= 0: none;
+// cap > 0: scores become cap * tanh(score / cap).
 TB_API int tb_window_attn(int dtype, const void* q, const void* kp, const void* vp, const int* cu, const int* slot,
                           const int* pos0, const int* ent, int E, int n, const int* table, int max_pages, int page_size, int H,
-                          int G, int dq, int dv, float scale, const float* bias, int far, int window, int keep, void* out,
-                          cudaStream_t stream) {
+                          int G, int dq, int dv, float scale, float cap, const float* bias, int far, int window, int chunk,
+                          int keep, void* out, cudaStream_t stream) {
   if (n <= 0) return 0;
   if (G <= 0 || H % G || dv > VREG * 32 || dq > 3000) return -2;
   RAGGED;
@@ -180,7 +261,7 @@ TB_API int tb_window_attn(int dtype, const void* q, const void* kp, const void* 
   const dim3 grid((unsigned)((warps + 3) / 4));
 #define RUN(T)                                                                                                              \
   return launch_pdl(window_attn_kernel<T>, grid, dim3(128), (size_t)4 * dq * 4, stream, (const T*)q, (const T*)kp,           \
-                    (const T*)vp, rb, pg, H, G, dq, dv, scale, bias, far, window, keep, (T*)out) == cudaSuccess ? 0 : -5
+                    (const T*)vp, rb, pg, H, G, dq, dv, scale, cap, bias, far, window, chunk, keep, (T*)out) == cudaSuccess ? 0 : -5
   if (dtype == 0) RUN(__nv_bfloat16);
   RUN(float);
 #undef RUN

@@ -9,15 +9,21 @@ sizes and constants in a spec, its parameters in a module and its per-sequence c
   MatrixMemory            mLSTM: matrix memory with exponential input gate, capped gate pre-activations, per-head norm
                           and sigmoid output gate
   ParallelMixer           two mixers on the same input, half the sum of their normed outputs
+  TokenShiftMemory        RWKV time mixing: every projection reads its own mix of a token and the one before it, matrix
+                          memory with a data-dependent decay per key channel and a bonus for the current token, per-head
+                          norm and silu output gate
+  ForgetGateMemory        HGRN2: matrix memory whose forget gate (bounded from below) also decides what is written
+  RotaryAttention         grouped-query attention with rotary positions, RMS-normed query and key heads, score cap, chunks
+                          of positions; may read the keys and values of another layer
 
-A spec's `kv_rows()` names the paged cache rows a pass through the layer needs (key columns, value columns), or None;
-`state_shapes()` the fp32 state it keeps per sequence slot. The kernels are launched by `models/stack_exec.py`.
+A spec's `kv_rows()` names the paged cache rows a pass through the layer needs (key columns, value columns), or None (also
+for attention that reads another layer's, `kv_from`); `state_shapes()` the fp32 state it keeps per sequence slot. The kernels are launched by `models/stack_exec.py`.
 """
 from __future__ import annotations
 
 import math
 from dataclasses import dataclass
-from typing import Optional
+from typing import ClassVar, Optional
 
 import torch
 import torch.nn as nn
@@ -52,6 +58,8 @@ class WindowAttentionSpec:
     window: int                  # 0 = unlimited
     keep_first: int = 0          # leading tokens of the sequence that stay visible
     buckets: int = 32            # rows of the bias table
+    chunk: ClassVar[int] = 0
+    softcap: ClassVar[float] = 0.0
 
     def kv_rows(self):
         return (self.kv_heads * self.dim, self.kv_heads * self.vdim)
@@ -85,6 +93,55 @@ class ParallelSpec:
 
     def state_shapes(self) -> dict:
         return self.right.state_shapes()
+
+
+@dataclass(frozen=True)
+class RotaryAttentionSpec:
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot_dims: int                # leading dimensions of a head that turn
+    rot_base: float
+    softcap: float = 0.0         # scores become softcap * tanh(score / softcap); 0 = as they are
+    chunk: int = 0               # a query sees the keys of its own chunk of that many positions; 0 = all before it
+    kv_from: Optional[int] = None    # index of the layer whose keys and values this one reads
+    window: ClassVar[int] = 0
+    keep_first: ClassVar[int] = 0
+
+    def kv_rows(self):
+        return None if self.kv_from is not None else (self.kv_heads * self.dim, self.kv_heads * self.vdim)
+
+    def state_shapes(self) -> dict:
+        return {}
+
+
+@dataclass(frozen=True)
+class TokenShiftMemorySpec:
+    heads: int
+    dim: int                     # key and value size of a head
+    decay_rank: int              # width of the bottleneck that makes the decays
+    width: int                   # the mixer's input: the last one of a sequence is part of the state
+
+    def kv_rows(self):
+        return None
+
+    def state_shapes(self) -> dict:
+        return {"S": (self.heads, self.dim, self.dim), "last": (self.width,)}
+
+
+@dataclass(frozen=True)
+class ForgetGateMemorySpec:
+    heads: int
+    dim: int
+    vdim: int
+
+    def kv_rows(self):
+        return None
+
+    def state_shapes(self) -> dict:
+        return {"S": (self.heads, self.dim, self.vdim)}
 
 
 # ------------------------------------------------------------------------------------------------- bias table
@@ -196,7 +253,76 @@ class ParallelMixer(nn.Module):
                 [rt.i_proj, rt.f_proj]]
 
 
-MIXERS = {RGLRUSpec: RGLRUMixer, ParallelSpec: ParallelMixer}
+class RotaryAttention(nn.Module):
+    def __init__(self, spec: RotaryAttentionSpec, width: int, eps: float, dtype, device=None):
+        super().__init__()
+        if spec.heads % spec.kv_heads:
+            raise ValueError(f"{spec.heads} query heads over {spec.kv_heads} key / value heads")
+        if spec.rot_dims % 2 or spec.rot_dims > spec.dim:
+            raise ValueError(f"{spec.rot_dims} rotated dimensions of {spec.dim}")
+        self.spec, self.eps = spec, eps
+        self.q_proj = Linear(width, spec.heads * spec.dim, True, dtype, device)
+        own = spec.kv_from is None
+        self.k_proj = Linear(width, spec.kv_heads * spec.dim, True, dtype, device) if own else None
+        self.v_proj = Linear(width, spec.kv_heads * spec.vdim, True, dtype, device) if own else None
+        self.o_proj = Linear(spec.heads * spec.vdim, width, True, dtype, device)
+
+    def init_special(self) -> None:
+        pass
+
+    def fused_groups(self) -> list:
+        return [[self.q_proj] + ([self.k_proj, self.v_proj] if self.k_proj is not None else [])]
+
+
+class TokenShiftMemory(nn.Module):
+    MIXES = ("r", "k", "v", "g", "w")
+
+    def __init__(self, spec: TokenShiftMemorySpec, width: int, eps: float, dtype, device=None):
+        super().__init__()
+        self.spec, self.eps = spec, eps
+        C = spec.heads * spec.dim
+        for n in self.MIXES:
+            setattr(self, "mu_" + n, _param(width, dtype=dtype, device=device, fill=0.5))
+        for n in ("r", "k", "v", "g"):
+            setattr(self, n + "_proj", Linear(width, C, False, dtype, device))
+        self.w1_proj = Linear(width, spec.decay_rank, False, dtype, device)
+        self.w2_proj = Linear(spec.decay_rank, C, False, dtype, device)
+        self.w0 = _param(C, dtype=dtype, device=device)
+        self.u = _param(spec.heads, spec.dim, dtype=dtype, device=device)
+        self.norm = RMSNorm(C, eps, False, dtype, device)
+        self.o_proj = Linear(C, width, False, dtype, device)
+
+    def mu(self) -> torch.Tensor:
+        return torch.stack([getattr(self, "mu_" + n).data for n in self.MIXES])
+
+    def init_special(self) -> None:
+        n = self.w0.numel()
+        self.w0.copy_(torch.linspace(-6.0, 0.0, n, device=self.w0.device))      # slow to fast decays over the channels
+
+    def fused_groups(self) -> list:
+        return []
+
+
+class ForgetGateMemory(nn.Module):
+    def __init__(self, spec: ForgetGateMemorySpec, width: int, eps: float, dtype, device=None):
+        super().__init__()
+        self.spec, self.eps = spec, eps
+        self.q_proj = Linear(width, spec.heads * spec.dim, False, dtype, device)
+        self.v_proj = Linear(width, spec.heads * spec.vdim, False, dtype, device)
+        self.f_proj = Linear(width, spec.heads * spec.dim, True, dtype, device)
+        self.lower = _param(spec.heads * spec.dim, dtype=dtype, device=device, fill=0.5)
+        self.norm = RMSNorm(spec.vdim, eps, False, dtype, device)
+        self.o_proj = Linear(spec.heads * spec.vdim, width, False, dtype, device)
+
+    def init_special(self) -> None:
+        self.f_proj.bias.fill_(2.0)
+
+    def fused_groups(self) -> list:
+        return [[self.q_proj, self.v_proj], [self.f_proj]]
+
+
+MIXERS = {RGLRUSpec: RGLRUMixer, ParallelSpec: ParallelMixer, RotaryAttentionSpec: RotaryAttention,
+          TokenShiftMemorySpec: TokenShiftMemory, ForgetGateMemorySpec: ForgetGateMemory}
 
 
 def create_mixer(spec, width: int, eps: float, dtype, device: Optional[torch.device] = None) -> nn.Module:

@@ -74,11 +74,29 @@ _KEY_MAPS = {
         (r"l(\d+)\.mix\.(conv|ra|ri)", r"layers.\1.mixer.\2_weight"),
         (r"l(\d+)\.mix\.lam", r"layers.\1.mixer.lam"),
     ],
+    "tovalix": [
+        (r"embed", "embed_tokens"),
+        (r"embed\.norm", "embed_norm.weight"),
+        (r"side\.embed", "side_embed"),
+        (r"head", "lm_head"),
+        (r"final\.norm", "norm.weight"),
+        (r"l(\d+)\.norm1", r"layers.\1.input_layernorm.weight"),
+        (r"l(\d+)\.norm2", r"layers.\1.post_attention_layernorm.weight"),
+        (r"l(\d+)\.mlp\.(up|down)", r"layers.\1.mlp.\2_proj.weight"),
+        (r"l(\d+)\.mlp\.act", r"layers.\1.mlp.act"),
+        (r"l(\d+)\.side\.gate", r"layers.\1.side.gate_proj.weight"),
+        (r"l(\d+)\.side\.(proj|norm)", r"layers.\1.side.\2.weight"),
+        (r"l(\d+)\.mix\.mu\.(r|k|v|g|w)", r"layers.\1.mixer.mu_\2"),
+        (r"l(\d+)\.mix\.(w0|u|lower)", r"layers.\1.mixer.\2"),
+        (r"l(\d+)\.mix\.norm", r"layers.\1.mixer.norm.weight"),
+        (r"l(\d+)\.mix\.(q|k|v|o|f)\.b", r"layers.\1.mixer.\2_proj.bias"),
+        (r"l(\d+)\.mix\.(r|k|v|g|q|f|o|w1|w2)", r"layers.\1.mixer.\2_proj.weight"),
+    ],
 }
 
 
 def key_map_for(cfg) -> list:
-    if cfg.family in ("gemma4", "roluzen"):
+    if cfg.family in ("gemma4", "roluzen", "tovalix"):
         return _KEY_MAPS[cfg.family]
     return _KEY_MAPS["gemma_post_norms" if cfg.post_norms else "default"]
 
@@ -95,8 +113,8 @@ def map_key(hf_key: str, table: list) -> Optional[str]:
 
 def inverse_map_key(our_key: str, cfg) -> str:
     """Our parameter name -> HF key (used by the saver)."""
-    if cfg.family == "roluzen":
-        return _inverse_stack_key(our_key)
+    if cfg.family in _STACK_INVERSE:
+        return _inverse_stack_key(our_key, cfg.family)
     if our_key == "embed_tokens":
         return "model.embed_tokens.weight"
     if our_key == "lm_head":
@@ -112,11 +130,13 @@ def inverse_map_key(our_key: str, cfg) -> str:
     return k
 
 
-# parameter name -> checkpoint name of layer-stack models, the inverse of _KEY_MAPS["roluzen"]
-_STACK_INVERSE = [
+# parameter name -> checkpoint name of layer-stack models, the inverse of their tables in _KEY_MAPS
+_STACK_ENDS = [
     (r"embed_tokens", "embed"), (r"lm_head", "head"), (r"norm\.weight", "final.norm"),
     (r"layers\.(\d+)\.input_layernorm\.weight", r"l\1.norm1"),
     (r"layers\.(\d+)\.post_attention_layernorm\.weight", r"l\1.norm2"),
+]
+_STACK_INVERSE = {"roluzen": _STACK_ENDS + [
     (r"layers\.(\d+)\.(hc\d)\.weight_(in|out)", r"l\1.\2.\3"),
     (r"layers\.(\d+)\.(hc\d)\.mix", r"l\1.\2.mix"),
     (r"layers\.(\d+)\.mlp\.(gate|up|down)_proj\.weight", r"l\1.mlp.\2"),
@@ -131,11 +151,22 @@ _STACK_INVERSE = [
     (r"layers\.(\d+)\.mixer\.(conv|ra|ri)_bias", r"l\1.mix.\2.b"),
     (r"layers\.(\d+)\.mixer\.(conv|ra|ri)_weight", r"l\1.mix.\2"),
     (r"layers\.(\d+)\.mixer\.lam", r"l\1.mix.lam"),
-]
+], "tovalix": _STACK_ENDS + [
+    (r"embed_norm\.weight", "embed.norm"), (r"side_embed", "side.embed"),
+    (r"layers\.(\d+)\.mlp\.(up|down)_proj\.weight", r"l\1.mlp.\2"),
+    (r"layers\.(\d+)\.mlp\.act", r"l\1.mlp.act"),
+    (r"layers\.(\d+)\.side\.gate_proj\.weight", r"l\1.side.gate"),
+    (r"layers\.(\d+)\.side\.(proj|norm)\.weight", r"l\1.side.\2"),
+    (r"layers\.(\d+)\.mixer\.mu_(\w)", r"l\1.mix.mu.\2"),
+    (r"layers\.(\d+)\.mixer\.(w0|u|lower)", r"l\1.mix.\2"),
+    (r"layers\.(\d+)\.mixer\.norm\.weight", r"l\1.mix.norm"),
+    (r"layers\.(\d+)\.mixer\.(\w+)_proj\.bias", r"l\1.mix.\2.b"),
+    (r"layers\.(\d+)\.mixer\.(\w+)_proj\.weight", r"l\1.mix.\2"),
+]}
 
 
-def _inverse_stack_key(our_key: str) -> str:
-    for pat, repl in _STACK_INVERSE:
+def _inverse_stack_key(our_key: str, family: str) -> str:
+    for pat, repl in _STACK_INVERSE[family]:
         m = re.fullmatch(pat, our_key)
         if m:
             return m.expand(repl)

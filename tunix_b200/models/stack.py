@@ -1,15 +1,18 @@
 """Layer-stack models: decoders whose layers are listed one by one, each with its own mixer (`models/mixers.py`) and
-feed-forward, a range of layers that may run several times with the same weights, and parallel residual streams joined by
-hyper-connections. Roluzen is the first design of this kind.
+feed-forward, a range of layers that may run several times with the same weights, parallel residual streams joined by
+hyper-connections, norms over groups of a row, and inputs per token and layer. Designs of this kind: Roluzen, Tovalix.
 
 The residual streams are fp32. A sublayer q of a layer reads u = sum_s in[s] x_s, computes y = f(norm(u)) and leaves
-x_t = sum_s mix[s, t] x_s + out[t] y on every stream; the model's output is the norm of the streams' sum.
+x_t = sum_s mix[s, t] x_s + out[t] y on every stream; the model's output is the norm of the streams' sum. A layer's token
+input adds norm(proj(gelu(gate(x)) * e)) after the feed-forward, e being the layer's part of the token's row in a second
+embedding table.
 
 The model holds parameters; `models/stack_exec.py` runs it on ragged batches over the paged cache and the slot states of
 `generate/engine.py`. `forward` scores whole sequences through that same path on a temporary cache (no gradients).
 """
 from __future__ import annotations
 
+import dataclasses
 import json
 import os
 from dataclasses import dataclass, field
@@ -20,14 +23,16 @@ import torch.nn as nn
 
 from ..ops import functional as F
 from .config import ModelConfig
-from .mixers import MatrixMemorySpec, ParallelSpec, RGLRUSpec, WindowAttentionSpec, create_mixer
-from .transformer import MLP, RMSNorm
+from .mixers import (ForgetGateMemorySpec, MatrixMemorySpec, ParallelSpec, RGLRUSpec, RotaryAttentionSpec, TokenShiftMemorySpec,
+                     WindowAttentionSpec, create_mixer)
+from .transformer import MLP, Linear, RMSNorm
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     mixer: object                       # one of the specs of models/mixers.py
-    ff: Optional[int]                   # width of the gated feed-forward; None = the layer has none
+    ff: Optional[int]                   # width of the feed-forward; None = the layer has none
+    ff_kind: str = "glu"                # "glu": silu-gated; "xielu": up, xIELU with two learned numbers, down
 
 
 @dataclass
@@ -35,6 +40,9 @@ class StackConfig(ModelConfig):
     layer_specs: tuple = field(default_factory=tuple)
     loop: Optional[tuple] = None        # (start, stop, times): these layers run `times` times in a row
     streams: int = 0                    # residual streams with hyper-connections; 0 = one plain residual
+    norm_groups: int = 1                # equal parts of a row that the norms before sublayers and at the ends are taken over
+    embed_norm: bool = False            # the embedding rows are normed
+    token_side: int = 0                 # width of the per-layer token inputs; 0 = none
 
     def __post_init__(self):
         if not self.layer_specs:
@@ -42,13 +50,26 @@ class StackConfig(ModelConfig):
         self.num_layers = len(self.layer_specs)
         ffs = [s.ff for s in self.layer_specs if s.ff is not None]
         self.hidden_dim = max(ffs) if ffs else 0
-        att = [s.mixer.left for s in self.layer_specs if isinstance(s.mixer, ParallelSpec)]
+        att = [getattr(s.mixer, "left", s.mixer) for s in self.layer_specs]
+        att = [a for a in att if isinstance(a, (WindowAttentionSpec, RotaryAttentionSpec))]
         if att:                         # what generic callers size caches and reports by: the first attention layer
             self.num_heads, self.num_kv_heads, self.head_dim = att[0].heads, att[0].kv_heads, att[0].dim
         if self.loop is not None:
             a, b, times = self.loop
             if not (0 <= a <= b <= self.num_layers and times >= 0):
                 raise ValueError(f"loop {self.loop} does not fit {self.num_layers} layers")
+        if self.embed_dim % self.norm_groups:
+            raise ValueError(f"a width of {self.embed_dim} does not split into {self.norm_groups} norm groups")
+        for i, s in enumerate(self.layer_specs):
+            j = getattr(s.mixer, "kv_from", None)
+            if j is None:
+                continue
+            src = self.layer_specs[j].mixer if 0 <= j < i else None
+            if not isinstance(src, RotaryAttentionSpec) or src.kv_from is not None:
+                raise ValueError(f"layer {i} reads keys and values of layer {j}, which keeps none before it")
+            if (src.kv_heads, src.dim, src.vdim) != (s.mixer.kv_heads, s.mixer.dim, s.mixer.vdim):
+                raise ValueError(f"layers {i} and {j} share keys and values of unequal sizes")
+        self.kv_sources()
 
     def runs(self) -> list:
         """Layer index of every pass, in order. Each pass has its own cache and state."""
@@ -61,6 +82,17 @@ class StackConfig(ModelConfig):
     # ---- what the engine's cache manager allocates, per pass
     def kv_rows(self) -> list:
         return [self.layer_specs[i].mixer.kv_rows() for i in self.runs()]
+
+    def kv_sources(self) -> list:
+        """Per pass, the pass whose cache its attention reads: its own, or the last pass of the layer it shares with."""
+        last, out = {}, []
+        for r, i in enumerate(self.runs()):
+            j = getattr(self.layer_specs[i].mixer, "kv_from", None)
+            if j is not None and j not in last:
+                raise ValueError(f"layer {i} reads keys and values of layer {j}, which has not run before it")
+            out.append(r if j is None else last[j])
+            last[i] = r
+        return out
 
     def state_shapes(self) -> list:
         return [self.layer_specs[i].mixer.state_shapes() for i in self.runs()]
@@ -94,9 +126,38 @@ class StackConfig(ModelConfig):
     def roluzen_8b(cls) -> "StackConfig":
         return cls._roluzen(4096, 12288, 32, 8, 128, 8, 256, 512, 4096, 16, 24, (0, 3, 2))
 
+    @classmethod
+    def _tovalix(cls, D, ff, heads, kv, dim, mh, mdim, fh, fdim, fvdim, n, chunk, side, groups=1, rank=64, vocab=151936, rot=None):
+        att = RotaryAttentionSpec(heads=heads, kv_heads=kv, dim=dim, vdim=dim, scale=dim ** -0.5, rot_dims=rot or dim,
+                                  rot_base=500000.0, softcap=30.0, chunk=chunk)
+        specs, source = [], None
+        for i in range(n):
+            if i % 3 == 0:
+                mixer = TokenShiftMemorySpec(mh, mdim, rank, D)
+            elif i % 3 == 1:
+                mixer = ForgetGateMemorySpec(fh, fdim, fvdim)
+            else:                                 # every other attention layer reads the cache of the one before it
+                mixer = att if source is None else dataclasses.replace(att, kv_from=source)
+                source = i if source is None else None
+            specs.append(LayerSpec(mixer, ff, "xielu"))
+        return cls(family="tovalix", vocab_size=vocab, embed_dim=D, layer_specs=tuple(specs), norm_groups=groups, embed_norm=True,
+                   token_side=side)
+
+    @classmethod
+    def tovalix_tiny(cls) -> "StackConfig":
+        return cls._tovalix(96, 160, 4, 2, 32, 3, 32, 2, 40, 24, 6, 24, 8, groups=3, rank=8, vocab=384, rot=16)
+
+    @classmethod
+    def tovalix_2b(cls) -> "StackConfig":
+        return cls._tovalix(2048, 8192, 16, 8, 128, 32, 64, 16, 128, 128, 24, 1024, 64)
+
+    @classmethod
+    def tovalix_8b(cls) -> "StackConfig":
+        return cls._tovalix(4096, 16384, 32, 8, 128, 64, 64, 32, 128, 128, 30, 1024, 128)
+
 
 # ------------------------------------------------------------------------------------------ config.json reader
-def _parallel_spec(m: dict, shapes, prefix: str) -> ParallelSpec:
+def _parallel_spec(m: dict, shapes, prefix: str, width: int) -> ParallelSpec:
     lf, rt = m["left"], m["right"]
     mask = lf.get("mask") or {}
     rel = (shapes or {}).get(prefix + "left.rel")
@@ -107,12 +168,40 @@ def _parallel_spec(m: dict, shapes, prefix: str) -> ParallelSpec:
                                                gate_cap=float(rt["gate_cap"])))
 
 
-def _rglru_spec(m: dict, shapes, prefix: str) -> RGLRUSpec:
+def _rglru_spec(m: dict, shapes, prefix: str, width: int) -> RGLRUSpec:
     return RGLRUSpec(width=int(m["width"]), blocks=int(m["blocks"]), conv=int(m["conv"]))
 
 
-MIXER_READERS = {"rglru": _rglru_spec, "parallel": _parallel_spec}
-ARCHITECTURES = {"Roluzen": "roluzen"}
+def _rotary_spec(m: dict, shapes, prefix: str, width: int) -> RotaryAttentionSpec:
+    mask, rot = m.get("mask") or {}, m.get("rot") or {}
+    return RotaryAttentionSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                               scale=float(m["scale"]), rot_dims=int(rot.get("dims") or 0), rot_base=float(rot.get("base") or 1.0),
+                               softcap=float(m.get("softcap") or 0.0), chunk=int(mask.get("size") or 0),
+                               kv_from=None if m.get("kv_from") is None else int(m["kv_from"]))
+
+
+def _wkv_spec(m: dict, shapes, prefix: str, width: int) -> TokenShiftMemorySpec:
+    w1 = (shapes or {}).get(prefix + "w1")
+    return TokenShiftMemorySpec(heads=int(m["heads"]), dim=int(m["dim"]), decay_rank=int(w1[0]) if w1 else 64, width=width)
+
+
+def _hgrn2_spec(m: dict, shapes, prefix: str, width: int) -> ForgetGateMemorySpec:
+    return ForgetGateMemorySpec(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]))
+
+
+@dataclass(frozen=True)
+class Design:
+    family: str
+    mixers: dict                        # layer type in config.json -> reader of its mixer
+    ff_kind: str                        # what a "dense" feed-forward is
+    embed_norm: bool = False
+
+
+ARCHITECTURES = {
+    "Roluzen": Design("roluzen", {"rglru": _rglru_spec, "parallel": _parallel_spec}, "glu"),
+    "Tovalix": Design("tovalix", {"wkv": _wkv_spec, "hgrn2": _hgrn2_spec, "attention": _rotary_spec}, "xielu", embed_norm=True),
+}
+STACK_FAMILIES = tuple(d.family for d in ARCHITECTURES.values())
 
 
 def is_stack_json(c: dict) -> bool:
@@ -131,7 +220,7 @@ def describes_layer_stack(path: str) -> bool:
 def config_from_stack_json(src: Union[str, dict], dtype: Optional[torch.dtype] = None, shapes: Optional[dict] = None,
                            **overrides) -> StackConfig:
     """`src`: a checkpoint directory, a config.json path or the parsed dict. Sizes that only a tensor's shape tells (rows
-    of the bias tables) come from the safetensors headers of the directory, or from `shapes` (name -> shape)."""
+    of the bias tables, the decays' bottleneck) come from the safetensors headers of the directory, or from `shapes` (name -> shape)."""
     c = src
     if isinstance(src, str):
         path = os.path.join(src, "config.json") if os.path.isdir(src) else src
@@ -140,17 +229,18 @@ def config_from_stack_json(src: Union[str, dict], dtype: Optional[torch.dtype] =
         if shapes is None:
             from .safetensors_loader import tensor_shapes
             shapes = tensor_shapes(os.path.dirname(path))
-    specs = []
+    design, width, specs = ARCHITECTURES[c["architecture"]], int(c["width"]), []
     for i, layer in enumerate(c["layers"]):
-        if layer["type"] not in MIXER_READERS:
+        if layer["type"] not in design.mixers:
             raise ValueError(f"layer {i}: no mixer {layer['type']!r} in this framework")
         mlp = layer.get("mlp")
         if mlp is not None and mlp.get("kind") != "dense":
             raise ValueError(f"layer {i}: no feed-forward {mlp.get('kind')!r} in this framework")
-        specs.append(LayerSpec(MIXER_READERS[layer["type"]](layer["mixer"], shapes, f"l{i}.mix."),
-                               None if mlp is None else int(mlp["ff"])))
+        specs.append(LayerSpec(design.mixers[layer["type"]](layer["mixer"], shapes, f"l{i}.mix.", width),
+                               None if mlp is None else int(mlp["ff"]), design.ff_kind))
     lp = c.get("loop")
-    kw = dict(family=ARCHITECTURES[c["architecture"]], vocab_size=int(c["vocab"]), embed_dim=int(c["width"]),
+    kw = dict(family=design.family, vocab_size=int(c["vocab"]), embed_dim=width, norm_groups=int(c["norm"].get("groups") or 1),
+              embed_norm=design.embed_norm, token_side=int((c.get("token_side") or {}).get("dim") or 0),
               norm_eps=float(c["norm"]["eps"]), layer_specs=tuple(specs),
               loop=None if not lp else (int(lp["start"]), int(lp["stop"]), int(lp["times"])),
               streams=int(c.get("streams") or 0), dtype=dtype or torch.bfloat16)
@@ -170,6 +260,26 @@ class HyperConnection(nn.Module):
         self.mix = nn.Parameter(torch.eye(S, dtype=dtype, device=device))
 
 
+class PlainMLP(nn.Module):
+    """down(xielu(up x)); `act` holds the activation's two numbers."""
+
+    def __init__(self, width: int, ff: int, dtype, device=None):
+        super().__init__()
+        self.up_proj = Linear(width, ff, False, dtype, device)
+        self.down_proj = Linear(ff, width, False, dtype, device)
+        self.act = nn.Parameter(torch.full((2,), 0.5, dtype=dtype, device=device))
+
+
+class TokenSide(nn.Module):
+    """A layer's token input: norm(proj(gelu(gate x) * e))."""
+
+    def __init__(self, width: int, dim: int, eps: float, dtype, device=None):
+        super().__init__()
+        self.gate_proj = Linear(width, dim, False, dtype, device)
+        self.proj = Linear(dim, width, False, dtype, device)
+        self.norm = RMSNorm(width, eps, False, dtype, device)
+
+
 class StackLayer(nn.Module):
     def __init__(self, cfg: StackConfig, spec: LayerSpec, device=None):
         super().__init__()
@@ -182,8 +292,10 @@ class StackLayer(nn.Module):
         if spec.ff is not None:
             self.post_attention_layernorm = RMSNorm(D, eps, False, dt, device)
             # the generic gated MLP reads only these sizes
-            self.mlp = MLP(ModelConfig(embed_dim=D, hidden_dim=spec.ff, activation=cfg.activation, dtype=dt), device)
+            self.mlp = PlainMLP(D, spec.ff, dt, device) if spec.ff_kind == "xielu" else \
+                MLP(ModelConfig(embed_dim=D, hidden_dim=spec.ff, activation=cfg.activation, dtype=dt), device)
             self.hc2 = HyperConnection(cfg.streams, dt, device) if cfg.streams else None
+        self.side = TokenSide(D, cfg.token_side, eps, dt, device) if cfg.token_side else None
 
 
 class StackModel(nn.Module):
@@ -192,6 +304,10 @@ class StackModel(nn.Module):
         self.config = cfg
         dt = cfg.dtype
         self.embed_tokens = nn.Parameter(torch.empty(cfg.vocab_size, cfg.embed_dim, dtype=dt, device=device))
+        self.embed_norm = RMSNorm(cfg.embed_dim, cfg.norm_eps, False, dt, device) if cfg.embed_norm else None
+        self.side_embed = None
+        if cfg.token_side:          # row of a token: one part of `token_side` columns per layer
+            self.side_embed = nn.Parameter(torch.empty(cfg.vocab_size, cfg.num_layers * cfg.token_side, dtype=dt, device=device))
         self.layers = nn.ModuleList([StackLayer(cfg, s, device) for s in cfg.layer_specs])
         self.norm = RMSNorm(cfg.embed_dim, cfg.norm_eps, False, dt, device)
         self.lm_head = nn.Parameter(torch.empty(cfg.vocab_size, cfg.embed_dim, dtype=dt, device=device))

@@ -283,8 +283,8 @@ _lib.register_cuda_sigs({
     "tb_attn_fwd": [_lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.I, _lib.I, _lib.I, _lib.I, _lib.I, _lib.I,
                     _lib.LL, _lib.LL, _lib.LL, _lib.LL, _lib.F, _lib.F, _lib.I, _lib.I, _lib.I, _lib.P, _lib.P,
                     _lib.P, _lib.P],
-    "tb_attn_fwd_paged": [_lib.P, _lib.P, _lib.P, _lib.P, _lib.I, _lib.LL, _lib.I, _lib.I, _lib.I, _lib.F, _lib.I, _lib.I, _lib.P,
-                          _lib.I, _lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.I, _lib.P, _lib.I, _lib.I, _lib.P, _lib.P],
+    "tb_attn_fwd_paged": [_lib.P, _lib.P, _lib.P, _lib.P, _lib.I, _lib.LL, _lib.I, _lib.I, _lib.I, _lib.F, _lib.F, _lib.I, _lib.I,
+                          _lib.I, _lib.P, _lib.I, _lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.I, _lib.P, _lib.I, _lib.I, _lib.P, _lib.P],
     "tb_attn_delta": [_lib.P, _lib.LL, _lib.P, _lib.LL, _lib.P, _lib.I, _lib.I, _lib.I, _lib.I, _lib.P],
     "tb_attn_bwd": [_lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.I, _lib.I,
                     _lib.I, _lib.I, _lib.I, _lib.I, _lib.LL, _lib.LL, _lib.LL, _lib.LL, _lib.LL, _lib.LL,
@@ -321,17 +321,17 @@ def attn_fwd(q, k, v, *, scale: float, causal: bool = True, window: int = 0, sof
 
 
 def attn_fwd_paged(q, k_pool, v_pool, rb, table, page_size: int, *, num_heads: int, num_kv_heads: int, head_dim: int, scale: float,
-                   window: int = 0, keep_first: int = 0, bias=None) -> torch.Tensor:
+                   softcap: float = 0.0, window: int = 0, chunk: int = 0, keep_first: int = 0, bias=None) -> torch.Tensor:
     """Flash attention of the entries of a `ops.ragged.RaggedBatch` (prompt portions) over the paged cache that already
     holds their keys and values. q [n, N * H] bf16 -> [n, N * H]; pools [pages, page_size, KH * H], page_size a multiple of
-    64. `window` / `keep_first` / `bias` as in `paged_decode`."""
+    64. `softcap` / `window` / `chunk` / `keep_first` / `bias` as in `paged_decode`."""
     n = q.shape[0]
     assert q.is_contiguous() and page_size % 64 == 0 and k_pool.is_contiguous() and k_pool.shape == v_pool.shape
     out = torch.empty_like(q)
     t0, ent, _, tiles = rb.tiles(128)
     rc = _lib.cuda().tb_attn_fwd_paged(q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(), out.data_ptr(), n,
-                                       k_pool.shape[0] * page_size, num_heads, num_kv_heads, head_dim, float(scale), int(window),
-                                       int(keep_first), _lib.ptr(bias), 0 if bias is None else bias.shape[1] - 1,
+                                       k_pool.shape[0] * page_size, num_heads, num_kv_heads, head_dim, float(scale), float(softcap),
+                                       int(window), int(chunk), int(keep_first), _lib.ptr(bias), 0 if bias is None else bias.shape[1] - 1,
                                        rb.cu.data_ptr(), rb.slot.data_ptr(), rb.pos0.data_ptr(), t0.data_ptr(), ent.data_ptr(),
                                        tiles, table.data_ptr(), table.shape[1], page_size,
                                        _lib.status_buffer(q.device).data_ptr(), _lib.stream_ptr())
@@ -372,7 +372,7 @@ def attn_bwd(dout, q, k, v, o, lse, *, scale: float, causal: bool = True, window
 _lib.register_cuda_sigs({
     "tb_kv_write": [_lib.P, _lib.P, _lib.LL, _lib.P, _lib.P, _lib.P, _lib.I, _lib.I, _lib.P, _lib.P, _lib.I, _lib.I, _lib.P],
     "tb_paged_decode": [_lib.P, _lib.LL, _lib.P, _lib.P, _lib.P, _lib.I, _lib.I, _lib.P, _lib.P, _lib.I, _lib.I, _lib.I,
-                        _lib.I, _lib.I, _lib.F, _lib.F, _lib.I, _lib.I, _lib.P, _lib.I, _lib.I, _lib.LL, _lib.P, _lib.P, _lib.P,
+                        _lib.I, _lib.I, _lib.F, _lib.F, _lib.I, _lib.I, _lib.I, _lib.P, _lib.I, _lib.I, _lib.LL, _lib.P, _lib.P, _lib.P,
                         _lib.LL, _lib.P, _lib.P],
     "tb_qkv_post": [_lib.P, _lib.LL, _lib.P, _lib.P, _lib.P, _lib.P, _lib.F, _lib.F, _lib.P, _lib.P, _lib.P, _lib.I,
                     _lib.I, _lib.P, _lib.P, _lib.I, _lib.I, _lib.I, _lib.I, _lib.P],
@@ -444,10 +444,11 @@ def decode_split_tokens(batch: int, num_kv_heads: int, max_ctx: int = 0) -> int:
 
 
 def paged_decode(q, k_pool, v_pool, page_table, seq_ids, seq_lens, *, num_kv_heads: int, page_size: int, max_ctx: int,
-                 scale: float, softcap: float = 0.0, window: int = 0, keep_first: int = 0, bias=None, workspace=None, out=None,
-                 split_tokens: int = 0):
+                 scale: float, softcap: float = 0.0, window: int = 0, chunk: int = 0, keep_first: int = 0, bias=None,
+                 workspace=None, out=None, split_tokens: int = 0):
     """Single-token attention over a paged KV cache. q [B, N, H] bf16 (row stride free) -> out [B, N, H] bf16.
-    With a window, the first `keep_first` tokens of a sequence stay visible. `bias` fp32 [N, far + 1] is added to the
+    `chunk` > 0: a query sees the keys of its own chunk of that many positions, counted from the sequence's start.
+    With a window or chunks, the first `keep_first` tokens of a sequence stay visible. `bias` fp32 [N, far + 1] is added to the
     scaled score of a key at distance min(distance, far).
     `workspace` (two fp32 buffers) must be sized for ceil(max_ctx / split_tokens) splits."""
     B, N, H = q.shape
@@ -464,8 +465,9 @@ def paged_decode(q, k_pool, v_pool, page_table, seq_ids, seq_lens, *, num_kv_hea
         out = torch.empty((B, N, H), dtype=q.dtype, device=q.device)
     rc = _lib.cuda().tb_paged_decode(q.data_ptr(), q.stride(0), k_pool.data_ptr(), v_pool.data_ptr(), page_table.data_ptr(),
                                      page_table.shape[1], page_size, seq_ids.data_ptr(), seq_lens.data_ptr(), B, N,
-                                     num_kv_heads, H, max_ctx, float(scale), float(softcap), int(window), int(keep_first),
-                                     _lib.ptr(bias), 0 if bias is None else bias.shape[1] - 1, int(split_tokens), pool_rows, workspace[0].data_ptr(), workspace[1].data_ptr(),
+                                     num_kv_heads, H, max_ctx, float(scale), float(softcap), int(window), int(chunk),
+                                     int(keep_first), _lib.ptr(bias), 0 if bias is None else bias.shape[1] - 1, int(split_tokens),
+                                     pool_rows, workspace[0].data_ptr(), workspace[1].data_ptr(),
                                      out.data_ptr(), N * H, _lib.status_buffer(q.device).data_ptr(), _lib.stream_ptr())
     _lib.check(rc, "tb_paged_decode")
     _count(2)

@@ -1,4 +1,4 @@
-"""Launchers of the layer-stack kernels (csrc/stack.cu, recurrent.cu, window_attention.cu). Activations and weights are
+"""Launchers of the layer-stack kernels (csrc/stack.cu, recurrent.cu, linear_attention.cu, window_attention.cu). Activations and weights are
 bf16 or float (the `dtype` argument of the entry points), residual streams, states and gates fp32."""
 from __future__ import annotations
 
@@ -13,8 +13,13 @@ from .ragged import RaggedBatch
 _P, _I, _LL, _F = _lib.P, _lib.I, _lib.LL, _lib.F
 _RB = [_P, _P, _P, _P, _I, _I]
 _lib.register_cuda_sigs({
-    "tb_stream_step": [_I, _P, _I, _I, _I, _F, _P, _P, _P, _P, _P, _P, _P, _P, _I, _P, _P, _P, _P, _P],
-    "tb_few_outputs": [_P, _P, _I, _I, _I, _P, _P],
+    "tb_stream_step": [_I, _P, _I, _I, _I, _F, _P, _P, _P, _P, _P, _P, _P, _P, _I, _P, _I, _P, _P, _P, _P, _P, _I, _P, _P, _P, _P, _P],
+    "tb_few_outputs": [_P, _P, _I, _I, _I, _I, _P, _I, _P, _LL, _I, _P, _I, _P],
+    "tb_small_act": [_I, _P, _I, _I, _I, _P, _I, _P, _LL, _I, _P, _P],
+    "tb_token_shift": [_I, _P, _P, _I, _P, *_RB, _I, _P, _P],
+    "tb_xielu": [_I, _P, _P, _LL, _P],
+    "tb_gated_linear": [_I, _I, _P, _LL, _P, _LL, _P, _LL, _P, _LL, _P, _LL, _P, _P, *_RB, _I, _I, _I, _P, _P, _P, _I, _P, _I, _F,
+                        _P, _P, _I, _I, _P],
     "tb_silu_mul": [_I, _P, _P, _LL, _I, _P],
     "tb_gate_outputs": [_I, _P, _P, _P, _LL, _I, _I, _P, _F, _I, _I, _I, _I, _P, _P, _P],
     "tb_rglru": [_I, _P, _LL, _I, _I, _P, _P, _P, _P, _P, _P, _P, *_RB, _I, _I, _I, _P, _P, _P, _P, _P, _P, _I, _P, _P,
@@ -22,7 +27,8 @@ _lib.register_cuda_sigs({
     "tb_mlstm_slices": [_I],
     "tb_mlstm": [_I, _P, _LL, _I, _I, _I, _P, _P, _P, _F, *_RB, _I, _I, _I, _P, _P, _P, _P, _I, _I, _P],
     "tb_qk_norm_write": [_I, _P, _LL, _I, _I, _I, _P, _P, _F, *_RB, _P, _I, _I, _I, _I, _I, _P, _P, _P, _P],
-    "tb_window_attn": [_I, _P, _P, _P, *_RB, _P, _I, _I, _I, _I, _I, _I, _F, _P, _I, _I, _I, _P, _P],
+    "tb_rope_norm_write": [_I, _P, _LL, _I, _I, _I, _P, _P, _I, _F, *_RB, _P, _I, _I, _I, _I, _I, _I, _P, _P, _P, _P],
+    "tb_window_attn": [_I, _P, _P, _P, *_RB, _P, _I, _I, _I, _I, _I, _I, _F, _F, _P, _I, _I, _I, _I, _P, _P],
 })
 
 
@@ -35,20 +41,50 @@ def _dt(t: torch.Tensor) -> int:
 
 
 def stream_step(x: torch.Tensor, eps: float, *, y=None, y2=None, wy=None, wy2=None, mix=None, w_out=None, tokens=None, embed=None,
-                w_in=None, norm_w=None, sum_out: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
-    """Close one sublayer (y [, y2 with their norms], mix, w_out; or start from the embedding rows of `tokens`) and open
-    the next: returns h = norm(sum_s w_in[s] x_s) * norm_w (w_in None: the plain sum; norm_w None: nothing follows).
-    x fp32 [n, S, D] is updated in place; `sum_out` fp32 [n, D] receives the sum of the streams."""
+                embed_w=None, groups: int = 1, w_in=None, norm_w=None, raw: bool = False, shift=None, rb: Optional[RaggedBatch] = None,
+                sum_out: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """Close one sublayer (y [, y2 with their norms; y alone with its norm wy], mix, w_out; or start from the embedding rows
+    of `tokens`, normed with embed_w if given) and open the next: returns h = norm(sum_s w_in[s] x_s) * norm_w (w_in None:
+    the plain sum; norm_w None: nothing follows, or with `raw` the sum itself). The norms of rows and embeddings are taken
+    over `groups` equal parts. x fp32 [n, S, D] is updated in place; `sum_out` fp32 [n, D] receives the sum of the streams.
+    `shift` = (mu [m, D], carry fp32 [slots, D]), for batches `rb` of single tokens: returns the m mixes
+    h + (carry - h) mu [m, n, D] instead of h and replaces the slots' carry by h."""
     n, S, D = x.shape
     ref = norm_w if norm_w is not None else (y if y is not None else embed)
-    h = torch.empty((n, D), dtype=ref.dtype, device=x.device) if norm_w is not None else None
+    mu, carry = shift or (None, None)
+    mixes = torch.empty((mu.shape[0], n, D), dtype=ref.dtype, device=x.device) if shift else None
+    h = torch.empty((n, D), dtype=ref.dtype, device=x.device) if (norm_w is not None and not shift) or raw else None
     rc = _lib.cuda().tb_stream_step(_dt(ref), x.data_ptr(), n, S, D, float(eps), _lib.ptr(y), _lib.ptr(y2), _lib.ptr(wy),
                                     _lib.ptr(wy2), _lib.ptr(mix), _lib.ptr(w_out), _lib.ptr(tokens), _lib.ptr(embed),
-                                    0 if embed is None else embed.shape[0], _lib.ptr(w_in), _lib.ptr(norm_w), _lib.ptr(h),
-                                    _lib.ptr(sum_out), _lib.stream_ptr())
+                                    0 if embed is None else embed.shape[0], _lib.ptr(embed_w), int(groups), _lib.ptr(w_in),
+                                    _lib.ptr(norm_w), _lib.ptr(h), _lib.ptr(sum_out), _lib.ptr(mu), 0 if mu is None else mu.shape[0],
+                                    _lib.ptr(carry), _lib.ptr(mixes), rb.slot.data_ptr() if shift else 0,
+                                    rb.pos0.data_ptr() if shift else 0, _lib.stream_ptr())
     _lib.check(rc, "tb_stream_step")
     _count()
-    return h
+    return mixes if shift else h
+
+
+def token_shift(h, mu, carry, rb: RaggedBatch) -> torch.Tensor:
+    """h [n, D] + (row of the token before - h) * mu[m] -> [m, n, D]; the row before a portion is its slot's `carry` (zero at
+    the start of a sequence). The carry is replaced by the recurrence that runs on the mixes."""
+    n, D = h.shape
+    assert h.is_contiguous() and mu.is_contiguous()
+    mixes = torch.empty((mu.shape[0], n, D), dtype=h.dtype, device=h.device)
+    rc = _lib.cuda().tb_token_shift(_dt(h), h.data_ptr(), mu.data_ptr(), mu.shape[0], carry.data_ptr(), *rb.args(), D,
+                                    mixes.data_ptr(), _lib.stream_ptr())
+    _lib.check(rc, "tb_token_shift")
+    _count()
+    return mixes
+
+
+def xielu_(x: torch.Tensor, act: torch.Tensor) -> torch.Tensor:
+    """xIELU in place, act = its two numbers (before softplus)."""
+    assert x.is_contiguous() and act.dtype == x.dtype
+    rc = _lib.cuda().tb_xielu(_dt(x), x.data_ptr(), act.data_ptr(), x.numel(), _lib.stream_ptr())
+    _lib.check(rc, "tb_xielu")
+    _count()
+    return x
 
 
 def silu_mul(gu: torch.Tensor) -> torch.Tensor:
@@ -61,13 +97,59 @@ def silu_mul(gu: torch.Tensor) -> torch.Tensor:
     return h
 
 
-def few_outputs(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
-    """x bf16 [n, K] @ w^T [N, K] -> fp32 [n, N] for a handful of outputs and decode-size n (a GEMM tile would leave one CTA
-    with the whole contraction)."""
+ACT_NONE, ACT_TANH, ACT_GELU_ROW = 0, 1, 2      # csrc/stack.cu: apply_small
+
+
+def few_outputs(x: torch.Tensor, w: torch.Tensor, act: int = ACT_NONE, tokens=None, rows=None, col: int = 0) -> torch.Tensor:
+    """act(x bf16 [n, K] @ w^T [N, K]) for a handful of outputs and decode-size n (a GEMM tile would leave one CTA with the
+    whole contraction): fp32 [n, N], or bf16 after an activation. ACT_GELU_ROW multiplies by columns col .. col + N of the
+    tokens' rows of the table `rows`."""
     assert x.dtype == w.dtype == torch.bfloat16 and x.is_contiguous() and w.is_contiguous() and x.shape[1] % 8 == 0
-    out = torch.empty((x.shape[0], w.shape[0]), dtype=torch.float32, device=x.device)
-    rc = _lib.cuda().tb_few_outputs(x.data_ptr(), w.data_ptr(), x.shape[0], x.shape[1], w.shape[0], out.data_ptr(), _lib.stream_ptr())
+    out = torch.empty((x.shape[0], w.shape[0]), dtype=torch.float32 if act == ACT_NONE else torch.bfloat16, device=x.device)
+    rc = _lib.cuda().tb_few_outputs(x.data_ptr(), w.data_ptr(), x.shape[0], x.shape[1], w.shape[0], act, _lib.ptr(tokens),
+                                    0 if rows is None else rows.shape[0], _lib.ptr(rows), 0 if rows is None else rows.shape[1],
+                                    col, out.data_ptr(), int(act != ACT_NONE), _lib.stream_ptr())
     _lib.check(rc, "tb_few_outputs")
+    _count()
+    return out
+
+
+def small_act(z: torch.Tensor, dtype, act: int, tokens=None, rows=None, col: int = 0) -> torch.Tensor:
+    """The activations of `few_outputs` on fp32 products z [n, N] of any size."""
+    assert z.dtype == torch.float32 and z.is_contiguous()
+    out = torch.empty(z.shape, dtype=dtype, device=z.device)
+    rc = _lib.cuda().tb_small_act(_dt(out), z.data_ptr(), z.shape[0], z.shape[1], act, _lib.ptr(tokens),
+                                  0 if rows is None else rows.shape[0], _lib.ptr(rows), 0 if rows is None else rows.shape[1], col,
+                                  out.data_ptr(), _lib.stream_ptr())
+    _lib.check(rc, "tb_small_act")
+    _count()
+    return out
+
+
+GATES_BONUS, GATES_LOWER = 0, 1                 # csrc/linear_attention.cu: Mode
+
+
+def gated_linear(mode: int, q, k, v, z, c0, c1, rb: RaggedBatch, heads: int, dk: int, dv: int, state, norm_w, eps: float, *,
+                 gate=None, per_head: bool = False, carry=None, h=None, plain: bool = False) -> torch.Tensor:
+    """Matrix state with a decay per head and channel over a ragged batch, its head norm and output gate; [n, heads * dv].
+    GATES_BONUS: decay exp(-exp(z + c0)), keys k, bonus c1 for the current token. GATES_LOWER: decay
+    c1 + (1 - c1) sigmoid(z + c0), key 1 - decay, silu(q). q, k, v, gate: column views of rows [n, ..]; z fp32.
+    norm_w [dv], or [heads * dv] with per_head. carry / h: see `token_shift` (portions only).
+    `plain`: the token by token kernel of the 32-bit path, also for bf16."""
+    n = q.shape[0]
+    assert z.dtype == torch.float32 and all(t is None or t.stride(1) == 1 for t in (q, k, v, z, gate))
+    one = rb.decode and not plain
+    raw = torch.empty((n, heads * dv), dtype=torch.float32, device=q.device) if not one or dv > 256 else None
+    out = torch.empty((n, heads * dv), dtype=q.dtype, device=q.device)
+    ld = lambda t: 0 if t is None else t.stride(0)  # noqa: E731
+    if rb.decode:
+        carry = h = None                        # the launch that made the mixes has replaced it
+    rc = _lib.cuda().tb_gated_linear(_dt(q), mode, q.data_ptr(), ld(q), _lib.ptr(k), ld(k), v.data_ptr(), ld(v), _lib.ptr(gate),
+                                     ld(gate), z.data_ptr(), ld(z), c0.data_ptr(), c1.data_ptr(), *rb.args(), heads, dk, dv,
+                                     state.data_ptr(), _lib.ptr(h), _lib.ptr(carry), 0 if h is None else h.shape[1],
+                                     norm_w.data_ptr(), int(per_head), float(eps), _lib.ptr(raw), out.data_ptr(), int(one),
+                                     int(not plain), _lib.stream_ptr())
+    _lib.check(rc, "tb_gated_linear")
     _count()
     return out
 
@@ -139,14 +221,30 @@ def qk_norm_write(proj, q_off: int, k_off: int, v_off: int, q_w, k_w, eps: float
     return q
 
 
+def rope_norm_write(proj, q_off: int, k_off: int, v_off: int, cos, sin, rot_dims: int, eps: float, rb: RaggedBatch, table,
+                    page_size: int, heads: int, kv_heads: int, dim: int, vdim: int, k_pool, v_pool) -> torch.Tensor:
+    """Rotation of the first rot_dims dimensions of every query and key head (cos / sin fp32 [positions, rot_dims / 2]), then
+    each head divided by its root mean square; q [n, heads * dim] is returned, k and v rows go to their pages. kv_heads 0: the
+    rows hold queries only and nothing is written."""
+    n = proj.shape[0]
+    q = torch.empty((n, heads * dim), dtype=proj.dtype, device=proj.device)
+    rc = _lib.cuda().tb_rope_norm_write(_dt(proj), proj.data_ptr(), proj.stride(0), q_off, k_off, v_off, _lib.ptr(cos),
+                                        _lib.ptr(sin), rot_dims, float(eps), *rb.args(), table.data_ptr(), table.shape[1],
+                                        page_size, heads, kv_heads, dim, vdim, q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(),
+                                        _lib.stream_ptr())
+    _lib.check(rc, "tb_rope_norm_write")
+    _count()
+    return q
+
+
 def window_attn(q, k_pool, v_pool, rb: RaggedBatch, table, page_size: int, sp, bias) -> torch.Tensor:
-    """`sp`: models.mixers.WindowAttentionSpec; bias fp32 [heads, far + 1]. Returns [n, heads * vdim]."""
+    """`sp`: an attention spec of models.mixers; bias fp32 [heads, far + 1] or None. Returns [n, heads * vdim]."""
     n = q.shape[0]
     out = torch.empty((n, sp.heads * sp.vdim), dtype=q.dtype, device=q.device)
     rc = _lib.cuda().tb_window_attn(_dt(q), q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(), *rb.args(), table.data_ptr(),
                                     table.shape[1], page_size, sp.heads, sp.kv_heads, sp.dim, sp.vdim, float(sp.scale),
-                                    bias.data_ptr(), bias.shape[1] - 1, sp.window, sp.keep_first, out.data_ptr(),
-                                    _lib.stream_ptr())
+                                    float(sp.softcap), _lib.ptr(bias), 0 if bias is None else bias.shape[1] - 1, sp.window,
+                                    sp.chunk, sp.keep_first, out.data_ptr(), _lib.stream_ptr())
     _lib.check(rc, "tb_window_attn")
     _count()
     return out
