@@ -1,9 +1,17 @@
-"""Small Roluzen checkpoints with random weights for the layer-stack tests (config.json dict + tensors by name)."""
+"""Small Roluzen and Tovalix checkpoints with random weights for the layer-stack tests (config.json dict + tensors by name)."""
 import json
 import os
 
 import torch
 
+from tests import roluzen_oracle, tovalix_oracle
+
+
+def oracle(cfg):
+    return {"Roluzen": roluzen_oracle, "Tovalix": tovalix_oracle}[cfg["architecture"]]
+
+
+# ---- Roluzen
 
 def attention(heads=4, kv_heads=2, dim=16, vdim=24, scale=0.3, bias_max=40, size=20, keep_first=3):
     return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "bias_max": bias_max,
@@ -29,6 +37,29 @@ def config(layers, width=48, vocab=101, streams=3, loop=None, eps=1e-5):
             "width": width}
 
 
+# ---- Tovalix
+def wkv(heads=3, dim=16, ff=56):
+    return {"type": "wkv", "mixer": {"heads": heads, "dim": dim}, "mlp": None if ff is None else {"kind": "dense", "ff": ff}}
+
+
+def hgrn2(heads=2, dim=24, vdim=40, ff=72):
+    return {"type": "hgrn2", "mixer": {"heads": heads, "dim": dim, "vdim": vdim},
+            "mlp": None if ff is None else {"kind": "dense", "ff": ff}}
+
+
+def rotary(heads=4, kv_heads=2, dim=16, vdim=24, rot=8, base=900.0, scale=0.6, cap=6.0, chunk=20, kv_from=None, ff=64):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "rot": {"dims": rot, "base": base}, "scale": scale,
+         "softcap": cap, "mask": {"size": chunk}}
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return {"type": "attention", "mixer": m, "mlp": None if ff is None else {"kind": "dense", "ff": ff}}
+
+
+def tovalix(layers, width=48, vocab=101, groups=3, side=8, eps=1e-5):
+    return {"architecture": "Tovalix", "layers": layers, "norm": {"eps": eps, "groups": groups}, "token_side": {"dim": side},
+            "vocab": vocab, "width": width}
+
+
 # sizes apart from each other, layers with and without feed-forward, loops and none, one stream and several, odd widths;
 # "wide" has the head sizes and widths of the tensor-core kernels
 CASES = {
@@ -40,12 +71,24 @@ CASES = {
     "wide": config([parallel(attention(heads=6, kv_heads=3, dim=64, vdim=64, scale=0.11, size=70, keep_first=5, bias_max=90),
                              memory(2, 40, 72), ff=128), rglru(128, 2, 4, ff=96)], width=128, streams=4, vocab=300,
                    loop={"start": 0, "stop": 1, "times": 3}),
+    # keys and values shared by layers with unequal chunks and query heads
+    "shared": tovalix([wkv(), rotary(), hgrn2(ff=None), rotary(heads=2, chunk=33, cap=3.0, kv_from=1, ff=None), wkv(2, 24)]),
+    # widths that fit no vector load or tensor-core tile, one norm group, a shared cache read twice
+    "uneven": tovalix([hgrn2(3, 12, 6, ff=31), rotary(3, 1, 10, 6, rot=6, chunk=9, cap=40.0, ff=33), wkv(3, 10, ff=45),
+                       rotary(3, 1, 10, 6, rot=6, chunk=70, kv_from=1), rotary(3, 1, 10, 6, rot=6, chunk=14, kv_from=1, ff=None)],
+                      width=36, vocab=67, groups=1, side=3, eps=1e-3),
+    # the head sizes of the tensor-core kernels, values wider than one slice
+    "tiles": tovalix([rotary(6, 3, 64, 64, rot=32, chunk=70, scale=0.3, cap=9.0, ff=128), wkv(2, 64, ff=96), hgrn2(2, 104, 136, ff=64),
+                      rotary(3, 3, 64, 64, rot=32, chunk=130, scale=0.3, cap=12.0, kv_from=0, ff=None), wkv(1, 128, ff=None)],
+                     width=128, vocab=300, groups=4, side=16),
 }
 
 
 def weights(cfg, seed=0, buckets=11):
-    """Random tensors of the checkpoint, in bf16-representable fp32. Decays reach from fast to very slow and the bias table
-    is large, so that far tokens, window edges and kept tokens matter."""
+    """Random tensors of the checkpoint, in bf16-representable fp32. Decays reach from fast to very slow, the bias table is
+    large and attention is sharp, so that far tokens, window and chunk edges and kept tokens matter."""
+    if cfg["architecture"] == "Tovalix":
+        return tovalix_weights(cfg, seed)
     g = torch.Generator().manual_seed(seed)
     w = {}
 
@@ -104,6 +147,67 @@ def weights(cfg, seed=0, buckets=11):
             put(p + "hc2.out", S, mean=0.4)
             put(p + "hc2.mix", S, S, std=0.15)
             w[p + "hc2.mix"] = (w[p + "hc2.mix"] + 0.75 * torch.eye(S)).to(torch.bfloat16).float()
+    return w
+
+
+def tovalix_weights(cfg, seed=0, rank=6):
+    g = torch.Generator().manual_seed(seed)
+    w = {}
+
+    def put(name, *shape, std=None, mean=0.0, uniform=None):
+        x = torch.randn(*shape, generator=g)
+        if uniform is not None:
+            x = uniform[0] + (uniform[1] - uniform[0]) * torch.rand(*shape, generator=g)
+        else:
+            x = mean + ((shape[-1] ** -0.5 if len(shape) > 1 else 0.2) if std is None else std) * x
+        w[name] = x.to(torch.bfloat16).float()
+
+    D, V, dim, n = cfg["width"], cfg["vocab"], cfg["token_side"]["dim"], len(cfg["layers"])
+    put("embed", V, D, std=0.7)
+    put("embed.norm", D, mean=1.0)
+    put("side.embed", V, n * dim, std=1.0)
+    put("head", V, D)
+    put("final.norm", D, mean=1.0)
+    for i, layer in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", layer["mixer"]
+        put(p + "norm1", D, mean=1.0)
+        if layer["type"] == "wkv":
+            C = m["heads"] * m["dim"]
+            for s in "rkvgw":
+                put(f"{p}mix.mu.{s}", D, uniform=(0.0, 1.0))
+            for s in "rkvg":
+                put(f"{p}mix.{s}", C, D)
+            put(p + "mix.w1", rank, D)
+            put(p + "mix.w2", C, rank, std=0.5)
+            put(p + "mix.w0", C, uniform=(-7.0, 1.5))
+            put(p + "mix.u", m["heads"], m["dim"], std=1.0)
+            put(p + "mix.norm", C, mean=1.0)
+            put(p + "mix.o", D, C)
+        elif layer["type"] == "hgrn2":
+            K, C = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+            for s, rows in (("q", K), ("f", K), ("v", C)):
+                put(f"{p}mix.{s}", rows, D)
+            put(p + "mix.f.b", K, std=2.0, mean=2.0)
+            put(p + "mix.lower", K, uniform=(0.0, 0.99))
+            put(p + "mix.norm", m["vdim"], mean=1.0)
+            put(p + "mix.o", D, C)
+        else:
+            H, G = m["heads"], m["kv_heads"]
+            own = m.get("kv_from") is None
+            for s, rows in (("q", H * m["dim"]),) + ((("k", G * m["dim"]), ("v", G * m["vdim"])) if own else ()):
+                put(f"{p}mix.{s}", rows, D)
+                put(f"{p}mix.{s}.b", rows, std=0.5)
+            put(p + "mix.o", D, H * m["vdim"])
+            put(p + "mix.o.b", D)
+        if layer["mlp"] is not None:
+            ff = layer["mlp"]["ff"]
+            put(p + "norm2", D, mean=1.0)
+            put(p + "mlp.up", ff, D)
+            put(p + "mlp.down", D, ff)
+            put(p + "mlp.act", 2, std=1.0)
+        put(p + "side.gate", dim, D)
+        put(p + "side.proj", D, dim)
+        put(p + "side.norm", D, std=0.3)
     return w
 
 

@@ -1,11 +1,12 @@
-"""Distance-biased sliding-window attention with kept first tokens over the paged cache, in its three kernels (general, flash
-attention over pages, paged decode): against a dense restatement, with queries whose scores single out one key at an edge."""
+"""Attention of layer-stack models over the paged cache (distance-biased sliding windows with kept first tokens; rotary, capped
+attention inside chunks), in its three kernels (general, flash attention over pages, paged decode): against a dense restatement, with queries whose scores single out one key at an edge."""
 import math
 
 import pytest
 import torch
 
 from tests import roluzen_oracle as O
+from tests import tovalix_oracle as TO
 from tests.test_stack_kernels_gpu import batch, rand, rel
 
 pytestmark = pytest.mark.gpu
@@ -61,7 +62,7 @@ def run(kind, cache, rb, q, sp, bias, split=0):
     n = q.shape[0]
     if kind == "general":
         return SK.window_attn(q.reshape(n, -1), cache.k, cache.v, rb, cache.table, cache.page, sp, bias).view(n, sp.heads, sp.vdim)
-    kw = dict(scale=sp.scale, window=sp.window, keep_first=sp.keep_first, bias=bias)
+    kw = dict(scale=sp.scale, softcap=sp.softcap, window=sp.window, chunk=sp.chunk, keep_first=sp.keep_first, bias=bias)
     if kind == "decode":
         return K.paged_decode(q, cache.k, cache.v, cache.table, rb.slot, rb.pos0 + 1, num_kv_heads=sp.kv_heads, page_size=cache.page,
                               max_ctx=cache.table.shape[1] * cache.page, split_tokens=split, **kw)
@@ -203,3 +204,117 @@ def test_existing_decode_attention_without_bias_is_unchanged_by_the_tile_walk():
         out = run("decode", cache, rb, q, sp, None, split)
         for s, (k, v) in enumerate(cache.seqs):
             assert rel(out[s:s + 1], dense(q[s:s + 1], k, v, k.shape[0] - 1, sp.scale, zero, 100, 0)) < 1.2e-2
+
+
+# ------------------------------------------------------------------------------------------------ rotary, capped, in chunks
+def rotary(H, G, dq, dv, chunk, cap=0.0, scale=0.2, rot=0):
+    from tunix_b200.models.mixers import RotaryAttentionSpec
+    return RotaryAttentionSpec(heads=H, kv_heads=G, dim=dq, vdim=dv, scale=scale, rot_dims=rot, rot_base=100.0, softcap=cap, chunk=chunk)
+
+
+def dense_chunks(q, k, v, i0, sp):
+    q, k, v = (t.double().cpu() for t in (q, k, v))
+    out = torch.zeros(*q.shape[:2], v.shape[2], dtype=torch.float64)
+    for t in range(q.shape[0]):
+        js = [j for j in range(k.shape[0]) if TO.visible(i0 + t, j, sp.chunk or 10 ** 9)]
+        for h in range(sp.heads):
+            g = h // (sp.heads // sp.kv_heads)
+            s = k[js, g] @ q[t, h] * sp.scale
+            if sp.softcap:
+                s = sp.softcap * torch.tanh(s / sp.softcap)
+            out[t, h] = torch.softmax(s, -1) @ v[js, g]
+    return out
+
+
+CHUNKS = [(20, 3.0), (64, 0.0), (65, 8.0), (70, 50.0), (200, 1.5), (1, 4.0), (0, 2.0)]
+
+
+@pytest.mark.parametrize("chunk,cap", CHUNKS)
+@pytest.mark.parametrize("kind,dtype,H,G,dq,dv", GENERAL + FLASH)
+def test_chunked_portions(kind, dtype, H, G, dq, dv, chunk, cap):
+    sp = rotary(H, G, dq, dv, chunk, cap)
+    cache = Cache([300, 64, 130, 7], G, dq, dv, dtype, seed=21)
+    parts = [(0, 120, 180), (1, 0, 64), (2, 128, 2), (3, 0, 7), (0, 69, 131)]
+    q = rand(sum(n for _, _, n in parts), H, dq, dtype=dtype, std=2.0)
+    out, at = run(kind, cache, batch(parts), q, sp, None), 0
+    for s, p, n in parts:
+        k, v = cache.seqs[s]
+        assert rel(out[at:at + n], dense_chunks(q[at:at + n], k[:p + n], v[:p + n], p, sp)) < tol(dtype), s
+        at += n
+
+
+@pytest.mark.parametrize("chunk,cap", CHUNKS)
+@pytest.mark.parametrize("kind,dtype,H,G,dq,dv", GENERAL[:2] + DECODE)
+def test_chunked_single_tokens(kind, dtype, H, G, dq, dv, chunk, cap):
+    sp = rotary(H, G, dq, dv, chunk, cap)
+    lens = [1, 20, 21, 63, 64, 65, 66, 129, 140, 141, 300]
+    cache = Cache(lens, G, dq, dv, dtype, seed=22)
+    rb = batch([(s, n - 1, 1) for s, n in enumerate(lens)] + [(len(lens), 0, 1)])
+    rb.pos0[-1] = -1                                                    # idle
+    q = rand(len(lens) + 1, H, dq, dtype=dtype, std=2.0)
+    want = [dense_chunks(q[s:s + 1], k, v, lens[s] - 1, sp) for s, (k, v) in enumerate(cache.seqs)]
+    for split in (0, 64, 128, 512):
+        out = run(kind, cache, rb, q, sp, None, split)
+        for s, w in enumerate(want):
+            assert rel(out[s:s + 1], w) < tol(dtype), (s, split)
+        assert out[-1].abs().max() == 0
+        if kind == "general":
+            break
+
+
+@pytest.mark.parametrize("chunk", [20, 64, 70, 129, 200])
+@pytest.mark.parametrize("kind,dtype,H,G,dq,dv,decoded", [(*c, d) for d, cs in ((False, GENERAL[:2] + FLASH[:2]), (True, GENERAL[:2] + DECODE[:2]))
+                                                          for c in cs])
+def test_one_key_at_a_chunk_edge(kind, dtype, H, G, dq, dv, chunk, decoded):
+    """Every query asks for one key: the first of its chunk, the one before it, page edges, the sequence's first token, itself."""
+    sp = rotary(H, G, dq, dv, chunk, cap=60.0, scale=0.3)
+    cache = Cache([330], G, dq, dv, dtype, seed=23, unit=True)
+    k, v = cache.seqs[0]
+    pairs = sorted({(i, j) for i in (chunk - 1, chunk, chunk + 1, 63, 64, 128, 2 * chunk, 3 * chunk + 7, 255, 256, 329) if i < 330
+                    for j in (i, i - 1, i - i % chunk, i - i % chunk - 1, 0, 63, 64, 127, 128) if 0 <= j <= i})
+    if decoded:
+        got = torch.cat([run(kind, cache, batch([(0, i, 1)]), outstanding(cache, 0, [i], [j], H, dq), sp, None) for i, j in pairs])
+    else:
+        rows = []
+        for i, j in pairs:
+            lo = max(0, i - 2)
+            q = outstanding(cache, 0, range(lo, i + 1), [*range(lo, i), j], H, dq)
+            rows.append(run(kind, cache, batch([(0, lo, i + 1 - lo)]), q, sp, None)[-1:])
+        got = torch.cat(rows)
+    for (i, j), o in zip(pairs, got):
+        val = torch.stack([v[j, h // (H // G)] for h in range(H)]).double().cpu()
+        err = ((o.double().cpu() - val).norm() / val.norm()).item()
+        assert err < 0.05 if TO.visible(i, j, chunk) else err > 0.3, (i, j, err)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("H,G,dq,dv,rot", [(4, 2, 16, 24, 16), (3, 1, 10, 6, 6), (8, 4, 64, 64, 64), (2, 2, 128, 128, 32), (5, 1, 24, 8, 0),
+                                           (1, 1, 300, 20, 200), (4, 2, 256, 128, 256), (2, 1, 72, 200, 48)])
+def test_rotation_norm_and_page_write(H, G, dq, dv, rot, dtype):
+    """Rotation before the norm, far positions, pass-through dimensions, pages; queries alone for a layer that shares its keys."""
+    from tunix_b200.models.stack_exec import rope_table
+    from tunix_b200.ops import stack_kernels as SK
+    NQ, NK, NV, eps = H * dq, G * dq, G * dv, 1e-2
+    rb = batch([(1, 62, 4), (0, 0, 3), (2, 5, 1), (3, 700, 1)])
+    rb.pos0[2] = -1
+    off, n = 8, 9
+    proj = rand(n, off + NQ + NK + NV, dtype=dtype, std=0.3)
+    table = torch.full((4, 12), -1, dtype=torch.int32)
+    table[0, 0], table[1, 0], table[1, 1], table[3, 10] = 4, 2, 0, 1
+    table = table.cuda()
+    kp, vp = torch.zeros(5, 64, NK, device="cuda", dtype=dtype), torch.zeros(5, 64, NV, device="cuda", dtype=dtype)
+    cos, sin = rope_table(768, rot, 100.0, "cuda")
+    args = (cos, sin, rot, eps, rb, table, 64)
+    q = SK.rope_norm_write(proj, off, off + NQ, off + NQ + NK, *args, H, G, dq, dv, kp, vp)
+    pos = torch.tensor([62, 63, 64, 65, 0, 1, 2, 5, 700])
+    d = proj.double().cpu()
+    turn = lambda x, heads: TO.rms(TO.rotate(x.reshape(n, heads, dq), pos, rot, 100.0), eps).reshape(n, -1)  # noqa: E731
+    wq, wk = turn(d[:, off:off + NQ], H), turn(d[:, off + NQ:off + NQ + NK], G)
+    t, live = 2e-6 if dtype == torch.float32 else 5e-3, [0, 1, 2, 3, 4, 5, 6, 8]
+    assert rel(q[live], wq[live]) < t and q[7].abs().max() == 0
+    for row, (pg, o) in zip(live, [(2, 62), (2, 63), (0, 0), (0, 1), (4, 0), (4, 1), (4, 2), (1, 60)]):
+        assert rel(kp[pg, o], wk[row]) < t and torch.equal(vp[pg, o], proj[row, off + NQ + NK:])
+    assert (kp.abs().sum(-1) > 0).sum() == 8 and (vp.abs().sum(-1) > 0).sum() == 8
+    alone = proj[:, off:off + NQ].contiguous()
+    before = kp.clone()
+    assert torch.equal(SK.rope_norm_write(alone, 0, NQ, NQ, *args, H, 0, dq, dv, kp, vp), q) and torch.equal(kp, before)

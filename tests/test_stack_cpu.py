@@ -8,6 +8,7 @@ import torch
 
 from tests import roluzen_oracle as O
 from tests import stack_cases as C
+from tests import tovalix_oracle as TO
 
 
 @pytest.mark.parametrize("name", sorted(C.CASES))
@@ -17,7 +18,7 @@ def test_checkpoint_round_trip(tmp_path, name):
     from tunix_b200.models.safetensors_saver import save_lora_merged_model_as_safetensors
     from tunix_b200.models.stack import StackModel
     cfg = C.CASES[name]
-    src = C.write(tmp_path / "roluzen-tiny", cfg, C.weights(cfg))      # a directory name that could be taken for a preset
+    src = C.write(tmp_path / (cfg["architecture"].lower() + "-tiny"), cfg, C.weights(cfg))      # a directory name that could be taken for a preset
     model, path = AutoModel.from_pretrained(src, model_source="local")
     assert isinstance(model, StackModel) and path == src
     assert model.config.runs() == O.layer_runs(cfg) and model.config.norm_eps == cfg["norm"]["eps"]
@@ -55,6 +56,43 @@ def test_cache_layout_is_per_pass():
     assert states[1] == {"S": (2, 24, 40), "n": (2, 2, 24), "m": (2, 2)}
 
 
+def test_tovalix_constants_come_from_config_json(tmp_path):
+    from tunix_b200.models.hf_config import config_from_hf
+    cfg = C.CASES["shared"]
+    src = C.write(tmp_path / "m", cfg, C.tovalix_weights(cfg, rank=5))
+    c = config_from_hf(src)
+    assert (c.norm_groups, c.token_side, c.embed_norm, c.norm_eps, c.streams, c.loop) == (3, 8, True, 1e-5, 0, None)
+    a, b = c.layer_specs[1].mixer, c.layer_specs[3].mixer
+    assert (a.scale, a.softcap, a.chunk, a.rot_dims, a.rot_base, a.kv_from) == (0.6, 6.0, 20, 8, 900.0, None)
+    assert (b.heads, b.chunk, b.softcap, b.kv_from) == (2, 33, 3.0, 1)
+    assert c.layer_specs[0].mixer.decay_rank == 5                      # told by the tensor's shape only
+    assert [s.ff for s in c.layer_specs] == [56, 64, None, None, 56] and c.layer_specs[0].ff_kind == "xielu"
+    assert (c.num_heads, c.num_kv_heads, c.head_dim) == (4, 2, 16)
+    with pytest.raises(ValueError, match="mixer"):                     # a design has its own layer types only
+        config_from_hf(dict(cfg, layers=[C.rglru()]))
+    for layers in ([C.rotary(kv_from=1), C.rotary()], [C.wkv(), C.rotary(kv_from=0)], [C.rotary(), C.rotary(kv_from=0), C.rotary(kv_from=1)],
+                   [C.rotary(), C.rotary(kv_heads=4, kv_from=0)]):
+        with pytest.raises(ValueError, match="keys and values"):
+            config_from_hf(dict(cfg, layers=layers))
+    with pytest.raises(ValueError, match="groups"):
+        config_from_hf(dict(cfg, norm={"eps": 1e-5, "groups": 5}))
+
+
+def test_shared_keys_take_no_pages():
+    from tunix_b200.generate.engine import PagePool
+    from tunix_b200.models.hf_config import config_from_hf
+    c = config_from_hf(C.CASES["shared"])
+    assert c.kv_rows() == [None, (32, 48), None, None, None] and c.kv_sources() == [0, 1, 2, 1, 4]
+    assert c.replace(loop=(0, 2, 2)).kv_sources() == [0, 1, 2, 3, 4, 3, 6]      # the latest pass of the layer
+    with pytest.raises(ValueError, match="has not run"):
+        c.replace(loop=(0, 2, 0))
+    states = c.state_shapes()
+    assert states[0] == {"S": (3, 16, 16), "last": (48,)} and states[2] == {"S": (2, 24, 40)} and states[1] == states[3] == {}
+    pool = PagePool(c, 4, 16, 2, 4, "cpu", torch.float32, prefix_caching=False)
+    assert pool.k[3] is None and pool.v[1].shape == (4, 16, 48)
+    assert pool.state.nbytes_per_slot() == 4 * (3 * 256 + 48 + 2 * 960 + 2 * 576 + 48)
+
+
 def test_pool_and_states_on_cpu():
     from tunix_b200.generate.engine import PagePool
     from tunix_b200.models.hf_config import config_from_hf
@@ -81,6 +119,11 @@ def test_registry_presets_and_names():
     model = create_model(get_config("roluzen_tiny"), seed=3)
     assert model.config.runs() == [0, 1, 2, 1, 2]
     assert torch.equal(model.layers[0].hc1.mix, torch.eye(3)) and model.layers[1].mixer.right.f_proj.bias.eq(3).all()
+    assert registry.get_family("tovalix").family == "tovalix" and naming.config_for("tovalix-8b") == get_config("tovalix_8b")
+    assert naming.get_model_family("x/Tovalix-2B") == "tovalix"
+    small = create_model(get_config("tovalix_tiny"), seed=3)
+    assert small.config.kv_sources() == [0, 1, 2, 3, 4, 2] and small.layers[5].mixer.k_proj is None
+    assert small.num_params == get_config("tovalix_tiny").num_params()
     with pytest.raises(ValueError, match="loop"):
         get_config("roluzen_tiny").replace(loop=(2, 5, 1))
     with pytest.raises(NotImplementedError):
@@ -132,6 +175,56 @@ def test_joint_weights_share_memory_and_follow_updates():
     model.layers[1].mixer.left.q_proj.lora_a = torch.nn.Parameter(torch.zeros(1, 1))
     with pytest.raises(NotImplementedError, match="adapters"):
         ex.refresh()
+
+
+def test_joint_weights_of_memories_and_rotary_attention():
+    from tunix_b200.models.config import get_config
+    from tunix_b200.models.stack_exec import StackExecutor, rope_table
+    from tunix_b200.models.transformer import create_model
+    model = create_model(get_config("tovalix_tiny"), seed=0)
+    ex = StackExecutor(model)
+    before = {k: v.data_ptr() for d in ex.w for k, v in d.items() if v is not None}
+    with torch.no_grad():
+        model.layers[0].mixer.mu_g.fill_(0.125)
+        model.layers[2].mixer.v_proj.bias.fill_(3.0)
+        model.layers[1].mixer.v_proj.weight.fill_(2.0)
+    ex.refresh()
+    assert {k: v.data_ptr() for d in ex.w for k, v in d.items() if v is not None} == before
+    assert ex.w[0]["mu"][3].eq(0.125).all() and "proj" not in ex.w[0]
+    assert ex.w[2]["proj_bias"][-1] == 3.0 and ex.w[1]["proj"][-1].eq(2).all() and ex.w[1]["gates_bias"] is None
+    assert ex.w[5]["proj"].shape[0] == 4 * 32                           # queries only
+    cos, sin = rope_table(3000, 6, 900.0, "cpu")
+    a = 2999 * 900.0 ** (-4 / 6)
+    assert cos[0].eq(1).all() and abs(cos[2999, 2].item() - math.cos(a)) < 1e-7 and abs(sin[2999, 2].item() - math.sin(a)) < 1e-7
+
+
+def test_oracle_recurrences_against_their_unrolled_sums():
+    """The token-by-token memories of the second oracle against direct sums over all earlier tokens."""
+    torch.manual_seed(1)
+    T, H, d, dv = 20, 2, 5, 4
+    q, k, v = (torch.randn(T, H, n, dtype=torch.float64) for n in (d, d, dv))
+    f, u = torch.rand(T, H, d, dtype=torch.float64), torch.randn(H, d, dtype=torch.float64)
+    wkv, hgrn = TO.wkv_recurrence(q, k, v, f, u), TO.hgrn2_recurrence(q, f, v)
+    for t in range(T):
+        a, b = torch.zeros(H, dv).double(), torch.zeros(H, dv).double()
+        for s in range(t + 1):
+            after = f[s + 1:t].prod(0) if s < t else u                  # decays between the two tokens, or the bonus
+            a += (q[t] * after * k[s]).sum(-1, keepdim=True) * v[s]
+            b += (q[t] * f[s + 1:t + 1].prod(0) * (1 - f[s])).sum(-1, keepdim=True) * v[s]
+        assert torch.allclose(wkv[t], a) and torch.allclose(hgrn[t], b)
+
+
+def test_oracle_details():
+    x = torch.tensor([[3.0, 4.0, 0.0, 2.0]], dtype=torch.float64)
+    got = TO.group_norm(x, torch.tensor([1.0, 1.0, 1.0, 2.0]).double(), 2, 0.0)
+    assert torch.allclose(got, torch.tensor([[3 / 12.5 ** 0.5, 4 / 12.5 ** 0.5, 0.0, 2 * 2 ** 0.5]]).double())
+    z, p, q = torch.tensor([-1.0, 0.0, 2.0]).double(), torch.tensor(0.3).double(), torch.tensor(-0.7).double()
+    sp = lambda a: math.log(1 + math.exp(a))  # noqa: E731
+    want = [(0.5 + sp(-0.7)) * (math.exp(-1) - 1 + 1) - 0.5, 0.0, sp(0.3) * 4 + 1]
+    assert torch.allclose(TO.xielu(z, p, q), torch.tensor(want).double())
+    assert TO.visible(19, 0, 20) and not TO.visible(20, 19, 20) and not TO.visible(20, 21, 20)
+    h = torch.randn(5, 3).double()
+    assert torch.equal(TO.token_shift(h, torch.ones(3).double())[1:], h[:-1]) and TO.token_shift(h, torch.ones(3).double())[0].eq(0).all()
 
 
 def test_oracle_memory_against_its_unrolled_sum():

@@ -1,12 +1,11 @@
-"""Layer-stack models on the GPU against the plain oracle (tests/roluzen_oracle.py): whole prompts, portions, mixed batches,
+"""Layer-stack models on the GPU against the plain oracles (tests/roluzen_oracle.py, tovalix_oracle.py): whole prompts, portions, mixed batches,
 decoding, slots and pages that are used again, greedy generation through the engine. Mechanism tests are in
-test_stack_kernels_gpu.py."""
+test_stack_kernels_gpu.py and test_gated_linear_gpu.py."""
 import functools
 
 import pytest
 import torch
 
-from tests import roluzen_oracle as O
 from tests import stack_cases as C
 
 pytestmark = pytest.mark.gpu
@@ -47,7 +46,7 @@ def case(name, dtype, tmp=None):
 @functools.lru_cache(None)
 def oracle(name, toks):
     cfg, w = C.CASES[name], C.weights(C.CASES[name], seed=len(name))
-    return O.forward(cfg, w, list(toks))
+    return C.oracle(cfg).forward(cfg, w, list(toks))
 
 
 def engine(model, pages=16, slots=3, page=64, ctx=None, **kw):
@@ -69,9 +68,10 @@ def error(got, want):
 
 
 def close(got, want, dtype):
-    """All rows together within the tolerance, and no single row far off (a random model amplifies rounding at some)."""
+    """All rows together within the tolerance (if they are enough for an average), and no single row far off (a random model
+    amplifies rounding at some)."""
     print(f"rms {error(got, want):.2e}, worst row {worst_row(got, want):.2e}")
-    return error(got, want) < TOL[dtype] and worst_row(got, want) < 8 * TOL[dtype]
+    return (got.shape[0] < 4 or error(got, want) < TOL[dtype]) and worst_row(got, want) < 8 * TOL[dtype]
 
 
 def worst_row(got, want):
@@ -86,7 +86,7 @@ def test_whole_prompt_and_layers(name, dtype):
     from tunix_b200.ops.ragged import RaggedBatch
     cfg, w, model = case(name, dtype)
     toks = C.tokens(cfg, 150)
-    want, layers = O.forward(cfg, w, toks, want_layers=True)
+    want, layers = C.oracle(cfg).forward(cfg, w, toks, want_layers=True)
     pool = PagePool(model.config, 4, 64, 2, 4, "cuda", dtype, prefix_caching=False)
     pool.open(1, toks, 0)
     pool.sync_table()
@@ -122,7 +122,7 @@ def test_portions_and_decoding_agree_with_the_oracle(name, dtype):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("name", ["mixed", "wide"])
+@pytest.mark.parametrize("name", ["mixed", "wide", "shared", "tiles", "uneven"])
 def test_mixed_batches_and_reused_slots(name, dtype):
     """Unequal requests: portions beside decoded tokens, requests that sit out steps, ends in between; six requests share
     three slots and a pool that holds two of the longest, so that pages and slots change owners."""
@@ -157,9 +157,10 @@ def test_mixed_batches_and_reused_slots(name, dtype):
         assert close(torch.cat(got[i]), want, dtype), i
 
 
-def test_a_batch_equals_each_request_alone_in_bf16():
+@pytest.mark.parametrize("name", ["wide", "tiles"])
+def test_a_batch_equals_each_request_alone_in_bf16(name):
     """bf16 results do not depend on the company beyond rounding: compared with the single request, not with the oracle."""
-    cfg, _, model = case("wide", torch.bfloat16)
+    cfg, _, model = case(name, torch.bfloat16)
     seqs = [C.tokens(cfg, n, 30 + n) for n in (33, 190, 70)]
     ses = session(model, pages=8, slots=3)
     together = ses.step([(i, s, range(len(s))) for i, s in enumerate(seqs)])
@@ -174,11 +175,12 @@ def test_a_batch_equals_each_request_alone_in_bf16():
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-def test_long_decoding(dtype):
-    """Several hundred decoded tokens: states, rings and windows that have turned over many times."""
-    cfg, _, model = case("mixed", dtype)
+@pytest.mark.parametrize("name", ["mixed", "shared", "tiles"])
+def test_long_decoding(name, dtype):
+    """Several hundred decoded tokens: states, rings, windows and chunks that have turned over many times."""
+    cfg, _, model = case(name, dtype)
     toks = C.tokens(cfg, 460, 2)
-    want = oracle("mixed", tuple(toks))
+    want = oracle(name, tuple(toks))
     ses = session(model, pages=8, slots=2)
     ses.step([("r", toks[:30], [])])
     rows = [ses.step([("r", [t], [0])]) for t in toks[30:]]
@@ -205,7 +207,7 @@ def greedy_reference(name, prompt, steps):
     cfg, w = C.CASES[name], C.weights(C.CASES[name], seed=len(name))
     toks, margins = list(prompt), []
     for _ in range(steps):
-        z = O.forward(cfg, w, toks)[-1]
+        z = C.oracle(cfg).forward(cfg, w, toks)[-1]
         top = z.topk(2).values
         margins.append((top[0] - top[1]).item() / z.std().item())
         toks.append(int(z.argmax()))
@@ -213,17 +215,18 @@ def greedy_reference(name, prompt, steps):
 
 
 @pytest.mark.parametrize("graph", [True, False])
-def test_greedy_generation_matches_the_oracle(graph):
+@pytest.mark.parametrize("name", ["mixed", "shared", "uneven"])
+def test_greedy_generation_matches_the_oracle(name, graph):
     """Through the engine's entry point and scheduler in 32-bit: four prompts over two slots and a pool that forces
     pre-emption, decode step captured in a graph or not; logits of the oracle decide."""
-    cfg, _, model = case("mixed", torch.float32)
+    cfg, _, model = case(name, torch.float32)
     prompts = [C.tokens(cfg, n, 50 + n) for n in (14, 33, 20, 7)]
     steps = 12
     eng = engine(model, pages=5, slots=2, page=16, ctx=64, use_cuda_graph=graph, check_every=4)
     out = eng(prompt_token_ids=prompts, max_generation_steps=steps, max_prompt_length=40, temperature=0.0, eos_tokens=[-1],
               return_logprobs=True)
     for p, got, lps in zip(prompts, out.tokens, out.logprobs):
-        want, margins = greedy_reference("mixed", p, steps)
+        want, margins = greedy_reference(name, p, steps)
         for a, b, mg, lp in zip(got.tolist(), want, margins, lps):
             if a != b:
                 assert mg < 1e-3, (a, b, mg)
@@ -231,9 +234,10 @@ def test_greedy_generation_matches_the_oracle(graph):
             assert lp <= 0.0
 
 
-def test_generation_is_the_same_under_portions_preemption_and_graphs():
+@pytest.mark.parametrize("name", ["wide", "tiles"])
+def test_generation_is_the_same_under_portions_preemption_and_graphs(name):
     """bf16 and the tensor-core kernels: sampled tokens of one engine against engines with other schedules."""
-    cfg, _, model = case("wide", torch.bfloat16)
+    cfg, _, model = case(name, torch.bfloat16)
     prompts = [C.tokens(cfg, n, 70 + n) for n in (120, 3, 64, 65, 31)]
 
     def gen(**kw):
@@ -254,8 +258,9 @@ def test_generation_is_the_same_under_portions_preemption_and_graphs():
                 assert abs(la[k] - lb[k]) < 0.3, kw
 
 
-def test_stop_tokens_and_sampling_run_through_the_engine():
-    cfg, _, model = case("wide", torch.bfloat16)
+@pytest.mark.parametrize("name", ["wide", "tiles"])
+def test_stop_tokens_and_sampling_run_through_the_engine(name):
+    cfg, _, model = case(name, torch.bfloat16)
     eng = engine(model, pages=12, slots=4, ctx=192)
     prompts = [C.tokens(cfg, 9, 90 + i) for i in range(4)]
     kw = dict(prompt_token_ids=prompts, max_generation_steps=16, max_prompt_length=16, temperature=0.8, top_p=0.9, top_k=40, seed=5)
@@ -267,9 +272,10 @@ def test_stop_tokens_and_sampling_run_through_the_engine():
     assert c.tokens[0].tolist() == a.tokens[0].tolist()[:first + 1]
 
 
-def test_engine_server_serves_the_model():
+@pytest.mark.parametrize("name", ["wide", "tiles"])
+def test_engine_server_serves_the_model(name):
     from tunix_b200.generate.engine import EngineServer
-    cfg, _, model = case("wide", torch.bfloat16)
+    cfg, _, model = case(name, torch.bfloat16)
     prompts = [C.tokens(cfg, n, 120 + n) for n in (5, 40, 12)]
     with EngineServer(engine(model, pages=12, slots=2, ctx=192, check_every=4), max_new_tokens=8, max_prompt_length=64,
                       temperature=0.0, eos_tokens=[-1]) as srv:
@@ -281,30 +287,32 @@ def test_engine_server_serves_the_model():
     assert all(len(t) == 8 for t in first)
 
 
-def test_scoring_with_padding_matches_unpadded_rows():
-    cfg, _, model = case("wide", torch.float32)
+@pytest.mark.parametrize("name", ["wide", "tiles"])
+def test_scoring_with_padding_matches_unpadded_rows(name):
+    cfg, _, model = case(name, torch.float32)
     rows = [C.tokens(cfg, n, 140 + n) for n in (6, 19)]
     T = 24
     toks, seg = torch.zeros(2, T, dtype=torch.long), torch.zeros(2, T, dtype=torch.int32)
     toks[0, T - 6:], seg[0, T - 6:] = torch.tensor(rows[0]), 1          # left padding, as prompts have
     toks[1, :19], seg[1, :19] = torch.tensor(rows[1]), 1                # right padding, as completions have
     z, _ = model(toks, segment_ids=seg)
-    assert close(z[0, T - 6:], oracle("wide", tuple(rows[0])), torch.float32)
-    assert close(z[1, :19], oracle("wide", tuple(rows[1])), torch.float32)
+    assert close(z[0, T - 6:], oracle(name, tuple(rows[0])), torch.float32)
+    assert close(z[1, :19], oracle(name, tuple(rows[1])), torch.float32)
 
 
-def test_trace_runner_replays_steps(tmp_path):
+@pytest.mark.parametrize("name", ["mixed", "shared"])
+def test_trace_runner_replays_steps(name, tmp_path):
     import json
     import os
     import subprocess
     import sys
 
     import numpy as np
-    cfg = C.CASES["mixed"]
+    cfg = C.CASES[name]
     w = C.weights(cfg, seed=3)
     src = C.write(tmp_path / "model", cfg, w)
     toks = C.tokens(cfg, 70, 5)
-    want = O.forward(cfg, w, toks)
+    want = C.oracle(cfg).forward(cfg, w, toks)
     steps = [{"step": 0, "entries": [{"id": "a", "tokens": toks[:40], "want": [0, 39]}], "end": []},
              {"step": 1, "entries": [{"id": "a", "tokens": toks[40:41], "want": []}, {"id": "b", "tokens": toks[:9], "want": [8]}],
               "end": ["b"]},

@@ -1,4 +1,4 @@
-"""The layer-stack kernels one mechanism at a time against tests/roluzen_oracle.py: odd and even sizes, 32-bit and bf16, the
+"""The layer-stack kernels one mechanism at a time against tests/roluzen_oracle.py and tovalix_oracle.py: odd and even sizes, 32-bit and bf16, the
 simple and the tensor-core forms, and inputs in which one key stands out at a window's, a page's or the kept tokens' edge."""
 import math
 
@@ -6,6 +6,7 @@ import pytest
 import torch
 
 from tests import roluzen_oracle as O
+from tests import tovalix_oracle as TO
 
 pytestmark = pytest.mark.gpu
 DT = [torch.float32, torch.bfloat16]
@@ -79,6 +80,59 @@ def test_few_outputs(K, N):
     from tunix_b200.ops import stack_kernels as SK
     x, w = rand(5, K, dtype=torch.bfloat16), rand(N, K, dtype=torch.bfloat16, seed=1)
     assert rel(SK.few_outputs(x, w), x.double() @ w.double().T) < 1e-5
+
+
+@pytest.mark.parametrize("dtype", DT)
+@pytest.mark.parametrize("D,groups", [(48, 3), (36, 1), (37, 1), (1024, 4), (60, 15), (66, 6)])
+def test_stream_step_norm_groups_embedding_norm_and_normed_updates(D, groups, dtype):
+    from tunix_b200.ops import stack_kernels as SK
+    n, eps, tol = 5, 1e-2, 1e-6 if dtype == torch.float32 else 5e-3
+    one = torch.ones(1, device="cuda", dtype=dtype)
+    embed, nw, ew, wy, y = (rand(*s, dtype=dtype, std=t, seed=i) for i, (s, t) in enumerate([((20, D), 0.1), ((D,), 1), ((D,), 1), ((D,), 1), ((n, D), 0.1)]))
+    embed[:, : D // groups] *= 9                            # groups of unequal size
+    toks = torch.tensor([3, 0, 19, 7, 7], device="cuda")
+    d = lambda t: t.double().cpu()  # noqa: E731
+    x = torch.empty(n, 1, D, device="cuda")
+    h = SK.stream_step(x, eps, tokens=toks, embed=embed, embed_w=ew, groups=groups, w_in=one, norm_w=nw)
+    ref = TO.group_norm(d(embed)[toks.cpu()], d(ew), groups, eps)
+    assert rel(x[:, 0], ref) < 1e-6 and rel(h, TO.group_norm(ref, d(nw), groups, eps)) < tol
+    h = SK.stream_step(x, eps, y=y, wy=wy, mix=one, w_out=one, w_in=one, norm_w=nw, groups=groups)    # the update has a plain norm
+    ref = ref + TO.rms(d(y), eps) * d(wy)
+    assert rel(x[:, 0], ref) < 1e-6 and rel(h, TO.group_norm(ref, d(nw), groups, eps)) < tol
+    h = SK.stream_step(x, eps, y=y, mix=one, w_out=one, raw=True, groups=groups)
+    ref = ref + d(y)
+    assert rel(x[:, 0], ref) < 1e-6 and rel(h, ref) < tol
+
+
+@pytest.mark.parametrize("dtype", DT)
+@pytest.mark.parametrize("rows,F", [(3, 8), (5, 31), (64, 500)])
+@pytest.mark.parametrize("p,q", [(0.5, -1.25), (-3.0, 4.0), (6.0, 0.0)])
+def test_xielu(rows, F, p, q, dtype):
+    from tunix_b200.ops import stack_kernels as SK
+    z = rand(rows, F, dtype=dtype, std=3)
+    z.view(-1)[:4] = torch.tensor([0.0, -1e-3, -60.0, 1e-3], device="cuda")
+    act = torch.tensor([p, q], device="cuda", dtype=dtype)
+    want = TO.xielu(z.double().cpu(), torch.tensor(p).double(), torch.tensor(q).double())
+    got = SK.xielu_(z.clone(), act)
+    assert rel(got, want) < (1e-6 if dtype == torch.float32 else 5e-3)
+    assert torch.allclose(got.view(-1)[:4].double().cpu(), want.view(-1)[:4], rtol=1e-6 if dtype == torch.float32 else 5e-3, atol=1e-7)
+
+
+@pytest.mark.parametrize("dtype", DT)
+@pytest.mark.parametrize("K,N", [(40, 3), (64, 16), (256, 70)])
+def test_few_outputs_with_their_activations(K, N, dtype):
+    """tanh, and gelu times the token's own columns of a table; the narrow product and the two-step form."""
+    from tunix_b200.ops import stack_kernels as SK
+    x, w, rows = rand(5, K, dtype=dtype), rand(N, K, dtype=dtype, std=0.3, seed=1), rand(11, N + 9, dtype=dtype, seed=2)
+    toks = torch.tensor([10, 0, 3, 3, 7], device="cuda")
+    z = x.double().cpu() @ w.double().cpu().T
+    e = rows.double().cpu()[toks.cpu(), 4:4 + N]
+    kw = dict(tokens=toks, rows=rows, col=4)
+    for act, want, args in ((SK.ACT_TANH, torch.tanh(z), {}), (SK.ACT_GELU_ROW, TO.gelu_tanh(z) * e, kw)):
+        t = 2e-6 if dtype == torch.float32 else 5e-3
+        assert rel(SK.small_act(z.float().cuda(), dtype, act, **args), want) < t
+        if dtype == torch.bfloat16:
+            assert rel(SK.few_outputs(x, w, act, **args), want) < t
 
 
 # ------------------------------------------------------------------------------------------------ gated recurrence

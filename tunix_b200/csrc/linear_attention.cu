@@ -51,12 +51,16 @@ __device__ __forceinline__ void gates_exact(float z, float c0, float c1, float& 
     f = k < 0.5f ? 1.f - k : c1 + (1.f - c1) * sigmoid(z + c0);
   }
 }
-// log f for bf16 models; bounded, so that sums of it stay finite
+// log2 f for bf16 models; bounded, so that sums of it stay finite. b0 = gates_offset(c0)
 template <int MODE>
-__device__ __forceinline__ float gates_log(float z, float c0, float c1, float& k) {
-  if (MODE == BONUS) return -fminf(quick_exp(z + c0), 1e4f);
-  k = (1.f - c1) * quick_sigmoid(-(z + c0));
-  return k < 0.5f ? log1pf(-k) : logf(fmaxf(c1 + (1.f - c1) * quick_sigmoid(z + c0), 1e-30f));
+__device__ __forceinline__ float gates_offset(float c0) { return c0 * LOG2_E + (MODE == BONUS ? 0.5287663729448977f : 0.f); }   // + log2(log2 e)
+template <int MODE>
+__device__ __forceinline__ float gates_log2(float z, float b0, float c1, float& k) {
+  const float e = quick_exp2(fminf(fmaf(z, LOG2_E, b0), 100.f));
+  if (MODE == BONUS) return -fminf(e, 1e4f);
+  const float s = quick_rcp(1.f + e), r = 1.f - c1;    // sigmoid of the negative; e s: of the positive
+  k = r * s;
+  return quick_log2_decay(k, fmaf(r, e * s, c1));
 }
 
 template <typename T>
@@ -264,54 +268,56 @@ head_norm_kernel(const GlaArgs a, const float* __restrict__ o, T* __restrict__ o
 }
 
 // ------------------------------------------------------------------------------------------------ portions, tensor cores
-// A CTA owns 64 value columns of one head, 16 per warp, and walks its entry in blocks of 16 tokens. With L_t the sum of log f
-// from the block's start through token t and L its end,
-//   o_t = (q_t e^(L_t)) S + sum_{s <= t} (q_t e^(L_t) . k_s e^(-L_s)) v_s,    S' = diag(e^L) S + sum_s (k_s e^(L - L_s)) v_s^T
+// A CTA owns 64 or 128 value columns of one head, 16 per warp, and walks its entry in blocks of 16 tokens. With L_t the sum of log f (in the code: of log2 f)
+// from the block's start through token t, m its value at the block's middle and L at its end,
+//   o_t = (q_t e^(L_t - m)) (diag(e^m) S) + sum_{s <= t} (q_t e^(L_t - m) . k_s e^(m - L_s)) v_s,
+//   S' = diag(e^(L - m)) diag(e^m) S + sum_s (k_s e^(L - L_s)) v_s^T
 // (BONUS reads S before the token: L_(t-1), s < t, and the current token weighs q . (c1 k)).
 // S^T stays in fp32 accumulators [16 values, dk]: their layout is that of the B operand of q S, so the state is packed to bf16
 // for the read-out without leaving registers. The updates k e^(L - L_s) go to the tensor cores as bf16 pairs hi + lo, v is
 // bf16 and exact. Several blocks are prepared at once (TT tokens); every warp prepares one block (half of its channels at
 // dk > 64), so a tile of tokens costs two barriers.
-// e^(-L_s) must stay finite: where some channel decays by more than e^-SAFE within a block, the tile's weights are summed
-// directly, with e^(L_t - L_s) per pair and channel.
-constexpr int DV = 64;
-constexpr float SAFE = 60.f;
-constexpr int VPITCH = DV * 2 + 16;
+// The factors around m must stay finite: where some channel decays by more than e^-SAFE within half a block, the tile takes
+// m = 0 and sums its weights directly, with e^(L_t - L_s) per pair and channel.
+constexpr float SAFE = 70.f * LOG2_E;
 constexpr int PPITCH = 48;
 
 struct ChunkSmem {
-  int tt, pitch, q, k, z, v, Q, Ki, Kh, Kl, P, D, dg, ssq, total;
+  int tt, pitch, vpitch, q, k, z, v, Q, Ki, Kh, Kl, P, D, E, dg, ssq, total;
 };
-__host__ __device__ constexpr ChunkSmem chunk_smem(int KP) {
+__host__ __device__ constexpr ChunkSmem chunk_smem(int KP, int warps) {
   ChunkSmem L{};
-  L.tt = 4096 / KP;
+  L.tt = 16 * warps * 64 / KP;
   L.pitch = KP * 2 + 16;
+  L.vpitch = 16 * warps * 2 + 16;
   L.q = 0;
   L.k = L.q + L.tt * L.pitch;
   L.z = L.k + L.tt * L.pitch;
   L.v = L.z + L.tt * KP * 4;
-  L.Q = L.v + 2 * L.tt * VPITCH;
+  L.Q = L.v + 2 * L.tt * L.vpitch;
   L.Ki = L.Q + L.tt * L.pitch;
   L.Kh = L.Ki + L.tt * L.pitch;
   L.Kl = L.Kh + L.tt * L.pitch;
   L.P = L.Kl + L.tt * L.pitch;
   L.D = L.P + (L.tt / 16) * 16 * PPITCH;
-  L.dg = L.D + (L.tt / 16) * KP * 4;
+  L.E = L.D + (L.tt / 16) * KP * 4;
+  L.dg = L.E + (L.tt / 16) * KP * 4;
   L.ssq = L.dg + (KP / 64) * L.tt * 4;
-  L.total = L.ssq + 4 * L.tt * 4;
+  L.total = L.ssq + warps * L.tt * 4;
   return L;
 }
 
-template <int KP, int MODE>
-__global__ void __launch_bounds__(128)
+template <int KP, int MODE, int WARPS>
+__global__ void __launch_bounds__(32 * WARPS)
 gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out) {
   extern __shared__ __align__(16) uint8_t smem[];
-  constexpr ChunkSmem M = chunk_smem(KP);
-  constexpr int TT = M.tt, SUBS = TT / 16, HALVES = KP / 64, KT = KP / 8;
+  constexpr ChunkSmem M = chunk_smem(KP, WARPS);
+  constexpr int TT = M.tt, SUBS = TT / 16, HALVES = KP / 64, KT = KP / 8, DV = 16 * WARPS, NT = 32 * WARPS, VPITCH = M.vpitch;
   const uint32_t sb = smem_u32(smem);
-  float* Dd = reinterpret_cast<float*>(smem + M.D);     // [SUBS][KP] e^L
+  float* Dd = reinterpret_cast<float*>(smem + M.D);     // [SUBS][KP] e^(L - m)
+  float* De = reinterpret_cast<float*>(smem + M.E);     // [SUBS][KP] e^m
   float* Dg = reinterpret_cast<float*>(smem + M.dg);    // [HALVES][TT] q . (c1 k)
-  float* Ssq = reinterpret_cast<float*>(smem + M.ssq);  // [4][TT]
+  float* Ssq = reinterpret_cast<float*>(smem + M.ssq);  // [WARPS][TT]
   const float* Z = reinterpret_cast<const float*>(smem + M.z);
   pdl_trigger();
   pdl_wait();
@@ -329,21 +335,28 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
   const bf* kg = MODE == BONUS ? static_cast<const bf*>(a.k) + (long long)t0 * a.ldk + hd * dk : nullptr;
   const bf* vg = static_cast<const bf*>(a.v) + (long long)t0 * a.ldv + hd * dv + c0;
   const float* zg = a.z + (long long)t0 * a.ldz + hd * dk;
+  const bf* gg = a.gate ? static_cast<const bf*>(a.gate) + (long long)t0 * a.ldg + hd * dv + c0 : nullptr;
+  uint32_t nw[2];                       // norm weights of this lane's columns
+#pragma unroll
+  for (int j = 0; j < 2; ++j) {
+    const int c = c0 + v0 + j * 8 + 2 * (lane & 3);
+    nw[j] = c < dv ? *reinterpret_cast<const uint32_t*>(static_cast<const bf*>(a.nw) + (a.per_head ? hd * dv + c : c)) : 0u;
+  }
   auto load = [&](int tile) {
     const int at = tile * TT, rows = min(TT, len - at);
-    for (int i = tid; i < TT * (KP / 8); i += 128) {
+    for (int i = tid; i < TT * (KP / 8); i += NT) {
       const int r = i / (KP / 8), c = i % (KP / 8);
       const bool ok = r < rows && c * 8 < dk;
       cp_async16(sb + M.q + r * M.pitch + c * 16, qg + (ok ? (at + r) * a.ldq + c * 8 : 0), ok ? 16 : 0);
       if (MODE == BONUS) cp_async16(sb + M.k + r * M.pitch + c * 16, kg + (ok ? (at + r) * a.ldk + c * 8 : 0), ok ? 16 : 0);
     }
-    for (int i = tid; i < TT * (KP / 4); i += 128) {
+    for (int i = tid; i < TT * (KP / 4); i += NT) {
       const int r = i / (KP / 4), c = i % (KP / 4);
       const bool ok = r < rows && c * 4 < dk;
       cp_async16(sb + M.z + r * (KP * 4) + c * 16, zg + (ok ? (at + r) * a.ldz + c * 4 : 0), ok ? 16 : 0);
     }
     const uint32_t vb = sb + M.v + (tile & 1) * TT * VPITCH;
-    for (int i = tid; i < TT * (DV / 8); i += 128) {
+    for (int i = tid; i < TT * (DV / 8); i += NT) {
       const int r = i / (DV / 8), c = i % (DV / 8);
       const bool ok = r < rows && c * 8 < nc;
       cp_async16(vb + r * VPITCH + c * 16, vg + (ok ? (at + r) * a.ldv + c * 8 : 0), ok ? 16 : 0);
@@ -368,7 +381,7 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     const bool ok = pd + i < dk;
-    b0[i] = ok ? to_f(static_cast<const bf*>(a.c0)[hd * dk + pd + i]) : 0.f;
+    b0[i] = gates_offset<MODE>(ok ? to_f(static_cast<const bf*>(a.c0)[hd * dk + pd + i]) : 0.f);
     b1[i] = ok ? to_f(static_cast<const bf*>(a.c1)[hd * dk + pd + i]) : (MODE == LOWER ? 1.f : 0.f);
   }
 
@@ -384,7 +397,7 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
       for (int t = 0; t < 16; ++t) {
         const int row = psub * 16 + t;
         const float2 z = *reinterpret_cast<const float2*>(Z + row * KP + pd);
-        float l0 = gates_log<MODE>(z.x, b0[0], b1[0], kk[t][0]), l1 = gates_log<MODE>(z.y, b0[1], b1[1], kk[t][1]);
+        float l0 = gates_log2<MODE>(z.x, b0[0], b1[0], kk[t][0]), l1 = gates_log2<MODE>(z.y, b0[1], b1[1], kk[t][1]);
         if (MODE == BONUS) {
           const uint32_t k2 = *reinterpret_cast<const uint32_t*>(smem + M.k + row * M.pitch + pd * 2);
           kk[t][0] = bf16_lo(k2);
@@ -398,6 +411,9 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
       }
     }
     const float e0 = L[15][0], e1 = L[15][1];
+    float m0 = L[7][0], m1 = L[7][1];
+    const bool direct = __syncthreads_or(fminf(fminf(m0, e0 - m0), fminf(m1, e1 - m1)) < -SAFE);
+    if (direct) m0 = m1 = 0.f;
     float dg[16];
 #pragma unroll
     for (int t = 0; t < 16; ++t) {
@@ -407,27 +423,33 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
       float q0 = bf16_lo(q2), q1 = bf16_hi(q2);
       if (MODE == LOWER) { q0 = silu<bf>(q0); q1 = silu<bf>(q1); }
       else dg[t] = q0 * b1[0] * kk[t][0] + q1 * b1[1] * kk[t][1];
-      float x0, x1;                     // decay from the block's start to the read-out
-      if (MODE == LOWER) { x0 = quick_exp(L[t][0]); x1 = quick_exp(L[t][1]); }
-      else if (t == 0) x0 = x1 = 1.f;
-      else { x0 = quick_exp(L[t > 0 ? t - 1 : 0][0]); x1 = quick_exp(L[t > 0 ? t - 1 : 0][1]); }
-      *reinterpret_cast<uint32_t*>(smem + M.Q + at) = pack_bf16(q0 * x0, q1 * x1);
-      *reinterpret_cast<uint32_t*>(smem + M.Ki + at) = pack_bf16(kk[t][0] * quick_exp(fminf(-L[t][0], SAFE)), kk[t][1] * quick_exp(fminf(-L[t][1], SAFE)));
+      const int tr = MODE == LOWER ? t : t - 1;         // the last token whose decay the read-out has seen
+      const float r0 = tr >= 0 ? L[tr < 0 ? 0 : tr][0] : 0.f, r1 = tr >= 0 ? L[tr < 0 ? 0 : tr][1] : 0.f;
+      *reinterpret_cast<uint32_t*>(smem + M.Q + at) = pack_bf16(q0 * quick_exp2(r0 - m0), q1 * quick_exp2(r1 - m1));
+      if (!direct)
+        *reinterpret_cast<uint32_t*>(smem + M.Ki + at) = pack_bf16(kk[t][0] * quick_exp2(m0 - L[t][0]), kk[t][1] * quick_exp2(m1 - L[t][1]));
       bf h0, h1, l0, l1;
-      split_bf16(kk[t][0] * quick_exp(e0 - L[t][0]), h0, l0);
-      split_bf16(kk[t][1] * quick_exp(e1 - L[t][1]), h1, l1);
+      split_bf16(kk[t][0] * quick_exp2(e0 - L[t][0]), h0, l0);
+      split_bf16(kk[t][1] * quick_exp2(e1 - L[t][1]), h1, l1);
       *reinterpret_cast<__nv_bfloat162*>(smem + M.Kh + at) = __halves2bfloat162(h0, h1);
       *reinterpret_cast<__nv_bfloat162*>(smem + M.Kl + at) = __halves2bfloat162(l0, l1);
     }
-    *reinterpret_cast<float2*>(Dd + psub * KP + pd) = make_float2(quick_exp(e0), quick_exp(e1));
+    *reinterpret_cast<float2*>(De + psub * KP + pd) = make_float2(quick_exp2(m0), quick_exp2(m1));
+    *reinterpret_cast<float2*>(Dd + psub * KP + pd) = make_float2(quick_exp2(e0 - m0), quick_exp2(e1 - m1));
     if (MODE == BONUS) {
+      // 16 sums over the warp: halve the values a lane holds at every step
 #pragma unroll
-      for (int t = 0; t < 16; ++t) {
-        const float s = warp_sum(dg[t]);
-        if (lane == 0) Dg[(warp % HALVES) * TT + psub * 16 + t] = s;
+      for (int w = 8; w >= 1; w >>= 1) {
+#pragma unroll
+        for (int t = 0; t < w; ++t) {
+          const float mine = (lane & w) ? dg[t + w] : dg[t], other = (lane & w) ? dg[t] : dg[t + w];
+          dg[t] = mine + __shfl_xor_sync(0xffffffffu, other, w);
+        }
       }
+      dg[0] += __shfl_xor_sync(0xffffffffu, dg[0], 16);
+      if (lane < 16) Dg[(warp % HALVES) * TT + psub * 16 + lane] = dg[0];
     }
-    const bool direct = __syncthreads_or(fminf(e0, e1) < -SAFE);
+    __syncthreads();
     if (direct) {
       // L, q and k of the whole tile go to shared memory, then one thread per weight
 #pragma unroll
@@ -442,7 +464,7 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
         }
       }
       __syncthreads();
-      for (int i = tid; i < SUBS * 256; i += 128) {
+      for (int i = tid; i < SUBS * 256; i += NT) {
         const int sub = i >> 8, t = (i >> 4) & 15, s = i & 15, rt = sub * 16 + t, rs = sub * 16 + s;
         float p = 0.f;
         if (MODE == BONUS && s == t) {
@@ -452,7 +474,7 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
           const bf* q = reinterpret_cast<const bf*>(smem + M.q + rt * M.pitch);
           const bf* k = reinterpret_cast<const bf*>(smem + M.k + rs * M.pitch);
           const float *Lt = Z + (MODE == BONUS ? rt - 1 : rt) * KP, *Ls = Z + rs * KP;
-          for (int d = 0; d < dk; ++d) p += to_f(q[d]) * to_f(k[d]) * quick_exp(Lt[d] - Ls[d]);
+          for (int d = 0; d < dk; ++d) p += to_f(q[d]) * to_f(k[d]) * quick_exp2(Lt[d] - Ls[d]);
         }
         *reinterpret_cast<bf*>(smem + M.P + (sub * 16 + t) * PPITCH + s * 2) = __float2bfloat16(p);
       }
@@ -460,6 +482,19 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
     }
     if (tile + 1 < tiles) load(tile + 1);
 
+    // the gates of this lane's outputs, on their way while the products run
+    uint32_t gate[SUBS][2][2];
+    if (active && out != nullptr && a.gate) {
+#pragma unroll
+      for (int sub = 0; sub < SUBS; ++sub)
+#pragma unroll
+        for (int h = 0; h < 2; ++h)
+#pragma unroll
+          for (int j = 0; j < 2; ++j) {
+            const int r = sub * 16 + g + h * 8, c = v0 + j * 8 + qd;
+            gate[sub][h][j] = r < rows && c < nc ? __ldg(reinterpret_cast<const uint32_t*>(gg + (tile * TT + r) * a.ldg + c)) : 0u;
+          }
+    }
     float O[SUBS][2][4];
     const uint32_t vb = sb + M.v + (tile & 1) * TT * VPITCH;
     if (active) {
@@ -475,11 +510,18 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
         for (int ks = 0; ks < KP / 16; ++ks) {
           uint32_t q[4], k[4];
           ldsm_x4(q, sb + M.Q + r_nt * M.pitch + (ks * 2 + (li >> 1)) * 16);
-          ldsm_x4(k, sb + M.Ki + r_b * M.pitch + (ks * 2 + (li & 1)) * 16);
-          mma_16816(P[0], q, k[0], k[1]);
-          mma_16816(P[1], q, k[2], k[3]);
-          mma_16816(O[sub][0], q, pack_bf16(S[2 * ks][0], S[2 * ks][1]), pack_bf16(S[2 * ks + 1][0], S[2 * ks + 1][1]));
-          mma_16816(O[sub][1], q, pack_bf16(S[2 * ks][2], S[2 * ks][3]), pack_bf16(S[2 * ks + 1][2], S[2 * ks + 1][3]));
+          if (!direct) {
+            ldsm_x4(k, sb + M.Ki + r_b * M.pitch + (ks * 2 + (li & 1)) * 16);
+            mma_16816(P[0], q, k[0], k[1]);
+            mma_16816(P[1], q, k[2], k[3]);
+          }
+          const float2 f0 = *reinterpret_cast<const float2*>(De + sub * KP + ks * 16 + qd);
+          const float2 f1 = *reinterpret_cast<const float2*>(De + sub * KP + ks * 16 + 8 + qd);
+          float (&s0)[4] = S[2 * ks], (&s1)[4] = S[2 * ks + 1];
+          s0[0] *= f0.x; s0[1] *= f0.y; s0[2] *= f0.x; s0[3] *= f0.y;
+          s1[0] *= f1.x; s1[1] *= f1.y; s1[2] *= f1.x; s1[3] *= f1.y;
+          mma_16816(O[sub][0], q, pack_bf16(s0[0], s0[1]), pack_bf16(s1[0], s1[1]));
+          mma_16816(O[sub][1], q, pack_bf16(s0[2], s0[3]), pack_bf16(s1[2], s1[3]));
         }
         uint32_t ap[4], bv[4], av[4];
         if (direct) {
@@ -547,7 +589,12 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
           if (r >= rows) continue;
           const long long t = t0 + tile * TT + r;
           float rstd = 1.f;
-          if (out != nullptr) rstd = 1.f / sqrtf((Ssq[r] + Ssq[TT + r] + Ssq[2 * TT + r] + Ssq[3 * TT + r]) / (float)dv + a.eps);
+          if (out != nullptr) {
+            float s = 0.f;
+#pragma unroll
+            for (int w = 0; w < WARPS; ++w) s += Ssq[w * TT + r];
+            rstd = rsqrtf(s / (float)dv + a.eps);
+          }
 #pragma unroll
           for (int j = 0; j < 2; ++j) {
             const int c = c0 + v0 + j * 8 + qd;
@@ -556,12 +603,10 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
             if (out == nullptr) {
               *reinterpret_cast<float2*>(raw + (t * a.heads + hd) * dv + c) = make_float2(x0, x1);
             } else {
-              const uint32_t w2 = *reinterpret_cast<const uint32_t*>(static_cast<const bf*>(a.nw) + (a.per_head ? hd * dv + c : c));
-              float y0 = x0 * rstd * bf16_lo(w2), y1 = x1 * rstd * bf16_hi(w2);
+              float y0 = x0 * rstd * bf16_lo(nw[j]), y1 = x1 * rstd * bf16_hi(nw[j]);
               if (a.gate) {
-                const uint32_t g2 = *reinterpret_cast<const uint32_t*>(static_cast<const bf*>(a.gate) + t * a.ldg + hd * dv + c);
-                y0 *= silu<bf>(bf16_lo(g2));
-                y1 *= silu<bf>(bf16_hi(g2));
+                y0 *= silu<bf>(bf16_lo(gate[sub][h][j]));
+                y1 *= silu<bf>(bf16_hi(gate[sub][h][j]));
               }
               *reinterpret_cast<uint32_t*>(out + t * a.heads * dv + hd * dv + c) = pack_bf16(y0, y1);
             }
@@ -579,14 +624,15 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
   carry_rows<bf>(a, t0 + len - 1, slot, hd * gridDim.x + sl, gridDim.x * gridDim.y);
 }
 
-template <int KP, int MODE>
+template <int KP, int MODE, int WARPS>
 int launch_chunk(const GlaArgs& a, float* raw, bf* out, cudaStream_t stream) {
-  constexpr int smem = chunk_smem(KP).total;
+  constexpr int smem = chunk_smem(KP, WARPS).total, DV = 16 * WARPS;
+  bf* o = a.dv <= DV ? out : nullptr;
   static DeviceOnce once;
   if (once.first() &&
-      cudaFuncSetAttribute(gla_chunk_kernel<KP, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -5;
+      cudaFuncSetAttribute(gla_chunk_kernel<KP, MODE, WARPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -5;
   const dim3 grid((a.dv + DV - 1) / DV, a.heads, a.rb.E);
-  return launch_pdl(gla_chunk_kernel<KP, MODE>, grid, dim3(128), smem, stream, a, raw, out) == cudaSuccess ? 0 : -5;
+  return launch_pdl(gla_chunk_kernel<KP, MODE, WARPS>, grid, dim3(32 * WARPS), smem, stream, a, raw, o) == cudaSuccess ? 0 : -5;
 }
 
 template <typename T, int MODE, int V>
@@ -607,19 +653,18 @@ int run(const GlaArgs& a, float* raw, T* out, int one, int chunked, cudaStream_t
     if (vec && a.dv <= 4 * GT) return launch_step<T, MODE, 4>(a, out, stream);
     if (a.dv <= GT) return launch_step<T, MODE, 1>(a, out, stream);
   }
-  bool normed = false;
+  bool sliced = false;
   if constexpr (sizeof(T) == 2) {
     if (chunked && !one && a.dk <= 128 && a.dk % 8 == 0 && a.dv % 8 == 0 && a.ldq % 8 == 0 && a.ldv % 8 == 0 && a.ldz % 4 == 0 &&
         (MODE == LOWER || a.ldk % 8 == 0) && a.ldg % 2 == 0) {
-      normed = a.dv <= DV;
-      bf* o = normed ? out : nullptr;
-      const int rc = a.dk <= 64 ? launch_chunk<64, MODE>(a, raw, o, stream) : launch_chunk<128, MODE>(a, raw, o, stream);
-      if (rc) return rc;
-      if (normed) return 0;
-      chunked = 2;
+      const bool wide = a.dv > 64;
+      const int rc = a.dk <= 64 ? (wide ? launch_chunk<64, MODE, 8>(a, raw, out, stream) : launch_chunk<64, MODE, 4>(a, raw, out, stream))
+                                : (wide ? launch_chunk<128, MODE, 8>(a, raw, out, stream) : launch_chunk<128, MODE, 4>(a, raw, out, stream));
+      if (rc || a.dv <= 128) return rc;
+      sliced = true;
     }
   }
-  if (chunked != 2) {
+  if (!sliced) {
     const size_t smem = ((size_t)a.dk * (SV + 4) + SV + (GT / 32) * SV) * 4;
     static DeviceOnce once;
     if (smem > 220 * 1024) return -2;

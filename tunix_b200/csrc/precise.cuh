@@ -78,15 +78,29 @@ __device__ __forceinline__ void store_v(__nv_bfloat16* p, const float (&v)[V]) {
 // The same functions for kernels that only bf16 models run: hardware exponential and division (relative error of a few
 // units in the last place), which is far below the rounding of their bf16 inputs and outputs. quick_expm1 keeps its relative
 // accuracy near zero (Taylor series there), as the decays of a recurrence need it.
-__device__ __forceinline__ float quick_exp(float z) {
+constexpr float LOG2_E = 1.4426950408889634f;
+__device__ __forceinline__ float quick_exp2(float z) {
   float r;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(z * 1.4426950408889634f));
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(z));
   return r;
 }
-__device__ __forceinline__ float quick_sigmoid(float z) {
+__device__ __forceinline__ float quick_log2(float z) {
   float r;
-  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + quick_exp(-z)));
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(z));
   return r;
+}
+__device__ __forceinline__ float quick_rcp(float z) {
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(z));
+  return r;
+}
+__device__ __forceinline__ float quick_exp(float z) { return quick_exp2(z * LOG2_E); }
+__device__ __forceinline__ float quick_sigmoid(float z) { return quick_rcp(1.f + quick_exp(-z)); }
+// log2(1 - k) for 0 <= k < 1, f = 1 - k: relative accuracy near k = 0 by -2 atanh(k / (2 - k)), whose series is short there
+__device__ __forceinline__ float quick_log2_decay(float k, float f) {
+  const float s = k * quick_rcp(2.f - k), s2 = s * s;
+  const float series = s * fmaf(s2, fmaf(s2, fmaf(s2, fmaf(s2, 1.f / 9.f, 1.f / 7.f), 0.2f), 1.f / 3.f), 1.f);
+  return k < 0.5f ? -2.f * LOG2_E * series : quick_log2(fmaxf(f, 1e-30f));
 }
 __device__ __forceinline__ float quick_expm1(float z) {
   const float t = z * fmaf(z, fmaf(z, fmaf(z, fmaf(z, fmaf(z, fmaf(z, 1.f / 5040.f, 1.f / 720.f), 1.f / 120.f), 1.f / 24.f), 1.f / 6.f), 0.5f), 1.f);

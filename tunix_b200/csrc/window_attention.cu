@@ -79,6 +79,68 @@ qk_norm_write_kernel(const T* __restrict__ proj, long long ldp, int q_off, int k
   }
 }
 
+// Heads of a multiple of 8 dimensions that turn by a multiple of 16: LPH lanes per head, 8 elements per lane; the partner of a
+// rotation sits rd / 16 lanes away. Otherwise like rope_norm_write_kernel.
+template <int LPH>
+__global__ void __launch_bounds__(256)
+rope_norm_write_vec_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int q_off, int k_off, int v_off,
+                           const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rd, float eps, Ragged rb, Paged pg,
+                           int H, int G, int dq, int dv, __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ kp,
+                           __nv_bfloat16* __restrict__ vp) {
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x, lane = threadIdx.x & 31, sub = threadIdx.x % LPH, e = rb.ent[t], p0 = rb.pos0[e];
+  const int heads = H + 2 * G, base = lane - sub, half8 = rd >> 4;
+  const __nv_bfloat16* row = proj + (long long)t * ldp;
+  const int p = p0 + t - rb.cu[e];
+  long long pr = 0;
+  if (p0 >= 0 && G > 0) pr = page_row(pg, pg.table + (long long)rb.slot[e] * pg.max_pages, p);
+  const bool turns = sub < 2 * half8 && p0 >= 0;
+  const int partner = turns ? (sub < half8 ? sub + half8 : sub - half8) : sub;
+  float c[8], s[8];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) { c[i] = 1.f; s[i] = 0.f; }
+  if (turns) {
+    const long long at = (long long)p * (rd >> 1) + (sub < half8 ? sub : sub - half8) * 8;
+    load_v<8>(cos_t + at, c);
+    load_v<8>(sin_t + at, s);
+    if (sub < half8) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) s[i] = -s[i];
+    }
+  }
+  for (int h0 = 0; h0 < heads; h0 += 256 / LPH) {       // whole warps stay together for the shuffles
+    const int hh = h0 + threadIdx.x / LPH;
+    const bool is_v = hh >= H + G, ok = hh < heads && sub * 8 < (is_v ? dv : dq) && p0 >= 0;
+    float v[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] = 0.f;
+    if (ok) load_v<8>(row + (hh < H ? q_off + hh * dq : is_v ? v_off + (hh - H - G) * dv : k_off + (hh - H) * dq) + sub * 8, v);
+    float o[8], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      o[i] = v[i] * c[i] + __shfl_sync(0xffffffffu, v[i], base + partner) * s[i];
+      ss += o[i] * o[i];
+    }
+#pragma unroll
+    for (int w = LPH / 2; w >= 1; w >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, w);
+    const float r = 1.f / sqrtf(ss / (float)dq + eps);
+    if (hh < H) {
+      if (sub * 8 < dq) {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) o[i] *= r;
+        store_v<8>(q + ((long long)t * H + hh) * dq + sub * 8, o);
+      }
+    } else if (ok && !is_v) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) o[i] *= r;
+      store_v<8>(kp + (pr * G + hh - H) * dq + sub * 8, o);
+    } else if (ok) {
+      store_v<8>(vp + (pr * G + hh - H - G) * dv + sub * 8, v);
+    }
+  }
+}
+
 // One warp per (token, head) over the query heads, then key heads, then value heads of a row. cos / sin [positions, rd / 2].
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -238,6 +300,16 @@ TB_API int tb_rope_norm_write(int dtype, const void* proj, long long ldp, int q_
   if (rd < 0 || rd % 2 || rd > dq) return -2;
   RAGGED;
   PAGED;
+  const int wide = dq > dv ? dq : dv;
+  if (dtype == 0 && dq % 8 == 0 && dv % 8 == 0 && rd % 16 == 0 && wide <= 256 && ldp % 8 == 0 && q_off % 8 == 0 && k_off % 8 == 0 &&
+      v_off % 8 == 0) {
+    typedef __nv_bfloat16 bf;
+#define VEC(L)                                                                                                              \
+  launch_pdl(rope_norm_write_vec_kernel<L>, dim3(n), dim3(256), 0, stream, (const bf*)proj, ldp, q_off, k_off, v_off, cos_t,  \
+             sin_t, rd, eps, rb, pg, H, G, dq, dv, (bf*)q, (bf*)kp, (bf*)vp)
+    return (wide <= 64 ? VEC(8) : wide <= 128 ? VEC(16) : VEC(32)) == cudaSuccess ? 0 : -5;
+#undef VEC
+  }
   const long long warps = (long long)n * (H + 2 * G);
   const dim3 grid((unsigned)((warps + 7) / 8));
 #define RUN(T)                                                                                                              \

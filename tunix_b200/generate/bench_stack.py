@@ -1,10 +1,12 @@
 """Serving throughput of layer-stack models beside the closest uniform decoder of equal size:
-`python bench.py --workload stack_serving` or `python -m tunix_b200.generate.bench_stack [--models roluzen_2b,roluzen_8b]`.
+`python bench.py --workload stack_serving` or
+`python -m tunix_b200.generate.bench_stack [--models roluzen_2b,roluzen_8b,tovalix_2b,tovalix_8b]`.
 
 For every size: prefill tokens/s (`--prefill-seqs` prompts of `--prefill-len` tokens, one sampled token each) and decode
 tokens/s (`--decode-seqs` sequences at context `--decode-ctx`, `--decode-steps` captured steps), both through
-`PagedEngine.__call__`, random-init weights, uniform random token ids. The other model has the same width, feed-forward,
-attention heads, vocabulary and number of layer passes, with sliding-window attention of the same window in every layer.
+`PagedEngine.__call__`, random-init weights, uniform random token ids. The other model has the same width, feed-forward
+(of equal size where only one of them is gated), attention heads, vocabulary and number of layer passes, with
+sliding-window attention in every layer, of the same window or as long as the chunks.
 Times are CUDA events around the call after a warm-up call; a decode step streams the weights (far more than L2), the
 prefill's activations exceed L2 too."""
 from __future__ import annotations
@@ -37,11 +39,12 @@ class _Ids:
 def closest_config(cfg):
     """Uniform decoder with the sizes of a layer-stack config: one attention + MLP layer per layer pass."""
     from ..models.config import ModelConfig
-    from ..models.mixers import ParallelSpec
-    att = next(s.mixer.left for s in cfg.layer_specs if isinstance(s.mixer, ParallelSpec))
+    att = next(a for a in (getattr(s.mixer, "left", s.mixer) for s in cfg.layer_specs) if hasattr(a, "kv_heads"))
+    gated = all(s.ff_kind == "glu" for s in cfg.layer_specs)
     return ModelConfig(family="qwen3", num_layers=len(cfg.runs()), vocab_size=cfg.vocab_size, embed_dim=cfg.embed_dim,
-                       hidden_dim=cfg.hidden_dim, num_heads=att.heads, head_dim=att.dim, num_kv_heads=att.kv_heads, qk_norm=True,
-                       sliding_window=att.window, layer_pattern=("local",), dtype=torch.bfloat16)
+                       hidden_dim=cfg.hidden_dim if gated else round(cfg.hidden_dim * 2 / 3 / 128) * 128, num_heads=att.heads,
+                       head_dim=att.dim, num_kv_heads=att.kv_heads, qk_norm=True, sliding_window=att.window or att.chunk,
+                       layer_pattern=("local",), dtype=torch.bfloat16)
 
 
 def flops_per_token(model) -> float:

@@ -4,7 +4,8 @@
 One JSON line per kernel at the sizes of a preset: median time with L2 flushed between iterations, the algorithmic bytes and
 operations (every input read once, every output written once; no repeated or split work counted), and the fraction of the
 roofline, i.e. the larger of bytes / copy bandwidth and operations / GEMM throughput over the measured time. The like kernels
-of uniform decoders (flash attention with the same window as a prefill calls it, paged decode, RMS norm) come beside them."""
+of uniform decoders (flash attention with the same window as a prefill calls it, paged decode, RMS norm, gated activation)
+come beside them."""
 from __future__ import annotations
 
 import json
@@ -12,19 +13,8 @@ import json
 import torch
 
 
-def run(args, peaks, timer) -> None:
-    from ..models.config import get_config
-    from ..models.mixers import MatrixMemory, ParallelSpec, RGLRUMixer, RGLRUSpec
-    from . import functional as F
-    from . import kernels as K
-    from . import stack_kernels as SK
-    from .ragged import RaggedBatch
+def reporter(args, peaks, timer):
     peak_tf, peak_gb, which = peaks
-    dev, bf = torch.device("cuda"), torch.bfloat16
-    cfg = get_config(args.model)
-    par = next(s.mixer for s in cfg.layer_specs if isinstance(s.mixer, ParallelSpec))
-    rec = next(s.mixer for s in cfg.layer_specs if isinstance(s.mixer, RGLRUSpec))
-    a, mm, D, S = par.left, par.right, cfg.embed_dim, max(cfg.streams, 1)
     only = set(args.only.split(",")) if args.only else None
 
     def report(name, fn, nbytes, flops=0.0, note=None):
@@ -37,19 +27,135 @@ def run(args, peaks, timer) -> None:
         if note:
             line["note"] = note
         print(json.dumps(line), flush=True)
+    return report
 
-    def pool(B, ctx):
-        pages = -(-ctx // 64)
-        mk = lambda n: torch.randn(B * pages, 64, n, device=dev).to(bf)  # noqa: E731
-        return mk(a.kv_heads * a.dim), mk(a.kv_heads * a.vdim), torch.randperm(B * pages, device=dev).int().view(B, pages)
 
+def phases(args):
+    """(phase, batch, entries, context) of a prefill and a decode step."""
+    from .ragged import RaggedBatch
+    for phase, ls in (("prefill", [args.seq] * args.batch), ("decode", [1] * args.decode_batch)):
+        ctx = args.decode_ctx if phase == "decode" else args.seq
+        work = [(i, ctx - 1 if phase == "decode" else 0, [1] * L) for i, L in enumerate(ls)]
+        yield phase, RaggedBatch.build(work, torch.device("cuda")), len(ls), ctx
+
+
+def page_pool(B, ctx, k_cols, v_cols):
+    pages = -(-ctx // 64)
+    mk = lambda n: torch.randn(B * pages, 64, n, device="cuda").to(torch.bfloat16)  # noqa: E731
+    return mk(k_cols), mk(v_cols), torch.randperm(B * pages, device="cuda").int().view(B, pages)
+
+
+def run(args, peaks, timer) -> None:
+    from ..models.config import get_config
+    if get_config(args.model).family == "tovalix":
+        run_tovalix(args, peaks, timer)
+    else:
+        run_roluzen(args, peaks, timer)
+
+
+def run_tovalix(args, peaks, timer) -> None:
+    from ..models.config import get_config
+    from ..models.mixers import ForgetGateMemorySpec, RotaryAttentionSpec, TokenShiftMemorySpec
+    from ..models.stack_exec import FEW_OUTPUTS, rope_table
+    from . import functional as F
+    from . import kernels as K
+    from . import stack_kernels as SK
+    report = reporter(args, peaks, timer)
+    dev, bf = torch.device("cuda"), torch.bfloat16
+    cfg = get_config(args.model)
+    first = lambda t: next(s.mixer for s in cfg.layer_specs if isinstance(s.mixer, t))  # noqa: E731
+    a, wk, fg, D = first(RotaryAttentionSpec), first(TokenShiftMemorySpec), first(ForgetGateMemorySpec), cfg.embed_dim
+    rand = lambda *s: torch.randn(*s, device=dev).to(bf)  # noqa: E731
+    for phase, rb, B, ctx in phases(args):
+        n, one = rb.n, phase == "decode"
+        # --- residual, norms, token shift
+        x, y, w, h = torch.randn(n, 1, D, device=dev), rand(n, D), torch.ones(D, device=dev, dtype=bf), rand(n, D)
+        unit, mu, last = torch.ones(1, device=dev, dtype=bf), rand(5, D), torch.zeros(B, D, device=dev)
+        kw = dict(y=y, mix=unit, w_out=unit, w_in=unit, groups=cfg.norm_groups)
+        report(f"stream_step_{phase}", lambda: SK.stream_step(x, 1e-6, norm_w=w, **kw), n * D * 12.0)
+        report(f"stream_step_groups4_{phase}", lambda: SK.stream_step(x, 1e-6, norm_w=w, **{**kw, "groups": 4}), n * D * 12.0)
+        report(f"stream_step_row_{phase}", lambda: SK.stream_step(x, 1e-6, raw=True, **kw), n * D * 12.0)
+        report(f"stream_step_normed_{phase}", lambda: SK.stream_step(x, 1e-6, norm_w=w, wy=w, **kw), n * D * 12.0)
+        if one:
+            report("stream_step_shift_decode", lambda: SK.stream_step(x, 1e-6, norm_w=w, shift=(mu, last), rb=rb, **kw), n * D * 28.0)
+        else:
+            report("token_shift_prefill", lambda: SK.token_shift(h, mu, last, rb), n * D * 12.0)
+        report(f"like_rmsnorm_{phase}", lambda: K.rmsnorm_fwd(y, w, 1e-6, want_rstd=False), n * D * 4.0)
+        # --- per-layer token input
+        N = cfg.token_side
+        table, gw, z = rand(cfg.vocab_size, 4 * N), rand(N, D), torch.randn(n, N, device=dev)
+        rows = dict(tokens=rb.tokens, rows=table, col=N)
+        if one and N <= FEW_OUTPUTS:
+            report("side_gate_decode", lambda: SK.few_outputs(h, gw, SK.ACT_GELU_ROW, **rows), n * D * 2.0 + N * D * 2)
+        report(f"small_act_{phase}", lambda: SK.small_act(z, bf, SK.ACT_GELU_ROW, **rows), n * N * 6.0)
+        # --- feed-forward activation
+        ff = cfg.hidden_dim
+        up, act = rand(n, ff), rand(2)
+        report(f"xielu_{phase}", lambda: SK.xielu_(up, act), n * ff * 4.0)
+        half = rand(n, ff)
+        report(f"like_glu_{phase}", lambda: K.glu_fwd(half, up, K.GLU_SILU), n * ff * 6.0)
+        del up, half
+        # --- matrix memories
+        for name, sp, mode in (("wkv", wk, SK.GATES_BONUS), ("hgrn2", fg, SK.GATES_LOWER)):
+            H, dk, dv = sp.heads, sp.dim, getattr(sp, "vdim", sp.dim)
+            bonus = mode == SK.GATES_BONUS
+            q, k, v, g = rand(n, H * dk), rand(n, H * dk) if bonus else None, rand(n, H * dv), rand(n, H * dv) if bonus else None
+            z, c0, c1 = torch.randn(n, H * dk, device=dev), rand(H * dk) + (-3 if bonus else 2), torch.rand(H * dk, device=dev).to(bf)
+            S, nw = torch.zeros(B, H, dk, dv, device=dev), torch.ones(H * dv if bonus else dv, device=dev, dtype=bf)
+            nb = n * H * (dk * (6.0 + 2 * bonus) + dv * (4.0 + 2 * bonus)) + B * H * dk * dv * 8.0
+            fl = 0.0 if one else n * H * (4.0 * dk * dv + 16 * (dk + dv))
+            report(f"{name}_{phase}", lambda: SK.gated_linear(mode, q, k, v, z, c0, c1, rb, H, dk, dv, S, nw, 1e-6, gate=g,  # noqa: B023
+                                                              per_head=bonus), nb, fl)
+            del q, k, v, g, z, S
+        # --- attention
+        NQ, NK, NV = a.heads * a.dim, a.kv_heads * a.dim, a.kv_heads * a.vdim
+        kp, vp, table = page_pool(B, ctx, NK, NV)
+        proj, q = rand(n, NQ + NK + NV), rand(n, NQ)
+        cos, sin = rope_table(ctx, a.rot_dims, a.rot_base, dev)
+        report(f"rope_norm_write_{phase}", lambda: SK.rope_norm_write(proj, 0, NQ, NQ + NK, cos, sin, a.rot_dims, 1e-6, rb, table, 64,
+                                                                      a.heads, a.kv_heads, a.dim, a.vdim, kp, vp),
+               n * (NQ + NK + NV) * 4.0)
+        if one:
+            keys = (ctx - 1) % a.chunk + 1
+            nb = B * keys * (NK + NV) * 2.0 + n * NQ * 4.0
+            split = K.decode_split_tokens(B, a.kv_heads, min(ctx, a.chunk + 128))
+            dkw = dict(num_kv_heads=a.kv_heads, page_size=64, max_ctx=ctx, split_tokens=split, scale=a.scale)
+            q3, lens_t = q.view(B, a.heads, a.dim), rb.pos0 + 1
+            pd = lambda **o: K.paged_decode(q3, kp, vp, table, rb.slot, lens_t, **dkw, **o)  # noqa: E731
+            report("attention_decode", lambda: pd(softcap=a.softcap, chunk=a.chunk), nb)
+            report("like_paged_decode", lambda: pd(window=keys), nb, note="as many keys")
+        else:
+            full = sum(i % a.chunk + 1 for i in range(args.seq)) * float(B)
+            fl, nb = full * a.heads * a.dim * 4.0, n * (2 * NQ + NK + NV) * 2.0
+            pk = dict(num_heads=a.heads, num_kv_heads=a.kv_heads, head_dim=a.dim, scale=a.scale)
+            report("attention_prefill", lambda: K.attn_fwd_paged(q, kp, vp, rb, table, 64, softcap=a.softcap, chunk=a.chunk, **pk), nb, fl)
+            report("attention_prefill_uncapped", lambda: K.attn_fwd_paged(q, kp, vp, rb, table, 64, chunk=a.chunk, **pk), nb, fl)
+            q4 = q.view(B, args.seq, a.heads, a.dim)
+            k4, v4 = (rand(B, args.seq, a.kv_heads, a.dim) for _ in range(2))
+            seg = torch.ones(B, args.seq, dtype=torch.int32, device=dev)
+            win = sum(min(i + 1, a.chunk) for i in range(args.seq)) * float(B) * a.heads * a.dim * 4.0
+            att = lambda s: F.attention(q4, k4, v4, scale=a.scale, causal=True, window=a.chunk, seg_q=s, seg_k=s)  # noqa: E731
+            with torch.no_grad():
+                report("like_attn_fwd", lambda: att(None), nb, win, note="window as long as a chunk")
+                report("like_attn_fwd_segments", lambda: att(seg), nb, win, note="as the padded prefill of uniform decoders calls it")
+
+
+def run_roluzen(args, peaks, timer) -> None:
+    from ..models.config import get_config
+    from ..models.mixers import ParallelSpec, RGLRUMixer, RGLRUSpec
+    from . import functional as F
+    from . import kernels as K
+    from . import stack_kernels as SK
+    report = reporter(args, peaks, timer)
+    dev, bf = torch.device("cuda"), torch.bfloat16
+    cfg = get_config(args.model)
+    par = next(s.mixer for s in cfg.layer_specs if isinstance(s.mixer, ParallelSpec))
+    rec = next(s.mixer for s in cfg.layer_specs if isinstance(s.mixer, RGLRUSpec))
+    a, mm, D, S = par.left, par.right, cfg.embed_dim, max(cfg.streams, 1)
     bias = torch.randn(a.heads, a.bias_max + 1, device=dev)
     aw = dict(scale=a.scale, window=a.window)
-    lens = {"prefill": [args.seq] * args.batch, "decode": [1] * args.decode_batch}
-    for phase, ls in lens.items():
-        B, n, one = len(ls), sum(ls), phase == "decode"
-        ctx = args.decode_ctx if one else args.seq
-        rb = RaggedBatch.build([(i, ctx - 1 if one else 0, [1] * L) for i, L in enumerate(ls)], dev)
+    for phase, rb, B, ctx in phases(args):
+        n, one = rb.n, phase == "decode"
         # --- streams
         x = torch.randn(n, S, D, device=dev)
         y, y2 = (torch.randn(n, D, device=dev).to(bf) for _ in range(2))
@@ -83,8 +189,8 @@ def run(args, peaks, timer) -> None:
                n * H * (4.0 * dk + 2 * dv + 4 * dv) + B * H * dk * dv * 8.0, 0.0 if one else fl)
         del proj
         # --- attention
-        kp, vp, table = pool(B, ctx)
         NQ, NK, NV = a.heads * a.dim, a.kv_heads * a.dim, a.kv_heads * a.vdim
+        kp, vp, table = page_pool(B, ctx, NK, NV)
         proj = torch.randn(n, NQ + NK + NV, device=dev).to(bf)
         qw, kwt = torch.ones(NQ, device=dev, dtype=bf), torch.ones(NK, device=dev, dtype=bf)
         report(f"qk_norm_write_{phase}", lambda: SK.qk_norm_write(proj, 0, NQ, NQ + NK, qw, kwt, 1e-6, rb, table, 64, kp, vp, NQ),
