@@ -78,8 +78,9 @@ def test_gate_outputs(C1, heads, vdim, dtype):
 @pytest.mark.parametrize("K,N", [(40, 4), (1024, 6), (4096, 16), (256, 70)])
 def test_few_outputs(K, N):
     from tunix_b200.ops import stack_kernels as SK
-    x, w = rand(5, K, dtype=torch.bfloat16), rand(N, K, dtype=torch.bfloat16, seed=1)
-    assert rel(SK.few_outputs(x, w), x.double() @ w.double().T) < 1e-5
+    for n in (5, 16, 35):
+        x, w = rand(n, K, dtype=torch.bfloat16), rand(N, K, dtype=torch.bfloat16, seed=1)
+        assert rel(SK.few_outputs(x, w), x.double() @ w.double().T) < 1e-5
 
 
 @pytest.mark.parametrize("dtype", DT)
@@ -116,6 +117,15 @@ def test_xielu(rows, F, p, q, dtype):
     got = SK.xielu_(z.clone(), act)
     assert rel(got, want) < (1e-6 if dtype == torch.float32 else 5e-3)
     assert torch.allclose(got.view(-1)[:4].double().cpu(), want.view(-1)[:4], rtol=1e-6 if dtype == torch.float32 else 5e-3, atol=1e-7)
+
+
+@pytest.mark.parametrize("M,N,K", [(5, 64, 128), (64, 16640, 256), (130, 200, 64)])
+def test_packed_product_with_xielu(M, N, K):
+    from tunix_b200.ops import kernels as K_
+    x, w = rand(M, K, dtype=torch.bfloat16), rand(N, K, dtype=torch.bfloat16, std=0.2, seed=1)
+    act = torch.tensor([0.5, 1.25], device="cuda", dtype=torch.bfloat16)
+    want = TO.xielu((x.double() @ w.double().T).cpu(), *act.double().cpu())
+    assert rel(K_.gemm_packed(x, K_.PackedWeight(w), xielu=act), want) < 5e-3
 
 
 @pytest.mark.parametrize("dtype", DT)

@@ -40,6 +40,8 @@ enum GemmFlags : int {
   // groups of 16 = [8 gate | 8 up] (tb_pack_weight_glu); the kernel writes act(gate) * up, N / 2 bf16 columns.
   GF_GLU_SILU = 64,
   GF_GLU_GELU = 128,
+  // packed weights only: xIELU on the result; `bias` holds its two numbers (bf16) instead of a bias
+  GF_XIELU = 256,
 };
 
 // Grouped mode (mixture-of-experts): the tile list lives in device memory, built by a planning kernel from
@@ -589,6 +591,13 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
     const bool has_bias = args.flags & GF_BIAS;
     const bool has_res = args.flags & GF_RESIDUAL;
     const int glu_kind = (args.flags & GF_GLU_SILU) ? 1 : (args.flags & GF_GLU_GELU) ? 2 : 0;
+    const bool xielu = args.flags & GF_XIELU;
+    float xi_pos = 0.f, xi_neg = 0.f;
+    if (xielu) {
+      const float p = __bfloat162float(args.bias[0]), q2 = __bfloat162float(args.bias[1]);
+      xi_pos = fmaxf(p, 0.f) + log1pf(__expf(-fabsf(p)));
+      xi_neg = 0.5f + fmaxf(q2, 0.f) + log1pf(__expf(-fabsf(q2)));
+    }
     const float alpha = args.alpha;
     const bool c_al16 = (reinterpret_cast<uintptr_t>(args.C) & 15) == 0;      // vector paths need aligned bases
     const bool r_al16 = (reinterpret_cast<uintptr_t>(args.resid) & 15) == 0;
@@ -652,6 +661,13 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
               *reinterpret_cast<uint4*>(cp + 8 * g) = pk;       // ldc % 8 == 0 and col0 % 32 == 0: 16-byte aligned
             }
             continue;
+          }
+          if (xielu) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i) {
+              const float z = v[i];
+              v[i] = (z > 0.f ? xi_pos * z * z : xi_neg * (__expf(fminf(z, 0.f)) - 1.f - z)) + 0.5f * z;
+            }
           }
           if (has_bias) {
 #pragma unroll
@@ -1073,13 +1089,14 @@ TB_API int tb_gemm_packed_bf16(const void* A, long long lda, const void* P, int 
   if (glu && ((flags & (GF_OUT_F32 | GF_ACCUM | GF_BIAS | GF_RESIDUAL)) || (N % 16) || (ldc % 8) ||
               (reinterpret_cast<uintptr_t>(C) & 15) || alpha != 1.0f))
     return -2;
+  if ((flags & GF_XIELU) && ((flags & (GF_ACCUM | GF_BIAS | GF_RESIDUAL)) || glu || bias == nullptr)) return -2;
   if (g_sm_count == 0) {
     int dev = 0;
     cudaGetDevice(&dev);
     cudaDeviceGetAttribute(&g_sm_count, cudaDevAttrMultiProcessorCount, dev);
   }
   static const bool no_splitk = getenv("TUNIX_B200_NO_SPLITK") != nullptr;
-  if (w == 256 && !no_splitk && !glu) {
+  if (w == 256 && !no_splitk && !glu && !(flags & GF_XIELU)) {
     const int sk = tb_gemm_splitk_try(A, nullptr, C, M, N, K, lda, 8, ldc, flags, bias, resid, ldr, alpha, status, stream, P);
     if (sk != 0) return sk < 0 ? sk : 0;
   }

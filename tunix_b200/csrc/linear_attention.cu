@@ -51,13 +51,13 @@ __device__ __forceinline__ void gates_exact(float z, float c0, float c1, float& 
     f = k < 0.5f ? 1.f - k : c1 + (1.f - c1) * sigmoid(z + c0);
   }
 }
-// log2 f for bf16 models; bounded, so that sums of it stay finite. b0 = gates_offset(c0)
+// log2 f for bf16 models; bounded where f is zero in any sum of them. b0 = gates_offset(c0)
 template <int MODE>
 __device__ __forceinline__ float gates_offset(float c0) { return c0 * LOG2_E + (MODE == BONUS ? 0.5287663729448977f : 0.f); }   // + log2(log2 e)
 template <int MODE>
 __device__ __forceinline__ float gates_log2(float z, float b0, float c1, float& k) {
   const float e = quick_exp2(fminf(fmaf(z, LOG2_E, b0), 100.f));
-  if (MODE == BONUS) return -fminf(e, 1e4f);
+  if (MODE == BONUS) return -fminf(e, 150.f);
   const float s = quick_rcp(1.f + e), r = 1.f - c1;    // sigmoid of the negative; e s: of the positive
   k = r * s;
   return quick_log2_decay(k, fmaf(r, e * s, c1));
@@ -390,53 +390,66 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
     const int rows = min(TT, len - tile * TT);
     cp_async_wait<0>();
     __syncthreads();                    // the tile is in; nobody reads the last tile's operands any more
-    float L[16][2], kk[16][2];
-    {
-      float run0 = 0.f, run1 = 0.f;
-#pragma unroll
-      for (int t = 0; t < 16; ++t) {
-        const int row = psub * 16 + t;
-        const float2 z = *reinterpret_cast<const float2*>(Z + row * KP + pd);
-        float l0 = gates_log2<MODE>(z.x, b0[0], b1[0], kk[t][0]), l1 = gates_log2<MODE>(z.y, b0[1], b1[1], kk[t][1]);
-        if (MODE == BONUS) {
-          const uint32_t k2 = *reinterpret_cast<const uint32_t*>(smem + M.k + row * M.pitch + pd * 2);
-          kk[t][0] = bf16_lo(k2);
-          kk[t][1] = bf16_hi(k2);
-        }
-        if (row >= rows) l0 = l1 = kk[t][0] = kk[t][1] = 0.f;
-        run0 += l0;
-        run1 += l1;
-        L[t][0] = run0;
-        L[t][1] = run1;
-      }
-    }
-    const float e0 = L[15][0], e1 = L[15][1];
-    float m0 = L[7][0], m1 = L[7][1];
-    const bool direct = __syncthreads_or(fminf(fminf(m0, e0 - m0), fminf(m1, e1 - m1)) < -SAFE);
-    if (direct) m0 = m1 = 0.f;
-    float dg[16];
+    // log2 f and k of this lane's two channels. Every factor below is the power of a sum of its own, never of a difference
+    // of sums: where one token decays much, the others keep their accuracy.
+    float l[16][2], h0[2] = {0.f, 0.f}, h1[2] = {0.f, 0.f};      // h0, h1: sums over the halves of the block
 #pragma unroll
     for (int t = 0; t < 16; ++t) {
       const int row = psub * 16 + t;
-      const uint32_t at = row * M.pitch + pd * 2;
-      const uint32_t q2 = *reinterpret_cast<const uint32_t*>(smem + M.q + at);
-      float q0 = bf16_lo(q2), q1 = bf16_hi(q2);
-      if (MODE == LOWER) { q0 = silu<bf>(q0); q1 = silu<bf>(q1); }
-      else dg[t] = q0 * b1[0] * kk[t][0] + q1 * b1[1] * kk[t][1];
-      const int tr = MODE == LOWER ? t : t - 1;         // the last token whose decay the read-out has seen
-      const float r0 = tr >= 0 ? L[tr < 0 ? 0 : tr][0] : 0.f, r1 = tr >= 0 ? L[tr < 0 ? 0 : tr][1] : 0.f;
-      *reinterpret_cast<uint32_t*>(smem + M.Q + at) = pack_bf16(q0 * quick_exp2(r0 - m0), q1 * quick_exp2(r1 - m1));
-      if (!direct)
-        *reinterpret_cast<uint32_t*>(smem + M.Ki + at) = pack_bf16(kk[t][0] * quick_exp2(m0 - L[t][0]), kk[t][1] * quick_exp2(m1 - L[t][1]));
-      bf h0, h1, l0, l1;
-      split_bf16(kk[t][0] * quick_exp2(e0 - L[t][0]), h0, l0);
-      split_bf16(kk[t][1] * quick_exp2(e1 - L[t][1]), h1, l1);
-      *reinterpret_cast<__nv_bfloat162*>(smem + M.Kh + at) = __halves2bfloat162(h0, h1);
-      *reinterpret_cast<__nv_bfloat162*>(smem + M.Kl + at) = __halves2bfloat162(l0, l1);
+      const float2 z = *reinterpret_cast<const float2*>(Z + row * KP + pd);
+      float2 k;
+      l[t][0] = gates_log2<MODE>(z.x, b0[0], b1[0], k.x);
+      l[t][1] = gates_log2<MODE>(z.y, b0[1], b1[1], k.y);
+      if (row >= rows) l[t][0] = l[t][1] = k.x = k.y = 0.f;
+      // keys made from the gates take the place of z: only the sums stay in registers
+      if (MODE == LOWER) *reinterpret_cast<float2*>(smem + M.z + (row * KP + pd) * 4) = k;
+#pragma unroll
+      for (int i = 0; i < 2; ++i) (t < 8 ? h0[i] : h1[i]) += l[t][i];
     }
-    *reinterpret_cast<float2*>(De + psub * KP + pd) = make_float2(quick_exp2(m0), quick_exp2(m1));
-    *reinterpret_cast<float2*>(Dd + psub * KP + pd) = make_float2(quick_exp2(e0 - m0), quick_exp2(e1 - m1));
+    const bool direct = __syncthreads_or(fminf(fminf(h0[0], h1[0]), fminf(h0[1], h1[1])) < -SAFE);
+    auto queries = [&](int row, float& q0, float& q1) {
+      const uint32_t q2 = *reinterpret_cast<const uint32_t*>(smem + M.q + row * M.pitch + pd * 2);
+      q0 = bf16_lo(q2);
+      q1 = bf16_hi(q2);
+      if (MODE == LOWER) { q0 = silu<bf>(q0); q1 = silu<bf>(q1); }
+    };
+    auto keys = [&](int row) {                          // rows past the end hold zeros
+      if (MODE == LOWER) return *reinterpret_cast<const float2*>(smem + M.z + (row * KP + pd) * 4);
+      const uint32_t k2 = *reinterpret_cast<const uint32_t*>(smem + M.k + row * M.pitch + pd * 2);
+      return make_float2(bf16_lo(k2), bf16_hi(k2));
+    };
+    // token t: read-out scaled by e^(log2 r), key by e^(log2 w)
+    auto scaled = [&](int t, float r0, float r1, float w0, float w1) {
+      const int row = psub * 16 + t;
+      const uint32_t at = row * M.pitch + pd * 2;
+      float q0, q1;
+      queries(row, q0, q1);
+      const float2 k = keys(row);
+      *reinterpret_cast<uint32_t*>(smem + M.Q + at) = pack_bf16(q0 * quick_exp2(r0), q1 * quick_exp2(r1));
+      *reinterpret_cast<uint32_t*>(smem + M.Ki + at) = pack_bf16(k.x * quick_exp2(w0), k.y * quick_exp2(w1));
+    };
+    float end0 = 0.f, end1 = 0.f;                       // sums from the token after t to the block's end
+#pragma unroll
+    for (int t = 15; t >= 0; --t) {
+      const uint32_t at = (psub * 16 + t) * M.pitch + pd * 2;
+      const float2 k = keys(psub * 16 + t);
+      bf hi0, hi1, lo0, lo1;
+      split_bf16(k.x * quick_exp2(end0), hi0, lo0);
+      split_bf16(k.y * quick_exp2(end1), hi1, lo1);
+      *reinterpret_cast<__nv_bfloat162*>(smem + M.Kh + at) = __halves2bfloat162(hi0, hi1);
+      *reinterpret_cast<__nv_bfloat162*>(smem + M.Kl + at) = __halves2bfloat162(lo0, lo1);
+      end0 += l[t][0];
+      end1 += l[t][1];
+    }
     if (MODE == BONUS) {
+      float dg[16];
+#pragma unroll
+      for (int t = 0; t < 16; ++t) {
+        float q0, q1;
+        queries(psub * 16 + t, q0, q1);
+        const float2 k = keys(psub * 16 + t);
+        dg[t] = q0 * b1[0] * k.x + q1 * b1[1] * k.y;
+      }
       // 16 sums over the warp: halve the values a lane holds at every step
 #pragma unroll
       for (int w = 8; w >= 1; w >>= 1) {
@@ -449,21 +462,46 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
       dg[0] += __shfl_xor_sync(0xffffffffu, dg[0], 16);
       if (lane < 16) Dg[(warp % HALVES) * TT + psub * 16 + lane] = dg[0];
     }
-    __syncthreads();
-    if (direct) {
-      // L, q and k of the whole tile go to shared memory, then one thread per weight
+    if (!direct) {
+      float c0s = 0.f, c1s = 0.f;                       // from the token after t to the middle
+#pragma unroll
+      for (int t = 7; t >= 0; --t) {
+        const float n0 = c0s + l[t][0], n1 = c1s + l[t][1];
+        scaled(t, MODE == LOWER ? -c0s : -n0, MODE == LOWER ? -c1s : -n1, c0s, c1s);
+        c0s = n0;
+        c1s = n1;
+      }
+      c0s = c1s = 0.f;                                  // from the middle to the token
+#pragma unroll
+      for (int t = 8; t < 16; ++t) {
+        const float n0 = c0s + l[t][0], n1 = c1s + l[t][1];
+        scaled(t, MODE == LOWER ? n0 : c0s, MODE == LOWER ? n1 : c1s, -n0, -n1);
+        c0s = n0;
+        c1s = n1;
+      }
+    } else {
+      // read-outs from the block's start; sums, queries and keys of the whole tile for the weights below
+      float c0s = 0.f, c1s = 0.f;
 #pragma unroll
       for (int t = 0; t < 16; ++t) {
         const int row = psub * 16 + t;
         const uint32_t at = row * M.pitch + pd * 2;
-        *reinterpret_cast<float2*>(smem + M.z + (row * KP + pd) * 4) = make_float2(L[t][0], L[t][1]);
-        *reinterpret_cast<uint32_t*>(smem + M.k + at) = pack_bf16(kk[t][0], kk[t][1]);
-        if (MODE == LOWER) {
-          uint32_t* q2 = reinterpret_cast<uint32_t*>(smem + M.q + at);
-          *q2 = pack_bf16(silu<bf>(bf16_lo(*q2)), silu<bf>(bf16_hi(*q2)));
-        }
+        const float n0 = c0s + l[t][0], n1 = c1s + l[t][1];
+        float q0, q1;
+        queries(row, q0, q1);
+        const float2 k = keys(row);
+        *reinterpret_cast<uint32_t*>(smem + M.Q + at) = pack_bf16(q0 * quick_exp2(MODE == LOWER ? n0 : c0s), q1 * quick_exp2(MODE == LOWER ? n1 : c1s));
+        *reinterpret_cast<float2*>(smem + M.z + (row * KP + pd) * 4) = make_float2(n0, n1);
+        *reinterpret_cast<uint32_t*>(smem + M.k + at) = pack_bf16(k.x, k.y);
+        *reinterpret_cast<uint32_t*>(smem + M.q + at) = pack_bf16(q0, q1);
+        c0s = n0;
+        c1s = n1;
       }
-      __syncthreads();
+    }
+    *reinterpret_cast<float2*>(De + psub * KP + pd) = direct ? make_float2(1.f, 1.f) : make_float2(quick_exp2(h0[0]), quick_exp2(h0[1]));
+    *reinterpret_cast<float2*>(Dd + psub * KP + pd) = direct ? make_float2(quick_exp2(end0), quick_exp2(end1)) : make_float2(quick_exp2(h1[0]), quick_exp2(h1[1]));
+    __syncthreads();
+    if (direct) {                       // one thread per weight
       for (int i = tid; i < SUBS * 256; i += NT) {
         const int sub = i >> 8, t = (i >> 4) & 15, s = i & 15, rt = sub * 16 + t, rs = sub * 16 + s;
         float p = 0.f;

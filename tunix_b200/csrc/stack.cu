@@ -16,6 +16,7 @@
 //   xielu       : the activation of feed-forwards without a gate.
 //
 // This file is compiled without fast-math: the same kernels serve the 32-bit mode.
+#include "mma.cuh"
 #include "precise.cuh"
 
 using namespace tb;
@@ -362,29 +363,47 @@ __device__ __forceinline__ float apply_small(int act, float z, const long long* 
   return z;
 }
 
-// out[t, o] = act(sum_k x[t, k] w[o, k]) with an fp32 sum, for a handful of outputs and few rows (gates of a decode step):
-// one CTA per row, a warp per output.
+// out[t, o] = act(sum_k x[t, k] w[o, k]) with an fp32 sum, for few outputs and few rows (gates and bottlenecks of a decode
+// step): a CTA owns 16 rows x 8 outputs, its warps split the contraction and meet in shared memory. A lane loads 8 consecutive
+// k of its two rows and its output at once; both operands see the same permutation of k, so no shuffle is needed.
+constexpr int FW = 8;           // warps
 template <typename TO>
-__global__ void __launch_bounds__(512)
-few_outputs_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ w, int K, int N, int act,
+__global__ void __launch_bounds__(32 * FW)
+few_outputs_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ w, int n, int K, int N, int act,
                    const long long* __restrict__ tokens, int vocab, const __nv_bfloat16* __restrict__ e, long long lde, int e_off,
                    TO* __restrict__ out) {
+  __shared__ float part[FW][16][9];
   pdl_trigger();
   pdl_wait();
-  const long long t = blockIdx.x;
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
-  for (int o = warp; o < N; o += nw) {
-    float acc = 0.f;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, q8 = (lane & 3) * 8;
+  const int r0 = blockIdx.y * 16 + g, r1 = r0 + 8, o = blockIdx.x * 8 + g;
+  const __nv_bfloat16 *x0 = x + (long long)min(r0, n - 1) * K, *x1 = x + (long long)min(r1, n - 1) * K, *wo = w + (long long)min(o, N - 1) * K;
+  float acc[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll 4
-    for (int k = lane * 8; k < K; k += 256) {
-      float a[8], b[8];
-      load_v<8>(x + t * K + k, a);
-      load_v<8>(w + (long long)o * K + k, b);
+  for (int kb = warp * 32; kb < K; kb += FW * 32) {             // whole warps stay together for the products
+    const int k = kb + q8;                                      // K is a multiple of 8: a lane's 8 elements are in or out
+    const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+    const uint4 a = k < K ? *reinterpret_cast<const uint4*>(x0 + k) : zero, b = k < K ? *reinterpret_cast<const uint4*>(x1 + k) : zero;
+    const uint4 c = k < K ? *reinterpret_cast<const uint4*>(wo + k) : zero;
+    const uint32_t s0[4] = {a.x, b.x, a.y, b.y}, s1[4] = {a.z, b.z, a.w, b.w};
+    mma_16816(acc, s0, c.x, c.y);
+    mma_16816(acc, s1, c.z, c.w);
+  }
+  const int c2 = 2 * (lane & 3);
+  part[warp][g][c2] = acc[0];
+  part[warp][g][c2 + 1] = acc[1];
+  part[warp][g + 8][c2] = acc[2];
+  part[warp][g + 8][c2 + 1] = acc[3];
+  __syncthreads();
+  if (threadIdx.x < 128) {
+    const int r = threadIdx.x >> 3, c = threadIdx.x & 7, oo = blockIdx.x * 8 + c;
+    const long long t = blockIdx.y * 16 + r;
+    if (t < n && oo < N) {
+      float v = 0.f;
 #pragma unroll
-      for (int i = 0; i < 8; ++i) acc += a[i] * b[i];
+      for (int i = 0; i < FW; ++i) v += part[i][r][c];
+      out[t * N + oo] = from_f<TO>(apply_small(act, v, tokens, vocab, e, lde, e_off, t, oo));
     }
-    acc = warp_sum(acc);
-    if (lane == 0) out[t * N + o] = from_f<TO>(apply_small(act, acc, tokens, vocab, e, lde, e_off, t, o));
   }
 }
 
@@ -549,10 +568,11 @@ TB_API int tb_few_outputs(const void* x, const void* w, int n, int K, int N, int
                           const void* e, long long lde, int e_off, void* out, int out_bf16, cudaStream_t stream) {
   if (n <= 0 || N <= 0) return 0;
   if (K % 8) return -2;
-  const int threads = N >= 16 ? 512 : N >= 8 ? 256 : 128;
   typedef __nv_bfloat16 bf;
+  const dim3 grid((N + 7) / 8, (n + 15) / 16);
+  if (grid.y > 65535) return -2;
 #define FO(TO)                                                                                                              \
-  launch_pdl(few_outputs_kernel<TO>, dim3(n), dim3(threads), 0, stream, (const bf*)x, (const bf*)w, K, N, act, tokens, vocab, \
+  launch_pdl(few_outputs_kernel<TO>, grid, dim3(32 * FW), 0, stream, (const bf*)x, (const bf*)w, n, K, N, act, tokens, vocab, \
              (const bf*)e, lde, e_off, (TO*)out)
   return (out_bf16 ? FO(bf) : FO(float)) == cudaSuccess ? 0 : -5;
 #undef FO

@@ -90,8 +90,10 @@ def measure(cfg, args) -> dict:
     prompts = rng.integers(3, cfg.vocab_size, (args.decode_seqs, args.decode_ctx)).tolist()
     short, long = 5, 5 + args.decode_steps
     timed(eng, prompts, args.decode_ctx, long)
-    a = min(timed(eng, prompts, args.decode_ctx, short) for _ in range(args.repeats))
-    b = min(timed(eng, prompts, args.decode_ctx, long) for _ in range(args.repeats))
+    a = b = float("inf")                # alternating, so that a change of clocks reaches both
+    for _ in range(args.repeats):
+        a = min(a, timed(eng, prompts, args.decode_ctx, short))
+        b = min(b, timed(eng, prompts, args.decode_ctx, long))
     _lib.raise_if_kernel_error()
     step = (b - a) / args.decode_steps
     n_pre = args.prefill_seqs * args.prefill_len
@@ -107,7 +109,7 @@ def measure(cfg, args) -> dict:
 
 
 def add_arguments(ap) -> None:
-    ap.add_argument("--models", default="roluzen_2b,roluzen_8b", help="layer-stack presets (stack_serving)")
+    ap.add_argument("--models", default="roluzen_2b,roluzen_8b,tovalix_2b,tovalix_8b", help="layer-stack presets (stack_serving)")
     ap.add_argument("--prefill-seqs", type=int, default=4)
     ap.add_argument("--prefill-len", type=int, default=4096)
     ap.add_argument("--decode-seqs", type=int, default=64)

@@ -61,7 +61,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
         torch.backends.cuda.matmul.allow_tf32 = prev
 
 
-FEW_OUTPUTS = 32        # in a decode step, products with fewer outputs than this run one CTA per row
+FEW_OUTPUTS = 512       # in a decode step, products with at most this many outputs split the contraction inside a CTA
 
 
 def rope_table(positions: int, dims: int, base: float, device) -> tuple:
@@ -224,7 +224,8 @@ class StackExecutor:
 
     def _mlp(self, i, mlp, h, rb: RaggedBatch):
         if isinstance(mlp, PlainMLP):
-            act = SK.xielu_(linear(h, self.w[i]["up"], packed=self.pk(i, "up") if rb.decode else None), mlp.act)
+            pup = self.pk(i, "up") if rb.decode else None
+            act = K.gemm_packed(h, pup, xielu=mlp.act) if pup is not None else SK.xielu_(linear(h, self.w[i]["up"]), mlp.act)
             return linear(act, mlp.down_proj.weight, packed=self.pk(i, "down") if rb.decode else None)
         gu_w = self.w[i]["gu"]
         F = gu_w.shape[0] // 2

@@ -1,4 +1,4 @@
-"""Micro-benchmarks of the layer-stack kernels: `python -m tunix_b200.ops.bench_kernels stack [--model roluzen_8b]
+"""Micro-benchmarks of the layer-stack kernels: `python -m tunix_b200.ops.bench_kernels stack [--model roluzen_8b|tovalix_8b]
 [--batch 4 --seq 4096] [--decode-batch 64 --decode-ctx 1024] [--only mlstm_prefill,...]`.
 
 One JSON line per kernel at the sizes of a preset: median time with L2 flushed between iterations, the algorithmic bytes and
@@ -87,7 +87,9 @@ def run_tovalix(args, peaks, timer) -> None:
         rows = dict(tokens=rb.tokens, rows=table, col=N)
         if one and N <= FEW_OUTPUTS:
             report("side_gate_decode", lambda: SK.few_outputs(h, gw, SK.ACT_GELU_ROW, **rows), n * D * 2.0 + N * D * 2)
-        report(f"small_act_{phase}", lambda: SK.small_act(z, bf, SK.ACT_GELU_ROW, **rows), n * N * 6.0)
+            report("like_narrow_gemm_decode", lambda: K.gemm(h, gw), n * D * 2.0 + N * D * 2)
+        else:
+            report(f"small_act_{phase}", lambda: SK.small_act(z, bf, SK.ACT_GELU_ROW, **rows), n * N * 6.0)
         # --- feed-forward activation
         ff = cfg.hidden_dim
         up, act = rand(n, ff), rand(2)

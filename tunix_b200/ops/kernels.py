@@ -9,7 +9,7 @@ import torch
 
 from .. import _lib
 
-GF_A_MN, GF_B_MN, GF_OUT_F32, GF_ACCUM, GF_BIAS, GF_RESIDUAL, GF_GLU_SILU, GF_GLU_GELU = 1, 2, 4, 8, 16, 32, 64, 128
+GF_A_MN, GF_B_MN, GF_OUT_F32, GF_ACCUM, GF_BIAS, GF_RESIDUAL, GF_GLU_SILU, GF_GLU_GELU, GF_XIELU = 1, 2, 4, 8, 16, 32, 64, 128, 256
 
 launch_count = 0  # number of native kernel launches issued through this module
 
@@ -821,8 +821,9 @@ class PackedWeight:
 
 def gemm_packed(a: torch.Tensor, pw: PackedWeight, *, out: torch.Tensor | None = None, out_dtype: torch.dtype = torch.bfloat16,
                 accumulate: bool = False, bias: torch.Tensor | None = None, residual: torch.Tensor | None = None,
-                alpha: float = 1.0, glu: int | None = None) -> torch.Tensor:
-    """C = alpha * A @ W^T with W given as a PackedWeight; same epilogue options as `gemm`. `glu` (GLU_SILU / GLU_GELU)
+                alpha: float = 1.0, glu: int | None = None, xielu: torch.Tensor | None = None) -> torch.Tensor:
+    """C = alpha * A @ W^T with W given as a PackedWeight; same epilogue options as `gemm`. `xielu` (the activation's two
+    numbers, before softplus): xIELU on the result, computed in the epilogue. `glu` (GLU_SILU / GLU_GELU)
     with a weight packed with `glu=True`: C [M, N / 2] = act(A @ Wgate^T) * (A @ Wup^T), computed in the epilogue."""
     assert a.dtype == torch.bfloat16 and _is2d_rowmajor(a)
     M, K = a.shape
@@ -856,6 +857,10 @@ def gemm_packed(a: torch.Tensor, pw: PackedWeight, *, out: torch.Tensor | None =
     if bias is not None:
         assert bias.dtype == torch.bfloat16 and bias.numel() == N and bias.is_contiguous()
         flags |= GF_BIAS
+    if xielu is not None:
+        assert not accumulate and bias is None and residual is None and xielu.dtype == torch.bfloat16 and xielu.numel() == 2
+        flags |= GF_XIELU
+        bias = xielu
     ldr = 0
     if residual is not None:
         assert residual.dtype == torch.bfloat16 and residual.shape == (M, N) and residual.stride(1) == 1

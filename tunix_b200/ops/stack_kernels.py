@@ -101,8 +101,8 @@ ACT_NONE, ACT_TANH, ACT_GELU_ROW = 0, 1, 2      # csrc/stack.cu: apply_small
 
 
 def few_outputs(x: torch.Tensor, w: torch.Tensor, act: int = ACT_NONE, tokens=None, rows=None, col: int = 0) -> torch.Tensor:
-    """act(x bf16 [n, K] @ w^T [N, K]) for a handful of outputs and decode-size n (a GEMM tile would leave one CTA with the
-    whole contraction): fp32 [n, N], or bf16 after an activation. ACT_GELU_ROW multiplies by columns col .. col + N of the
+    """act(x bf16 [n, K] @ w^T [N, K]) for few outputs and decode-size n (GEMM tiles would leave a few CTAs with the whole
+    contraction): fp32 [n, N], or bf16 after an activation. ACT_GELU_ROW multiplies by columns col .. col + N of the
     tokens' rows of the table `rows`."""
     assert x.dtype == w.dtype == torch.bfloat16 and x.is_contiguous() and w.is_contiguous() and x.shape[1] % 8 == 0
     out = torch.empty((x.shape[0], w.shape[0]), dtype=torch.float32 if act == ACT_NONE else torch.bfloat16, device=x.device)
