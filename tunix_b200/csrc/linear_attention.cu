@@ -668,7 +668,10 @@ int launch_chunk(const GlaArgs& a, float* raw, bf* out, cudaStream_t stream) {
   bf* o = a.dv <= DV ? out : nullptr;
   static DeviceOnce once;
   if (once.first() &&
-      cudaFuncSetAttribute(gla_chunk_kernel<KP, MODE, WARPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -5;
+      (cudaFuncSetAttribute(gla_chunk_kernel<KP, MODE, WARPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess ||
+       // two of the smaller CTAs fit an SM only if the launches around them leave it this carveout
+       cudaFuncSetAttribute(gla_chunk_kernel<KP, MODE, WARPS>, cudaFuncAttributePreferredSharedMemoryCarveout,
+                            cudaSharedmemCarveoutMaxShared) != cudaSuccess)) return -5;
   const dim3 grid((a.dv + DV - 1) / DV, a.heads, a.rb.E);
   return launch_pdl(gla_chunk_kernel<KP, MODE, WARPS>, grid, dim3(32 * WARPS), smem, stream, a, raw, o) == cudaSuccess ? 0 : -5;
 }

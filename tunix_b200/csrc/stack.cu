@@ -379,7 +379,7 @@ few_outputs_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __r
   const int r0 = blockIdx.y * 16 + g, r1 = r0 + 8, o = blockIdx.x * 8 + g;
   const __nv_bfloat16 *x0 = x + (long long)min(r0, n - 1) * K, *x1 = x + (long long)min(r1, n - 1) * K, *wo = w + (long long)min(o, N - 1) * K;
   float acc[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll 4
+#pragma unroll 8
   for (int kb = warp * 32; kb < K; kb += FW * 32) {             // whole warps stay together for the products
     const int k = kb + q8;                                      // K is a multiple of 8: a lane's 8 elements are in or out
     const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
