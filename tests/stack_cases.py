@@ -1,14 +1,14 @@
-"""Small Roluzen and Tovalix checkpoints with random weights for the layer-stack tests (config.json dict + tensors by name)."""
+"""Small Roluzen, Tovalix and Zikezen checkpoints with random weights for the layer-stack tests (config.json dict + tensors by name)."""
 import json
 import os
 
 import torch
 
-from tests import roluzen_oracle, tovalix_oracle
+from tests import roluzen_oracle, tovalix_oracle, zikezen_oracle
 
 
 def oracle(cfg):
-    return {"Roluzen": roluzen_oracle, "Tovalix": tovalix_oracle}[cfg["architecture"]]
+    return {"Roluzen": roluzen_oracle, "Tovalix": tovalix_oracle, "Zikezen": zikezen_oracle}[cfg["architecture"]]
 
 
 # ---- Roluzen
@@ -60,6 +60,35 @@ def tovalix(layers, width=48, vocab=101, groups=3, side=8, eps=1e-5):
             "vocab": vocab, "width": width}
 
 
+# ---- Zikezen
+def scaled_rot(dims=8, base=700.0, factor=5.0, low=1.0, high=3.5, original=60):
+    return {"dims": dims, "base": base, "scaling": {"factor": factor, "low": low, "high": high, "original": original}}
+
+
+def sink_attention(heads=4, kv_heads=2, dim=16, vdim=24, scale=0.4, size=20, rot=None):
+    return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "mask": {"size": size},
+            "rot": rot or scaled_rot()}
+
+
+def gated(heads=2, dim=24, vdim=40, tau=12.0):
+    return {"heads": heads, "dim": dim, "vdim": vdim, "tau": tau}
+
+
+def beside(left=None, right=None, ff=72, scales=(0.7, 1.3), experts=None):
+    """`experts`: (number, chosen), of width ff each."""
+    mlp = None if ff is None else {"kind": "dense", "ff": ff}
+    if experts:
+        mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts[0], "top": experts[1]}}
+    return {"type": "parallel", "mlp": mlp, "mixer": {"left": left or sink_attention(), "right": right or gated(),
+                                                      "left_scale": scales[0], "right_scale": scales[1]}}
+
+
+def zikezen(layers, width=48, vocab=101, loop=None, side=8, eps=1e-5, cap=12.0, scale=1.7, positions=512):
+    return {"architecture": "Zikezen", "embedding": {"scale": scale}, "layers": layers, "logit_softcap": cap,
+            "loop": None if loop is None else dict(zip(("start", "stop", "times"), loop)), "max_positions": positions,
+            "norm": {"eps": eps}, "token_side": {"dim": side}, "vocab": vocab, "width": width}
+
+
 # sizes apart from each other, layers with and without feed-forward, loops and none, one stream and several, odd widths;
 # "wide" has the head sizes and widths of the tensor-core kernels
 CASES = {
@@ -81,6 +110,20 @@ CASES = {
     "tiles": tovalix([rotary(6, 3, 64, 64, rot=32, chunk=70, scale=0.3, cap=9.0, ff=128), wkv(2, 64, ff=96), hgrn2(2, 104, 136, ff=64),
                       rotary(3, 3, 64, 64, rot=32, chunk=130, scale=0.3, cap=12.0, kv_from=0, ff=None), wkv(1, 128, ff=None)],
                      width=128, vocab=300, groups=4, side=16),
+    # a loop over the middle layers, unequal mixers, experts and no feed-forward, the loop's first layer without one before it
+    "looped": zikezen([beside(ff=40, experts=(6, 2)), beside(sink_attention(heads=2, kv_heads=2, size=7), gated(3, 16, 24), ff=None,
+                                                             scales=(1.1, 0.4)),
+                       beside(right=gated(1, 8, 16, tau=1.0), ff=56, experts=(5, 5)), beside()], loop=(0, 3, 3)),
+    # widths that fit no vector load or tensor-core tile, one rotated pair, no scaled frequencies, one expert of many
+    "ragged": zikezen([beside(sink_attention(3, 1, 10, 6, size=33, rot={"dims": 2, "base": 40.0}), gated(2, 7, 9, tau=5.0), ff=31),
+                       beside(sink_attention(3, 3, 6, 14, size=70, rot=scaled_rot(dims=6)), gated(1, 30, 6), ff=13, experts=(9, 1)),
+                       beside(ff=None)], width=36, vocab=67, side=3, eps=1e-3, loop=(1, 2, 2), cap=4.0),
+    # the sizes of the tensor-core kernels: heads that are stored wider than they are, whole heads, experts
+    "blocks": zikezen([beside(sink_attention(6, 3, 40, 56, size=70, scale=0.2, rot=scaled_rot(dims=24)), gated(2, 40, 72), ff=64,
+                              experts=(7, 3)),
+                       beside(sink_attention(4, 1, 96, 80, size=130, scale=0.15, rot=scaled_rot(dims=96)), gated(1, 104, 136), ff=96),
+                       beside(sink_attention(2, 2, 128, 128, size=65, scale=0.1, rot=scaled_rot(dims=64)), gated(3, 64, 64), ff=40,
+                              experts=(40, 2))], width=128, vocab=300, side=16, loop=(1, 3, 2)),
 }
 
 
@@ -89,6 +132,8 @@ def weights(cfg, seed=0, buckets=11):
     large and attention is sharp, so that far tokens, window and chunk edges and kept tokens matter."""
     if cfg["architecture"] == "Tovalix":
         return tovalix_weights(cfg, seed)
+    if cfg["architecture"] == "Zikezen":
+        return zikezen_weights(cfg, seed)
     g = torch.Generator().manual_seed(seed)
     w = {}
 
@@ -205,6 +250,58 @@ def tovalix_weights(cfg, seed=0, rank=6):
             put(p + "mlp.up", ff, D)
             put(p + "mlp.down", D, ff)
             put(p + "mlp.act", 2, std=1.0)
+        put(p + "side.gate", dim, D)
+        put(p + "side.proj", D, dim)
+        put(p + "side.norm", D, std=0.3)
+    return w
+
+
+def zikezen_weights(cfg, seed=0, rank=8):
+    g = torch.Generator().manual_seed(seed)
+    w = {}
+
+    def put(name, *shape, std=None, mean=0.0):
+        std = (shape[-1] ** -0.5 if len(shape) > 1 else 0.2) if std is None else std
+        w[name] = (mean + std * torch.randn(*shape, generator=g)).to(torch.bfloat16).float()
+
+    D, V, dim, n = cfg["width"], cfg["vocab"], cfg["token_side"]["dim"], len(cfg["layers"])
+    if D % 8:
+        rank = 5
+    put("embed", V, D, std=0.5)
+    put("pos", cfg["max_positions"], D, std=0.4)
+    put("side.embed", V, n * dim, std=1.0)
+    put("head", V, D, std=3.0 * D ** -0.5)
+    put("final.norm", D, mean=1.0)
+    for i, layer in enumerate(cfg["layers"]):
+        p, a, r, mlp = f"l{i}.", layer["mixer"]["left"], layer["mixer"]["right"], layer["mlp"]
+        for s in ("norm1", "norm1b") + (() if mlp is None else ("norm2", "norm2b")):
+            put(p + s, D, mean=1.0)
+        H, G = a["heads"], a["kv_heads"]
+        for s, rows in (("q", H * a["dim"]), ("k", G * a["dim"]), ("v", G * a["vdim"])):
+            put(f"{p}mix.left.{s}", rows, D)
+            put(f"{p}mix.left.{s}.b", rows, std=0.5)
+        put(p + "mix.left.q.norm", a["dim"], mean=1.3, std=0.5)
+        put(p + "mix.left.k.norm", a["dim"], mean=1.3, std=0.5)
+        put(p + "mix.left.o", D, H * a["vdim"])
+        K, C = r["heads"] * r["dim"], r["heads"] * r["vdim"]
+        for s, rows in (("q", K), ("k", K), ("v", C), ("g", C)):
+            put(f"{p}mix.right.{s}", rows, D)
+        put(p + "mix.right.a1", rank, D)
+        put(p + "mix.right.a2", K, rank, std=0.7)
+        put(p + "mix.right.a2.b", K, std=3.0)
+        put(p + "mix.right.norm", r["vdim"], mean=1.0)
+        put(p + "mix.right.o", D, C)
+        if mlp is not None and mlp["kind"] == "dense":
+            for s, shape in (("gate", (mlp["ff"], D)), ("up", (mlp["ff"], D)), ("down", (D, mlp["ff"]))):
+                put(f"{p}mlp.{s}", *shape)
+        elif mlp is not None:
+            F, E = mlp["expert"]["ff"], mlp["router"]["experts"]
+            for e in range(E):
+                for s, shape in (("gate", (F, D)), ("up", (F, D)), ("down", (D, F))):
+                    put(f"{p}mlp.e{e}.{s}", *shape)
+            # scores spread enough that rounding rarely changes a choice
+            put(p + "mlp.router", E, D, std=3.0 * D ** -0.5)
+            put(p + "mlp.correction", E, std=0.3, mean=0.5)
         put(p + "side.gate", dim, D)
         put(p + "side.proj", D, dim)
         put(p + "side.norm", D, std=0.3)

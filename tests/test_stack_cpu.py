@@ -9,6 +9,7 @@ import torch
 from tests import roluzen_oracle as O
 from tests import stack_cases as C
 from tests import tovalix_oracle as TO
+from tests import zikezen_oracle as ZO
 
 
 @pytest.mark.parametrize("name", sorted(C.CASES))

@@ -46,6 +46,9 @@ struct AttnArgs {
   int keep;                  // with a window: the first `keep` tokens of a sequence stay visible
   const float* bias;         // [N, far + 1] added to the score of a key at distance min(distance, far), or null
   int far;
+  int vd;                    // paged: value columns of a head that are written (heads may be stored with zeros behind them)
+  float sink2;               // paged: one more score without a value in the sum of the weights, in log2 units (-inf: none)
+  float out_scale;           // paged: factor of the output
 };
 
 template <int H>
@@ -341,8 +344,9 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     if (ok && nblk > 0)
       ok = mbar_wait_bounded(barPV, (nblk - 1) & 1, abort_flag, a.status, ST_TIMEOUT_EPILOGUE);
     tc_fence_after();
-    const float inv_l = (l > 0.f) ? 1.f / l : 0.f;
-    __nv_bfloat16* orow = a.O + (long long)(row0 + r) * a.ldo + (long long)n * H;
+    const int vd = PAGED ? a.vd : H;
+    const float inv_l = PAGED ? a.out_scale / (l + exp2f(a.sink2 - m_used)) : (l > 0.f) ? 1.f / l : 0.f;
+    __nv_bfloat16* orow = a.O + (long long)(row0 + r) * a.ldo + (long long)n * vd;
 #pragma unroll 1
     for (int c = 0; c < H / 32; ++c) {
       uint32_t o[32];
@@ -356,6 +360,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       if (row_valid) {
 #pragma unroll
         for (int g = 0; g < 4; ++g) {
+          if (PAGED && c * 32 + g * 8 >= vd) break;
           uint4 v;
           v.x = pack_bf16(__uint_as_float(o[8 * g + 0]) * inv_l, __uint_as_float(o[8 * g + 1]) * inv_l);
           v.y = pack_bf16(__uint_as_float(o[8 * g + 2]) * inv_l, __uint_as_float(o[8 * g + 3]) * inv_l);
@@ -842,17 +847,21 @@ static int launch_fwd_paged(const void* q, const void* k, const void* v, const A
 // Causal attention of the query tiles (at most 128 rows of one entry each) of a ragged batch over paged keys and values:
 // q / out [n, N * H]; pools [pool_rows, KH * H] with page_size a multiple of 64; a key block of 64 tokens lies in one page
 // and is fetched by TMA through the page table. window, chunk <= 0: none; softcap <= 0: none. The unused tail of a page must hold finite values.
-TB_API int tb_attn_fwd_paged(const void* q, const void* k_pool, const void* v_pool, void* out, int n, long long pool_rows, int N,
-                             int KH, int H, float scale, float softcap, int window, int chunk, int keep, const float* bias, int far, const int* cu,
+// sink: one more score without a value in the sum of the weights (-inf: none). out [n, ldo], 16-byte aligned, head h at columns
+// h * vd (the first vd <= H value columns, a multiple of 8), times out_scale.
+TB_API int tb_attn_fwd_paged(const void* q, const void* k_pool, const void* v_pool, void* out, long long ldo, int n, long long pool_rows, int N,
+                             int KH, int H, int vd, float scale, float softcap, int window, int chunk, int keep, float sink,
+                             float out_scale, const float* bias, int far, const int* cu,
                              const int* slot, const int* pos0, const int* tile_t0, const int* tile_ent, int tiles,
                              const int* table, int max_pages, int page_size, int* status, cudaStream_t stream) {
   if (n <= 0 || tiles <= 0) return 0;
-  if (KH <= 0 || N % KH || page_size % BKV || N > 65535) return -2;
+  if (KH <= 0 || N % KH || page_size % BKV || N > 65535 || vd <= 0 || vd > H || vd % 8 || ldo % 8 || ((uintptr_t)out & 15)) return -2;
   AttnArgs a = {};
+  a.vd = vd; a.sink2 = sink * LOG2E; a.out_scale = out_scale;
   a.N = N; a.KH = KH; a.scale = scale; a.causal = 1; a.window = window > 0 ? window : 0;
   a.softcap = softcap; a.chunk = chunk > 0 ? chunk : 0;
   a.keep = a.window > 0 || a.chunk > 0 ? keep : 0; a.bias = bias; a.far = far;
-  a.O = reinterpret_cast<__nv_bfloat16*>(out); a.ldo = (long long)N * H; a.status = status;
+  a.O = reinterpret_cast<__nv_bfloat16*>(out); a.ldo = ldo; a.status = status;
   a.cu = cu; a.slot = slot; a.pos0 = pos0; a.tile_t0 = tile_t0; a.tile_ent = tile_ent; a.table = table;
   a.max_pages = max_pages; a.page_size = page_size;
   switch (H) {

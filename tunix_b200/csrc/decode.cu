@@ -153,7 +153,8 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_consta
                     const __nv_bfloat16* __restrict__ k_pool, const __nv_bfloat16* __restrict__ v_pool,
                     const int* __restrict__ page_table, int max_pages, int page_size,
                     const int* __restrict__ seq_ids, const int* __restrict__ seq_lens, int KH, int G, float scale,
-                    float softcap, int window, int chunk, int keep, const float* __restrict__ bias, int far,   // bias [N, far + 1] or null
+                    float softcap, int window, int chunk, int keep, float sink, float out_scale, int vd,
+                    const float* __restrict__ bias, int far,                   // bias [N, far + 1] or null
                     int num_splits, int split_tokens,
                     float* __restrict__ part_acc,                                               // [B, N, splits, H]
                     float* __restrict__ part_ml,                                                // [B, N, splits, 2]
@@ -178,8 +179,8 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_consta
   const int n_tiles = min(kt.total - tile0, split_tokens / TILE_KEYS);
   if (len <= 0 || n_tiles <= 0) { // past the end of this sequence: the combine kernel never reads this split
     if (num_splits == 1)          // (an empty slot with a single split: its output row is zero)
-      for (int idx = threadIdx.x; idx < G * H; idx += 128)
-        out[(long long)b * ldo + (long long)(kh * G) * H + idx] = __float2bfloat16(0.f);
+      for (int idx = threadIdx.x; idx < G * vd; idx += 128)
+        out[(long long)b * ldo + (long long)(kh * G) * vd + idx] = __float2bfloat16(0.f);
     return;
   }
   auto visible = [&](int t) { return t < len && (t >= kt.w_lo || t < keep); };
@@ -356,6 +357,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_consta
   __syncthreads();
   for (int idx = tid; idx < G * H; idx += 128) {
     const int g = idx / H, d = idx - g * H;
+    if (d >= vd) continue;
     float mm = -INFINITY;
 #pragma unroll
     for (int w = 0; w < 4; ++w) mm = fmaxf(mm, sm_m[w][g]);
@@ -367,7 +369,8 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_consta
       aa += sm_acc[(w * 16 + g) * H + d] * c;
     }
     if (num_splits == 1) {                 // the whole context in this CTA: no partial state, no combine kernel
-      out[(long long)b * ldo + (long long)(kh * G + g) * H + d] = __float2bfloat16(ll > 0.f ? aa / ll : 0.f);
+      ll += __expf(sink - mm);
+      out[(long long)b * ldo + (long long)(kh * G + g) * vd + d] = __float2bfloat16(ll > 0.f ? out_scale * aa / ll : 0.f);
       continue;
     }
     const long long oidx = (((long long)b * N + kh * G + g) * num_splits + split);
@@ -379,10 +382,11 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_consta
   }
 }
 
-// out[b, n, :] = sum_s acc_s * exp(m_s - M) / sum_s l_s * exp(m_s - M)
+// out[b, n, :vd] = out_scale * sum_s acc_s * exp(m_s - M) / (exp(sink - M) + sum_s l_s * exp(m_s - M))
 __global__ void paged_decode_combine_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
                                             const int* __restrict__ seq_lens, int N, int H, int num_splits, int split_tokens,
-                                            int window, int chunk, int keep, __nv_bfloat16* __restrict__ out, long long ldo) {
+                                            int window, int chunk, int keep, float sink, float out_scale, int vd,
+                                            __nv_bfloat16* __restrict__ out, long long ldo) {
   pdl_trigger();
   pdl_wait();
   const int b = blockIdx.x, n = blockIdx.y;
@@ -392,19 +396,19 @@ __global__ void paged_decode_combine_kernel(const float* __restrict__ part_acc, 
   const long long base = ((long long)b * N + n) * num_splits;
   float M = -INFINITY;
   for (int s = 0; s < used; ++s) M = fmaxf(M, part_ml[(base + s) * 2]);
-  float L = 0.f;
+  float L = used > 0 ? __expf(sink - M) : 0.f;
   for (int s = 0; s < used; ++s) {
     const float ms = part_ml[(base + s) * 2];
     if (ms != -INFINITY) L += part_ml[(base + s) * 2 + 1] * __expf(ms - M);
   }
-  const float inv = L > 0.f ? 1.f / L : 0.f;
-  for (int d = threadIdx.x; d < H; d += blockDim.x) {
+  const float inv = L > 0.f ? out_scale / L : 0.f;
+  for (int d = threadIdx.x; d < vd; d += blockDim.x) {
     float a = 0.f;
     for (int s = 0; s < used; ++s) {
       const float ms = part_ml[(base + s) * 2];
       if (ms != -INFINITY) a += part_acc[(base + s) * H + d] * __expf(ms - M);
     }
-    out[(long long)b * ldo + (long long)n * H + d] = __float2bfloat16(a * inv);
+    out[(long long)b * ldo + (long long)n * vd + d] = __float2bfloat16(a * inv);
   }
 }
 
@@ -412,7 +416,7 @@ template <int H, bool TMA, int STAGES>
 int launch_decode_v(int G, dim3 grid, cudaStream_t stream, const CUtensorMap& tmK, const CUtensorMap& tmV,
                     const __nv_bfloat16* q, long long ldq, const __nv_bfloat16* kp, const __nv_bfloat16* vp, const int* pt,
                     int max_pages, int page_size, const int* seq_ids, const int* seq_lens, int KH, float scale, float softcap,
-                    int window, int chunk, int keep, const float* bias, int far, int splits, int split_tokens, float* pa, float* pml,
+                    int window, int chunk, int keep, float sink, float out_scale, int vd, const float* bias, int far, int splits, int split_tokens, float* pa, float* pml,
                     __nv_bfloat16* out, long long ldo, int* status) {
   constexpr int TILE2 = 2 * TILE_KEYS * H * 2;                       // one stage: a K tile and a V tile
   constexpr int SMEM = STAGES * TILE2 + (TMA ? 1024 : 0);
@@ -423,7 +427,7 @@ int launch_decode_v(int G, dim3 grid, cudaStream_t stream, const CUtensorMap& tm
   // a split of one 64-key tile needs one stage only: more CTAs fit on an SM
   const int smem = split_tokens > TILE_KEYS ? SMEM : TILE2 + (TMA ? 1024 : 0);
   return launch_pdl(paged_decode_kernel<H, TMA, STAGES>, grid, dim3(128), smem, stream, tmK, tmV, q, ldq, kp, vp, pt, max_pages,
-                    page_size, seq_ids, seq_lens, KH, G, scale, softcap, window, chunk, keep, bias, far, splits, split_tokens, pa, pml, out, ldo,
+                    page_size, seq_ids, seq_lens, KH, G, scale, softcap, window, chunk, keep, sink, out_scale, vd, bias, far, splits, split_tokens, pa, pml, out, ldo,
                     status) == cudaSuccess ? 0 : -5;
 }
 
@@ -432,7 +436,8 @@ template <int H>
 int launch_decode(int G, dim3 grid, cudaStream_t stream, const __nv_bfloat16* q, long long ldq,
                   const __nv_bfloat16* kp, const __nv_bfloat16* vp, long long pool_rows, const int* pt, int max_pages,
                   int page_size, const int* seq_ids, const int* seq_lens, int KH, float scale, float softcap, int window,
-                  int chunk, int keep, const float* bias, int far, int splits, int split_tokens, float* pa, float* pml, __nv_bfloat16* out,
+                  int chunk, int keep, float sink, float out_scale, int vd, const float* bias, int far, int splits, int split_tokens, float* pa,
+                  float* pml, __nv_bfloat16* out,
                   long long ldo, int* status) {
   static const bool no_tma = getenv("TUNIX_B200_DECODE_NO_TMA") != nullptr;
   static const char* stages_env = getenv("TUNIX_B200_DECODE_STAGES");
@@ -443,7 +448,7 @@ int launch_decode(int G, dim3 grid, cudaStream_t stream, const __nv_bfloat16* q,
                    tb_make_tmap_2d_bf16(&tmK, kp, (uint64_t)pool_rows, (uint64_t)KH * H, (uint64_t)KH * H, TILE_KEYS, 64, 1) == 0 &&
                    tb_make_tmap_2d_bf16(&tmV, vp, (uint64_t)pool_rows, (uint64_t)KH * H, (uint64_t)KH * H, TILE_KEYS, 64, 1) == 0;
 #define LD(T, S) launch_decode_v<H, T, S>(G, grid, stream, tmK, tmV, q, ldq, kp, vp, pt, max_pages, page_size, seq_ids, seq_lens, \
-                                         KH, scale, softcap, window, chunk, keep, bias, far, splits, split_tokens, pa, pml, out, ldo, status)
+                                         KH, scale, softcap, window, chunk, keep, sink, out_scale, vd, bias, far, splits, split_tokens, pa, pml, out, ldo, status)
   if (!tma) return LD(false, 2);
   // measured at head dim 128 (8 kv heads, 256 sequences x 768 tokens): 2 / 3 / 4 stages take 157 / 161 / 194 us,
   // cp.async staging 190 us: three CTAs per SM with two stages each beat deeper rings on fewer CTAs
@@ -499,14 +504,15 @@ TB_API int tb_qkv_post(void* qkv, long long ld, const int* seq_ids, const int* p
 // split_tokens = context tokens per CTA, a multiple of 64 in [64, 2048] (0 = 256). CTAs of splits that lie past the
 // end of their sequence return at once. pool_rows = num_pages * page_size (rows of the pools, for the tensor maps;
 // 0 = no TMA staging). window > 0: keys at distance < window, chunk > 0: keys of the query's chunk, and the sequence's first `keep` tokens. bias fp32
-// [N, far + 1] (null = none) is added to the scaled score of a key at distance min(distance, far). status: word that a bounded mbarrier wait writes its code to.
+// [N, far + 1] (null = none) is added to the scaled score of a key at distance min(distance, far). sink: one more score without a
+// value in the sum of the weights (-inf: none). out [B, ldo]: head n at columns n * vd, its first vd <= H value columns, times out_scale. status: word that a bounded mbarrier wait writes its code to.
 TB_API int tb_paged_decode(const void* q, long long ldq, const void* k_pool, const void* v_pool,
                            const int* page_table, int max_pages, int page_size, const int* seq_ids,
                            const int* seq_lens, int B, int N, int KH, int H, int max_ctx, float scale, float softcap,
-                           int window, int chunk, int keep, const float* bias, int far, int split_tokens, long long pool_rows,
-                           float* part_acc, float* part_ml, void* out, long long ldo, int* status, cudaStream_t stream) {
+                           int window, int chunk, int keep, float sink, float out_scale, int vd, const float* bias, int far,
+                           int split_tokens, long long pool_rows, float* part_acc, float* part_ml, void* out, long long ldo, int* status, cudaStream_t stream) {
   if (B <= 0) return 0;
-  if (KH <= 0 || N % KH || (ldq % 8)) return -2;
+  if (KH <= 0 || N % KH || (ldq % 8) || vd <= 0 || vd > H) return -2;
   const int G = N / KH;
   if (G > MAX_G) return -2;
   if (split_tokens <= 0) split_tokens = 256;
@@ -524,15 +530,15 @@ TB_API int tb_paged_decode(const void* q, long long ldq, const void* k_pool, con
   auto kp = (const __nv_bfloat16*)k_pool;
   auto vp = (const __nv_bfloat16*)v_pool;
   switch (H) {
-    case 64: rc = launch_decode<64>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, chunk, keep, bias, far, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
-    case 128: rc = launch_decode<128>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, chunk, keep, bias, far, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
-    case 256: rc = launch_decode<256>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, chunk, keep, bias, far, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
+    case 64: rc = launch_decode<64>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, chunk, keep, sink, out_scale, vd, bias, far, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
+    case 128: rc = launch_decode<128>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, chunk, keep, sink, out_scale, vd, bias, far, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
+    case 256: rc = launch_decode<256>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, chunk, keep, sink, out_scale, vd, bias, far, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
     default: return -2;
   }
   if (rc) return rc;
   if (splits == 1) return 0;
   return launch_pdl(paged_decode_combine_kernel, dim3(B, N), dim3(128), 0, stream, (const float*)part_acc,
-                    (const float*)part_ml, seq_lens, N, H, splits, split_tokens, window, chunk, keep, (__nv_bfloat16*)out, ldo) == cudaSuccess ? 0 : -5;
+                    (const float*)part_ml, seq_lens, N, H, splits, split_tokens, window, chunk, keep, sink, out_scale, vd, (__nv_bfloat16*)out, ldo) == cudaSuccess ? 0 : -5;
 }
 
 // ------------------------------------------------------------------ per-step bookkeeping of the decode loop

@@ -4,10 +4,12 @@
 // What makes f, k and the read-out differs per mechanism (MODE):
 //   BONUS (RWKV time mixing)  f = exp(-exp(z + c0)); o = (S_before + diag(c1) k v^T)^T q
 //   LOWER (HGRN2)             f = c1 + (1 - c1) sigmoid(z + c0), k = 1 - f, q = silu(q); o = S^T q
+//   ROOT (gated linear attention)  f = sigmoid(z + c0)^(1 / tau), q times a constant; o = S^T q
 // with z fp32 from a projection and c0, c1 parameters per head and channel. Then every head's o is divided by its root mean
-// square over dv, weighted (one weight for all heads or one per head), and gated by silu if there is a gate.
+// square over dv, weighted (one weight for all heads or one per head), gated by silu if there is a gate, and scaled.
 //
-//   gla_step  : one token per entry. The state streams through registers once; norm and gate in the same launch.
+//   gla_step  : one token per entry. The state streams through registers once; norm and gate in the same launch. z may be given
+//               as the product of a short row per token (a bottleneck) with a weight row per channel, which is formed here.
 //   gla_chunk : portions of prompts, bf16, on tensor cores (below).
 //   gla_seq   : token by token, any sizes, also 32-bit; head_norm after it.
 //
@@ -20,14 +22,21 @@ using namespace tb;
 namespace {
 
 typedef __nv_bfloat16 bf;
-enum Mode { BONUS = 0, LOWER = 1 };
+enum Mode { BONUS = 0, LOWER = 1, ROOT = 2 };
+__host__ __device__ constexpr bool has_keys(int mode) { return mode != LOWER; }      // else made from the gates
+__host__ __device__ constexpr bool reads_after(int mode) { return mode != BONUS; }   // the read-out sees the token's own update
 
 struct GlaArgs {
   const void *q, *k, *v, *gate;       // T [n, ld*], head h at columns h * dk or h * dv; k null with LOWER, gate may be null
   long long ldq, ldk, ldv, ldg;
-  const float* z;                     // fp32 [n, ldz]
+  const float* z;                     // fp32 [n, ldz], or null (gla_step): z = w2 x
   long long ldz;
-  const void *c0, *c1;                // T [heads * dk]
+  const void* x;                      // T [n, ldx], the first `rank` columns
+  const void* w2;                     // T [heads * dk, rank]
+  long long ldx;
+  int rank;
+  const void *c0, *c1;                // T [heads * dk]; c1 not with ROOT
+  float qscale, inv_tau;              // ROOT
   int heads, dk, dv;
   Ragged rb;
   float* S;                           // fp32 [slots, heads, dk, dv]
@@ -38,13 +47,16 @@ struct GlaArgs {
   // output norm
   const void* nw;                     // T [dv] or [heads * dv]
   int per_head;
-  float eps;
+  float eps, out_scale;
+  long long ldo;                      // row stride of the output
 };
 
 template <int MODE>
-__device__ __forceinline__ void gates_exact(float z, float c0, float c1, float& f, float& k) {
+__device__ __forceinline__ void gates_exact(const GlaArgs& a, float z, float c0, float c1, float& f, float& k) {
   if (MODE == BONUS) {
     f = decay_exp(-expf(z + c0));
+  } else if (MODE == ROOT) {
+    f = decay_exp(log_sigmoid(z + c0) * a.inv_tau);
   } else {
     // near 1 the decay is rounded once: 1 - k
     k = (1.f - c1) * sigmoid(-(z + c0));
@@ -55,10 +67,11 @@ __device__ __forceinline__ void gates_exact(float z, float c0, float c1, float& 
 template <int MODE>
 __device__ __forceinline__ float gates_offset(float c0) { return c0 * LOG2_E + (MODE == BONUS ? 0.5287663729448977f : 0.f); }   // + log2(log2 e)
 template <int MODE>
-__device__ __forceinline__ float gates_log2(float z, float b0, float c1, float& k) {
-  const float e = quick_exp2(fminf(fmaf(z, LOG2_E, b0), 100.f));
+__device__ __forceinline__ float gates_log2(const GlaArgs& a, float z, float b0, float c1, float& k) {
+  const float y = fmaf(z, LOG2_E, b0), e = quick_exp2(fminf(y, 100.f));
   if (MODE == BONUS) return -fminf(e, 150.f);
   const float s = quick_rcp(1.f + e), r = 1.f - c1;    // sigmoid of the negative; e s: of the positive
+  if (MODE == ROOT) return fmaxf((y > 0.f ? quick_log2_decay(s, 1.f) : y - quick_log2(1.f + e)) * a.inv_tau, -150.f);
   k = r * s;
   return quick_log2_decay(k, fmaf(r, e * s, c1));
 }
@@ -66,6 +79,25 @@ __device__ __forceinline__ float gates_log2(float z, float b0, float c1, float& 
 template <typename T>
 __device__ __forceinline__ float silu(float z) {
   return z * (sizeof(T) == 2 ? quick_sigmoid(z) : sigmoid(z));
+}
+
+// z of channel c for token t from its bottleneck row
+template <typename T>
+__device__ __forceinline__ float low_rank(const GlaArgs& a, int t, int c) {
+  const T *x = static_cast<const T*>(a.x) + t * a.ldx, *w = static_cast<const T*>(a.w2) + (long long)c * a.rank;
+  float z = 0.f;
+  int r = 0;
+  if (sizeof(T) == 2 && a.rank % 8 == 0 && ((uintptr_t)x & 15) == 0) {
+    for (; r < a.rank; r += 8) {
+      float xv[8], wv[8];
+      load_v<8>(x + r, xv);
+      load_v<8>(w + r, wv);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) z += xv[i] * wv[i];
+    }
+  }
+  for (; r < a.rank; ++r) z += to_f(x[r]) * to_f(w[r]);
+  return z;
 }
 
 template <typename T>
@@ -92,7 +124,7 @@ gla_step_kernel(const GlaArgs a, T* __restrict__ out) {
   pdl_trigger();
   pdl_wait();
   const int p0 = a.rb.pos0[e];
-  T* o = out + ((long long)e * a.heads + hd) * dv;
+  T* o = out + e * a.ldo + hd * dv;
   if (p0 < 0) {
     for (int c = tid; c < dv; c += GT) o[c] = from_f<T>(0.f);
     return;
@@ -101,11 +133,12 @@ gla_step_kernel(const GlaArgs a, T* __restrict__ out) {
   float* S = a.S + ((long long)a.rb.slot[e] * a.heads + hd) * dk * dv;
   for (int d = tid; d < dk; d += GT) {
     const int c = hd * dk + d;
-    const float c1 = to_f(static_cast<const T*>(a.c1)[c]);
+    const float c1 = MODE == ROOT ? 0.f : to_f(static_cast<const T*>(a.c1)[c]);
     float q = to_f(static_cast<const T*>(a.q)[e * a.ldq + c]), k = 0.f, f;
-    if (MODE == BONUS) k = to_f(static_cast<const T*>(a.k)[e * a.ldk + c]);
-    else q = silu<T>(q);
-    gates_exact<MODE>(a.z[e * a.ldz + c], to_f(static_cast<const T*>(a.c0)[c]), c1, f, k);
+    if (has_keys(MODE)) k = to_f(static_cast<const T*>(a.k)[e * a.ldk + c]);
+    if (MODE == LOWER) q = silu<T>(q);
+    if (MODE == ROOT) q *= a.qscale;
+    gates_exact<MODE>(a, a.z ? a.z[e * a.ldz + c] : low_rank<T>(a, e, c), to_f(static_cast<const T*>(a.c0)[c]), c1, f, k);
     qs[d] = q;
     ks[d] = k;
     fs[d] = f;
@@ -138,9 +171,9 @@ gla_step_kernel(const GlaArgs a, T* __restrict__ out) {
           const float k = ks[d], f = fs[d], q = qs[d], uk = us[d] * k;
 #pragma unroll
           for (int i = 0; i < V; ++i) {
-            if (MODE == BONUS) acc[i] += q * (s[j][i] + uk * v[i]);
+            if (!reads_after(MODE)) acc[i] += q * (s[j][i] + uk * v[i]);
             s[j][i] = f * s[j][i] + k * v[i];
-            if (MODE == LOWER) acc[i] += q * s[j][i];
+            if (reads_after(MODE)) acc[i] += q * s[j][i];
           }
           store_v<V>(S + (long long)d * dv + col, s[j]);
         }
@@ -157,7 +190,7 @@ gla_step_kernel(const GlaArgs a, T* __restrict__ out) {
     ss += x * x;
   }
   ss = block_sum(ss, red);
-  const float rstd = 1.f / sqrtf(ss / (float)dv + a.eps);
+  const float rstd = a.out_scale / sqrtf(ss / (float)dv + a.eps);
   for (int c = tid; c < dv; c += GT) {
     float x = part[c] * rstd * to_f(static_cast<const T*>(a.nw)[a.per_head ? hd * dv + c : c]);
     if (a.gate) x *= silu<T>(to_f(static_cast<const T*>(a.gate)[e * a.ldg + hd * dv + c]));
@@ -199,11 +232,12 @@ gla_seq_kernel(const GlaArgs a, float* __restrict__ out) {
   for (int t = t0; t < t1; ++t) {
     for (int d = tid; d < dk; d += GT) {
       const int c = hd * dk + d;
-      const float c1 = to_f(static_cast<const T*>(a.c1)[c]);
+      const float c1 = MODE == ROOT ? 0.f : to_f(static_cast<const T*>(a.c1)[c]);
       float q = to_f(static_cast<const T*>(a.q)[t * a.ldq + c]), k = 0.f, f;
-      if (MODE == BONUS) k = to_f(static_cast<const T*>(a.k)[t * a.ldk + c]);
-      else q = silu<T>(q);
-      gates_exact<MODE>(a.z[t * a.ldz + c], to_f(static_cast<const T*>(a.c0)[c]), c1, f, k);
+      if (has_keys(MODE)) k = to_f(static_cast<const T*>(a.k)[t * a.ldk + c]);
+      if (MODE == LOWER) q = silu<T>(q);
+      if (MODE == ROOT) q *= a.qscale;
+      gates_exact<MODE>(a, a.z[t * a.ldz + c], to_f(static_cast<const T*>(a.c0)[c]), c1, f, k);
       qs[d] = q;
       ks[d] = k;
       fs[d] = f;
@@ -254,7 +288,7 @@ head_norm_kernel(const GlaArgs a, const float* __restrict__ o, T* __restrict__ o
 #pragma unroll
       for (int i = 0; i < V; ++i) ss += v[i] * v[i];
     }
-    const float r = 1.f / sqrtf(warp_sum(ss) / (float)dv + a.eps);
+    const float r = a.out_scale / sqrtf(warp_sum(ss) / (float)dv + a.eps);
     for (int c = lane * V; c < dv; c += 32 * V) {
       float v[V], ww[V], g[V];
       load_v<V>(x + c, v);
@@ -262,7 +296,7 @@ head_norm_kernel(const GlaArgs a, const float* __restrict__ o, T* __restrict__ o
       if (gate) load_v<V>(gate + hd * dv + c, g);
 #pragma unroll
       for (int i = 0; i < V; ++i) v[i] *= r * ww[i] * (gate ? silu<T>(g[i]) : 1.f);
-      store_v<V>(out + t * a.heads * dv + hd * dv + c, v);
+      store_v<V>(out + t * a.ldo + hd * dv + c, v);
     }
   }
 }
@@ -332,7 +366,7 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
   float* Sg = a.S + (slot * a.heads + hd) * dk * dv + c0;
 
   const bf* qg = static_cast<const bf*>(a.q) + (long long)t0 * a.ldq + hd * dk;
-  const bf* kg = MODE == BONUS ? static_cast<const bf*>(a.k) + (long long)t0 * a.ldk + hd * dk : nullptr;
+  const bf* kg = has_keys(MODE) ? static_cast<const bf*>(a.k) + (long long)t0 * a.ldk + hd * dk : nullptr;
   const bf* vg = static_cast<const bf*>(a.v) + (long long)t0 * a.ldv + hd * dv + c0;
   const float* zg = a.z + (long long)t0 * a.ldz + hd * dk;
   const bf* gg = a.gate ? static_cast<const bf*>(a.gate) + (long long)t0 * a.ldg + hd * dv + c0 : nullptr;
@@ -348,7 +382,7 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
       const int r = i / (KP / 8), c = i % (KP / 8);
       const bool ok = r < rows && c * 8 < dk;
       cp_async16(sb + M.q + r * M.pitch + c * 16, qg + (ok ? (at + r) * a.ldq + c * 8 : 0), ok ? 16 : 0);
-      if (MODE == BONUS) cp_async16(sb + M.k + r * M.pitch + c * 16, kg + (ok ? (at + r) * a.ldk + c * 8 : 0), ok ? 16 : 0);
+      if (has_keys(MODE)) cp_async16(sb + M.k + r * M.pitch + c * 16, kg + (ok ? (at + r) * a.ldk + c * 8 : 0), ok ? 16 : 0);
     }
     for (int i = tid; i < TT * (KP / 4); i += NT) {
       const int r = i / (KP / 4), c = i % (KP / 4);
@@ -382,7 +416,7 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
   for (int i = 0; i < 2; ++i) {
     const bool ok = pd + i < dk;
     b0[i] = gates_offset<MODE>(ok ? to_f(static_cast<const bf*>(a.c0)[hd * dk + pd + i]) : 0.f);
-    b1[i] = ok ? to_f(static_cast<const bf*>(a.c1)[hd * dk + pd + i]) : (MODE == LOWER ? 1.f : 0.f);
+    b1[i] = MODE == ROOT ? 0.f : ok ? to_f(static_cast<const bf*>(a.c1)[hd * dk + pd + i]) : (MODE == LOWER ? 1.f : 0.f);
   }
 
   const int tiles = (len + TT - 1) / TT;
@@ -398,8 +432,8 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
       const int row = psub * 16 + t;
       const float2 z = *reinterpret_cast<const float2*>(Z + row * KP + pd);
       float2 k;
-      l[t][0] = gates_log2<MODE>(z.x, b0[0], b1[0], k.x);
-      l[t][1] = gates_log2<MODE>(z.y, b0[1], b1[1], k.y);
+      l[t][0] = gates_log2<MODE>(a, z.x, b0[0], b1[0], k.x);
+      l[t][1] = gates_log2<MODE>(a, z.y, b0[1], b1[1], k.y);
       if (row >= rows) l[t][0] = l[t][1] = k.x = k.y = 0.f;
       // keys made from the gates take the place of z: only the sums stay in registers
       if (MODE == LOWER) *reinterpret_cast<float2*>(smem + M.z + (row * KP + pd) * 4) = k;
@@ -412,6 +446,7 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
       q0 = bf16_lo(q2);
       q1 = bf16_hi(q2);
       if (MODE == LOWER) { q0 = silu<bf>(q0); q1 = silu<bf>(q1); }
+      if (MODE == ROOT) { q0 *= a.qscale; q1 *= a.qscale; }
     };
     auto keys = [&](int row) {                          // rows past the end hold zeros
       if (MODE == LOWER) return *reinterpret_cast<const float2*>(smem + M.z + (row * KP + pd) * 4);
@@ -467,7 +502,7 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
 #pragma unroll
       for (int t = 7; t >= 0; --t) {
         const float n0 = c0s + l[t][0], n1 = c1s + l[t][1];
-        scaled(t, MODE == LOWER ? -c0s : -n0, MODE == LOWER ? -c1s : -n1, c0s, c1s);
+        scaled(t, reads_after(MODE) ? -c0s : -n0, reads_after(MODE) ? -c1s : -n1, c0s, c1s);
         c0s = n0;
         c1s = n1;
       }
@@ -475,7 +510,7 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
 #pragma unroll
       for (int t = 8; t < 16; ++t) {
         const float n0 = c0s + l[t][0], n1 = c1s + l[t][1];
-        scaled(t, MODE == LOWER ? n0 : c0s, MODE == LOWER ? n1 : c1s, -n0, -n1);
+        scaled(t, reads_after(MODE) ? n0 : c0s, reads_after(MODE) ? n1 : c1s, -n0, -n1);
         c0s = n0;
         c1s = n1;
       }
@@ -490,7 +525,7 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
         float q0, q1;
         queries(row, q0, q1);
         const float2 k = keys(row);
-        *reinterpret_cast<uint32_t*>(smem + M.Q + at) = pack_bf16(q0 * quick_exp2(MODE == LOWER ? n0 : c0s), q1 * quick_exp2(MODE == LOWER ? n1 : c1s));
+        *reinterpret_cast<uint32_t*>(smem + M.Q + at) = pack_bf16(q0 * quick_exp2(reads_after(MODE) ? n0 : c0s), q1 * quick_exp2(reads_after(MODE) ? n1 : c1s));
         *reinterpret_cast<float2*>(smem + M.z + (row * KP + pd) * 4) = make_float2(n0, n1);
         *reinterpret_cast<uint32_t*>(smem + M.k + at) = pack_bf16(k.x, k.y);
         *reinterpret_cast<uint32_t*>(smem + M.q + at) = pack_bf16(q0, q1);
@@ -631,7 +666,7 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
             float s = 0.f;
 #pragma unroll
             for (int w = 0; w < WARPS; ++w) s += Ssq[w * TT + r];
-            rstd = rsqrtf(s / (float)dv + a.eps);
+            rstd = a.out_scale * rsqrtf(s / (float)dv + a.eps);
           }
 #pragma unroll
           for (int j = 0; j < 2; ++j) {
@@ -646,7 +681,7 @@ gla_chunk_kernel(const GlaArgs a, float* __restrict__ raw, bf* __restrict__ out)
                 y0 *= silu<bf>(bf16_lo(gate[sub][h][j]));
                 y1 *= silu<bf>(bf16_hi(gate[sub][h][j]));
               }
-              *reinterpret_cast<uint32_t*>(out + t * a.heads * dv + hd * dv + c) = pack_bf16(y0, y1);
+              *reinterpret_cast<uint32_t*>(out + t * a.ldo + hd * dv + c) = pack_bf16(y0, y1);
             }
           }
         }
@@ -687,17 +722,21 @@ int launch_step(const GlaArgs& a, T* out, cudaStream_t stream) {
   return launch_pdl(gla_step_kernel<T, MODE, V>, dim3(a.heads, a.rb.E), dim3(GT), smem, stream, a, out) == cudaSuccess ? 0 : -5;
 }
 
+bool aligned(const void* p, int bytes) { return ((uintptr_t)p & (bytes - 1)) == 0; }
+
 template <typename T, int MODE>
 int run(const GlaArgs& a, float* raw, T* out, int one, int chunked, cudaStream_t stream) {
   if (one) {
-    const bool vec = a.dv % 4 == 0 && a.ldv % 4 == 0 && a.dk % 4 == 0;
+    const bool vec = a.dv % 4 == 0 && a.ldv % 4 == 0 && a.dk % 4 == 0 && aligned(a.v, 4 * sizeof(T));
     if (vec && a.dv <= 4 * GT) return launch_step<T, MODE, 4>(a, out, stream);
     if (a.dv <= GT) return launch_step<T, MODE, 1>(a, out, stream);
   }
+  if (!a.z || !raw) return -2;
   bool sliced = false;
   if constexpr (sizeof(T) == 2) {
     if (chunked && !one && a.dk <= 128 && a.dk % 8 == 0 && a.dv % 8 == 0 && a.ldq % 8 == 0 && a.ldv % 8 == 0 && a.ldz % 4 == 0 &&
-        (MODE == LOWER || a.ldk % 8 == 0) && a.ldg % 2 == 0) {
+        (!has_keys(MODE) || (a.ldk % 8 == 0 && aligned(a.k, 16))) && a.ldg % 2 == 0 && a.ldo % 2 == 0 && aligned(a.q, 16) &&
+        aligned(a.v, 16) && aligned(a.z, 16) && aligned(a.gate, 4) && aligned(out, 4)) {
       const bool wide = a.dv > 64;
       const int rc = a.dk <= 64 ? (wide ? launch_chunk<64, MODE, 8>(a, raw, out, stream) : launch_chunk<64, MODE, 4>(a, raw, out, stream))
                                 : (wide ? launch_chunk<128, MODE, 8>(a, raw, out, stream) : launch_chunk<128, MODE, 4>(a, raw, out, stream));
@@ -714,7 +753,7 @@ int run(const GlaArgs& a, float* raw, T* out, int one, int chunked, cudaStream_t
     const dim3 grid((a.dv + SV - 1) / SV, a.heads, a.rb.E);
     if (launch_pdl(gla_seq_kernel<T, MODE>, grid, dim3(GT), smem, stream, a, raw) != cudaSuccess) return -5;
   }
-  const bool vec = a.dv % 4 == 0 && a.ldg % 4 == 0;
+  const bool vec = a.dv % 4 == 0 && a.ldg % 4 == 0 && a.ldo % 4 == 0 && aligned(a.gate, 4 * sizeof(T)) && aligned(out, 4 * sizeof(T));
   const dim3 grid(a.rb.n);
   const cudaError_t err = vec ? launch_pdl(head_norm_kernel<T, 4>, grid, dim3(256), 0, stream, a, (const float*)raw, out)
                               : launch_pdl(head_norm_kernel<T, 1>, grid, dim3(256), 0, stream, a, (const float*)raw, out);
@@ -723,21 +762,27 @@ int run(const GlaArgs& a, float* raw, T* out, int one, int chunked, cudaStream_t
 
 }  // namespace
 
-// mode: 0 BONUS, 1 LOWER. q, k [n, heads * dk], v, gate [n, heads * dv] (row strides ld*; k null with LOWER, gate may be null),
-// z fp32 [n, heads * dk] with row stride ldz; c0, c1 T [heads * dk]; S fp32 [slots, heads, dk, dv].
+// mode: 0 BONUS, 1 LOWER, 2 ROOT. q, k [n, heads * dk], v, gate [n, heads * dv] (row strides ld*; k null with LOWER, gate may be
+// null), z fp32 [n, heads * dk] with row stride ldz, or (with `one`) null: x T [n, rank] with row stride ldx times w2 T
+// [heads * dk, rank]; c0, c1 T [heads * dk] (c1 null with ROOT); qscale, inv_tau: ROOT's constants; S fp32 [slots, heads, dk, dv].
 // h T [n, D] / carry fp32 [slots, D] (or null): last rows of portions kept for the token shift (not with `one`).
-// nw T [dv], or [heads * dv] with per_head; raw fp32 [n, heads * dv] workspace; out T [n, heads * dv].
+// nw T [dv], or [heads * dv] with per_head; raw fp32 [n, heads * dv] workspace; out T [n, heads * dv] with row stride ldo, times
+// out_scale.
 // one: every entry is one token. chunked: bf16 portions take the tensor-core form where the sizes allow.
 TB_API int tb_gated_linear(int dtype, int mode, const void* q, long long ldq, const void* k, long long ldk, const void* v,
-                           long long ldv, const void* gate, long long ldg, const float* z, long long ldz, const void* c0,
-                           const void* c1, const int* cu, const int* slot, const int* pos0, const int* ent, int E, int n,
+                           long long ldv, const void* gate, long long ldg, const float* z, long long ldz, const void* x,
+                           long long ldx, const void* w2, int rank, const void* c0, const void* c1, float qscale, float inv_tau,
+                           const int* cu, const int* slot, const int* pos0, const int* ent, int E, int n,
                            int heads, int dk, int dv, float* S, const void* h, float* carry, int D, const void* nw, int per_head,
-                           float eps, float* raw, void* out, int one, int chunked, cudaStream_t stream) {
+                           float eps, float out_scale, float* raw, void* out, long long ldo, int one, int chunked,
+                           cudaStream_t stream) {
   if (n <= 0 || E <= 0) return 0;
-  if (heads <= 0 || dk <= 0 || dv <= 0 || E > 65535 || heads > 65535 || (mode != BONUS && mode != LOWER) || (mode == BONUS && !k)) return -2;
-  GlaArgs a{q, k, v, gate, ldq, ldk, ldv, ldg, z, ldz, c0, c1, heads, dk, dv, Ragged{cu, slot, pos0, ent, E, n}, S, h, carry, D,
-            nw, per_head, eps};
-  if (dtype == 0)
-    return mode == BONUS ? run<bf, BONUS>(a, raw, (bf*)out, one, chunked, stream) : run<bf, LOWER>(a, raw, (bf*)out, one, chunked, stream);
-  return mode == BONUS ? run<float, BONUS>(a, raw, (float*)out, one, chunked, stream) : run<float, LOWER>(a, raw, (float*)out, one, chunked, stream);
+  if (heads <= 0 || dk <= 0 || dv <= 0 || E > 65535 || heads > 65535 || mode < BONUS || mode > ROOT || (has_keys(mode) && !k) ||
+      (mode != ROOT && !c1) || (!z && (!one || !x || !w2 || rank <= 0))) return -2;
+  GlaArgs a{q, k, v, gate, ldq, ldk, ldv, ldg, z, ldz, x, w2, ldx, rank, c0, c1, qscale, inv_tau, heads, dk, dv,
+            Ragged{cu, slot, pos0, ent, E, n}, S, h, carry, D, nw, per_head, eps, out_scale, ldo};
+#define GL(T) (mode == BONUS ? run<T, BONUS>(a, raw, (T*)out, one, chunked, stream) : mode == LOWER \
+                   ? run<T, LOWER>(a, raw, (T*)out, one, chunked, stream) : run<T, ROOT>(a, raw, (T*)out, one, chunked, stream))
+  return dtype == 0 ? GL(bf) : GL(float);
+#undef GL
 }

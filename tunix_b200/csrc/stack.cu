@@ -7,9 +7,11 @@
 //                 read and written once per sublayer. y is one tensor, or half the sum of two tensors that are
 //                 RMS-normed first (two mixers side by side), or one tensor that is RMS-normed first (an update with a
 //                 norm of its own). The first launch of a forward pass takes the embedding rows (normed, if the model
-//                 norms them) instead of streams, the last one has no successor but the final norm. Norms may run over
-//                 equal groups of a row. Without a norm the row itself is written in the activation type. In a decode
-//                 step the launch can also mix the new row with the one before it (token shift).
+//                 norms them; scaled; with a learned row per position added) instead of streams, the last one has no
+//                 successor but the final norm. A launch between two passes of a loop can add the embedding rows again,
+//                 after the sum of the streams is reported. Norms may run over equal groups of a row. Without a norm
+//                 the row itself is written in the activation type. In a decode step the launch can also mix the new
+//                 row with the one before it (token shift).
 //   token_shift : the same mixes for portions of prompts.
 //   few_outputs, small_act : products with a handful of outputs, and what is applied to them (tanh; gelu times a row
 //                 that belongs to the token).
@@ -36,11 +38,15 @@ struct StreamArgs {
   const void* wy2;            // T [D]
   const void* mix;            // T [S, S], row = from, column = to
   const void* out;            // T [S]
-  // the start of a forward pass (instead of the above)
+  // the start of a forward pass (instead of the above), or with y: rows that are added after it
   const long long* tokens;    // [n] or null
   const void* embed;          // T [V, D]
   int vocab;
   const void* embed_w;        // T [D] or null: weight of the norm of the embedding rows
+  float embed_scale;          // factor of the (normed) embedding rows
+  const void* pos;            // T [positions, D] or null: a row per position, added to the embedding rows
+  int positions;
+  const int *cu, *ent;        // the batch's entries, with pos0 below (read with pos only)
   int groups;                 // equal parts of a row that the norms of embedding and streams are taken over
   // the sublayer that follows
   const void* in;             // T [S]; null = all ones (the sum of the streams)
@@ -126,8 +132,12 @@ __global__ void __launch_bounds__(512) stream_step_kernel(const StreamArgs a) {
     r1 = 0.5f / sqrtf(s1 / (float)D + a.eps);
     r2 = 0.5f / sqrtf(s2 / (float)D + a.eps);
   }
-  const T* emb = nullptr;
+  const T *emb = nullptr, *pos = nullptr;
   if (a.tokens) {
+    if (a.pos) {
+      const int e = a.ent[row], p = a.pos0[e] + (int)row - a.cu[e];
+      pos = static_cast<const T*>(a.pos) + (long long)min(max(p, 0), a.positions - 1) * D;
+    }
     long long t = a.tokens[row];
     t = t < 0 ? 0 : (t >= a.vocab ? a.vocab - 1 : t);
     emb = static_cast<const T*>(a.embed) + t * D;
@@ -142,9 +152,8 @@ __global__ void __launch_bounds__(512) stream_step_kernel(const StreamArgs a) {
   }
   float ss = 0.f;
   for (int d = threadIdx.x * V; d < D; d += step) {
-    float v[S][V];
+    float v[S][V], ev[V];
     if (emb) {
-      float ev[V];
       load_v<V>(emb + d, ev);
       if (a.embed_w) {
         float w[V];
@@ -152,6 +161,16 @@ __global__ void __launch_bounds__(512) stream_step_kernel(const StreamArgs a) {
 #pragma unroll
         for (int i = 0; i < V; ++i) ev[i] *= rs[(d + i) / glen] * w[i];
       }
+#pragma unroll
+      for (int i = 0; i < V; ++i) ev[i] *= a.embed_scale;
+      if (pos) {
+        float pv[V];
+        load_v<V>(pos + d, pv);
+#pragma unroll
+        for (int i = 0; i < V; ++i) ev[i] += pv[i];
+      }
+    }
+    if (emb && !y) {
 #pragma unroll
       for (int s = 0; s < S; ++s)
 #pragma unroll
@@ -192,17 +211,32 @@ __global__ void __launch_bounds__(512) stream_step_kernel(const StreamArgs a) {
           for (int i = 0; i < V; ++i) v[t][i] = o[t][i];
       }
     }
+    if (a.sum_out) {
+      float tot[V];
+#pragma unroll
+      for (int i = 0; i < V; ++i) {
+        tot[i] = 0.f;
+#pragma unroll
+        for (int s = 0; s < S; ++s) tot[i] += v[s][i];
+      }
+      store_v<V>(a.sum_out + row * D + d, tot);
+    }
+    if (emb && y) {
+#pragma unroll
+      for (int s = 0; s < S; ++s)
+#pragma unroll
+        for (int i = 0; i < V; ++i) v[s][i] += ev[i];
+    }
 #pragma unroll
     for (int s = 0; s < S; ++s) store_v<V>(x + (long long)s * D + d, v[s]);
-    float u[V], tot[V];
+    float u[V];
 #pragma unroll
     for (int i = 0; i < V; ++i) {
-      u[i] = tot[i] = 0.f;
+      u[i] = 0.f;
 #pragma unroll
-      for (int s = 0; s < S; ++s) { u[i] += inw[s] * v[s][i]; tot[i] += v[s][i]; }
+      for (int s = 0; s < S; ++s) u[i] += inw[s] * v[s][i];
       ss += u[i] * u[i];
     }
-    if (a.sum_out) store_v<V>(a.sum_out + row * D + d, tot);
     store_v<V>(u_s + d, u);
   }
   if (!a.h && !a.mu) return;
@@ -486,14 +520,15 @@ token_shift_kernel(const T* __restrict__ h, const T* __restrict__ mu, const floa
 // dtype: 0 = bf16, 1 = float (activations and weights). x fp32 [n, S, D]; see StreamArgs.
 TB_API int tb_stream_step(int dtype, float* x, int n, int S, int D, float eps, const void* y, const void* y2, const void* wy,
                           const void* wy2, const void* mix, const void* out, const long long* tokens, const void* embed,
-                          int vocab, const void* embed_w, int groups, const void* in, const void* w, void* h, float* sum_out,
-                          const void* mu, int n_mix, float* before, void* mixes, const int* slot, const int* pos0,
-                          cudaStream_t stream) {
+                          int vocab, const void* embed_w, float embed_scale, const void* pos, int positions, int groups,
+                          const void* in, const void* w, void* h, float* sum_out, const void* mu, int n_mix, float* before,
+                          void* mixes, const int* cu, const int* slot, const int* pos0, const int* ent, cudaStream_t stream) {
   if (n <= 0) return 0;
-  if (S < 1 || S > MAX_STREAMS || D <= 0 || D > 11000 || (y && tokens) || (y2 && !y)) return -2;
+  if (S < 1 || S > MAX_STREAMS || D <= 0 || D > 11000 || (y2 && !y)) return -2;
+  if (pos && (!tokens || positions <= 0 || !cu || !pos0 || !ent)) return -2;
   if (groups < 1 || groups > 256 || D % groups || (mu && (!w || !before || !mixes))) return -2;
-  StreamArgs a{x, D, eps, y, y2, wy, wy2, mix, out, tokens, embed, vocab, embed_w, groups, in, w, h, sum_out,
-               mu, n_mix, before, mixes, slot, pos0};
+  StreamArgs a{x, D, eps, y, y2, wy, wy2, mix, out, tokens, embed, vocab, embed_w, embed_scale, pos, positions, cu, ent,
+               groups, in, w, h, sum_out, mu, n_mix, before, mixes, slot, pos0};
   return dtype == 0 ? dispatch_stream_step<__nv_bfloat16>(a, S, n, stream) : dispatch_stream_step<float>(a, S, n, stream);
 }
 

@@ -4,12 +4,15 @@
 //   qk_norm_write : after the fused projection of a step: RMS norm of q and of k over the WHOLE projection (all heads at
 //                   once), q to a compact buffer, k and v rows to their pages (value rows may be wider or narrower than
 //                   key rows).
-//   rope_norm_write : the same place for rotary attention: the first `rd` dimensions of every query and key head turn by
-//                   the angles of the token's position (element i together with i + rd / 2), then each head is divided by
-//                   its root mean square. A layer that reads another layer's cache has queries only.
+//   rope_norm_write : the same place for rotary attention: every query and key head is divided by its root mean square
+//                   (and weighted, if the model has weights), then its first `rd` dimensions turn by the angles of the
+//                   token's position, element i together with i + rd / 2, or (interleaved) 2 i together with 2 i + 1. Heads
+//                   can be stored wider than they are, with zeros behind them, so that the tensor-core kernels fit them. A
+//                   layer that reads another layer's cache has queries only.
 //   window_attn   : any head sizes, bf16 or float: one warp per (token, query head), lanes over keys for the scores and
 //                   over value columns for the output, online softmax in fp32. Position i sees j <= i with
-//                   (i - j < window and j in i's chunk) or j < keep. Models whose heads fit the tensor-core kernels (attention_fwd.cu,
+//                   (i - j < window and j in i's chunk) or j < keep. A sink is one more score, without a value, in the sum
+//                   of the weights (-inf: none). Models whose heads fit the tensor-core kernels (attention_fwd.cu,
 //                   decode.cu) use those instead.
 //
 // This file is compiled without fast-math: the same kernels serve the 32-bit mode.
@@ -79,13 +82,14 @@ qk_norm_write_kernel(const T* __restrict__ proj, long long ldp, int q_off, int k
   }
 }
 
-// Heads of a multiple of 8 dimensions that turn by a multiple of 16: LPH lanes per head, 8 elements per lane; the partner of a
-// rotation sits rd / 16 lanes away. Otherwise like rope_norm_write_kernel.
-template <int LPH>
+// Heads of a multiple of 8 dimensions that turn by a multiple of 16 (8 if interleaved): LPH lanes per head, 8 elements per lane;
+// the partner of a rotation sits rd / 16 lanes away, or in the same lane. Otherwise like rope_norm_write_kernel.
+template <int LPH, bool INTER>
 __global__ void __launch_bounds__(256)
 rope_norm_write_vec_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int q_off, int k_off, int v_off,
-                           const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rd, float eps, Ragged rb, Paged pg,
-                           int H, int G, int dq, int dv, __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ kp,
+                           const __nv_bfloat16* __restrict__ qw, const __nv_bfloat16* __restrict__ kw, const float* __restrict__ cos_t,
+                           const float* __restrict__ sin_t, int rd, float eps, Ragged rb, Paged pg, int H, int G, int dq, int dv,
+                           int wq, int wv, __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ kp,
                            __nv_bfloat16* __restrict__ vp) {
   pdl_trigger();
   pdl_wait();
@@ -95,12 +99,18 @@ rope_norm_write_vec_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp
   const int p = p0 + t - rb.cu[e];
   long long pr = 0;
   if (p0 >= 0 && G > 0) pr = page_row(pg, pg.table + (long long)rb.slot[e] * pg.max_pages, p);
-  const bool turns = sub < 2 * half8 && p0 >= 0;
+  const bool turns = sub * 8 < rd && p0 >= 0;
   const int partner = turns ? (sub < half8 ? sub + half8 : sub - half8) : sub;
   float c[8], s[8];
 #pragma unroll
   for (int i = 0; i < 8; ++i) { c[i] = 1.f; s[i] = 0.f; }
-  if (turns) {
+  if (INTER && turns) {
+    float c4[4], s4[4];
+    load_v<4>(cos_t + (long long)p * (rd >> 1) + sub * 4, c4);
+    load_v<4>(sin_t + (long long)p * (rd >> 1) + sub * 4, s4);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) { c[i] = c4[i >> 1]; s[i] = (i & 1) ? s4[i >> 1] : -s4[i >> 1]; }
+  } else if (turns) {
     const long long at = (long long)p * (rd >> 1) + (sub < half8 ? sub : sub - half8) * 8;
     load_v<8>(cos_t + at, c);
     load_v<8>(sin_t + at, s);
@@ -109,6 +119,11 @@ rope_norm_write_vec_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp
       for (int i = 0; i < 8; ++i) s[i] = -s[i];
     }
   }
+  float wa[8], wb[8];                                   // norm weights of this lane's elements of a query / key head
+#pragma unroll
+  for (int i = 0; i < 8; ++i) wa[i] = wb[i] = 1.f;
+  if (qw && sub * 8 < dq) load_v<8>(qw + sub * 8, wa);
+  if (kw && sub * 8 < dq) load_v<8>(kw + sub * 8, wb);
   for (int h0 = 0; h0 < heads; h0 += 256 / LPH) {       // whole warps stay together for the shuffles
     const int hh = h0 + threadIdx.x / LPH;
     const bool is_v = hh >= H + G, ok = hh < heads && sub * 8 < (is_v ? dv : dq) && p0 >= 0;
@@ -118,25 +133,22 @@ rope_norm_write_vec_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp
     if (ok) load_v<8>(row + (hh < H ? q_off + hh * dq : is_v ? v_off + (hh - H - G) * dv : k_off + (hh - H) * dq) + sub * 8, v);
     float o[8], ss = 0.f;
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      o[i] = v[i] * c[i] + __shfl_sync(0xffffffffu, v[i], base + partner) * s[i];
-      ss += o[i] * o[i];
-    }
+    for (int i = 0; i < 8; ++i) ss += v[i] * v[i];
 #pragma unroll
     for (int w = LPH / 2; w >= 1; w >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, w);
-    const float r = 1.f / sqrtf(ss / (float)dq + eps);
+    if (!is_v) {
+      const float r = 1.f / sqrtf(ss / (float)dq + eps);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) v[i] *= r * (hh < H ? wa[i] : wb[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+      o[i] = v[i] * c[i] + (INTER ? v[i ^ 1] : __shfl_sync(0xffffffffu, v[i], base + partner)) * s[i];
     if (hh < H) {
-      if (sub * 8 < dq) {
-#pragma unroll
-        for (int i = 0; i < 8; ++i) o[i] *= r;
-        store_v<8>(q + ((long long)t * H + hh) * dq + sub * 8, o);
-      }
-    } else if (ok && !is_v) {
-#pragma unroll
-      for (int i = 0; i < 8; ++i) o[i] *= r;
-      store_v<8>(kp + (pr * G + hh - H) * dq + sub * 8, o);
-    } else if (ok) {
-      store_v<8>(vp + (pr * G + hh - H - G) * dv + sub * 8, v);
+      if (sub * 8 < wq) store_v<8>(q + ((long long)t * H + hh) * wq + sub * 8, o);
+    } else if (hh < heads && p0 >= 0) {
+      if (!is_v && sub * 8 < wq) store_v<8>(kp + (pr * G + hh - H) * wq + sub * 8, o);
+      if (is_v && sub * 8 < wv) store_v<8>(vp + (pr * G + hh - H - G) * wv + sub * 8, v);
     }
   }
 }
@@ -144,9 +156,10 @@ rope_norm_write_vec_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp
 // One warp per (token, head) over the query heads, then key heads, then value heads of a row. cos / sin [positions, rd / 2].
 template <typename T>
 __global__ void __launch_bounds__(256)
-rope_norm_write_kernel(const T* __restrict__ proj, long long ldp, int q_off, int k_off, int v_off, const float* __restrict__ cos_t,
-                       const float* __restrict__ sin_t, int rd, float eps, Ragged rb, Paged pg, int H, int G, int dq, int dv,
-                       T* __restrict__ q, T* __restrict__ kp, T* __restrict__ vp) {
+rope_norm_write_kernel(const T* __restrict__ proj, long long ldp, int q_off, int k_off, int v_off, const T* __restrict__ qw,
+                       const T* __restrict__ kw, const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rd, int inter,
+                       float eps, Ragged rb, Paged pg, int H, int G, int dq, int dv, int wq, int wv, T* __restrict__ q,
+                       T* __restrict__ kp, T* __restrict__ vp) {
   pdl_trigger();
   pdl_wait();
   const int heads = H + 2 * G;
@@ -158,7 +171,7 @@ rope_norm_write_kernel(const T* __restrict__ proj, long long ldp, int q_off, int
   const T* row = proj + (long long)t * ldp;
   if (p0 < 0) {
     if (hh < H)
-      for (int c = lane; c < dq; c += 32) q[((long long)t * H + hh) * dq + c] = from_f<T>(0.f);
+      for (int c = lane; c < wq; c += 32) q[((long long)t * H + hh) * wq + c] = from_f<T>(0.f);
     return;
   }
   const int p = p0 + t - rb.cu[e];
@@ -166,35 +179,30 @@ rope_norm_write_kernel(const T* __restrict__ proj, long long ldp, int q_off, int
   if (hh >= H) pr = page_row(pg, pg.table + (long long)rb.slot[e] * pg.max_pages, p);
   if (hh >= H + G) {
     const int g = hh - H - G;
-    for (int c = lane; c < dv; c += 32) vp[(pr * G + g) * dv + c] = row[v_off + g * dv + c];
+    for (int c = lane; c < wv; c += 32) vp[(pr * G + g) * wv + c] = c < dv ? row[v_off + g * dv + c] : from_f<T>(0.f);
     return;
   }
   const T* src = row + (hh < H ? q_off + hh * dq : k_off + (hh - H) * dq);
-  T* dst = hh < H ? q + ((long long)t * H + hh) * dq : kp + (pr * G + hh - H) * dq;
+  const T* w = hh < H ? qw : kw;
+  T* dst = hh < H ? q + ((long long)t * H + hh) * wq : kp + (pr * G + hh - H) * wq;
   const int half = rd >> 1;
   const float *ct = cos_t + (long long)p * half, *st = sin_t + (long long)p * half;
-  // the turned head stays in registers up to 256 dimensions (lane + 32 j), wider ones are turned twice
-  auto turned = [&](int c) {
-    const float x = to_f(src[c]);
-    if (c < half) return x * ct[c] - to_f(src[c + half]) * st[c];
-    if (c < 2 * half) return x * ct[c - half] + to_f(src[c - half]) * st[c - half];
-    return x;
-  };
-  float v[8], ss = 0.f;
-#pragma unroll
-  for (int j = 0; j < 8; ++j) {
-    const int c = lane + 32 * j;
-    v[j] = c < dq ? turned(c) : 0.f;
-    ss += v[j] * v[j];
-  }
-  for (int c = lane + 256; c < dq; c += 32) { const float x = turned(c); ss += x * x; }
+  float ss = 0.f;
+  for (int c = lane; c < dq; c += 32) { const float x = to_f(src[c]); ss += x * x; }
   const float r = 1.f / sqrtf(warp_sum(ss) / (float)dq + eps);
-#pragma unroll
-  for (int j = 0; j < 8; ++j) {
-    const int c = lane + 32 * j;
-    if (c < dq) dst[c] = from_f<T>(v[j] * r);
+  auto normed = [&](int c) { return to_f(src[c]) * r * (w ? to_f(w[c]) : 1.f); };
+  for (int c = lane; c < wq; c += 32) {
+    float x = 0.f;
+    if (c >= rd) {
+      if (c < dq) x = normed(c);
+    } else if (inter) {
+      const float a = normed(c), b = normed(c ^ 1);
+      x = (c & 1) ? a * ct[c >> 1] + b * st[c >> 1] : a * ct[c >> 1] - b * st[c >> 1];
+    } else {
+      x = c < half ? normed(c) * ct[c] - normed(c + half) * st[c] : normed(c) * ct[c - half] + normed(c - half) * st[c - half];
+    }
+    dst[c] = from_f<T>(x);
   }
-  for (int c = lane + 256; c < dq; c += 32) dst[c] = from_f<T>(turned(c) * r);
 }
 
 constexpr int VREG = 16;        // value columns per lane: value heads up to 512 wide
@@ -202,8 +210,8 @@ constexpr int VREG = 16;        // value columns per lane: value heads up to 512
 template <typename T>
 __global__ void __launch_bounds__(128)
 window_attn_kernel(const T* __restrict__ q, const T* __restrict__ kp, const T* __restrict__ vp, Ragged rb, Paged pg, int H,
-                   int G, int dq, int dv, float scale, float cap, const float* __restrict__ bias, int far, int window, int chunk,
-                   int keep, T* __restrict__ out) {
+                   int G, int dq, int dv, int wq, int wv, float scale, float cap, const float* __restrict__ bias, int far, int window,
+                   int chunk, int keep, float sink, float out_scale, T* __restrict__ out, long long ldo) {
   extern __shared__ float qs_all[];               // [4][dq]
   pdl_trigger();
   pdl_wait();
@@ -212,13 +220,13 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ kp, const T* _
   if (wid >= (long long)rb.n * H) return;
   const int t = (int)(wid / H), h = (int)(wid - (long long)t * H), g = h / (H / G);
   const int e = rb.ent[t], p0 = rb.pos0[e];
-  T* o = out + ((long long)t * H + h) * dv;
+  T* o = out + (long long)t * ldo + (long long)h * dv;
   if (p0 < 0) {
     for (int c = lane; c < dv; c += 32) o[c] = from_f<T>(0.f);
     return;
   }
   float* qs = qs_all + warp * dq;
-  for (int d = lane; d < dq; d += 32) qs[d] = to_f(q[((long long)t * H + h) * dq + d]) * scale;
+  for (int d = lane; d < dq; d += 32) qs[d] = to_f(q[((long long)t * H + h) * wq + d]) * scale;
   __syncwarp();
   const int i = p0 + t - rb.cu[e];
   const int lo = first_visible(i, window, chunk);
@@ -236,7 +244,7 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ kp, const T* _
     if (x < cnt) {
       const int j = x < kept ? x : lo + x - kept;
       row = page_row(pg, pt, j);
-      const T* k = kp + (row * G + g) * dq;
+      const T* k = kp + (row * G + g) * wq;
       float dot = 0.f;
       for (int d = 0; d < dq; ++d) dot += qs[d] * to_f(k[d]);
       s = cap > 0.f ? cap * tanhf(dot / cap) : dot;
@@ -252,7 +260,7 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ kp, const T* _
     for (int y = 0; y < lim; ++y) {
       const float py = __shfl_sync(0xffffffffu, p, y);
       const long long ry = __shfl_sync(0xffffffffu, row, y);
-      const T* v = vp + (ry * G + g) * dv;
+      const T* v = vp + (ry * G + g) * wv;
 #pragma unroll
       for (int r = 0; r < VREG; ++r) {
         const int cc = r * 32 + lane;
@@ -260,7 +268,7 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ kp, const T* _
       }
     }
   }
-  const float inv = 1.f / l;
+  const float inv = out_scale / (l + expf(sink - m));
 #pragma unroll
   for (int r = 0; r < VREG; ++r) {
     const int cc = r * 32 + lane;
@@ -290,41 +298,46 @@ TB_API int tb_qk_norm_write(int dtype, const void* proj, long long ldp, int q_of
   return err == cudaSuccess ? 0 : -5;
 }
 
-// q | k | v: columns of proj [n, ldp]; H query heads, G key / value heads (0: queries only), rd rotated dimensions with tables
-// cos / sin fp32 [positions, rd / 2]; q [n, H * dq]; pools [pages, page_size, G * dq] and [.., G * dv].
-TB_API int tb_rope_norm_write(int dtype, const void* proj, long long ldp, int q_off, int k_off, int v_off, const float* cos_t,
-                              const float* sin_t, int rd, float eps, const int* cu, const int* slot, const int* pos0,
-                              const int* ent, int E, int n, const int* table, int max_pages, int page_size, int H, int G, int dq,
-                              int dv, void* q, void* kp, void* vp, cudaStream_t stream) {
+// q | k | v: columns of proj [n, ldp]; H query heads of dq, G key / value heads (0: queries only) of dq / dv; qw, kw T [dq] or
+// null: weights of the heads' norms; rd rotated dimensions (inter: neighbours turn together) with tables cos / sin fp32
+// [positions, rd / 2]. Heads are stored wq / wv wide: q [n, H * wq]; pools [pages, page_size, G * wq] and [.., G * wv].
+TB_API int tb_rope_norm_write(int dtype, const void* proj, long long ldp, int q_off, int k_off, int v_off, const void* qw,
+                              const void* kw, const float* cos_t, const float* sin_t, int rd, int inter, float eps, const int* cu,
+                              const int* slot, const int* pos0, const int* ent, int E, int n, const int* table, int max_pages,
+                              int page_size, int H, int G, int dq, int dv, int wq, int wv, void* q, void* kp, void* vp,
+                              cudaStream_t stream) {
   if (n <= 0) return 0;
-  if (rd < 0 || rd % 2 || rd > dq) return -2;
+  if (rd < 0 || rd % 2 || rd > dq || wq < dq || wv < dv) return -2;
   RAGGED;
   PAGED;
-  const int wide = dq > dv ? dq : dv;
-  if (dtype == 0 && dq % 8 == 0 && dv % 8 == 0 && rd % 16 == 0 && wide <= 256 && ldp % 8 == 0 && q_off % 8 == 0 && k_off % 8 == 0 &&
-      v_off % 8 == 0) {
+  const int wide = wq > wv ? wq : wv;
+  if (dtype == 0 && dq % 8 == 0 && dv % 8 == 0 && wq % 8 == 0 && wv % 8 == 0 && rd % (inter ? 8 : 16) == 0 && wide <= 256 &&
+      ldp % 8 == 0 && q_off % 8 == 0 && k_off % 8 == 0 && v_off % 8 == 0) {
     typedef __nv_bfloat16 bf;
-#define VEC(L)                                                                                                              \
-  launch_pdl(rope_norm_write_vec_kernel<L>, dim3(n), dim3(256), 0, stream, (const bf*)proj, ldp, q_off, k_off, v_off, cos_t,  \
-             sin_t, rd, eps, rb, pg, H, G, dq, dv, (bf*)q, (bf*)kp, (bf*)vp)
-    return (wide <= 64 ? VEC(8) : wide <= 128 ? VEC(16) : VEC(32)) == cudaSuccess ? 0 : -5;
+#define VEC(L, I)                                                                                                           \
+  launch_pdl(rope_norm_write_vec_kernel<L, I>, dim3(n), dim3(256), 0, stream, (const bf*)proj, ldp, q_off, k_off, v_off,     \
+             (const bf*)qw, (const bf*)kw, cos_t, sin_t, rd, eps, rb, pg, H, G, dq, dv, wq, wv, (bf*)q, (bf*)kp, (bf*)vp)
+    const cudaError_t err = inter ? (wide <= 64 ? VEC(8, true) : wide <= 128 ? VEC(16, true) : VEC(32, true))
+                                  : (wide <= 64 ? VEC(8, false) : wide <= 128 ? VEC(16, false) : VEC(32, false));
+    return err == cudaSuccess ? 0 : -5;
 #undef VEC
   }
   const long long warps = (long long)n * (H + 2 * G);
   const dim3 grid((unsigned)((warps + 7) / 8));
 #define RUN(T)                                                                                                              \
-  launch_pdl(rope_norm_write_kernel<T>, grid, dim3(256), 0, stream, (const T*)proj, ldp, q_off, k_off, v_off, cos_t, sin_t,  \
-             rd, eps, rb, pg, H, G, dq, dv, (T*)q, (T*)kp, (T*)vp)
+  launch_pdl(rope_norm_write_kernel<T>, grid, dim3(256), 0, stream, (const T*)proj, ldp, q_off, k_off, v_off, (const T*)qw,  \
+             (const T*)kw, cos_t, sin_t, rd, inter, eps, rb, pg, H, G, dq, dv, wq, wv, (T*)q, (T*)kp, (T*)vp)
   return (dtype == 0 ? RUN(__nv_bfloat16) : RUN(float)) == cudaSuccess ? 0 : -5;
 #undef RUN
 }
 
 // bias fp32 [H, far + 1] or null: what is added to the score of a key at distance min(i - j, far). window, chunk <= 0: none;
-// cap > 0: scores become cap * tanh(score / cap).
+// cap > 0: scores become cap * tanh(score / cap). sink: one more score without a value in the sum of the weights (-inf: none).
+// Heads are stored wq / wv wide; out T [n, ldo], head h at columns h * dv, times out_scale.
 TB_API int tb_window_attn(int dtype, const void* q, const void* kp, const void* vp, const int* cu, const int* slot,
                           const int* pos0, const int* ent, int E, int n, const int* table, int max_pages, int page_size, int H,
-                          int G, int dq, int dv, float scale, float cap, const float* bias, int far, int window, int chunk,
-                          int keep, void* out, cudaStream_t stream) {
+                          int G, int dq, int dv, int wq, int wv, float scale, float cap, const float* bias, int far, int window,
+                          int chunk, int keep, float sink, float out_scale, void* out, long long ldo, cudaStream_t stream) {
   if (n <= 0) return 0;
   if (G <= 0 || H % G || dv > VREG * 32 || dq > 3000) return -2;
   RAGGED;
@@ -333,7 +346,8 @@ TB_API int tb_window_attn(int dtype, const void* q, const void* kp, const void* 
   const dim3 grid((unsigned)((warps + 3) / 4));
 #define RUN(T)                                                                                                              \
   return launch_pdl(window_attn_kernel<T>, grid, dim3(128), (size_t)4 * dq * 4, stream, (const T*)q, (const T*)kp,           \
-                    (const T*)vp, rb, pg, H, G, dq, dv, scale, cap, bias, far, window, chunk, keep, (T*)out) == cudaSuccess ? 0 : -5
+                    (const T*)vp, rb, pg, H, G, dq, dv, wq, wv, scale, cap, bias, far, window, chunk, keep, sink, out_scale, \
+                    (T*)out, ldo) == cudaSuccess ? 0 : -5
   if (dtype == 0) RUN(__nv_bfloat16);
   RUN(float);
 #undef RUN

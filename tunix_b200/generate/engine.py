@@ -65,7 +65,7 @@ class PagePool:
         from ..experimental.generate import kv_cache_manager as kvm
         self.page_size, self.num_pages, self.max_pages = page_size, num_pages, max_pages_per_seq
         if hasattr(cfg, "kv_rows"):                # layer-stack models: rows and states per layer pass
-            rows, self.state = cfg.kv_rows(), SlotStates(cfg.state_shapes(), max_seqs, device)
+            rows, self.state = cfg.kv_rows(dtype), SlotStates(cfg.state_shapes(), max_seqs, device)
         else:
             row = (kv_heads or cfg.num_kv_heads) * cfg.head_dim   # a tensor-parallel rank keeps its own kv heads only
             rows, self.state = [(row, row)] * cfg.num_layers, None
@@ -205,6 +205,11 @@ class PagedEngine(BaseSampler):
         for name, w in updated_weights.items():
             if own[name].data_ptr() != w.data_ptr():
                 own[name].copy_(w.to(own[name].device, own[name].dtype))
+
+    def _check_length(self, tokens: int) -> None:
+        limit = getattr(self.cfg, "positions", 0)
+        if limit and tokens > limit:
+            raise ValueError(f"a sequence of {tokens} tokens: the model has {limit} positions")
 
     def delete_cache(self) -> None:
         self.pool = None
@@ -539,6 +544,7 @@ class PagedEngine(BaseSampler):
         plen = max_prompt_length if max_prompt_length else next_power_of_2(max(len(r) for r in rows))
         if plen + max_generation_steps > self.cache_size:
             raise ValueError("prompt + generation exceeds the configured cache size")
+        self._check_length(max(len(r) for r in rows) + max_generation_steps)
         was_training = self._model.training
         self._model.eval()
         prompts_all, plens_all = pad_prompts_left(rows, plen, pad_id)
@@ -894,6 +900,7 @@ class StepSession:
             if not tokens:
                 continue
             req = self._live.get(rid)
+            eng._check_length((req[1] if req else 0) + len(tokens))
             if req is None:
                 if not self._free:
                     raise RuntimeError(f"request {rid!r}: all {eng.max_running} slots are in use")
@@ -913,6 +920,9 @@ class StepSession:
             h = eng.exec.forward(RaggedBatch.build(work, eng.device), pool)
             if rows:
                 logits = eng._logits(h[torch.tensor(rows, dtype=torch.int64, device=eng.device)])
+                cap = float(eng.cfg.final_logit_softcap or 0.0)
+                if cap > 0.0:
+                    logits = cap * torch.tanh(logits / cap)
         for rid in end:
             self.end(rid)
         return logits
@@ -941,6 +951,7 @@ class EngineServer:
         import threading
         if max_prompt_length + max_new_tokens > engine.cache_size:
             raise ValueError("prompt + generation exceeds the configured cache size")
+        engine._check_length(max_prompt_length + max_new_tokens)
         self.engine = engine
         self.max_new_tokens = int(max_new_tokens)
         self.P = int(max_prompt_length)

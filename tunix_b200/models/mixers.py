@@ -13,11 +13,17 @@ sizes and constants in a spec, its parameters in a module and its per-sequence c
                           memory with a data-dependent decay per key channel and a bonus for the current token, per-head
                           norm and silu output gate
   ForgetGateMemory        HGRN2: matrix memory whose forget gate (bounded from below) also decides what is written
-  RotaryAttention         grouped-query attention with rotary positions, RMS-normed query and key heads, score cap, chunks
-                          of positions; may read the keys and values of another layer
+  RotaryAttention         grouped-query attention with rotary positions (halves of a head or neighbouring dimensions turn
+                          together, frequencies may be scaled), RMS-normed query and key heads with or without weights, score
+                          cap, sliding window, chunks of positions, a sink in the softmax; may read the keys and values of
+                          another layer
+  GatedLinearAttention    matrix memory with a decay per key channel, a root of a sigmoid behind a bottleneck; per-head norm
+                          and silu output gate
+  SumMixer                rotary attention and gated linear attention on the same input, each times a constant, summed
 
-A spec's `kv_rows()` names the paged cache rows a pass through the layer needs (key columns, value columns), or None (also
-for attention that reads another layer's, `kv_from`); `state_shapes()` the fp32 state it keeps per sequence slot. The kernels are launched by `models/stack_exec.py`.
+A spec's `kv_rows(dtype)` names the paged cache rows a pass through the layer needs (key columns, value columns), or None
+(also for attention that reads another layer's, `kv_from`); `state_shapes()` the fp32 state it keeps per sequence slot. Heads
+of attention are stored `stored(dtype)` wide. The kernels are launched by `models/stack_exec.py`.
 """
 from __future__ import annotations
 
@@ -31,6 +37,8 @@ import torch.nn as nn
 from .transformer import Linear, RMSNorm
 
 MEMORY_SLICE = 32       # value columns a CTA of the matrix-memory kernels owns (csrc/recurrent.cu: MV)
+TILE_HEADS = (64, 128, 256)     # head sizes of the tensor-core attention kernels
+NO_SINK = -math.inf
 
 
 # ---------------------------------------------------------------------------------------------------- specs
@@ -40,7 +48,7 @@ class RGLRUSpec:
     blocks: int
     conv: int                    # taps of the causal convolution
 
-    def kv_rows(self):
+    def kv_rows(self, dtype):
         return None
 
     def state_shapes(self) -> dict:
@@ -60,8 +68,12 @@ class WindowAttentionSpec:
     buckets: int = 32            # rows of the bias table
     chunk: ClassVar[int] = 0
     softcap: ClassVar[float] = 0.0
+    sink: ClassVar[float] = NO_SINK
 
-    def kv_rows(self):
+    def stored(self, dtype):
+        return self.dim, self.vdim
+
+    def kv_rows(self, dtype):
         return (self.kv_heads * self.dim, self.kv_heads * self.vdim)
 
     def state_shapes(self) -> dict:
@@ -75,7 +87,7 @@ class MatrixMemorySpec:
     vdim: int
     gate_cap: float
 
-    def kv_rows(self):
+    def kv_rows(self, dtype):
         return None
 
     def state_shapes(self) -> dict:
@@ -88,8 +100,8 @@ class ParallelSpec:
     left: WindowAttentionSpec
     right: MatrixMemorySpec
 
-    def kv_rows(self):
-        return self.left.kv_rows()
+    def kv_rows(self, dtype):
+        return self.left.kv_rows(dtype)
 
     def state_shapes(self) -> dict:
         return self.right.state_shapes()
@@ -107,11 +119,27 @@ class RotaryAttentionSpec:
     softcap: float = 0.0         # scores become softcap * tanh(score / softcap); 0 = as they are
     chunk: int = 0               # a query sees the keys of its own chunk of that many positions; 0 = all before it
     kv_from: Optional[int] = None    # index of the layer whose keys and values this one reads
-    window: ClassVar[int] = 0
+    window: int = 0              # a query sees itself and the window - 1 keys before it; 0 = all
+    interleaved: bool = False    # dimensions 2 i and 2 i + 1 turn together; otherwise i and i + rot_dims / 2
+    rot_scaling: Optional[tuple] = None    # (factor, low, high, original context): see stack_exec.rope_frequencies
+    head_weights: bool = False   # the norms of query and key heads have weights
+    sink: float = NO_SINK        # one more score, without a value, in the sum of the weights
+    out_bias: bool = True
+    fit_heads: bool = False      # bf16 heads are stored as wide as the tensor-core kernels want them, zeros behind them
     keep_first: ClassVar[int] = 0
 
-    def kv_rows(self):
-        return None if self.kv_from is not None else (self.kv_heads * self.dim, self.kv_heads * self.vdim)
+    def stored(self, dtype):
+        wide = max(self.dim, self.vdim)
+        fit = next((w for w in TILE_HEADS if w >= wide), 0)
+        if self.fit_heads and dtype == torch.bfloat16 and fit <= 2 * wide and fit and self.vdim % 8 == 0:
+            return fit, fit
+        return self.dim, self.vdim
+
+    def kv_rows(self, dtype):
+        if self.kv_from is not None:
+            return None
+        k, v = self.stored(dtype)
+        return self.kv_heads * k, self.kv_heads * v
 
     def state_shapes(self) -> dict:
         return {}
@@ -124,7 +152,7 @@ class TokenShiftMemorySpec:
     decay_rank: int              # width of the bottleneck that makes the decays
     width: int                   # the mixer's input: the last one of a sequence is part of the state
 
-    def kv_rows(self):
+    def kv_rows(self, dtype):
         return None
 
     def state_shapes(self) -> dict:
@@ -137,11 +165,40 @@ class ForgetGateMemorySpec:
     dim: int
     vdim: int
 
-    def kv_rows(self):
+    def kv_rows(self, dtype):
         return None
 
     def state_shapes(self) -> dict:
         return {"S": (self.heads, self.dim, self.vdim)}
+
+
+@dataclass(frozen=True)
+class GatedLinearSpec:
+    heads: int
+    dim: int
+    vdim: int
+    tau: float                   # the decay is the tau-th root of a sigmoid
+    decay_rank: int              # width of the bottleneck that makes the decays
+
+    def kv_rows(self, dtype):
+        return None
+
+    def state_shapes(self) -> dict:
+        return {"S": (self.heads, self.dim, self.vdim)}
+
+
+@dataclass(frozen=True)
+class SumSpec:
+    left: RotaryAttentionSpec
+    right: GatedLinearSpec
+    left_scale: float
+    right_scale: float
+
+    def kv_rows(self, dtype):
+        return self.left.kv_rows(dtype)
+
+    def state_shapes(self) -> dict:
+        return self.right.state_shapes()
 
 
 # ------------------------------------------------------------------------------------------------- bias table
@@ -265,7 +322,9 @@ class RotaryAttention(nn.Module):
         own = spec.kv_from is None
         self.k_proj = Linear(width, spec.kv_heads * spec.dim, True, dtype, device) if own else None
         self.v_proj = Linear(width, spec.kv_heads * spec.vdim, True, dtype, device) if own else None
-        self.o_proj = Linear(spec.heads * spec.vdim, width, True, dtype, device)
+        self.o_proj = Linear(spec.heads * spec.vdim, width, spec.out_bias, dtype, device)
+        self.q_norm = RMSNorm(spec.dim, eps, False, dtype, device) if spec.head_weights else None
+        self.k_norm = RMSNorm(spec.dim, eps, False, dtype, device) if spec.head_weights and own else None
 
     def init_special(self) -> None:
         pass
@@ -321,8 +380,47 @@ class ForgetGateMemory(nn.Module):
         return [[self.q_proj, self.v_proj], [self.f_proj]]
 
 
+class GatedLinearAttention(nn.Module):
+    def __init__(self, spec: GatedLinearSpec, width: int, eps: float, dtype, device=None):
+        super().__init__()
+        self.spec, self.eps = spec, eps
+        K, C = spec.heads * spec.dim, spec.heads * spec.vdim
+        self.q_proj = Linear(width, K, False, dtype, device)
+        self.k_proj = Linear(width, K, False, dtype, device)
+        self.v_proj = Linear(width, C, False, dtype, device)
+        self.g_proj = Linear(width, C, False, dtype, device)
+        self.a1_proj = Linear(width, spec.decay_rank, False, dtype, device)
+        self.a2_proj = Linear(spec.decay_rank, K, True, dtype, device)
+        self.norm = RMSNorm(spec.vdim, eps, False, dtype, device)
+        self.o_proj = Linear(C, width, False, dtype, device)
+
+    def init_special(self) -> None:
+        self.a2_proj.bias.fill_(2.0)
+
+    def fused_groups(self) -> list:
+        return [[self.q_proj, self.k_proj, self.v_proj, self.g_proj, self.a1_proj]]
+
+
+class SumMixer(nn.Module):
+    def __init__(self, spec: SumSpec, width: int, eps: float, dtype, device=None):
+        super().__init__()
+        if spec.left.out_bias or spec.left.kv_from is not None:
+            raise ValueError("attention beside another mixer has keys of its own and no output bias")
+        self.spec = spec
+        self.left = RotaryAttention(spec.left, width, eps, dtype, device)
+        self.right = GatedLinearAttention(spec.right, width, eps, dtype, device)
+
+    def init_special(self) -> None:
+        self.left.init_special()
+        self.right.init_special()
+
+    def fused_groups(self) -> list:
+        return [self.left.fused_groups()[0] + self.right.fused_groups()[0]]
+
+
 MIXERS = {RGLRUSpec: RGLRUMixer, ParallelSpec: ParallelMixer, RotaryAttentionSpec: RotaryAttention,
-          TokenShiftMemorySpec: TokenShiftMemory, ForgetGateMemorySpec: ForgetGateMemory}
+          TokenShiftMemorySpec: TokenShiftMemory, ForgetGateMemorySpec: ForgetGateMemory, GatedLinearSpec: GatedLinearAttention,
+          SumSpec: SumMixer}
 
 
 def create_mixer(spec, width: int, eps: float, dtype, device: Optional[torch.device] = None) -> nn.Module:

@@ -52,5 +52,6 @@ for _fam, _pref, _tmpl in (("llama3", ("llama-3", "meta-llama-3", "llama3"), "ll
                            ("gemma3", ("gemma-3-",), "gemma"),
                            ("gemma4", ("gemma-4-",), "gemma4"),
                            ("roluzen", ("roluzen",), "default"),
-                           ("tovalix", ("tovalix",), "default")):
+                           ("tovalix", ("tovalix",), "default"),
+                           ("zikezen", ("zikezen",), "default")):
     register_family(FamilyEntry(_fam, config_lib.get_config, _pref, _tmpl))

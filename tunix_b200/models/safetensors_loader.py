@@ -92,11 +92,32 @@ _KEY_MAPS = {
         (r"l(\d+)\.mix\.(q|k|v|o|f)\.b", r"layers.\1.mixer.\2_proj.bias"),
         (r"l(\d+)\.mix\.(r|k|v|g|q|f|o|w1|w2)", r"layers.\1.mixer.\2_proj.weight"),
     ],
+    "zikezen": [
+        (r"embed", "embed_tokens"),
+        (r"pos", "pos_embed"),
+        (r"side\.embed", "side_embed"),
+        (r"head", "lm_head"),
+        (r"final\.norm", "norm.weight"),
+        (r"l(\d+)\.norm1", r"layers.\1.input_layernorm.weight"),
+        (r"l(\d+)\.norm2", r"layers.\1.post_attention_layernorm.weight"),
+        (r"l(\d+)\.norm1b", r"layers.\1.post_attn_norm.weight"),
+        (r"l(\d+)\.norm2b", r"layers.\1.post_ffw_norm.weight"),
+        (r"l(\d+)\.mlp\.(gate|up|down)", r"layers.\1.mlp.\2_proj.weight"),
+        (r"l(\d+)\.mlp\.e(\d+)\.(gate|up|down)", r"layers.\1.mlp.\3_proj#\2"),
+        (r"l(\d+)\.mlp\.router", r"layers.\1.mlp.router.weight"),
+        (r"l(\d+)\.mlp\.correction", r"layers.\1.mlp.correction"),
+        (r"l(\d+)\.side\.gate", r"layers.\1.side.gate_proj.weight"),
+        (r"l(\d+)\.side\.(proj|norm)", r"layers.\1.side.\2.weight"),
+        (r"l(\d+)\.mix\.left\.(q|k)\.norm", r"layers.\1.mixer.left.\2_norm.weight"),
+        (r"l(\d+)\.mix\.right\.norm", r"layers.\1.mixer.right.norm.weight"),
+        (r"l(\d+)\.mix\.(left|right)\.(q|k|v|a2)\.b", r"layers.\1.mixer.\2.\3_proj.bias"),
+        (r"l(\d+)\.mix\.(left|right)\.(q|k|v|g|o|a1|a2)", r"layers.\1.mixer.\2.\3_proj.weight"),
+    ],
 }
 
 
 def key_map_for(cfg) -> list:
-    if cfg.family in ("gemma4", "roluzen", "tovalix"):
+    if cfg.family == "gemma4" or cfg.family in _STACK_INVERSE:
         return _KEY_MAPS[cfg.family]
     return _KEY_MAPS["gemma_post_norms" if cfg.post_norms else "default"]
 
@@ -162,6 +183,20 @@ _STACK_INVERSE = {"roluzen": _STACK_ENDS + [
     (r"layers\.(\d+)\.mixer\.norm\.weight", r"l\1.mix.norm"),
     (r"layers\.(\d+)\.mixer\.(\w+)_proj\.bias", r"l\1.mix.\2.b"),
     (r"layers\.(\d+)\.mixer\.(\w+)_proj\.weight", r"l\1.mix.\2"),
+], "zikezen": _STACK_ENDS + [
+    (r"pos_embed", "pos"), (r"side_embed", "side.embed"),
+    (r"layers\.(\d+)\.post_attn_norm\.weight", r"l\1.norm1b"),
+    (r"layers\.(\d+)\.post_ffw_norm\.weight", r"l\1.norm2b"),
+    (r"layers\.(\d+)\.mlp\.(gate|up|down)_proj\.weight", r"l\1.mlp.\2"),
+    (r"layers\.(\d+)\.mlp\.(gate|up|down)_proj#(\d+)", r"l\1.mlp.e\3.\2"),
+    (r"layers\.(\d+)\.mlp\.router\.weight", r"l\1.mlp.router"),
+    (r"layers\.(\d+)\.mlp\.correction", r"l\1.mlp.correction"),
+    (r"layers\.(\d+)\.side\.gate_proj\.weight", r"l\1.side.gate"),
+    (r"layers\.(\d+)\.side\.(proj|norm)\.weight", r"l\1.side.\2"),
+    (r"layers\.(\d+)\.mixer\.left\.(q|k)_norm\.weight", r"l\1.mix.left.\2.norm"),
+    (r"layers\.(\d+)\.mixer\.right\.norm\.weight", r"l\1.mix.right.norm"),
+    (r"layers\.(\d+)\.mixer\.(left|right)\.(\w+)_proj\.bias", r"l\1.mix.\2.\3.b"),
+    (r"layers\.(\d+)\.mixer\.(left|right)\.(\w+)_proj\.weight", r"l\1.mix.\2.\3"),
 ]}
 
 
@@ -231,7 +266,8 @@ def load_safetensors_into(model, path: str, dtype: Optional[torch.dtype] = None,
         for n, p in params.items():
             if "lora_" in n or (n, None) in seen:
                 continue
-            if p.dim() == 3 and n.endswith(("gate_proj", "up_proj", "down_proj")) and model.config.is_moe:
+            if p.dim() == 3 and n.endswith(("gate_proj", "up_proj", "down_proj")) and \
+                    (model.config.is_moe or model.config.family in _STACK_INVERSE):
                 missing += [f"{n}#{e}" for e in range(p.shape[0]) if (n, e) not in seen]
             elif (n, None) not in seen:
                 missing.append(n)

@@ -9,7 +9,7 @@ from typing import Optional
 import torch
 
 from ..lora import merged_weight
-from .safetensors_loader import inverse_map_key
+from .safetensors_loader import _STACK_INVERSE, inverse_map_key
 from .transformer import Linear
 
 
@@ -58,6 +58,10 @@ def state_dict_for_export(model, merge_lora: bool = True) -> dict:
             t = p.detach()
         if cfg.family == "gemma4":
             out[name] = t.contiguous().cpu()
+            continue
+        if cfg.family in _STACK_INVERSE and p.dim() == 3 and name.endswith(("gate_proj", "up_proj", "down_proj")):
+            for e in range(p.shape[0]):
+                out[inverse_map_key(f"{name}#{e}", cfg)] = t[e].contiguous().cpu()
             continue
         if cfg.is_moe and p.dim() == 3 and name.endswith(("gate_proj", "up_proj", "down_proj")):
             base = inverse_map_key(name, cfg).rsplit(".", 1)

@@ -1,10 +1,12 @@
 """Layer-stack models: decoders whose layers are listed one by one, each with its own mixer (`models/mixers.py`) and
 feed-forward, a range of layers that may run several times with the same weights, parallel residual streams joined by
-hyper-connections, norms over groups of a row, and inputs per token and layer. Designs of this kind: Roluzen, Tovalix.
+hyper-connections, norms over groups of a row and behind sublayers, learned position rows, mixtures of experts, and inputs per
+token and layer. Designs of this kind: Roluzen, Tovalix, Zikezen.
 
 The residual streams are fp32. A sublayer q of a layer reads u = sum_s in[s] x_s, computes y = f(norm(u)) and leaves
-x_t = sum_s mix[s, t] x_s + out[t] y on every stream; the model's output is the norm of the streams' sum. A layer's token
-input adds norm(proj(gelu(gate(x)) * e)) after the feed-forward, e being the layer's part of the token's row in a second
+x_t = sum_s mix[s, t] x_s + out[t] y on every stream (`post_norms`: y is normed once more); the model's output is the norm of
+the streams' sum. With `loop_embed` the embedding output is added again before every pass of the loop but the first. A layer's
+token input adds norm(proj(gelu(gate(x)) * e)) after the feed-forward, e being the layer's part of the token's row in a second
 embedding table.
 
 The model holds parameters; `models/stack_exec.py` runs it on ragged batches over the paged cache and the slot states of
@@ -23,16 +25,18 @@ import torch.nn as nn
 
 from ..ops import functional as F
 from .config import ModelConfig
-from .mixers import (ForgetGateMemorySpec, MatrixMemorySpec, ParallelSpec, RGLRUSpec, RotaryAttentionSpec, TokenShiftMemorySpec,
-                     WindowAttentionSpec, create_mixer)
+from .mixers import (ForgetGateMemorySpec, GatedLinearSpec, MatrixMemorySpec, ParallelSpec, RGLRUSpec, RotaryAttentionSpec, SumSpec,
+                     TokenShiftMemorySpec, WindowAttentionSpec, create_mixer)
 from .transformer import MLP, Linear, RMSNorm
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     mixer: object                       # one of the specs of models/mixers.py
-    ff: Optional[int]                   # width of the feed-forward; None = the layer has none
-    ff_kind: str = "glu"                # "glu": silu-gated; "xielu": up, xIELU with two learned numbers, down
+    ff: Optional[int]                   # width of the feed-forward (of an expert); None = the layer has none
+    ff_kind: str = "glu"                # "glu": silu-gated; "xielu": up, xIELU with two learned numbers, down; "experts"
+    experts: int = 0                    # silu-gated experts, of which a token uses `top`
+    top: int = 0
 
 
 @dataclass
@@ -43,6 +47,9 @@ class StackConfig(ModelConfig):
     norm_groups: int = 1                # equal parts of a row that the norms before sublayers and at the ends are taken over
     embed_norm: bool = False            # the embedding rows are normed
     token_side: int = 0                 # width of the per-layer token inputs; 0 = none
+    embed_factor: float = 1.0           # of the embedding rows
+    positions: int = 0                  # rows of the learned position table, the longest sequence; 0 = no table
+    loop_embed: bool = False            # the embedding output is added again before each pass of the loop but the first
 
     def __post_init__(self):
         if not self.layer_specs:
@@ -61,6 +68,10 @@ class StackConfig(ModelConfig):
         if self.embed_dim % self.norm_groups:
             raise ValueError(f"a width of {self.embed_dim} does not split into {self.norm_groups} norm groups")
         for i, s in enumerate(self.layer_specs):
+            if s.ff_kind == "experts" and s.ff is not None and not 1 <= s.top <= s.experts:
+                raise ValueError(f"layer {i}: {s.top} of {s.experts} experts")
+            if self.post_norms and isinstance(s.mixer, ParallelSpec):
+                raise ValueError(f"layer {i}: the halves of this mixer are normed already")
             j = getattr(s.mixer, "kv_from", None)
             if j is None:
                 continue
@@ -79,9 +90,16 @@ class StackConfig(ModelConfig):
         a, b, times = self.loop
         return list(range(a)) + list(range(a, b)) * times + list(range(b, n))
 
+    def restarts(self) -> set:
+        """The passes (indices into `runs`) that begin a repetition of the loop."""
+        if self.loop is None:
+            return set()
+        a, b, times = self.loop
+        return {a + t * (b - a) for t in range(1, times)} if b > a else set()
+
     # ---- what the engine's cache manager allocates, per pass
-    def kv_rows(self) -> list:
-        return [self.layer_specs[i].mixer.kv_rows() for i in self.runs()]
+    def kv_rows(self, dtype: Optional[torch.dtype] = None) -> list:
+        return [self.layer_specs[i].mixer.kv_rows(dtype or self.dtype) for i in self.runs()]
 
     def kv_sources(self) -> list:
         """Per pass, the pass whose cache its attention reads: its own, or the last pass of the layer it shares with."""
@@ -156,6 +174,30 @@ class StackConfig(ModelConfig):
         return cls._tovalix(4096, 16384, 32, 8, 128, 64, 64, 32, 128, 128, 30, 1024, 128)
 
 
+    @classmethod
+    def _zikezen(cls, D, ff, heads, kv, dim, mh, mdim, mvdim, n, loop, window, experts, top, eff, side, rank=64, vocab=151936,
+                 positions=16384, rot=None) -> "StackConfig":
+        att = RotaryAttentionSpec(heads=heads, kv_heads=kv, dim=dim, vdim=dim, scale=dim ** -0.5, rot_dims=rot or dim // 2,
+                                  rot_base=500000.0, window=window, interleaved=True, rot_scaling=(8.0, 1.0, 4.0, positions // 2),
+                                  head_weights=True, sink=0.0, out_bias=False, fit_heads=True)
+        mixer = SumSpec(att, GatedLinearSpec(mh, mdim, mvdim, 16.0, rank), 0.7, 0.6)
+        specs = tuple(LayerSpec(mixer, eff, "experts", experts, top) if i % 2 else LayerSpec(mixer, ff) for i in range(n))
+        return cls(family="zikezen", vocab_size=vocab, embed_dim=D, layer_specs=specs, loop=loop, token_side=side, embed_factor=2.0,
+                   positions=positions, max_position=positions, loop_embed=True, post_norms=True, final_logit_softcap=30.0)
+
+    @classmethod
+    def zikezen_tiny(cls) -> "StackConfig":
+        return cls._zikezen(96, 160, 4, 2, 24, 3, 16, 32, 4, (1, 3, 2), 24, 6, 2, 40, 8, rank=8, vocab=384, positions=512)
+
+    @classmethod
+    def zikezen_2b(cls) -> "StackConfig":
+        return cls._zikezen(2048, 4096, 16, 8, 128, 16, 64, 128, 14, (4, 10, 2), 1024, 32, 4, 1024, 64)
+
+    @classmethod
+    def zikezen_8b(cls) -> "StackConfig":
+        return cls._zikezen(4096, 8192, 32, 8, 128, 32, 64, 128, 16, (5, 11, 2), 1024, 32, 4, 2048, 128)
+
+
 # ------------------------------------------------------------------------------------------ config.json reader
 def _parallel_spec(m: dict, shapes, prefix: str, width: int) -> ParallelSpec:
     lf, rt = m["left"], m["right"]
@@ -180,6 +222,24 @@ def _rotary_spec(m: dict, shapes, prefix: str, width: int) -> RotaryAttentionSpe
                                kv_from=None if m.get("kv_from") is None else int(m["kv_from"]))
 
 
+def _rot_scaling(rot: dict) -> Optional[tuple]:
+    s = rot.get("scaling")
+    return None if not s else (float(s["factor"]), float(s["low"]), float(s["high"]), float(s["original"]))
+
+
+def _sum_spec(m: dict, shapes, prefix: str, width: int) -> SumSpec:
+    lf, rt = m["left"], m["right"]
+    mask, rot = lf.get("mask") or {}, lf.get("rot") or {}
+    left = RotaryAttentionSpec(heads=int(lf["heads"]), kv_heads=int(lf["kv_heads"]), dim=int(lf["dim"]), vdim=int(lf["vdim"]),
+                               scale=float(lf["scale"]), rot_dims=int(rot.get("dims") or 0), rot_base=float(rot.get("base") or 1.0),
+                               window=int(mask.get("size") or 0), interleaved=True, rot_scaling=_rot_scaling(rot), head_weights=True,
+                               sink=0.0, out_bias=False, fit_heads=True)
+    a1 = (shapes or {}).get(prefix + "right.a1")
+    right = GatedLinearSpec(heads=int(rt["heads"]), dim=int(rt["dim"]), vdim=int(rt["vdim"]), tau=float(rt["tau"]),
+                            decay_rank=int(a1[0]) if a1 else 16)
+    return SumSpec(left, right, float(m["left_scale"]), float(m["right_scale"]))
+
+
 def _wkv_spec(m: dict, shapes, prefix: str, width: int) -> TokenShiftMemorySpec:
     w1 = (shapes or {}).get(prefix + "w1")
     return TokenShiftMemorySpec(heads=int(m["heads"]), dim=int(m["dim"]), decay_rank=int(w1[0]) if w1 else 64, width=width)
@@ -195,11 +255,15 @@ class Design:
     mixers: dict                        # layer type in config.json -> reader of its mixer
     ff_kind: str                        # what a "dense" feed-forward is
     embed_norm: bool = False
+    experts: bool = False               # layers may have a mixture of experts
+    post_norms: bool = False            # a norm behind every sublayer
+    loop_embed: bool = False
 
 
 ARCHITECTURES = {
     "Roluzen": Design("roluzen", {"rglru": _rglru_spec, "parallel": _parallel_spec}, "glu"),
     "Tovalix": Design("tovalix", {"wkv": _wkv_spec, "hgrn2": _hgrn2_spec, "attention": _rotary_spec}, "xielu", embed_norm=True),
+    "Zikezen": Design("zikezen", {"parallel": _sum_spec}, "glu", experts=True, post_norms=True, loop_embed=True),
 }
 STACK_FAMILIES = tuple(d.family for d in ARCHITECTURES.values())
 
@@ -234,16 +298,26 @@ def config_from_stack_json(src: Union[str, dict], dtype: Optional[torch.dtype] =
         if layer["type"] not in design.mixers:
             raise ValueError(f"layer {i}: no mixer {layer['type']!r} in this framework")
         mlp = layer.get("mlp")
-        if mlp is not None and mlp.get("kind") != "dense":
+        mixer = design.mixers[layer["type"]](layer["mixer"], shapes, f"l{i}.mix.", width)
+        if mlp is None:
+            specs.append(LayerSpec(mixer, None, design.ff_kind))
+        elif mlp.get("kind") == "dense":
+            specs.append(LayerSpec(mixer, int(mlp["ff"]), design.ff_kind))
+        elif mlp.get("kind") == "moe" and design.experts:
+            specs.append(LayerSpec(mixer, int(mlp["expert"]["ff"]), "experts", int(mlp["router"]["experts"]), int(mlp["router"]["top"])))
+        else:
             raise ValueError(f"layer {i}: no feed-forward {mlp.get('kind')!r} in this framework")
-        specs.append(LayerSpec(design.mixers[layer["type"]](layer["mixer"], shapes, f"l{i}.mix.", width),
-                               None if mlp is None else int(mlp["ff"]), design.ff_kind))
     lp = c.get("loop")
+    positions = int(c.get("max_positions") or 0)
     kw = dict(family=design.family, vocab_size=int(c["vocab"]), embed_dim=width, norm_groups=int(c["norm"].get("groups") or 1),
               embed_norm=design.embed_norm, token_side=int((c.get("token_side") or {}).get("dim") or 0),
               norm_eps=float(c["norm"]["eps"]), layer_specs=tuple(specs),
               loop=None if not lp else (int(lp["start"]), int(lp["stop"]), int(lp["times"])),
-              streams=int(c.get("streams") or 0), dtype=dtype or torch.bfloat16)
+              streams=int(c.get("streams") or 0), dtype=dtype or torch.bfloat16, post_norms=design.post_norms,
+              loop_embed=design.loop_embed, embed_factor=float((c.get("embedding") or {}).get("scale") or 1.0),
+              final_logit_softcap=float(c.get("logit_softcap") or 0.0), positions=positions)
+    if positions:
+        kw["max_position"] = positions
     kw.update(overrides)
     return StackConfig(**kw)
 
@@ -270,6 +344,20 @@ class PlainMLP(nn.Module):
         self.act = nn.Parameter(torch.full((2,), 0.5, dtype=dtype, device=device))
 
 
+class ExpertsMLP(nn.Module):
+    """sum_j s_j expert_j(x) over the `top` experts with the largest softmax score + correction, weighted by the score itself;
+    an expert is silu-gated. Expert weights are stacked [E, F, D] (gate, up) and [E, D, F] (down)."""
+
+    def __init__(self, width: int, ff: int, experts: int, top: int, dtype, device=None):
+        super().__init__()
+        self.top = top
+        self.router = Linear(width, experts, False, dtype, device)
+        self.correction = nn.Parameter(torch.zeros(experts, dtype=dtype, device=device))
+        self.gate_proj = nn.Parameter(torch.empty(experts, ff, width, dtype=dtype, device=device))
+        self.up_proj = nn.Parameter(torch.empty(experts, ff, width, dtype=dtype, device=device))
+        self.down_proj = nn.Parameter(torch.empty(experts, width, ff, dtype=dtype, device=device))
+
+
 class TokenSide(nn.Module):
     """A layer's token input: norm(proj(gelu(gate x) * e))."""
 
@@ -288,12 +376,19 @@ class StackLayer(nn.Module):
         self.input_layernorm = RMSNorm(D, eps, False, dt, device)
         self.mixer = create_mixer(spec.mixer, D, eps, dt, device)
         self.hc1 = HyperConnection(cfg.streams, dt, device) if cfg.streams else None
-        self.post_attention_layernorm = self.mlp = self.hc2 = None
+        self.post_attention_layernorm = self.mlp = self.hc2 = self.post_attn_norm = self.post_ffw_norm = None
+        if cfg.post_norms:
+            self.post_attn_norm = RMSNorm(D, eps, False, dt, device)
         if spec.ff is not None:
             self.post_attention_layernorm = RMSNorm(D, eps, False, dt, device)
-            # the generic gated MLP reads only these sizes
-            self.mlp = PlainMLP(D, spec.ff, dt, device) if spec.ff_kind == "xielu" else \
-                MLP(ModelConfig(embed_dim=D, hidden_dim=spec.ff, activation=cfg.activation, dtype=dt), device)
+            if cfg.post_norms:
+                self.post_ffw_norm = RMSNorm(D, eps, False, dt, device)
+            if spec.ff_kind == "experts":
+                self.mlp = ExpertsMLP(D, spec.ff, spec.experts, spec.top, dt, device)
+            elif spec.ff_kind == "xielu":
+                self.mlp = PlainMLP(D, spec.ff, dt, device)
+            else:                       # the generic gated MLP reads only these sizes
+                self.mlp = MLP(ModelConfig(embed_dim=D, hidden_dim=spec.ff, activation=cfg.activation, dtype=dt), device)
             self.hc2 = HyperConnection(cfg.streams, dt, device) if cfg.streams else None
         self.side = TokenSide(D, cfg.token_side, eps, dt, device) if cfg.token_side else None
 
@@ -305,7 +400,9 @@ class StackModel(nn.Module):
         dt = cfg.dtype
         self.embed_tokens = nn.Parameter(torch.empty(cfg.vocab_size, cfg.embed_dim, dtype=dt, device=device))
         self.embed_norm = RMSNorm(cfg.embed_dim, cfg.norm_eps, False, dt, device) if cfg.embed_norm else None
-        self.side_embed = None
+        self.pos_embed = self.side_embed = None
+        if cfg.positions:
+            self.pos_embed = nn.Parameter(torch.empty(cfg.positions, cfg.embed_dim, dtype=dt, device=device))
         if cfg.token_side:          # row of a token: one part of `token_side` columns per layer
             self.side_embed = nn.Parameter(torch.empty(cfg.vocab_size, cfg.num_layers * cfg.token_side, dtype=dt, device=device))
         self.layers = nn.ModuleList([StackLayer(cfg, s, device) for s in cfg.layer_specs])
@@ -364,6 +461,8 @@ class StackModel(nn.Module):
             raise NotImplementedError("packed rows (several segments) are not scored by layer-stack models")
         toks = input_tokens.cpu()
         rows = [toks[b][keep[b]].tolist() for b in range(B)]
+        if self.config.positions and max(map(len, rows), default=0) > self.config.positions:
+            raise ValueError(f"rows of more than {self.config.positions} tokens: the model has no position beyond")
         pages = [-(-max(len(r), 1) // 64) for r in rows]
         pool = PagePool(self.config, sum(pages), 64, B, max(pages), dev, self.config.dtype, prefix_caching=False)
         work = []

@@ -6,6 +6,7 @@ read and norm). Projections that share an input run as one GEMM over weights joi
 package's tcgen05 GEMMs, with fp32 accumulation; 32-bit models use library GEMMs in full precision (no TF32)."""
 from __future__ import annotations
 
+import math
 from typing import Callable, Optional
 
 import torch
@@ -13,15 +14,20 @@ import torch
 from ..ops import kernels as K
 from ..ops import stack_kernels as SK
 from ..ops.ragged import RaggedBatch
-from .mixers import ForgetGateMemory, ParallelMixer, RGLRUMixer, RotaryAttention, TokenShiftMemory
-from .stack import PlainMLP
+from .mixers import (TILE_HEADS, ForgetGateMemory, GatedLinearAttention, ParallelMixer, RGLRUMixer, RotaryAttention, SumMixer,
+                     TokenShiftMemory)
+from .stack import ExpertsMLP, PlainMLP
+
+
+def _plain(mods) -> None:
+    if any(m.quant is not None or (m.lora_a is not None and m.lora_enabled) for m in mods):
+        raise NotImplementedError("layer-stack models run without adapters or quantised weights")
 
 
 def joint_weight(mods):
     """One [sum(out_i), in] tensor over the weights of `mods` (moved there once; the modules keep views), and the joint
-    bias or None. Adapters and quantised bases are not supported on these models."""
-    if any(m.quant is not None or (m.lora_a is not None and m.lora_enabled) for m in mods):
-        raise NotImplementedError("layer-stack models run without adapters or quantised weights")
+    bias (zeros for modules without one) or None. Adapters and quantised bases are not supported on these models."""
+    _plain(mods)
     ws = [m.weight for m in mods]
     rows, base = sum(w.shape[0] for w in ws), ws[0].data
     off, adjacent = base.storage_offset(), True
@@ -38,8 +44,32 @@ def joint_weight(mods):
         for w in ws:
             w.data = joint[r:r + w.shape[0]]
             r += w.shape[0]
-    bias = torch.cat([m.bias.data for m in mods]) if mods[0].bias is not None else None
+    bias = None
+    if any(m.bias is not None for m in mods):
+        bias = torch.cat([m.weight.new_zeros(m.weight.shape[0]) if m.bias is None else m.bias.data for m in mods])
     return joint, bias
+
+
+def side_by_side(params, dim: int) -> torch.Tensor:
+    """The parameters joined along `dim` in one contiguous tensor (moved there once; they stay views of it)."""
+    sizes = [p.shape[dim] for p in params]
+    shape = list(params[0].shape)
+    shape[dim] = sum(sizes)
+    base, off = params[0].data, 0
+    stride = [1] * len(shape)
+    for i in range(len(shape) - 2, -1, -1):
+        stride[i] = stride[i + 1] * shape[i + 1]
+    for p, n in zip(params, sizes):
+        if p.data.untyped_storage().data_ptr() != base.untyped_storage().data_ptr() or list(p.stride()) != stride or \
+                p.storage_offset() != base.storage_offset() + off * stride[dim]:
+            break
+        off += n
+    else:
+        return base.as_strided(shape, stride, base.storage_offset())
+    joint = torch.cat([p.data for p in params], dim)
+    for p, part in zip(params, joint.split(sizes, dim)):
+        p.data = part
+    return joint
 
 
 def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None,
@@ -50,6 +80,8 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
         if packed is not None:
             return K.gemm_packed(x, packed, bias=bias, out_dtype=out_dtype)
         if x.shape[1] % 8 == 0:
+            if x.stride(0) % 8 or x.data_ptr() % 16:        # columns of a wider row that TMA cannot address
+                x = x.contiguous()
             return K.gemm(x, w, bias=bias, out_dtype=out_dtype)
     prev = torch.backends.cuda.matmul.allow_tf32
     torch.backends.cuda.matmul.allow_tf32 = False
@@ -64,9 +96,22 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
 FEW_OUTPUTS = 512       # in a decode step, products with at most this many outputs split the contraction inside a CTA
 
 
-def rope_table(positions: int, dims: int, base: float, device) -> tuple:
-    """cos / sin fp32 [positions, dims / 2] of the angles position * base^(-2 i / dims), from fp64."""
+def rope_frequencies(dims: int, base: float, scaling: Optional[tuple] = None, device=None) -> torch.Tensor:
+    """fp64 [dims / 2]: base^(-2 i / dims). `scaling` = (factor, low, high, original context), as Llama 3.1 has it: frequencies
+    that turn fewer than `low` times over the original context are divided by the factor, those that turn more than `high` times
+    stay, in between the two are mixed linearly in the number of turns."""
     f = base ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64, device=device) / max(dims, 1))
+    if scaling is None:
+        return f
+    factor, low, high, original = scaling
+    turns = original * f / (2.0 * math.pi)
+    keep = ((turns - low) / (high - low)).clamp(0.0, 1.0) if high > low else (turns >= low).to(f.dtype)
+    return torch.where(turns > high, f, torch.where(turns < low, f / factor, (1.0 - keep) * f / factor + keep * f))
+
+
+def rope_table(positions: int, dims: int, base: float, device, scaling: Optional[tuple] = None) -> tuple:
+    """cos / sin fp32 [positions, dims / 2] of the angles position * frequency, from fp64."""
+    f = rope_frequencies(dims, base, scaling, device)
     a = torch.arange(positions, dtype=torch.float64, device=device)[:, None] * f
     return a.cos().float(), a.sin().float()
 
@@ -78,7 +123,9 @@ class StackExecutor:
         self.runs = self.cfg.runs()
         self.kv_src = self.cfg.kv_sources()
         self._mix = {RGLRUMixer: self._rglru, ParallelMixer: self._parallel, RotaryAttention: self._rotary,
-                     TokenShiftMemory: self._shift_memory, ForgetGateMemory: self._forget_memory}
+                     TokenShiftMemory: self._shift_memory, ForgetGateMemory: self._forget_memory,
+                     GatedLinearAttention: self._gated_linear, SumMixer: self._sum}
+        self.restarts = self.cfg.restarts() if self.cfg.loop_embed else set()
         self._rope: dict = {}       # kept for good: captured decode graphs point at the tables
         self.dtype = model.embed_tokens.dtype
         self.pk: Callable = lambda i, name: None        # packed decode weights, set by the engine
@@ -104,8 +151,15 @@ class StackExecutor:
                 d["gates_bias"] = None
             if isinstance(layer.mixer, TokenShiftMemory):
                 d["mu"] = layer.mixer.mu()
+            if isinstance(layer.mixer, SumMixer):
+                outs = [layer.mixer.left.o_proj, layer.mixer.right.o_proj]
+                _plain(outs)
+                d["o"] = side_by_side([m.weight for m in outs], 1)
             if isinstance(layer.mlp, PlainMLP):
                 d["up"], _ = joint_weight([layer.mlp.up_proj])
+            elif isinstance(layer.mlp, ExpertsMLP):
+                _plain([layer.mlp.router])
+                d["experts_gu"] = side_by_side([layer.mlp.gate_proj, layer.mlp.up_proj], 1)
             elif layer.mlp is not None:
                 d["gu"], _ = joint_weight([layer.mlp.gate_proj, layer.mlp.up_proj])
             fresh.append(d)
@@ -121,8 +175,8 @@ class StackExecutor:
         """Per layer, the weights the engine may keep in packed form for decoding (`PagedEngine._pack_all`)."""
         out = []
         for layer, d in zip(self.model.layers, self.w):
-            src = {k: d[k] for k in ("proj", "gates", "gu", "up") if k in d}
-            if layer.mlp is not None:
+            src = {k: d[k] for k in ("proj", "gates", "gu", "up", "o") if k in d}
+            if layer.mlp is not None and not isinstance(layer.mlp, ExpertsMLP):
                 src["down"] = layer.mlp.down_proj.weight.data
             out.append(src)
         return out
@@ -163,17 +217,24 @@ class StackExecutor:
         return (linear(a1, lf.o_proj.weight), linear(a2, rt.o_proj.weight), m.left_norm.weight, m.right_norm.weight)
 
     def _rotary(self, i, m: RotaryAttention, h, rb: RaggedBatch, pool, r):
-        d, a, src = self.w[i], m.spec, self.kv_src[r]
+        d = self.w[i]
         proj = linear(h, d["proj"], d["proj_bias"], packed=self.pk(i, "proj") if rb.decode else None)
-        key = (a.rot_dims, a.rot_base, pool.max_pages * pool.page_size)
+        att = self._rotary_heads(m, proj, rb, pool, r)
+        return (linear(att, m.o_proj.weight, m.o_proj.bias), None, None, None)
+
+    def _rotary_heads(self, m: RotaryAttention, proj, rb: RaggedBatch, pool, r, **kw):
+        """Attention of the projected rows (queries, keys and values in their first columns), before the output projection."""
+        a, src = m.spec, self.kv_src[r]
+        key = (a.rot_dims, a.rot_base, a.rot_scaling, pool.max_pages * pool.page_size)
         if key not in self._rope:
-            self._rope[key] = rope_table(key[2], a.rot_dims, a.rot_base, h.device)
+            self._rope[key] = rope_table(key[3], a.rot_dims, a.rot_base, proj.device, a.rot_scaling)
         cos, sin = self._rope[key]
         nq, kv = a.heads * a.dim, 0 if a.kv_from is not None else a.kv_heads
         q = SK.rope_norm_write(proj, 0, nq, nq + kv * a.dim, cos, sin, a.rot_dims, m.eps, rb, pool.table, pool.page_size, a.heads,
-                               kv, a.dim, a.vdim, pool.k[src], pool.v[src])
-        att = self._attend(q, a, None, rb, pool, src)
-        return (linear(att, m.o_proj.weight, m.o_proj.bias), None, None, None)
+                               kv, a.dim, a.vdim, pool.k[src], pool.v[src], q_w=None if m.q_norm is None else m.q_norm.weight,
+                               k_w=None if m.k_norm is None else m.k_norm.weight, interleaved=a.interleaved,
+                               stored=a.stored(proj.dtype))
+        return self._attend(q, a, None, rb, pool, src, **kw)
 
     def _shift_memory(self, i, m: TokenShiftMemory, h, rb: RaggedBatch, pool, r):
         """h: the mixes [5, n, D] in a decode step (made by the launch before), else the normed rows."""
@@ -194,6 +255,32 @@ class StackExecutor:
                             pool.state[r]["S"], m.norm.weight, m.eps, plain=self.plain)
         return (linear(o, m.o_proj.weight), None, None, None)
 
+    def _gated_linear(self, i, m: GatedLinearAttention, h, rb: RaggedBatch, pool, r):
+        proj = linear(h, self.w[i]["proj"], packed=self.pk(i, "proj") if rb.decode else None)
+        return (linear(self._gated_heads(m, proj, rb, pool, r), m.o_proj.weight), None, None, None)
+
+    def _gated_heads(self, m: GatedLinearAttention, proj, rb: RaggedBatch, pool, r, **kw):
+        """The memory's read-outs, normed and gated, from the projected rows (q, k, v, gate, bottleneck)."""
+        sp = m.spec
+        nk, nv = sp.heads * sp.dim, sp.heads * sp.vdim
+        q, k, v, g, x = proj.split([nk, nk, nv, nv, sp.decay_rank], 1)
+        low = (x, m.a2_proj.weight)
+        z = None if rb.decode and not self.plain and sp.vdim <= SK.STEP_WIDTH else linear(x, m.a2_proj.weight, out_dtype=torch.float32)
+        return SK.gated_linear(SK.GATES_ROOT, q, k, v, z, m.a2_proj.bias, None, rb, sp.heads, sp.dim, sp.vdim, pool.state[r]["S"],
+                               m.norm.weight, m.eps, gate=g, plain=self.plain, low_rank=low, q_scale=sp.dim ** -0.5, tau=sp.tau, **kw)
+
+    def _sum(self, i, m: SumMixer, h, rb: RaggedBatch, pool, r):
+        """Both mixers' heads land, scaled, in one row, which a single product takes to the residual's width."""
+        d, sp = self.w[i], m.spec
+        a, s = sp.left, sp.right
+        proj = linear(h, d["proj"], d["proj_bias"], packed=self.pk(i, "proj") if rb.decode else None)
+        na, ns = a.heads * a.vdim, s.heads * s.vdim
+        o = torch.empty((h.shape[0], na + ns), dtype=h.dtype, device=h.device)
+        left = a.heads * a.dim + a.kv_heads * (a.dim + a.vdim)
+        self._rotary_heads(m.left, proj, rb, pool, r, out=o[:, :na], out_scale=sp.left_scale)
+        self._gated_heads(m.right, proj[:, left:], rb, pool, r, out=o[:, na:], out_scale=sp.right_scale)
+        return (linear(o, d["o"], packed=self.pk(i, "o") if rb.decode else None), None, None, None)
+
     def _few(self, x, w, rb: RaggedBatch, act: int, **rows) -> torch.Tensor:
         """act(x w^T) for narrow w."""
         if rb.decode and x.dtype == torch.bfloat16 and x.shape[1] % 8 == 0 and w.shape[0] <= FEW_OUTPUTS:
@@ -205,28 +292,33 @@ class StackExecutor:
         y = self._few(x, side.gate_proj.weight, rb, SK.ACT_GELU_ROW, tokens=rb.tokens, rows=self.model.side_embed, col=i * dim)
         return (linear(y, side.proj.weight), None, side.norm.weight, None)
 
-    def _attend(self, q, a, bias, rb: RaggedBatch, pool, r):
-        """Tensor-core kernels where the heads fit them (the framework's paged decode and flash attention, extended by the
-        bias and the kept tokens); otherwise, and in 32-bit, the general kernel."""
-        fits = q.dtype == torch.bfloat16 and a.dim == a.vdim and a.dim in (64, 128, 256) and not self.plain
-        kw = dict(scale=a.scale, softcap=a.softcap, window=a.window, chunk=a.chunk, keep_first=a.keep_first, bias=bias)
+    def _attend(self, q, a, bias, rb: RaggedBatch, pool, r, out=None, out_scale: float = 1.0):
+        """Tensor-core kernels where the stored heads fit them (the framework's paged decode and flash attention, extended by the
+        bias, the kept tokens and the sink); otherwise, and in 32-bit, the general kernel. `out`: columns that take the result."""
+        wide, wide_v = a.stored(q.dtype)
+        fits = q.dtype == torch.bfloat16 and wide == wide_v and wide in TILE_HEADS and not self.plain and a.vdim % 8 == 0 and \
+            (out is None or (out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0))
+        kw = dict(scale=a.scale, softcap=a.softcap, window=a.window, chunk=a.chunk, keep_first=a.keep_first, sink=a.sink, bias=bias,
+                  value_dim=a.vdim, out=out, out_scale=out_scale)
         if fits and rb.decode and a.heads // a.kv_heads <= 16:
             max_ctx = pool.table.shape[1] * pool.page_size
             span = min((s for s in (a.window, a.chunk) if s > 0), default=0)       # most keys a query sees besides the kept ones
             split = K.decode_split_tokens(rb.n, a.kv_heads, min(max_ctx, span + a.keep_first + 128) if span else max_ctx)
-            return K.paged_decode(q.view(rb.n, a.heads, a.dim), pool.k[r], pool.v[r], pool.table, rb.slot, self._lens,
+            return K.paged_decode(q.view(rb.n, a.heads, wide), pool.k[r], pool.v[r], pool.table, rb.slot, self._lens,
                                   num_kv_heads=a.kv_heads, page_size=pool.page_size, max_ctx=max_ctx, split_tokens=split,
                                   **kw).view(rb.n, -1)
         if fits and not rb.decode and pool.page_size % 64 == 0:
             return K.attn_fwd_paged(q, pool.k[r], pool.v[r], rb, pool.table, pool.page_size, num_heads=a.heads,
-                                    num_kv_heads=a.kv_heads, head_dim=a.dim, **kw)
-        return SK.window_attn(q, pool.k[r], pool.v[r], rb, pool.table, pool.page_size, a, bias)
+                                    num_kv_heads=a.kv_heads, head_dim=wide, **kw)
+        return SK.window_attn(q, pool.k[r], pool.v[r], rb, pool.table, pool.page_size, a, bias, out=out, out_scale=out_scale)
 
     def _mlp(self, i, mlp, h, rb: RaggedBatch):
         if isinstance(mlp, PlainMLP):
             pup = self.pk(i, "up") if rb.decode else None
             act = K.gemm_packed(h, pup, xielu=mlp.act) if pup is not None else SK.xielu_(linear(h, self.w[i]["up"]), mlp.act)
             return linear(act, mlp.down_proj.weight, packed=self.pk(i, "down") if rb.decode else None)
+        if isinstance(mlp, ExpertsMLP):
+            return SK.moe(h, self._router(h, mlp.router.weight, rb), mlp.correction, self.w[i]["experts_gu"], mlp.down_proj, mlp.top, rb)
         gu_w = self.w[i]["gu"]
         F = gu_w.shape[0] // 2
         pgu = self.pk(i, "gu") if rb.decode else None
@@ -237,6 +329,12 @@ class StackExecutor:
             act = K.glu_fwd(gu[:, :F], gu[:, F:], K.GLU_SILU) if gu.dtype == torch.bfloat16 and F % 8 == 0 else SK.silu_mul(gu)
         return linear(act, mlp.down_proj.weight, packed=self.pk(i, "down") if rb.decode else None)
 
+    def _router(self, h, w, rb: RaggedBatch) -> torch.Tensor:
+        """fp32 router logits."""
+        if h.dtype == torch.bfloat16 and h.shape[1] % 8 == 0 and (rb.n <= SK.ROWS_TOKENS and w.shape[0] <= FEW_OUTPUTS):
+            return SK.few_outputs(h, w)
+        return linear(h, w, out_dtype=torch.float32)
+
     # ------------------------------------------------------------------------------------------------ the stack
     @torch.no_grad()
     def forward(self, rb: RaggedBatch, pool, layer_sums: Optional[list] = None) -> torch.Tensor:
@@ -245,11 +343,14 @@ class StackExecutor:
         cfg, model = self.cfg, self.model
         eps, n = cfg.norm_eps, rb.n
         x = torch.empty((n, max(cfg.streams, 1), cfg.embed_dim), dtype=torch.float32, device=rb.tokens.device)
-        close = dict(tokens=rb.tokens, embed=model.embed_tokens,       # what the next stream_step closes
-                     embed_w=None if model.embed_norm is None else model.embed_norm.weight)
+        start = dict(tokens=rb.tokens, embed=model.embed_tokens, embed_w=None if model.embed_norm is None else model.embed_norm.weight,
+                     embed_scale=cfg.embed_factor, pos=model.pos_embed)
+        close = start                                                  # what the next stream_step closes
 
-        def pending(out, hc):
+        def pending(out, hc, norm=None):
             y, y2, wy, wy2 = out
+            if norm is not None:
+                wy = norm.weight
             _, w_out, mix = self._hc(hc)
             return dict(y=y, y2=y2, wy=wy, wy2=wy2, mix=mix, w_out=w_out)
 
@@ -263,17 +364,19 @@ class StackExecutor:
                 total = torch.empty((n, cfg.embed_dim), dtype=torch.float32, device=x.device)
                 layer_sums.append(total)
             ended = False
-            return SK.stream_step(x, eps, groups=cfg.norm_groups, w_in=w_in, norm_w=norm_w, sum_out=total, **close, **kw)
+            return SK.stream_step(x, eps, groups=cfg.norm_groups, w_in=w_in, norm_w=norm_w, sum_out=total, rb=rb, **close, **kw)
 
         for r, i in enumerate(self.runs):
             layer = model.layers[i]
             shifts = rb.decode and isinstance(layer.mixer, TokenShiftMemory)
+            if r in self.restarts:
+                close = dict(close, **start)
             h = step(self._hc(layer.hc1)[0], layer.input_layernorm.weight,
-                     **(dict(shift=(self.w[i]["mu"], pool.state[r]["last"]), rb=rb) if shifts else {}))
-            close = pending(self._mix[type(layer.mixer)](i, layer.mixer, h, rb, pool, r), layer.hc1)
+                     **(dict(shift=(self.w[i]["mu"], pool.state[r]["last"])) if shifts else {}))
+            close = pending(self._mix[type(layer.mixer)](i, layer.mixer, h, rb, pool, r), layer.hc1, layer.post_attn_norm)
             if layer.mlp is not None:
                 h = step(self._hc(layer.hc2)[0], layer.post_attention_layernorm.weight)
-                close = pending((self._mlp(i, layer.mlp, h, rb), None, None, None), layer.hc2)
+                close = pending((self._mlp(i, layer.mlp, h, rb), None, None, None), layer.hc2, layer.post_ffw_norm)
             if layer.side is not None:
                 close = pending(self._side(i, layer.side, step(None, None, raw=True), rb), None)
             ended = True

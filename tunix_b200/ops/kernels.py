@@ -283,13 +283,17 @@ _lib.register_cuda_sigs({
     "tb_attn_fwd": [_lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.I, _lib.I, _lib.I, _lib.I, _lib.I, _lib.I,
                     _lib.LL, _lib.LL, _lib.LL, _lib.LL, _lib.F, _lib.F, _lib.I, _lib.I, _lib.I, _lib.P, _lib.P,
                     _lib.P, _lib.P],
-    "tb_attn_fwd_paged": [_lib.P, _lib.P, _lib.P, _lib.P, _lib.I, _lib.LL, _lib.I, _lib.I, _lib.I, _lib.F, _lib.F, _lib.I, _lib.I,
-                          _lib.I, _lib.P, _lib.I, _lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.I, _lib.P, _lib.I, _lib.I, _lib.P, _lib.P],
+    "tb_attn_fwd_paged": [_lib.P, _lib.P, _lib.P, _lib.P, _lib.LL, _lib.I, _lib.LL, _lib.I, _lib.I, _lib.I, _lib.I, _lib.F, _lib.F,
+                          _lib.I, _lib.I, _lib.I, _lib.F, _lib.F, _lib.P, _lib.I, _lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.I,
+                          _lib.P, _lib.I, _lib.I, _lib.P, _lib.P],
     "tb_attn_delta": [_lib.P, _lib.LL, _lib.P, _lib.LL, _lib.P, _lib.I, _lib.I, _lib.I, _lib.I, _lib.P],
     "tb_attn_bwd": [_lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.I, _lib.I,
                     _lib.I, _lib.I, _lib.I, _lib.I, _lib.LL, _lib.LL, _lib.LL, _lib.LL, _lib.LL, _lib.LL,
                     _lib.F, _lib.F, _lib.I, _lib.I, _lib.I, _lib.P, _lib.P, _lib.P, _lib.P],
 })
+
+
+NO_SINK = float("-inf")
 
 
 def _attn_views(q, k, v):
@@ -321,17 +325,22 @@ def attn_fwd(q, k, v, *, scale: float, causal: bool = True, window: int = 0, sof
 
 
 def attn_fwd_paged(q, k_pool, v_pool, rb, table, page_size: int, *, num_heads: int, num_kv_heads: int, head_dim: int, scale: float,
-                   softcap: float = 0.0, window: int = 0, chunk: int = 0, keep_first: int = 0, bias=None) -> torch.Tensor:
+                   softcap: float = 0.0, window: int = 0, chunk: int = 0, keep_first: int = 0, sink: float = NO_SINK, bias=None,
+                   out=None, value_dim: int = 0, out_scale: float = 1.0) -> torch.Tensor:
     """Flash attention of the entries of a `ops.ragged.RaggedBatch` (prompt portions) over the paged cache that already
-    holds their keys and values. q [n, N * H] bf16 -> [n, N * H]; pools [pages, page_size, KH * H], page_size a multiple of
-    64. `softcap` / `window` / `chunk` / `keep_first` / `bias` as in `paged_decode`."""
-    n = q.shape[0]
+    holds their keys and values. q [n, N * H] bf16 -> [n, N * value_dim]; pools [pages, page_size, KH * H], page_size a multiple
+    of 64. `softcap` / `window` / `chunk` / `keep_first` / `sink` / `bias` / `out_scale` as in `paged_decode`. `value_dim` (0: H):
+    the heads' values stand in the first columns of the stored ones. `out`: columns of wider rows."""
+    n, vd = q.shape[0], value_dim or head_dim
     assert q.is_contiguous() and page_size % 64 == 0 and k_pool.is_contiguous() and k_pool.shape == v_pool.shape
-    out = torch.empty_like(q)
+    if out is None:
+        out = torch.empty((n, num_heads * vd), dtype=q.dtype, device=q.device)
+    assert out.shape == (n, num_heads * vd) and out.stride(1) == 1
     t0, ent, _, tiles = rb.tiles(128)
-    rc = _lib.cuda().tb_attn_fwd_paged(q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(), out.data_ptr(), n,
-                                       k_pool.shape[0] * page_size, num_heads, num_kv_heads, head_dim, float(scale), float(softcap),
-                                       int(window), int(chunk), int(keep_first), _lib.ptr(bias), 0 if bias is None else bias.shape[1] - 1,
+    rc = _lib.cuda().tb_attn_fwd_paged(q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(), out.data_ptr(), out.stride(0), n,
+                                       k_pool.shape[0] * page_size, num_heads, num_kv_heads, head_dim, vd, float(scale), float(softcap),
+                                       int(window), int(chunk), int(keep_first), float(sink), float(out_scale), _lib.ptr(bias),
+                                       0 if bias is None else bias.shape[1] - 1,
                                        rb.cu.data_ptr(), rb.slot.data_ptr(), rb.pos0.data_ptr(), t0.data_ptr(), ent.data_ptr(),
                                        tiles, table.data_ptr(), table.shape[1], page_size,
                                        _lib.status_buffer(q.device).data_ptr(), _lib.stream_ptr())
@@ -372,8 +381,8 @@ def attn_bwd(dout, q, k, v, o, lse, *, scale: float, causal: bool = True, window
 _lib.register_cuda_sigs({
     "tb_kv_write": [_lib.P, _lib.P, _lib.LL, _lib.P, _lib.P, _lib.P, _lib.I, _lib.I, _lib.P, _lib.P, _lib.I, _lib.I, _lib.P],
     "tb_paged_decode": [_lib.P, _lib.LL, _lib.P, _lib.P, _lib.P, _lib.I, _lib.I, _lib.P, _lib.P, _lib.I, _lib.I, _lib.I,
-                        _lib.I, _lib.I, _lib.F, _lib.F, _lib.I, _lib.I, _lib.I, _lib.P, _lib.I, _lib.I, _lib.LL, _lib.P, _lib.P, _lib.P,
-                        _lib.LL, _lib.P, _lib.P],
+                        _lib.I, _lib.I, _lib.F, _lib.F, _lib.I, _lib.I, _lib.I, _lib.F, _lib.F, _lib.I, _lib.P, _lib.I, _lib.I, _lib.LL,
+                        _lib.P, _lib.P, _lib.P, _lib.LL, _lib.P, _lib.P],
     "tb_qkv_post": [_lib.P, _lib.LL, _lib.P, _lib.P, _lib.P, _lib.P, _lib.F, _lib.F, _lib.P, _lib.P, _lib.P, _lib.I,
                     _lib.I, _lib.P, _lib.P, _lib.I, _lib.I, _lib.I, _lib.I, _lib.P],
     "tb_decode_advance": [_lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.LL, _lib.P, _lib.P, _lib.P, _lib.I, _lib.LL, _lib.P,
@@ -444,9 +453,11 @@ def decode_split_tokens(batch: int, num_kv_heads: int, max_ctx: int = 0) -> int:
 
 
 def paged_decode(q, k_pool, v_pool, page_table, seq_ids, seq_lens, *, num_kv_heads: int, page_size: int, max_ctx: int,
-                 scale: float, softcap: float = 0.0, window: int = 0, chunk: int = 0, keep_first: int = 0, bias=None,
-                 workspace=None, out=None, split_tokens: int = 0):
-    """Single-token attention over a paged KV cache. q [B, N, H] bf16 (row stride free) -> out [B, N, H] bf16.
+                 scale: float, softcap: float = 0.0, window: int = 0, chunk: int = 0, keep_first: int = 0, sink: float = NO_SINK,
+                 bias=None, workspace=None, out=None, split_tokens: int = 0, value_dim: int = 0, out_scale: float = 1.0):
+    """Single-token attention over a paged KV cache. q [B, N, H] bf16 (row stride free) -> out [B, N, H] bf16, or with
+    `value_dim` [B, N, value_dim] (the heads' values stand in the first columns of the stored ones); `out` [B, N * value_dim] may
+    be columns of wider rows. `sink`: one more score in the sum of the weights, without a value. The output is scaled by `out_scale`.
     `chunk` > 0: a query sees the keys of its own chunk of that many positions, counted from the sequence's start.
     With a window or chunks, the first `keep_first` tokens of a sequence stay visible. `bias` fp32 [N, far + 1] is added to the
     scaled score of a key at distance min(distance, far).
@@ -461,14 +472,17 @@ def paged_decode(q, k_pool, v_pool, page_table, seq_ids, seq_lens, *, num_kv_hea
     if workspace is None:
         workspace = (torch.empty(B * N * splits * H, dtype=torch.float32, device=q.device),
                      torch.empty(B * N * splits * 2, dtype=torch.float32, device=q.device))
+    vd = value_dim or H
     if out is None:
-        out = torch.empty((B, N, H), dtype=q.dtype, device=q.device)
+        out = torch.empty((B, N, vd), dtype=q.dtype, device=q.device)
+    assert out.numel() == B * N * vd and out.stride(-1) == 1
     rc = _lib.cuda().tb_paged_decode(q.data_ptr(), q.stride(0), k_pool.data_ptr(), v_pool.data_ptr(), page_table.data_ptr(),
                                      page_table.shape[1], page_size, seq_ids.data_ptr(), seq_lens.data_ptr(), B, N,
                                      num_kv_heads, H, max_ctx, float(scale), float(softcap), int(window), int(chunk),
-                                     int(keep_first), _lib.ptr(bias), 0 if bias is None else bias.shape[1] - 1, int(split_tokens),
+                                     int(keep_first), float(sink), float(out_scale), vd, _lib.ptr(bias),
+                                     0 if bias is None else bias.shape[1] - 1, int(split_tokens),
                                      pool_rows, workspace[0].data_ptr(), workspace[1].data_ptr(),
-                                     out.data_ptr(), N * H, _lib.status_buffer(q.device).data_ptr(), _lib.stream_ptr())
+                                     out.data_ptr(), out.stride(0), _lib.status_buffer(q.device).data_ptr(), _lib.stream_ptr())
     _lib.check(rc, "tb_paged_decode")
     _count(2)
     return out
@@ -504,13 +518,13 @@ def _grouped_bn(n: int) -> int:
 
 def moe_tiles_rows(seg_off: torch.Tensor, max_rows: int, n_out: int, k_contract: int, b_rows_per_expert: int) -> TileList:
     """Tiles of a GEMM whose output rows are the permuted token rows: [max_rows, n_out] with the contraction
-    (k_contract, a multiple of 64) over the feature dimension and B = the stacked expert weights."""
-    assert k_contract % 64 == 0
+    k_contract over the feature dimension (the operands' inner one where it is no multiple of 64: reads past it are zeros) and
+    B = the stacked expert weights."""
     E = seg_off.numel() - 1
     bn = _grouped_bn(n_out)
     num_n = (n_out + bn - 1) // bn
     tl = TileList((max_rows // 128) * num_n, bn, seg_off.device)
-    rc = _lib.cuda().tb_moe_tiles_rows(seg_off.data_ptr(), E, num_n, bn, k_contract // 64, b_rows_per_expert,
+    rc = _lib.cuda().tb_moe_tiles_rows(seg_off.data_ptr(), E, num_n, bn, -(-k_contract // 64), b_rows_per_expert,
                                        tl.desc.data_ptr(), tl.count.data_ptr(), _lib.stream_ptr())
     _lib.check(rc, "tb_moe_tiles_rows")
     _count()

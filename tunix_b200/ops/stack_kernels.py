@@ -1,5 +1,5 @@
-"""Launchers of the layer-stack kernels (csrc/stack.cu, recurrent.cu, linear_attention.cu, window_attention.cu). Activations and weights are
-bf16 or float (the `dtype` argument of the entry points), residual streams, states and gates fp32."""
+"""Launchers of the layer-stack kernels (csrc/stack.cu, recurrent.cu, linear_attention.cu, window_attention.cu,
+moe_infer.cu). Activations and weights are bf16 or float (the `dtype` argument of the entry points), residual streams, states and gates fp32."""
 from __future__ import annotations
 
 from typing import Optional
@@ -7,19 +7,21 @@ from typing import Optional
 import torch
 
 from .. import _lib
+from . import kernels as K
 from .kernels import _count
 from .ragged import RaggedBatch
 
 _P, _I, _LL, _F = _lib.P, _lib.I, _lib.LL, _lib.F
 _RB = [_P, _P, _P, _P, _I, _I]
 _lib.register_cuda_sigs({
-    "tb_stream_step": [_I, _P, _I, _I, _I, _F, _P, _P, _P, _P, _P, _P, _P, _P, _I, _P, _I, _P, _P, _P, _P, _P, _I, _P, _P, _P, _P, _P],
+    "tb_stream_step": [_I, _P, _I, _I, _I, _F, _P, _P, _P, _P, _P, _P, _P, _P, _I, _P, _F, _P, _I, _I, _P, _P, _P, _P, _P, _I, _P, _P,
+                       _P, _P, _P, _P, _P],
     "tb_few_outputs": [_P, _P, _I, _I, _I, _I, _P, _I, _P, _LL, _I, _P, _I, _P],
     "tb_small_act": [_I, _P, _I, _I, _I, _P, _I, _P, _LL, _I, _P, _P],
     "tb_token_shift": [_I, _P, _P, _I, _P, *_RB, _I, _P, _P],
     "tb_xielu": [_I, _P, _P, _LL, _P],
-    "tb_gated_linear": [_I, _I, _P, _LL, _P, _LL, _P, _LL, _P, _LL, _P, _LL, _P, _P, *_RB, _I, _I, _I, _P, _P, _P, _I, _P, _I, _F,
-                        _P, _P, _I, _I, _P],
+    "tb_gated_linear": [_I, _I, _P, _LL, _P, _LL, _P, _LL, _P, _LL, _P, _LL, _P, _LL, _P, _I, _P, _P, _F, _F, *_RB, _I, _I, _I, _P, _P,
+                        _P, _I, _P, _I, _F, _F, _P, _P, _LL, _I, _I, _P],
     "tb_silu_mul": [_I, _P, _P, _LL, _I, _P],
     "tb_gate_outputs": [_I, _P, _P, _P, _LL, _I, _I, _P, _F, _I, _I, _I, _I, _P, _P, _P],
     "tb_rglru": [_I, _P, _LL, _I, _I, _P, _P, _P, _P, _P, _P, _P, *_RB, _I, _I, _I, _P, _P, _P, _P, _P, _P, _I, _P, _P,
@@ -27,8 +29,11 @@ _lib.register_cuda_sigs({
     "tb_mlstm_slices": [_I],
     "tb_mlstm": [_I, _P, _LL, _I, _I, _I, _P, _P, _P, _F, *_RB, _I, _I, _I, _P, _P, _P, _P, _I, _I, _P],
     "tb_qk_norm_write": [_I, _P, _LL, _I, _I, _I, _P, _P, _F, *_RB, _P, _I, _I, _I, _I, _I, _P, _P, _P, _P],
-    "tb_rope_norm_write": [_I, _P, _LL, _I, _I, _I, _P, _P, _I, _F, *_RB, _P, _I, _I, _I, _I, _I, _I, _P, _P, _P, _P],
-    "tb_window_attn": [_I, _P, _P, _P, *_RB, _P, _I, _I, _I, _I, _I, _I, _F, _F, _P, _I, _I, _I, _I, _P, _P],
+    "tb_rope_norm_write": [_I, _P, _LL, _I, _I, _I, _P, _P, _P, _P, _I, _I, _F, *_RB, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P, _P, _P],
+    "tb_window_attn": [_I, _P, _P, _P, *_RB, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _P, _I, _I, _I, _I, _F, _F, _P, _LL, _P],
+    "tb_moe_route": [_I, _P, _P, *_RB, _I, _I, _P, _P, _P, _P, _P, _P],
+    "tb_moe_route_lists": [_I, _P, _P, *_RB, _I, _I, _P, _P, _P, _P, _P],
+    "tb_moe_experts": [_I, _I, _P, _LL, _P, _P, _I, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P, _P],
 })
 
 
@@ -41,10 +46,11 @@ def _dt(t: torch.Tensor) -> int:
 
 
 def stream_step(x: torch.Tensor, eps: float, *, y=None, y2=None, wy=None, wy2=None, mix=None, w_out=None, tokens=None, embed=None,
-                embed_w=None, groups: int = 1, w_in=None, norm_w=None, raw: bool = False, shift=None, rb: Optional[RaggedBatch] = None,
-                sum_out: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+                embed_w=None, embed_scale: float = 1.0, pos=None, groups: int = 1, w_in=None, norm_w=None, raw: bool = False,
+                shift=None, rb: Optional[RaggedBatch] = None, sum_out: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
     """Close one sublayer (y [, y2 with their norms; y alone with its norm wy], mix, w_out; or start from the embedding rows
-    of `tokens`, normed with embed_w if given) and open the next: returns h = norm(sum_s w_in[s] x_s) * norm_w (w_in None:
+    of `tokens`, normed with embed_w if given, times embed_scale, plus the rows `pos` [positions, D] of the tokens' positions in
+    the batch `rb`; or both: the embedding rows are added to every stream after the sublayer, not to sum_out) and open the next: returns h = norm(sum_s w_in[s] x_s) * norm_w (w_in None:
     the plain sum; norm_w None: nothing follows, or with `raw` the sum itself). The norms of rows and embeddings are taken
     over `groups` equal parts. x fp32 [n, S, D] is updated in place; `sum_out` fp32 [n, D] receives the sum of the streams.
     `shift` = (mu [m, D], carry fp32 [slots, D]), for batches `rb` of single tokens: returns the m mixes
@@ -56,10 +62,10 @@ def stream_step(x: torch.Tensor, eps: float, *, y=None, y2=None, wy=None, wy2=No
     h = torch.empty((n, D), dtype=ref.dtype, device=x.device) if (norm_w is not None and not shift) or raw else None
     rc = _lib.cuda().tb_stream_step(_dt(ref), x.data_ptr(), n, S, D, float(eps), _lib.ptr(y), _lib.ptr(y2), _lib.ptr(wy),
                                     _lib.ptr(wy2), _lib.ptr(mix), _lib.ptr(w_out), _lib.ptr(tokens), _lib.ptr(embed),
-                                    0 if embed is None else embed.shape[0], _lib.ptr(embed_w), int(groups), _lib.ptr(w_in),
-                                    _lib.ptr(norm_w), _lib.ptr(h), _lib.ptr(sum_out), _lib.ptr(mu), 0 if mu is None else mu.shape[0],
-                                    _lib.ptr(carry), _lib.ptr(mixes), rb.slot.data_ptr() if shift else 0,
-                                    rb.pos0.data_ptr() if shift else 0, _lib.stream_ptr())
+                                    0 if embed is None else embed.shape[0], _lib.ptr(embed_w), float(embed_scale), _lib.ptr(pos),
+                                    0 if pos is None else pos.shape[0], int(groups), _lib.ptr(w_in), _lib.ptr(norm_w), _lib.ptr(h),
+                                    _lib.ptr(sum_out), _lib.ptr(mu), 0 if mu is None else mu.shape[0], _lib.ptr(carry),
+                                    _lib.ptr(mixes), *((0, 0, 0, 0) if rb is None else rb.args()[:4]), _lib.stream_ptr())
     _lib.check(rc, "tb_stream_step")
     _count()
     return mixes if shift else h
@@ -126,29 +132,36 @@ def small_act(z: torch.Tensor, dtype, act: int, tokens=None, rows=None, col: int
     return out
 
 
-GATES_BONUS, GATES_LOWER = 0, 1                 # csrc/linear_attention.cu: Mode
+GATES_BONUS, GATES_LOWER, GATES_ROOT = 0, 1, 2  # csrc/linear_attention.cu: Mode
+STEP_WIDTH = 256        # heads with wider values may not fit the decode kernel and take the token by token one
 
 
 def gated_linear(mode: int, q, k, v, z, c0, c1, rb: RaggedBatch, heads: int, dk: int, dv: int, state, norm_w, eps: float, *,
-                 gate=None, per_head: bool = False, carry=None, h=None, plain: bool = False) -> torch.Tensor:
+                 gate=None, per_head: bool = False, carry=None, h=None, plain: bool = False, low_rank=None, q_scale: float = 1.0,
+                 tau: float = 1.0, out=None, out_scale: float = 1.0) -> torch.Tensor:
     """Matrix state with a decay per head and channel over a ragged batch, its head norm and output gate; [n, heads * dv].
     GATES_BONUS: decay exp(-exp(z + c0)), keys k, bonus c1 for the current token. GATES_LOWER: decay
-    c1 + (1 - c1) sigmoid(z + c0), key 1 - decay, silu(q). q, k, v, gate: column views of rows [n, ..]; z fp32.
-    norm_w [dv], or [heads * dv] with per_head. carry / h: see `token_shift` (portions only).
+    c1 + (1 - c1) sigmoid(z + c0), key 1 - decay, silu(q). GATES_ROOT: decay sigmoid(z + c0)^(1 / tau), keys k, q * q_scale.
+    q, k, v, gate: column views of rows [n, ..]; z fp32, or None with `low_rank` = (x [n, rank], w [heads * dk, rank]) in a decode
+    step: z = x w^T, formed in the kernel. norm_w [dv], or [heads * dv] with per_head. carry / h: see `token_shift` (portions
+    only). `out`: columns of wider rows; the result is scaled by out_scale.
     `plain`: the token by token kernel of the 32-bit path, also for bf16."""
     n = q.shape[0]
-    assert z.dtype == torch.float32 and all(t is None or t.stride(1) == 1 for t in (q, k, v, z, gate))
+    x, w2 = low_rank if z is None else (None, None)
+    assert (z is None or z.dtype == torch.float32) and all(t is None or t.stride(1) == 1 for t in (q, k, v, z, x, gate, out))
     one = rb.decode and not plain
-    raw = torch.empty((n, heads * dv), dtype=torch.float32, device=q.device) if not one or dv > 256 else None
-    out = torch.empty((n, heads * dv), dtype=q.dtype, device=q.device)
+    raw = torch.empty((n, heads * dv), dtype=torch.float32, device=q.device) if not one or dv > STEP_WIDTH else None
+    if out is None:
+        out = torch.empty((n, heads * dv), dtype=q.dtype, device=q.device)
     ld = lambda t: 0 if t is None else t.stride(0)  # noqa: E731
     if rb.decode:
         carry = h = None                        # the launch that made the mixes has replaced it
     rc = _lib.cuda().tb_gated_linear(_dt(q), mode, q.data_ptr(), ld(q), _lib.ptr(k), ld(k), v.data_ptr(), ld(v), _lib.ptr(gate),
-                                     ld(gate), z.data_ptr(), ld(z), c0.data_ptr(), c1.data_ptr(), *rb.args(), heads, dk, dv,
+                                     ld(gate), _lib.ptr(z), ld(z), _lib.ptr(x), ld(x), _lib.ptr(w2), 0 if x is None else x.shape[1],
+                                     c0.data_ptr(), _lib.ptr(c1), float(q_scale), 1.0 / tau, *rb.args(), heads, dk, dv,
                                      state.data_ptr(), _lib.ptr(h), _lib.ptr(carry), 0 if h is None else h.shape[1],
-                                     norm_w.data_ptr(), int(per_head), float(eps), _lib.ptr(raw), out.data_ptr(), int(one),
-                                     int(not plain), _lib.stream_ptr())
+                                     norm_w.data_ptr(), int(per_head), float(eps), float(out_scale), _lib.ptr(raw), out.data_ptr(),
+                                     out.stride(0), int(one), int(not plain), _lib.stream_ptr())
     _lib.check(rc, "tb_gated_linear")
     _count()
     return out
@@ -222,29 +235,83 @@ def qk_norm_write(proj, q_off: int, k_off: int, v_off: int, q_w, k_w, eps: float
 
 
 def rope_norm_write(proj, q_off: int, k_off: int, v_off: int, cos, sin, rot_dims: int, eps: float, rb: RaggedBatch, table,
-                    page_size: int, heads: int, kv_heads: int, dim: int, vdim: int, k_pool, v_pool) -> torch.Tensor:
-    """Rotation of the first rot_dims dimensions of every query and key head (cos / sin fp32 [positions, rot_dims / 2]), then
-    each head divided by its root mean square; q [n, heads * dim] is returned, k and v rows go to their pages. kv_heads 0: the
-    rows hold queries only and nothing is written."""
+                    page_size: int, heads: int, kv_heads: int, dim: int, vdim: int, k_pool, v_pool, *, q_w=None, k_w=None,
+                    interleaved: bool = False, stored: Optional[tuple] = None) -> torch.Tensor:
+    """Every query and key head divided by its root mean square (times q_w / k_w [dim]) and its first rot_dims dimensions turned
+    (cos / sin fp32 [positions, rot_dims / 2]; halves of them together, or neighbours if `interleaved`); q is returned, k and v
+    rows go to their pages. `stored`: widths the key / value heads are kept at, with zeros behind them (queries like keys; default:
+    as they are). kv_heads 0: the rows hold queries only and nothing is written."""
     n = proj.shape[0]
-    q = torch.empty((n, heads * dim), dtype=proj.dtype, device=proj.device)
-    rc = _lib.cuda().tb_rope_norm_write(_dt(proj), proj.data_ptr(), proj.stride(0), q_off, k_off, v_off, _lib.ptr(cos),
-                                        _lib.ptr(sin), rot_dims, float(eps), *rb.args(), table.data_ptr(), table.shape[1],
-                                        page_size, heads, kv_heads, dim, vdim, q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(),
-                                        _lib.stream_ptr())
+    wq, wv = stored or (dim, vdim)
+    q = torch.empty((n, heads * wq), dtype=proj.dtype, device=proj.device)
+    rc = _lib.cuda().tb_rope_norm_write(_dt(proj), proj.data_ptr(), proj.stride(0), q_off, k_off, v_off, _lib.ptr(q_w), _lib.ptr(k_w),
+                                        _lib.ptr(cos), _lib.ptr(sin), rot_dims, int(interleaved), float(eps), *rb.args(),
+                                        table.data_ptr(), table.shape[1], page_size, heads, kv_heads, dim, vdim, wq, wv, q.data_ptr(),
+                                        k_pool.data_ptr(), v_pool.data_ptr(), _lib.stream_ptr())
     _lib.check(rc, "tb_rope_norm_write")
     _count()
     return q
 
 
-def window_attn(q, k_pool, v_pool, rb: RaggedBatch, table, page_size: int, sp, bias) -> torch.Tensor:
-    """`sp`: an attention spec of models.mixers; bias fp32 [heads, far + 1] or None. Returns [n, heads * vdim]."""
+def window_attn(q, k_pool, v_pool, rb: RaggedBatch, table, page_size: int, sp, bias, out=None, out_scale: float = 1.0) -> torch.Tensor:
+    """`sp`: an attention spec of models.mixers; bias fp32 [heads, far + 1] or None. Returns out_scale * [n, heads * vdim]; `out`:
+    columns of wider rows."""
     n = q.shape[0]
-    out = torch.empty((n, sp.heads * sp.vdim), dtype=q.dtype, device=q.device)
+    wq, wv = sp.stored(q.dtype)
+    if out is None:
+        out = torch.empty((n, sp.heads * sp.vdim), dtype=q.dtype, device=q.device)
     rc = _lib.cuda().tb_window_attn(_dt(q), q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(), *rb.args(), table.data_ptr(),
-                                    table.shape[1], page_size, sp.heads, sp.kv_heads, sp.dim, sp.vdim, float(sp.scale),
+                                    table.shape[1], page_size, sp.heads, sp.kv_heads, sp.dim, sp.vdim, wq, wv, float(sp.scale),
                                     float(sp.softcap), _lib.ptr(bias), 0 if bias is None else bias.shape[1] - 1, sp.window,
-                                    sp.chunk, sp.keep_first, out.data_ptr(), _lib.stream_ptr())
+                                    sp.chunk, sp.keep_first, float(sp.sink), float(out_scale), out.data_ptr(), out.stride(0),
+                                    _lib.stream_ptr())
     _lib.check(rc, "tb_window_attn")
     _count()
+    return out
+
+
+# ------------------------------------------------------------------------------------------------ experts
+ROWS_TOKENS = 128       # up to this many tokens an expert's weights are streamed past its few rows
+
+
+def moe(h, logits, correction, gate_up, down, top: int, rb: RaggedBatch) -> torch.Tensor:
+    """sum_j s_j expert_j(h) over the `top` experts with the largest score (+ correction [E] for the choice only); s: softmax of
+    the fp32 router logits over all experts, not renormalised. gate_up [E, 2 F, D] (gate rows, then up rows), down [E, D, F];
+    expert: down(silu(gate h) * up h). Returns [n, D] in h's type."""
+    n, D = h.shape
+    E, F2, _ = gate_up.shape
+    F, dev = F2 // 2, h.device
+    assert logits.dtype == torch.float32 and logits.shape == (n, E) and logits.is_contiguous() and h.stride(1) == 1
+    assert gate_up.is_contiguous() and down.is_contiguous() and down.shape == (E, D, F)
+    idx = torch.empty((n, top), dtype=torch.int32, device=dev)
+    wts = torch.empty((n, top), dtype=torch.float32, device=dev)
+    fits = h.dtype == torch.bfloat16 and D % 8 == 0 and F % 8 == 0 and h.stride(0) % 8 == 0 and h.data_ptr() % 16 == 0
+    if fits and n > ROWS_TOKENS:
+        hist = torch.empty((-(-n // 128), E), dtype=torch.int32, device=dev)
+        seg = torch.empty(E + 1, dtype=torch.int32, device=dev)
+        pos = torch.empty((n, top), dtype=torch.int32, device=dev)
+        rc = _lib.cuda().tb_moe_route(_dt(h), logits.data_ptr(), _lib.ptr(correction), *rb.args(), E, top, idx.data_ptr(), wts.data_ptr(),
+                                      hist.data_ptr(), seg.data_ptr(), pos.data_ptr(), _lib.stream_ptr())
+        _lib.check(rc, "tb_moe_route")
+        _count(3)
+        rows = (n * top + E * 127 + 127) // 128 * 128
+        xp = torch.empty((rows, D), dtype=h.dtype, device=dev)
+        K.moe_scatter_rows(h, pos, None, xp)
+        gu = torch.empty((rows, F2), dtype=h.dtype, device=dev)
+        K.gemm_grouped(xp, gate_up.view(E * F2, D), gu, F2, K.moe_tiles_rows(seg, rows, F2, D, F2))
+        y = K.gemm_grouped(K.glu_fwd(gu[:, :F], gu[:, F:], K.GLU_SILU), down.view(E * D, F), xp, D, K.moe_tiles_rows(seg, rows, D, F, D))
+        return K.moe_gather_sum(y, pos, wts)
+    off = torch.empty(E + 1, dtype=torch.int32, device=dev)
+    order = torch.empty(n * top, dtype=torch.int32, device=dev)
+    rc = _lib.cuda().tb_moe_route_lists(_dt(h), logits.data_ptr(), _lib.ptr(correction), *rb.args(), E, top, idx.data_ptr(),
+                                        wts.data_ptr(), off.data_ptr(), order.data_ptr(), _lib.stream_ptr())
+    _lib.check(rc, "tb_moe_route_lists")
+    act = torch.empty((n * top, F), dtype=h.dtype, device=dev)
+    y = torch.empty((n * top, D), dtype=torch.float32, device=dev)
+    out = torch.empty((n, D), dtype=h.dtype, device=dev)
+    rc = _lib.cuda().tb_moe_experts(_dt(h), int(fits), h.data_ptr(), h.stride(0), gate_up.data_ptr(), down.data_ptr(), n, D, F, E, top,
+                                    idx.data_ptr(), wts.data_ptr(), off.data_ptr(), order.data_ptr(), act.data_ptr(), y.data_ptr(),
+                                    out.data_ptr(), _lib.stream_ptr())
+    _lib.check(rc, "tb_moe_experts")
+    _count(4)
     return out
