@@ -256,7 +256,12 @@ def tovalix_weights(cfg, seed=0, rank=6):
     return w
 
 
+ROUTED = 4       # leading dimensions that only the embedding writes and the routers read
+
+
 def zikezen_weights(cfg, seed=0, rank=8):
+    """Routers read a few dimensions that no sublayer writes, and the embedding rows are drawn such that no choice between experts
+    is close: rounding then never sends a token to another expert. Which experts a token takes differs from layer to layer."""
     g = torch.Generator().manual_seed(seed)
     w = {}
 
@@ -274,8 +279,11 @@ def zikezen_weights(cfg, seed=0, rank=8):
     put("final.norm", D, mean=1.0)
     for i, layer in enumerate(cfg["layers"]):
         p, a, r, mlp = f"l{i}.", layer["mixer"]["left"], layer["mixer"]["right"], layer["mlp"]
-        for s in ("norm1", "norm1b") + (() if mlp is None else ("norm2", "norm2b")):
+        for s in ("norm1",) + (() if mlp is None else ("norm2",)):
             put(p + s, D, mean=1.0)
+        for s in ("norm1b",) + (() if mlp is None else ("norm2b",)):
+            put(p + s, D, mean=0.6)
+            w[p + s][:ROUTED] = 0
         H, G = a["heads"], a["kv_heads"]
         for s, rows in (("q", H * a["dim"]), ("k", G * a["dim"]), ("v", G * a["vdim"])):
             put(f"{p}mix.left.{s}", rows, D)
@@ -299,12 +307,27 @@ def zikezen_weights(cfg, seed=0, rank=8):
             for e in range(E):
                 for s, shape in (("gate", (F, D)), ("up", (F, D)), ("down", (D, F))):
                     put(f"{p}mlp.e{e}.{s}", *shape)
-            # scores spread enough that rounding rarely changes a choice
-            put(p + "mlp.router", E, D, std=3.0 * D ** -0.5)
-            put(p + "mlp.correction", E, std=0.3, mean=0.5)
+            put(p + "mlp.router", E, D, std=1.3)
+            w[p + "mlp.router"][:, ROUTED:] = 0
+            put(p + "mlp.correction", E, std=0.2, mean=0.5)
+            w[p + "norm2"][:ROUTED] = 1
         put(p + "side.gate", dim, D)
         put(p + "side.proj", D, dim)
         put(p + "side.norm", D, std=0.3)
+        w[p + "side.norm"][:ROUTED] = 0
+    w["pos"][:, :ROUTED] = 0
+    rows = (2 * torch.randn(60 * V, ROUTED, generator=g)).to(torch.bfloat16).float()
+    clear = torch.ones(len(rows), dtype=torch.bool)
+    for i, layer in enumerate(cfg["layers"]):
+        if layer["mlp"] is not None and layer["mlp"]["kind"] == "moe" and layer["mlp"]["router"]["top"] < layer["mlp"]["router"]["experts"]:
+            top = layer["mlp"]["router"]["top"]
+            for size in torch.linspace(0.15, 1.2, 22):              # whatever the norm makes of a row's size
+                s = torch.softmax(size * rows @ w[f"l{i}.mlp.router"][:, :ROUTED].T, -1) + w[f"l{i}.mlp.correction"]
+                s = s.sort(-1, descending=True).values
+                clear &= s[:, top - 1] - s[:, top] > 0.015
+    assert clear.sum() >= V, clear.sum()
+    w["embed"][:, :ROUTED] = rows[clear][:V] / cfg["embedding"]["scale"]
+    w["embed"] = w["embed"].to(torch.bfloat16).float()
     return w
 
 

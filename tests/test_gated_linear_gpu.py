@@ -1,15 +1,16 @@
 """Matrix memories with a decay per head and channel (csrc/linear_attention.cu) and what feeds them: token shift and output norm
-against tests/tovalix_oracle.py, in their three kernels (token by token, tensor-core blocks, decode step), with decays from
+against tests/tovalix_oracle.py and zikezen_oracle.py, in their three kernels (token by token, tensor-core blocks, decode step), with decays from
 none to total, keys that stand out far away, and slots that start over."""
 import pytest
 import torch
 
 from tests import tovalix_oracle as O
+from tests import zikezen_oracle as ZO
 from tests.test_stack_kernels_gpu import batch, rand, rel
 
 pytestmark = pytest.mark.gpu
 FORMS = [(torch.float32, False), (torch.bfloat16, True), (torch.bfloat16, False)]
-MODES = ["bonus", "lower"]
+MODES = ["bonus", "lower", "root"]
 # heads, key size, value size
 SIZES = [(2, 64, 64), (3, 16, 24), (1, 128, 128), (2, 104, 136), (2, 10, 6), (1, 40, 200), (2, 136, 16), (4, 8, 8)]
 
@@ -21,15 +22,19 @@ def d(t):
 class Memory:
     """One head group's parameters and a reference state per slot."""
 
-    def __init__(self, mode, H, dk, dv, dtype, slots=4, gated=True, per_head=True, strength=(-7.0, 1.5), seed=0):
+    def __init__(self, mode, H, dk, dv, dtype, slots=4, gated=True, per_head=True, strength=(-7.0, 1.5), seed=0, tau=1.5):
+        self.tau = tau
         self.mode, self.H, self.dk, self.dv, self.dtype, self.per_head = mode, H, dk, dv, dtype, per_head
         u = torch.rand(H * dk, generator=torch.Generator().manual_seed(seed))
         lo, hi = strength
-        if mode == "bonus":
+        if mode == "root":
+            self.c0, self.c1 = (-tau * (lo + (hi - lo) * u)).to(dtype).cuda(), None
+        elif mode == "bonus":
             self.c0, self.c1 = (lo + (hi - lo) * u).to(dtype).cuda(), rand(H * dk, dtype=dtype, seed=seed + 1)
         else:
             self.c0, self.c1 = (-(lo + (hi - lo) * u)).to(dtype).cuda(), (u.flip(0) * 0.98).to(dtype).cuda()
             self.c1[::3] = 0
+        self.keyed = mode != "lower"
         self.nw = rand(H * dv if per_head else dv, dtype=dtype, seed=seed + 2)
         self.gated = gated
         self.S = rand(slots, H, dk, dv, seed=seed + 3, std=5)          # left by earlier owners
@@ -46,11 +51,15 @@ class Memory:
     def run(self, x, rb, eps=1e-3, plain=False, **kw):
         from tunix_b200.ops import stack_kernels as SK
         q, k, v, g, z = x
-        mode = SK.GATES_BONUS if self.mode == "bonus" else SK.GATES_LOWER
-        return SK.gated_linear(mode, q, k if self.mode == "bonus" else None, v, z, self.c0, self.c1, rb, self.H, self.dk, self.dv, self.S,
+        mode = {"bonus": SK.GATES_BONUS, "lower": SK.GATES_LOWER, "root": SK.GATES_ROOT}[self.mode]
+        if self.mode == "root":
+            kw = dict(q_scale=0.3, tau=self.tau, **kw)
+        return SK.gated_linear(mode, q, k if self.keyed else None, v, z, self.c0, self.c1, rb, self.H, self.dk, self.dv, self.S,
                                self.nw, eps, gate=g if self.gated else None, per_head=self.per_head, plain=plain, **kw)
 
     def decays(self, z):
+        if self.mode == "root":
+            return ZO.decays(z + d(self.c0), self.tau).view(-1, self.H, self.dk)
         c0, c1 = d(self.c0), d(self.c1)
         f = torch.exp(-torch.exp(z + c0)) if self.mode == "bonus" else c1 + (1 - c1) * torch.sigmoid(z + c0)
         return f.view(-1, self.H, self.dk)
@@ -59,7 +68,9 @@ class Memory:
         q, k, v, g, z = (d(t[sl]) for t in x)
         H, dk, dv = self.H, self.dk, self.dv
         q, k, v, f = q.reshape(-1, H, dk), k.reshape(-1, H, dk), v.reshape(-1, H, dv), self.decays(z)
-        u, S, out = d(self.c1).view(H, dk, 1), self.ref[s], []
+        u, S, out = None if self.c1 is None else d(self.c1).view(H, dk, 1), self.ref[s], []
+        if self.mode == "root":
+            q = q * 0.3
         if self.mode == "lower":
             q, k = O.silu(q), 1 - f
         for t in range(q.shape[0]):
@@ -139,7 +150,8 @@ def test_total_decay_of_one_channel(channel, dtype, plain):
     """One token empties one channel in the middle of a block: the others go on, what follows is kept."""
     for mode in MODES:
         m = Memory(mode, 1, 72, 16, dtype, strength=(-6.0, -3.0), gated=False, per_head=False)
-        m.c1[:] = 0.0
+        if m.c1 is not None:
+            m.c1[:] = 0.0
         for t in (5, 7, 8, 15):
             m.ref[0].zero_()
             x = m.inputs(40, 500 + t)
@@ -157,10 +169,11 @@ def test_a_key_far_away(dtype, plain, cuts):
     n, far = sum(cuts), 1
     for mode in MODES:
         m = Memory(mode, 2, 32, 16, dtype, strength=(-14.0, -12.0), gated=False, per_head=False)
-        m.c1[:] = 0.0
+        if m.c1 is not None:
+            m.c1[:] = 0.0
         q, k, v, g, z = m.inputs(n, 600)
         z[:] = 0.0
-        if mode == "bonus":
+        if m.keyed:
             k *= 0.01
             k[far] = 30.0
         else:
@@ -222,3 +235,52 @@ def test_token_shift_of_single_tokens(D, groups, dtype):
     t = 1e-6 if dtype == torch.float32 else 1e-2
     assert got.shape == (5, 4, D) and rel(got[:, :3], h[:3] + (before - h[:3]) * d(mu)[:, None]) < t
     assert rel(carry[[5, 0, 2]], h[:3]) < t and torch.equal(carry[[1, 3, 4]], old[[1, 3, 4]])
+
+
+@pytest.mark.parametrize("dtype,plain", FORMS)
+@pytest.mark.parametrize("tau", [1.0, 16.0, 40.0])
+@pytest.mark.parametrize("cuts", [[900], [1] * 2 + [600] + [1] * 298])
+def test_roots_of_sigmoids_over_many_tokens(tau, cuts, dtype, plain):
+    """Decays from nearly one to small, as the root's degree sets them, over portions and hundreds of decoded tokens."""
+    m = Memory("root", 2, 40, 24, dtype, tau=tau, gated=False, per_head=False)
+    m.c0 = (torch.linspace(-9.0, 9.0, 80)).to(dtype).cuda()
+    x, at, got = m.inputs(sum(cuts), 700), 0, []
+    for c in cuts:
+        got.append(m.run(tuple(t[at:at + c] for t in x), batch([(3, at, c)]), plain=plain))
+        at += c
+    assert rel(torch.cat(got), m.reference(x, 3, slice(None))) < tol(dtype)
+    assert rel(m.S[3], m.ref[3]) < (2e-5 if dtype == torch.float32 else 1e-4)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("rank", [8, 16, 5, 72])
+def test_gates_from_a_bottleneck_in_a_decode_step(rank, dtype):
+    """The gates' product inside the step kernel against the same gates given to it."""
+    from tunix_b200.ops import stack_kernels as SK
+    for H, dk, dv in ((2, 64, 64), (3, 7, 9), (1, 40, 136)):
+        a, b = Memory("root", H, dk, dv, dtype, seed=3), Memory("root", H, dk, dv, dtype, seed=3)
+        rb = batch([(2, 5, 1), (0, 0, 1), (1, 64, 1)])
+        rb.pos0[2] = -1
+        q, k, v, g, _ = a.inputs(3, 800)
+        for lead in (8, 3):                                # columns of a wider row, with and without 16-byte alignment
+            x, w2 = rand(3, lead + rank, dtype=dtype, seed=9)[:, lead:], rand(H * dk, rank, dtype=dtype, seed=10, std=0.5)
+            z = (d(x) @ d(w2).T).float().cuda()
+            want = a.run((q, k, v, g, z), rb)
+            got = SK.gated_linear(SK.GATES_ROOT, q, k, v, None, b.c0, None, rb, H, dk, dv, b.S, b.nw, 1e-3, gate=g, per_head=True,
+                                  low_rank=(x, w2), q_scale=0.3, tau=b.tau)
+            assert rel(got[:2], want[:2]) < (1e-5 if dtype == torch.float32 else 5e-3) and rel(b.S[[0, 2]], a.S[[0, 2]]) < 1e-5
+            assert got[2].abs().max() == 0 and torch.equal(b.S[1], a.S[1])
+
+
+@pytest.mark.parametrize("dtype,plain", FORMS)
+@pytest.mark.parametrize("H,dk,dv", [(2, 16, 24), (1, 16, 136), (3, 10, 6), (2, 64, 64)])
+def test_output_into_columns_of_a_row(H, dk, dv, dtype, plain):
+    for lead, factor in ((8, 0.5), (3, 1.75), (16, -2.0)):
+        for n in (70, 1):
+            a, b = (Memory("root", H, dk, dv, dtype, seed=5) for _ in range(2))
+            x, rb = a.inputs(n, 900), batch([(1, 0, n)])
+            want = a.run(x, rb, plain=plain)
+            rows = torch.full((n, lead + H * dv + 5), 7.0, dtype=dtype, device="cuda")
+            out = b.run(x, rb, plain=plain, out=rows[:, lead:lead + H * dv], out_scale=factor)
+            assert rel(out, want.double() * factor) < (1e-6 if dtype == torch.float32 else 5e-3)
+            assert rows[:, :lead].eq(7).all() and rows[:, lead + H * dv:].eq(7).all()

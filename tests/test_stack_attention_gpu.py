@@ -7,6 +7,7 @@ import torch
 
 from tests import roluzen_oracle as O
 from tests import tovalix_oracle as TO
+from tests import zikezen_oracle as ZO
 from tests.test_stack_kernels_gpu import batch, rand, rel
 
 pytestmark = pytest.mark.gpu
@@ -56,18 +57,19 @@ class Cache:
         self.page = page
 
 
-def run(kind, cache, rb, q, sp, bias, split=0):
+def run(kind, cache, rb, q, sp, bias, split=0, **kw):
     from tunix_b200.ops import kernels as K
     from tunix_b200.ops import stack_kernels as SK
     n = q.shape[0]
     if kind == "general":
-        return SK.window_attn(q.reshape(n, -1), cache.k, cache.v, rb, cache.table, cache.page, sp, bias).view(n, sp.heads, sp.vdim)
-    kw = dict(scale=sp.scale, softcap=sp.softcap, window=sp.window, chunk=sp.chunk, keep_first=sp.keep_first, bias=bias)
+        return SK.window_attn(q.reshape(n, -1), cache.k, cache.v, rb, cache.table, cache.page, sp, bias, **kw).view(n, sp.heads, sp.vdim)
+    kw = dict(scale=sp.scale, softcap=sp.softcap, window=sp.window, chunk=sp.chunk, keep_first=sp.keep_first, sink=sp.sink, bias=bias,
+              value_dim=sp.vdim, **kw)
     if kind == "decode":
         return K.paged_decode(q, cache.k, cache.v, cache.table, rb.slot, rb.pos0 + 1, num_kv_heads=sp.kv_heads, page_size=cache.page,
-                              max_ctx=cache.table.shape[1] * cache.page, split_tokens=split, **kw)
+                              max_ctx=cache.table.shape[1] * cache.page, split_tokens=split, **kw).view(n, sp.heads, sp.vdim)
     return K.attn_fwd_paged(q.reshape(n, -1).contiguous(), cache.k, cache.v, rb, cache.table, cache.page, num_heads=sp.heads,
-                            num_kv_heads=sp.kv_heads, head_dim=sp.dim, **kw).view(n, sp.heads, sp.vdim)
+                            num_kv_heads=sp.kv_heads, head_dim=sp.stored(q.dtype)[0], **kw).view(n, sp.heads, sp.vdim)
 
 
 def spec(H, G, dq, dv, window, keep, scale=0.2):
@@ -318,3 +320,180 @@ def test_rotation_norm_and_page_write(H, G, dq, dv, rot, dtype):
     alone = proj[:, off:off + NQ].contiguous()
     before = kp.clone()
     assert torch.equal(SK.rope_norm_write(alone, 0, NQ, NQ, *args, H, 0, dq, dv, kp, vp), q) and torch.equal(kp, before)
+
+
+# ------------------------------------------------------------------------------------------------ windows with a sink, wider stored heads
+def sinking(H, G, dq, dv, window, scale=0.2, sink=0.0, rot=0, fit=True, **kw):
+    from tunix_b200.models.mixers import RotaryAttentionSpec
+    return RotaryAttentionSpec(heads=H, kv_heads=G, dim=dq, vdim=dv, scale=scale, rot_dims=rot, rot_base=100.0, window=window, sink=sink,
+                               fit_heads=fit, **kw)
+
+
+class Widened(Cache):
+    """The cache of a spec whose heads may be stored wider than they are, zeros behind them."""
+
+    def __init__(self, lens, sp, dtype, **kw):
+        wk, wv = sp.stored(dtype)
+        G = sp.kv_heads
+        super().__init__(lens, G, wk, wv, dtype, **kw)
+        for t, width, w in ((self.k, sp.dim, wk), (self.v, sp.vdim, wv)):
+            t.view(*t.shape[:2], G, w)[..., width:] = 0
+        seqs = []
+        for k, v in self.seqs:
+            k, v = k[..., :sp.dim].clone(), v[..., :sp.vdim].clone()
+            if kw.get("unit"):
+                k = (k / k.float().norm(dim=-1, keepdim=True)).to(dtype)
+            seqs.append((k, v))
+        if kw.get("unit"):                                 # cut to the heads' size and scaled again
+            for s, (k, _) in enumerate(seqs):
+                own = self.table[s].tolist()
+                for j in range(k.shape[0]):
+                    self.k[own[j // self.page], j % self.page].view(G, wk)[:, :sp.dim] = k[j]
+        self.seqs = seqs
+
+
+def widen(q, sp):
+    return torch.nn.functional.pad(q, (0, sp.stored(q.dtype)[0] - sp.dim)).contiguous()
+
+
+def dense_sink(q, k, v, i0, sp):
+    """The oracle's attention of the last rows of a sequence."""
+    q, k, v = (t.double().cpu() for t in (q, k, v))
+    T, P = q.shape[0], k.shape[0]
+    pad = torch.zeros(P, *q.shape[1:], dtype=torch.float64)
+    pad[i0:i0 + T] = q
+    m = {"heads": sp.heads, "kv_heads": sp.kv_heads, "vdim": sp.vdim, "scale": sp.scale, "mask": {"size": sp.window or 10 ** 9}}
+    return ZO.attend(pad, k, v, m)[i0:i0 + T].view(T, sp.heads, sp.vdim)
+
+
+SINK_GENERAL = [("general", torch.float32, 4, 2, 12, 20), ("general", torch.bfloat16, 3, 1, 17, 9), ("general", torch.bfloat16, 4, 2, 40, 56)]
+SINK_FLASH = [("flash", torch.bfloat16, 4, 2, 64, 48), ("flash", torch.bfloat16, 3, 1, 72, 128), ("flash", torch.bfloat16, 2, 2, 256, 256),
+              ("flash", torch.bfloat16, 6, 3, 40, 64)]
+SINK_DECODE = [("decode", torch.bfloat16, 6, 2, 64, 48), ("decode", torch.bfloat16, 16, 1, 128, 128), ("decode", torch.bfloat16, 3, 3, 96, 200)]
+WINDOWS = [20, 64, 65, 63, 200, 0, 1, 129]
+
+
+@pytest.mark.parametrize("window", WINDOWS)
+@pytest.mark.parametrize("kind,dtype,H,G,dq,dv", SINK_GENERAL + SINK_FLASH)
+def test_sink_in_portions(kind, dtype, H, G, dq, dv, window):
+    """Weights that the sink takes a large part of, heads stored wider, the result in columns of a wider row and scaled."""
+    sp = sinking(H, G, dq, dv, window)
+    cache = Widened([300, 64, 130, 7], sp, dtype, seed=31)
+    parts = [(0, 120, 180), (1, 0, 64), (2, 128, 2), (3, 0, 7), (0, 69, 131)]
+    n = sum(p[2] for p in parts)
+    q = rand(n, H, dq, dtype=dtype, std=0.5)
+    rows = torch.full((n, 8 + H * dv + 8 + (-H * dv) % 8), 9.0, dtype=dtype, device="cuda")
+    out, at = run(kind, cache, batch(parts), widen(q, sp), sp, None, out=rows[:, 8:8 + H * dv], out_scale=0.5), 0
+    assert rows[:, :8].eq(9).all() and rows[:, 8 + H * dv:].eq(9).all()
+    for s, p, m in parts:
+        k, v = cache.seqs[s]
+        assert rel(out[at:at + m], 0.5 * dense_sink(q[at:at + m], k[:p + m], v[:p + m], p, sp)) < tol(dtype), s
+        at += m
+
+
+@pytest.mark.parametrize("window", WINDOWS)
+@pytest.mark.parametrize("kind,dtype,H,G,dq,dv", SINK_GENERAL[:2] + SINK_DECODE)
+def test_sink_in_single_tokens(kind, dtype, H, G, dq, dv, window):
+    sp = sinking(H, G, dq, dv, window)
+    lens = [1, 20, 21, 63, 64, 65, 66, 129, 140, 200, 201, 300]
+    cache = Widened(lens, sp, dtype, seed=32)
+    rb = batch([(s, n - 1, 1) for s, n in enumerate(lens)] + [(len(lens), 0, 1)])
+    rb.pos0[-1] = -1                                                    # idle
+    n = len(lens) + 1
+    q = rand(n, H, dq, dtype=dtype, std=0.5)
+    want = [-3.0 * dense_sink(q[s:s + 1], k, v, lens[s] - 1, sp) for s, (k, v) in enumerate(cache.seqs)]
+    for split in (0, 64, 128, 512):
+        rows = torch.full((n, 3 + H * dv + 2), 9.0, dtype=dtype, device="cuda")
+        out = run(kind, cache, rb, widen(q, sp), sp, None, split, out=rows[:, 3:3 + H * dv], out_scale=-3.0)
+        assert rows[:, :3].eq(9).all() and rows[:, 3 + H * dv:].eq(9).all()
+        for s, w in enumerate(want):
+            assert rel(out[s:s + 1], w) < tol(dtype), (s, split)
+        assert out[-1].abs().max() == 0
+        if kind == "general":
+            break
+
+
+@pytest.mark.parametrize("score", [-60.0, -8.0, 0.0, 12.0, 60.0])
+@pytest.mark.parametrize("kind,dtype,H,G,dq,dv", SINK_GENERAL[:2] + SINK_FLASH[:2] + SINK_DECODE[:2])
+def test_sink_against_scores_of_every_size(kind, dtype, H, G, dq, dv, score):
+    """All keys score the same: the sink takes everything, its exact share, or nothing."""
+    window, n = 40, 100
+    sp = sinking(H, G, dq, dv, window, scale=1.0)
+    cache = Widened([n], sp, dtype, seed=33)
+    wk, _ = sp.stored(dtype)
+    cache.k.view(*cache.k.shape[:2], G, wk)[..., 0] = 1.0
+    q = torch.zeros(1, H, dq, dtype=dtype, device="cuda")
+    q[..., 0] = score
+    out = run(kind, cache, batch([(0, n - 1, 1)]), widen(q, sp), sp, None)[0].double().cpu()
+    v = cache.seqs[0][1].double().cpu()[n - window:]
+    share = 1 / (math.exp(-score) + window)                             # e^s / (1 + window e^s)
+    want = torch.stack([v[:, h // (H // G)].sum(0) * share for h in range(H)])
+    if score == -60.0:
+        assert out.abs().max() < 1e-20
+    else:
+        assert rel(out, want) < tol(dtype)
+
+
+@pytest.mark.parametrize("window", [20, 64, 70, 129, 128])
+@pytest.mark.parametrize("kind,dtype,H,G,dq,dv,decoded", [(*c, d) for d, cs in ((False, SINK_GENERAL + SINK_FLASH), (True, SINK_GENERAL[:2] + SINK_DECODE))
+                                                          for c in cs])
+def test_one_key_at_a_window_edge_beside_the_sink(kind, dtype, H, G, dq, dv, window, decoded):
+    """Every query asks for one key: seen, the output is its value; just outside, it must be something else, also when nothing
+    else scores above the sink."""
+    sp = sinking(H, G, dq, dv, window, scale=0.3)
+    cache = Widened([330], sp, dtype, seed=34, unit=True)
+    k, v = cache.seqs[0]
+    pairs = sorted({(i, j) for i in (63, 64, 127, 128, 191, 200, 255, 256, 320, 329)
+                    for j in (i, i - 1, i - window + 1, i - window, 0, 63, 64, 127, 128) if 0 <= j <= i})
+    ask = lambda ps, js: widen(outstanding(cache, 0, ps, js, H, dq), sp)  # noqa: E731
+    if decoded:
+        got = torch.cat([run(kind, cache, batch([(0, i, 1)]), ask([i], [j]), sp, None) for i, j in pairs])
+    else:
+        rows = []
+        for i, j in pairs:
+            lo = max(0, i - 2)
+            rows.append(run(kind, cache, batch([(0, lo, i + 1 - lo)]), ask(range(lo, i + 1), [*range(lo, i), j]), sp, None)[-1:])
+        got = torch.cat(rows)
+    for (i, j), o in zip(pairs, got):
+        val = torch.stack([v[j, h // (H // G)] for h in range(H)]).double().cpu()
+        err = ((o.double().cpu() - val).norm() / val.norm()).item()
+        assert err < 0.05 if ZO.visible(i, j, window) else err > 0.3, (i, j, err)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("H,G,dq,dv,rot", [(4, 2, 16, 24, 16), (3, 1, 10, 6, 6), (8, 4, 64, 64, 64), (2, 2, 72, 128, 8), (5, 1, 24, 8, 0),
+                                           (6, 2, 40, 48, 24), (4, 2, 256, 128, 128), (2, 1, 96, 200, 2), (1, 1, 300, 20, 200)])
+def test_weighted_norm_interleaved_rotation_and_wider_pages(H, G, dq, dv, rot, dtype):
+    """Norm with weights before the rotation of neighbours, scaled frequencies; what lies behind a head is zero."""
+    from tunix_b200.models.stack_exec import rope_table
+    from tunix_b200.ops import stack_kernels as SK
+    sp = sinking(H, G, dq, dv, 0, rot=rot)
+    wk, wv = sp.stored(dtype)
+    NQ, NK, NV, eps = H * dq, G * dq, G * dv, 1e-2
+    rb = batch([(1, 62, 4), (0, 0, 3), (2, 5, 1), (3, 700, 1)])
+    rb.pos0[2] = -1
+    off, n = 8, 9
+    proj = rand(n, off + NQ + NK + NV, dtype=dtype, std=0.3)
+    qw, kw = rand(dq, dtype=dtype, seed=1), rand(dq, dtype=dtype, seed=2)
+    table = torch.full((4, 12), -1, dtype=torch.int32)
+    table[0, 0], table[1, 0], table[1, 1], table[3, 10] = 4, 2, 0, 1
+    kp, vp = torch.full((5, 64, G * wk), 3.0, device="cuda", dtype=dtype), torch.full((5, 64, G * wv), 3.0, device="cuda", dtype=dtype)
+    scaling = {"factor": 6.0, "low": 1.0, "high": 4.0, "original": 400}
+    cos, sin = rope_table(768, rot, 100.0, "cuda", tuple(scaling.values()))
+    q = SK.rope_norm_write(proj, off, off + NQ, off + NQ + NK, cos, sin, rot, eps, rb, table.cuda(), 64, H, G, dq, dv, kp, vp, q_w=qw,
+                           k_w=kw, interleaved=True, stored=(wk, wv))
+    pos = torch.tensor([62, 63, 64, 65, 0, 1, 2, 5, 700])
+    p, rt = proj.double().cpu(), {"dims": rot, "base": 100.0, "scaling": scaling}
+
+    def turn(x, heads, w):
+        x = ZO.rotate(ZO.rms(x.reshape(n, heads, dq), eps) * w.double().cpu(), pos, rt)
+        return torch.nn.functional.pad(x, (0, wk - dq)).reshape(n, -1)
+    wantq, wantk = turn(p[:, off:off + NQ], H, qw), turn(p[:, off + NQ:off + NQ + NK], G, kw)
+    wantv = torch.nn.functional.pad(p[:, off + NQ + NK:].reshape(n, G, dv), (0, wv - dv)).reshape(n, -1)
+    t, live = 2e-6 if dtype == torch.float32 else 5e-3, [0, 1, 2, 3, 4, 5, 6, 8]
+    assert rel(q[live], wantq[live]) < t and q[7].abs().max() == 0
+    assert q[live].view(8, H, wk)[..., dq:].abs().sum() == 0
+    for row, (pg, o) in zip(live, [(2, 62), (2, 63), (0, 0), (0, 1), (4, 0), (4, 1), (4, 2), (1, 60)]):
+        assert rel(kp[pg, o], wantk[row]) < t and torch.equal(vp[pg, o].double().cpu(), wantv[row])
+        assert kp[pg, o].view(G, wk)[:, dq:].abs().sum() == 0
+    assert (kp != 3).any(-1).sum() == 8 and (vp != 3).any(-1).sum() == 8

@@ -266,3 +266,149 @@ def test_trace_runner_help_names_its_options():
 def test_configs_are_json():
     for cfg in C.CASES.values():
         assert json.loads(json.dumps(cfg)) == cfg
+
+
+# ------------------------------------------------------------------------------------------------ Zikezen
+def test_zikezen_constants_come_from_config_json(tmp_path):
+    from tunix_b200.models.hf_config import config_from_hf
+    cfg = C.CASES["looped"]
+    src = C.write(tmp_path / "m", cfg, C.zikezen_weights(cfg, rank=7))
+    c = config_from_hf(src)
+    assert (c.family, c.embed_factor, c.positions, c.max_position, c.final_logit_softcap, c.token_side) == ("zikezen", 1.7, 512, 512, 12.0, 8)
+    assert c.post_norms and c.loop_embed and c.loop == (0, 3, 3) and c.streams == 0 and not c.is_moe
+    m = c.layer_specs[1].mixer
+    assert (m.left_scale, m.right_scale, m.right.tau, m.right.decay_rank) == (1.1, 0.4, 12.0, 7)
+    a = m.left
+    assert (a.heads, a.kv_heads, a.window, a.scale, a.rot_dims, a.rot_base, a.rot_scaling) == (2, 2, 7, 0.4, 8, 700.0, (5.0, 1.0, 3.5, 60.0))
+    assert a.interleaved and a.head_weights and a.sink == 0.0 and not a.out_bias and a.softcap == 0.0 and a.chunk == 0
+    assert [(s.ff, s.ff_kind, s.experts, s.top) for s in c.layer_specs] == [(40, "experts", 6, 2), (None, "glu", 0, 0), (56, "experts", 5, 5),
+                                                                            (72, "glu", 0, 0)]
+    assert c.runs() == [0, 1, 2] * 3 + [3] and c.restarts() == {3, 6}
+    assert config_from_hf(C.CASES["ragged"]).restarts() == {2} and config_from_hf(C.CASES["ragged"]).layer_specs[0].mixer.left.rot_scaling is None
+    plain = config_from_hf(dict(cfg, loop=None, logit_softcap=None))
+    assert plain.restarts() == set() and plain.final_logit_softcap == 0.0
+    with pytest.raises(ValueError, match="mixer"):
+        config_from_hf(dict(cfg, layers=[C.hgrn2()]))
+    with pytest.raises(ValueError, match="feed-forward"):               # only designs that have experts take them
+        config_from_hf(dict(C.CASES["shared"], layers=[dict(C.wkv(), mlp=cfg["layers"][0]["mlp"])]))
+    with pytest.raises(ValueError, match="experts"):
+        config_from_hf(dict(cfg, loop=None, layers=[C.beside(experts=(3, 4))]))
+
+
+def test_stored_heads_and_cache_rows():
+    from tunix_b200.models.hf_config import config_from_hf
+    c = config_from_hf(C.CASES["blocks"])
+    specs = [s.mixer.left for s in c.layer_specs]
+    assert [a.stored(torch.bfloat16) for a in specs] == [(64, 64), (128, 128), (128, 128)]
+    assert [a.stored(torch.float32) for a in specs] == [(40, 56), (96, 80), (128, 128)]
+    assert c.kv_rows() == [(192, 192), (128, 128), (256, 256), (128, 128), (256, 256)]
+    assert c.kv_rows(torch.float32)[:2] == [(120, 168), (96, 80)]
+    assert config_from_hf(C.CASES["ragged"]).kv_rows() == [(10, 6), (18, 42), (18, 42), (32, 48)]
+    assert c.state_shapes()[0] == {"S": (2, 40, 72)} and len(c.state_shapes()) == 5
+
+
+def test_zikezen_presets_and_parameters():
+    from tunix_b200.models import naming, registry
+    from tunix_b200.models.config import get_config
+    from tunix_b200.models.transformer import create_model
+    assert registry.get_family("zikezen").family == "zikezen" and registry.family_of_hf_id("x/Zikezen-2B").family == "zikezen"
+    assert naming.config_for("zikezen-8b") == get_config("zikezen_8b") and naming.get_model_family("x/Zikezen-2B") == "zikezen"
+    model = create_model(get_config("zikezen_tiny"), seed=3)
+    assert model.num_params == get_config("zikezen_tiny").num_params() and model.config.runs() == [0, 1, 2, 1, 2, 3]
+    assert model.layers[0].post_attn_norm.weight.eq(1).all() and model.layers[1].mlp.correction.eq(0).all()
+    assert model.layers[0].mixer.right.a2_proj.bias.eq(2).all() and model.layers[1].mlp.gate_proj.std() > 0.01
+    with pytest.raises(ValueError, match="position"):
+        model(torch.zeros(1, 513, dtype=torch.long))
+
+
+def test_missing_experts_are_named(tmp_path):
+    from safetensors.torch import load_file, save_file
+    from tunix_b200.models.automodel import AutoModel
+    cfg = C.CASES["looped"]
+    src = C.write(tmp_path / "m", cfg, C.weights(cfg))
+    t = load_file(src + "/model.safetensors")
+    del t["l0.mlp.e3.up"]
+    save_file(t, src + "/model.safetensors")
+    with pytest.raises(KeyError, match="up_proj#3"):
+        AutoModel.from_pretrained(src, model_source="local")
+
+
+def test_parameters_joined_side_by_side_follow_updates():
+    from tunix_b200.models.config import get_config
+    from tunix_b200.models.stack_exec import StackExecutor
+    from tunix_b200.models.transformer import create_model
+    model = create_model(get_config("zikezen_tiny"), seed=0)
+    ex = StackExecutor(model)
+    before = {(i, k): v.data_ptr() for i, d in enumerate(ex.w) for k, v in d.items() if v is not None}
+    mix, mlp = model.layers[1].mixer, model.layers[1].mlp
+    want = torch.cat([mix.left.o_proj.weight, mix.right.o_proj.weight], 1)
+    with torch.no_grad():
+        mix.right.o_proj.weight.mul_(2.0)
+        mlp.up_proj[3].fill_(0.5)
+        mix.left.v_proj.bias.fill_(3.0)
+    ex.refresh()
+    assert {(i, k): v.data_ptr() for i, d in enumerate(ex.w) for k, v in d.items() if v is not None} == before
+    n = mix.left.o_proj.weight.shape[1]
+    assert torch.equal(ex.w[1]["o"][:, :n], want[:, :n]) and torch.equal(ex.w[1]["o"][:, n:], 2 * want[:, n:])
+    gu, F = ex.w[1]["experts_gu"], mlp.gate_proj.shape[1]
+    assert gu.is_contiguous() and torch.equal(gu[:, :F], mlp.gate_proj) and gu[3, F:].eq(0.5).all() and "experts_gu" not in ex.w[0]
+    a = mix.spec.left
+    q, kv = a.heads * a.dim, a.kv_heads * (a.dim + a.vdim)
+    b = ex.w[1]["proj_bias"]
+    assert b[q + a.kv_heads * a.dim:q + kv].eq(3).all() and b[q + kv:].eq(0).all() and b.numel() == ex.w[1]["proj"].shape[0]
+    assert set(ex.pack_sources()[1]) == {"proj", "o"} and "down" in ex.pack_sources()[0]
+
+
+@pytest.mark.parametrize("scaling", [None, (5.0, 1.0, 3.5, 60.0), (8.0, 1.0, 4.0, 8192.0), (3.0, 2.0, 2.0, 500.0), (1.0, 1.0, 4.0, 100.0)])
+def test_rope_frequencies(scaling):
+    from tunix_b200.models.stack_exec import rope_frequencies
+    for dims, base in ((32, 5e5), (8, 700.0), (2, 40.0), (0, 1.0)):
+        rot = {"dims": dims, "base": base}
+        if scaling:
+            rot["scaling"] = dict(zip(("factor", "low", "high", "original"), scaling))
+            rot["scaling"]["high"] += 1e-9 * (scaling[1] == scaling[2])        # the oracle divides by the band's width
+        assert torch.allclose(rope_frequencies(dims, base, scaling), ZO.frequencies(rot), rtol=1e-6)
+
+
+def test_zikezen_oracle_details():
+    s = torch.tensor([0.0, math.log(2.0), -math.inf]).double()
+    assert torch.allclose(ZO.sink_softmax(s), torch.tensor([0.25, 0.5, 0.0]).double())
+    assert torch.allclose(ZO.sink_softmax(s + 300), torch.tensor([1 / 3, 2 / 3, 0.0]).double()) and ZO.sink_softmax(s - 300).sum() < 1e-100
+    x = torch.tensor([[[1.0, 0.0, 0.0, 2.0, 5.0]]]).double()
+    got = ZO.rotate(x, torch.tensor([3]), {"dims": 4, "base": 100.0})[0, 0]
+    a, b = 3.0, 0.3
+    assert torch.allclose(got, torch.tensor([math.cos(a), math.sin(a), -2 * math.sin(b), 2 * math.cos(b), 5.0]).double())
+    f = ZO.frequencies({"dims": 6, "base": 1000.0, "scaling": {"factor": 4.0, "low": 1.0, "high": 4.0, "original": 100}})
+    turns = [100 / (2 * math.pi) * 1000.0 ** (-i / 3) for i in range(3)]                 # 15.9, 1.59, 0.159
+    mid = (turns[1] - 1) / 3
+    assert torch.allclose(f, torch.tensor([1.0, 0.1 * (mid + (1 - mid) / 4), 0.01 / 4]).double())
+    r = ZO.route(torch.tensor([[0.0, 1.0, 2.0]]).double(), torch.eye(3).double(), torch.tensor([0.9, 0.0, 0.0]).double(), 2)
+    p = torch.softmax(torch.tensor([0.0, 1.0, 2.0]).double(), 0)
+    assert torch.allclose(r[0], torch.stack([p[0], p[1] * 0, p[2]]))
+    assert torch.allclose(ZO.decays(torch.tensor([0.0, -800.0]).double(), 4.0), torch.tensor([0.5 ** 0.25, math.exp(-200)]).double())
+    assert ZO.visible(19, 0, 20) and not ZO.visible(20, 0, 20) and not ZO.visible(3, 4, 20)
+    assert ZO.layer_runs({"layers": [0] * 4, "loop": {"start": 1, "stop": 3, "times": 2}}) == \
+        [(0, False), (1, False), (2, False), (1, True), (2, False), (3, False)]
+
+
+def test_zikezen_memory_against_its_unrolled_sum():
+    torch.manual_seed(2)
+    T, H, d, dv = 12, 2, 4, 3
+    q, k, v, a = (torch.randn(T, H, n, dtype=torch.float64) for n in (d, d, dv, d))
+    a = torch.sigmoid(a)
+    got = ZO.gla_recurrence(q, k, v, a)
+    for t in range(T):
+        want = sum((q[t] * a[s + 1:t + 1].prod(0) * k[s]).sum(-1, keepdim=True) * v[s] for s in range(t + 1))
+        assert torch.allclose(got[t], want)
+
+
+def test_sequences_stay_within_the_learned_positions():
+    from tunix_b200.generate.engine import PagedEngine
+    from tunix_b200.models.hf_config import config_from_hf
+    eng = PagedEngine.__new__(PagedEngine)
+    eng.cfg = config_from_hf(C.CASES["looped"])
+    eng._check_length(512)
+    with pytest.raises(ValueError, match="positions"):
+        eng._check_length(513)
+    eng.cfg = config_from_hf(C.CASES["shared"])
+    eng._check_length(10 ** 6)

@@ -1,5 +1,5 @@
-"""Layer-stack models on the GPU against the plain oracles (tests/roluzen_oracle.py, tovalix_oracle.py): whole prompts, portions, mixed batches,
-decoding, slots and pages that are used again, greedy generation through the engine. Mechanism tests are in
+"""Layer-stack models on the GPU against the plain oracles (tests/roluzen_oracle.py, tovalix_oracle.py, zikezen_oracle.py): whole
+prompts, portions, mixed batches, decoding, slots and pages that are used again, greedy generation through the engine. Mechanism tests are in
 test_stack_kernels_gpu.py and test_gated_linear_gpu.py."""
 import functools
 
@@ -10,6 +10,7 @@ from tests import stack_cases as C
 
 pytestmark = pytest.mark.gpu
 TOL = {torch.float32: 1e-5, torch.bfloat16: 1.5e-2}       # relative rms error of the logits against the oracle, all rows
+NOISY = {"looped": 2.0}     # models whose longer chain of sublayers amplifies rounding: factor of the bf16 tolerance
 
 
 class Ids:
@@ -98,9 +99,12 @@ def test_whole_prompt_and_layers(name, dtype):
     assert len(sums) == len(model.config.runs())
     for s, ref in zip(sums, layers):
         assert close(s, ref, dtype)
-    assert close(ex.logits(h), want, dtype)
+    logits, cap = ex.logits(h), model.config.final_logit_softcap
+    if cap:
+        logits = cap * torch.tanh(logits / cap)
+    assert close(logits, want, dtype)
     z, _ = model(torch.tensor([toks]))
-    assert torch.allclose(z[0].float(), ex.logits(h), atol=1e-4 if dtype == torch.float32 else 0.15)
+    assert torch.allclose(z[0].float(), logits, atol=1e-4 if dtype == torch.float32 else 0.15)
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
@@ -122,7 +126,7 @@ def test_portions_and_decoding_agree_with_the_oracle(name, dtype):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("name", ["mixed", "wide", "shared", "tiles", "uneven"])
+@pytest.mark.parametrize("name", ["mixed", "wide", "shared", "tiles", "uneven", "looped", "ragged", "blocks"])
 def test_mixed_batches_and_reused_slots(name, dtype):
     """Unequal requests: portions beside decoded tokens, requests that sit out steps, ends in between; six requests share
     three slots and a pool that holds two of the longest, so that pages and slots change owners."""
@@ -157,7 +161,7 @@ def test_mixed_batches_and_reused_slots(name, dtype):
         assert close(torch.cat(got[i]), want, dtype), i
 
 
-@pytest.mark.parametrize("name", ["wide", "tiles"])
+@pytest.mark.parametrize("name", ["wide", "tiles", "blocks"])
 def test_a_batch_equals_each_request_alone_in_bf16(name):
     """bf16 results do not depend on the company beyond rounding: compared with the single request, not with the oracle."""
     cfg, _, model = case(name, torch.bfloat16)
@@ -175,7 +179,7 @@ def test_a_batch_equals_each_request_alone_in_bf16(name):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("name", ["mixed", "shared", "tiles"])
+@pytest.mark.parametrize("name", ["mixed", "shared", "tiles", "looped", "blocks"])
 def test_long_decoding(name, dtype):
     """Several hundred decoded tokens: states, rings, windows and chunks that have turned over many times."""
     cfg, _, model = case(name, dtype)
@@ -215,7 +219,7 @@ def greedy_reference(name, prompt, steps):
 
 
 @pytest.mark.parametrize("graph", [True, False])
-@pytest.mark.parametrize("name", ["mixed", "shared", "uneven"])
+@pytest.mark.parametrize("name", ["mixed", "shared", "uneven", "looped", "ragged"])
 def test_greedy_generation_matches_the_oracle(name, graph):
     """Through the engine's entry point and scheduler in 32-bit: four prompts over two slots and a pool that forces
     pre-emption, decode step captured in a graph or not; logits of the oracle decide."""
@@ -234,7 +238,7 @@ def test_greedy_generation_matches_the_oracle(name, graph):
             assert lp <= 0.0
 
 
-@pytest.mark.parametrize("name", ["wide", "tiles"])
+@pytest.mark.parametrize("name", ["wide", "tiles", "blocks"])
 def test_generation_is_the_same_under_portions_preemption_and_graphs(name):
     """bf16 and the tensor-core kernels: sampled tokens of one engine against engines with other schedules."""
     cfg, _, model = case(name, torch.bfloat16)
@@ -258,7 +262,7 @@ def test_generation_is_the_same_under_portions_preemption_and_graphs(name):
                 assert abs(la[k] - lb[k]) < 0.3, kw
 
 
-@pytest.mark.parametrize("name", ["wide", "tiles"])
+@pytest.mark.parametrize("name", ["wide", "tiles", "blocks"])
 def test_stop_tokens_and_sampling_run_through_the_engine(name):
     cfg, _, model = case(name, torch.bfloat16)
     eng = engine(model, pages=12, slots=4, ctx=192)
@@ -272,7 +276,7 @@ def test_stop_tokens_and_sampling_run_through_the_engine(name):
     assert c.tokens[0].tolist() == a.tokens[0].tolist()[:first + 1]
 
 
-@pytest.mark.parametrize("name", ["wide", "tiles"])
+@pytest.mark.parametrize("name", ["wide", "tiles", "blocks"])
 def test_engine_server_serves_the_model(name):
     from tunix_b200.generate.engine import EngineServer
     cfg, _, model = case(name, torch.bfloat16)
@@ -287,7 +291,7 @@ def test_engine_server_serves_the_model(name):
     assert all(len(t) == 8 for t in first)
 
 
-@pytest.mark.parametrize("name", ["wide", "tiles"])
+@pytest.mark.parametrize("name", ["wide", "tiles", "blocks"])
 def test_scoring_with_padding_matches_unpadded_rows(name):
     cfg, _, model = case(name, torch.float32)
     rows = [C.tokens(cfg, n, 140 + n) for n in (6, 19)]
@@ -300,7 +304,7 @@ def test_scoring_with_padding_matches_unpadded_rows(name):
     assert close(z[1, :19], oracle(name, tuple(rows[1])), torch.float32)
 
 
-@pytest.mark.parametrize("name", ["mixed", "shared"])
+@pytest.mark.parametrize("name", ["mixed", "shared", "looped"])
 def test_trace_runner_replays_steps(name, tmp_path):
     import json
     import os

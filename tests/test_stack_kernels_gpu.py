@@ -7,6 +7,7 @@ import torch
 
 from tests import roluzen_oracle as O
 from tests import tovalix_oracle as TO
+from tests import zikezen_oracle as ZO
 
 pytestmark = pytest.mark.gpu
 DT = [torch.float32, torch.bfloat16]
@@ -256,3 +257,104 @@ def test_matrix_memory(H, dk, dv, cap, dtype, plain):
                 assert rel(state["n"][s][:, x], nn) < 2e-5
                 assert (state["m"][s][:, x].double().cpu() - m).abs().max() < 1e-4
             at += k
+
+
+# ------------------------------------------------------------------------------------------------ learned positions, loops
+@pytest.mark.parametrize("dtype", DT)
+@pytest.mark.parametrize("S,D", [(1, 48), (1, 37), (3, 64), (1, 1024)])
+def test_stream_step_scaled_embedding_positions_and_repetition(S, D, dtype):
+    """The embedding output at the start, and once more on top of a closed sublayer, whose sum is reported without it."""
+    from tunix_b200.ops import stack_kernels as SK
+    eps, tol, scale = 1e-3, 1e-6 if dtype == torch.float32 else 5e-3, 2.5
+    rb = batch([(1, 7, 3), (0, 0, 2), (2, 40, 1), (3, 5, 1)])
+    rb.pos0[3] = -1
+    n, at = 7, [7, 8, 9, 0, 1, 40, 0]
+    rb.tokens.copy_(torch.tensor([3, 0, 49, 7, 7, 1, 2]))
+    embed, pos, nw, wy, y = (rand(*s, dtype=dtype, seed=50 + i) for i, s in enumerate([(50, D), (41, D), (D,), (D,), (n, D)]))
+    one, mix = torch.ones(S, device="cuda", dtype=dtype), torch.eye(S, device="cuda", dtype=dtype)
+    d = lambda t: t.double().cpu()  # noqa: E731
+    cfg, w = {"embedding": {"scale": scale}}, {"embed": d(embed), "pos": d(pos)}
+    rows = torch.cat([ZO.embedding(cfg, w, rb.tokens[t:t + 1].cpu(), p) for t, p in enumerate(at)])
+    kw = dict(tokens=rb.tokens, embed=embed, embed_scale=scale, pos=pos, rb=rb)
+    x = torch.empty(n, S, D, device="cuda")
+    h = SK.stream_step(x, eps, w_in=one, norm_w=nw, **kw)
+    assert rel(x, rows[:, None].repeat(1, S, 1)) < 1e-6 and rel(h, ZO.rms(S * rows, eps) * d(nw)) < tol
+    total = torch.empty(n, D, device="cuda")
+    h = SK.stream_step(x, eps, y=y, wy=wy, mix=mix, w_out=one, w_in=one, norm_w=nw, sum_out=total, **kw)
+    closed = rows + ZO.rms(d(y), eps) * d(wy)
+    assert rel(total, S * closed) < 1e-6 and rel(x, (closed + rows)[:, None].repeat(1, S, 1)) < 1e-6
+    assert rel(h, ZO.rms(S * (closed + rows), eps) * d(nw)) < tol
+
+
+# ------------------------------------------------------------------------------------------------ experts
+def expert_case(D, F, E, top, n, dtype, seed=0):
+    h, gu, down = rand(n, D, dtype=dtype, seed=seed), rand(E, 2 * F, D, dtype=dtype, std=D ** -0.5, seed=seed + 1), \
+        rand(E, D, F, dtype=dtype, std=F ** -0.5, seed=seed + 2)
+    return h, gu, down, rand(n, E, seed=seed + 3, std=1.5), rand(E, dtype=dtype, seed=seed + 4, std=0.3)
+
+
+def expert_reference(h, gu, down, logits, correction, top):
+    h, gu, down, z = (t.double().cpu() for t in (h, gu, down, logits))
+    E, F2, _ = gu.shape
+    # the oracle's router reads the logits as they are
+    r = ZO.route(z, torch.eye(E).double(), 0.0 if correction is None else correction.double().cpu(), top)
+    out = torch.zeros_like(h)
+    for e in range(E):
+        t = r[:, e] > 0
+        w = {"gate": gu[e, :F2 // 2], "up": gu[e, F2 // 2:], "down": down[e]}
+        out[t] += r[t, e:e + 1] * ZO.glu(w, "", h[t])
+    return out, r
+
+
+EXPERTS = [(64, 64, 8, 2), (128, 40, 33, 4), (48, 24, 5, 5), (36, 13, 7, 3), (256, 128, 64, 8), (72, 200, 130, 6), (40, 8, 3, 1), (64, 64, 1, 1)]
+
+
+@pytest.mark.parametrize("dtype", DT)
+@pytest.mark.parametrize("D,F,E,top", EXPERTS)
+def test_experts(D, F, E, top, dtype):
+    """Few and many tokens (lists of few rows per expert, row segments for the grouped product, choice by choice), experts that
+    nobody takes, a correction that changes the choice and not the weights."""
+    from tunix_b200.ops import stack_kernels as SK
+    for n in (1, 5, 64, 128, 129, 300):
+        h, gu, down, z, corr = expert_case(D, F, E, top, n, dtype, seed=n)
+        for c in (corr, None):
+            want, _ = expert_reference(h, gu, down, z, c, top)
+            assert rel(SK.moe(h, z, c, gu, down, top, batch([(0, 0, n)])), want) < (2e-6 if dtype == torch.float32 else 1.2e-2), (n, c is None)
+
+
+@pytest.mark.parametrize("dtype", DT)
+@pytest.mark.parametrize("n", [40, 400])
+def test_one_expert_takes_every_token(n, dtype):
+    """Segments of very unequal length, and scores that the choice must not follow."""
+    from tunix_b200.ops import stack_kernels as SK
+    D, F, E = 64, 32, 12
+    h, gu, down, z, corr = expert_case(D, F, E, 2, n, dtype, seed=3)
+    corr[:], z[:, 7] = 0.0, -9.0
+    corr[7], corr[2] = 5.0, 3.0                                          # chosen by everyone for the correction's sake
+    want, r = expert_reference(h, gu, down, z, corr, 2)
+    assert ((r > 0).sum(0).tolist()) == [n if e in (2, 7) else 0 for e in range(E)] and r[:, 7].max() < 1e-2
+    assert rel(SK.moe(h, z, corr, gu, down, 2, batch([(0, 0, n)])), want) < (2e-6 if dtype == torch.float32 else 1.2e-2)
+
+
+@pytest.mark.parametrize("dtype", DT)
+@pytest.mark.parametrize("D,F", [(64, 32), (36, 13)])
+def test_idle_slots_choose_no_expert(D, F, dtype):
+    from tunix_b200.ops import stack_kernels as SK
+    h, gu, down, z, corr = expert_case(D, F, 6, 2, 5, dtype, seed=4)
+    rb = batch([(s, 3, 1) for s in range(5)])
+    rb.pos0[[1, 4]] = -1
+    h[[1, 4]], z[[1, 4]] = float("nan"), float("nan")                    # whatever an idle row holds
+    got = SK.moe(h, z, corr, gu, down, 2, rb)
+    live = [0, 2, 3]
+    want, _ = expert_reference(h[live], gu, down, z[live], corr, 2)
+    assert rel(got[live], want) < (2e-6 if dtype == torch.float32 else 1.2e-2) and got[[1, 4]].eq(0).all()
+
+
+def test_rows_of_experts_do_not_depend_on_the_company():
+    """A token alone, in a decode batch and inside a long portion: the same result to rounding."""
+    from tunix_b200.ops import stack_kernels as SK
+    h, gu, down, z, corr = expert_case(128, 64, 16, 4, 300, torch.bfloat16, seed=8)
+    full = SK.moe(h, z, corr, gu, down, 4, batch([(0, 0, 300)]))
+    for at, n in ((0, 1), (17, 40), (299, 1), (100, 128)):
+        part = SK.moe(h[at:at + n], z[at:at + n].contiguous(), corr, gu, down, 4, batch([(0, at, n)]))
+        assert rel(part, full[at:at + n]) < 8e-3
