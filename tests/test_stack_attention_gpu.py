@@ -462,7 +462,8 @@ def test_one_key_at_a_window_edge_beside_the_sink(kind, dtype, H, G, dq, dv, win
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("H,G,dq,dv,rot", [(4, 2, 16, 24, 16), (3, 1, 10, 6, 6), (8, 4, 64, 64, 64), (2, 2, 72, 128, 8), (5, 1, 24, 8, 0),
-                                           (6, 2, 40, 48, 24), (4, 2, 256, 128, 128), (2, 1, 96, 200, 2), (1, 1, 300, 20, 200)])
+                                           (6, 2, 40, 48, 24), (4, 2, 256, 128, 128), (2, 1, 96, 200, 2), (1, 1, 300, 20, 200),
+                                           (4, 2, 52, 40, 12), (3, 3, 40, 64, 10)])
 def test_weighted_norm_interleaved_rotation_and_wider_pages(H, G, dq, dv, rot, dtype):
     """Norm with weights before the rotation of neighbours, scaled frequencies; what lies behind a head is zero."""
     from tunix_b200.models.stack_exec import rope_table

@@ -1,12 +1,13 @@
 """Serving throughput of layer-stack models beside the closest uniform decoder of equal size:
 `python bench.py --workload stack_serving` or
-`python -m tunix_b200.generate.bench_stack [--models roluzen_2b,roluzen_8b,tovalix_2b,tovalix_8b]`.
+`python -m tunix_b200.generate.bench_stack [--models roluzen_2b,roluzen_8b,tovalix_2b,tovalix_8b,zikezen_2b,zikezen_8b]`.
 
 For every size: prefill tokens/s (`--prefill-seqs` prompts of `--prefill-len` tokens, one sampled token each) and decode
 tokens/s (`--decode-seqs` sequences at context `--decode-ctx`, `--decode-steps` captured steps), both through
 `PagedEngine.__call__`, random-init weights, uniform random token ids. The other model has the same width, feed-forward
-(of equal size where only one of them is gated), attention heads, vocabulary and number of layer passes, with
-sliding-window attention in every layer, of the same window or as long as the chunks.
+(of equal size where only one of them is gated, as much as a token passes where there are experts), attention heads, vocabulary and number of layer passes, with
+sliding-window attention in every layer, of the same window or as long as the chunks. Models with experts stand beside a second
+one, whose feed-forwards are all such experts.
 Times are CUDA events around the call after a warm-up call; a decode step streams the weights (far more than L2), the
 prefill's activations exceed L2 too."""
 from __future__ import annotations
@@ -47,10 +48,29 @@ def closest_config(cfg):
                        layer_pattern=("local",), dtype=torch.bfloat16)
 
 
+def closest_experts_config(cfg):
+    """The same with the experts of `cfg` in every layer, or None."""
+    ex = next((s for s in cfg.layer_specs if s.ff_kind == "experts"), None)
+    if ex is None:
+        return None
+    return closest_config(cfg).replace(num_experts=ex.experts, num_experts_per_tok=ex.top, moe_hidden_dim=ex.ff)
+
+
 def flops_per_token(model) -> float:
-    """2 x the weights of the projections a token passes (each layer pass counted), head excluded."""
-    runs = model.config.runs() if hasattr(model.config, "runs") else range(model.config.num_layers)
-    return 2.0 * sum(p.numel() for i in runs for p in model.layers[i].parameters() if p.dim() >= 2)
+    """2 x the weights of the projections a token passes (each layer pass and the experts it takes counted), head excluded."""
+    cfg = model.config
+    runs = cfg.runs() if hasattr(cfg, "runs") else range(cfg.num_layers)
+
+    def weights(i):
+        total = 0.0
+        for p in model.layers[i].parameters():
+            if p.dim() == 3:            # stacked experts
+                top = cfg.layer_specs[i].top if hasattr(cfg, "layer_specs") else cfg.num_experts_per_tok
+                total += p.numel() * (top / p.shape[0] if top else 1.0)
+            elif p.dim() == 2:
+                total += p.numel()
+        return total
+    return 2.0 * sum(weights(i) for i in runs)
 
 
 def measure(cfg, args) -> dict:
@@ -109,7 +129,7 @@ def measure(cfg, args) -> dict:
 
 
 def add_arguments(ap) -> None:
-    ap.add_argument("--models", default="roluzen_2b,roluzen_8b,tovalix_2b,tovalix_8b", help="layer-stack presets (stack_serving)")
+    ap.add_argument("--models", default="roluzen_2b,roluzen_8b,tovalix_2b,tovalix_8b,zikezen_2b,zikezen_8b", help="layer-stack presets (stack_serving)")
     ap.add_argument("--prefill-seqs", type=int, default=4)
     ap.add_argument("--prefill-len", type=int, default=4096)
     ap.add_argument("--decode-seqs", type=int, default=64)
@@ -123,12 +143,13 @@ def run(args) -> int:
     for name in args.models.split(","):
         cfg = get_config(name)
         ours = measure(cfg, args)
-        near = measure(closest_config(cfg), args)
+        near, experts = measure(closest_config(cfg), args), closest_experts_config(cfg)
         print(json.dumps({"metric": "stack_serving", "model": name, "unit": "tokens/s", "value": ours["prefill_tokens_per_sec"],
                           "higher_is_better": True, "dtype": "bf16", "data": "synthetic uniform token ids, random-init weights",
                           "prefill": f"{args.prefill_seqs} x {args.prefill_len}",
                           "decode": f"{args.decode_seqs} sequences at context {args.decode_ctx}, {args.decode_steps} steps",
-                          "stack": ours, "closest_uniform_decoder": near}), flush=True)
+                          "stack": ours, "closest_uniform_decoder": near,
+                          **({} if experts is None else {"closest_with_experts": measure(experts, args)})}), flush=True)
     return 0
 
 

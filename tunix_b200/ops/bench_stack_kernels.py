@@ -1,11 +1,11 @@
-"""Micro-benchmarks of the layer-stack kernels: `python -m tunix_b200.ops.bench_kernels stack [--model roluzen_8b|tovalix_8b]
+"""Micro-benchmarks of the layer-stack kernels: `python -m tunix_b200.ops.bench_kernels stack [--model roluzen_8b|tovalix_8b|zikezen_8b]
 [--batch 4 --seq 4096] [--decode-batch 64 --decode-ctx 1024] [--only mlstm_prefill,...]`.
 
 One JSON line per kernel at the sizes of a preset: median time with L2 flushed between iterations, the algorithmic bytes and
 operations (every input read once, every output written once; no repeated or split work counted), and the fraction of the
 roofline, i.e. the larger of bytes / copy bandwidth and operations / GEMM throughput over the measured time. The like kernels
-of uniform decoders (flash attention with the same window as a prefill calls it, paged decode, RMS norm, gated activation)
-come beside them."""
+of uniform decoders (flash attention with the same window as a prefill calls it, paged decode, RMS norm, gated activation,
+expert layer) come beside them."""
 from __future__ import annotations
 
 import json
@@ -47,8 +47,11 @@ def page_pool(B, ctx, k_cols, v_cols):
 
 def run(args, peaks, timer) -> None:
     from ..models.config import get_config
-    if get_config(args.model).family == "tovalix":
+    family = get_config(args.model).family
+    if family == "tovalix":
         run_tovalix(args, peaks, timer)
+    elif family == "zikezen":
+        run_zikezen(args, peaks, timer)
     else:
         run_roluzen(args, peaks, timer)
 
@@ -140,6 +143,100 @@ def run_tovalix(args, peaks, timer) -> None:
             with torch.no_grad():
                 report("like_attn_fwd", lambda: att(None), nb, win, note="window as long as a chunk")
                 report("like_attn_fwd_segments", lambda: att(seg), nb, win, note="as the padded prefill of uniform decoders calls it")
+
+
+def run_zikezen(args, peaks, timer) -> None:
+    from ..models.config import get_config
+    from ..models.stack_exec import rope_table
+    from . import functional as F
+    from . import kernels as K
+    from . import moe as uniform_moe
+    from . import reference as R
+    from . import stack_kernels as SK
+    report = reporter(args, peaks, timer)
+    dev, bf = torch.device("cuda"), torch.bfloat16
+    cfg = get_config(args.model)
+    sp = cfg.layer_specs[0].mixer
+    ex = next(s for s in cfg.layer_specs if s.ff_kind == "experts")
+    a, gl, D = sp.left, sp.right, cfg.embed_dim
+    rand = lambda *s: torch.randn(*s, device=dev).to(bf)  # noqa: E731
+    E, top, ff = ex.experts, ex.top, ex.ff
+    gate_up, down, router, corr = rand(E, 2 * ff, D), rand(E, D, ff), rand(E, D), rand(E)
+    for phase, rb, B, ctx in phases(args):
+        n, one = rb.n, phase == "decode"
+        # --- residual
+        x, y, w, h = torch.randn(n, 1, D, device=dev), rand(n, D), torch.ones(D, device=dev, dtype=bf), rand(n, D)
+        unit, table, pos = torch.ones(1, device=dev, dtype=bf), rand(cfg.vocab_size, D), rand(cfg.positions, D)
+        kw = dict(y=y, wy=w, mix=unit, w_out=unit, w_in=unit, norm_w=w)
+        report(f"stream_step_normed_{phase}", lambda: SK.stream_step(x, 1e-6, **kw), n * D * 12.0)
+        report(f"stream_step_again_{phase}", lambda: SK.stream_step(x, 1e-6, tokens=rb.tokens, embed=table, embed_scale=2.0, pos=pos, rb=rb,
+                                                                    **kw), n * D * 14.0, note="tokens of one row")
+        report(f"like_rmsnorm_{phase}", lambda: K.rmsnorm_fwd(y, w, 1e-6, want_rstd=False), n * D * 4.0)
+        del x, table, pos
+        # --- gated linear attention
+        H, dk, dv, rank = gl.heads, gl.dim, gl.vdim, gl.decay_rank
+        q, k, v, g = rand(n, H * dk), rand(n, H * dk), rand(n, H * dv), rand(n, H * dv)
+        z, c0, xr, w2 = torch.randn(n, H * dk, device=dev), rand(H * dk) + 2, rand(n, rank), rand(H * dk, rank) * rank ** -0.5
+        S, nw, nwh = torch.zeros(B, H, dk, dv, device=dev), torch.ones(dv, device=dev, dtype=bf), torch.ones(H * dv, device=dev, dtype=bf)
+        nb, fl = n * H * (dk * 8.0 + dv * 6) + B * H * dk * dv * 8.0, 0.0 if one else n * H * (4.0 * dk * dv + 16 * (dk + dv))
+        run_ = lambda mode, zz, kk, c1, **o: SK.gated_linear(mode, q, kk, v, zz, c0, c1, rb, H, dk, dv, S, o.pop("nw", nw), 1e-6, gate=g, **o)  # noqa: E731
+        report(f"gla_{phase}", lambda: run_(SK.GATES_ROOT, z, k, None, q_scale=0.1, tau=16.0), nb, fl)
+        if one:
+            report("gla_bottleneck_decode", lambda: run_(SK.GATES_ROOT, None, k, None, q_scale=0.1, tau=16.0, low_rank=(xr, w2)),
+                   nb - n * H * dk * 4.0 + n * rank * 2 + H * dk * rank * 2)
+        report(f"like_wkv_{phase}", lambda: run_(SK.GATES_BONUS, z, k, c0, per_head=True, nw=nwh), nb, fl, note="same sizes")
+        report(f"like_hgrn2_{phase}", lambda: run_(SK.GATES_LOWER, z, None, torch.sigmoid(c0)), nb - n * H * dk * 2, fl, note="same sizes")
+        report(f"gates_product_{phase}", lambda: K.gemm(xr, w2, out_dtype=torch.float32), n * (rank * 2.0 + H * dk * 4) + H * dk * rank * 2)
+        del q, k, v, g, z, S
+        # --- attention
+        NQ, NK = a.heads * a.dim, a.kv_heads * a.dim
+        kp, vp, table = page_pool(B, ctx, NK, NK)
+        proj, q, hw = rand(n, NQ + 2 * NK), rand(n, NQ), torch.ones(a.dim, device=dev, dtype=bf)
+        cos, sin = rope_table(ctx, a.rot_dims, a.rot_base, dev)
+        rope = lambda **o: SK.rope_norm_write(proj, 0, NQ, NQ + NK, cos, sin, a.rot_dims, 1e-6, rb, table, 64, a.heads, a.kv_heads, a.dim, a.vdim,  # noqa: E731
+                                              kp, vp, **o)
+        report(f"rope_norm_write_{phase}", lambda: rope(q_w=hw, k_w=hw, interleaved=True), n * (NQ + 2 * NK) * 4.0)
+        report(f"like_rope_norm_write_{phase}", lambda: rope(), n * (NQ + 2 * NK) * 4.0, note="halves, no weights")
+        if one:
+            keys = min(ctx, a.window)
+            nb = B * keys * 2 * NK * 2.0 + n * NQ * 4.0
+            split = K.decode_split_tokens(B, a.kv_heads, min(ctx, a.window + 128))
+            q3, lens_t = q.view(B, a.heads, a.dim), rb.pos0 + 1
+            pd = lambda **o: K.paged_decode(q3, kp, vp, table, rb.slot, lens_t, num_kv_heads=a.kv_heads, page_size=64, max_ctx=ctx,  # noqa: E731
+                                            split_tokens=split, scale=a.scale, window=a.window, **o)
+            report("attention_decode", lambda: pd(sink=0.0, out_scale=0.7), nb)
+            report("like_paged_decode", lambda: pd(), nb, note="no sink")
+        else:
+            fl = sum(min(i + 1, a.window) for i in range(args.seq)) * float(B) * a.heads * a.dim * 4.0
+            nb = n * (2 * NQ + 2 * NK) * 2.0
+            pk = dict(num_heads=a.heads, num_kv_heads=a.kv_heads, head_dim=a.dim, scale=a.scale, window=a.window)
+            report("attention_prefill", lambda: K.attn_fwd_paged(q, kp, vp, rb, table, 64, sink=0.0, out_scale=0.7, **pk), nb, fl)
+            q4 = q.view(B, args.seq, a.heads, a.dim)
+            k4, v4 = (rand(B, args.seq, a.kv_heads, a.dim) for _ in range(2))
+            seg = torch.ones(B, args.seq, dtype=torch.int32, device=dev)
+            att = lambda s: F.attention(q4, k4, v4, scale=a.scale, causal=True, window=a.window, seg_q=s, seg_k=s)  # noqa: E731
+            with torch.no_grad():
+                report("like_attn_fwd", lambda: att(None), nb, fl, note="same window")
+                report("like_attn_fwd_segments", lambda: att(seg), nb, fl, note="as the padded prefill of uniform decoders calls it")
+            del q4, k4, v4
+        del kp, vp, proj, q
+        # --- experts
+        logits = torch.randn(n, E, device=dev)
+        used = min(E, n * top)
+        nb, fl = n * D * 4.0 + used * 6.0 * ff * D + n * E * 4, n * top * 6.0 * ff * D
+        report(f"router_{phase}", (lambda: SK.few_outputs(h, router)) if one else (lambda: K.gemm(h, router, out_dtype=torch.float32)),
+               n * (D * 2.0 + E * 4) + E * D * 2)
+        report(f"experts_{phase}", lambda: SK.moe(h, logits, corr, gate_up, down, top, rb), nb, fl)
+        gw, uw = gate_up[:, :ff].contiguous(), gate_up[:, ff:].contiguous()
+
+        def uniform():
+            wts, idx, _ = R.topk_router_ref(logits, top, True)
+            return uniform_moe.experts(h, wts, idx, gw, uw, down)
+        with torch.no_grad():
+            report(f"like_experts_{phase}", uniform, nb, fl, note="expert layer of uniform decoders, routing included")
+        half, up = rand(n, cfg.hidden_dim), rand(n, cfg.hidden_dim)
+        report(f"glu_{phase}", lambda: K.glu_fwd(half, up, K.GLU_SILU), n * cfg.hidden_dim * 6.0)
+        del half, up, gw, uw
 
 
 def run_roluzen(args, peaks, timer) -> None:
