@@ -316,17 +316,19 @@ def zikezen_weights(cfg, seed=0, rank=8):
         put(p + "side.norm", D, std=0.3)
         w[p + "side.norm"][:ROUTED] = 0
     w["pos"][:, :ROUTED] = 0
-    rows = (2 * torch.randn(30 * V, ROUTED, generator=g)).to(torch.bfloat16).float()
-    clear = torch.ones(len(rows), dtype=torch.bool)
-    for i, layer in enumerate(cfg["layers"]):
-        if layer["mlp"] is not None and layer["mlp"]["kind"] == "moe" and layer["mlp"]["router"]["top"] < layer["mlp"]["router"]["experts"]:
-            top = layer["mlp"]["router"]["top"]
-            for size in torch.linspace(0.1, 1.4, 150):             # whatever the norm makes of a row's size
-                s = torch.softmax(size * rows @ w[f"l{i}.mlp.router"][:, :ROUTED].T, -1) + w[f"l{i}.mlp.correction"]
-                s = s.sort(-1, descending=True).values
-                clear &= s[:, top - 1] - s[:, top] > 0.015
-    assert clear.sum() >= V, clear.sum()
-    w["embed"][:, :ROUTED] = rows[clear][:V] / cfg["embedding"]["scale"]
+    kept = []
+    while sum(map(len, kept)) < V:
+        rows = (2 * torch.randn(20 * V, ROUTED, generator=g)).to(torch.bfloat16).float()
+        clear = torch.ones(len(rows), dtype=torch.bool)
+        for i, layer in enumerate(cfg["layers"]):
+            if layer["mlp"] is not None and layer["mlp"]["kind"] == "moe" and layer["mlp"]["router"]["top"] < layer["mlp"]["router"]["experts"]:
+                top = layer["mlp"]["router"]["top"]
+                for size in torch.linspace(0.1, 1.4, 150):             # whatever the norm makes of a row's size
+                    s = torch.softmax(size * rows @ w[f"l{i}.mlp.router"][:, :ROUTED].T, -1) + w[f"l{i}.mlp.correction"]
+                    s = s.topk(top + 1, -1).values
+                    clear &= s[:, top - 1] - s[:, top] > 0.015
+        kept.append(rows[clear])
+    w["embed"][:, :ROUTED] = torch.cat(kept)[:V] / cfg["embedding"]["scale"]
     w["embed"] = w["embed"].to(torch.bfloat16).float()
     return w
 

@@ -5,8 +5,8 @@
 //   moe_plan, moe_place : a row segment per expert (multiples of 128 rows) for the grouped tcgen05 GEMM (gemm.cu), and the row of
 //                      every (token, choice). Padding rows of a segment are never read back, so nothing zeroes them.
 //   moe_route_lists  : the same choice in one CTA for a decode step, with the choices sorted by expert.
-//   expert_rows      : few rows per expert: a CTA streams 32 weight rows of one expert once (16 gate and 16 up rows, or 32 down
-//                      rows) past the rows that chose it, 16 at a time on mma.sync; its warps split the contraction.
+//   expert_rows      : few rows per expert: a CTA streams 32 weight rows of one expert (16 gate and 16 up rows, or 32 down rows)
+//                      past the rows that chose it, up to 64 at a time on mma.sync.
 //   expert_plain     : any sizes, also 32-bit: a warp per choice and output.
 //   moe_sum          : the sum over a token's choices.
 // A choice is numbered token * top + j. Tokens of idle slots choose nothing (expert -1).
@@ -189,59 +189,56 @@ moe_route_lists_kernel(const float* __restrict__ z, const T* __restrict__ correc
   }
 }
 
-// Rows of one expert, 16 at a time, times 32 of its weight rows. GLU: x rows belong to tokens, out[choice, f] = silu(gate) * up
-// for 16 f, T. Otherwise x rows belong to choices, out[choice, d] = weight * product for 32 d, fp32.
+// Rows of one expert, up to 64 at a time, times 32 of its weight rows. GLU: x rows belong to tokens, out[choice, f] = silu(gate) *
+// up for 16 f, T. Otherwise x rows belong to choices, out[choice, d] = weight * product for 32 d, fp32. The warps of a CTA split
+// the contraction and meet in shared memory; both operands of a product see the same permutation of k, so nothing is shuffled.
 constexpr int RW = 8;           // warps
-template <bool GLU>
-__global__ void __launch_bounds__(32 * RW)
-expert_rows_kernel(const bf* __restrict__ x, long long ldx, const bf* __restrict__ w, int K, int N, const int* __restrict__ off,
-                   const int* __restrict__ list, const float* __restrict__ wts, int top, void* __restrict__ out) {
-  __shared__ float part[RW][16][33];
-  pdl_trigger();
-  pdl_wait();
-  const int e = blockIdx.y, i0 = off[e], i1 = off[e + 1];
-  if (i0 >= i1) return;
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, q8 = (lane & 3) * 8;
+template <bool GLU, int MT>
+__device__ __forceinline__ void expert_pass(const bf* x, long long ldx, const bf* const (&wr)[4], int K, int N, const int* list, int left,
+                                            const float* wts, int top, int n0, float (&part)[RW][16][33], void* out) {
   constexpr int TILE = GLU ? 16 : 32;
-  const int n0 = blockIdx.x * TILE;
-  // this lane's four weight rows: GLU gate n0 + g, + 8, then up; otherwise n0 + g + 8 j. Rows past N repeat the last one.
-  const bf* wr[4];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, q8 = (lane & 3) * 8;
+  const bf* xr[MT][2];
+  float acc[MT][4][4];
 #pragma unroll
-  for (int j = 0; j < 4; ++j) {
-    const int r = GLU ? min(n0 + (j & 1) * 8 + g, N - 1) + (j >> 1) * N : min(n0 + j * 8 + g, N - 1);
-    wr[j] = w + ((long long)e * (GLU ? 2 * N : N) + r) * K;
-  }
-  for (int r0 = i0; r0 < i1; r0 += 16) {
-    const int ca = list[min(r0 + g, i1 - 1)], cb = list[min(r0 + g + 8, i1 - 1)];
-    const bf *xa = x + (GLU ? ca / top : ca) * ldx, *xb = x + (GLU ? cb / top : cb) * ldx;
-    float acc[4][4];
+  for (int m = 0; m < MT; ++m)
 #pragma unroll
-    for (int j = 0; j < 4; ++j)
+    for (int h = 0; h < 2; ++h) {
+      const int c = list[min(m * 16 + h * 8 + g, left - 1)];
+      xr[m][h] = x + (GLU ? c / top : c) * ldx;
 #pragma unroll
-      for (int i = 0; i < 4; ++i) acc[j][i] = 0.f;
-#pragma unroll 4
-    for (int kb = warp * 32; kb < K; kb += RW * 32) {           // whole warps stay together for the products
-      const int k = kb + q8;                                    // K is a multiple of 8: a lane's 8 elements are in or out
-      const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
-      const uint4 a = k < K ? *reinterpret_cast<const uint4*>(xa + k) : zero, b = k < K ? *reinterpret_cast<const uint4*>(xb + k) : zero;
+      for (int j = 0; j < 4; ++j) acc[m][j][2 * h] = acc[m][j][2 * h + 1] = 0.f;
+    }
+#pragma unroll (MT == 1 ? 4 : MT == 2 ? 2 : 1)
+  for (int kb = warp * 32; kb < K; kb += RW * 32) {             // whole warps stay together for the products
+    const int k = kb + q8;                                      // K is a multiple of 8: a lane's 8 elements are in or out
+    const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+    uint4 w[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) w[j] = k < K ? __ldg(reinterpret_cast<const uint4*>(wr[j] + k)) : zero;
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+      const uint4 a = k < K ? *reinterpret_cast<const uint4*>(xr[m][0] + k) : zero, b = k < K ? *reinterpret_cast<const uint4*>(xr[m][1] + k) : zero;
       const uint32_t s0[4] = {a.x, b.x, a.y, b.y}, s1[4] = {a.z, b.z, a.w, b.w};
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        const uint4 c = k < K ? __ldg(reinterpret_cast<const uint4*>(wr[j] + k)) : zero;
-        mma_16816(acc[j], s0, c.x, c.y);
-        mma_16816(acc[j], s1, c.z, c.w);
+        mma_16816(acc[m][j], s0, w[j].x, w[j].y);
+        mma_16816(acc[m][j], s1, w[j].z, w[j].w);
       }
     }
-    const int c2 = 2 * (lane & 3);
+  }
+  const int c2 = 2 * (lane & 3);
+#pragma unroll
+  for (int m = 0; m < MT; ++m) {
 #pragma unroll
     for (int j = 0; j < 4; ++j)
 #pragma unroll
-      for (int i = 0; i < 4; ++i) part[warp][g + (i >> 1) * 8][j * 8 + c2 + (i & 1)] = acc[j][i];
+      for (int i = 0; i < 4; ++i) part[warp][g + (i >> 1) * 8][j * 8 + c2 + (i & 1)] = acc[m][j][i];
     __syncthreads();
     for (int i = threadIdx.x; i < 16 * TILE; i += 32 * RW) {
       const int r = i / TILE, c = i % TILE, col = n0 + c;
-      if (r0 + r < i1 && col < N) {
-        const int choice = list[r0 + r];
+      if (m * 16 + r < left && col < N) {
+        const int choice = list[m * 16 + r];
         float v = 0.f, u = 0.f;
 #pragma unroll
         for (int j = 0; j < RW; ++j) {
@@ -253,6 +250,38 @@ expert_rows_kernel(const bf* __restrict__ x, long long ldx, const bf* __restrict
       }
     }
     __syncthreads();
+  }
+}
+
+template <bool GLU>
+__global__ void __launch_bounds__(32 * RW, 2)
+expert_rows_kernel(const bf* __restrict__ x, long long ldx, const bf* __restrict__ w, int K, int N, const int* __restrict__ off,
+                   const int* __restrict__ list, const float* __restrict__ wts, int top, void* __restrict__ out) {
+  __shared__ float part[RW][16][33];
+  pdl_trigger();
+  pdl_wait();
+  const int e = blockIdx.y, i0 = off[e], i1 = off[e + 1];
+  if (i0 >= i1) return;
+  const int g = (threadIdx.x & 31) >> 2, n0 = blockIdx.x * (GLU ? 16 : 32);
+  // this lane's four weight rows: GLU gate n0 + g, + 8, then up; otherwise n0 + g + 8 j. Rows past N repeat the last one.
+  const bf* wr[4];
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const int r = GLU ? min(n0 + (j & 1) * 8 + g, N - 1) + (j >> 1) * N : min(n0 + j * 8 + g, N - 1);
+    wr[j] = w + ((long long)e * (GLU ? 2 * N : N) + r) * K;
+  }
+  for (int r0 = i0; r0 < i1;) {
+    const int left = i1 - r0;
+    if (left > 32) {
+      expert_pass<GLU, 4>(x, ldx, wr, K, N, list + r0, left, wts, top, n0, part, out);
+      r0 += 64;
+    } else if (left > 16) {
+      expert_pass<GLU, 2>(x, ldx, wr, K, N, list + r0, left, wts, top, n0, part, out);
+      r0 += 32;
+    } else {
+      expert_pass<GLU, 1>(x, ldx, wr, K, N, list + r0, left, wts, top, n0, part, out);
+      r0 += 16;
+    }
   }
 }
 
