@@ -161,7 +161,7 @@ def run_zikezen(args, peaks, timer) -> None:
     a, gl, D = sp.left, sp.right, cfg.embed_dim
     rand = lambda *s: torch.randn(*s, device=dev).to(bf)  # noqa: E731
     E, top, ff = ex.experts, ex.top, ex.ff
-    gate_up, down, router, corr = rand(E, 2 * ff, D), rand(E, D, ff), rand(E, D), rand(E)
+    gate_up, down, router, corr = rand(E, 2 * ff, D), rand(E, D, ff), rand(E, D), rand(E) * 0.01
     for phase, rb, B, ctx in phases(args):
         n, one = rb.n, phase == "decode"
         # --- residual
@@ -222,7 +222,7 @@ def run_zikezen(args, peaks, timer) -> None:
         del kp, vp, proj, q
         # --- experts
         logits = torch.randn(n, E, device=dev)
-        used = min(E, n * top)
+        used = (torch.softmax(logits, -1) + corr).topk(top, -1).indices.unique().numel()
         nb, fl = n * D * 4.0 + used * 6.0 * ff * D + n * E * 4, n * top * 6.0 * ff * D
         report(f"router_{phase}", (lambda: SK.few_outputs(h, router)) if one else (lambda: K.gemm(h, router, out_dtype=torch.float32)),
                n * (D * 2.0 + E * 4) + E * D * 2)
