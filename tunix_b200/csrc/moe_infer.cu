@@ -192,8 +192,8 @@ moe_route_lists_kernel(const float* __restrict__ z, const T* __restrict__ correc
 // Rows of one expert, up to 64 at a time, times 32 of its weight rows. GLU: x rows belong to tokens, out[choice, f] = silu(gate) *
 // up for 16 f, T. Otherwise x rows belong to choices, out[choice, d] = weight * product for 32 d, fp32. The warps of a CTA split
 // the contraction and meet in shared memory; both operands of a product see the same permutation of k, so nothing is shuffled.
-constexpr int RW = 8;           // warps
-template <bool GLU, int MT>
+__host__ __device__ constexpr int row_warps(bool glu) { return glu ? 8 : 4; }      // shorter contractions: fewer warps, more CTAs
+template <bool GLU, int MT, int RW>
 __device__ __forceinline__ void expert_pass(const bf* x, long long ldx, const bf* const (&wr)[4], int K, int N, const int* list, int left,
                                             const float* wts, int top, int n0, float (&part)[RW][16][33], void* out) {
   constexpr int TILE = GLU ? 16 : 32;
@@ -254,9 +254,10 @@ __device__ __forceinline__ void expert_pass(const bf* x, long long ldx, const bf
 }
 
 template <bool GLU>
-__global__ void __launch_bounds__(32 * RW, 2)
+__global__ void __launch_bounds__(32 * row_warps(GLU), 16 / row_warps(GLU))
 expert_rows_kernel(const bf* __restrict__ x, long long ldx, const bf* __restrict__ w, int K, int N, const int* __restrict__ off,
                    const int* __restrict__ list, const float* __restrict__ wts, int top, void* __restrict__ out) {
+  constexpr int RW = row_warps(GLU);
   __shared__ float part[RW][16][33];
   pdl_trigger();
   pdl_wait();
@@ -273,13 +274,13 @@ expert_rows_kernel(const bf* __restrict__ x, long long ldx, const bf* __restrict
   for (int r0 = i0; r0 < i1;) {
     const int left = i1 - r0;
     if (left > 32) {
-      expert_pass<GLU, 4>(x, ldx, wr, K, N, list + r0, left, wts, top, n0, part, out);
+      expert_pass<GLU, 4, RW>(x, ldx, wr, K, N, list + r0, left, wts, top, n0, part, out);
       r0 += 64;
     } else if (left > 16) {
-      expert_pass<GLU, 2>(x, ldx, wr, K, N, list + r0, left, wts, top, n0, part, out);
+      expert_pass<GLU, 2, RW>(x, ldx, wr, K, N, list + r0, left, wts, top, n0, part, out);
       r0 += 32;
     } else {
-      expert_pass<GLU, 1>(x, ldx, wr, K, N, list + r0, left, wts, top, n0, part, out);
+      expert_pass<GLU, 1, RW>(x, ldx, wr, K, N, list + r0, left, wts, top, n0, part, out);
       r0 += 16;
     }
   }
@@ -388,10 +389,10 @@ TB_API int tb_moe_experts(int dtype, int rows, const void* x, long long ldx, con
   cudaError_t err;
   if (rows) {
     if (dtype != 0 || D % 8 || F % 8 || ldx % 8 || E > 65535 || ((uintptr_t)x & 15) || ((uintptr_t)wgu & 15) || ((uintptr_t)wd & 15)) return -2;
-    err = launch_pdl(expert_rows_kernel<true>, dim3((F + 15) / 16, E), dim3(32 * RW), 0, stream, (const bf*)x, ldx, (const bf*)wgu, D, F,
+    err = launch_pdl(expert_rows_kernel<true>, dim3((F + 15) / 16, E), dim3(32 * row_warps(true)), 0, stream, (const bf*)x, ldx, (const bf*)wgu, D, F,
                      off, list, wts, top, act);
     if (err != cudaSuccess) return -5;
-    err = launch_pdl(expert_rows_kernel<false>, dim3((D + 31) / 32, E), dim3(32 * RW), 0, stream, (const bf*)act, (long long)F,
+    err = launch_pdl(expert_rows_kernel<false>, dim3((D + 31) / 32, E), dim3(32 * row_warps(false)), 0, stream, (const bf*)act, (long long)F,
                      (const bf*)wd, F, D, off, list, wts, top, (void*)y);
     if (err != cudaSuccess) return -5;
   } else {
