@@ -403,12 +403,13 @@ def test_zikezen_memory_against_its_unrolled_sum():
 
 
 def test_sequences_stay_within_the_learned_positions():
-    from tunix_b200.generate.engine import PagedEngine
+    from types import SimpleNamespace
+
+    from tunix_b200.generate.engine import check_length
     from tunix_b200.models.hf_config import config_from_hf
-    eng = PagedEngine.__new__(PagedEngine)
-    eng.cfg = config_from_hf(C.CASES["looped"])
-    eng._check_length(512)
+    eng = SimpleNamespace(cfg=config_from_hf(C.CASES["looped"]))
+    check_length(eng, 512)
     with pytest.raises(ValueError, match="positions"):
-        eng._check_length(513)
-    eng.cfg = config_from_hf(C.CASES["shared"])
-    eng._check_length(10 ** 6)
+        check_length(eng, 513)
+    check_length(SimpleNamespace(cfg=config_from_hf(C.CASES["shared"])), 10 ** 6)
+    check_length(SimpleNamespace(), 10 ** 6)

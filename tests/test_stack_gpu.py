@@ -330,3 +330,16 @@ def test_trace_runner_replays_steps(name, tmp_path):
     for step, rows in ((0, [0, 39]), (1, [8]), (2, [69])):
         got = torch.from_numpy(np.fromfile(tmp_path / f"{step}.f32", "<f4")).view(len(rows), -1)
         assert close(got, want[rows], torch.float32)
+
+
+def test_sequences_longer_than_the_learned_positions_are_refused():
+    cfg, _, model = case("looped", torch.bfloat16)
+    ses = session(model, pages=10, slots=1)
+    toks = C.tokens(cfg, cfg["max_positions"], 160)
+    z = ses.step([("a", toks[:500], [499])])
+    assert ses.step([("a", toks[500:], [11])]).isfinite().all() and z.isfinite().all()
+    with pytest.raises(ValueError, match="positions"):
+        ses.step([("a", [1], [0])])
+    eng = engine(model, pages=10, slots=1)
+    with pytest.raises(ValueError, match="positions"):
+        eng(prompt_token_ids=[toks[:500]], max_generation_steps=20, max_prompt_length=512, eos_tokens=[-1])

@@ -133,6 +133,13 @@ class PagePool:
         self.table.copy_(torch.from_numpy(self.table_host), non_blocking=False)
 
 
+def check_length(engine, tokens: int) -> None:
+    """Refuse a sequence that is longer than a model's learned positions (`StackConfig.positions`; other models have none)."""
+    limit = getattr(getattr(engine, "cfg", None), "positions", 0)
+    if limit and tokens > limit:
+        raise ValueError(f"a sequence of {tokens} tokens: the model has {limit} positions")
+
+
 class PagedEngine(BaseSampler):
     def __init__(self, transformer, tokenizer, cache_config: CacheConfig, page_size: int = 64,
                  max_running_requests: int = 64, use_cuda_graph: bool = True, check_every: int = 16,
@@ -205,11 +212,6 @@ class PagedEngine(BaseSampler):
         for name, w in updated_weights.items():
             if own[name].data_ptr() != w.data_ptr():
                 own[name].copy_(w.to(own[name].device, own[name].dtype))
-
-    def _check_length(self, tokens: int) -> None:
-        limit = getattr(self.cfg, "positions", 0)
-        if limit and tokens > limit:
-            raise ValueError(f"a sequence of {tokens} tokens: the model has {limit} positions")
 
     def delete_cache(self) -> None:
         self.pool = None
@@ -544,7 +546,7 @@ class PagedEngine(BaseSampler):
         plen = max_prompt_length if max_prompt_length else next_power_of_2(max(len(r) for r in rows))
         if plen + max_generation_steps > self.cache_size:
             raise ValueError("prompt + generation exceeds the configured cache size")
-        self._check_length(max(len(r) for r in rows) + max_generation_steps)
+        check_length(self, max(len(r) for r in rows) + max_generation_steps)
         was_training = self._model.training
         self._model.eval()
         prompts_all, plens_all = pad_prompts_left(rows, plen, pad_id)
@@ -900,7 +902,7 @@ class StepSession:
             if not tokens:
                 continue
             req = self._live.get(rid)
-            eng._check_length((req[1] if req else 0) + len(tokens))
+            check_length(eng, (req[1] if req else 0) + len(tokens))
             if req is None:
                 if not self._free:
                     raise RuntimeError(f"request {rid!r}: all {eng.max_running} slots are in use")
@@ -951,7 +953,7 @@ class EngineServer:
         import threading
         if max_prompt_length + max_new_tokens > engine.cache_size:
             raise ValueError("prompt + generation exceeds the configured cache size")
-        engine._check_length(max_prompt_length + max_new_tokens)
+        check_length(engine, max_prompt_length + max_new_tokens)
         self.engine = engine
         self.max_new_tokens = int(max_new_tokens)
         self.P = int(max_prompt_length)
