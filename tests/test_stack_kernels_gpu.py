@@ -7,6 +7,7 @@ import torch
 
 from tests import roluzen_oracle as O
 from tests import tovalix_oracle as TO
+from tests import zigipel_oracle as ZG
 from tests import zikezen_oracle as ZO
 
 pytestmark = pytest.mark.gpu
@@ -56,11 +57,15 @@ def test_stream_step(S, D, dtype):
 
 @pytest.mark.parametrize("dtype", DT)
 @pytest.mark.parametrize("F", [8, 31, 500])
-def test_silu_mul(F, dtype):
+def test_glu(F, dtype):
+    from tunix_b200.ops import kernels as K
     from tunix_b200.ops import stack_kernels as SK
     gu = rand(17, 2 * F, dtype=dtype, std=3)
-    ref = O.silu(gu[:, :F].double()) * gu[:, F:].double()
-    assert rel(SK.silu_mul(gu), ref) < (1e-6 if dtype == torch.float32 else 5e-3)
+    tol = 1e-6 if dtype == torch.float32 else 5e-3
+    assert rel(SK.glu(gu, K.GLU_SILU), O.silu(gu[:, :F].double()) * gu[:, F:].double()) < tol
+    wide = torch.full((17, F + 5), 7.0, dtype=dtype, device="cuda")
+    got = SK.glu(gu, K.GLU_GELU, wide[:, 2:F + 2])
+    assert rel(got, ZG.gelu_tanh(gu[:, :F].double()) * gu[:, F:].double()) < tol and wide[:, :2].eq(7).all() and wide[:, F + 2:].eq(7).all()
 
 
 @pytest.mark.parametrize("dtype", DT)

@@ -28,7 +28,7 @@ NVCC_FLAGS = [
     "--expt-relaxed-constexpr",
 ]
 # kernels that also serve the 32-bit mode of a model (see csrc/precise.cuh) keep full-precision math functions
-PRECISE_SOURCES = {"stack.cu", "recurrent.cu", "linear_attention.cu", "window_attention.cu", "moe_infer.cu"}
+PRECISE_SOURCES = {"stack.cu", "recurrent.cu", "linear_attention.cu", "window_attention.cu", "moe_infer.cu", "latent_attention.cu"}
 CXX_FLAGS = ["-O3", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread"]
 
 

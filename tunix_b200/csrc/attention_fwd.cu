@@ -10,7 +10,8 @@
 //   warp 4     : one elected thread issues every TMA load (no multicast) and every
 //                tcgen05.mma: S_{j+1} = Q K_{j+1}^T is in flight while the softmax of block j runs.
 // Masks: causal (with offset for Tq != Tk), sliding window, segment ids (packing / padding),
-// key length. Logit soft-cap (Gemma-2). Head dim 64 / 128 / 256.
+// key length. Logit soft-cap (Gemma-2). Head dim 64 / 128 / 256; the paged form also takes unequal key and value sizes,
+// learned sinks and output gates per head, and queries and keys whose heads lie further apart than they are wide.
 // Every mbarrier wait is bounded; a timeout sets *status and the CTA unwinds.
 //
 // Replaces the eager [B,N,T,S] attention and the TPU-only splash attention of the reference
@@ -48,31 +49,42 @@ struct AttnArgs {
   int far;
   int vd;                    // paged: value columns of a head that are written (heads may be stored with zeros behind them)
   float sink2;               // paged: one more score without a value in the sum of the weights, in log2 units (-inf: none)
+  const float* sinks;        // paged: [N] or null, a sink per head instead
+  const __nv_bfloat16* gate; // paged: rows ldg apart, or null: head n's output is multiplied by sigmoid(gate[row, n])
+  long long ldg;
+  int q_heads;               // paged: columns from one query head to the next
   float out_scale;           // paged: factor of the output
 };
 
-template <int H>
+// H: query / key head size, HV: value head size
+template <int H, int HV>
 struct FwdCfg {
   static constexpr int HS = H / 64;                 // 64-column slabs along the head dim
+  static constexpr int HVS = HV / 64;
   static constexpr int Q_BYTES = HS * BQ * 128;     // K-major slabs [128 x 128B]
-  static constexpr int KV_BYTES = HS * BKV * 128;   // slabs [64 x 128B]
+  static constexpr int K_BYTES = HS * BKV * 128;    // slabs [64 x 128B]
+  static constexpr int V_BYTES = HVS * BKV * 128;
   static constexpr int P_BYTES = BQ * 128;
+  // two V buffers, or one where that lets a second CTA share the SM
+  static constexpr int FIXED = Q_BYTES + K_BYTES + P_BYTES + 128 + 1024;
+  static constexpr int NV = FIXED + 2 * V_BYTES > 113 * 1024 && FIXED + V_BYTES <= 113 * 1024 ? 1 : 2;
   static constexpr int OFF_Q = 0;
   static constexpr int OFF_K = OFF_Q + Q_BYTES;
-  static constexpr int OFF_V = OFF_K + KV_BYTES;    // two V buffers
-  static constexpr int OFF_P = OFF_V + 2 * KV_BYTES;
+  static constexpr int OFF_V = OFF_K + K_BYTES;
+  static constexpr int OFF_P = OFF_V + NV * V_BYTES;
   static constexpr int OFF_BAR = OFF_P + P_BYTES;
   static constexpr int SMEM_BYTES = OFF_BAR + 128 + 1024;
   static constexpr int TMEM_S = 0;                  // two S buffers of 64 columns
   static constexpr int TMEM_O = 128;
-  static constexpr int TMEM_COLS = (128 + H) <= 256 ? 256 : 512;
+  static constexpr int TMEM_COLS = (128 + HV) <= 256 ? 256 : 512;
 };
 
-template <int H, bool PAGED>
+template <int H, int HV, bool PAGED>
 __global__ void __launch_bounds__(160, 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                 const __grid_constant__ CUtensorMap tmV, const AttnArgs a) {
-  using C_ = FwdCfg<H>;
+  using C_ = FwdCfg<H, HV>;
+  constexpr int NV = C_::NV;
   extern __shared__ uint8_t smem_raw[];
   const uint32_t sbase = (smem_u32(smem_raw) + 1023u) & ~1023u;
   uint8_t* sptr = smem_raw + (sbase - smem_u32(smem_raw));
@@ -145,21 +157,22 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     // ------------------------------------------------------------ issuer warp
     if (nblk > 0 && elect_one()) {
       const uint32_t idesc_s = make_idesc_bf16(BQ, BKV, 0, 0);
-      const uint32_t idesc_o = make_idesc_bf16(BQ, H, 0, 1);
+      const uint32_t idesc_o = make_idesc_bf16(BQ, HV, 0, 1);
       auto load_k = [&](int j) {
-        mbar_expect_tx(barK, C_::KV_BYTES);
+        mbar_expect_tx(barK, C_::K_BYTES);
         const int row = block_row(j);
 #pragma unroll
         for (int c = 0; c < C_::HS; ++c)
           tma_load_2d(sK + c * (BKV * 128), &tmK, barK, kvh * H + 64 * c, row);
       };
       auto load_v = [&](int j) {
-        const uint32_t bar = barV0 + 8 * (j & 1);
-        mbar_expect_tx(bar, C_::KV_BYTES);
+        const int buf = j % NV;
+        const uint32_t bar = barV0 + 8 * buf;
+        mbar_expect_tx(bar, C_::V_BYTES);
         const int row = block_row(j);
 #pragma unroll
-        for (int c = 0; c < C_::HS; ++c)
-          tma_load_2d(sV + (j & 1) * C_::KV_BYTES + c * (BKV * 128), &tmV, bar, kvh * H + 64 * c, row);
+        for (int c = 0; c < C_::HVS; ++c)
+          tma_load_2d(sV + buf * C_::V_BYTES + c * (BKV * 128), &tmV, bar, kvh * HV + 64 * c, row);
       };
       auto issue_s = [&](int j) {
         const uint32_t d = tmem + C_::TMEM_S + (j & 1) * BKV;
@@ -175,7 +188,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       mbar_expect_tx(barQ, C_::Q_BYTES);
 #pragma unroll
       for (int c = 0; c < C_::HS; ++c)
-        tma_load_2d(sQ + c * (BQ * 128), &tmQ, barQ, n * H + 64 * c, row0);
+        tma_load_2d(sQ + c * (BQ * 128), &tmQ, barQ, n * (PAGED ? a.q_heads : H) + 64 * c, row0);
       load_k(0);
       load_v(0);
       ok = ok && mbar_wait_bounded(barQ, 0, abort_flag, a.status, ST_TIMEOUT_PRODUCER);
@@ -193,13 +206,20 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           tc_fence_after();
           issue_s(j + 1);
           // V buffer (j+1)&1 was last read by PV_{j-1}
-          if (j >= 1 && !mbar_wait_bounded(barPV, (j - 1) & 1, abort_flag, a.status, ST_TIMEOUT_MMA)) { ok = false; break; }
-          load_v(j + 1);
+          if (NV == 2) {
+            if (j >= 1 && !mbar_wait_bounded(barPV, (j - 1) & 1, abort_flag, a.status, ST_TIMEOUT_MMA)) { ok = false; break; }
+            load_v(j + 1);
+          }
+        }
+        // the only V buffer was last read by PV_{j-1}
+        if (NV == 1 && j >= 1) {
+          if (!mbar_wait_bounded(barPV, (j - 1) & 1, abort_flag, a.status, ST_TIMEOUT_MMA)) { ok = false; break; }
+          load_v(j);
         }
         if (!mbar_wait_bounded(barP, j & 1, abort_flag, a.status, ST_TIMEOUT_MMA)) { ok = false; break; }
-        if (!mbar_wait_bounded(barV0 + 8 * (j & 1), (j >> 1) & 1, abort_flag, a.status, ST_TIMEOUT_PRODUCER)) { ok = false; break; }
+        if (!mbar_wait_bounded(barV0 + 8 * (j % NV), (j / NV) & 1, abort_flag, a.status, ST_TIMEOUT_PRODUCER)) { ok = false; break; }
         tc_fence_after();
-        const uint32_t vb = sV + (j & 1) * C_::KV_BYTES;
+        const uint32_t vb = sV + (j % NV) * C_::V_BYTES;
 #pragma unroll
         for (int kk = 0; kk < BKV / 16; ++kk) {
           const uint64_t ad = make_smem_desc(sP + kk * 32, 16, 1024);
@@ -318,7 +338,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         tc_fence_after();
         if (warp_need) {
 #pragma unroll 1
-          for (int c = 0; c < H / 16; ++c) {
+          for (int c = 0; c < HV / 16; ++c) {
             uint32_t o[16];
             tmem_ld_32x16(tmem + lane_addr + C_::TMEM_O + c * 16, o);
             tmem_ld_wait();
@@ -344,11 +364,15 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     if (ok && nblk > 0)
       ok = mbar_wait_bounded(barPV, (nblk - 1) & 1, abort_flag, a.status, ST_TIMEOUT_EPILOGUE);
     tc_fence_after();
-    const int vd = PAGED ? a.vd : H;
-    const float inv_l = PAGED ? a.out_scale / (l + exp2f(a.sink2 - m_used)) : (l > 0.f) ? 1.f / l : 0.f;
+    const int vd = PAGED ? a.vd : HV;
+    float inv_l = (l > 0.f) ? 1.f / l : 0.f;
+    if (PAGED) {
+      inv_l = a.out_scale / (l + exp2f((a.sinks ? a.sinks[n] * LOG2E : a.sink2) - m_used));
+      if (a.gate && row_valid) inv_l /= 1.f + exp2f(-LOG2E * __bfloat162float(a.gate[(long long)(row0 + r) * a.ldg + n]));
+    }
     __nv_bfloat16* orow = a.O + (long long)(row0 + r) * a.ldo + (long long)n * vd;
 #pragma unroll 1
-    for (int c = 0; c < H / 32; ++c) {
+    for (int c = 0; c < HV / 32; ++c) {
       uint32_t o[32];
       if (nblk > 0 && ok) {
         tmem_ld_32x32(tmem + lane_addr + C_::TMEM_O + c * 32, o);
@@ -388,17 +412,17 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
 template <int H>
 int launch_fwd(const void* q, const void* k, const void* v, const AttnArgs& a, long long ldq,
                long long ldk, long long ldv, cudaStream_t stream) {
-  using C_ = FwdCfg<H>;
+  using C_ = FwdCfg<H, H>;
   CUtensorMap tq, tk, tv;
   if (tb_make_tmap_2d_bf16(&tq, q, (uint64_t)a.B * a.Tq, (uint64_t)a.N * H, ldq, BQ, 64, 1)) return -3;
   if (tb_make_tmap_2d_bf16(&tk, k, (uint64_t)a.B * a.Tk, (uint64_t)a.KH * H, ldk, BKV, 64, 1)) return -3;
   if (tb_make_tmap_2d_bf16(&tv, v, (uint64_t)a.B * a.Tk, (uint64_t)a.KH * H, ldv, BKV, 64, 1)) return -3;
   static DeviceOnce once;
   if (once.first() &&
-      cudaFuncSetAttribute(attn_fwd_kernel<H, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, C_::SMEM_BYTES) != cudaSuccess)
+      cudaFuncSetAttribute(attn_fwd_kernel<H, H, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, C_::SMEM_BYTES) != cudaSuccess)
     return -5;
   dim3 grid((a.Tq + BQ - 1) / BQ, a.N, a.B);
-  attn_fwd_kernel<H, false><<<grid, 160, C_::SMEM_BYTES, stream>>>(tq, tk, tv, a);
+  attn_fwd_kernel<H, H, false><<<grid, 160, C_::SMEM_BYTES, stream>>>(tq, tk, tv, a);
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
 }
 
@@ -827,47 +851,57 @@ TB_API int tb_attn_fwd(const void* q, const void* k, const void* v, void* o, flo
   }
 }
 
-template <int H>
-static int launch_fwd_paged(const void* q, const void* k, const void* v, const AttnArgs& a, long long rows, long long pool_rows,
-                            int tiles, cudaStream_t stream) {
-  using C_ = FwdCfg<H>;
+template <int H, int HV>
+static int launch_fwd_paged(const void* q, long long ldq, int q_cols, const void* k, long long ldk, const void* v, long long ldv, const AttnArgs& a,
+                            long long rows, long long pool_rows, int tiles, cudaStream_t stream) {
+  using C_ = FwdCfg<H, HV>;
   CUtensorMap tq, tk, tv;
-  const uint64_t qc = (uint64_t)a.N * H, kc = (uint64_t)a.KH * H;
-  if (tb_make_tmap_2d_bf16(&tq, q, (uint64_t)rows, qc, qc, BQ, 64, 1) || tb_make_tmap_2d_bf16(&tk, k, (uint64_t)pool_rows, kc, kc, BKV, 64, 1) ||
-      tb_make_tmap_2d_bf16(&tv, v, (uint64_t)pool_rows, kc, kc, BKV, 64, 1))
+  // heads that lie closer than H columns: the columns behind a head meet the zeros behind the stored key
+  if (tb_make_tmap_2d_bf16(&tq, q, (uint64_t)rows, (uint64_t)q_cols, (uint64_t)ldq, BQ, 64, 1) ||
+      tb_make_tmap_2d_bf16(&tk, k, (uint64_t)pool_rows, (uint64_t)a.KH * H, (uint64_t)ldk, BKV, 64, 1) ||
+      tb_make_tmap_2d_bf16(&tv, v, (uint64_t)pool_rows, (uint64_t)a.KH * HV, (uint64_t)ldv, BKV, 64, 1))
     return -3;
   static DeviceOnce once;
   if (once.first() &&
-      cudaFuncSetAttribute(attn_fwd_kernel<H, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, C_::SMEM_BYTES) != cudaSuccess)
+      cudaFuncSetAttribute(attn_fwd_kernel<H, HV, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, C_::SMEM_BYTES) != cudaSuccess)
     return -5;
-  attn_fwd_kernel<H, true><<<dim3(tiles, a.N), 160, C_::SMEM_BYTES, stream>>>(tq, tk, tv, a);
+  attn_fwd_kernel<H, HV, true><<<dim3(tiles, a.N), 160, C_::SMEM_BYTES, stream>>>(tq, tk, tv, a);
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
 }
 
 // Causal attention of the query tiles (at most 128 rows of one entry each) of a ragged batch over paged keys and values:
-// q / out [n, N * H]; pools [pool_rows, KH * H] with page_size a multiple of 64; a key block of 64 tokens lies in one page
-// and is fetched by TMA through the page table. window, chunk <= 0: none; softcap <= 0: none. The unused tail of a page must hold finite values.
-// sink: one more score without a value in the sum of the weights (-inf: none). out [n, ldo], 16-byte aligned, head h at columns
-// h * vd (the first vd <= H value columns, a multiple of 8), times out_scale.
-TB_API int tb_attn_fwd_paged(const void* q, const void* k_pool, const void* v_pool, void* out, long long ldo, int n, long long pool_rows, int N,
-                             int KH, int H, int vd, float scale, float softcap, int window, int chunk, int keep, float sink,
-                             float out_scale, const float* bias, int far, const int* cu,
+// q_cols columns of q [n, ldq] with heads q_heads apart (a multiple of 8; queries may be narrower than H if the keys have zeros behind their own
+// columns); pools of pool_rows rows, ldk / ldv apart, of KH heads of H / HV, with page_size a multiple of 64; a key block of 64
+// tokens lies in one page and is fetched by TMA through the page table. window, chunk <= 0: none; softcap <= 0: none. The unused
+// tail of a page must hold finite values. sink: one more score without a value in the sum of the weights (-inf: none), or sinks
+// fp32 [N], one per head. gate bf16, rows ldg apart, or null: head h's output is multiplied by sigmoid(gate[row, h]). out [n, ldo],
+// 16-byte aligned, head h at columns h * vd (the first vd <= HV value columns, a multiple of 8), times out_scale.
+// (H, HV): (64, 64), (128, 64), (128, 128), (192, 128), (256, 256).
+TB_API int tb_attn_fwd_paged(const void* q, long long ldq, int q_cols, int q_heads, const void* k_pool, long long ldk, const void* v_pool,
+                             long long ldv, void* out, long long ldo, int n, long long pool_rows, int N, int KH, int H, int HV, int vd,
+                             float scale, float softcap, int window, int chunk, int keep, float sink, const float* sinks,
+                             const void* gate, long long ldg, float out_scale, const float* bias, int far, const int* cu,
                              const int* slot, const int* pos0, const int* tile_t0, const int* tile_ent, int tiles,
                              const int* table, int max_pages, int page_size, int* status, cudaStream_t stream) {
   if (n <= 0 || tiles <= 0) return 0;
-  if (KH <= 0 || N % KH || page_size % BKV || N > 65535 || vd <= 0 || vd > H || vd % 8 || ldo % 8 || ((uintptr_t)out & 15)) return -2;
+  if (KH <= 0 || N % KH || page_size % BKV || N > 65535 || vd <= 0 || vd > HV || vd % 8 || ldo % 8 || ((uintptr_t)out & 15)) return -2;
+  if (q_heads % 8 || ldq % 8 || ldk % 8 || ldv % 8 || ((uintptr_t)q & 15) || ((uintptr_t)k_pool & 15) || ((uintptr_t)v_pool & 15)) return -2;
   AttnArgs a = {};
-  a.vd = vd; a.sink2 = sink * LOG2E; a.out_scale = out_scale;
+  a.vd = vd; a.sink2 = sink * LOG2E; a.sinks = sinks; a.out_scale = out_scale;
+  a.gate = reinterpret_cast<const __nv_bfloat16*>(gate); a.ldg = ldg; a.q_heads = q_heads;
   a.N = N; a.KH = KH; a.scale = scale; a.causal = 1; a.window = window > 0 ? window : 0;
   a.softcap = softcap; a.chunk = chunk > 0 ? chunk : 0;
   a.keep = a.window > 0 || a.chunk > 0 ? keep : 0; a.bias = bias; a.far = far;
   a.O = reinterpret_cast<__nv_bfloat16*>(out); a.ldo = ldo; a.status = status;
   a.cu = cu; a.slot = slot; a.pos0 = pos0; a.tile_t0 = tile_t0; a.tile_ent = tile_ent; a.table = table;
   a.max_pages = max_pages; a.page_size = page_size;
-  switch (H) {
-    case 64: return launch_fwd_paged<64>(q, k_pool, v_pool, a, n, pool_rows, tiles, stream);
-    case 128: return launch_fwd_paged<128>(q, k_pool, v_pool, a, n, pool_rows, tiles, stream);
-    case 256: return launch_fwd_paged<256>(q, k_pool, v_pool, a, n, pool_rows, tiles, stream);
-    default: return -2;
-  }
+#define PAIR(K, V) \
+  if (H == K && HV == V) return launch_fwd_paged<K, V>(q, ldq, q_cols, k_pool, ldk, v_pool, ldv, a, n, pool_rows, tiles, stream)
+  PAIR(64, 64);
+  PAIR(128, 64);
+  PAIR(128, 128);
+  PAIR(192, 128);
+  PAIR(256, 256);
+#undef PAIR
+  return -2;
 }

@@ -12,13 +12,15 @@
 //                    max / sum per query head, partial results of the splits merged by `paged_decode_combine`.
 //                    Sliding window (optionally with kept first tokens), chunks of positions, a bias per (distance, head)
 //                    added to the scores, and logit soft-cap supported; with a window or chunks only the tiles that hold
-//                    visible keys are walked and split over CTAs. Memory-bound by construction: every K / V
+//                    visible keys are walked and split over CTAs; a sink in the sum of the weights, the same or a learned
+//                    one per head, and a gate per head on the output. Memory-bound by construction: every K / V
 //                    byte of the sequence is read exactly once per kv head.
 //
 // The reference keeps only host-side page-table logic (tunix/experimental/generate/*) and runs decode on a
 // dense cache through XLA (tunix/generate/sampler.py:732-793); these kernels are the device side of the
 // in-framework engine that replaces its vLLM / SGLang integrations.
 #include "mma.cuh"
+#include "decode_splits.cuh"
 
 using namespace tb;
 
@@ -111,8 +113,6 @@ qkv_post_kernel(__nv_bfloat16* __restrict__ qkv, long long ld, const int* __rest
 
 // ---- tensor-core fragments (warp-level mma.sync of mma.cuh: with at most 16 query rows per kv head there is no 64/128-row
 // tile to give to tcgen05, and the kernel is bound by the K/V stream, not by math) --------------------------------
-constexpr int TILE_KEYS = 64;   // keys staged per pipeline stage; 16 per warp
-
 // byte offset of 16-byte chunk c of row r in a [rows, H] bf16 tile whose 128-byte groups are XOR-swizzled by row
 template <int H>
 __device__ __forceinline__ uint32_t swz(int r, int c) {
@@ -127,19 +127,6 @@ __device__ __forceinline__ uint32_t tile_off(int r, int c) {
   return swz<H>(r, c);
 }
 
-// The key tiles a single query at position len - 1 walks: the tiles that hold kept first tokens, then those of the window.
-struct KeyTiles {
-  int w_lo, first, n_sink, total;
-  __device__ __forceinline__ KeyTiles(int len, int window, int chunk, int keep) {
-    w_lo = window > 0 ? max(0, len - window) : 0;
-    if (chunk > 0 && len > 0) w_lo = max(w_lo, len - 1 - (len - 1) % chunk);
-    first = w_lo / TILE_KEYS;
-    n_sink = min((min(keep, len) + TILE_KEYS - 1) / TILE_KEYS, first);
-    total = n_sink + (len + TILE_KEYS - 1) / TILE_KEYS - first;
-  }
-  __device__ __forceinline__ int start(int tile) const { return (tile < n_sink ? tile : first + tile - n_sink) * TILE_KEYS; }
-};
-
 // One CTA per (sequence, kv head, context split): the G (<= 16) query heads of the kv head are the 16 rows of the
 // A operand, a warp owns 16 keys of each 64-key stage, S = Q K^T and O += P V run on mma.sync and read K / V with
 // ldmatrix; every K / V byte is read once. Staging: with pages of a multiple of 64 tokens a tile lies in one page
@@ -149,11 +136,11 @@ struct KeyTiles {
 template <int H, bool TMA, int STAGES>
 __global__ void __launch_bounds__(128)
 paged_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
-                    const __nv_bfloat16* __restrict__ q, long long ldq,        // [B, N*H]
+                    const __nv_bfloat16* __restrict__ q, long long ldq,        // [B, ldq], heads q_heads apart
                     const __nv_bfloat16* __restrict__ k_pool, const __nv_bfloat16* __restrict__ v_pool,
                     const int* __restrict__ page_table, int max_pages, int page_size,
                     const int* __restrict__ seq_ids, const int* __restrict__ seq_lens, int KH, int G, float scale,
-                    float softcap, int window, int chunk, int keep, float sink, float out_scale, int vd,
+                    float softcap, int window, int chunk, int keep, float out_scale, int vd, const HeadExtras ex, int q_heads,
                     const float* __restrict__ bias, int far,                   // bias [N, far + 1] or null
                     int num_splits, int split_tokens,
                     float* __restrict__ part_acc,                                               // [B, N, splits, H]
@@ -193,7 +180,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_consta
   for (int idx = tid; idx < 16 * CPR; idx += 128) {
     const int r = idx / CPR, c = idx - r * CPR;
     uint4 u = make_uint4(0, 0, 0, 0);
-    if (r < G) u = *reinterpret_cast<const uint4*>(q + (long long)b * ldq + (long long)(kh * G + r) * H + c * 8);
+    if (r < G) u = *reinterpret_cast<const uint4*>(q + (long long)b * ldq + (long long)(kh * G + r) * q_heads + c * 8);
     *reinterpret_cast<uint4*>(q_s + swz<H>(r, c)) = u;
   }
 
@@ -369,8 +356,9 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_consta
       aa += sm_acc[(w * 16 + g) * H + d] * c;
     }
     if (num_splits == 1) {                 // the whole context in this CTA: no partial state, no combine kernel
-      ll += __expf(sink - mm);
-      out[(long long)b * ldo + (long long)(kh * G + g) * vd + d] = __float2bfloat16(ll > 0.f ? out_scale * aa / ll : 0.f);
+      ll += __expf(ex.sink_of(kh * G + g) - mm);
+      out[(long long)b * ldo + (long long)(kh * G + g) * vd + d] =
+          __float2bfloat16(ll > 0.f ? out_scale * ex.gate_of(b, kh * G + g) * aa / ll : 0.f);
       continue;
     }
     const long long oidx = (((long long)b * N + kh * G + g) * num_splits + split);
@@ -382,42 +370,12 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_consta
   }
 }
 
-// out[b, n, :vd] = out_scale * sum_s acc_s * exp(m_s - M) / (exp(sink - M) + sum_s l_s * exp(m_s - M))
-__global__ void paged_decode_combine_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
-                                            const int* __restrict__ seq_lens, int N, int H, int num_splits, int split_tokens,
-                                            int window, int chunk, int keep, float sink, float out_scale, int vd,
-                                            __nv_bfloat16* __restrict__ out, long long ldo) {
-  pdl_trigger();
-  pdl_wait();
-  const int b = blockIdx.x, n = blockIdx.y;
-  const int len = seq_lens[b];
-  const int tps = split_tokens / TILE_KEYS;
-  const int used = len > 0 ? min(num_splits, (KeyTiles(len, window, chunk, keep).total + tps - 1) / tps) : 0;
-  const long long base = ((long long)b * N + n) * num_splits;
-  float M = -INFINITY;
-  for (int s = 0; s < used; ++s) M = fmaxf(M, part_ml[(base + s) * 2]);
-  float L = used > 0 ? __expf(sink - M) : 0.f;
-  for (int s = 0; s < used; ++s) {
-    const float ms = part_ml[(base + s) * 2];
-    if (ms != -INFINITY) L += part_ml[(base + s) * 2 + 1] * __expf(ms - M);
-  }
-  const float inv = L > 0.f ? out_scale / L : 0.f;
-  for (int d = threadIdx.x; d < vd; d += blockDim.x) {
-    float a = 0.f;
-    for (int s = 0; s < used; ++s) {
-      const float ms = part_ml[(base + s) * 2];
-      if (ms != -INFINITY) a += part_acc[(base + s) * H + d] * __expf(ms - M);
-    }
-    out[(long long)b * ldo + (long long)n * vd + d] = __float2bfloat16(a * inv);
-  }
-}
-
 template <int H, bool TMA, int STAGES>
 int launch_decode_v(int G, dim3 grid, cudaStream_t stream, const CUtensorMap& tmK, const CUtensorMap& tmV,
                     const __nv_bfloat16* q, long long ldq, const __nv_bfloat16* kp, const __nv_bfloat16* vp, const int* pt,
                     int max_pages, int page_size, const int* seq_ids, const int* seq_lens, int KH, float scale, float softcap,
-                    int window, int chunk, int keep, float sink, float out_scale, int vd, const float* bias, int far, int splits, int split_tokens, float* pa, float* pml,
-                    __nv_bfloat16* out, long long ldo, int* status) {
+                    int window, int chunk, int keep, float out_scale, int vd, HeadExtras ex, int q_heads, const float* bias, int far, int splits,
+                    int split_tokens, float* pa, float* pml, __nv_bfloat16* out, long long ldo, int* status) {
   constexpr int TILE2 = 2 * TILE_KEYS * H * 2;                       // one stage: a K tile and a V tile
   constexpr int SMEM = STAGES * TILE2 + (TMA ? 1024 : 0);
   static DeviceOnce once;
@@ -427,7 +385,7 @@ int launch_decode_v(int G, dim3 grid, cudaStream_t stream, const CUtensorMap& tm
   // a split of one 64-key tile needs one stage only: more CTAs fit on an SM
   const int smem = split_tokens > TILE_KEYS ? SMEM : TILE2 + (TMA ? 1024 : 0);
   return launch_pdl(paged_decode_kernel<H, TMA, STAGES>, grid, dim3(128), smem, stream, tmK, tmV, q, ldq, kp, vp, pt, max_pages,
-                    page_size, seq_ids, seq_lens, KH, G, scale, softcap, window, chunk, keep, sink, out_scale, vd, bias, far, splits, split_tokens, pa, pml, out, ldo,
+                    page_size, seq_ids, seq_lens, KH, G, scale, softcap, window, chunk, keep, out_scale, vd, ex, q_heads, bias, far, splits, split_tokens, pa, pml, out, ldo,
                     status) == cudaSuccess ? 0 : -5;
 }
 
@@ -436,9 +394,8 @@ template <int H>
 int launch_decode(int G, dim3 grid, cudaStream_t stream, const __nv_bfloat16* q, long long ldq,
                   const __nv_bfloat16* kp, const __nv_bfloat16* vp, long long pool_rows, const int* pt, int max_pages,
                   int page_size, const int* seq_ids, const int* seq_lens, int KH, float scale, float softcap, int window,
-                  int chunk, int keep, float sink, float out_scale, int vd, const float* bias, int far, int splits, int split_tokens, float* pa,
-                  float* pml, __nv_bfloat16* out,
-                  long long ldo, int* status) {
+                  int chunk, int keep, float out_scale, int vd, HeadExtras ex, int q_heads, const float* bias, int far, int splits,
+                  int split_tokens, float* pa, float* pml, __nv_bfloat16* out, long long ldo, int* status) {
   static const bool no_tma = getenv("TUNIX_B200_DECODE_NO_TMA") != nullptr;
   static const char* stages_env = getenv("TUNIX_B200_DECODE_STAGES");
   CUtensorMap tmK, tmV;
@@ -448,7 +405,7 @@ int launch_decode(int G, dim3 grid, cudaStream_t stream, const __nv_bfloat16* q,
                    tb_make_tmap_2d_bf16(&tmK, kp, (uint64_t)pool_rows, (uint64_t)KH * H, (uint64_t)KH * H, TILE_KEYS, 64, 1) == 0 &&
                    tb_make_tmap_2d_bf16(&tmV, vp, (uint64_t)pool_rows, (uint64_t)KH * H, (uint64_t)KH * H, TILE_KEYS, 64, 1) == 0;
 #define LD(T, S) launch_decode_v<H, T, S>(G, grid, stream, tmK, tmV, q, ldq, kp, vp, pt, max_pages, page_size, seq_ids, seq_lens, \
-                                         KH, scale, softcap, window, chunk, keep, sink, out_scale, vd, bias, far, splits, split_tokens, pa, pml, out, ldo, status)
+                                         KH, scale, softcap, window, chunk, keep, out_scale, vd, ex, q_heads, bias, far, splits, split_tokens, pa, pml, out, ldo, status)
   if (!tma) return LD(false, 2);
   // measured at head dim 128 (8 kv heads, 256 sequences x 768 tokens): 2 / 3 / 4 stages take 157 / 161 / 194 us,
   // cp.async staging 190 us: three CTAs per SM with two stages each beat deeper rings on fewer CTAs
@@ -499,20 +456,22 @@ TB_API int tb_qkv_post(void* qkv, long long ld, const int* seq_ids, const int* p
   return err == cudaSuccess ? 0 : -5;
 }
 
-// q [B, N*H]; pools [num_pages, page_size, KH*H]; page_table [*, max_pages]; seq_ids [B]; seq_lens [B];
+// q [B, ldq], heads q_heads apart (each read H wide); pools [num_pages, page_size, KH*H]; page_table [*, max_pages]; seq_ids [B]; seq_lens [B];
 // workspace: part_acc fp32 [B*N*splits*H], part_ml fp32 [B*N*splits*2] with splits = ceil(max_ctx / split_tokens);
 // split_tokens = context tokens per CTA, a multiple of 64 in [64, 2048] (0 = 256). CTAs of splits that lie past the
 // end of their sequence return at once. pool_rows = num_pages * page_size (rows of the pools, for the tensor maps;
 // 0 = no TMA staging). window > 0: keys at distance < window, chunk > 0: keys of the query's chunk, and the sequence's first `keep` tokens. bias fp32
 // [N, far + 1] (null = none) is added to the scaled score of a key at distance min(distance, far). sink: one more score without a
-// value in the sum of the weights (-inf: none). out [B, ldo]: head n at columns n * vd, its first vd <= H value columns, times out_scale. status: word that a bounded mbarrier wait writes its code to.
-TB_API int tb_paged_decode(const void* q, long long ldq, const void* k_pool, const void* v_pool,
+// value in the sum of the weights (-inf: none), or sinks fp32 [N], one per head. gate bf16, rows ldg apart, or null: head n's
+// output is multiplied by sigmoid(gate[row, n]). out [B, ldo]: head n at columns n * vd, its first vd <= H value columns, times out_scale. status: word that a bounded mbarrier wait writes its code to.
+TB_API int tb_paged_decode(const void* q, long long ldq, int q_heads, const void* k_pool, const void* v_pool,
                            const int* page_table, int max_pages, int page_size, const int* seq_ids,
                            const int* seq_lens, int B, int N, int KH, int H, int max_ctx, float scale, float softcap,
-                           int window, int chunk, int keep, float sink, float out_scale, int vd, const float* bias, int far,
-                           int split_tokens, long long pool_rows, float* part_acc, float* part_ml, void* out, long long ldo, int* status, cudaStream_t stream) {
+                           int window, int chunk, int keep, float sink, const float* sinks, const void* gate, long long ldg, float out_scale,
+                           int vd, const float* bias, int far, int split_tokens, long long pool_rows, float* part_acc, float* part_ml, void* out, long long ldo, int* status, cudaStream_t stream) {
   if (B <= 0) return 0;
-  if (KH <= 0 || N % KH || (ldq % 8) || vd <= 0 || vd > H) return -2;
+  if (KH <= 0 || N % KH || (ldq % 8) || (q_heads % 8) || vd <= 0 || vd > H) return -2;
+  const HeadExtras ex{sink, sinks, (const __nv_bfloat16*)gate, ldg};
   const int G = N / KH;
   if (G > MAX_G) return -2;
   if (split_tokens <= 0) split_tokens = 256;
@@ -530,15 +489,15 @@ TB_API int tb_paged_decode(const void* q, long long ldq, const void* k_pool, con
   auto kp = (const __nv_bfloat16*)k_pool;
   auto vp = (const __nv_bfloat16*)v_pool;
   switch (H) {
-    case 64: rc = launch_decode<64>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, chunk, keep, sink, out_scale, vd, bias, far, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
-    case 128: rc = launch_decode<128>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, chunk, keep, sink, out_scale, vd, bias, far, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
-    case 256: rc = launch_decode<256>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, chunk, keep, sink, out_scale, vd, bias, far, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
+    case 64: rc = launch_decode<64>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, chunk, keep, out_scale, vd, ex, q_heads, bias, far, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
+    case 128: rc = launch_decode<128>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, chunk, keep, out_scale, vd, ex, q_heads, bias, far, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
+    case 256: rc = launch_decode<256>(G, grid, stream, qq, ldq, kp, vp, pool_rows, page_table, max_pages, page_size, seq_ids, seq_lens, KH, scale, softcap, window, chunk, keep, out_scale, vd, ex, q_heads, bias, far, splits, split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, ldo, status); break;
     default: return -2;
   }
   if (rc) return rc;
   if (splits == 1) return 0;
   return launch_pdl(paged_decode_combine_kernel, dim3(B, N), dim3(128), 0, stream, (const float*)part_acc,
-                    (const float*)part_ml, seq_lens, N, H, splits, split_tokens, window, chunk, keep, sink, out_scale, vd, (__nv_bfloat16*)out, ldo) == cudaSuccess ? 0 : -5;
+                    (const float*)part_ml, seq_lens, N, H, splits, split_tokens, window, chunk, keep, out_scale, vd, ex, (__nv_bfloat16*)out, ldo) == cudaSuccess ? 0 : -5;
 }
 
 // ------------------------------------------------------------------ per-step bookkeeping of the decode loop

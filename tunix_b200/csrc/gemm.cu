@@ -643,7 +643,11 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
               float o[8];
 #pragma unroll
               for (int j = 0; j < 8; ++j) {
-                const float gt = v[16 * g + j], up = v[16 * g + 8 + j];
+                float gt = v[16 * g + j], up = v[16 * g + 8 + j];
+                if (has_bias) {                                   // stored as the weight's rows: gates, then ups
+                  gt += __bfloat162float(args.bias[(col0 >> 1) + 8 * g + j]);
+                  up += __bfloat162float(args.bias[(args.N >> 1) + (col0 >> 1) + 8 * g + j]);
+                }
                 float act;
                 if (glu_kind == 1) {
                   act = gt / (1.f + __expf(-gt));
@@ -1085,8 +1089,8 @@ TB_API int tb_gemm_packed_bf16(const void* A, long long lda, const void* P, int 
       w < 16 || w > 256 || (w % 16) || (flags & (GF_A_MN | GF_B_MN)))
     return -2;
   const bool glu = flags & (GF_GLU_SILU | GF_GLU_GELU);
-  // gated epilogue: bf16 output of N / 2 columns, nothing else in the epilogue, 16-byte aligned rows
-  if (glu && ((flags & (GF_OUT_F32 | GF_ACCUM | GF_BIAS | GF_RESIDUAL)) || (N % 16) || (ldc % 8) ||
+  // gated epilogue: bf16 output of N / 2 columns, a bias [gates | ups] at most, 16-byte aligned rows
+  if (glu && ((flags & (GF_OUT_F32 | GF_ACCUM | GF_RESIDUAL)) || (N % 16) || (ldc % 8) ||
               (reinterpret_cast<uintptr_t>(C) & 15) || alpha != 1.0f))
     return -2;
   if ((flags & GF_XIELU) && ((flags & (GF_ACCUM | GF_BIAS | GF_RESIDUAL)) || glu || bias == nullptr)) return -2;

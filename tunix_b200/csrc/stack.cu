@@ -11,11 +11,12 @@
 //                 successor but the final norm. A launch between two passes of a loop can add the embedding rows again,
 //                 after the sum of the streams is reported. Norms may run over equal groups of a row. Without a norm
 //                 the row itself is written in the activation type. In a decode step the launch can also mix the new
-//                 row with the one before it (token shift).
-//   token_shift : the same mixes for portions of prompts.
+//                 row with the one before it (token shift). The embedding may add a row of a table of token pairs; its
+//                 sum can be written out for a product that reads it again.
+//   token_shift, keep_last : the same mixes for portions of prompts, and the rows that the next portions start from.
 //   few_outputs, small_act : products with a handful of outputs, and what is applied to them (tanh; gelu times a row
 //                 that belongs to the token).
-//   xielu       : the activation of feed-forwards without a gate.
+//   xielu, glu  : the activations of feed-forwards without and with a gate.
 //
 // This file is compiled without fast-math: the same kernels serve the 32-bit mode.
 #include "mma.cuh"
@@ -46,13 +47,21 @@ struct StreamArgs {
   float embed_scale;          // factor of the (normed) embedding rows
   const void* pos;            // T [positions, D] or null: a row per position, added to the embedding rows
   int positions;
-  const int *cu, *ent;        // the batch's entries, with pos0 below (read with pos only)
+  const void* pairs;          // T [buckets + 1, D] or null: a row per pair of a token and the one before it, added as well;
+  long long buckets, mul_prev, mul_cur;     //     row (before * mul_prev + token * mul_cur) mod buckets, the last row for a first token
+  const long long* last;      // [slots] the token before an entry's first one
+  void* start;                // T, rows ld_start apart, or null: the embedding rows as they are added
+  long long ld_start;
+  const int *cu, *ent;        // the batch's entries, with slot and pos0 below (read with pos, pairs, keep)
   int groups;                 // equal parts of a row that the norms of embedding and streams are taken over
   // the sublayer that follows
   const void* in;             // T [S]; null = all ones (the sum of the streams)
   const void* w;              // T [D] norm weight
-  void* h;                    // T [n, D]
+  void* h;                    // T, rows ldh apart
+  long long ldh;
   float* sum_out;             // fp32 [n, D] or null: the sum of the streams
+  long long* keep;            // [slots] or null: receives the last token of every entry, from ids [n]
+  const long long* ids;
   // token shift of a batch of single tokens (row = entry): mixes T [n_mix, n, D] instead of h
   const void* mu;             // T [n_mix, D] or null
   int n_mix;
@@ -132,7 +141,11 @@ __global__ void __launch_bounds__(512) stream_step_kernel(const StreamArgs a) {
     r1 = 0.5f / sqrtf(s1 / (float)D + a.eps);
     r2 = 0.5f / sqrtf(s2 / (float)D + a.eps);
   }
-  const T *emb = nullptr, *pos = nullptr;
+  const T *emb = nullptr, *pos = nullptr, *pair = nullptr;
+  if (a.keep && threadIdx.x == 0) {
+    const int e = a.ent[row];
+    if (row + 1 == a.cu[e + 1] && a.pos0[e] >= 0) a.keep[a.slot[e]] = a.ids[row];
+  }
   if (a.tokens) {
     if (a.pos) {
       const int e = a.ent[row], p = a.pos0[e] + (int)row - a.cu[e];
@@ -141,6 +154,18 @@ __global__ void __launch_bounds__(512) stream_step_kernel(const StreamArgs a) {
     long long t = a.tokens[row];
     t = t < 0 ? 0 : (t >= a.vocab ? a.vocab - 1 : t);
     emb = static_cast<const T*>(a.embed) + t * D;
+    if (a.pairs) {
+      const int e = a.ent[row], p0 = a.pos0[e];
+      const bool inside = row > a.cu[e];
+      long long b = a.buckets;
+      if (inside || p0 > 0) {
+        long long before = inside ? a.tokens[row - 1] : a.last[a.slot[e]];
+        before = before < 0 ? 0 : (before >= a.vocab ? a.vocab - 1 : before);
+        b = (before * a.mul_prev + t * a.mul_cur) % a.buckets;
+        if (b < 0) b += a.buckets;
+      }
+      pair = static_cast<const T*>(a.pairs) + b * D;
+    }
     if (a.embed_w) {
       for (int d = threadIdx.x * V; d < D; d += step) {
         float ev[V];
@@ -169,6 +194,13 @@ __global__ void __launch_bounds__(512) stream_step_kernel(const StreamArgs a) {
 #pragma unroll
         for (int i = 0; i < V; ++i) ev[i] += pv[i];
       }
+      if (pair) {
+        float pv[V];
+        load_v<V>(pair + d, pv);
+#pragma unroll
+        for (int i = 0; i < V; ++i) ev[i] += pv[i];
+      }
+      if (a.start) store_v<V>(static_cast<T*>(a.start) + row * a.ld_start + d, ev);
     }
     if (emb && !y) {
 #pragma unroll
@@ -241,7 +273,7 @@ __global__ void __launch_bounds__(512) stream_step_kernel(const StreamArgs a) {
   }
   if (!a.h && !a.mu) return;
   if (!a.w) {                                            // the row itself
-    T* h = static_cast<T*>(a.h) + row * D;
+    T* h = static_cast<T*>(a.h) + row * a.ldh;
     for (int d = threadIdx.x * V; d < D; d += step) {
       float u[V];
       load_v<V>(u_s + d, u);
@@ -255,7 +287,7 @@ __global__ void __launch_bounds__(512) stream_step_kernel(const StreamArgs a) {
   } else {
     r = 1.f / sqrtf(block_sum(ss, red) / (float)D + a.eps);
   }
-  T* h = a.h ? static_cast<T*>(a.h) + row * D : nullptr;
+  T* h = a.h ? static_cast<T*>(a.h) + row * a.ldh : nullptr;
   const int p0 = a.mu ? a.pos0[row] : 0;
   float* before = a.mu ? a.before + (long long)a.slot[row] * D : nullptr;
   for (int d = threadIdx.x * V; d < D; d += step) {      // each thread reads back what it wrote
@@ -295,7 +327,7 @@ __global__ void __launch_bounds__(512) stream_step_kernel(const StreamArgs a) {
 
 template <typename T, int S>
 cudaError_t launch_stream_step(const StreamArgs& a, int n, cudaStream_t stream) {
-  const bool vec = a.D % 4 == 0;
+  const bool vec = a.D % 4 == 0 && (!a.h || a.ldh % 4 == 0) && (!a.start || a.ld_start % 4 == 0);
   const int per = vec ? a.D / 4 : a.D;
   int threads = n <= 296 ? 512 : 256;              // few rows: the latency of one row counts
   while (threads > 128 && threads / 2 >= per) threads /= 2;
@@ -321,9 +353,9 @@ int dispatch_stream_step(const StreamArgs& a, int S, int n, cudaStream_t stream)
   return err == cudaSuccess ? 0 : -5;
 }
 
-// h[r, f] = silu(gu[r, f]) * gu[r, F + f] for any F
+// h[r, f] = act(gu[r, f]) * gu[r, F + f] for any F; act: 0 silu, 1 gelu (tanh form)
 template <typename T>
-__global__ void silu_mul_kernel(const T* __restrict__ gu, T* __restrict__ h, long long rows, int F) {
+__global__ void glu_kernel(int kind, const T* __restrict__ gu, T* __restrict__ h, long long ldh, long long rows, int F) {
   pdl_trigger();
   pdl_wait();
   const long long total = rows * F;
@@ -331,7 +363,7 @@ __global__ void silu_mul_kernel(const T* __restrict__ gu, T* __restrict__ h, lon
     const long long r = i / F;
     const int f = (int)(i - r * F);
     const float g = to_f(gu[r * 2 * F + f]), u = to_f(gu[r * 2 * F + F + f]);
-    h[i] = from_f<T>(g * sigmoid(g) * u);
+    h[r * ldh + f] = from_f<T>((kind == 0 ? g * sigmoid(g) : gelu_tanh(g)) * u);
   }
 }
 
@@ -515,20 +547,34 @@ token_shift_kernel(const T* __restrict__ h, const T* __restrict__ mu, const floa
   }
 }
 
+// carry[slot[e]] = the last row of entry e of h (fp32 copies)
+template <typename T>
+__global__ void __launch_bounds__(256) keep_last_kernel(const T* __restrict__ h, float* __restrict__ carry, Ragged rb, int D) {
+  pdl_trigger();
+  pdl_wait();
+  const int e = blockIdx.y, d = blockIdx.x * blockDim.x + threadIdx.x;
+  if (d < D && rb.pos0[e] >= 0) carry[(long long)rb.slot[e] * D + d] = to_f(h[(long long)(rb.cu[e + 1] - 1) * D + d]);
+}
+
 }  // namespace
 
 // dtype: 0 = bf16, 1 = float (activations and weights). x fp32 [n, S, D]; see StreamArgs.
 TB_API int tb_stream_step(int dtype, float* x, int n, int S, int D, float eps, const void* y, const void* y2, const void* wy,
                           const void* wy2, const void* mix, const void* out, const long long* tokens, const void* embed,
                           int vocab, const void* embed_w, float embed_scale, const void* pos, int positions, int groups,
-                          const void* in, const void* w, void* h, float* sum_out, const void* mu, int n_mix, float* before,
-                          void* mixes, const int* cu, const int* slot, const int* pos0, const int* ent, cudaStream_t stream) {
+                          const void* in, const void* w, void* h, long long ldh, float* sum_out, const void* mu, int n_mix, float* before,
+                          void* mixes, const void* pairs, long long buckets, long long mul_prev, long long mul_cur,
+                          const long long* last, void* start, long long ld_start, long long* keep, const long long* ids,
+                          const int* cu, const int* slot, const int* pos0, const int* ent, cudaStream_t stream) {
   if (n <= 0) return 0;
   if (S < 1 || S > MAX_STREAMS || D <= 0 || D > 11000 || (y2 && !y)) return -2;
   if (pos && (!tokens || positions <= 0 || !cu || !pos0 || !ent)) return -2;
   if (groups < 1 || groups > 256 || D % groups || (mu && (!w || !before || !mixes))) return -2;
-  StreamArgs a{x, D, eps, y, y2, wy, wy2, mix, out, tokens, embed, vocab, embed_w, embed_scale, pos, positions, cu, ent,
-               groups, in, w, h, sum_out, mu, n_mix, before, mixes, slot, pos0};
+  if (pairs && (!tokens || buckets <= 0 || !last || !cu || !slot || !pos0 || !ent)) return -2;
+  if (keep && (!ids || !cu || !slot || !pos0 || !ent)) return -2;
+  StreamArgs a{x, D, eps, y, y2, wy, wy2, mix, out, tokens, embed, vocab, embed_w, embed_scale, pos, positions, pairs, buckets,
+               mul_prev, mul_cur, last, start, ld_start, cu, ent, groups, in, w, h, ldh, sum_out, keep, ids, mu, n_mix, before,
+               mixes, slot, pos0};
   return dtype == 0 ? dispatch_stream_step<__nv_bfloat16>(a, S, n, stream) : dispatch_stream_step<float>(a, S, n, stream);
 }
 
@@ -542,8 +588,22 @@ TB_API int tb_token_shift(int dtype, const void* h, const void* mu, int n_mix, c
 #define TS(T, V, NM)                                                                                                        \
   launch_pdl(token_shift_kernel<T, V, NM>, dim3((D / V + 127) / 128, (n + ST - 1) / ST), dim3(128), 0, stream, (const T*)h,  \
              (const T*)mu, carry, rb, D, n_mix, (T*)mixes)
-  cudaError_t err = dtype != 0 ? TS(float, 1, 8) : D % 4 ? TS(bf, 1, 8) : n_mix <= 5 ? TS(bf, 4, 5) : TS(bf, 4, 8);
+  cudaError_t err = dtype != 0 ? TS(float, 1, 8)
+                    : n_mix == 1 && D % 8 == 0 ? TS(bf, 8, 1)
+                    : D % 4 ? TS(bf, 1, 8) : n_mix <= 5 ? TS(bf, 4, 5) : TS(bf, 4, 8);
 #undef TS
+  return err == cudaSuccess ? 0 : -5;
+}
+
+// h T [n, D] contiguous -> carry fp32 [slots, D]: the last row of every entry
+TB_API int tb_keep_last(int dtype, const void* h, float* carry, const int* cu, const int* slot, const int* pos0, const int* ent, int E,
+                        int n, int D, cudaStream_t stream) {
+  if (n <= 0 || E <= 0) return 0;
+  if (E > 65535) return -2;
+  Ragged rb{cu, slot, pos0, ent, E, n};
+  const dim3 grid((D + 255) / 256, E);
+  const cudaError_t err = dtype == 0 ? launch_pdl(keep_last_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, (const __nv_bfloat16*)h, carry, rb, D)
+                                     : launch_pdl(keep_last_kernel<float>, grid, dim3(256), 0, stream, (const float*)h, carry, rb, D);
   return err == cudaSuccess ? 0 : -5;
 }
 
@@ -574,13 +634,14 @@ TB_API int tb_small_act(int dtype, const float* z, int n, int N, int act, const 
   return err == cudaSuccess ? 0 : -5;
 }
 
-TB_API int tb_silu_mul(int dtype, const void* gu, void* h, long long rows, int F, cudaStream_t stream) {
+// gu T [rows, 2 F] (gates, then ups) -> h T [rows, F], rows ldh apart; kind as in glu_kernel
+TB_API int tb_glu(int dtype, int kind, const void* gu, void* h, long long ldh, long long rows, int F, cudaStream_t stream) {
   if (rows <= 0 || F <= 0) return 0;
   const long long want = (rows * F + 255) / 256;
   const dim3 grid((unsigned)(want < 148 * 16 ? want : 148 * 16));
   cudaError_t err = dtype == 0
-      ? launch_pdl(silu_mul_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)h, rows, F)
-      : launch_pdl(silu_mul_kernel<float>, grid, dim3(256), 0, stream, (const float*)gu, (float*)h, rows, F);
+      ? launch_pdl(glu_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, kind, (const __nv_bfloat16*)gu, (__nv_bfloat16*)h, ldh, rows, F)
+      : launch_pdl(glu_kernel<float>, grid, dim3(256), 0, stream, kind, (const float*)gu, (float*)h, ldh, rows, F);
   return err == cudaSuccess ? 0 : -5;
 }
 

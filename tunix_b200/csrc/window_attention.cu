@@ -8,12 +8,13 @@
 //                   (and weighted, if the model has weights), then its first `rd` dimensions turn by the angles of the
 //                   token's position, element i together with i + rd / 2, or (interleaved) 2 i together with 2 i + 1. Heads
 //                   can be stored wider than they are, with zeros behind them, so that the tensor-core kernels fit them. A
-//                   layer that reads another layer's cache has queries only.
+//                   layer that reads another layer's cache has queries only. Which heads are normed (queries and keys,
+//                   values) is the caller's choice; without query heads only keys and values are written.
 //   window_attn   : any head sizes, bf16 or float: one warp per (token, query head), lanes over keys for the scores and
 //                   over value columns for the output, online softmax in fp32. Position i sees j <= i with
 //                   (i - j < window and j in i's chunk) or j < keep. A sink is one more score, without a value, in the sum
-//                   of the weights (-inf: none). Models whose heads fit the tensor-core kernels (attention_fwd.cu,
-//                   decode.cu) use those instead.
+//                   of the weights (-inf: none), the same or a learned one per head. A head's output may have a gate of
+//                   its own. Models whose heads fit the tensor-core kernels (attention_fwd.cu, decode.cu) use those instead.
 //
 // This file is compiled without fast-math: the same kernels serve the 32-bit mode.
 #include "precise.cuh"
@@ -82,14 +83,16 @@ qk_norm_write_kernel(const T* __restrict__ proj, long long ldp, int q_off, int k
   }
 }
 
+constexpr int NORM_QK = 1, NORM_V = 2;     // which heads are divided by their root mean square
+
 // Heads of a multiple of 8 dimensions that turn by a multiple of 16 (8 if interleaved): LPH lanes per head, 8 elements per lane;
 // the partner of a rotation sits rd / 16 lanes away, or in the same lane. Otherwise like rope_norm_write_kernel.
 template <int LPH, bool INTER>
 __global__ void __launch_bounds__(256)
 rope_norm_write_vec_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp, int q_off, int k_off, int v_off,
                            const __nv_bfloat16* __restrict__ qw, const __nv_bfloat16* __restrict__ kw, const float* __restrict__ cos_t,
-                           const float* __restrict__ sin_t, int rd, float eps, Ragged rb, Paged pg, int H, int G, int dq, int dv,
-                           int wq, int wv, __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ kp,
+                           const float* __restrict__ sin_t, int rd, float eps, int norms, Ragged rb, Paged pg, int H, int G, int dq,
+                           int dv, int wq, int wv, __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ kp,
                            __nv_bfloat16* __restrict__ vp) {
   pdl_trigger();
   pdl_wait();
@@ -136,10 +139,10 @@ rope_norm_write_vec_kernel(const __nv_bfloat16* __restrict__ proj, long long ldp
     for (int i = 0; i < 8; ++i) ss += v[i] * v[i];
 #pragma unroll
     for (int w = LPH / 2; w >= 1; w >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, w);
-    if (!is_v) {
-      const float r = 1.f / sqrtf(ss / (float)dq + eps);
+    if (norms & (is_v ? NORM_V : NORM_QK)) {
+      const float r = 1.f / sqrtf(ss / (float)(is_v ? dv : dq) + eps);
 #pragma unroll
-      for (int i = 0; i < 8; ++i) v[i] *= r * (hh < H ? wa[i] : wb[i]);
+      for (int i = 0; i < 8; ++i) v[i] *= is_v ? r : r * (hh < H ? wa[i] : wb[i]);
     }
 #pragma unroll
     for (int i = 0; i < 8; ++i)
@@ -158,7 +161,7 @@ template <typename T>
 __global__ void __launch_bounds__(256)
 rope_norm_write_kernel(const T* __restrict__ proj, long long ldp, int q_off, int k_off, int v_off, const T* __restrict__ qw,
                        const T* __restrict__ kw, const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rd, int inter,
-                       float eps, Ragged rb, Paged pg, int H, int G, int dq, int dv, int wq, int wv, T* __restrict__ q,
+                       float eps, int norms, Ragged rb, Paged pg, int H, int G, int dq, int dv, int wq, int wv, T* __restrict__ q,
                        T* __restrict__ kp, T* __restrict__ vp) {
   pdl_trigger();
   pdl_wait();
@@ -179,7 +182,13 @@ rope_norm_write_kernel(const T* __restrict__ proj, long long ldp, int q_off, int
   if (hh >= H) pr = page_row(pg, pg.table + (long long)rb.slot[e] * pg.max_pages, p);
   if (hh >= H + G) {
     const int g = hh - H - G;
-    for (int c = lane; c < wv; c += 32) vp[(pr * G + g) * wv + c] = c < dv ? row[v_off + g * dv + c] : from_f<T>(0.f);
+    const T* src = row + v_off + g * dv;
+    float ss = 0.f, r = 1.f;
+    if (norms & NORM_V) {
+      for (int c = lane; c < dv; c += 32) { const float x = to_f(src[c]); ss += x * x; }
+      r = 1.f / sqrtf(warp_sum(ss) / (float)dv + eps);
+    }
+    for (int c = lane; c < wv; c += 32) vp[(pr * G + g) * wv + c] = from_f<T>(c < dv ? to_f(src[c]) * r : 0.f);
     return;
   }
   const T* src = row + (hh < H ? q_off + hh * dq : k_off + (hh - H) * dq);
@@ -189,7 +198,7 @@ rope_norm_write_kernel(const T* __restrict__ proj, long long ldp, int q_off, int
   const float *ct = cos_t + (long long)p * half, *st = sin_t + (long long)p * half;
   float ss = 0.f;
   for (int c = lane; c < dq; c += 32) { const float x = to_f(src[c]); ss += x * x; }
-  const float r = 1.f / sqrtf(warp_sum(ss) / (float)dq + eps);
+  const float r = norms & NORM_QK ? 1.f / sqrtf(warp_sum(ss) / (float)dq + eps) : 1.f;
   auto normed = [&](int c) { return to_f(src[c]) * r * (w ? to_f(w[c]) : 1.f); };
   for (int c = lane; c < wq; c += 32) {
     float x = 0.f;
@@ -205,13 +214,14 @@ rope_norm_write_kernel(const T* __restrict__ proj, long long ldp, int q_off, int
   }
 }
 
-constexpr int VREG = 16;        // value columns per lane: value heads up to 512 wide
+constexpr int VREG = 16;        // value columns per lane: wider value heads are cut over blockIdx.y
 
 template <typename T>
 __global__ void __launch_bounds__(128)
-window_attn_kernel(const T* __restrict__ q, const T* __restrict__ kp, const T* __restrict__ vp, Ragged rb, Paged pg, int H,
-                   int G, int dq, int dv, int wq, int wv, float scale, float cap, const float* __restrict__ bias, int far, int window,
-                   int chunk, int keep, float sink, float out_scale, T* __restrict__ out, long long ldo) {
+window_attn_kernel(const T* __restrict__ q, long long ldq, int qs_heads, const T* __restrict__ kp, const T* __restrict__ vp, Ragged rb,
+                   Paged pg, int H, int G, int dq, int dv, int wq, int wv, float scale, float cap, const float* __restrict__ bias, int far,
+                   int window, int chunk, int keep, float sink, const float* __restrict__ sinks, const T* __restrict__ gate,
+                   long long ldg, float out_scale, T* __restrict__ out, long long ldo) {
   extern __shared__ float qs_all[];               // [4][dq]
   pdl_trigger();
   pdl_wait();
@@ -221,12 +231,13 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ kp, const T* _
   const int t = (int)(wid / H), h = (int)(wid - (long long)t * H), g = h / (H / G);
   const int e = rb.ent[t], p0 = rb.pos0[e];
   T* o = out + (long long)t * ldo + (long long)h * dv;
+  const int c0 = blockIdx.y * VREG * 32;          // first value column of this block
   if (p0 < 0) {
-    for (int c = lane; c < dv; c += 32) o[c] = from_f<T>(0.f);
+    for (int c = c0 + lane; c < min(dv, c0 + VREG * 32); c += 32) o[c] = from_f<T>(0.f);
     return;
   }
   float* qs = qs_all + warp * dq;
-  for (int d = lane; d < dq; d += 32) qs[d] = to_f(q[((long long)t * H + h) * wq + d]) * scale;
+  for (int d = lane; d < dq; d += 32) qs[d] = to_f(q[(long long)t * ldq + (long long)h * qs_heads + d]) * scale;
   __syncwarp();
   const int i = p0 + t - rb.cu[e];
   const int lo = first_visible(i, window, chunk);
@@ -263,15 +274,15 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ kp, const T* _
       const T* v = vp + (ry * G + g) * wv;
 #pragma unroll
       for (int r = 0; r < VREG; ++r) {
-        const int cc = r * 32 + lane;
+        const int cc = c0 + r * 32 + lane;
         if (cc < dv) acc[r] += py * to_f(v[cc]);
       }
     }
   }
-  const float inv = out_scale / (l + expf(sink - m));
+  const float inv = out_scale * (gate ? sigmoid(to_f(gate[(long long)t * ldg + h])) : 1.f) / (l + expf((sinks ? sinks[h] : sink) - m));
 #pragma unroll
   for (int r = 0; r < VREG; ++r) {
-    const int cc = r * 32 + lane;
+    const int cc = c0 + r * 32 + lane;
     if (cc < dv) o[cc] = from_f<T>(acc[r] * inv);
   }
 }
@@ -299,15 +310,16 @@ TB_API int tb_qk_norm_write(int dtype, const void* proj, long long ldp, int q_of
 }
 
 // q | k | v: columns of proj [n, ldp]; H query heads of dq, G key / value heads (0: queries only) of dq / dv; qw, kw T [dq] or
-// null: weights of the heads' norms; rd rotated dimensions (inter: neighbours turn together) with tables cos / sin fp32
-// [positions, rd / 2]. Heads are stored wq / wv wide: q [n, H * wq]; pools [pages, page_size, G * wq] and [.., G * wv].
+// null: weights of the heads' norms; norms: bit 0 query and key heads, bit 1 value heads; rd rotated dimensions (inter: neighbours turn together) with tables cos / sin fp32
+// [positions, rd / 2]. Heads are stored wq / wv wide: q [n, H * wq] (H 0: keys and values only); pools [pages, page_size, G * wq]
+// and [.., G * wv].
 TB_API int tb_rope_norm_write(int dtype, const void* proj, long long ldp, int q_off, int k_off, int v_off, const void* qw,
-                              const void* kw, const float* cos_t, const float* sin_t, int rd, int inter, float eps, const int* cu,
+                              const void* kw, const float* cos_t, const float* sin_t, int rd, int inter, float eps, int norms, const int* cu,
                               const int* slot, const int* pos0, const int* ent, int E, int n, const int* table, int max_pages,
                               int page_size, int H, int G, int dq, int dv, int wq, int wv, void* q, void* kp, void* vp,
                               cudaStream_t stream) {
   if (n <= 0) return 0;
-  if (rd < 0 || rd % 2 || rd > dq || wq < dq || wv < dv) return -2;
+  if (rd < 0 || rd % 2 || rd > dq || wq < dq || wv < dv || (rd > 0 && (!cos_t || !sin_t))) return -2;
   RAGGED;
   PAGED;
   const int wide = wq > wv ? wq : wv;
@@ -316,7 +328,7 @@ TB_API int tb_rope_norm_write(int dtype, const void* proj, long long ldp, int q_
     typedef __nv_bfloat16 bf;
 #define VEC(L, I)                                                                                                           \
   launch_pdl(rope_norm_write_vec_kernel<L, I>, dim3(n), dim3(256), 0, stream, (const bf*)proj, ldp, q_off, k_off, v_off,     \
-             (const bf*)qw, (const bf*)kw, cos_t, sin_t, rd, eps, rb, pg, H, G, dq, dv, wq, wv, (bf*)q, (bf*)kp, (bf*)vp)
+             (const bf*)qw, (const bf*)kw, cos_t, sin_t, rd, eps, norms, rb, pg, H, G, dq, dv, wq, wv, (bf*)q, (bf*)kp, (bf*)vp)
     const cudaError_t err = inter ? (wide <= 64 ? VEC(8, true) : wide <= 128 ? VEC(16, true) : VEC(32, true))
                                   : (wide <= 64 ? VEC(8, false) : wide <= 128 ? VEC(16, false) : VEC(32, false));
     return err == cudaSuccess ? 0 : -5;
@@ -326,28 +338,31 @@ TB_API int tb_rope_norm_write(int dtype, const void* proj, long long ldp, int q_
   const dim3 grid((unsigned)((warps + 7) / 8));
 #define RUN(T)                                                                                                              \
   launch_pdl(rope_norm_write_kernel<T>, grid, dim3(256), 0, stream, (const T*)proj, ldp, q_off, k_off, v_off, (const T*)qw,  \
-             (const T*)kw, cos_t, sin_t, rd, inter, eps, rb, pg, H, G, dq, dv, wq, wv, (T*)q, (T*)kp, (T*)vp)
+             (const T*)kw, cos_t, sin_t, rd, inter, eps, norms, rb, pg, H, G, dq, dv, wq, wv, (T*)q, (T*)kp, (T*)vp)
   return (dtype == 0 ? RUN(__nv_bfloat16) : RUN(float)) == cudaSuccess ? 0 : -5;
 #undef RUN
 }
 
 // bias fp32 [H, far + 1] or null: what is added to the score of a key at distance min(i - j, far). window, chunk <= 0: none;
-// cap > 0: scores become cap * tanh(score / cap). sink: one more score without a value in the sum of the weights (-inf: none).
-// Heads are stored wq / wv wide; out T [n, ldo], head h at columns h * dv, times out_scale.
-TB_API int tb_window_attn(int dtype, const void* q, const void* kp, const void* vp, const int* cu, const int* slot,
+// cap > 0: scores become cap * tanh(score / cap). sink: one more score without a value in the sum of the weights (-inf: none), or
+// sinks fp32 [H], one per head. gate T, rows ldg apart, or null: head h's output is multiplied by sigmoid(gate[row, h]).
+// q T, rows ldq and heads q_heads apart. Cached heads are stored wq / wv wide; out T [n, ldo], head h at columns h * dv, times
+// out_scale.
+TB_API int tb_window_attn(int dtype, const void* q, long long ldq, int q_heads, const void* kp, const void* vp, const int* cu, const int* slot,
                           const int* pos0, const int* ent, int E, int n, const int* table, int max_pages, int page_size, int H,
                           int G, int dq, int dv, int wq, int wv, float scale, float cap, const float* bias, int far, int window,
-                          int chunk, int keep, float sink, float out_scale, void* out, long long ldo, cudaStream_t stream) {
+                          int chunk, int keep, float sink, const float* sinks, const void* gate, long long ldg, float out_scale, void* out,
+                          long long ldo, cudaStream_t stream) {
   if (n <= 0) return 0;
-  if (G <= 0 || H % G || dv > VREG * 32 || dq > 3000) return -2;
+  if (G <= 0 || H % G || dv <= 0 || dq > 3000) return -2;
   RAGGED;
   PAGED;
   const long long warps = (long long)n * H;
-  const dim3 grid((unsigned)((warps + 3) / 4));
+  const dim3 grid((unsigned)((warps + 3) / 4), (dv + VREG * 32 - 1) / (VREG * 32));
 #define RUN(T)                                                                                                              \
-  return launch_pdl(window_attn_kernel<T>, grid, dim3(128), (size_t)4 * dq * 4, stream, (const T*)q, (const T*)kp,           \
-                    (const T*)vp, rb, pg, H, G, dq, dv, wq, wv, scale, cap, bias, far, window, chunk, keep, sink, out_scale, \
-                    (T*)out, ldo) == cudaSuccess ? 0 : -5
+  return launch_pdl(window_attn_kernel<T>, grid, dim3(128), (size_t)4 * dq * 4, stream, (const T*)q, ldq, q_heads, (const T*)kp, \
+                    (const T*)vp, rb, pg, H, G, dq, dv, wq, wv, scale, cap, bias, far, window, chunk, keep, sink, sinks,     \
+                    (const T*)gate, ldg, out_scale, (T*)out, ldo) == cudaSuccess ? 0 : -5
   if (dtype == 0) RUN(__nv_bfloat16);
   RUN(float);
 #undef RUN

@@ -38,17 +38,18 @@ from .sampler import next_power_of_2, pad_prompts_left
 
 
 class SlotStates:
-    """Recurrent state of every layer pass: fp32 tensors with one row per slot. A kernel that runs a sequence's first
+    """Recurrent state of every layer pass: fp32 tensors with one row per slot, and token ids per slot. A kernel that runs a sequence's first
     token starts from zero whatever the slot held before, so a slot needs no clearing when its owner changes."""
 
-    def __init__(self, shapes: Sequence[dict], max_seqs: int, device):
+    def __init__(self, shapes: Sequence[dict], max_seqs: int, device, tokens: Sequence[str] = ()):
         self.tensors = [{k: torch.zeros((max_seqs, *s), dtype=torch.float32, device=device) for k, s in d.items()} for d in shapes]
+        self.tokens = {k: torch.zeros(max_seqs, dtype=torch.int64, device=device) for k in tokens}     # token ids, one per slot
 
     def __getitem__(self, layer_pass: int) -> dict:
         return self.tensors[layer_pass]
 
     def nbytes_per_slot(self) -> int:
-        return sum(t[0].numel() * 4 for d in self.tensors for t in d.values())
+        return sum(t[0].numel() * 4 for d in self.tensors for t in d.values()) + 8 * len(self.tokens)
 
 
 class PagePool:
@@ -65,14 +66,15 @@ class PagePool:
         from ..experimental.generate import kv_cache_manager as kvm
         self.page_size, self.num_pages, self.max_pages = page_size, num_pages, max_pages_per_seq
         if hasattr(cfg, "kv_rows"):                # layer-stack models: rows and states per layer pass
-            rows, self.state = cfg.kv_rows(dtype), SlotStates(cfg.state_shapes(), max_seqs, device)
+            rows = cfg.kv_rows(dtype)
+            self.state = SlotStates(cfg.state_shapes(), max_seqs, device, cfg.token_states())
         else:
             row = (kv_heads or cfg.num_kv_heads) * cfg.head_dim   # a tensor-parallel rank keeps its own kv heads only
             rows, self.state = [(row, row)] * cfg.num_layers, None
         # zero-initialised: rows of a page that were never written must hold finite values
         pages = lambda n: torch.zeros(num_pages, page_size, n, dtype=dtype, device=device)  # noqa: E731
         self.k = [None if r is None else pages(r[0]) for r in rows]
-        self.v = [None if r is None else pages(r[1]) for r in rows]
+        self.v = [None if r is None or not r[1] else pages(r[1]) for r in rows]      # latents serve as keys and values
         self.table_host = np.full((max_seqs, max_pages_per_seq), -1, np.int32)
         self.table = torch.full((max_seqs, max_pages_per_seq), -1, dtype=torch.int32, device=device)
         self.Error = kvm.PagePoolError

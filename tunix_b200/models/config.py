@@ -287,7 +287,7 @@ def get_config(name: str) -> ModelConfig:
         for n in ("gemma4_e2b", "gemma4_e4b", "gemma4_12b", "gemma4_31b", "gemma4_26b_a4b"):
             PRESETS[n] = getattr(Gemma4Config, n)
             PRESETS[n + "_it"] = getattr(Gemma4Config, n)
-    if key.startswith(("roluzen", "tovalix", "zikezen")) and key not in PRESETS:
+    if key.startswith(("roluzen", "tovalix", "zikezen", "zigipel")) and key not in PRESETS:
         from .stack import STACK_FAMILIES, StackConfig
         for n in (f"{fam}_{size}" for fam in STACK_FAMILIES for size in ("tiny", "2b", "8b")):
             PRESETS[n] = getattr(StackConfig, n)

@@ -20,6 +20,10 @@ sizes and constants in a spec, its parameters in a module and its per-sequence c
   GatedLinearAttention    matrix memory with a decay per key channel, a root of a sigmoid behind a bottleneck; per-head norm
                           and silu output gate
   SumMixer                rotary attention and gated linear attention on the same input, each times a constant, summed
+  DistanceAttention       grouped-query attention without rotation: a logarithm of the distance is taken off the scores, value
+                          heads are normed, sliding window with kept first tokens, per head a learned sink and an output gate
+  LatentAttention         heads of keys and values made from one normed latent per token (which is what is cached), plus one
+                          rotated key part that all heads share; sliding window, per head a learned sink
 
 A spec's `kv_rows(dtype)` names the paged cache rows a pass through the layer needs (key columns, value columns), or None
 (also for attention that reads another layer's, `kv_from`); `state_shapes()` the fp32 state it keeps per sequence slot. Heads
@@ -29,7 +33,7 @@ from __future__ import annotations
 
 import math
 from dataclasses import dataclass
-from typing import ClassVar, Optional
+from typing import ClassVar, NamedTuple, Optional
 
 import torch
 import torch.nn as nn
@@ -38,7 +42,31 @@ from .transformer import Linear, RMSNorm
 
 MEMORY_SLICE = 32       # value columns a CTA of the matrix-memory kernels owns (csrc/recurrent.cu: MV)
 TILE_HEADS = (64, 128, 256)     # head sizes of the tensor-core attention kernels
+TILE_PAIRS = ((64, 64), (128, 64), (128, 128), (192, 128), (256, 256))    # (key, value) head sizes of the one for portions
 NO_SINK = -math.inf
+LATENT_RANK, LATENT_WIDTH = 512, 640    # widest latent, and latent with its rotated part, of the tensor-core decode kernel
+
+
+def fitted_heads(dim: int, vdim: int, dtype) -> tuple:
+    """Widths that heads are stored at: as wide as the tensor-core kernels want them, zeros behind them, where that is bf16 and
+    at most twice the size."""
+    wide = max(dim, vdim)
+    fit = next((w for w in TILE_HEADS if w >= wide), 0)
+    return (fit, fit) if dtype == torch.bfloat16 and 0 < fit <= 2 * wide and vdim % 8 == 0 else (dim, vdim)
+
+
+class YarnScaling(NamedTuple):
+    """Rotary frequencies for longer contexts: pairs that turn more than `fast` times over the original context keep theirs,
+    those that turn fewer than `slow` times have it divided by the factor, and the pairs between change over linearly; turned
+    vectors grow by `size`."""
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+    @property
+    def size(self) -> float:
+        return 0.1 * math.log(self.factor) + 1.0
 
 
 # ---------------------------------------------------------------------------------------------------- specs
@@ -129,11 +157,7 @@ class RotaryAttentionSpec:
     keep_first: ClassVar[int] = 0
 
     def stored(self, dtype):
-        wide = max(self.dim, self.vdim)
-        fit = next((w for w in TILE_HEADS if w >= wide), 0)
-        if self.fit_heads and dtype == torch.bfloat16 and fit <= 2 * wide and fit and self.vdim % 8 == 0:
-            return fit, fit
-        return self.dim, self.vdim
+        return fitted_heads(self.dim, self.vdim, dtype) if self.fit_heads else (self.dim, self.vdim)
 
     def kv_rows(self, dtype):
         if self.kv_from is not None:
@@ -199,6 +223,73 @@ class SumSpec:
 
     def state_shapes(self) -> dict:
         return self.right.state_shapes()
+
+
+@dataclass(frozen=True)
+class DistanceAttentionSpec:
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    window: int                  # 0 = unlimited
+    keep_first: int = 0          # leading tokens of the sequence that stay visible
+    chunk: ClassVar[int] = 0
+    softcap: ClassVar[float] = 0.0
+    sink: ClassVar[float] = NO_SINK         # the learned ones take its place
+
+    def stored(self, dtype):
+        return fitted_heads(self.dim, self.vdim, dtype)
+
+    def kv_rows(self, dtype):
+        k, v = self.stored(dtype)
+        return self.kv_heads * k, self.kv_heads * v
+
+    def state_shapes(self) -> dict:
+        return {}
+
+
+@dataclass(frozen=True)
+class LatentAttentionSpec:
+    heads: int
+    dim: int                     # unrotated query / key dimensions of a head
+    rot_dim: int                 # rotated ones; their key part is shared by all heads
+    vdim: int
+    kv_rank: int                 # size of the latent
+    scale: float
+    window: int                  # 0 = unlimited
+    rot_dims: int                # leading dimensions of the rotated part that turn
+    rot_base: float
+    rot_scaling: Optional[tuple] = None     # see stack_exec.rope_frequencies
+    kv_heads: ClassVar[int] = 1             # one row of latents serves every head
+    chunk: ClassVar[int] = 0
+    softcap: ClassVar[float] = 0.0
+    sink: ClassVar[float] = NO_SINK
+    keep_first: ClassVar[int] = 0
+
+    @property
+    def width(self) -> int:
+        return self.kv_rank + self.rot_dim
+
+    def tiled(self, dtype) -> bool:
+        """Whether the tensor-core kernels take these sizes."""
+        return dtype == torch.bfloat16 and not any(n % 8 for n in (self.kv_rank, self.dim, self.rot_dim, self.vdim)) and \
+            self.kv_rank <= LATENT_RANK and self.width <= LATENT_WIDTH and self.tile_heads() is not None
+
+    def tile_heads(self) -> Optional[tuple]:
+        """Widths of the key and value heads that portions of prompts expand the latents to."""
+        return next((p for p in TILE_PAIRS if p[0] >= self.dim + self.rot_dim and p[1] >= self.vdim), None)
+
+    def stored(self, dtype):
+        """Width of a cached row as key and as value: the latent, the rotated part, and zeros up to a multiple of 64."""
+        w = -(-self.width // 64) * 64 if self.tiled(dtype) else self.width
+        return w, w
+
+    def kv_rows(self, dtype):
+        return self.stored(dtype)[0], 0
+
+    def state_shapes(self) -> dict:
+        return {}
 
 
 # ------------------------------------------------------------------------------------------------- bias table
@@ -418,7 +509,71 @@ class SumMixer(nn.Module):
         return [self.left.fused_groups()[0] + self.right.fused_groups()[0]]
 
 
-MIXERS = {RGLRUSpec: RGLRUMixer, ParallelSpec: ParallelMixer, RotaryAttentionSpec: RotaryAttention,
+class DistanceAttention(nn.Module):
+    def __init__(self, spec: DistanceAttentionSpec, width: int, eps: float, dtype, device=None):
+        super().__init__()
+        if spec.heads % spec.kv_heads:
+            raise ValueError(f"{spec.heads} query heads over {spec.kv_heads} key / value heads")
+        self.spec, self.eps = spec, eps
+        H, G = spec.heads, spec.kv_heads
+        self.q_proj = Linear(width, H * spec.dim, False, dtype, device)
+        self.k_proj = Linear(width, G * spec.dim, False, dtype, device)
+        self.v_proj = Linear(width, G * spec.vdim, False, dtype, device)
+        self.g_proj = Linear(width, H, False, dtype, device)
+        self.o_proj = Linear(H * spec.vdim, width, False, dtype, device)
+        self.r1 = _param(H, dtype=dtype, device=device, fill=1.0)
+        self.r2 = _param(H, dtype=dtype, device=device, fill=1.0)
+        self.sink = _param(H, dtype=dtype, device=device)
+
+    def bias_table(self, positions: int) -> torch.Tensor:
+        """fp32 [heads, positions]: what is added to the score of a key at every distance, -r1 ln(1 + r2 distance)."""
+        r1, r2 = (r.detach().double()[:, None] for r in (self.r1, self.r2))
+        gap = torch.arange(positions, dtype=torch.float64, device=r1.device)
+        return (-r1 * torch.log1p(r2 * gap)).float()
+
+    def init_special(self) -> None:
+        self.r1.fill_(1.0)
+        self.r2.fill_(1.0)
+
+    def fused_groups(self) -> list:
+        return [[self.q_proj, self.k_proj, self.v_proj, self.g_proj]]
+
+
+class LatentAttention(nn.Module):
+    def __init__(self, spec: LatentAttentionSpec, width: int, eps: float, dtype, device=None):
+        super().__init__()
+        if spec.rot_dims % 2 or spec.rot_dims > spec.rot_dim:
+            raise ValueError(f"{spec.rot_dims} rotated dimensions of {spec.rot_dim}")
+        self.spec, self.eps = spec, eps
+        H = spec.heads
+        self.q_proj = Linear(width, H * (spec.dim + spec.rot_dim), False, dtype, device)
+        self.dkv_proj = Linear(width, spec.width, False, dtype, device)
+        self.kv_norm = RMSNorm(spec.kv_rank, eps, False, dtype, device)
+        self.uk_proj = Linear(spec.kv_rank, H * spec.dim, False, dtype, device)
+        self.uv_proj = Linear(spec.kv_rank, H * spec.vdim, False, dtype, device)
+        self.o_proj = Linear(H * spec.vdim, width, False, dtype, device)
+        self.sink = _param(H, dtype=dtype, device=device)
+
+    @torch.no_grad()
+    def expansion(self, stored: int, wide: int, wide_v: int) -> torch.Tensor:
+        """[heads * (wide + wide_v), stored]: takes a cached row to the heads' keys (made from the latent, then the shared rotated
+        part, then zeros) and behind all of them to their values."""
+        sp, H = self.spec, self.spec.heads
+        w = self.uk_proj.weight.new_zeros(H * (wide + wide_v), stored)
+        k, v = w[:H * wide].view(H, wide, stored), w[H * wide:].view(H, wide_v, stored)
+        k[:, :sp.dim, :sp.kv_rank] = self.uk_proj.weight.view(H, sp.dim, sp.kv_rank)
+        k[:, sp.dim:sp.dim + sp.rot_dim, sp.kv_rank:sp.width] = torch.eye(sp.rot_dim, dtype=w.dtype, device=w.device)
+        v[:, :sp.vdim, :sp.kv_rank] = self.uv_proj.weight.view(H, sp.vdim, sp.kv_rank)
+        return w
+
+    def init_special(self) -> None:
+        pass
+
+    def fused_groups(self) -> list:
+        return [[self.q_proj, self.dkv_proj]]
+
+
+MIXERS = {DistanceAttentionSpec: DistanceAttention, LatentAttentionSpec: LatentAttention, RGLRUSpec: RGLRUMixer, ParallelSpec: ParallelMixer, RotaryAttentionSpec: RotaryAttention,
           TokenShiftMemorySpec: TokenShiftMemory, ForgetGateMemorySpec: ForgetGateMemory, GatedLinearSpec: GatedLinearAttention,
           SumSpec: SumMixer}
 

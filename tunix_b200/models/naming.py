@@ -9,7 +9,7 @@ from .config import PRESETS, ModelConfig, get_config
 _FAMILY_PATTERNS = [
     (r"llama[-_]?3", "llama3"), (r"qwen[-_]?3", "qwen3"), (r"qwen[-_]?2", "qwen2"), (r"deepseek[-_]?r1[-_]?distill[-_]?qwen", "qwen2"),
     (r"gemma[-_]?4", "gemma4"), (r"gemma[-_]?3", "gemma3"), (r"gemma[-_]?2", "gemma2"), (r"gemma", "gemma"), (r"roluzen", "roluzen"),
-    (r"tovalix", "tovalix"), (r"zikezen", "zikezen"),
+    (r"tovalix", "tovalix"), (r"zikezen", "zikezen"), (r"zigipel", "zigipel"),
 ]
 
 
@@ -42,7 +42,7 @@ def get_model_config_id(model_name: str) -> str:
     n = n.replace("-", "_").replace(".", "p")
     if n.startswith("gemma4"):
         get_config("gemma4_e2b")          # Gemma-4 presets register on first use
-    for fam in ("roluzen", "tovalix", "zikezen"):
+    for fam in ("roluzen", "tovalix", "zikezen", "zigipel"):
         if n.startswith(fam):
             get_config(fam + "_tiny")
     if n in PRESETS:

@@ -53,5 +53,6 @@ for _fam, _pref, _tmpl in (("llama3", ("llama-3", "meta-llama-3", "llama3"), "ll
                            ("gemma4", ("gemma-4-",), "gemma4"),
                            ("roluzen", ("roluzen",), "default"),
                            ("tovalix", ("tovalix",), "default"),
-                           ("zikezen", ("zikezen",), "default")):
+                           ("zikezen", ("zikezen",), "default"),
+                           ("zigipel", ("zigipel",), "default")):
     register_family(FamilyEntry(_fam, config_lib.get_config, _pref, _tmpl))

@@ -113,6 +113,21 @@ _KEY_MAPS = {
         (r"l(\d+)\.mix\.(left|right)\.(q|k|v|a2)\.b", r"layers.\1.mixer.\2.\3_proj.bias"),
         (r"l(\d+)\.mix\.(left|right)\.(q|k|v|g|o|a1|a2)", r"layers.\1.mixer.\2.\3_proj.weight"),
     ],
+    "zigipel": [
+        (r"embed", "embed_tokens"),
+        (r"bigram", "bigram_embed"),
+        (r"loop\.in", "loop_in.weight"),
+        (r"loop\.step", "loop_step"),
+        (r"head", "lm_head"),
+        (r"final\.norm", "norm.weight"),
+        (r"l(\d+)\.norm1", r"layers.\1.input_layernorm.weight"),
+        (r"l(\d+)\.shift", r"layers.\1.shift"),
+        (r"l(\d+)\.mlp\.(gate|up|down)\.b", r"layers.\1.mlp.\2_proj.bias"),
+        (r"l(\d+)\.mlp\.(gate|up|down)", r"layers.\1.mlp.\2_proj.weight"),
+        (r"l(\d+)\.mix\.dkv\.norm", r"layers.\1.mixer.kv_norm.weight"),
+        (r"l(\d+)\.mix\.(r1|r2|sink)", r"layers.\1.mixer.\2"),
+        (r"l(\d+)\.mix\.(q|k|v|g|o|dkv|uk|uv)", r"layers.\1.mixer.\2_proj.weight"),
+    ],
 }
 
 
@@ -197,6 +212,14 @@ _STACK_INVERSE = {"roluzen": _STACK_ENDS + [
     (r"layers\.(\d+)\.mixer\.right\.norm\.weight", r"l\1.mix.right.norm"),
     (r"layers\.(\d+)\.mixer\.(left|right)\.(\w+)_proj\.bias", r"l\1.mix.\2.\3.b"),
     (r"layers\.(\d+)\.mixer\.(left|right)\.(\w+)_proj\.weight", r"l\1.mix.\2.\3"),
+], "zigipel": _STACK_ENDS + [
+    (r"bigram_embed", "bigram"), (r"loop_in\.weight", "loop.in"), (r"loop_step", "loop.step"),
+    (r"layers\.(\d+)\.shift", r"l\1.shift"),
+    (r"layers\.(\d+)\.mlp\.(gate|up|down)_proj\.bias", r"l\1.mlp.\2.b"),
+    (r"layers\.(\d+)\.mlp\.(gate|up|down)_proj\.weight", r"l\1.mlp.\2"),
+    (r"layers\.(\d+)\.mixer\.kv_norm\.weight", r"l\1.mix.dkv.norm"),
+    (r"layers\.(\d+)\.mixer\.(r1|r2|sink)", r"l\1.mix.\2"),
+    (r"layers\.(\d+)\.mixer\.(\w+)_proj\.weight", r"l\1.mix.\2"),
 ]}
 
 

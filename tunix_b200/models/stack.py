@@ -1,13 +1,15 @@
 """Layer-stack models: decoders whose layers are listed one by one, each with its own mixer (`models/mixers.py`) and
 feed-forward, a range of layers that may run several times with the same weights, parallel residual streams joined by
 hyper-connections, norms over groups of a row and behind sublayers, learned position rows, mixtures of experts, and inputs per
-token and layer. Designs of this kind: Roluzen, Tovalix, Zikezen.
+token and layer. Designs of this kind: Roluzen, Tovalix, Zikezen, Zigipel.
 
 The residual streams are fp32. A sublayer q of a layer reads u = sum_s in[s] x_s, computes y = f(norm(u)) and leaves
 x_t = sum_s mix[s, t] x_s + out[t] y on every stream (`post_norms`: y is normed once more); the model's output is the norm of
-the streams' sum. With `loop_embed` the embedding output is added again before every pass of the loop but the first. A layer's
-token input adds norm(proj(gelu(gate(x)) * e)) after the feed-forward, e being the layer's part of the token's row in a second
-embedding table.
+the streams' sum. With `loop_embed` the embedding output is added again before every pass of the loop but the first; with
+`loop_input` every pass t begins with x = W [x; embedding output] + step_t. A layer's token input adds
+norm(proj(gelu(gate(x)) * e)) after the feed-forward, e being the layer's part of the token's row in a second embedding table.
+With `parallel_ff` mixer and feed-forward of a layer read the same norm and are added together; with `token_shift` a mixer reads
+h + (row before - h) * mu instead of h. The embedding may add a row per pair of neighbouring tokens (`bigram`).
 
 The model holds parameters; `models/stack_exec.py` runs it on ragged batches over the paged cache and the slot states of
 `generate/engine.py`. `forward` scores whole sequences through that same path on a temporary cache (no gradients).
@@ -25,8 +27,8 @@ import torch.nn as nn
 
 from ..ops import functional as F
 from .config import ModelConfig
-from .mixers import (ForgetGateMemorySpec, GatedLinearSpec, MatrixMemorySpec, ParallelSpec, RGLRUSpec, RotaryAttentionSpec, SumSpec,
-                     TokenShiftMemorySpec, WindowAttentionSpec, create_mixer)
+from .mixers import (DistanceAttentionSpec, ForgetGateMemorySpec, GatedLinearSpec, LatentAttentionSpec, MatrixMemorySpec, ParallelSpec,
+                     RGLRUSpec, RotaryAttentionSpec, SumSpec, TokenShiftMemorySpec, WindowAttentionSpec, YarnScaling, create_mixer)
 from .transformer import MLP, Linear, RMSNorm
 
 
@@ -34,7 +36,7 @@ from .transformer import MLP, Linear, RMSNorm
 class LayerSpec:
     mixer: object                       # one of the specs of models/mixers.py
     ff: Optional[int]                   # width of the feed-forward (of an expert); None = the layer has none
-    ff_kind: str = "glu"                # "glu": silu-gated; "xielu": up, xIELU with two learned numbers, down; "experts"
+    ff_kind: str = "glu"                # "glu": gated by the model's activation; "xielu": up, xIELU with two learned numbers, down; "experts"
     experts: int = 0                    # silu-gated experts, of which a token uses `top`
     top: int = 0
 
@@ -50,6 +52,12 @@ class StackConfig(ModelConfig):
     embed_factor: float = 1.0           # of the embedding rows
     positions: int = 0                  # rows of the learned position table, the longest sequence; 0 = no table
     loop_embed: bool = False            # the embedding output is added again before each pass of the loop but the first
+    loop_input: bool = False            # each pass of the loop begins with a product of [x; embedding output] and a vector of its own
+    bigram: Optional[tuple] = None      # (buckets, factor of the token before, factor of the token): hashed rows of token pairs
+    parallel_ff: bool = False           # mixer and feed-forward of a layer read the same norm
+    token_shift: bool = False           # mixers read a mix of a token's normed row and the one before it
+    ff_bias: bool = False               # biases of the feed-forward's projections
+    logit_scale: float = 1.0
 
     def __post_init__(self):
         if not self.layer_specs:
@@ -58,13 +66,22 @@ class StackConfig(ModelConfig):
         ffs = [s.ff for s in self.layer_specs if s.ff is not None]
         self.hidden_dim = max(ffs) if ffs else 0
         att = [getattr(s.mixer, "left", s.mixer) for s in self.layer_specs]
-        att = [a for a in att if isinstance(a, (WindowAttentionSpec, RotaryAttentionSpec))]
+        att = [a for a in att if isinstance(a, (WindowAttentionSpec, RotaryAttentionSpec, DistanceAttentionSpec, LatentAttentionSpec))]
         if att:                         # what generic callers size caches and reports by: the first attention layer
             self.num_heads, self.num_kv_heads, self.head_dim = att[0].heads, att[0].kv_heads, att[0].dim
         if self.loop is not None:
             a, b, times = self.loop
             if not (0 <= a <= b <= self.num_layers and times >= 0):
                 raise ValueError(f"loop {self.loop} does not fit {self.num_layers} layers")
+        if self.parallel_ff and (self.post_norms or self.streams or self.token_side):
+            raise ValueError("layers whose sublayers run side by side have one plain residual and no norms behind sublayers")
+        if (self.parallel_ff or self.token_shift) and not all(
+                isinstance(s.mixer, (DistanceAttentionSpec, LatentAttentionSpec)) and s.ff_kind == "glu" for s in self.layer_specs):
+            raise ValueError("this layer form takes distance or latent attention and gated feed-forwards")
+        if self.parallel_ff != self.token_shift:
+            raise ValueError("shifted mixers and side by side sublayers come together")
+        if self.logit_scale != 1.0 and (self.final_logit_softcap or self.logit_scale <= 0):
+            raise ValueError(f"a logit scale of {self.logit_scale}" + (" beside a score cap" if self.final_logit_softcap else ""))
         if self.embed_dim % self.norm_groups:
             raise ValueError(f"a width of {self.embed_dim} does not split into {self.norm_groups} norm groups")
         for i, s in enumerate(self.layer_specs):
@@ -97,6 +114,13 @@ class StackConfig(ModelConfig):
         a, b, times = self.loop
         return {a + t * (b - a) for t in range(1, times)} if b > a else set()
 
+    def loop_starts(self) -> dict:
+        """Pass (index into `runs`) -> number of the loop's repetition that it begins."""
+        if self.loop is None:
+            return {}
+        a, b, times = self.loop
+        return {a + t * (b - a): t for t in range(times)} if b > a else {}
+
     # ---- what the engine's cache manager allocates, per pass
     def kv_rows(self, dtype: Optional[torch.dtype] = None) -> list:
         return [self.layer_specs[i].mixer.kv_rows(dtype or self.dtype) for i in self.runs()]
@@ -113,7 +137,12 @@ class StackConfig(ModelConfig):
         return out
 
     def state_shapes(self) -> list:
-        return [self.layer_specs[i].mixer.state_shapes() for i in self.runs()]
+        before = {"before": (self.embed_dim,)} if self.token_shift else {}     # the normed row of the sequence's last token
+        return [{**self.layer_specs[i].mixer.state_shapes(), **before} for i in self.runs()]
+
+    def token_states(self) -> tuple:
+        """Token ids that a sequence keeps besides the states of its layer passes."""
+        return ("last",) if self.bigram else ()
 
     def num_params(self) -> int:
         return sum(p.numel() for p in StackModel(self, device=torch.device("meta")).parameters())
@@ -198,6 +227,28 @@ class StackConfig(ModelConfig):
         return cls._zikezen(4096, 8192, 32, 8, 128, 32, 64, 128, 16, (5, 11, 2), 1024, 32, 4, 2048, 128)
 
 
+    @classmethod
+    def _zigipel(cls, D, ff, heads, kv, dim, lheads, ldim, rot, lvdim, rank, n, loop, window, lwindow, vocab=151936, buckets=65521) -> "StackConfig":
+        att = DistanceAttentionSpec(heads=heads, kv_heads=kv, dim=dim, vdim=dim, scale=dim ** -0.5, window=window, keep_first=4)
+        lat = LatentAttentionSpec(heads=lheads, dim=ldim, rot_dim=rot, vdim=lvdim, kv_rank=rank, scale=(ldim + rot) ** -0.5,
+                                  window=lwindow, rot_dims=rot, rot_base=500000.0, rot_scaling=YarnScaling(4.0, 4096.0, 32.0, 1.0))
+        specs = tuple(LayerSpec(lat if i % 2 else att, ff) for i in range(n))
+        return cls(family="zigipel", vocab_size=vocab, embed_dim=D, layer_specs=specs, loop=loop, loop_input=True,
+                   bigram=(buckets, 31, 7), parallel_ff=True, token_shift=True, ff_bias=True, activation="gelu", logit_scale=0.5)
+
+    @classmethod
+    def zigipel_tiny(cls) -> "StackConfig":
+        return cls._zigipel(96, 160, 4, 2, 24, 3, 16, 8, 24, 40, 4, (1, 3, 2), 24, 20, vocab=384, buckets=211)
+
+    @classmethod
+    def zigipel_2b(cls) -> "StackConfig":
+        return cls._zigipel(2048, 6144, 16, 8, 128, 16, 128, 64, 128, 512, 18, (6, 12, 2), 1024, 1024)
+
+    @classmethod
+    def zigipel_8b(cls) -> "StackConfig":
+        return cls._zigipel(4096, 12288, 32, 8, 128, 32, 128, 64, 128, 512, 24, (8, 14, 2), 1024, 1024)
+
+
 # ------------------------------------------------------------------------------------------ config.json reader
 def _parallel_spec(m: dict, shapes, prefix: str, width: int) -> ParallelSpec:
     lf, rt = m["left"], m["right"]
@@ -249,6 +300,24 @@ def _hgrn2_spec(m: dict, shapes, prefix: str, width: int) -> ForgetGateMemorySpe
     return ForgetGateMemorySpec(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]))
 
 
+def _distance_spec(m: dict, shapes, prefix: str, width: int) -> DistanceAttentionSpec:
+    mask = m.get("mask") or {}
+    return DistanceAttentionSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                                 scale=float(m["scale"]), window=int(mask.get("size") or 0), keep_first=int(mask.get("keep_first") or 0))
+
+
+def _yarn(rot: dict) -> Optional[YarnScaling]:
+    s = rot.get("scaling")
+    return None if not s else YarnScaling(float(s["factor"]), float(s["original"]), float(s["fast"]), float(s["slow"]))
+
+
+def _latent_spec(m: dict, shapes, prefix: str, width: int) -> LatentAttentionSpec:
+    mask, rot = m.get("mask") or {}, m["rot"]
+    return LatentAttentionSpec(heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]), vdim=int(m["vdim"]),
+                               kv_rank=int(m["kv_rank"]), scale=float(m["scale"]), window=int(mask.get("size") or 0),
+                               rot_dims=int(rot["dims"]), rot_base=float(rot["base"]), rot_scaling=_yarn(rot))
+
+
 @dataclass(frozen=True)
 class Design:
     family: str
@@ -258,12 +327,16 @@ class Design:
     experts: bool = False               # layers may have a mixture of experts
     post_norms: bool = False            # a norm behind every sublayer
     loop_embed: bool = False
+    options: tuple = ()                 # further fields of StackConfig that the design fixes: (name, value)
 
 
 ARCHITECTURES = {
     "Roluzen": Design("roluzen", {"rglru": _rglru_spec, "parallel": _parallel_spec}, "glu"),
     "Tovalix": Design("tovalix", {"wkv": _wkv_spec, "hgrn2": _hgrn2_spec, "attention": _rotary_spec}, "xielu", embed_norm=True),
     "Zikezen": Design("zikezen", {"parallel": _sum_spec}, "glu", experts=True, post_norms=True, loop_embed=True),
+    "Zigipel": Design("zigipel", {"attention": _distance_spec, "latent_attention": _latent_spec}, "glu",
+                      options=(("loop_input", True), ("parallel_ff", True), ("token_shift", True), ("ff_bias", True),
+                               ("activation", "gelu"))),
 }
 STACK_FAMILIES = tuple(d.family for d in ARCHITECTURES.values())
 
@@ -309,13 +382,17 @@ def config_from_stack_json(src: Union[str, dict], dtype: Optional[torch.dtype] =
             raise ValueError(f"layer {i}: no feed-forward {mlp.get('kind')!r} in this framework")
     lp = c.get("loop")
     positions = int(c.get("max_positions") or 0)
+    emb = c.get("embedding") or {}
+    pairs = emb.get("bigram")
     kw = dict(family=design.family, vocab_size=int(c["vocab"]), embed_dim=width, norm_groups=int(c["norm"].get("groups") or 1),
               embed_norm=design.embed_norm, token_side=int((c.get("token_side") or {}).get("dim") or 0),
               norm_eps=float(c["norm"]["eps"]), layer_specs=tuple(specs),
               loop=None if not lp else (int(lp["start"]), int(lp["stop"]), int(lp["times"])),
               streams=int(c.get("streams") or 0), dtype=dtype or torch.bfloat16, post_norms=design.post_norms,
-              loop_embed=design.loop_embed, embed_factor=float((c.get("embedding") or {}).get("scale") or 1.0),
-              final_logit_softcap=float(c.get("logit_softcap") or 0.0), positions=positions)
+              loop_embed=design.loop_embed, embed_factor=float(emb.get("scale") or 1.0),
+              final_logit_softcap=float(c.get("logit_softcap") or 0.0), positions=positions,
+              bigram=None if not pairs else (int(pairs["buckets"]), int(pairs["mul_prev"]), int(pairs["mul_cur"])),
+              logit_scale=1.0 if c.get("logit_scale") is None else float(c["logit_scale"]), **dict(design.options))
     if positions:
         kw["max_position"] = positions
     kw.update(overrides)
@@ -379,8 +456,11 @@ class StackLayer(nn.Module):
         self.post_attention_layernorm = self.mlp = self.hc2 = self.post_attn_norm = self.post_ffw_norm = None
         if cfg.post_norms:
             self.post_attn_norm = RMSNorm(D, eps, False, dt, device)
+        # how much of the row before a mixer reads, per channel
+        self.shift = nn.Parameter(torch.full((D,), 0.5, dtype=dt, device=device)) if cfg.token_shift else None
         if spec.ff is not None:
-            self.post_attention_layernorm = RMSNorm(D, eps, False, dt, device)
+            if not cfg.parallel_ff:
+                self.post_attention_layernorm = RMSNorm(D, eps, False, dt, device)
             if cfg.post_norms:
                 self.post_ffw_norm = RMSNorm(D, eps, False, dt, device)
             if spec.ff_kind == "experts":
@@ -388,7 +468,7 @@ class StackLayer(nn.Module):
             elif spec.ff_kind == "xielu":
                 self.mlp = PlainMLP(D, spec.ff, dt, device)
             else:                       # the generic gated MLP reads only these sizes
-                self.mlp = MLP(ModelConfig(embed_dim=D, hidden_dim=spec.ff, activation=cfg.activation, dtype=dt), device)
+                self.mlp = MLP(ModelConfig(embed_dim=D, hidden_dim=spec.ff, activation=cfg.activation, dtype=dt), device, cfg.ff_bias)
             self.hc2 = HyperConnection(cfg.streams, dt, device) if cfg.streams else None
         self.side = TokenSide(D, cfg.token_side, eps, dt, device) if cfg.token_side else None
 
@@ -400,7 +480,12 @@ class StackModel(nn.Module):
         dt = cfg.dtype
         self.embed_tokens = nn.Parameter(torch.empty(cfg.vocab_size, cfg.embed_dim, dtype=dt, device=device))
         self.embed_norm = RMSNorm(cfg.embed_dim, cfg.norm_eps, False, dt, device) if cfg.embed_norm else None
-        self.pos_embed = self.side_embed = None
+        self.pos_embed = self.side_embed = self.bigram_embed = self.loop_in = self.loop_step = None
+        if cfg.bigram:              # a row per bucket of token pairs, and one for a sequence's first token
+            self.bigram_embed = nn.Parameter(torch.empty(cfg.bigram[0] + 1, cfg.embed_dim, dtype=dt, device=device))
+        if cfg.loop_input and cfg.loop is not None:
+            self.loop_in = Linear(2 * cfg.embed_dim, cfg.embed_dim, False, dt, device)
+            self.loop_step = nn.Parameter(torch.zeros(cfg.loop[2], cfg.embed_dim, dtype=dt, device=device))
         if cfg.positions:
             self.pos_embed = nn.Parameter(torch.empty(cfg.positions, cfg.embed_dim, dtype=dt, device=device))
         if cfg.token_side:          # row of a token: one part of `token_side` columns per layer
@@ -429,11 +514,12 @@ class StackModel(nn.Module):
         return self.lm_head
 
     def compute_final_logits(self, hidden):
-        return F.lm_head_logits(hidden, self.head_weight(), softcap=self.config.final_logit_softcap)
+        z = F.lm_head_logits(hidden, self.head_weight(), softcap=self.config.final_logit_softcap)
+        return z if self.config.logit_scale == 1.0 else z * self.config.logit_scale
 
     def token_logprobs(self, hidden, targets, *, temperature: float = 1.0, want_entropy: bool = False, chunk: Optional[int] = None):
         return F.lm_head_logprobs(hidden, self.head_weight(), targets, softcap=self.config.final_logit_softcap,
-                                  temperature=temperature, want_entropy=want_entropy, chunk=chunk or self.config.logprob_chunk)
+                                  temperature=temperature / self.config.logit_scale, want_entropy=want_entropy, chunk=chunk or self.config.logprob_chunk)
 
     @property
     def num_params(self) -> int:

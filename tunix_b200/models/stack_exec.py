@@ -2,7 +2,8 @@
 through the same function, reading and writing the engine's paged cache and slot states.
 
 Between two sublayers one kernel closes the one before (hyper-connection write) and opens the one after (hyper-connection
-read and norm). Projections that share an input run as one GEMM over weights joined in memory. bf16 models run on the
+read and norm). Projections that share an input run as one GEMM over weights joined in memory; where mixer and feed-forward
+run side by side, the heads and the gated activation land in one row, which one GEMM takes back. bf16 models run on the
 package's tcgen05 GEMMs, with fp32 accumulation; 32-bit models use library GEMMs in full precision (no TF32)."""
 from __future__ import annotations
 
@@ -14,8 +15,8 @@ import torch
 from ..ops import kernels as K
 from ..ops import stack_kernels as SK
 from ..ops.ragged import RaggedBatch
-from .mixers import (TILE_HEADS, ForgetGateMemory, GatedLinearAttention, ParallelMixer, RGLRUMixer, RotaryAttention, SumMixer,
-                     TokenShiftMemory)
+from .mixers import (TILE_HEADS, DistanceAttention, ForgetGateMemory, GatedLinearAttention, LatentAttention, ParallelMixer, RGLRUMixer,
+                     RotaryAttention, SumMixer, TokenShiftMemory, YarnScaling)
 from .stack import ExpertsMLP, PlainMLP
 
 
@@ -73,16 +74,18 @@ def side_by_side(params, dim: int) -> torch.Tensor:
 
 
 def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None,
-           packed=None) -> torch.Tensor:
-    """x @ w^T (+ bias), fp32 accumulation, output in `out_dtype` (default: x's)."""
-    out_dtype = out_dtype or x.dtype
+           packed=None, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """x @ w^T (+ bias), fp32 accumulation, output in `out_dtype` (default: x's) or in `out`, which may be columns of wider rows."""
+    out_dtype = out_dtype or (x.dtype if out is None else out.dtype)
     if x.dtype == torch.bfloat16:
         if packed is not None:
-            return K.gemm_packed(x, packed, bias=bias, out_dtype=out_dtype)
+            return K.gemm_packed(x, packed, bias=bias, out_dtype=out_dtype, out=out)
         if x.shape[1] % 8 == 0:
             if x.stride(0) % 8 or x.data_ptr() % 16:        # columns of a wider row that TMA cannot address
                 x = x.contiguous()
-            return K.gemm(x, w, bias=bias, out_dtype=out_dtype)
+            return K.gemm(x, w, bias=bias, out_dtype=out_dtype, out=out)
+    if out is not None:
+        return out.copy_(linear(x, w, bias, out_dtype))
     prev = torch.backends.cuda.matmul.allow_tf32
     torch.backends.cuda.matmul.allow_tf32 = False
     try:
@@ -93,16 +96,32 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
         torch.backends.cuda.matmul.allow_tf32 = prev
 
 
+def _per_head(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """x [n, heads, K] with a matrix per head w [heads, K, N] -> [n, heads, N], by the library in full precision."""
+    prev = torch.backends.cuda.matmul.allow_tf32
+    torch.backends.cuda.matmul.allow_tf32 = False
+    try:
+        return torch.bmm(x.transpose(0, 1), w).transpose(0, 1)
+    finally:
+        torch.backends.cuda.matmul.allow_tf32 = prev
+
+
 FEW_OUTPUTS = 512       # in a decode step, products with at most this many outputs split the contraction inside a CTA
 
 
 def rope_frequencies(dims: int, base: float, scaling: Optional[tuple] = None, device=None) -> torch.Tensor:
     """fp64 [dims / 2]: base^(-2 i / dims). `scaling` = (factor, low, high, original context), as Llama 3.1 has it: frequencies
     that turn fewer than `low` times over the original context are divided by the factor, those that turn more than `high` times
-    stay, in between the two are mixed linearly in the number of turns."""
+    stay, in between the two are mixed linearly in the number of turns. With a `YarnScaling` the mix is linear in the number of the
+    pair, between the (rounded) pairs that turn `fast` and `slow` times."""
     f = base ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64, device=device) / max(dims, 1))
-    if scaling is None:
+    if scaling is None or not dims:
         return f
+    if isinstance(scaling, YarnScaling):
+        pair = lambda turns: dims * math.log(scaling.original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))  # noqa: E731
+        lo, hi = max(math.floor(pair(scaling.fast)), 0), min(math.ceil(pair(scaling.slow)), dims - 1)
+        far = ((torch.arange(dims // 2, dtype=torch.float64, device=device) - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+        return f / scaling.factor * far + f * (1.0 - far)
     factor, low, high, original = scaling
     turns = original * f / (2.0 * math.pi)
     keep = ((turns - low) / (high - low)).clamp(0.0, 1.0) if high > low else (turns >= low).to(f.dtype)
@@ -110,10 +129,11 @@ def rope_frequencies(dims: int, base: float, scaling: Optional[tuple] = None, de
 
 
 def rope_table(positions: int, dims: int, base: float, device, scaling: Optional[tuple] = None) -> tuple:
-    """cos / sin fp32 [positions, dims / 2] of the angles position * frequency, from fp64."""
+    """cos / sin fp32 [positions, dims / 2] of the angles position * frequency, from fp64 (times a `YarnScaling`'s size)."""
     f = rope_frequencies(dims, base, scaling, device)
     a = torch.arange(positions, dtype=torch.float64, device=device)[:, None] * f
-    return a.cos().float(), a.sin().float()
+    size = scaling.size if isinstance(scaling, YarnScaling) else 1.0
+    return (size * a.cos()).float(), (size * a.sin()).float()
 
 
 class StackExecutor:
@@ -125,8 +145,12 @@ class StackExecutor:
         self._mix = {RGLRUMixer: self._rglru, ParallelMixer: self._parallel, RotaryAttention: self._rotary,
                      TokenShiftMemory: self._shift_memory, ForgetGateMemory: self._forget_memory,
                      GatedLinearAttention: self._gated_linear, SumMixer: self._sum}
+        # mixers whose heads can land in columns of a wider row, before their output projection
+        self._heads = {DistanceAttention: self._distance_heads, LatentAttention: self._latent_heads}
         self.restarts = self.cfg.restarts() if self.cfg.loop_embed else set()
+        self.starts = self.cfg.loop_starts() if self.cfg.loop_input else {}
         self._rope: dict = {}       # kept for good: captured decode graphs point at the tables
+        self._far: dict = {}        # (layer, positions) -> distance bias, kept likewise
         self.dtype = model.embed_tokens.dtype
         self.pk: Callable = lambda i, name: None        # packed decode weights, set by the engine
         self.plain = False          # bf16 through the simple kernels of the 32-bit path (a cross-check, slow)
@@ -155,14 +179,28 @@ class StackExecutor:
                 outs = [layer.mixer.left.o_proj, layer.mixer.right.o_proj]
                 _plain(outs)
                 d["o"] = side_by_side([m.weight for m in outs], 1)
+            if self.cfg.parallel_ff:
+                outs = [layer.mixer.o_proj] + ([] if layer.mlp is None else [layer.mlp.down_proj])
+                _plain(outs)
+                d["o"] = side_by_side([m.weight for m in outs], 1)
+                d["o_bias"] = None if layer.mlp is None or layer.mlp.down_proj.bias is None else layer.mlp.down_proj.bias.data
+            if isinstance(layer.mixer, (DistanceAttention, LatentAttention)):
+                d["sinks"] = layer.mixer.sink.detach().float()
+            if isinstance(layer.mixer, LatentAttention):
+                sp, w = layer.mixer.spec, layer.mixer.uk_proj.weight
+                _plain([layer.mixer.uk_proj, layer.mixer.uv_proj])
+                if sp.tiled(w.dtype):
+                    d["expand"] = layer.mixer.expansion(sp.stored(w.dtype)[0], *sp.tile_heads())
             if isinstance(layer.mlp, PlainMLP):
                 d["up"], _ = joint_weight([layer.mlp.up_proj])
             elif isinstance(layer.mlp, ExpertsMLP):
                 _plain([layer.mlp.router])
                 d["experts_gu"] = side_by_side([layer.mlp.gate_proj, layer.mlp.up_proj], 1)
             elif layer.mlp is not None:
-                d["gu"], _ = joint_weight([layer.mlp.gate_proj, layer.mlp.up_proj])
+                d["gu"], d["gu_bias"] = joint_weight([layer.mlp.gate_proj, layer.mlp.up_proj])
             fresh.append(d)
+        for (i, positions), table in self._far.items():
+            table.copy_(self.model.layers[i].mixer.bias_table(positions))
         for new, old in zip(fresh, self.w):
             for k, v in old.items():
                 if v is not None and v.shape == new[k].shape:
@@ -176,7 +214,7 @@ class StackExecutor:
         out = []
         for layer, d in zip(self.model.layers, self.w):
             src = {k: d[k] for k in ("proj", "gates", "gu", "up", "o") if k in d}
-            if layer.mlp is not None and not isinstance(layer.mlp, ExpertsMLP):
+            if layer.mlp is not None and not isinstance(layer.mlp, ExpertsMLP) and not self.cfg.parallel_ff:
                 src["down"] = layer.mlp.down_proj.weight.data
             out.append(src)
         return out
@@ -225,16 +263,77 @@ class StackExecutor:
     def _rotary_heads(self, m: RotaryAttention, proj, rb: RaggedBatch, pool, r, **kw):
         """Attention of the projected rows (queries, keys and values in their first columns), before the output projection."""
         a, src = m.spec, self.kv_src[r]
-        key = (a.rot_dims, a.rot_base, a.rot_scaling, pool.max_pages * pool.page_size)
-        if key not in self._rope:
-            self._rope[key] = rope_table(key[3], a.rot_dims, a.rot_base, proj.device, a.rot_scaling)
-        cos, sin = self._rope[key]
+        cos, sin = self._rope_tables(a, pool, proj.device)
         nq, kv = a.heads * a.dim, 0 if a.kv_from is not None else a.kv_heads
         q = SK.rope_norm_write(proj, 0, nq, nq + kv * a.dim, cos, sin, a.rot_dims, m.eps, rb, pool.table, pool.page_size, a.heads,
                                kv, a.dim, a.vdim, pool.k[src], pool.v[src], q_w=None if m.q_norm is None else m.q_norm.weight,
                                k_w=None if m.k_norm is None else m.k_norm.weight, interleaved=a.interleaved,
                                stored=a.stored(proj.dtype))
         return self._attend(q, a, None, rb, pool, src, **kw)
+
+    def _rope_tables(self, a, pool, device) -> tuple:
+        key = (a.rot_dims, a.rot_base, a.rot_scaling, pool.max_pages * pool.page_size)
+        if key not in self._rope:
+            self._rope[key] = rope_table(key[3], a.rot_dims, a.rot_base, device, a.rot_scaling)
+        return self._rope[key]
+
+    def _distance_heads(self, i, m: DistanceAttention, h, rb: RaggedBatch, pool, r, out) -> None:
+        d, a = self.w[i], m.spec
+        nq, nk, nv = a.heads * a.dim, a.kv_heads * a.dim, a.kv_heads * a.vdim
+        cols = nq + nk + nv + a.heads
+        row = torch.empty((h.shape[0], -(-cols // 8) * 8), dtype=h.dtype, device=h.device)
+        proj = linear(h, d["proj"], d["proj_bias"], packed=self.pk(i, "proj") if rb.decode else None, out=row[:, :cols])
+        wide, wide_v = a.stored(h.dtype)
+        # queries stay where they are: what a wider head reads behind its own columns meets the zeros behind the stored key
+        here = a.dim % 8 == 0 and (a.heads - 1) * a.dim + wide <= row.shape[1]
+        q = SK.rope_norm_write(proj, 0, nq, nq + nk, None, None, 0, m.eps, rb, pool.table, pool.page_size, 0 if here else a.heads,
+                               a.kv_heads, a.dim, a.vdim, pool.k[r], pool.v[r], stored=(wide, wide_v), norm_qk=False, norm_v=True)
+        if here:
+            q = row.as_strided((row.shape[0], a.heads, wide), (row.stride(0), a.dim, 1))
+        self._attend(q, a, self._distance_bias(i, m, pool), rb, pool, r, out=out, sinks=d["sinks"], gate=proj[:, nq + nk + nv:])
+
+    def _distance_bias(self, i, m: DistanceAttention, pool) -> torch.Tensor:
+        key = (i, pool.max_pages * pool.page_size)
+        if key not in self._far:
+            self._far[key] = m.bias_table(key[1])
+        return self._far[key]
+
+    def _latent_heads(self, i, m: LatentAttention, h, rb: RaggedBatch, pool, r, out) -> None:
+        """Portions of prompts expand the latents of their window to keys and values for the flash attention; single tokens and
+        short portions attend in the absorbed form, as everything does in the general kernel."""
+        d, sp, n = self.w[i], m.spec, h.shape[0]
+        H, qd, R, lat = sp.heads, sp.dim + sp.rot_dim, sp.kv_rank, pool.k[r]
+        proj = linear(h, d["proj"], d["proj_bias"], packed=self.pk(i, "proj") if rb.decode else None)
+        SK.latent_write(proj, H * qd, m.kv_norm.weight, *self._rope_tables(sp, pool, h.device), sp.rot_dims, m.eps, rb, pool.table,
+                        pool.page_size, H, sp.dim, sp.rot_dim, R, lat)
+        q, W = proj[:, :H * qd].unflatten(1, (H, qd)), lat.shape[-1]
+        uk, uv = m.uk_proj.weight.data.view(H, sp.dim, R), m.uv_proj.weight.data.view(H, sp.vdim, R)
+        if self.plain or not sp.tiled(h.dtype) or pool.page_size % 64:
+            full = q.new_zeros((n, H, W))
+            full[:, :, :R] = _per_head(q[:, :, :sp.dim], uk)
+            full[:, :, R:R + sp.rot_dim] = q[:, :, sp.dim:]
+            att = SK.window_attn(full, lat, lat, rb, pool.table, pool.page_size, sp, None, sinks=d["sinks"], sizes=(1, sp.width, R, W, W))
+            out.unflatten(1, (H, sp.vdim)).copy_(_per_head(att.view(n, H, R), uv.transpose(1, 2)))
+            return
+        to = out if out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0 else torch.empty(out.shape, dtype=out.dtype, device=out.device)
+        plan = rb.latent_plan(sp.window)
+        if plan.blocks is not None:
+            wide, wide_v = sp.tile_heads()
+            kv = linear(SK.latent_gather(lat, *plan.blocks, pool.table, pool.page_size), d["expand"])
+            qw = proj.as_strided((n, H, wide), (proj.stride(0), qd, 1)) if (H - 1) * qd + wide <= proj.shape[1] else \
+                torch.nn.functional.pad(q, (0, wide - qd))
+            K.attn_fwd_paged(qw, kv[:, :H * wide], kv[:, H * wide:], rb, plan.table, 64, num_heads=H, num_kv_heads=H, head_dim=wide,
+                             scale=sp.scale, window=sp.window, sinks=d["sinks"], out=to, value_dim=sp.vdim, tiles=plan.tiles,
+                             slots=plan.entries)
+        count = n if plan.rows is None else plan.rows.shape[0]
+        if count:
+            q1 = SK.head_product(q, uk, torch.empty((count, H, W), dtype=h.dtype, device=h.device), x_rows=plan.rows, rows=count,
+                                 tail=sp.rot_dim)
+            att = SK.latent_decode(q1, lat, pool.table, pool.page_size, plan.slots, self._lens if plan.lens is None else plan.lens, rank=R,
+                                   scale=sp.scale, window=sp.window, sinks=d["sinks"], max_ctx=pool.max_pages * pool.page_size)
+            SK.head_product(att, uv, to.unflatten(1, (H, sp.vdim)), transposed=True, out_rows=plan.rows, rows=count)
+        if to is not out:
+            out.copy_(to)
 
     def _shift_memory(self, i, m: TokenShiftMemory, h, rb: RaggedBatch, pool, r):
         """h: the mixes [5, n, D] in a decode step (made by the launch before), else the normed rows."""
@@ -292,25 +391,52 @@ class StackExecutor:
         y = self._few(x, side.gate_proj.weight, rb, SK.ACT_GELU_ROW, tokens=rb.tokens, rows=self.model.side_embed, col=i * dim)
         return (linear(y, side.proj.weight), None, side.norm.weight, None)
 
-    def _attend(self, q, a, bias, rb: RaggedBatch, pool, r, out=None, out_scale: float = 1.0):
+    def _attend(self, q, a, bias, rb: RaggedBatch, pool, r, out=None, out_scale: float = 1.0, sinks=None, gate=None):
         """Tensor-core kernels where the stored heads fit them (the framework's paged decode and flash attention, extended by the
-        bias, the kept tokens and the sink); otherwise, and in 32-bit, the general kernel. `out`: columns that take the result."""
+        bias, the kept tokens, the sink and the heads' gates); otherwise, and in 32-bit, the general kernel. q: [n, heads * stored], or a
+        view [n, heads, stored]. `out`: columns that take the result."""
         wide, wide_v = a.stored(q.dtype)
         fits = q.dtype == torch.bfloat16 and wide == wide_v and wide in TILE_HEADS and not self.plain and a.vdim % 8 == 0 and \
             (out is None or (out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0))
         kw = dict(scale=a.scale, softcap=a.softcap, window=a.window, chunk=a.chunk, keep_first=a.keep_first, sink=a.sink, bias=bias,
-                  value_dim=a.vdim, out=out, out_scale=out_scale)
+                  value_dim=a.vdim, out=out, out_scale=out_scale, sinks=sinks, gate=gate)
+        fits = fits and q.stride(0) % 8 == 0 and (q.dim() == 2 or q.stride(1) % 8 == 0)
         if fits and rb.decode and a.heads // a.kv_heads <= 16:
             max_ctx = pool.table.shape[1] * pool.page_size
             span = min((s for s in (a.window, a.chunk) if s > 0), default=0)       # most keys a query sees besides the kept ones
             split = K.decode_split_tokens(rb.n, a.kv_heads, min(max_ctx, span + a.keep_first + 128) if span else max_ctx)
-            return K.paged_decode(q.view(rb.n, a.heads, wide), pool.k[r], pool.v[r], pool.table, rb.slot, self._lens,
+            return K.paged_decode(q if q.dim() == 3 else q.view(rb.n, a.heads, wide), pool.k[r], pool.v[r], pool.table, rb.slot, self._lens,
                                   num_kv_heads=a.kv_heads, page_size=pool.page_size, max_ctx=max_ctx, split_tokens=split,
-                                  **kw).view(rb.n, -1)
+                                  **kw).flatten(1)
         if fits and not rb.decode and pool.page_size % 64 == 0:
             return K.attn_fwd_paged(q, pool.k[r], pool.v[r], rb, pool.table, pool.page_size, num_heads=a.heads,
                                     num_kv_heads=a.kv_heads, head_dim=wide, **kw)
-        return SK.window_attn(q, pool.k[r], pool.v[r], rb, pool.table, pool.page_size, a, bias, out=out, out_scale=out_scale)
+        return SK.window_attn(q, pool.k[r], pool.v[r], rb, pool.table, pool.page_size, a, bias, out=out, out_scale=out_scale,
+                              sinks=sinks, gate=gate)
+
+    def _side_by_side(self, i, layer, h, mixed, rb: RaggedBatch, pool, r):
+        """Mixer (on its own input `mixed`) and feed-forward of one norm: one row takes the heads and the gated activation."""
+        m, ff = layer.mixer, layer.spec.ff or 0
+        heads = m.spec.heads * m.spec.vdim
+        row = torch.empty((mixed.shape[0], heads + ff), dtype=mixed.dtype, device=mixed.device)
+        self._heads[type(m)](i, m, mixed, rb, pool, r, row[:, :heads])
+        if ff:
+            self._gated(i, h, rb, row[:, heads:])
+        return (linear(row, self.w[i]["o"], self.w[i]["o_bias"], packed=self.pk(i, "o") if rb.decode else None), None, None, None)
+
+    def _gated(self, i, h, rb: RaggedBatch, out=None) -> torch.Tensor:
+        """The gated activation of a feed-forward; `out`: columns of wider rows."""
+        d, kind = self.w[i], K.GLU_SILU if self.cfg.activation == "silu" else K.GLU_GELU
+        F = d["gu"].shape[0] // 2
+        pgu = self.pk(i, "gu") if rb.decode else None
+        aligned = out is None or (out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0)
+        if pgu is not None and pgu.glu:
+            act = K.gemm_packed(h, pgu, glu=kind, bias=d["gu_bias"], out=out if aligned else None)
+            return act if out is None or aligned else out.copy_(act)
+        gu = linear(h, d["gu"], d["gu_bias"], packed=pgu)
+        if gu.dtype == torch.bfloat16 and F % 8 == 0 and aligned:
+            return K.glu_fwd(gu[:, :F], gu[:, F:], kind, out)
+        return SK.glu(gu, kind, out)
 
     def _mlp(self, i, mlp, h, rb: RaggedBatch):
         if isinstance(mlp, PlainMLP):
@@ -319,15 +445,7 @@ class StackExecutor:
             return linear(act, mlp.down_proj.weight, packed=self.pk(i, "down") if rb.decode else None)
         if isinstance(mlp, ExpertsMLP):
             return SK.moe(h, self._router(h, mlp.router.weight, rb), mlp.correction, self.w[i]["experts_gu"], mlp.down_proj, mlp.top, rb)
-        gu_w = self.w[i]["gu"]
-        F = gu_w.shape[0] // 2
-        pgu = self.pk(i, "gu") if rb.decode else None
-        if pgu is not None and pgu.glu:
-            act = K.gemm_packed(h, pgu, glu=K.GLU_SILU)
-        else:
-            gu = linear(h, gu_w, packed=pgu)
-            act = K.glu_fwd(gu[:, :F], gu[:, F:], K.GLU_SILU) if gu.dtype == torch.bfloat16 and F % 8 == 0 else SK.silu_mul(gu)
-        return linear(act, mlp.down_proj.weight, packed=self.pk(i, "down") if rb.decode else None)
+        return linear(self._gated(i, h, rb), mlp.down_proj.weight, mlp.down_proj.bias, packed=self.pk(i, "down") if rb.decode else None)
 
     def _router(self, h, w, rb: RaggedBatch) -> torch.Tensor:
         """fp32 router logits."""
@@ -345,7 +463,13 @@ class StackExecutor:
         x = torch.empty((n, max(cfg.streams, 1), cfg.embed_dim), dtype=torch.float32, device=rb.tokens.device)
         start = dict(tokens=rb.tokens, embed=model.embed_tokens, embed_w=None if model.embed_norm is None else model.embed_norm.weight,
                      embed_scale=cfg.embed_factor, pos=model.pos_embed)
+        if cfg.bigram:
+            start["pairs"] = (model.bigram_embed, cfg.bigram, pool.state.tokens["last"])
         close = start                                                  # what the next stream_step closes
+        pair = None                                                    # [n, 2 D]: residual and embedding output, as a pass begins
+        if self.starts:
+            pair = torch.empty((n, 2 * cfg.embed_dim), dtype=self.dtype, device=x.device)
+            close = dict(start, start_out=pair[:, cfg.embed_dim:])
 
         def pending(out, hc, norm=None):
             y, y2, wy, wy2 = out
@@ -368,6 +492,21 @@ class StackExecutor:
 
         for r, i in enumerate(self.runs):
             layer = model.layers[i]
+            if r in self.starts:
+                step(None, None, raw=True, out=pair[:, :cfg.embed_dim])
+                linear(pair, model.loop_in.weight, model.loop_step[self.starts[r]], out=x.view(n, -1))
+                close = {}
+            if cfg.parallel_ff:
+                before = pool.state[r]["before"]
+                if rb.decode:
+                    h, mixed = step(self._hc(None)[0], layer.input_layernorm.weight, shift=(layer.shift[None], before), both=True)
+                else:
+                    h = step(self._hc(None)[0], layer.input_layernorm.weight)
+                    mixed = SK.token_shift(h, layer.shift[None], before, rb)
+                    SK.keep_last(h, before, rb)
+                close = pending(self._side_by_side(i, layer, h, mixed[0], rb, pool, r), None)
+                ended = True
+                continue
             shifts = rb.decode and isinstance(layer.mixer, TokenShiftMemory)
             if r in self.restarts:
                 close = dict(close, **start)
@@ -380,14 +519,15 @@ class StackExecutor:
             if layer.side is not None:
                 close = pending(self._side(i, layer.side, step(None, None, raw=True), rb), None)
             ended = True
-        return step(None, model.norm.weight)
+        return step(None, model.norm.weight, **({"keep": pool.state.tokens["last"]} if cfg.bigram else {}))
 
     def logits(self, hidden: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
         """fp32 logits of normed hidden rows."""
-        packed = self.pk(len(self.model.layers), "head")
+        packed, scale = self.pk(len(self.model.layers), "head"), self.cfg.logit_scale
         if hidden.dtype == torch.bfloat16 and packed is not None:
-            return K.gemm_packed(hidden, packed, out=out, out_dtype=torch.float32)
+            return K.gemm_packed(hidden, packed, out=out, out_dtype=torch.float32, alpha=scale)
         if hidden.dtype == torch.bfloat16 and hidden.shape[1] % 8 == 0:
-            return K.gemm(hidden, self.model.head_weight(), out=out, out_dtype=torch.float32)
+            return K.gemm(hidden, self.model.head_weight(), out=out, out_dtype=torch.float32, alpha=scale)
         z = linear(hidden, self.model.head_weight(), out_dtype=torch.float32)
+        z = z if scale == 1.0 else z.mul_(scale)
         return z if out is None else out.copy_(z)

@@ -220,12 +220,12 @@ class Attention(nn.Module):
 
 
 class MLP(nn.Module):
-    def __init__(self, cfg: ModelConfig, device=None):
+    def __init__(self, cfg: ModelConfig, device=None, bias: bool = False):
         super().__init__()
         D, Fd, dt = cfg.embed_dim, cfg.hidden_dim, cfg.dtype
-        self.gate_proj = Linear(D, Fd, False, dt, device)
-        self.up_proj = Linear(D, Fd, False, dt, device)
-        self.down_proj = Linear(Fd, D, False, dt, device)
+        self.gate_proj = Linear(D, Fd, bias, dt, device)
+        self.up_proj = Linear(D, Fd, bias, dt, device)
+        self.down_proj = Linear(Fd, D, bias, dt, device)
         self.kind = cfg.activation
 
     def forward(self, x, residual=None):

@@ -174,9 +174,10 @@ def rope_(x: torch.Tensor, positions: torch.Tensor, cos: torch.Tensor, sin: torc
 GLU_SILU, GLU_GELU = 0, 1
 
 
-def glu_fwd(g: torch.Tensor, u: torch.Tensor, kind: int) -> torch.Tensor:
+def glu_fwd(g: torch.Tensor, u: torch.Tensor, kind: int, out: torch.Tensor | None = None) -> torch.Tensor:
+    """act(g) * u; `out` may be columns of wider rows (16-byte aligned)."""
     rows, Fdim = g.shape
-    h = torch.empty((rows, Fdim), dtype=torch.bfloat16, device=g.device)
+    h = torch.empty((rows, Fdim), dtype=torch.bfloat16, device=g.device) if out is None else out
     rc = _lib.cuda().tb_glu_fwd(g.data_ptr(), g.stride(0), u.data_ptr(), u.stride(0), h.data_ptr(), h.stride(0),
                                 rows, Fdim, kind, _lib.stream_ptr())
     _lib.check(rc, "tb_glu_fwd")
@@ -283,9 +284,10 @@ _lib.register_cuda_sigs({
     "tb_attn_fwd": [_lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.I, _lib.I, _lib.I, _lib.I, _lib.I, _lib.I,
                     _lib.LL, _lib.LL, _lib.LL, _lib.LL, _lib.F, _lib.F, _lib.I, _lib.I, _lib.I, _lib.P, _lib.P,
                     _lib.P, _lib.P],
-    "tb_attn_fwd_paged": [_lib.P, _lib.P, _lib.P, _lib.P, _lib.LL, _lib.I, _lib.LL, _lib.I, _lib.I, _lib.I, _lib.I, _lib.F, _lib.F,
-                          _lib.I, _lib.I, _lib.I, _lib.F, _lib.F, _lib.P, _lib.I, _lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.I,
-                          _lib.P, _lib.I, _lib.I, _lib.P, _lib.P],
+    "tb_attn_fwd_paged": [_lib.P, _lib.LL, _lib.I, _lib.I, _lib.P, _lib.LL, _lib.P, _lib.LL, _lib.P, _lib.LL, _lib.I, _lib.LL, _lib.I,
+                          _lib.I, _lib.I, _lib.I, _lib.I, _lib.F, _lib.F, _lib.I, _lib.I, _lib.I, _lib.F, _lib.P, _lib.P, _lib.LL,
+                          _lib.F, _lib.P, _lib.I, _lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.I, _lib.P, _lib.I, _lib.I, _lib.P,
+                          _lib.P],
     "tb_attn_delta": [_lib.P, _lib.LL, _lib.P, _lib.LL, _lib.P, _lib.I, _lib.I, _lib.I, _lib.I, _lib.P],
     "tb_attn_bwd": [_lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.I, _lib.I,
                     _lib.I, _lib.I, _lib.I, _lib.I, _lib.LL, _lib.LL, _lib.LL, _lib.LL, _lib.LL, _lib.LL,
@@ -325,24 +327,34 @@ def attn_fwd(q, k, v, *, scale: float, causal: bool = True, window: int = 0, sof
 
 
 def attn_fwd_paged(q, k_pool, v_pool, rb, table, page_size: int, *, num_heads: int, num_kv_heads: int, head_dim: int, scale: float,
-                   softcap: float = 0.0, window: int = 0, chunk: int = 0, keep_first: int = 0, sink: float = NO_SINK, bias=None,
-                   out=None, value_dim: int = 0, out_scale: float = 1.0) -> torch.Tensor:
+                   softcap: float = 0.0, window: int = 0, chunk: int = 0, keep_first: int = 0, sink: float = NO_SINK, sinks=None,
+                   gate=None, bias=None, out=None, value_dim: int = 0, out_scale: float = 1.0, tiles=None, slots=None) -> torch.Tensor:
     """Flash attention of the entries of a `ops.ragged.RaggedBatch` (prompt portions) over the paged cache that already
-    holds their keys and values. q [n, N * H] bf16 -> [n, N * value_dim]; pools [pages, page_size, KH * H], page_size a multiple
-    of 64. `softcap` / `window` / `chunk` / `keep_first` / `sink` / `bias` / `out_scale` as in `paged_decode`. `value_dim` (0: H):
-    the heads' values stand in the first columns of the stored ones. `out`: columns of wider rows."""
-    n, vd = q.shape[0], value_dim or head_dim
-    assert q.is_contiguous() and page_size % 64 == 0 and k_pool.is_contiguous() and k_pool.shape == v_pool.shape
+    holds their keys and values. q [n, N * H] bf16, or a view [n, N, H] (heads may overlap where the stored keys have zeros behind
+    their own columns) -> [n, N * value_dim]; pools [pages, page_size, KH * H] (or [rows, KH * H], rows may lie apart), page_size a
+    multiple of 64; values may have heads of another size. `softcap` / `window` / `chunk` / `keep_first` / `sink` / `sinks` / `gate` /
+    `bias` / `out_scale` as in `paged_decode`. `value_dim` (0: as stored): the heads' values stand in the first columns of the stored
+    ones. `out`: columns of wider rows. `tiles`, `slots`: other query tiles (first row, entry, number) and page-table rows of the
+    entries than the batch's."""
+    rows = lambda p: p.shape[0] * (page_size if p.dim() == 3 else 1)  # noqa: E731
+    HV = v_pool.shape[-1] // num_kv_heads
+    n, vd = q.shape[0], value_dim or HV
+    q3 = q if q.dim() == 3 else q.view(n, num_heads, head_dim)
+    assert q3.shape == (n, num_heads, head_dim) and q3.stride(2) == 1 and page_size % 64 == 0
+    assert k_pool.shape[-1] == num_kv_heads * head_dim and rows(k_pool) == rows(v_pool) and k_pool.stride(-1) == v_pool.stride(-1) == 1
+    assert all(p.dim() == 2 or p.is_contiguous() for p in (k_pool, v_pool))
     if out is None:
         out = torch.empty((n, num_heads * vd), dtype=q.dtype, device=q.device)
     assert out.shape == (n, num_heads * vd) and out.stride(1) == 1
-    t0, ent, _, tiles = rb.tiles(128)
-    rc = _lib.cuda().tb_attn_fwd_paged(q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(), out.data_ptr(), out.stride(0), n,
-                                       k_pool.shape[0] * page_size, num_heads, num_kv_heads, head_dim, vd, float(scale), float(softcap),
-                                       int(window), int(chunk), int(keep_first), float(sink), float(out_scale), _lib.ptr(bias),
-                                       0 if bias is None else bias.shape[1] - 1,
-                                       rb.cu.data_ptr(), rb.slot.data_ptr(), rb.pos0.data_ptr(), t0.data_ptr(), ent.data_ptr(),
-                                       tiles, table.data_ptr(), table.shape[1], page_size,
+    t0, ent, n_tiles = tiles if tiles is not None else (lambda t: (t[0], t[1], t[3]))(rb.tiles(128))
+    rc = _lib.cuda().tb_attn_fwd_paged(q3.data_ptr(), q3.stride(0), (num_heads - 1) * q3.stride(1) + head_dim, q3.stride(1),
+                                       k_pool.data_ptr(), k_pool.stride(-2), v_pool.data_ptr(), v_pool.stride(-2), out.data_ptr(),
+                                       out.stride(0), n, rows(k_pool), num_heads, num_kv_heads, head_dim, HV, vd, float(scale),
+                                       float(softcap), int(window), int(chunk), int(keep_first), float(sink), _lib.ptr(sinks),
+                                       _lib.ptr(gate), 0 if gate is None else gate.stride(0), float(out_scale), _lib.ptr(bias),
+                                       0 if bias is None else bias.shape[1] - 1, rb.cu.data_ptr(),
+                                       (rb.slot if slots is None else slots).data_ptr(), rb.pos0.data_ptr(), t0.data_ptr(),
+                                       ent.data_ptr(), n_tiles, table.data_ptr(), table.shape[1], page_size,
                                        _lib.status_buffer(q.device).data_ptr(), _lib.stream_ptr())
     _lib.check(rc, "tb_attn_fwd_paged")
     _count()
@@ -380,8 +392,9 @@ def attn_bwd(dout, q, k, v, o, lse, *, scale: float, causal: bool = True, window
 
 _lib.register_cuda_sigs({
     "tb_kv_write": [_lib.P, _lib.P, _lib.LL, _lib.P, _lib.P, _lib.P, _lib.I, _lib.I, _lib.P, _lib.P, _lib.I, _lib.I, _lib.P],
-    "tb_paged_decode": [_lib.P, _lib.LL, _lib.P, _lib.P, _lib.P, _lib.I, _lib.I, _lib.P, _lib.P, _lib.I, _lib.I, _lib.I,
-                        _lib.I, _lib.I, _lib.F, _lib.F, _lib.I, _lib.I, _lib.I, _lib.F, _lib.F, _lib.I, _lib.P, _lib.I, _lib.I, _lib.LL,
+    "tb_paged_decode": [_lib.P, _lib.LL, _lib.I, _lib.P, _lib.P, _lib.P, _lib.I, _lib.I, _lib.P, _lib.P, _lib.I, _lib.I, _lib.I,
+                        _lib.I, _lib.I, _lib.F, _lib.F, _lib.I, _lib.I, _lib.I, _lib.F, _lib.P, _lib.P, _lib.LL, _lib.F, _lib.I,
+                        _lib.P, _lib.I, _lib.I, _lib.LL,
                         _lib.P, _lib.P, _lib.P, _lib.LL, _lib.P, _lib.P],
     "tb_qkv_post": [_lib.P, _lib.LL, _lib.P, _lib.P, _lib.P, _lib.P, _lib.F, _lib.F, _lib.P, _lib.P, _lib.P, _lib.I,
                     _lib.I, _lib.P, _lib.P, _lib.I, _lib.I, _lib.I, _lib.I, _lib.P],
@@ -454,16 +467,19 @@ def decode_split_tokens(batch: int, num_kv_heads: int, max_ctx: int = 0) -> int:
 
 def paged_decode(q, k_pool, v_pool, page_table, seq_ids, seq_lens, *, num_kv_heads: int, page_size: int, max_ctx: int,
                  scale: float, softcap: float = 0.0, window: int = 0, chunk: int = 0, keep_first: int = 0, sink: float = NO_SINK,
-                 bias=None, workspace=None, out=None, split_tokens: int = 0, value_dim: int = 0, out_scale: float = 1.0):
-    """Single-token attention over a paged KV cache. q [B, N, H] bf16 (row stride free) -> out [B, N, H] bf16, or with
+                 sinks=None, gate=None, bias=None, workspace=None, out=None, split_tokens: int = 0, value_dim: int = 0,
+                 out_scale: float = 1.0):
+    """Single-token attention over a paged KV cache. q [B, N, H] bf16 (row and head strides free: heads may overlap where the
+    stored keys have zeros behind their own columns) -> out [B, N, H] bf16, or with
     `value_dim` [B, N, value_dim] (the heads' values stand in the first columns of the stored ones); `out` [B, N * value_dim] may
-    be columns of wider rows. `sink`: one more score in the sum of the weights, without a value. The output is scaled by `out_scale`.
+    be columns of wider rows. `sink`: one more score in the sum of the weights, without a value; `sinks` fp32 [N]: one per head instead.
+    `gate` bf16 [B, N]: a head's output is multiplied by the gate's sigmoid. The output is scaled by `out_scale`.
     `chunk` > 0: a query sees the keys of its own chunk of that many positions, counted from the sequence's start.
     With a window or chunks, the first `keep_first` tokens of a sequence stay visible. `bias` fp32 [N, far + 1] is added to the
     scaled score of a key at distance min(distance, far).
     `workspace` (two fp32 buffers) must be sized for ceil(max_ctx / split_tokens) splits."""
     B, N, H = q.shape
-    assert q.stride(2) == 1 and q.stride(1) == H
+    assert q.stride(2) == 1
     split_tokens = split_tokens or decode_split_tokens(B, num_kv_heads, max_ctx)
     splits = (max_ctx + split_tokens - 1) // split_tokens
     # contiguous pools [pages, page_size, KH * H] can be staged by TMA (one tensor map per pool)
@@ -476,10 +492,11 @@ def paged_decode(q, k_pool, v_pool, page_table, seq_ids, seq_lens, *, num_kv_hea
     if out is None:
         out = torch.empty((B, N, vd), dtype=q.dtype, device=q.device)
     assert out.numel() == B * N * vd and out.stride(-1) == 1
-    rc = _lib.cuda().tb_paged_decode(q.data_ptr(), q.stride(0), k_pool.data_ptr(), v_pool.data_ptr(), page_table.data_ptr(),
+    rc = _lib.cuda().tb_paged_decode(q.data_ptr(), q.stride(0), q.stride(1), k_pool.data_ptr(), v_pool.data_ptr(), page_table.data_ptr(),
                                      page_table.shape[1], page_size, seq_ids.data_ptr(), seq_lens.data_ptr(), B, N,
                                      num_kv_heads, H, max_ctx, float(scale), float(softcap), int(window), int(chunk),
-                                     int(keep_first), float(sink), float(out_scale), vd, _lib.ptr(bias),
+                                     int(keep_first), float(sink), _lib.ptr(sinks), _lib.ptr(gate),
+                                     0 if gate is None else gate.stride(0), float(out_scale), vd, _lib.ptr(bias),
                                      0 if bias is None else bias.shape[1] - 1, int(split_tokens),
                                      pool_rows, workspace[0].data_ptr(), workspace[1].data_ptr(),
                                      out.data_ptr(), out.stride(0), _lib.status_buffer(q.device).data_ptr(), _lib.stream_ptr())
@@ -838,20 +855,23 @@ def gemm_packed(a: torch.Tensor, pw: PackedWeight, *, out: torch.Tensor | None =
                 alpha: float = 1.0, glu: int | None = None, xielu: torch.Tensor | None = None) -> torch.Tensor:
     """C = alpha * A @ W^T with W given as a PackedWeight; same epilogue options as `gemm`. `xielu` (the activation's two
     numbers, before softplus): xIELU on the result, computed in the epilogue. `glu` (GLU_SILU / GLU_GELU)
-    with a weight packed with `glu=True`: C [M, N / 2] = act(A @ Wgate^T) * (A @ Wup^T), computed in the epilogue."""
+    with a weight packed with `glu=True`: C [M, N / 2] = act(A @ Wgate^T) * (A @ Wup^T), computed in the epilogue; `bias` [N]:
+    the gates', then the ups'."""
     assert a.dtype == torch.bfloat16 and _is2d_rowmajor(a)
     M, K = a.shape
     assert K == pw.K, f"contraction mismatch {K} vs {pw.K}"
     N = pw.N
     if glu is not None:
-        assert pw.glu and not accumulate and bias is None and residual is None and alpha == 1.0
+        assert pw.glu and not accumulate and residual is None and alpha == 1.0
+        assert bias is None or (bias.dtype == torch.bfloat16 and bias.numel() == N and bias.is_contiguous())
         if out is None:
             out = torch.empty((M, N // 2), dtype=torch.bfloat16, device=a.device)
         assert out.shape == (M, N // 2) and out.dtype == torch.bfloat16 and out.stride(1) == 1
         if M == 0:
             return out
         rc = _lib.cuda().tb_gemm_packed_bf16(a.data_ptr(), a.stride(0), pw.data.data_ptr(), pw.width, out.data_ptr(),
-                                             out.stride(0), M, N, K, GF_GLU_SILU if glu == GLU_SILU else GF_GLU_GELU, 0, 0, 0, 1.0,
+                                             out.stride(0), M, N, K, (GF_GLU_SILU if glu == GLU_SILU else GF_GLU_GELU) |
+                                             (0 if bias is None else GF_BIAS), _lib.ptr(bias), 0, 0, 1.0,
                                              _lib.status_buffer(a.device).data_ptr(), _lib.stream_ptr())
         _lib.check(rc, "tb_gemm_packed_bf16")
         _count()

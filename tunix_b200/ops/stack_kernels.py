@@ -1,5 +1,5 @@
 """Launchers of the layer-stack kernels (csrc/stack.cu, recurrent.cu, linear_attention.cu, window_attention.cu,
-moe_infer.cu). Activations and weights are bf16 or float (the `dtype` argument of the entry points), residual streams, states and gates fp32."""
+latent_attention.cu, moe_infer.cu). Activations and weights are bf16 or float (the `dtype` argument of the entry points), residual streams, states and gates fp32."""
 from __future__ import annotations
 
 from typing import Optional
@@ -14,23 +14,29 @@ from .ragged import RaggedBatch
 _P, _I, _LL, _F = _lib.P, _lib.I, _lib.LL, _lib.F
 _RB = [_P, _P, _P, _P, _I, _I]
 _lib.register_cuda_sigs({
-    "tb_stream_step": [_I, _P, _I, _I, _I, _F, _P, _P, _P, _P, _P, _P, _P, _P, _I, _P, _F, _P, _I, _I, _P, _P, _P, _P, _P, _I, _P, _P,
-                       _P, _P, _P, _P, _P],
+    "tb_stream_step": [_I, _P, _I, _I, _I, _F, _P, _P, _P, _P, _P, _P, _P, _P, _I, _P, _F, _P, _I, _I, _P, _P, _P, _LL, _P, _P, _I, _P, _P,
+                       _P, _LL, _LL, _LL, _P, _P, _LL, _P, _P, _P, _P, _P, _P, _P],
     "tb_few_outputs": [_P, _P, _I, _I, _I, _I, _P, _I, _P, _LL, _I, _P, _I, _P],
     "tb_small_act": [_I, _P, _I, _I, _I, _P, _I, _P, _LL, _I, _P, _P],
     "tb_token_shift": [_I, _P, _P, _I, _P, *_RB, _I, _P, _P],
     "tb_xielu": [_I, _P, _P, _LL, _P],
     "tb_gated_linear": [_I, _I, _P, _LL, _P, _LL, _P, _LL, _P, _LL, _P, _LL, _P, _LL, _P, _I, _P, _P, _F, _F, *_RB, _I, _I, _I, _P, _P,
                         _P, _I, _P, _I, _F, _F, _P, _P, _LL, _I, _I, _P],
-    "tb_silu_mul": [_I, _P, _P, _LL, _I, _P],
+    "tb_glu": [_I, _I, _P, _P, _LL, _LL, _I, _P],
+    "tb_keep_last": [_I, _P, _P, *_RB, _I, _P],
     "tb_gate_outputs": [_I, _P, _P, _P, _LL, _I, _I, _P, _F, _I, _I, _I, _I, _P, _P, _P],
     "tb_rglru": [_I, _P, _LL, _I, _I, _P, _P, _P, _P, _P, _P, _P, *_RB, _I, _I, _I, _P, _P, _P, _P, _P, _P, _I, _P, _P,
                  _P, _I, _P, _P, _P],
     "tb_mlstm_slices": [_I],
     "tb_mlstm": [_I, _P, _LL, _I, _I, _I, _P, _P, _P, _F, *_RB, _I, _I, _I, _P, _P, _P, _P, _I, _I, _P],
     "tb_qk_norm_write": [_I, _P, _LL, _I, _I, _I, _P, _P, _F, *_RB, _P, _I, _I, _I, _I, _I, _P, _P, _P, _P],
-    "tb_rope_norm_write": [_I, _P, _LL, _I, _I, _I, _P, _P, _P, _P, _I, _I, _F, *_RB, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P, _P, _P],
-    "tb_window_attn": [_I, _P, _P, _P, *_RB, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _P, _I, _I, _I, _I, _F, _F, _P, _LL, _P],
+    "tb_rope_norm_write": [_I, _P, _LL, _I, _I, _I, _P, _P, _P, _P, _I, _I, _F, _I, *_RB, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P, _P, _P],
+    "tb_window_attn": [_I, _P, _LL, _I, _P, _P, *_RB, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _P, _I, _I, _I, _I, _F, _P, _P, _LL,
+                       _F, _P, _LL, _P],
+    "tb_latent_write": [_I, _P, _LL, _I, _I, _I, _I, _I, _P, _F, _P, _P, _I, *_RB, _P, _I, _I, _I, _P, _P],
+    "tb_latent_gather": [_P, _P, _P, _I, _P, _I, _I, _I, _P, _P],
+    "tb_head_product": [_I, _P, _LL, _I, _P, _P, _I, _I, _I, _P, _LL, _I, _P, _I, _I, _I, _P],
+    "tb_latent_decode": [_P, _P, _LL, _P, _I, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P, _I, _P, _P, _P, _P, _P],
     "tb_moe_route": [_I, _P, _P, *_RB, _I, _I, _P, _P, _P, _P, _P, _P],
     "tb_moe_route_lists": [_I, _P, _P, *_RB, _I, _I, _P, _P, _P, _P, _P],
     "tb_moe_experts": [_I, _I, _P, _LL, _P, _P, _I, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P, _P],
@@ -46,29 +52,40 @@ def _dt(t: torch.Tensor) -> int:
 
 
 def stream_step(x: torch.Tensor, eps: float, *, y=None, y2=None, wy=None, wy2=None, mix=None, w_out=None, tokens=None, embed=None,
-                embed_w=None, embed_scale: float = 1.0, pos=None, groups: int = 1, w_in=None, norm_w=None, raw: bool = False,
-                shift=None, rb: Optional[RaggedBatch] = None, sum_out: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+                embed_w=None, embed_scale: float = 1.0, pos=None, pairs=None, start_out=None, groups: int = 1, w_in=None, norm_w=None,
+                raw: bool = False, out=None, shift=None, both: bool = False, keep=None, rb: Optional[RaggedBatch] = None,
+                sum_out: Optional[torch.Tensor] = None):
     """Close one sublayer (y [, y2 with their norms; y alone with its norm wy], mix, w_out; or start from the embedding rows
     of `tokens`, normed with embed_w if given, times embed_scale, plus the rows `pos` [positions, D] of the tokens' positions in
     the batch `rb`; or both: the embedding rows are added to every stream after the sublayer, not to sum_out) and open the next: returns h = norm(sum_s w_in[s] x_s) * norm_w (w_in None:
     the plain sum; norm_w None: nothing follows, or with `raw` the sum itself). The norms of rows and embeddings are taken
     over `groups` equal parts. x fp32 [n, S, D] is updated in place; `sum_out` fp32 [n, D] receives the sum of the streams.
     `shift` = (mu [m, D], carry fp32 [slots, D]), for batches `rb` of single tokens: returns the m mixes
-    h + (carry - h) mu [m, n, D] instead of h and replaces the slots' carry by h."""
+    h + (carry - h) mu [m, n, D] instead of h (`both`: beside it) and replaces the slots' carry by h.
+    `pairs` = (table [buckets + 1, D], (buckets, p, c), last int64 [slots]): the embedding also has the table's row
+    (p * token before + c * token) mod buckets, `last` holding the tokens before the entries' first ones; a sequence's first token
+    takes the last row. `start_out`: columns that take the embedding rows as they are added. `out`: columns of wider rows for h.
+    `keep` int64 [slots] receives every entry's last token."""
     n, S, D = x.shape
     ref = norm_w if norm_w is not None else (y if y is not None else embed)
     mu, carry = shift or (None, None)
     mixes = torch.empty((mu.shape[0], n, D), dtype=ref.dtype, device=x.device) if shift else None
-    h = torch.empty((n, D), dtype=ref.dtype, device=x.device) if (norm_w is not None and not shift) or raw else None
+    h = out
+    if h is None and ((norm_w is not None and (not shift or both)) or raw):
+        h = torch.empty((n, D), dtype=ref.dtype, device=x.device)
+    table, (buckets, m_prev, m_cur), last = pairs or (None, (0, 0, 0), None)
     rc = _lib.cuda().tb_stream_step(_dt(ref), x.data_ptr(), n, S, D, float(eps), _lib.ptr(y), _lib.ptr(y2), _lib.ptr(wy),
                                     _lib.ptr(wy2), _lib.ptr(mix), _lib.ptr(w_out), _lib.ptr(tokens), _lib.ptr(embed),
                                     0 if embed is None else embed.shape[0], _lib.ptr(embed_w), float(embed_scale), _lib.ptr(pos),
                                     0 if pos is None else pos.shape[0], int(groups), _lib.ptr(w_in), _lib.ptr(norm_w), _lib.ptr(h),
-                                    _lib.ptr(sum_out), _lib.ptr(mu), 0 if mu is None else mu.shape[0], _lib.ptr(carry),
-                                    _lib.ptr(mixes), *((0, 0, 0, 0) if rb is None else rb.args()[:4]), _lib.stream_ptr())
+                                    0 if h is None else h.stride(0), _lib.ptr(sum_out), _lib.ptr(mu), 0 if mu is None else mu.shape[0],
+                                    _lib.ptr(carry), _lib.ptr(mixes), _lib.ptr(table), buckets, m_prev, m_cur, _lib.ptr(last),
+                                    _lib.ptr(start_out), 0 if start_out is None else start_out.stride(0), _lib.ptr(keep),
+                                    0 if keep is None else rb.tokens.data_ptr(),
+                                    *((0, 0, 0, 0) if rb is None else rb.args()[:4]), _lib.stream_ptr())
     _lib.check(rc, "tb_stream_step")
     _count()
-    return mixes if shift else h
+    return (h, mixes) if both else mixes if shift else h
 
 
 def token_shift(h, mu, carry, rb: RaggedBatch) -> torch.Tensor:
@@ -84,6 +101,14 @@ def token_shift(h, mu, carry, rb: RaggedBatch) -> torch.Tensor:
     return mixes
 
 
+def keep_last(h, carry, rb: RaggedBatch) -> None:
+    """carry fp32 [slots, D] of the batch's slots = the last rows of its entries in h [n, D]."""
+    assert h.is_contiguous()
+    rc = _lib.cuda().tb_keep_last(_dt(h), h.data_ptr(), carry.data_ptr(), *rb.args(), h.shape[1], _lib.stream_ptr())
+    _lib.check(rc, "tb_keep_last")
+    _count()
+
+
 def xielu_(x: torch.Tensor, act: torch.Tensor) -> torch.Tensor:
     """xIELU in place, act = its two numbers (before softplus)."""
     assert x.is_contiguous() and act.dtype == x.dtype
@@ -93,12 +118,13 @@ def xielu_(x: torch.Tensor, act: torch.Tensor) -> torch.Tensor:
     return x
 
 
-def silu_mul(gu: torch.Tensor) -> torch.Tensor:
-    """gu [rows, 2 F] -> silu(gu[:, :F]) * gu[:, F:], any F."""
+def glu(gu: torch.Tensor, kind: int, out=None) -> torch.Tensor:
+    """gu [rows, 2 F] -> act(gu[:, :F]) * gu[:, F:], any F; kind: K.GLU_SILU or K.GLU_GELU. `out`: columns of wider rows."""
     rows, F2 = gu.shape
-    h = torch.empty((rows, F2 // 2), dtype=gu.dtype, device=gu.device)
-    rc = _lib.cuda().tb_silu_mul(_dt(gu), gu.data_ptr(), h.data_ptr(), rows, F2 // 2, _lib.stream_ptr())
-    _lib.check(rc, "tb_silu_mul")
+    assert gu.is_contiguous()
+    h = torch.empty((rows, F2 // 2), dtype=gu.dtype, device=gu.device) if out is None else out
+    rc = _lib.cuda().tb_glu(_dt(gu), kind, gu.data_ptr(), h.data_ptr(), h.stride(0), rows, F2 // 2, _lib.stream_ptr())
+    _lib.check(rc, "tb_glu")
     _count()
     return h
 
@@ -236,16 +262,18 @@ def qk_norm_write(proj, q_off: int, k_off: int, v_off: int, q_w, k_w, eps: float
 
 def rope_norm_write(proj, q_off: int, k_off: int, v_off: int, cos, sin, rot_dims: int, eps: float, rb: RaggedBatch, table,
                     page_size: int, heads: int, kv_heads: int, dim: int, vdim: int, k_pool, v_pool, *, q_w=None, k_w=None,
-                    interleaved: bool = False, stored: Optional[tuple] = None) -> torch.Tensor:
+                    interleaved: bool = False, stored: Optional[tuple] = None, norm_qk: bool = True, norm_v: bool = False) -> torch.Tensor:
     """Every query and key head divided by its root mean square (times q_w / k_w [dim]) and its first rot_dims dimensions turned
     (cos / sin fp32 [positions, rot_dims / 2]; halves of them together, or neighbours if `interleaved`); q is returned, k and v
     rows go to their pages. `stored`: widths the key / value heads are kept at, with zeros behind them (queries like keys; default:
-    as they are). kv_heads 0: the rows hold queries only and nothing is written."""
+    as they are). kv_heads 0: the rows hold queries only and nothing is written; heads 0: keys and values only. `norm_qk`, `norm_v`:
+    whether query and key heads / value heads are divided by their root mean square."""
     n = proj.shape[0]
     wq, wv = stored or (dim, vdim)
     q = torch.empty((n, heads * wq), dtype=proj.dtype, device=proj.device)
     rc = _lib.cuda().tb_rope_norm_write(_dt(proj), proj.data_ptr(), proj.stride(0), q_off, k_off, v_off, _lib.ptr(q_w), _lib.ptr(k_w),
-                                        _lib.ptr(cos), _lib.ptr(sin), rot_dims, int(interleaved), float(eps), *rb.args(),
+                                        _lib.ptr(cos), _lib.ptr(sin), rot_dims, int(interleaved), float(eps),
+                                        int(norm_qk) + 2 * int(norm_v), *rb.args(),
                                         table.data_ptr(), table.shape[1], page_size, heads, kv_heads, dim, vdim, wq, wv, q.data_ptr(),
                                         k_pool.data_ptr(), v_pool.data_ptr(), _lib.stream_ptr())
     _lib.check(rc, "tb_rope_norm_write")
@@ -253,20 +281,96 @@ def rope_norm_write(proj, q_off: int, k_off: int, v_off: int, cos, sin, rot_dims
     return q
 
 
-def window_attn(q, k_pool, v_pool, rb: RaggedBatch, table, page_size: int, sp, bias, out=None, out_scale: float = 1.0) -> torch.Tensor:
-    """`sp`: an attention spec of models.mixers; bias fp32 [heads, far + 1] or None. Returns out_scale * [n, heads * vdim]; `out`:
-    columns of wider rows."""
+def window_attn(q, k_pool, v_pool, rb: RaggedBatch, table, page_size: int, sp, bias, out=None, out_scale: float = 1.0, sinks=None,
+                gate=None, sizes: Optional[tuple] = None) -> torch.Tensor:
+    """`sp`: an attention spec of models.mixers; bias fp32 [heads, far + 1] or None; `sinks` fp32 [heads], `gate` [n, heads] as in
+    kernels.paged_decode. q [n, heads * stored], or a view [n, heads, ..]. Returns out_scale * [n, heads * vdim]; `out`: columns of wider
+    rows. `sizes`: other (key heads, key size, value size, stored key, stored value) than the spec's."""
     n = q.shape[0]
-    wq, wv = sp.stored(q.dtype)
+    G, dq, dv, wq, wv = sizes or (sp.kv_heads, sp.dim, sp.vdim, *sp.stored(q.dtype))
+    if q.dim() == 2:
+        q = q.view(n, sp.heads, wq)
+    assert q.stride(2) == 1
     if out is None:
-        out = torch.empty((n, sp.heads * sp.vdim), dtype=q.dtype, device=q.device)
-    rc = _lib.cuda().tb_window_attn(_dt(q), q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(), *rb.args(), table.data_ptr(),
-                                    table.shape[1], page_size, sp.heads, sp.kv_heads, sp.dim, sp.vdim, wq, wv, float(sp.scale),
+        out = torch.empty((n, sp.heads * dv), dtype=q.dtype, device=q.device)
+    rc = _lib.cuda().tb_window_attn(_dt(q), q.data_ptr(), q.stride(0), q.stride(1), k_pool.data_ptr(), v_pool.data_ptr(), *rb.args(),
+                                    table.data_ptr(), table.shape[1], page_size, sp.heads, G, dq, dv, wq, wv, float(sp.scale),
                                     float(sp.softcap), _lib.ptr(bias), 0 if bias is None else bias.shape[1] - 1, sp.window,
-                                    sp.chunk, sp.keep_first, float(sp.sink), float(out_scale), out.data_ptr(), out.stride(0),
+                                    sp.chunk, sp.keep_first, float(sp.sink), _lib.ptr(sinks), _lib.ptr(gate),
+                                    0 if gate is None else gate.stride(0), float(out_scale), out.data_ptr(), out.stride(0),
                                     _lib.stream_ptr())
     _lib.check(rc, "tb_window_attn")
     _count()
+    return out
+
+
+# ------------------------------------------------------------------------------------------------ latents
+def latent_write(proj, c_off: int, norm_w, cos, sin, rot_dims: int, eps: float, rb: RaggedBatch, table, page_size: int, heads: int, dim: int,
+                 rot_dim: int, rank: int, pool) -> None:
+    """proj [n, ..]: query heads of dim + rot_dim columns, and at c_off the latent (rank) and the shared key part (rot_dim). The
+    first rot_dims of every rotated part turn (queries in place, halves together); the normed latent and the key part go to their
+    page rows."""
+    rc = _lib.cuda().tb_latent_write(_dt(proj), proj.data_ptr(), proj.stride(0), heads, dim, rot_dim, c_off, rank, norm_w.data_ptr(),
+                                     float(eps), cos.data_ptr(), sin.data_ptr(), rot_dims, *rb.args(), table.data_ptr(), table.shape[1],
+                                     page_size, pool.shape[-1], pool.data_ptr(), _lib.stream_ptr())
+    _lib.check(rc, "tb_latent_write")
+    _count()
+
+
+def latent_gather(pool, slot, pos, table, page_size: int) -> torch.Tensor:
+    """[blocks * 64, W]: the cached rows of positions pos[i] .. pos[i] + 63 of the sequences in slot[i]."""
+    out = torch.empty((slot.shape[0] * 64, pool.shape[-1]), dtype=pool.dtype, device=pool.device)
+    rc = _lib.cuda().tb_latent_gather(pool.data_ptr(), slot.data_ptr(), pos.data_ptr(), slot.shape[0], table.data_ptr(), table.shape[1],
+                                      page_size, pool.shape[-1], out.data_ptr(), _lib.stream_ptr())
+    _lib.check(rc, "tb_latent_gather")
+    _count()
+    return out
+
+
+def head_product(x, w, out, *, transposed: bool = False, x_rows=None, out_rows=None, rows: int = 0, tail: int = 0) -> torch.Tensor:
+    """out[t, h, :N] = x[t, h, :K] w[h], w bf16 [H, K, N] (or [H, N, K] `transposed`). x, out: views [.., H, ..] with free row and head
+    strides; `x_rows` / `out_rows` int32 [rows] name their rows. `tail`: that many columns behind x's K are copied behind out's N,
+    and what is left of out's columns becomes zero."""
+    H = w.shape[0]
+    K_, N = (w.shape[2], w.shape[1]) if transposed else (w.shape[1], w.shape[2])
+    T = rows or x.shape[0]
+    assert w.is_contiguous() and x.stride(2) == out.stride(2) == 1 and x.shape[2] >= K_ + tail and out.shape[2] >= N + tail
+    rc = _lib.cuda().tb_head_product(int(not transposed), x.data_ptr(), x.stride(0), x.stride(1), _lib.ptr(x_rows), w.data_ptr(), H, K_, N,
+                                     out.data_ptr(), out.stride(0), out.stride(1), _lib.ptr(out_rows), T, tail,
+                                     0 if transposed else out.shape[2] - N, _lib.stream_ptr())
+    _lib.check(rc, "tb_head_product")
+    _count()
+    return out
+
+
+def latent_splits(tokens: int, heads: int, tiles: int) -> int:
+    """Tiles of 64 keys per CTA of `latent_decode`: whole waves of one CTA per SM, each with a fixed cost of about two tiles."""
+    groups = -(-heads // (32 if heads > 16 else 16))
+    cost = lambda per: -(-tokens * groups * -(-tiles // per) // 148) * (per + 2)  # noqa: E731
+    return min(range(1, tiles + 1), key=lambda per: (cost(per), -per))
+
+
+def latent_decode(q, pool, table, page_size: int, slots, lens, *, rank: int, scale: float, window: int, sinks, max_ctx: int,
+                  split_tokens: int = 0) -> torch.Tensor:
+    """Attention of single queries q bf16 [T, H, W] in the absorbed form over cached rows [pages, page_size, W], whose first `rank`
+    columns are the values: bf16 [T, H, rank]. Query t sees the last `window` (0: all) of the first lens[t] rows of the
+    sequence in slots[t]; sinks fp32 [H]."""
+    T, H, W = q.shape
+    assert q.is_contiguous() and pool.is_contiguous() and pool.shape[-1] == W
+    tiles = -(-max_ctx // 64)
+    if window > 0:
+        tiles = min(tiles, -(-window // 64) + 1)
+    per = split_tokens // 64 if split_tokens else latent_splits(T, H, tiles)
+    splits = -(-tiles // per)
+    ws = torch.empty(T * H * splits * (rank + 2) if splits > 1 else 0, dtype=torch.float32, device=q.device)
+    out = torch.empty((T, H, rank), dtype=q.dtype, device=q.device)
+    acc = T * H * splits * rank * 4
+    rc = _lib.cuda().tb_latent_decode(q.data_ptr(), pool.data_ptr(), pool.shape[0] * page_size, table.data_ptr(), table.shape[1], page_size,
+                                      slots.data_ptr(), lens.data_ptr(), T, H, rank, W, tiles, float(scale), int(window), _lib.ptr(sinks),
+                                      per * 64, ws.data_ptr(), ws.data_ptr() + acc if splits > 1 else 0, out.data_ptr(),
+                                      _lib.status_buffer(q.device).data_ptr(), _lib.stream_ptr())
+    _lib.check(rc, "tb_latent_decode")
+    _count(1 if splits == 1 else 2)
     return out
 
 
