@@ -1,14 +1,14 @@
-"""Small Roluzen, Tovalix and Zikezen checkpoints with random weights for the layer-stack tests (config.json dict + tensors by name)."""
+"""Small Roluzen, Tovalix, Zikezen and Zigipel checkpoints with random weights for the layer-stack tests (config.json dict + tensors by name)."""
 import json
 import os
 
 import torch
 
-from tests import roluzen_oracle, tovalix_oracle, zikezen_oracle
+from tests import roluzen_oracle, tovalix_oracle, zigipel_oracle, zikezen_oracle
 
 
 def oracle(cfg):
-    return {"Roluzen": roluzen_oracle, "Tovalix": tovalix_oracle, "Zikezen": zikezen_oracle}[cfg["architecture"]]
+    return {"Roluzen": roluzen_oracle, "Tovalix": tovalix_oracle, "Zikezen": zikezen_oracle, "Zigipel": zigipel_oracle}[cfg["architecture"]]
 
 
 # ---- Roluzen
@@ -89,6 +89,29 @@ def zikezen(layers, width=48, vocab=101, loop=None, side=8, eps=1e-5, cap=12.0, 
             "norm": {"eps": eps}, "token_side": {"dim": side}, "vocab": vocab, "width": width}
 
 
+# ---- Zigipel
+def yarn_rot(dims=8, base=700.0, factor=5.0, fast=3.0, slow=0.5, original=60):
+    return {"dims": dims, "base": base, "scaling": {"factor": factor, "fast": fast, "slow": slow, "original": original}}
+
+
+def distance(heads=4, kv_heads=2, dim=16, vdim=24, scale=0.6, size=20, keep_first=3, ff=56):
+    return {"type": "attention", "mlp": None if ff is None else {"kind": "dense", "ff": ff},
+            "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale,
+                      "mask": {"size": size, "keep_first": keep_first}}}
+
+
+def latent(heads=3, dim=16, rot_dim=8, vdim=24, rank=40, scale=0.5, size=23, rot=None, ff=40):
+    return {"type": "latent_attention", "mlp": None if ff is None else {"kind": "dense", "ff": ff},
+            "mixer": {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": rank, "scale": scale, "mask": {"size": size},
+                      "rot": rot or yarn_rot(rot_dim)}}
+
+
+def zigipel(layers, width=48, vocab=101, loop=None, eps=1e-5, buckets=53, mul_prev=5, mul_cur=3, logit_scale=0.4):
+    return {"architecture": "Zigipel", "embedding": {"bigram": {"buckets": buckets, "mul_prev": mul_prev, "mul_cur": mul_cur}},
+            "layers": layers, "logit_scale": logit_scale, "loop": None if loop is None else dict(zip(("start", "stop", "times"), loop)),
+            "norm": {"eps": eps}, "vocab": vocab, "width": width}
+
+
 # sizes apart from each other, layers with and without feed-forward, loops and none, one stream and several, odd widths;
 # "wide" has the head sizes and widths of the tensor-core kernels
 CASES = {
@@ -124,6 +147,18 @@ CASES = {
                        beside(sink_attention(4, 1, 96, 80, size=130, scale=0.15, rot=scaled_rot(dims=96)), gated(1, 104, 136), ff=96),
                        beside(sink_attention(2, 2, 128, 128, size=65, scale=0.1, rot=scaled_rot(dims=64)), gated(3, 64, 64), ff=40,
                               experts=(40, 2))], width=128, vocab=300, side=16, loop=(1, 3, 2)),
+    # both mixers with and without feed-forward, small heads on the tensor-core kernels, a loop over the middle
+    "pairs": zigipel([distance(), latent(), latent(4, 24, 16, 8, 24, size=70, ff=None), distance(2, 1, 24, 16, size=33, keep_first=40, ff=None)],
+                     loop=(1, 3, 2)),
+    # widths that fit no vector load or tensor-core tile, the loop from the first layer to the last, kept tokens beyond the window
+    "crooked": zigipel([distance(3, 1, 10, 6, size=9, keep_first=12, ff=31), latent(3, 7, 6, 5, 13, size=30, rot=yarn_rot(6, base=40.0), ff=33),
+                        latent(1, 12, 2, 9, 50, size=66, ff=None)], width=36, vocab=67, eps=1e-3, loop=(0, 3, 3), buckets=11, mul_prev=1,
+                       mul_cur=1, logit_scale=1.0),
+    # the sizes of the tensor-core kernels: more heads than one group, wide latents, every pair of head sizes; no loop
+    "slabs": zigipel([distance(8, 2, 40, 56, size=70, scale=0.3, keep_first=5, ff=96), latent(20, 96, 64, 128, 136, scale=0.2, size=130, ff=64),
+                      distance(4, 4, 128, 112, size=129, scale=0.2, keep_first=1, ff=None), latent(3, 48, 16, 40, 264, scale=0.4, size=65, ff=72),
+                      latent(17, 104, 24, 64, 512, scale=0.2, size=200, rot=yarn_rot(24, original=500), ff=None),
+                      latent(5, 136, 32, 200, 72, scale=0.2, size=33)], width=128, vocab=300),
 }
 
 
@@ -134,6 +169,8 @@ def weights(cfg, seed=0, buckets=11):
         return tovalix_weights(cfg, seed)
     if cfg["architecture"] == "Zikezen":
         return zikezen_weights(cfg, seed)
+    if cfg["architecture"] == "Zigipel":
+        return zigipel_weights(cfg, seed)
     g = torch.Generator().manual_seed(seed)
     w = {}
 
@@ -330,6 +367,54 @@ def zikezen_weights(cfg, seed=0, rank=8):
         kept.append(rows[clear])
     w["embed"][:, :ROUTED] = torch.cat(kept)[:V] / cfg["embedding"]["scale"]
     w["embed"] = w["embed"].to(torch.bfloat16).float()
+    return w
+
+
+def zigipel_weights(cfg, seed=0):
+    """Attention is sharp, the distance takes a few units off a far key's score, and sinks stand among the scores."""
+    g = torch.Generator().manual_seed(seed)
+    w = {}
+
+    def put(name, *shape, std=None, mean=0.0, uniform=None):
+        x = torch.randn(*shape, generator=g)
+        if uniform is not None:
+            x = uniform[0] + (uniform[1] - uniform[0]) * torch.rand(*shape, generator=g)
+        else:
+            x = mean + ((shape[-1] ** -0.5 if len(shape) > 1 else 0.2) if std is None else std) * x
+        w[name] = x.to(torch.bfloat16).float()
+
+    D, V = cfg["width"], cfg["vocab"]
+    put("embed", V, D, std=0.7)
+    put("bigram", cfg["embedding"]["bigram"]["buckets"] + 1, D, std=0.7)
+    if cfg["loop"]:
+        put("loop.in", D, 2 * D)
+        put("loop.step", cfg["loop"]["times"], D, std=0.5)
+    put("head", V, D, std=3.0 * D ** -0.5)
+    put("final.norm", D, mean=1.0)
+    for i, layer in enumerate(cfg["layers"]):
+        p, m, H = f"l{i}.", layer["mixer"], layer["mixer"]["heads"]
+        put(p + "norm1", D, mean=1.0)
+        put(p + "shift", D, uniform=(0.0, 1.0))
+        if layer["type"] == "attention":
+            G = m["kv_heads"]
+            for s, rows in (("q", H * m["dim"]), ("k", G * m["dim"]), ("v", G * m["vdim"]), ("g", H)):
+                put(f"{p}mix.{s}", rows, D)
+            put(p + "mix.r1", H, uniform=(0.1, 0.8))
+            put(p + "mix.r2", H, uniform=(0.1, 2.0))
+        else:
+            R = m["kv_rank"]
+            put(p + "mix.q", H * (m["dim"] + m["rot_dim"]), D)
+            put(p + "mix.dkv", R + m["rot_dim"], D)
+            put(p + "mix.dkv.norm", R, mean=1.0)
+            put(p + "mix.uk", H * m["dim"], R)
+            put(p + "mix.uv", H * m["vdim"], R)
+        put(p + "mix.sink", H, std=1.5, mean=1.0)
+        put(p + "mix.o", D, H * m["vdim"])
+        if layer["mlp"] is not None:
+            ff = layer["mlp"]["ff"]
+            for s, shape in (("gate", (ff, D)), ("up", (ff, D)), ("down", (D, ff))):
+                put(f"{p}mlp.{s}", *shape)
+                put(f"{p}mlp.{s}.b", shape[0], std=0.5)
     return w
 
 

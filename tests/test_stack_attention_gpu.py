@@ -7,6 +7,7 @@ import torch
 
 from tests import roluzen_oracle as O
 from tests import tovalix_oracle as TO
+from tests import zigipel_oracle as ZG
 from tests import zikezen_oracle as ZO
 from tests.test_stack_kernels_gpu import batch, rand, rel
 
@@ -62,13 +63,13 @@ def run(kind, cache, rb, q, sp, bias, split=0, **kw):
     from tunix_b200.ops import stack_kernels as SK
     n = q.shape[0]
     if kind == "general":
-        return SK.window_attn(q.reshape(n, -1), cache.k, cache.v, rb, cache.table, cache.page, sp, bias, **kw).view(n, sp.heads, sp.vdim)
+        return SK.window_attn(q if q.stride(0) != q.shape[1] * q.shape[2] else q.reshape(n, -1), cache.k, cache.v, rb, cache.table, cache.page, sp, bias, **kw).view(n, sp.heads, sp.vdim)
     kw = dict(scale=sp.scale, softcap=sp.softcap, window=sp.window, chunk=sp.chunk, keep_first=sp.keep_first, sink=sp.sink, bias=bias,
               value_dim=sp.vdim, **kw)
     if kind == "decode":
         return K.paged_decode(q, cache.k, cache.v, cache.table, rb.slot, rb.pos0 + 1, num_kv_heads=sp.kv_heads, page_size=cache.page,
                               max_ctx=cache.table.shape[1] * cache.page, split_tokens=split, **kw).view(n, sp.heads, sp.vdim)
-    return K.attn_fwd_paged(q.reshape(n, -1).contiguous(), cache.k, cache.v, rb, cache.table, cache.page, num_heads=sp.heads,
+    return K.attn_fwd_paged(q if q.stride(0) != q.shape[1] * q.shape[2] else q.reshape(n, -1).contiguous(), cache.k, cache.v, rb, cache.table, cache.page, num_heads=sp.heads,
                             num_kv_heads=sp.kv_heads, head_dim=sp.stored(q.dtype)[0], **kw).view(n, sp.heads, sp.vdim)
 
 
@@ -498,3 +499,153 @@ def test_weighted_norm_interleaved_rotation_and_wider_pages(H, G, dq, dv, rot, d
         assert rel(kp[pg, o], wantk[row]) < t and torch.equal(vp[pg, o].double().cpu(), wantv[row])
         assert kp[pg, o].view(G, wk)[:, dq:].abs().sum() == 0
     assert (kp != 3).any(-1).sum() == 8 and (vp != 3).any(-1).sum() == 8
+
+
+# ------------------------------------------------------------------------------------------------ distance, learned sinks, gates
+def distant(H, G, dq, dv, window, keep, scale=0.3):
+    from tunix_b200.models.mixers import DistanceAttentionSpec
+    return DistanceAttentionSpec(heads=H, kv_heads=G, dim=dq, vdim=dv, scale=scale, window=window, keep_first=keep)
+
+
+def learned(sp, positions, seed=0):
+    """(r1, r2, sinks, distance bias) of a module with drawn numbers."""
+    from tunix_b200.models.mixers import DistanceAttention
+    m = DistanceAttention(sp, 8, 1e-5, torch.float32, "cuda")
+    g = torch.Generator("cuda").manual_seed(seed)
+    m.r1.data.uniform_(0.1, 0.9, generator=g)
+    m.r2.data.uniform_(0.1, 2.0, generator=g)
+    m.sink.data.normal_(0.5, 1.5, generator=g)
+    return m.r1.data, m.r2.data, m.sink.data, m.bias_table(positions)
+
+
+def dense_distance(q, k, v, i0, sp, r1, r2, sink, gate):
+    q, k, v, r1, r2, sink, gate = (t.double().cpu() for t in (q, k, v, r1, r2, sink, gate))
+    T, P = q.shape[0], k.shape[0]
+    pad = torch.zeros(P, *q.shape[1:], dtype=torch.float64)
+    pad[i0:i0 + T] = q
+    m = {"heads": sp.heads, "kv_heads": sp.kv_heads, "scale": sp.scale, "mask": {"size": sp.window or 10 ** 9, "keep_first": sp.keep_first}}
+    return ZG.attend(pad, k, v, m, r1, r2, sink)[i0:i0 + T] * torch.sigmoid(gate)[:, :, None]
+
+
+def apart(q, sp, extra=16):
+    """The same queries in rows that hold more behind them (and between heads nothing), read at the stored width."""
+    n, H, d = q.shape
+    wk = sp.stored(q.dtype)[0]
+    row = torch.full((n, H * d + max(wk - d, 0) + extra), 3.0, dtype=q.dtype, device="cuda")
+    row = torch.cat([q.reshape(n, -1), row[:, H * d:]], 1)
+    return row.as_strided((n, H, wk), (row.stride(0), d, 1)) if d % 8 == 0 and row.shape[1] % 8 == 0 else widen(q, sp)
+
+
+FAR = [("general", torch.float32, 4, 2, 12, 20), ("general", torch.bfloat16, 3, 1, 17, 9), ("general", torch.float32, 2, 1, 24, 600)]
+FAR_FLASH = [("flash", torch.bfloat16, 6, 2, 40, 56), ("flash", torch.bfloat16, 3, 1, 128, 128), ("flash", torch.bfloat16, 4, 4, 72, 80)]
+FAR_DECODE = [("decode", torch.bfloat16, 6, 2, 40, 56), ("decode", torch.bfloat16, 16, 1, 128, 128), ("decode", torch.bfloat16, 3, 3, 72, 80)]
+
+
+@pytest.mark.parametrize("window,keep", [(20, 3), (64, 5), (65, 64), (63, 70), (200, 0), (0, 0), (1, 1), (130, 129)])
+@pytest.mark.parametrize("kind,dtype,H,G,dq,dv", FAR + FAR_FLASH)
+def test_distance_sinks_and_gates_in_portions(kind, dtype, H, G, dq, dv, window, keep):
+    sp = distant(H, G, dq, dv, window, keep)
+    r1, r2, sink, bias = learned(sp, 384)
+    cache = Widened([300, 64, 130, 7], sp, dtype, seed=41)
+    parts = [(0, 120, 180), (1, 0, 64), (2, 128, 2), (3, 0, 7), (0, 69, 131)]
+    n = sum(p[2] for p in parts)
+    q, rows = rand(n, H, dq, dtype=dtype), torch.full((n, 8 + H * dv + 8 + (-H * dv) % 8), 9.0, dtype=dtype, device="cuda")
+    gate = rand(n, 3 + H, dtype=dtype, std=2.0, seed=4)[:, 3:]
+    out, at = run(kind, cache, batch(parts), apart(q, sp), sp, bias, out=rows[:, 8:8 + H * dv], sinks=sink, gate=gate), 0
+    assert rows[:, :8].eq(9).all() and rows[:, 8 + H * dv:].eq(9).all()
+    for s, p, m in parts:
+        k, v = cache.seqs[s]
+        want = dense_distance(q[at:at + m], k[:p + m], v[:p + m], p, sp, r1, r2, sink, gate[at:at + m])
+        assert rel(out[at:at + m], want) < tol(dtype), s
+        at += m
+
+
+@pytest.mark.parametrize("window,keep", [(20, 3), (64, 5), (65, 64), (63, 70), (200, 0), (0, 0), (1, 1), (130, 129)])
+@pytest.mark.parametrize("kind,dtype,H,G,dq,dv", FAR[:2] + FAR_DECODE)
+def test_distance_sinks_and_gates_in_single_tokens(kind, dtype, H, G, dq, dv, window, keep):
+    sp = distant(H, G, dq, dv, window, keep)
+    r1, r2, sink, bias = learned(sp, 384, seed=1)
+    lens = [1, 20, 21, 63, 64, 65, 66, 129, 140, 200, 201, 300]
+    cache = Widened(lens, sp, dtype, seed=42)
+    rb = batch([(s, n - 1, 1) for s, n in enumerate(lens)] + [(len(lens), 0, 1)])
+    rb.pos0[-1] = -1                                                    # idle
+    n = len(lens) + 1
+    q, gate = rand(n, H, dq, dtype=dtype), rand(n, H, dtype=dtype, std=2.0, seed=4)
+    want = [dense_distance(q[s:s + 1], k, v, lens[s] - 1, sp, r1, r2, sink, gate[s:s + 1]) for s, (k, v) in enumerate(cache.seqs)]
+    for split in (0, 64, 128, 512):
+        out = run(kind, cache, rb, apart(q, sp), sp, bias, split, sinks=sink, gate=gate)
+        for s, w in enumerate(want):
+            assert rel(out[s:s + 1], w) < tol(dtype), (s, split)
+        assert out[-1].abs().max() == 0
+        if kind == "general":
+            break
+
+
+@pytest.mark.parametrize("score", [-60.0, -8.0, 0.0, 12.0, 60.0])
+@pytest.mark.parametrize("kind,dtype,H,G,dq,dv", FAR[:2] + FAR_FLASH[:2] + FAR_DECODE[:2])
+def test_every_head_has_its_own_sink(kind, dtype, H, G, dq, dv, score):
+    """All keys score the same: a head's sink takes its exact share of the weights, also far below and above them."""
+    window, n = 40, 100
+    sp = distant(H, G, dq, dv, window, 0, scale=1.0)
+    cache = Widened([n], sp, dtype, seed=43)
+    wk, _ = sp.stored(dtype)
+    cache.k.view(*cache.k.shape[:2], G, wk)[..., 0] = 1.0
+    q = torch.zeros(1, H, dq, dtype=dtype, device="cuda")
+    q[..., 0] = score
+    sink = torch.linspace(-70.0, 70.0, H, device="cuda") if H > 1 else torch.zeros(1, device="cuda")
+    out = run(kind, cache, batch([(0, n - 1, 1)]), widen(q, sp), sp, None, sinks=sink)[0].double().cpu()
+    v = cache.seqs[0][1].double().cpu()[n - window:]
+    for h in range(H):
+        share = 1 / (math.exp(sink[h].item() - score) + window)
+        want = v[:, h // (H // G)].sum(0) * share
+        assert torch.allclose(out[h], want, rtol=tol(dtype), atol=tol(dtype) * want.abs().max().item() + 1e-30), h
+
+
+@pytest.mark.parametrize("window,keep", EDGES)
+@pytest.mark.parametrize("kind,dtype,H,G,dq,dv,decoded", [(*c, d) for d, cs in ((False, FAR[:2] + FAR_FLASH), (True, FAR[:2] + FAR_DECODE)) for c in cs])
+def test_one_key_at_an_edge_against_distance_and_sinks(kind, dtype, H, G, dq, dv, window, keep, decoded):
+    """Queries that ask for one key, whose score stands above what the distance takes off: seen, the output is its value."""
+    sp = distant(H, G, dq, dv, window, keep, scale=0.3)
+    r1, r2, sink, bias = learned(sp, 384, seed=2)
+    cache = Widened([330], sp, dtype, seed=44, unit=True)
+    k, v = cache.seqs[0]
+    pairs = sorted({(i, j) for i in (63, 64, 127, 128, 191, 200, 255, 256, 320, 329)
+                    for j in (i, i - 1, i - window + 1, i - window, 0, keep - 1, keep, 63, 64, 127, 128) if 0 <= j <= i})
+    ask = lambda ps, js: widen(outstanding(cache, 0, ps, js, H, dq), sp)  # noqa: E731
+    rows = []
+    for i, j in pairs:
+        lo = i if decoded else max(0, i - 2)
+        rows.append(run(kind, cache, batch([(0, lo, i + 1 - lo)]), ask(range(lo, i + 1), [*range(lo, i), j]), sp, bias, sinks=sink)[-1:])
+    for (i, j), o in zip(pairs, torch.cat(rows)):
+        val = torch.stack([v[j, h // (H // G)] for h in range(H)]).double().cpu()
+        err = ((o.double().cpu() - val).norm() / val.norm()).item()
+        assert err < 0.05 if ZG.visible(i, j, {"size": window, "keep_first": keep}) else err > 0.3, (i, j, err)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("H,G,dq,dv", [(4, 2, 16, 24), (3, 1, 10, 6), (8, 4, 64, 64), (2, 2, 72, 128), (6, 2, 40, 48), (4, 2, 52, 40), (3, 3, 24, 256)])
+def test_value_norm_and_page_write(H, G, dq, dv, dtype):
+    """Queries and keys as they are, value heads divided by their root mean square; with queries or without."""
+    from tunix_b200.ops import stack_kernels as SK
+    sp = distant(H, G, dq, dv, 0, 0)
+    wk, wv = sp.stored(dtype)
+    NQ, NK, NV, eps = H * dq, G * dq, G * dv, 1e-2
+    rb = batch([(1, 62, 4), (0, 0, 3), (2, 5, 1)])
+    rb.pos0[2] = -1
+    n = 8
+    proj = rand(n, 8 + NQ + NK + NV, dtype=dtype, std=0.3)
+    table = torch.tensor([[4, -1], [2, 0], [3, 3]], dtype=torch.int32, device="cuda")
+    t = 2e-6 if dtype == torch.float32 else 5e-3
+    p = proj.double().cpu()
+    wide = lambda x, heads, w: torch.nn.functional.pad(x.reshape(n, heads, -1), (0, w - x.shape[1] // heads)).reshape(n, -1)  # noqa: E731
+    wantk = wide(p[:, 8 + NQ:8 + NQ + NK], G, wk)
+    wantv = wide(ZG.rms(p[:, 8 + NQ + NK:].reshape(n, G, dv), eps).reshape(n, -1), G, wv)
+    for heads in (H, 0):
+        kp, vp = torch.full((5, 64, G * wk), 3.0, device="cuda", dtype=dtype), torch.full((5, 64, G * wv), 3.0, device="cuda", dtype=dtype)
+        q = SK.rope_norm_write(proj, 8, 8 + NQ, 8 + NQ + NK, None, None, 0, eps, rb, table, 64, heads, G, dq, dv, kp, vp, stored=(wk, wv),
+                               norm_qk=False, norm_v=True)
+        if heads:
+            assert torch.equal(q[:7].double().cpu(), wide(p[:, 8:8 + NQ], H, wk)[:7]) and q[7].abs().max() == 0
+        for row, (pg, o) in enumerate([(2, 62), (2, 63), (0, 0), (0, 1), (4, 0), (4, 1), (4, 2)]):
+            assert torch.equal(kp[pg, o].double().cpu(), wantk[row]) and rel(vp[pg, o], wantv[row]) < t
+        assert (kp != 3).any(-1).sum() == 7 and (vp != 3).any(-1).sum() == 7

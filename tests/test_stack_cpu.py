@@ -9,6 +9,7 @@ import torch
 from tests import roluzen_oracle as O
 from tests import stack_cases as C
 from tests import tovalix_oracle as TO
+from tests import zigipel_oracle as ZG
 from tests import zikezen_oracle as ZO
 
 
@@ -413,3 +414,183 @@ def test_sequences_stay_within_the_learned_positions():
         check_length(eng, 513)
     check_length(SimpleNamespace(cfg=config_from_hf(C.CASES["shared"])), 10 ** 6)
     check_length(SimpleNamespace(), 10 ** 6)
+
+
+# ------------------------------------------------------------------------------------------------ Zigipel
+def test_zigipel_constants_come_from_config_json():
+    from tunix_b200.models.hf_config import config_from_hf
+    from tunix_b200.models.mixers import YarnScaling
+    cfg = C.CASES["pairs"]
+    c = config_from_hf(cfg)
+    assert (c.family, c.bigram, c.logit_scale, c.activation, c.streams, c.token_side) == ("zigipel", (53, 5, 3), 0.4, "gelu", 0, 0)
+    assert c.parallel_ff and c.token_shift and c.ff_bias and c.loop_input and not c.loop_embed and not c.post_norms
+    assert c.loop == (1, 3, 2) and c.runs() == [0, 1, 2, 1, 2, 3] and c.loop_starts() == {1: 0, 3: 1}
+    a, b = c.layer_specs[0].mixer, c.layer_specs[2].mixer
+    assert (a.heads, a.kv_heads, a.dim, a.vdim, a.scale, a.window, a.keep_first) == (4, 2, 16, 24, 0.6, 20, 3)
+    assert (b.heads, b.dim, b.rot_dim, b.vdim, b.kv_rank, b.scale, b.window, b.rot_dims, b.rot_base) == (4, 24, 16, 8, 24, 0.5, 70, 16, 700.0)
+    assert b.rot_scaling == YarnScaling(5.0, 60.0, 3.0, 0.5) and [s.ff for s in c.layer_specs] == [56, 40, None, None]
+    assert config_from_hf(C.CASES["crooked"]).loop_starts() == {0: 0, 3: 1, 6: 2} and config_from_hf(C.CASES["slabs"]).loop_starts() == {}
+    assert config_from_hf(dict(cfg, logit_scale=None, embedding={})).bigram is None
+    plain = dict(cfg["layers"][1]["mixer"], rot={"dims": 8, "base": 5.0})
+    assert config_from_hf(dict(cfg, loop=None, layers=[dict(cfg["layers"][1], mixer=plain)])).layer_specs[0].mixer.rot_scaling is None
+    with pytest.raises(ValueError, match="mixer"):
+        config_from_hf(dict(cfg, layers=[C.wkv()]))
+    with pytest.raises(ValueError, match="feed-forward"):
+        config_from_hf(dict(cfg, layers=[dict(C.distance(), mlp={"kind": "moe", "expert": {"ff": 8}, "router": {"experts": 2, "top": 1}})]))
+    with pytest.raises(ValueError, match="logit scale"):
+        config_from_hf(dict(cfg, logit_scale=-1.0))
+
+
+def test_latent_cache_and_states():
+    from tunix_b200.generate.engine import PagePool
+    from tunix_b200.models.hf_config import config_from_hf
+    c = config_from_hf(C.CASES["slabs"])
+    assert c.kv_rows() == [(128, 128), (256, 0), (512, 512), (320, 0), (576, 0), (128, 0)]
+    assert c.kv_rows(torch.float32) == [(80, 112), (200, 0), (512, 448), (280, 0), (536, 0), (104, 0)]
+    assert [s.mixer.tile_heads() for s in c.layer_specs if hasattr(s.mixer, "kv_rank")] == [(192, 128), (64, 64), (128, 64), (256, 256)]
+    small = config_from_hf(C.CASES["crooked"])
+    assert not any(s.mixer.tiled(torch.bfloat16) for s in small.layer_specs[1:]) and small.kv_rows()[:3] == [(10, 6), (19, 0), (52, 0)]
+    pool = PagePool(c, 4, 16, 3, 4, "cpu", torch.float32, prefix_caching=False)
+    assert pool.k[1].shape == (4, 16, 200) and pool.v[1] is None and pool.state[1]["before"].shape == (3, 128)
+    assert pool.state.tokens["last"].dtype == torch.int64 and pool.state.nbytes_per_slot() == 6 * 128 * 4 + 8
+    assert config_from_hf(C.CASES["blocks"]).token_states() == ()
+
+
+def test_zigipel_presets_and_parameters():
+    from tunix_b200.models import naming, registry
+    from tunix_b200.models.config import get_config
+    from tunix_b200.models.transformer import create_model
+    assert registry.get_family("zigipel").family == "zigipel" and registry.family_of_hf_id("x/Zigipel-2B").family == "zigipel"
+    assert naming.config_for("zigipel-8b") == get_config("zigipel_8b") and naming.get_model_family("x/Zigipel-2B") == "zigipel"
+    cfg = get_config("zigipel_tiny")
+    model = create_model(cfg, seed=3)
+    assert model.num_params == cfg.num_params() and cfg.runs() == [0, 1, 2, 1, 2, 3]
+    assert model.layers[0].post_attention_layernorm is None and model.layers[0].mlp.down_proj.bias.eq(0).all()
+    assert model.loop_in.weight.shape == (96, 192) and model.loop_step.shape == (2, 96) and model.bigram_embed.shape == (212, 96)
+    assert create_model(cfg.replace(loop=None), init=False).loop_in is None
+    with pytest.raises(ValueError, match="side by side"):
+        cfg.replace(streams=2)
+    with pytest.raises(ValueError, match="distance or latent"):
+        get_config("tovalix_tiny").replace(parallel_ff=True, token_shift=True, token_side=0)
+
+
+def test_rows_of_both_sublayers_are_one_product():
+    """Weights joined along the contraction, derived arrays at fixed addresses, packed sources."""
+    from tunix_b200.models.config import get_config
+    from tunix_b200.models.stack_exec import StackExecutor
+    from tunix_b200.models.transformer import create_model
+    model = create_model(get_config("zigipel_tiny").replace(dtype=torch.bfloat16), seed=0)
+    ex = StackExecutor(model)
+    ex._far[(0, 32)] = model.layers[0].mixer.bias_table(32)
+    before = {(i, k): v.data_ptr() for i, d in enumerate(ex.w) for k, v in d.items() if v is not None}
+    lat, mlp = model.layers[1].mixer, model.layers[1].mlp
+    with torch.no_grad():
+        mlp.down_proj.weight.mul_(2.0)
+        lat.uk_proj.weight.mul_(0.5)
+        lat.sink.fill_(3.0)
+        model.layers[0].mixer.r1.fill_(0.25)
+    ex.refresh()
+    assert {(i, k): v.data_ptr() for i, d in enumerate(ex.w) for k, v in d.items() if v is not None} == before
+    n = lat.o_proj.weight.shape[1]
+    assert torch.equal(ex.w[1]["o"][:, n:], mlp.down_proj.weight) and torch.equal(ex.w[1]["o"][:, :n], lat.o_proj.weight)
+    sp, e = lat.spec, ex.w[1]["expand"]
+    wide, wide_v = sp.tile_heads()
+    row = torch.randn(sp.stored(torch.bfloat16)[0])
+    row[sp.width:] = 0
+    kv = e.float() @ row
+    k, v = kv[:sp.heads * wide].view(sp.heads, wide), kv[sp.heads * wide:].view(sp.heads, wide_v)
+    c = row[:sp.kv_rank]
+    assert torch.allclose(k[:, :sp.dim].flatten(), lat.uk_proj.weight.float() @ c, atol=1e-5)
+    assert torch.allclose(v[:, :sp.vdim].flatten(), lat.uv_proj.weight.float() @ c, atol=1e-5)
+    assert torch.equal(k[:, sp.dim:sp.dim + sp.rot_dim], row[sp.kv_rank:sp.width].expand(sp.heads, -1))
+    assert k[:, sp.dim + sp.rot_dim:].eq(0).all() and v[:, sp.vdim:].eq(0).all() and ex.w[1]["sinks"].eq(3).all()
+    want = -0.25 * torch.log1p(model.layers[0].mixer.r2.double()[:, None] * torch.arange(32).double())
+    assert torch.allclose(ex._far[(0, 32)].double(), want, atol=1e-6)
+    assert set(ex.pack_sources()[1]) == {"proj", "gu", "o"}
+
+
+@pytest.mark.parametrize("dims,base,factor,original,fast,slow", [(8, 700.0, 5.0, 60, 3.0, 0.5), (64, 1e6, 40.0, 4096, 32.0, 1.0), (16, 1e4, 2.0, 900, 7.0, 7.0),
+                                                                 (2, 30.0, 8.0, 100, 1.0, 0.1), (24, 5e5, 4.0, 20, 32.0, 1.0), (32, 1e4, 1.0, 128, 32.0, 1.0)])
+def test_yarn_frequencies(dims, base, factor, original, fast, slow):
+    from tunix_b200.models.mixers import YarnScaling
+    from tunix_b200.models.stack_exec import rope_frequencies, rope_table
+    rot = {"dims": dims, "base": base, "scaling": {"factor": factor, "original": original, "fast": fast, "slow": slow}}
+    s = YarnScaling(factor, float(original), fast, slow)
+    assert torch.allclose(rope_frequencies(dims, base, s), ZG.frequencies(rot), rtol=1e-9)
+    cos, sin = rope_table(40, dims, base, "cpu", s)
+    x = torch.randn(40, dims)
+    u, v = x[:, :dims // 2], x[:, dims // 2:]
+    got = torch.cat([u * cos - v * sin, v * cos + u * sin], 1)
+    assert torch.allclose(got, ZG.rotate(x.double(), torch.arange(40), rot).float(), atol=1e-5)
+
+
+def test_zigipel_oracle_details():
+    b = {"buckets": 10, "mul_prev": 3, "mul_cur": 7}
+    assert ZG.bigram_rows([4, 5, 0], b) == [10, (12 + 35) % 10, 15 % 10]
+    s, sink = torch.tensor([0.0, math.log(2.0), -math.inf]).double(), torch.tensor(math.log(3.0)).double()
+    assert torch.allclose(ZG.sink_softmax(s, sink), torch.tensor([1 / 6, 2 / 6, 0.0]).double())
+    mask = {"size": 20, "keep_first": 3}
+    assert ZG.visible(19, 0, {"size": 20}) and not ZG.visible(20, 0, {"size": 20}) and ZG.visible(40, 2, mask) and not ZG.visible(40, 3, mask)
+    assert not ZG.visible(1, 2, mask) and ZG.visible(40, 21, mask) and not ZG.visible(40, 20, mask)
+    T = 50
+    assert all(ZG.seen(T, mask)[i, j] == ZG.visible(i, j, mask) for i in range(T) for j in range(T))
+    h = torch.randn(5, 3).double()
+    assert torch.equal(ZG.token_shift(h, torch.ones(3).double())[1:], h[:-1]) and torch.equal(ZG.token_shift(h, torch.zeros(3).double()), h)
+    assert ZG.layer_runs({"layers": [0] * 4, "loop": {"start": 1, "stop": 3, "times": 2}}) == [(0, None), (1, 0), (2, None), (1, 1), (2, None), (3, None)]
+    # two visible keys, one head: e^(score - r1 ln(1 + r2 gap)) against the sink
+    m = {"heads": 1, "kv_heads": 1, "scale": 0.5, "mask": {"size": 2}}
+    q = k = torch.tensor([[[1.0]], [[2.0]], [[1.0]]]).double()
+    v = torch.tensor([[[1.0]], [[10.0]], [[100.0]]]).double()
+    one = lambda x: torch.tensor([x], dtype=torch.float64)  # noqa: E731
+    got = ZG.attend(q, k, v, m, one(2.0), one(3.0), one(0.3))[2, 0, 0].item()
+    e1, e2 = math.exp(1.0) / 4 ** 2, math.exp(0.5)
+    assert abs(got - (10 * e1 + 100 * e2) / (e1 + e2 + math.exp(0.3))) < 1e-9
+    # latent attention in its absorbed form
+    g = torch.Generator().manual_seed(0)
+    rnd = lambda *n: torch.randn(*n, generator=g, dtype=torch.float64)  # noqa: E731
+    T, H, d, r, R, dv = 9, 2, 4, 2, 5, 3
+    q, qr, c, kr, uk, uv, sinks = rnd(T, H, d), rnd(T, H, r), rnd(T, R), rnd(T, r), rnd(H, d, R), rnd(H, dv, R), rnd(H)
+    m = {"heads": H, "scale": 0.4, "mask": {"size": 4}}
+    got = ZG.latent_attend(q, qr, torch.einsum("tr,hdr->thd", c, uk), kr, torch.einsum("tr,hvr->thv", c, uv), m, sinks)
+    for t in range(T):
+        js = [j for j in range(T) if ZG.visible(t, j, m["mask"])]
+        for a in range(H):
+            s = torch.stack([(uk[a].T @ q[t, a]) @ c[j] + qr[t, a] @ kr[j] for j in js]) * 0.4
+            p = torch.exp(s) / (torch.exp(s).sum() + torch.exp(sinks[a]))
+            assert torch.allclose(got[t, a], uv[a] @ (p @ c[js]))
+
+
+def test_plan_of_latent_batches():
+    """Which tokens attend in which form, and the table of the expanded blocks."""
+    from tunix_b200.ops.ragged import EXPAND_MIN, EXPAND_RATIO, RaggedBatch
+    window = 20 * EXPAND_MIN
+    work = [(5, 0, [1] * 200), (2, 700, [1] * 3), (0, 130, [1] * (EXPAND_MIN * 3)), (1, 9, [1]), (3, 4000, [1] * EXPAND_MIN), (4, 0, [1] * EXPAND_MIN)]
+    rb = RaggedBatch.build(work, "cpu")
+    p = rb.latent_plan(window)
+    assert p is rb.latent_plan(window)
+    lens = [len(t) for _, _, t in work]
+    starts = [sum(lens[:e]) for e in range(len(lens))]
+    long = [0, 2, 5]                             # 4 has 20 cached rows per token before it, more than pay
+    assert EXPAND_RATIO < 19
+    rows = [t for e in (1, 3, 4) for t in range(starts[e], starts[e] + lens[e])]
+    assert p.rows.tolist() == rows and p.slots.tolist() == [work[e][0] for e in (1, 3, 4) for _ in range(lens[e])]
+    assert p.lens.tolist() == [work[e][1] + o + 1 for e in (1, 3, 4) for o in range(lens[e])]
+    assert list(zip(p.tiles[0].tolist(), p.tiles[1].tolist())) == [(0, 0), (128, 0), (starts[2], 2), (starts[5], 5)] and p.tiles[2] == 4
+    slots, pos = (t.tolist() for t in p.blocks)
+    for e in long:
+        slot, p0, toks = work[e]
+        first = max(0, p0 - window + 1)
+        for block in range(first // 64, (p0 + len(toks) - 1) // 64 + 1):
+            b = int(p.table[e, block])
+            assert (slots[b], pos[b]) == (slot, 64 * block)
+    assert len(pos) == sum((work[e][1] + lens[e] - 1) // 64 - max(0, work[e][1] - window + 1) // 64 + 1 for e in long)
+    one = RaggedBatch.build([(3, 7, [1]), (0, 0, [2])], "cpu").latent_plan(window)
+    assert one.blocks is None and one.rows is None and one.slots.tolist() == [3, 0]
+    short = RaggedBatch.build([(3, 7, [1, 2]), (0, 0, [2])], "cpu").latent_plan(window)
+    assert short.blocks is None and short.rows.tolist() == [0, 1, 2] and short.lens.tolist() == [8, 9, 1]
+
+
+def test_splits_of_the_absorbed_form():
+    from tunix_b200.ops.stack_kernels import latent_splits
+    assert latent_splits(64, 32, 17) == 9 and latent_splits(1000, 8, 17) == 17 and latent_splits(1, 16, 1) == 1
+    assert all(1 <= latent_splits(t, h, n) <= n for t in (1, 7, 64, 300) for h in (1, 16, 17, 128) for n in (1, 2, 17, 300))

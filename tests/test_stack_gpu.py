@@ -1,4 +1,4 @@
-"""Layer-stack models on the GPU against the plain oracles (tests/roluzen_oracle.py, tovalix_oracle.py, zikezen_oracle.py): whole
+"""Layer-stack models on the GPU against the plain oracles (tests/roluzen_oracle.py, tovalix_oracle.py, zikezen_oracle.py, zigipel_oracle.py): whole
 prompts, portions, mixed batches, decoding, slots and pages that are used again, greedy generation through the engine. Mechanism tests are in
 test_stack_kernels_gpu.py and test_gated_linear_gpu.py."""
 import functools
@@ -126,7 +126,7 @@ def test_portions_and_decoding_agree_with_the_oracle(name, dtype):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("name", ["mixed", "wide", "shared", "tiles", "uneven", "looped", "ragged", "blocks"])
+@pytest.mark.parametrize("name", ["mixed", "wide", "shared", "tiles", "uneven", "looped", "ragged", "blocks", "pairs", "crooked", "slabs"])
 def test_mixed_batches_and_reused_slots(name, dtype):
     """Unequal requests: portions beside decoded tokens, requests that sit out steps, ends in between; six requests share
     three slots and a pool that holds two of the longest, so that pages and slots change owners."""
@@ -161,7 +161,7 @@ def test_mixed_batches_and_reused_slots(name, dtype):
         assert close(torch.cat(got[i]), want, dtype), i
 
 
-@pytest.mark.parametrize("name", ["wide", "tiles", "blocks"])
+@pytest.mark.parametrize("name", ["wide", "tiles", "blocks", "slabs"])
 def test_a_batch_equals_each_request_alone_in_bf16(name):
     """bf16 results do not depend on the company beyond rounding: compared with the single request, not with the oracle."""
     cfg, _, model = case(name, torch.bfloat16)
@@ -179,7 +179,7 @@ def test_a_batch_equals_each_request_alone_in_bf16(name):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("name", ["mixed", "shared", "tiles", "looped", "blocks"])
+@pytest.mark.parametrize("name", ["mixed", "shared", "tiles", "looped", "blocks", "pairs", "slabs"])
 def test_long_decoding(name, dtype):
     """Several hundred decoded tokens: states, rings, windows and chunks that have turned over many times."""
     cfg, _, model = case(name, dtype)
@@ -219,7 +219,7 @@ def greedy_reference(name, prompt, steps):
 
 
 @pytest.mark.parametrize("graph", [True, False])
-@pytest.mark.parametrize("name", ["mixed", "shared", "uneven", "looped", "ragged"])
+@pytest.mark.parametrize("name", ["mixed", "shared", "uneven", "looped", "ragged", "pairs", "crooked"])
 def test_greedy_generation_matches_the_oracle(name, graph):
     """Through the engine's entry point and scheduler in 32-bit: four prompts over two slots and a pool that forces
     pre-emption, decode step captured in a graph or not; logits of the oracle decide."""
@@ -238,7 +238,7 @@ def test_greedy_generation_matches_the_oracle(name, graph):
             assert lp <= 0.0
 
 
-@pytest.mark.parametrize("name", ["wide", "tiles", "blocks"])
+@pytest.mark.parametrize("name", ["wide", "tiles", "blocks", "pairs", "slabs"])
 def test_generation_is_the_same_under_portions_preemption_and_graphs(name):
     """bf16 and the tensor-core kernels: sampled tokens of one engine against engines with other schedules."""
     cfg, _, model = case(name, torch.bfloat16)
@@ -262,7 +262,7 @@ def test_generation_is_the_same_under_portions_preemption_and_graphs(name):
                 assert abs(la[k] - lb[k]) < 0.3, kw
 
 
-@pytest.mark.parametrize("name", ["wide", "tiles", "blocks"])
+@pytest.mark.parametrize("name", ["wide", "tiles", "blocks", "slabs"])
 def test_stop_tokens_and_sampling_run_through_the_engine(name):
     cfg, _, model = case(name, torch.bfloat16)
     eng = engine(model, pages=12, slots=4, ctx=192)
@@ -276,7 +276,7 @@ def test_stop_tokens_and_sampling_run_through_the_engine(name):
     assert c.tokens[0].tolist() == a.tokens[0].tolist()[:first + 1]
 
 
-@pytest.mark.parametrize("name", ["wide", "tiles", "blocks"])
+@pytest.mark.parametrize("name", ["wide", "tiles", "blocks", "slabs"])
 def test_engine_server_serves_the_model(name):
     from tunix_b200.generate.engine import EngineServer
     cfg, _, model = case(name, torch.bfloat16)
@@ -291,7 +291,7 @@ def test_engine_server_serves_the_model(name):
     assert all(len(t) == 8 for t in first)
 
 
-@pytest.mark.parametrize("name", ["wide", "tiles", "blocks"])
+@pytest.mark.parametrize("name", ["wide", "tiles", "blocks", "slabs"])
 def test_scoring_with_padding_matches_unpadded_rows(name):
     cfg, _, model = case(name, torch.float32)
     rows = [C.tokens(cfg, n, 140 + n) for n in (6, 19)]
@@ -304,7 +304,7 @@ def test_scoring_with_padding_matches_unpadded_rows(name):
     assert close(z[1, :19], oracle(name, tuple(rows[1])), torch.float32)
 
 
-@pytest.mark.parametrize("name", ["mixed", "shared", "looped"])
+@pytest.mark.parametrize("name", ["mixed", "shared", "looped", "pairs"])
 def test_trace_runner_replays_steps(name, tmp_path):
     import json
     import os
@@ -330,6 +330,48 @@ def test_trace_runner_replays_steps(name, tmp_path):
     for step, rows in ((0, [0, 39]), (1, [8]), (2, [69])):
         got = torch.from_numpy(np.fromfile(tmp_path / f"{step}.f32", "<f4")).view(len(rows), -1)
         assert close(got, want[rows], torch.float32)
+
+
+def test_log_probabilities_of_scaled_logits():
+    """Scoring uses the scaled logits, as generation does."""
+    cfg, _, model = case("pairs", torch.float32)
+    toks = C.tokens(cfg, 30, 170)
+    want = torch.log_softmax(oracle("pairs", tuple(toks)) / 0.7, -1)
+    hidden, _ = model(torch.tensor([toks]), skip_lm_head=True)
+    targets = torch.tensor([toks[1:] + [0]], device="cuda")
+    got = model.token_logprobs(hidden, targets, temperature=0.7)
+    got = (got[0] if isinstance(got, tuple) else got).view(-1)
+    assert torch.allclose(got.double().cpu(), want[torch.arange(30), targets[0].cpu()], atol=2e-4)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("name", ["pairs", "slabs"])
+def test_portions_expand_and_single_tokens_absorb(name, dtype):
+    """Cuts on both sides of the length from which a portion's keys are expanded, behind prefixes longer than every window, beside
+    requests that do the other; every row against the oracle."""
+    from tunix_b200.ops.ragged import EXPAND_MIN, RaggedBatch
+    cfg, _, model = case(name, dtype)
+    windows = [L["mixer"]["mask"]["size"] for L in cfg["layers"] if L["type"] == "latent_attention"]
+    lens = [300, 290, 40]
+    seqs = [C.tokens(cfg, n, 180 + i) for i, n in enumerate(lens)]
+    wants = [oracle(name, tuple(s)) for s in seqs]
+    ses = session(model, pages=12, slots=3)
+    at, got = [0, 0, 0], [[], [], []]
+    cuts = [(128, 1, 15), (EXPAND_MIN - 1, 127, 1), (EXPAND_MIN, 2, 16), (1, EXPAND_MIN + 9, 0), (2, 64, 1), (65, 1, 2), (1, 1, 1),
+            (72, 69, 4)]
+    kinds = set()
+    for step in cuts:
+        entries = [(i, seqs[i][at[i]:at[i] + k], range(k)) for i, k in enumerate(step) if k]
+        for w in windows:
+            plan = RaggedBatch.build([(0, at[i], t) for i, t, _ in entries], "cuda").latent_plan(w)
+            kinds.add((plan.blocks is not None, plan.rows is None or len(plan.rows) > 0))
+        z, o = ses.step(entries), 0
+        for i, t, _ in entries:
+            got[i].append(z[o:o + len(t)])
+            at[i], o = at[i] + len(t), o + len(t)
+    assert at == lens and {(True, True), (False, True)} <= kinds
+    for i, want in enumerate(wants):
+        assert close(torch.cat(got[i]), want, dtype), i
 
 
 def test_sequences_longer_than_the_learned_positions_are_refused():

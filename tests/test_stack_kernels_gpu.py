@@ -363,3 +363,81 @@ def test_rows_of_experts_do_not_depend_on_the_company():
     for at, n in ((0, 1), (17, 40), (299, 1), (100, 128)):
         part = SK.moe(h[at:at + n], z[at:at + n].contiguous(), corr, gu, down, 4, batch([(0, at, n)]))
         assert rel(part, full[at:at + n]) < 8e-3
+
+
+# ------------------------------------------------------------------------------------------------ token pairs, shifted rows, gated products
+@pytest.mark.parametrize("dtype", DT)
+@pytest.mark.parametrize("D", [40, 37, 1024])
+def test_stream_step_token_pairs_and_rows_beside_it(D, dtype):
+    """The pair table's rows across portions, first tokens and idle slots; the embedding output in columns of a wider row; the tokens
+    that the next portions start from."""
+    from tunix_b200.ops import stack_kernels as SK
+    eps, tol = 1e-3, 1e-6 if dtype == torch.float32 else 5e-3
+    rb = batch([(1, 7, 3), (0, 0, 2), (2, 40, 1), (3, 5, 1), (4, 0, 1)])
+    rb.pos0[3] = -1
+    n, toks = 8, [3, 0, 49, 7, 7, 1, 2, 30]
+    rb.tokens.copy_(torch.tensor(toks))
+    rule = (13, 31, 5)
+    last = torch.tensor([11, 22, 33, 44, 55, 66], device="cuda")
+    embed, pairs, nw, y = (rand(*s, dtype=dtype, seed=80 + i) for i, s in enumerate([(50, D), (14, D), (D,), (n, D)]))
+    one = torch.ones(1, device="cuda", dtype=dtype)
+    d = lambda t: t.double().cpu()  # noqa: E731
+    cfg = {"embedding": {"bigram": dict(zip(("buckets", "mul_prev", "mul_cur"), rule))}}
+    w = {"embed": d(embed), "bigram": d(pairs)}
+    seq = lambda before, own: ZG.embedding(cfg, w, torch.tensor(before + own))[len(before):]  # noqa: E731
+    want = torch.cat([seq([22], toks[:3]), seq([], toks[3:5]), seq([33], toks[5:6]), seq([], toks[6:7]), seq([], toks[7:])])
+    x, row = torch.empty(n, 1, D, device="cuda"), torch.full((n, 2 * D + 3), 9.0, dtype=dtype, device="cuda")
+    h = SK.stream_step(x, eps, w_in=one, norm_w=nw, tokens=rb.tokens, embed=embed, pairs=(pairs, rule, last), start_out=row[:, D:2 * D], rb=rb)
+    assert rel(x[:, 0], want) < 1e-6 and rel(h, ZG.rms(want, eps) * d(nw)) < tol and rel(row[:, D:2 * D], want) < tol
+    got = SK.stream_step(x, eps, y=y, mix=one, w_out=one, raw=True, out=row[:, :D], keep=last, rb=rb)
+    assert got.data_ptr() == row.data_ptr() and rel(row[:, :D], want + d(y)) < tol and row[:, 2 * D:].eq(9).all()
+    assert rel(row[:, D:2 * D], want) < tol and last.tolist() == [7, 49, 1, 44, 30, 66]
+    h = SK.stream_step(x, eps, w_in=one, norm_w=nw)                     # nothing to close: the rows as they are
+    assert rel(h, ZG.rms(want + d(y), eps) * d(nw)) < tol
+
+
+@pytest.mark.parametrize("dtype", DT)
+@pytest.mark.parametrize("D", [40, 37, 1000])
+def test_token_shift_of_one_mix(D, dtype):
+    """Portions and single tokens: the same mixes beside the rows themselves, the same carried rows."""
+    from tunix_b200.ops import stack_kernels as SK
+    tol = 1e-6 if dtype == torch.float32 else 5e-3
+    mu, nw = rand(1, D, dtype=dtype, seed=1), torch.ones(D, device="cuda", dtype=dtype)
+    one, eps = torch.ones(1, device="cuda", dtype=dtype), 1e-3
+    seq = rand(41, D, dtype=dtype, seed=2)
+    h_all = (ZG.rms(seq.double().cpu(), eps)).to(dtype).double()
+    want = ZG.token_shift(h_all, mu[0].double().cpu())
+    carry = torch.full((3, D), 5.0, device="cuda")
+    at = 0
+    for k in (1, 19, 1, 2, 1, 17):
+        h = h_all[at:at + k].to(dtype).cuda()
+        if k == 1:
+            rb = batch([(2, at, 1)])
+            x = torch.empty(1, 1, D, device="cuda")
+            h2, mixed = SK.stream_step(x, eps, tokens=torch.zeros(1, dtype=torch.long, device="cuda"), embed=seq[at:at + 1], w_in=one, norm_w=nw,
+                                       shift=(mu, carry), both=True, rb=rb)
+            assert rel(h2, h) < tol
+        else:
+            rb = batch([(2, at, k)])
+            mixed = SK.token_shift(h, mu, carry, rb)
+            SK.keep_last(h, carry, rb)
+        assert mixed.shape == (1, k, D) and rel(mixed[0], want[at:at + k]) < 2 * tol
+        at += k
+        assert rel(carry[2], h_all[at - 1]) < tol and carry[:2].eq(5).all()
+    rb = batch([(0, 4, 2), (1, 0, 1)])
+    rb.pos0[1] = -1
+    SK.keep_last(seq[:3].contiguous(), carry, rb)                       # an idle slot keeps what it has
+    assert torch.equal(carry[0].to(dtype), seq[1]) and carry[1].eq(5).all()
+
+
+@pytest.mark.parametrize("M,N,K", [(5, 64, 128), (64, 16640, 256), (130, 224, 64)])
+def test_packed_gated_product_with_bias(M, N, K):
+    from tunix_b200.ops import kernels as K_
+    x, w, b = rand(M, K, dtype=torch.bfloat16), rand(N, K, dtype=torch.bfloat16, std=0.2, seed=1), rand(N, dtype=torch.bfloat16, seed=2)
+    z = (x.double() @ w.double().T + b.double()).cpu()
+    want = ZG.gelu_tanh(z[:, :N // 2]) * z[:, N // 2:]
+    pw = K_.PackedWeight(w, glu=True)
+    rows = torch.full((M, N // 2 + 16), 9.0, dtype=torch.bfloat16, device="cuda")
+    got = K_.gemm_packed(x, pw, glu=K_.GLU_GELU, bias=b, out=rows[:, 8:8 + N // 2])
+    assert rel(got, want) < 5e-3 and rows[:, :8].eq(9).all() and rows[:, 8 + N // 2:].eq(9).all()
+    assert rel(K_.glu_fwd(z[:, :N // 2].bfloat16().cuda(), z[:, N // 2:].bfloat16().cuda(), K_.GLU_GELU, rows[:, 8:8 + N // 2]), want) < 1e-2
