@@ -72,6 +72,21 @@ __device__ __forceinline__ bool mbar_try_wait(uint32_t bar, uint32_t parity) {
   return ok != 0;
 }
 
+// Whether a phase has completed, without waiting.
+__device__ __forceinline__ bool mbar_test(uint32_t bar, uint32_t parity) {
+  uint32_t ok;
+  asm volatile(
+      "{\n"
+      ".reg .pred p;\n"
+      "mbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\n"
+      "selp.u32 %0, 1, 0, p;\n"
+      "}\n"
+      : "=r"(ok)
+      : "r"(bar), "r"(parity)
+      : "memory");
+  return ok != 0;
+}
+
 // Bounded wait on an mbarrier phase. Returns false when the wait gave up
 // (either this waiter timed out or another role already raised `abort`).
 __device__ __forceinline__ bool mbar_wait_bounded(uint32_t bar, uint32_t parity,
@@ -349,3 +364,5 @@ inline cudaError_t launch_pdl(void (*kernel)(KArgs...), dim3 grid, dim3 block, s
 
 int tb_make_tmap_2d_bf16(CUtensorMap* out, const void* base, uint64_t rows, uint64_t cols,
                          uint64_t ld, uint32_t box_rows, uint32_t box_cols, int swizzle128);
+// Whole rows per box, as [cols / 64] slabs of [box_rows x 64] with the 128-byte swizzle: tma_load_3d at (0, row, 0). cols % 64 == 0.
+int tb_make_tmap_slabs_bf16(CUtensorMap* out, const void* base, uint64_t rows, uint64_t cols, uint64_t ld, uint32_t box_rows);

@@ -496,7 +496,7 @@ TB_API int tb_paged_decode(const void* q, long long ldq, int q_heads, const void
   }
   if (rc) return rc;
   if (splits == 1) return 0;
-  return launch_pdl(paged_decode_combine_kernel, dim3(B, N), dim3(128), 0, stream, (const float*)part_acc,
+  return launch_pdl(paged_decode_combine_kernel, dim3(B, N), dim3(H / 4 < 32 ? 32 : H / 4), 0, stream, (const float*)part_acc,
                     (const float*)part_ml, seq_lens, N, H, splits, split_tokens, window, chunk, keep, out_scale, vd, ex, (__nv_bfloat16*)out, ldo) == cudaSuccess ? 0 : -5;
 }
 

@@ -52,13 +52,22 @@ static __global__ void paged_decode_combine_kernel(const float* __restrict__ par
     if (ms != -INFINITY) L += part_ml[(base + s) * 2 + 1] * __expf(ms - M);
   }
   const float inv = L > 0.f ? out_scale * ex.gate_of(b, n) / L : 0.f;
-  for (int d = threadIdx.x; d < vd; d += blockDim.x) {
-    float a = 0.f;
+  __nv_bfloat16* to = out + (long long)b * ldo + (long long)n * vd;
+  for (int d = threadIdx.x * 4; d < vd; d += blockDim.x * 4) {          // H is a multiple of 4
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
     for (int s = 0; s < used; ++s) {
       const float ms = part_ml[(base + s) * 2];
-      if (ms != -INFINITY) a += part_acc[(base + s) * H + d] * __expf(ms - M);
+      if (ms == -INFINITY) continue;
+      const float w = __expf(ms - M) * inv;
+      const float4 v = *reinterpret_cast<const float4*>(part_acc + (base + s) * H + d);
+      a.x += v.x * w; a.y += v.y * w; a.z += v.z * w; a.w += v.w * w;
     }
-    out[(long long)b * ldo + (long long)n * vd + d] = __float2bfloat16(a * inv);
+    if (d + 4 <= vd && (((uintptr_t)to) & 7) == 0) {
+      *reinterpret_cast<uint2*>(to + d) = make_uint2(pack_bf16(a.x, a.y), pack_bf16(a.z, a.w));
+    } else {
+      const float v[4] = {a.x, a.y, a.z, a.w};
+      for (int k = 0; k < 4 && d + k < vd; ++k) to[d + k] = __float2bfloat16(v[k]);
+    }
   }
 }
 

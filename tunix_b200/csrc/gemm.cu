@@ -849,11 +849,12 @@ tb_encode_tiled_fn tb_get_encode_tiled() {
   return fn;
 }
 
-int tb_make_tmap_2d_bf16(CUtensorMap* out, const void* base, uint64_t rows, uint64_t cols,
-                         uint64_t ld, uint32_t box_rows, uint32_t box_cols, int swizzle128) {
+// slabs: a box holds all columns, 64 at a time: [cols / 64][box_rows][64] (a third dimension of the map)
+static int make_tmap(CUtensorMap* out, const void* base, uint64_t rows, uint64_t cols, uint64_t ld, uint32_t box_rows,
+                     uint32_t box_cols, int swizzle128, bool slabs) {
   tb_encode_tiled_fn enc = tb_get_encode_tiled();
   if (!enc) return -1;
-  TmapKey key{base, rows, cols, ld, box_rows, box_cols | (swizzle128 ? 0x80000000u : 0)};
+  TmapKey key{base, rows, cols, ld, box_rows, box_cols | (swizzle128 ? 0x80000000u : 0) | (slabs ? 0x40000000u : 0)};
   {
     std::lock_guard<std::mutex> lk(g_tmap_mu);
     auto it = g_tmap_cache.find(key);
@@ -862,12 +863,12 @@ int tb_make_tmap_2d_bf16(CUtensorMap* out, const void* base, uint64_t rows, uint
       return 0;
     }
   }
-  cuuint64_t dims[2] = {cols, rows};
-  cuuint64_t strides[1] = {ld * 2};
-  cuuint32_t box[2] = {box_cols, box_rows};
-  cuuint32_t estr[2] = {1, 1};
+  cuuint64_t dims[3] = {slabs ? box_cols : cols, rows, cols / box_cols};
+  cuuint64_t strides[2] = {ld * 2, (cuuint64_t)box_cols * 2};
+  cuuint32_t box[3] = {box_cols, box_rows, (cuuint32_t)(cols / box_cols)};
+  cuuint32_t estr[3] = {1, 1, 1};
   auto encode = [&] {
-    return enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
+    return enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, slabs ? 3 : 2, const_cast<void*>(base), dims, strides, box, estr,
                CU_TENSOR_MAP_INTERLEAVE_NONE, swizzle128 ? CU_TENSOR_MAP_SWIZZLE_128B : CU_TENSOR_MAP_SWIZZLE_NONE,
                CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
   };
@@ -884,6 +885,13 @@ int tb_make_tmap_2d_bf16(CUtensorMap* out, const void* base, uint64_t rows, uint
   if (g_tmap_cache.size() > 65536) g_tmap_cache.clear();
   g_tmap_cache.emplace(key, *out);
   return 0;
+}
+int tb_make_tmap_2d_bf16(CUtensorMap* out, const void* base, uint64_t rows, uint64_t cols,
+                         uint64_t ld, uint32_t box_rows, uint32_t box_cols, int swizzle128) {
+  return make_tmap(out, base, rows, cols, ld, box_rows, box_cols, swizzle128, false);
+}
+int tb_make_tmap_slabs_bf16(CUtensorMap* out, const void* base, uint64_t rows, uint64_t cols, uint64_t ld, uint32_t box_rows) {
+  return cols % 64 ? -2 : make_tmap(out, base, rows, cols, ld, box_rows, 64, 1, true);
 }
 
 namespace {

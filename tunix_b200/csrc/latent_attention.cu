@@ -8,9 +8,9 @@
 //   head_product  : a product with a matrix per head and few rows. Single tokens use the absorbed form: the score is
 //                   (U_h^T q) . c + rotated parts, and the weighted sum of latents goes through V_h once, so a query reads R + rot
 //                   columns per key whatever the number of heads.
-//   latent_decode : that attention. One CTA per (query token, up to 32 heads, split of the context): tiles of 64 rows come by TMA
-//                   and serve as keys and, in their first R columns, as values; the heads are the rows of mma.sync tiles. Eight
-//                   warps cut the scores into 16 keys x half of the contraction and the output into columns.
+//   latent_decode : that attention on tcgen05. One CTA per (query token, up to 32 heads, split of the context): tiles of 64 rows come
+//                   by TMA and serve as keys and, in their first R columns, as values. With a handful of heads the products are
+//                   taken the other way round: keys, then value columns, are the 128 rows of a product and heads its columns.
 //
 // Other sizes and 32-bit use window_attn (window_attention.cu) on the absorbed form: one key head, values = the key's columns.
 // This file is compiled without fast-math: latent_write serves the 32-bit mode as well.
@@ -178,233 +178,352 @@ head_product_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, int x_he
   }
 }
 
-// The layout of a CTA's shared memory: two stages of 64 cached rows, the queries, the weights of a tile, its scores (the two halves
-// of the contraction), and what the rows of heads are rescaled by.
+// The layout of a CTA's shared memory: two stages of 64 cached rows, the queries of NH heads, the weights of a tile as product
+// operand, what the softmax warps tell each other per head, barriers. An output product may read 64 columns past a stage (rows that
+// nobody uses), so at least that much follows the second one.
+constexpr int LD_THREADS = 192;
 struct LatentSmem {
-  int stage, q, p, s, row, total;
-  __host__ __device__ LatentSmem(int W, int rows)
-      : stage(64 * W * 2), q(2 * stage), p(q + rows * W * 2), s(p + rows * 128), row(s + 2 * rows * 68 * 4), total(row + 3 * rows * 4) {}
+  int stage, q, p, row, bars, total;
+  __host__ __device__ LatentSmem(int W, int NH) : stage(64 * W * 2), q(2 * stage), p(q + NH * W * 2), row(p + NH * 128), bars(row + 6 * NH * 4) {
+    total = (bars + 128 - q < 8192 ? q + 8192 : bars + 128);
+  }
 };
 
-// CB blocks of 16 output columns per warp, MT tiles of 16 heads. q [T, H, W] absorbed queries, pool rows of W columns.
-template <int CB, int MT>
-__global__ void __launch_bounds__(256, 1)
-latent_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __nv_bfloat16* __restrict__ q, const int* __restrict__ table,
+__device__ __forceinline__ void bar_sync(int id, int threads) { asm volatile("barrier.cta.sync %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
+__device__ __forceinline__ bool bar_any(int id, int threads, bool v) {
+  uint32_t r;
+  asm volatile("{\n.reg .pred p, q;\nsetp.ne.u32 p, %3, 0;\nbarrier.cta.red.or.pred q, %1, %2, p;\nselp.u32 %0, 1, 0, q;\n}"
+               : "=r"(r) : "r"(id), "r"(threads), "r"((uint32_t)v) : "memory");
+  return r != 0;
+}
+// Reduces 16 values per lane over the 16 lanes of a half warp: every exchange with the lane w away (w = 8, 4, 2, 1) halves the values,
+// so that lane i of the half ends up with the result of value half_slot(i).
+template <typename Op>
+__device__ __forceinline__ float half_reduce(float (&x)[16], int lane, Op op) {
+#pragma unroll
+  for (int w = 8; w >= 1; w >>= 1) {
+    const bool hi = lane & w;
+#pragma unroll
+    for (int c = 0; c < w; ++c) {
+      const float keep = hi ? x[w + c] : x[c], give = hi ? x[c] : x[w + c];
+      x[c] = op(keep, __shfl_xor_sync(0xffffffffu, give, w));
+    }
+  }
+  return x[0];
+}
+__device__ __forceinline__ int half_slot(int lane) { return lane & 15; }
+template <int NC>
+__device__ __forceinline__ void tmem_ld_cols(uint32_t addr, float (&v)[NC]) {
+  uint32_t r[NC];
+  if constexpr (NC == 32) tmem_ld_32x32(addr, r);
+  else tmem_ld_32x16(addr, r);
+  tmem_ld_wait();
+#pragma unroll
+  for (int i = 0; i < NC; ++i) v[i] = __uint_as_float(r[i]);
+}
+
+// NH heads (16 or 32) of one query. q [T * H, W] absorbed queries, pool rows of W columns. Products run on tcgen05 with keys or value
+// columns as the rows of a tile and heads as its columns: S^T = K Q^T, 64 rows, which lie in lanes 0-15 of every warp's 32; and
+// O^T += V^T P^T, 128 rows, V being the same shared memory read along its other dimension.
+//   warps 0-3 : softmax. A thread holds the scores of one key with 16 heads and keeps each head's maximum and its own share of the
+//               sums, so nothing crosses lanes unless a score outgrows a maximum by more than 2^8: then the new maxima are shared
+//               and O^T is rescaled. O^T leaves through all lanes (lane = value column).
+//   warp 4    : one thread issues the products, scores of the next tile and outputs of this one in the order in which their
+//               operands are ready.
+//   warp 5    : one thread fetches queries and tiles; a buffer is free when the output product of its tile has retired.
+template <int NH>
+__global__ void __launch_bounds__(LD_THREADS, 1)
+latent_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmQ, const int* __restrict__ table,
                      int max_pages, int page_size, const int* __restrict__ seq_ids, const int* __restrict__ seq_lens, int H, int R, int W,
-                     float scale, int window, const HeadExtras ex, int num_splits, int split_tokens, float* __restrict__ part_acc,
+                     float scale2, int window, const HeadExtras ex, int num_splits, int split_tokens, float* __restrict__ part_acc,
                      float* __restrict__ part_ml, __nv_bfloat16* __restrict__ out, int* __restrict__ status) {
-  constexpr int ROWS = MT * 16, TPR = 256 / ROWS, KPT = 64 / TPR;     // threads per row of scores, keys per thread
+  constexpr uint32_t TMEM_O = 2 * NH, TMEM_COLS = NH == 16 ? 128 : 256;
   extern __shared__ uint8_t smem_raw[];
-  __shared__ __align__(8) unsigned long long full_bars[2];
-  __shared__ int abort_flag;
-  uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);
-  const LatentSmem lay(W, ROWS);
+  const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
+  uint8_t* smem = smem_raw + (base - smem_u32(smem_raw));
+  const LatentSmem lay(W, NH);
+  const uint32_t sq = base + lay.q, sp = base + lay.p, bars = base + lay.bars;
+  // barriers: 0-1 tile arrived, 2-3 tile free, 4-5 scores, 6 weights, 7 outputs, 8 queries
+  const uint32_t bFull = bars, bFree = bars + 16, bS = bars + 32, bP = bars + 48, bO = bars + 56, bQ = bars + 64;
+  volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(smem + lay.bars + 80);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(smem + lay.bars + 84);
+  float* s_row = reinterpret_cast<float*>(smem + lay.row);      // [4][NH]: per warp, maxima and at the end sums
+  float* s_mul = s_row + 4 * NH;                                // [NH]: factors of the outputs
+  float* s_max = s_mul + NH;                                    // [NH]: maxima at the end
   pdl_trigger();
   pdl_wait();
-  const int b = blockIdx.x, h0 = blockIdx.y * ROWS, split = blockIdx.z;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, li = lane >> 3, lr = lane & 7;
+  const int b = blockIdx.x, h0 = blockIdx.y * NH, split = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int len = seq_lens[b];
   const KeyTiles kt(len, window, 0, 0);
   const int tile0 = split * (split_tokens / TILE_KEYS);
-  const int n_tiles = min(kt.total - tile0, split_tokens / TILE_KEYS);
-  if (len <= 0 || n_tiles <= 0) {       // past the end of this sequence: nobody reads this split
+  const int n = min(kt.total - tile0, split_tokens / TILE_KEYS);
+  if (len <= 0 || n <= 0) {             // past the end of this sequence: nobody reads this split
     if (num_splits == 1)
-      for (int i = tid; i < min(ROWS, H - h0) * R; i += 256) out[((long long)b * H + h0) * R + i] = __float2bfloat16(0.f);
+      for (int i = tid; i < min(NH, H - h0) * R; i += LD_THREADS) out[((long long)b * H + h0) * R + i] = __float2bfloat16(0.f);
     return;
   }
+  const int mtiles = (R + 127) >> 7;
   const int* pt = table + (long long)seq_ids[b] * max_pages;
-  const uint32_t base = smem_u32(smem), sq = base + lay.q, sp = base + lay.p;
-  float* s_s = reinterpret_cast<float*>(smem + lay.s);          // [2][ROWS][68]
-  float* s_alpha = reinterpret_cast<float*>(smem + lay.row);    // [ROWS], then the rows' maxima and sums
-  if (tid == 0) {
-    mbar_init(smem_u32(&full_bars[0]), 1);
-    mbar_init(smem_u32(&full_bars[1]), 1);
-    abort_flag = 0;
-    mbar_fence_init();
-  }
-  __syncthreads();
-  auto issue = [&](int tile) {
-    const int k = kt.start(tile0 + tile), buf = tile & 1;
-    const int row = pt[k / page_size] * page_size + k % page_size;
-    const uint32_t bar = smem_u32(&full_bars[buf]);
-    mbar_expect_tx(bar, lay.stage);
-    for (int s = 0; s < W / 64; ++s) tma_load_2d(base + buf * lay.stage + s * 8192, &tmK, bar, s * 64, row);
+  auto row_of = [&](int j) {
+    const int k = kt.start(tile0 + min(j, n - 1));
+    return pt[k / page_size] * page_size + k % page_size;
   };
-  if (tid == 0) {
-    issue(0);
-    if (n_tiles > 1) issue(1);
+  auto fetch = [&](int j, int row) {                    // one thread
+    const uint32_t bar = bFull + 8 * (j & 1), to = base + (j & 1) * lay.stage;
+    mbar_expect_tx(bar, lay.stage);
+    tma_load_3d(to, &tmK, bar, 0, row, 0);
+  };
+  if (tid == 160) {                                     // warp 5: what it fetches first needs no one else
+#pragma unroll
+    for (int i = 0; i < 6; ++i) mbar_init(bars + 8 * i, 1);
+    mbar_init(bP, 128);
+    mbar_init(bO, 1);
+    mbar_init(bQ, 1);
+    *abort_flag = 0;
+    mbar_fence_init();
+    fetch(0, row_of(0));
+    mbar_expect_tx(bQ, NH * W * 2);
+    tma_load_3d(sq, &tmQ, bQ, 0, b * H + h0, 0);
+    if (n > 1) fetch(1, row_of(1));
   }
-  const int cpr = W >> 3;
-  for (int i = tid; i < ROWS * cpr; i += 256) {
-    const int r = i / cpr, c = i - r * cpr;
-    uint4 u = make_uint4(0u, 0u, 0u, 0u);
-    if (h0 + r < H) u = *reinterpret_cast<const uint4*>(q + ((long long)b * H + h0 + r) * W + c * 8);
-    *reinterpret_cast<uint4*>(smem + lay.q + (c >> 3) * (ROWS * 128) + r * 128 + (((c ^ r) & 7) << 4)) = u;
+  if (warp == 4) {
+    tmem_alloc(smem_u32((const void*)tmem_slot), TMEM_COLS);
+    tmem_relinquish();
   }
+  tc_fence_before();
   __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = *tmem_slot;
 
-  const int kg = warp & 3, kh = warp >> 2, steps = W / 32;      // this warp's 16 keys and half of the contraction
-  const int srow = tid / TPR, skey = (tid % TPR) * KPT;         // this thread's row of scores and its keys
-  float m = -INFINITY, l = 0.f;
-  float o[MT][CB][8];
-#pragma unroll
-  for (int x = 0; x < MT; ++x)
-#pragma unroll
-    for (int i = 0; i < CB; ++i)
-#pragma unroll
-      for (int k = 0; k < 8; ++k) o[x][i][k] = 0.f;
-
-  for (int tile = 0; tile < n_tiles; ++tile) {
-    const uint32_t kb = base + (tile & 1) * lay.stage;
-    if (!mbar_wait_bounded(smem_u32(&full_bars[tile & 1]), (tile >> 1) & 1, &abort_flag, status, ST_TIMEOUT_PRODUCER)) break;
-    {
-      float s[MT][2][4];
-#pragma unroll
-      for (int x = 0; x < MT; ++x)
-#pragma unroll
-        for (int k = 0; k < 4; ++k) s[x][0][k] = s[x][1][k] = 0.f;
-#pragma unroll 4
-      for (int ks = kh * steps; ks < (kh + 1) * steps; ++ks) {
-        uint32_t kf[4];
-        {
-          const int r = kg * 16 + (li >> 1) * 8 + lr, c = ks * 2 + (li & 1);
-          ldsm_x4(kf, kb + (c >> 3) * 8192 + r * 128 + (((c ^ r) & 7) << 4));
-        }
-#pragma unroll
-        for (int x = 0; x < MT; ++x) {
-          uint32_t a[4];
-          const int r = x * 16 + (li & 1) * 8 + lr, c = ks * 2 + (li >> 1);
-          ldsm_x4(a, sq + (c >> 3) * (ROWS * 128) + r * 128 + (((c ^ r) & 7) << 4));
-          mma_16816(s[x][0], a, kf[0], kf[1]);
-          mma_16816(s[x][1], a, kf[2], kf[3]);
-        }
-      }
-#pragma unroll
-      for (int x = 0; x < MT; ++x)
-#pragma unroll
-        for (int nb = 0; nb < 2; ++nb) {
-          float* d = s_s + (kh * ROWS + x * 16 + (lane >> 2)) * 68 + kg * 16 + nb * 8 + 2 * (lane & 3);
-          *reinterpret_cast<float2*>(d) = make_float2(s[x][nb][0], s[x][nb][1]);
-          *reinterpret_cast<float2*>(d + 8 * 68) = make_float2(s[x][nb][2], s[x][nb][3]);
-        }
-    }
-    __syncthreads();
-    {
-      const int t0 = kt.start(tile0 + tile) + skey;
-      float v[KPT], mx = -INFINITY;
-#pragma unroll
-      for (int k = 0; k < KPT; k += 4) {
-        const float4 a = *reinterpret_cast<const float4*>(s_s + srow * 68 + skey + k);
-        const float4 c = *reinterpret_cast<const float4*>(s_s + (ROWS + srow) * 68 + skey + k);
-        v[k] = a.x + c.x; v[k + 1] = a.y + c.y; v[k + 2] = a.z + c.z; v[k + 3] = a.w + c.w;
-      }
-#pragma unroll
-      for (int k = 0; k < KPT; ++k) {
-        v[k] = t0 + k < len && t0 + k >= kt.w_lo ? v[k] * scale : -INFINITY;
-        mx = fmaxf(mx, v[k]);
-      }
-#pragma unroll
-      for (int x = TPR / 2; x >= 1; x >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, x));
-      const float mn = fmaxf(m, mx), c = m == -INFINITY ? 0.f : quick_exp(m - mn);
-      float ps = 0.f;
-#pragma unroll
-      for (int k = 0; k < KPT; ++k) {
-        v[k] = v[k] == -INFINITY ? 0.f : quick_exp(v[k] - mn);
-        ps += v[k];
-      }
-      l = l * c + ps;
-      m = mn;
-      if (tid % TPR == 0) s_alpha[srow] = c;
-      uint8_t* d = smem + lay.p + srow * 128 + ((((skey >> 3) ^ srow) & 7) << 4) + (skey & 7) * 2;
-      if (KPT == 8)
-        *reinterpret_cast<uint4*>(d) = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[KPT - 4], v[KPT - 3]), pack_bf16(v[KPT - 2], v[KPT - 1]));
-      else
-        *reinterpret_cast<uint2*>(d) = make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
-    }
-    __syncthreads();
-#pragma unroll
-    for (int x = 0; x < MT; ++x) {
-      const float a0 = s_alpha[x * 16 + (lane >> 2)], a1 = s_alpha[x * 16 + (lane >> 2) + 8];
-#pragma unroll
-      for (int i = 0; i < CB; ++i) {
-        o[x][i][0] *= a0; o[x][i][1] *= a0; o[x][i][4] *= a0; o[x][i][5] *= a0;
-        o[x][i][2] *= a1; o[x][i][3] *= a1; o[x][i][6] *= a1; o[x][i][7] *= a1;
+  if (warp == 5) {
+    if (tid == 160) {
+      for (int j = 2; j < n; ++j) {
+        const int row = row_of(j);
+        if (!mbar_wait_bounded(bFree + 8 * (j & 1), ((j >> 1) - 1) & 1, abort_flag, status, ST_TIMEOUT_PRODUCER)) break;
+        fetch(j, row);
       }
     }
-#pragma unroll
-    for (int kk = 0; kk < 4; ++kk) {
-      uint32_t a[MT][4];
-#pragma unroll
-      for (int x = 0; x < MT; ++x) {
-        const int r = x * 16 + (li & 1) * 8 + lr, c = kk * 2 + (li >> 1);
-        ldsm_x4(a[x], sp + r * 128 + (((c ^ r) & 7) << 4));
-      }
-#pragma unroll
-      for (int i = 0; i < CB; ++i) {
-        const int nb = warp + 8 * i;
-        if (nb * 16 < R) {                                      // the whole warp
-          uint32_t vf[4];
-          const int r = kk * 16 + (li & 1) * 8 + lr, c = nb * 2 + (li >> 1);
-          ldsm_x4_t(vf, kb + (c >> 3) * 8192 + r * 128 + (((c ^ r) & 7) << 4));
-#pragma unroll
-          for (int x = 0; x < MT; ++x) {
-            float(&lo)[4] = *reinterpret_cast<float(*)[4]>(&o[x][i][0]);
-            float(&hi)[4] = *reinterpret_cast<float(*)[4]>(&o[x][i][4]);
-            mma_16816(lo, a[x], vf[0], vf[1]);
-            mma_16816(hi, a[x], vf[2], vf[3]);
+  } else if (warp == 4) {
+    if (elect_one()) {
+      const uint32_t idesc_s = make_idesc_bf16(64, NH, 0, 0), idesc_o = make_idesc_bf16(128, NH, 1, 0);
+      // descriptors of a tile further along are the base plus (byte offset >> 4)
+      const uint64_t kd0 = make_smem_desc(base, 16, 1024), qd0 = make_smem_desc(sq, 16, 1024);
+      const uint64_t vd0 = make_smem_desc(base, 8192, 1024), pd0 = make_smem_desc(sp, 16, 1024);
+      bool ok = mbar_wait_bounded(bQ, 0, abort_flag, status, ST_TIMEOUT_PRODUCER);
+      int s = 0, o = 0, polls = 0;                      // next score product, next output product
+      long long t0 = clock64();
+      while (ok && o < n) {
+        bool idle = true;
+        if (s < n && s <= o + 1 && mbar_test(bFull + 8 * (s & 1), (s >> 1) & 1)) {
+          tc_fence_after();
+          uint64_t kd = kd0 + (uint64_t)(((s & 1) * lay.stage) >> 4), qd = qd0;
+          const uint32_t d = tmem + (s & 1) * NH;
+          for (int c = 0; c < W / 64; ++c, kd += 8192 >> 4, qd += (NH * 128) >> 4) {
+            umma_f16_ss(d, kd, qd, idesc_s, c != 0);
+            umma_f16_ss(d, kd + 2, qd + 2, idesc_s, 1);
+            umma_f16_ss(d, kd + 4, qd + 4, idesc_s, 1);
+            umma_f16_ss(d, kd + 6, qd + 6, idesc_s, 1);
+          }
+          umma_commit(bS + 8 * (s & 1));
+          ++s;
+          idle = false;
+        }
+        if (o < s && mbar_test(bP, o & 1)) {
+          tc_fence_after();
+          uint64_t vd = vd0 + (uint64_t)(((o & 1) * lay.stage) >> 4);
+          uint32_t d = tmem + TMEM_O;
+          for (int mt = 0; mt < mtiles; ++mt, vd += 16384 >> 4, d += NH) {
+            umma_f16_ss(d, vd, pd0, idesc_o, o != 0);
+            umma_f16_ss(d, vd + (2048 >> 4), pd0 + 2, idesc_o, 1);
+            umma_f16_ss(d, vd + (4096 >> 4), pd0 + 4, idesc_o, 1);
+            umma_f16_ss(d, vd + (6144 >> 4), pd0 + 6, idesc_o, 1);
+          }
+          umma_commit(bO);
+          if (o + 2 < n) umma_commit(bFree + 8 * (o & 1));
+          ++o;
+          idle = false;
+        }
+        if (!idle) {
+          t0 = clock64();
+        } else if ((++polls & 63) == 0) {
+          if (*abort_flag) break;
+          if (clock64() - t0 > SPIN_LIMIT_CYCLES) {
+            *abort_flag = 1;
+            if (status) atomicCAS(status, 0, (int)ST_TIMEOUT_MMA);
+            break;
           }
         }
       }
     }
-    __syncthreads();
-    if (tid == 0 && tile + 2 < n_tiles) issue(tile + 2);        // into the buffer that everyone has just left
-  }
+  } else {
+    const uint32_t lanes = (uint32_t)(warp * 32) << 16;
+    const int key = warp * 16 + (lane & 15);            // this thread's key of a tile
+    const int hb = NH == 32 ? (lane & 16) : 0;          // and the first of its 16 heads: lanes 16-31 take the second half
+    const bool active = NH == 32 || lane < 16;
+    float m[16], l[16];
 #pragma unroll
-  for (int x = TPR / 2; x >= 1; x >>= 1) l += __shfl_xor_sync(0xffffffffu, l, x);
-  if (tid % TPR == 0) {
-    s_alpha[ROWS + srow] = m;
-    s_alpha[2 * ROWS + srow] = l;
-    const int h = h0 + srow;
-    if (num_splits > 1 && h < H) {
-      float* ml = part_ml + (((long long)b * H + h) * num_splits + split) * 2;
-      ml[0] = m;
-      ml[1] = l;
+    for (int c = 0; c < 16; ++c) { m[c] = -INFINITY; l[c] = 0.f; }
+    bool ok = true;
+    for (int j = 0; j < n; ++j) {
+      ok = mbar_wait_bounded(bS + 8 * (j & 1), (j >> 1) & 1, abort_flag, status, ST_TIMEOUT_EPILOGUE);
+      ok = __all_sync(0xffffffffu, ok);
+      tc_fence_after();
+      float z[16];
+      {
+        float v[NH];
+        tmem_ld_cols<NH>(tmem + lanes + (j & 1) * NH, v);
+#pragma unroll
+        for (int c = 0; c < 16; ++c) {
+          z[c] = v[c];
+          if constexpr (NH == 32) {
+            const float other = __shfl_sync(0xffffffffu, v[16 + c], lane & 15);
+            z[c] = lane < 16 ? z[c] : other;
+          }
+        }
+      }
+      const int t0 = kt.start(tile0 + j);
+      if (t0 < kt.w_lo || t0 + TILE_KEYS > len) {       // a tile at an end: not all of its keys are visible
+        const bool seen = t0 + key < len && t0 + key >= kt.w_lo;
+#pragma unroll
+        for (int c = 0; c < 16; ++c) z[c] = seen ? z[c] : -INFINITY;
+      }
+      float over = -INFINITY;                           // how far scores lie above the maxima, in log2 units
+#pragma unroll
+      for (int c = 0; c < 16; ++c) over = fmaxf(over, fmaf(z[c], scale2, -m[c]));
+      if (bar_any(1, 128, (active && over > 8.f) || j == 0 || !ok)) {
+        // every tile has a visible key, so the maxima are finite from the first one on
+        float x[16];
+#pragma unroll
+        for (int c = 0; c < 16; ++c) x[c] = z[c] * scale2;
+        const float top = half_reduce(x, lane, [](float a, float c) { return fmaxf(a, c); });
+        if (active) s_row[warp * NH + hb + half_slot(lane)] = top;
+        if (bar_any(2, 128, !ok)) { ok = false; break; }
+#pragma unroll
+        for (int c = 0; c < 16; ++c) {
+          const float* r = s_row + hb + c;
+          const float y = fmaxf(fmaxf(r[0], r[NH]), fmaxf(r[2 * NH], r[3 * NH]));
+          const bool up = y > m[c] + 8.f;
+          const float alpha = up ? quick_exp2(m[c] - y) : 1.f;
+          if (up) m[c] = y;
+          l[c] *= alpha;
+          if (warp == 0 && (lane & 15) == 0 && active) s_mul[hb + c] = alpha;
+        }
+        if (j > 0) {
+          ok = __all_sync(0xffffffffu, mbar_wait_bounded(bO, (j - 1) & 1, abort_flag, status, ST_TIMEOUT_EPILOGUE));
+          tc_fence_after();
+          if (bar_any(1, 128, !ok)) { ok = false; break; }
+#pragma unroll 1
+          for (int c = 0; c < mtiles * NH; c += 16) {
+            uint32_t o[16];
+            tmem_ld_32x16(tmem + lanes + TMEM_O + c, o);
+            tmem_ld_wait();
+#pragma unroll
+            for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * s_mul[(c & (NH - 1)) + i]);
+            tmem_st_32x16(tmem + lanes + TMEM_O + c, o);
+          }
+          tmem_st_wait();
+        }
+      }
+#pragma unroll
+      for (int c = 0; c < 16; ++c) {
+        z[c] = quick_exp2(fmaf(z[c], scale2, -m[c]));
+        l[c] += z[c];
+      }
+      // the outputs of the tile before have retired: the weights' buffer is free
+      if (j > 0) ok = mbar_wait_bounded(bO, (j - 1) & 1, abort_flag, status, ST_TIMEOUT_EPILOGUE) && ok;
+      if (active) {
+        uint8_t* at = smem + lay.p + hb * 128 + (key & 7) * 2;
+#pragma unroll
+        for (int c = 0; c < 16; c += 2) {               // a pair of heads shares the conversion
+          const uint32_t two = pack_bf16(z[c], z[c + 1]);
+          *reinterpret_cast<uint16_t*>(at + c * 128 + ((((key >> 3) ^ c) & 7) << 4)) = (uint16_t)two;
+          *reinterpret_cast<uint16_t*>(at + c * 128 + 128 + ((((key >> 3) ^ (c + 1)) & 7) << 4)) = (uint16_t)(two >> 16);
+        }
+      }
+      fence_proxy_async_smem();
+      tc_fence_before();
+      mbar_arrive(bP);
+    }
+    bar_sync(1, 128);
+    if (warp == 0 && (lane & 15) == 0 && active) {
+#pragma unroll
+      for (int c = 0; c < 16; ++c) s_max[hb + c] = m[c];
+    }
+    const float sum_l = half_reduce(l, lane, [](float a, float c) { return a + c; });
+    if (active) s_row[warp * NH + hb + half_slot(lane)] = sum_l;
+    bar_sync(2, 128);
+    if (tid < NH) {
+      const float sum = s_row[tid] + s_row[NH + tid] + s_row[2 * NH + tid] + s_row[3 * NH + tid], top = s_max[tid];
+      const int h = h0 + tid;
+      s_mul[tid] = num_splits > 1 || h >= H ? 1.f : 1.f / (sum + quick_exp2(ex.sink_of(h) * LOG2_E - top));
+      if (num_splits > 1 && h < H) {
+        float* ml = part_ml + (((long long)b * H + h) * num_splits + split) * 2;
+        ml[0] = top * 0.6931471805599453f;              // natural units, as the merging kernel has them
+        ml[1] = sum;
+      }
+    }
+    ok = ok && mbar_wait_bounded(bO, (n - 1) & 1, abort_flag, status, ST_TIMEOUT_EPILOGUE);
+    tc_fence_after();
+    // O^T through shared memory (the tiles have been read) to rows of heads
+    if (!bar_any(1, 128, !ok)) {
+      float f[NH];
+#pragma unroll
+      for (int c = 0; c < NH; ++c) f[c] = s_mul[c];
+      for (int mt = 0; mt < mtiles; ++mt) {
+        float v[NH];
+        tmem_ld_cols<NH>(tmem + lanes + TMEM_O + mt * NH, v);
+        const int d = mt * 128 + warp * 32 + lane;
+        if (d < R && num_splits == 1) {
+          uint8_t* to = smem + d * 2;
+#pragma unroll
+          for (int c = 0; c < NH; ++c, to += R * 2 + 16) *reinterpret_cast<__nv_bfloat16*>(to) = __float2bfloat16(v[c] * f[c]);
+        } else if (d < R) {
+          uint8_t* to = smem + d * 4;
+#pragma unroll
+          for (int c = 0; c < NH; ++c, to += R * 4 + 16) *reinterpret_cast<float*>(to) = v[c];
+        }
+      }
     }
   }
   __syncthreads();
-#pragma unroll
-  for (int x = 0; x < MT; ++x)
-#pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      const int r = x * 16 + (lane >> 2) + 8 * half, h = h0 + r;
-      if (h >= H) continue;
-      const float inv = 1.f / (s_alpha[2 * ROWS + r] + quick_exp(ex.sink_of(h) - s_alpha[ROWS + r]));
-#pragma unroll
-      for (int i = 0; i < CB; ++i)
-#pragma unroll
-        for (int g = 0; g < 2; ++g) {
-          const int d = (warp + 8 * i) * 16 + g * 8 + 2 * (lane & 3);
-          if (d >= R) continue;
-          const float v0 = o[x][i][4 * g + 2 * half], v1 = o[x][i][4 * g + 2 * half + 1];
-          if (num_splits == 1)
-            *reinterpret_cast<uint32_t*>(out + ((long long)b * H + h) * R + d) = pack_bf16(v0 * inv, v1 * inv);
-          else
-            *reinterpret_cast<float2*>(part_acc + (((long long)b * H + h) * num_splits + split) * R + d) = make_float2(v0, v1);
-        }
+  if (!*abort_flag) {
+    const int size = num_splits == 1 ? 2 : 4, vec = R * size / 16;      // 16-byte pieces of a head
+    uint8_t* to = num_splits == 1 ? reinterpret_cast<uint8_t*>(out) : reinterpret_cast<uint8_t*>(part_acc);
+    const long long first = ((long long)b * H + h0) * num_splits + (num_splits == 1 ? 0 : split), step = (long long)num_splits * R * size;
+    to += first * R * size;
+    for (int i = tid; i < min(NH, H - h0) * vec; i += LD_THREADS) {
+      const int c = i / vec, k = i - c * vec;
+      *reinterpret_cast<uint4*>(to + c * step + k * 16) = *reinterpret_cast<const uint4*>(smem + c * (R * size + 16) + k * 16);
     }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (*abort_flag) {
+    for (int i = 0; i < 2000; ++i) __nanosleep(1000);   // copies in flight land before the CTA's memory goes away
+  }
+  if (warp == 4) {
+    tc_fence_after();
+    tmem_dealloc(tmem, TMEM_COLS);
+  }
 }
 
-template <int CB, int MT>
-int launch_latent_decode(const CUtensorMap& tm, dim3 grid, cudaStream_t stream, const __nv_bfloat16* q, const int* table, int max_pages,
-                         int page_size, const int* seq_ids, const int* seq_lens, int H, int R, int W, float scale, int window,
-                         HeadExtras ex, int splits, int split_tokens, float* pa, float* pml, __nv_bfloat16* out, int* status) {
+template <int NH>
+int launch_latent_decode(const void* pool, long long pool_rows, const void* q, int T, int H, int R, int W, const int* table, int max_pages,
+                         int page_size, const int* seq_ids, const int* seq_lens, float scale, int window, HeadExtras ex, int splits,
+                         int split_tokens, float* pa, float* pml, __nv_bfloat16* out, int* status, cudaStream_t stream) {
+  constexpr int LIMIT = 226 * 1024;
   static DeviceOnce once;
-  if (once.first() && cudaFuncSetAttribute(latent_decode_kernel<CB, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024) != cudaSuccess)
+  if (once.first() && cudaFuncSetAttribute(latent_decode_kernel<NH>, cudaFuncAttributeMaxDynamicSharedMemorySize, LIMIT) != cudaSuccess)
     return -5;
-  const int smem = LatentSmem(W, MT * 16).total + 1024;
-  if (smem > 226 * 1024) return -2;
-  return launch_pdl(latent_decode_kernel<CB, MT>, grid, dim3(256), smem, stream, tm, q, table, max_pages, page_size, seq_ids, seq_lens, H, R,
-                    W, scale, window, ex, splits, split_tokens, pa, pml, out, status) == cudaSuccess ? 0 : -5;
+  const int smem = LatentSmem(W, NH).total + 1024;
+  if (smem > LIMIT) return -2;
+  CUtensorMap tk, tq;
+  if (tb_make_tmap_slabs_bf16(&tk, pool, (uint64_t)pool_rows, (uint64_t)W, (uint64_t)W, TILE_KEYS) ||
+      tb_make_tmap_slabs_bf16(&tq, q, (uint64_t)T * H, (uint64_t)W, (uint64_t)W, NH))
+    return -3;
+  return launch_pdl(latent_decode_kernel<NH>, dim3(T, (H + NH - 1) / NH, splits), dim3(LD_THREADS), smem, stream, tk, tq, table, max_pages,
+                    page_size, seq_ids, seq_lens, H, R, W, scale * LOG2_E, window, ex, splits, split_tokens, pa, pml, out, status) == cudaSuccess
+             ? 0 : -5;
 }
 
 }  // namespace
@@ -473,22 +592,14 @@ TB_API int tb_latent_decode(const void* q, const void* pool, long long pool_rows
   if (T <= 0 || H <= 0) return 0;
   if (W % 64 || R % 8 || R <= 0 || R > 512 || R > W || page_size % TILE_KEYS || split_tokens <= 0 || split_tokens % TILE_KEYS || tiles <= 0)
     return -2;
-  CUtensorMap tm;
-  if (tb_make_tmap_2d_bf16(&tm, pool, (uint64_t)pool_rows, (uint64_t)W, (uint64_t)W, TILE_KEYS, 64, 1)) return -3;
   const int per = split_tokens / TILE_KEYS, splits = (tiles + per - 1) / per;
   const HeadExtras ex{-INFINITY, sinks, nullptr, 0};
-  const bool two = H > 16;
-  const dim3 grid(T, (H + (two ? 31 : 15)) / (two ? 32 : 16), splits);
-  typedef __nv_bfloat16 bf;
-  int rc;
-#define RUN(CB, MT)                                                                                                                   \
-  launch_latent_decode<CB, MT>(tm, grid, stream, (const bf*)q, table, max_pages, page_size, seq_ids, seq_lens, H, R, W, scale, window, ex, \
-                               splits, split_tokens, part_acc, part_ml, (bf*)out, status)
-  if (R <= 128) rc = two ? RUN(1, 2) : RUN(1, 1);
-  else if (R <= 256) rc = two ? RUN(2, 2) : RUN(2, 1);
-  else rc = two ? RUN(4, 2) : RUN(4, 1);
+#define RUN(NH)                                                                                                                       \
+  launch_latent_decode<NH>(pool, pool_rows, q, T, H, R, W, table, max_pages, page_size, seq_ids, seq_lens, scale, window, ex, splits, \
+                           split_tokens, part_acc, part_ml, (__nv_bfloat16*)out, status, stream)
+  const int rc = H > 16 ? RUN(32) : RUN(16);
 #undef RUN
   if (rc || splits == 1) return rc;
   return launch_pdl(paged_decode_combine_kernel, dim3(T, H), dim3(128), 0, stream, (const float*)part_acc, (const float*)part_ml, seq_lens, H,
-                    R, splits, split_tokens, window, 0, 0, 1.f, R, ex, (bf*)out, (long long)H * R) == cudaSuccess ? 0 : -5;
+                    R, splits, split_tokens, window, 0, 0, 1.f, R, ex, (__nv_bfloat16*)out, (long long)H * R) == cudaSuccess ? 0 : -5;
 }

@@ -1,6 +1,6 @@
 """Serving throughput of layer-stack models beside the closest uniform decoder of equal size:
 `python bench.py --workload stack_serving` or
-`python -m tunix_b200.generate.bench_stack [--models roluzen_2b,roluzen_8b,tovalix_2b,tovalix_8b,zikezen_2b,zikezen_8b]`.
+`python -m tunix_b200.generate.bench_stack [--models roluzen_2b,roluzen_8b,tovalix_2b,..,zigipel_2b,zigipel_8b]`.
 
 For every size: prefill tokens/s (`--prefill-seqs` prompts of `--prefill-len` tokens, one sampled token each) and decode
 tokens/s (`--decode-seqs` sequences at context `--decode-ctx`, `--decode-steps` captured steps), both through
@@ -70,7 +70,9 @@ def flops_per_token(model) -> float:
             elif p.dim() == 2:
                 total += p.numel()
         return total
-    return 2.0 * sum(weights(i) for i in runs)
+    loop_in = getattr(model, "loop_in", None)
+    starts = 0 if loop_in is None else len(cfg.loop_starts()) * loop_in.weight.numel()
+    return 2.0 * (sum(weights(i) for i in runs) + starts)
 
 
 def measure(cfg, args) -> dict:
@@ -129,7 +131,8 @@ def measure(cfg, args) -> dict:
 
 
 def add_arguments(ap) -> None:
-    ap.add_argument("--models", default="roluzen_2b,roluzen_8b,tovalix_2b,tovalix_8b,zikezen_2b,zikezen_8b", help="layer-stack presets (stack_serving)")
+    ap.add_argument("--models", default="roluzen_2b,roluzen_8b,tovalix_2b,tovalix_8b,zikezen_2b,zikezen_8b,zigipel_2b,zigipel_8b",
+                    help="layer-stack presets (stack_serving)")
     ap.add_argument("--prefill-seqs", type=int, default=4)
     ap.add_argument("--prefill-len", type=int, default=4096)
     ap.add_argument("--decode-seqs", type=int, default=64)

@@ -1,4 +1,4 @@
-"""Micro-benchmarks of the layer-stack kernels: `python -m tunix_b200.ops.bench_kernels stack [--model roluzen_8b|tovalix_8b|zikezen_8b]
+"""Micro-benchmarks of the layer-stack kernels: `python -m tunix_b200.ops.bench_kernels stack [--model roluzen_8b|tovalix_8b|zikezen_8b|zigipel_8b]
 [--batch 4 --seq 4096] [--decode-batch 64 --decode-ctx 1024] [--only mlstm_prefill,...]`.
 
 One JSON line per kernel at the sizes of a preset: median time with L2 flushed between iterations, the algorithmic bytes and
@@ -52,6 +52,8 @@ def run(args, peaks, timer) -> None:
         run_tovalix(args, peaks, timer)
     elif family == "zikezen":
         run_zikezen(args, peaks, timer)
+    elif family == "zigipel":
+        run_zigipel(args, peaks, timer)
     else:
         run_roluzen(args, peaks, timer)
 
@@ -237,6 +239,123 @@ def run_zikezen(args, peaks, timer) -> None:
         half, up = rand(n, cfg.hidden_dim), rand(n, cfg.hidden_dim)
         report(f"glu_{phase}", lambda: K.glu_fwd(half, up, K.GLU_SILU), n * cfg.hidden_dim * 6.0)
         del half, up, gw, uw
+
+
+def run_zigipel(args, peaks, timer) -> None:
+    from ..models.config import get_config
+    from ..models.mixers import DistanceAttention, DistanceAttentionSpec, LatentAttention, LatentAttentionSpec
+    from ..models.stack_exec import rope_table
+    from . import functional as F
+    from . import kernels as K
+    from . import stack_kernels as SK
+    report = reporter(args, peaks, timer)
+    dev, bf = torch.device("cuda"), torch.bfloat16
+    cfg = get_config(args.model)
+    first = lambda t: next(s.mixer for s in cfg.layer_specs if isinstance(s.mixer, t))  # noqa: E731
+    a, la, D, ff = first(DistanceAttentionSpec), first(LatentAttentionSpec), cfg.embed_dim, cfg.hidden_dim
+    rand = lambda *s: torch.randn(*s, device=dev).to(bf)  # noqa: E731
+    for phase, rb, B, ctx in phases(args):
+        n, one = rb.n, phase == "decode"
+        # --- residual, embedding, token shift
+        x, y, w, h = torch.randn(n, 1, D, device=dev), rand(n, D), torch.ones(D, device=dev, dtype=bf), rand(n, D)
+        unit, mu, before = torch.ones(1, device=dev, dtype=bf), rand(1, D), torch.zeros(B, D, device=dev)
+        table, pairs, last = rand(cfg.vocab_size, D), rand(cfg.bigram[0] + 1, D), torch.zeros(B, dtype=torch.int64, device=dev)
+        ids = torch.randint(0, cfg.vocab_size, (n,), device=dev)
+        kw = dict(y=y, mix=unit, w_out=unit, w_in=unit, norm_w=w)
+        if one:
+            report("stream_step_shift_decode", lambda: SK.stream_step(x, 1e-6, shift=(mu, before), both=True, rb=rb, **kw), n * D * 22.0)
+        else:
+            report("stream_step_prefill", lambda: SK.stream_step(x, 1e-6, **kw), n * D * 12.0)
+            report("token_shift_prefill", lambda: SK.token_shift(h, mu, before, rb), n * D * 4.0)
+        row = torch.empty(n, 2 * D, device=dev, dtype=bf)
+        report(f"embedding_{phase}", lambda: SK.stream_step(x, 1e-6, tokens=ids, embed=table, pairs=(pairs, cfg.bigram, last), rb=rb,
+                                                            start_out=row[:, D:], w_in=unit, norm_w=w), n * D * 12.0)
+        win = rand(D, 2 * D)
+        report(f"loop_product_{phase}", lambda: K.gemm(row, win, out=x.view(n, D), bias=y[0]), n * D * 8.0 + 4.0 * D * D, 4.0 * n * D * D)
+        report(f"like_rmsnorm_{phase}", lambda: K.rmsnorm_fwd(y, w, 1e-6, want_rstd=False), n * D * 4.0)
+        half, up, wide_row = rand(n, ff), rand(n, ff), torch.empty(n, ff + a.heads * a.vdim, device=dev, dtype=bf)
+        report(f"glu_gelu_{phase}", lambda: K.glu_fwd(half, up, K.GLU_GELU, wide_row[:, a.heads * a.vdim:]), n * ff * 6.0)
+        report(f"like_glu_{phase}", lambda: K.glu_fwd(half, up, K.GLU_SILU), n * ff * 6.0)
+        del x, table, pairs, half, up, wide_row, row, win
+        # --- distance attention
+        m = DistanceAttention(a, 8, 1e-6, bf, dev)
+        NQ, NK, NV = a.heads * a.dim, a.kv_heads * a.dim, a.kv_heads * a.vdim
+        kp, vp, pt = page_pool(B, ctx, NK, NV)
+        proj, gate, sinks, bias = rand(n, NQ + NK + NV), rand(n, a.heads), torch.zeros(a.heads, device=dev), m.bias_table(ctx)
+        report(f"value_norm_write_{phase}", lambda: SK.rope_norm_write(proj, 0, NQ, NQ + NK, None, None, 0, 1e-6, rb, pt, 64, 0, a.kv_heads,
+                                                                       a.dim, a.vdim, kp, vp, norm_qk=False, norm_v=True), n * (NK + NV) * 4.0)
+        cos, sin = rope_table(ctx, a.dim, 1e4, dev)
+        report(f"like_rope_norm_write_{phase}", lambda: SK.rope_norm_write(proj, 0, NQ, NQ + NK, cos, sin, a.dim, 1e-6, rb, pt, 64, a.heads,
+                                                                           a.kv_heads, a.dim, a.vdim, kp, vp), n * (NQ + NK + NV) * 4.0)
+        seen = sum(min(i + 1, a.window) + min(max(i + 1 - a.window, 0), a.keep_first) for i in range(args.seq)) * float(B)
+        ext = dict(keep_first=a.keep_first, bias=bias, sinks=sinks, gate=gate)
+        if one:
+            keys = min(ctx, a.window + a.keep_first)
+            nb = B * keys * (NK + NV) * 2.0 + n * NQ * 4.0
+            split = K.decode_split_tokens(B, a.kv_heads, min(ctx, a.window + a.keep_first + 128))
+            q3, lens_t = proj[:, :NQ].unflatten(1, (a.heads, a.dim)), rb.pos0 + 1
+            pd = lambda **o: K.paged_decode(q3, kp, vp, pt, rb.slot, lens_t, num_kv_heads=a.kv_heads, page_size=64, max_ctx=ctx,  # noqa: E731
+                                            split_tokens=split, scale=a.scale, window=a.window, **o)
+            report("attention_decode", lambda: pd(**ext), nb)
+            report("like_paged_decode", lambda: pd(), nb, note="same window; no bias, sinks, gates, kept tokens")
+        else:
+            nb, fl = n * (2 * NQ + NK + NV) * 2.0, seen * a.heads * (a.dim + a.vdim) * 2.0
+            pk = dict(num_heads=a.heads, num_kv_heads=a.kv_heads, head_dim=a.dim, scale=a.scale, window=a.window)
+            q3 = proj.as_strided((n, a.heads, a.dim), (proj.stride(0), a.dim, 1))
+            report("attention_prefill", lambda: K.attn_fwd_paged(q3, kp, vp, rb, pt, 64, **ext, **pk), nb, fl)
+            q4 = rand(B, args.seq, a.heads, a.dim)
+            k4, v4 = (rand(B, args.seq, a.kv_heads, a.dim) for _ in range(2))
+            seg = torch.ones(B, args.seq, dtype=torch.int32, device=dev)
+            win = sum(min(i + 1, a.window) for i in range(args.seq)) * float(B) * a.heads * a.dim * 4.0
+            att = lambda s: F.attention(q4, k4, v4, scale=a.scale, causal=True, window=a.window, seg_q=s, seg_k=s)  # noqa: E731
+            with torch.no_grad():
+                report("like_attn_fwd", lambda: att(None), nb, win, note="same window, no bias")
+                report("like_attn_fwd_segments", lambda: att(seg), nb, win, note="as the padded prefill of uniform decoders calls it")
+            del q4, k4, v4
+        del kp, vp, proj
+        # --- latent attention
+        m = LatentAttention(la, D, 1e-6, bf, dev)
+        for p in m.parameters():
+            p.data.normal_(0, 0.05)
+        H, R, qd, W = la.heads, la.kv_rank, la.dim + la.rot_dim, la.stored(bf)[0]
+        wide, wide_v = la.tile_heads()
+        pages = -(-ctx // 64)
+        pool = torch.randn(B * pages, 64, W, device=dev).to(bf)
+        pool[..., la.width:] = 0
+        pt = torch.randperm(B * pages, device=dev).int().view(B, pages)
+        proj, cos_sin = rand(n, H * qd + la.width), rope_table(ctx, la.rot_dims, la.rot_base, dev, la.rot_scaling)
+        report(f"latent_write_{phase}", lambda: SK.latent_write(proj, H * qd, m.kv_norm.weight, *cos_sin, la.rot_dims, 1e-6, rb, pt, 64, H, la.dim,
+                                                                la.rot_dim, R, pool), n * (H * la.rot_dim * 4.0 + la.width * 4.0))
+        sinks, q = torch.zeros(H, device=dev), proj[:, :H * qd].unflatten(1, (H, qd))
+        if one:
+            uk, uv = m.uk_proj.weight.data.view(H, la.dim, R), m.uv_proj.weight.data.view(H, la.vdim, R)
+            q1, out = torch.zeros(n, H, W, device=dev, dtype=bf), torch.empty(n, H, la.vdim, device=dev, dtype=bf)
+            report("head_product_keys_decode", lambda: SK.head_product(q, uk, q1, tail=la.rot_dim), n * H * (qd + W) * 2.0 + uk.numel() * 2,
+                   2.0 * n * H * la.dim * R)
+            dec = lambda: SK.latent_decode(q1, pool, pt, 64, rb.slot, rb.pos0 + 1, rank=R, scale=la.scale, window=la.window, sinks=sinks,  # noqa: E731
+                                           max_ctx=ctx)
+            keys = min(ctx, la.window)
+            report("latent_decode", dec, B * keys * la.width * 2.0 + n * H * (la.width + R) * 2.0, 2.0 * B * keys * H * (la.width + R))
+            att = dec()
+            report("head_product_values_decode", lambda: SK.head_product(att, uv, out, transposed=True), n * H * (R + la.vdim) * 2.0 + uv.numel() * 2,
+                   2.0 * n * H * la.vdim * R)
+            wk = rand(H * la.dim, D)
+            report("like_narrow_gemm_decode", lambda: K.gemm(h, wk), n * D * 2.0 + n * H * la.dim * 2 + wk.numel() * 2, note="a projection")
+        else:
+            plan, expand = rb.latent_plan(la.window), m.expansion(W, wide, wide_v)
+            rows = plan.blocks[0].shape[0] * 64
+            report("latent_gather_prefill", lambda: SK.latent_gather(pool, *plan.blocks, pt, 64), rows * W * 4.0)
+            g = SK.latent_gather(pool, *plan.blocks, pt, 64)
+            report("latent_expand_prefill", lambda: K.gemm(g, expand), rows * (W + H * (la.dim + la.rot_dim + la.vdim)) * 2.0,
+                   2.0 * rows * R * H * (la.dim + la.vdim))
+            kv = K.gemm(g, expand)
+            q3 = proj.as_strided((n, H, wide), (proj.stride(0), qd, 1))
+            fl = sum(min(i + 1, la.window) for i in range(args.seq)) * float(B) * H * (qd + la.vdim) * 2.0
+            report("latent_attention_prefill", lambda: K.attn_fwd_paged(q3, kv[:, :H * wide], kv[:, H * wide:], rb, plan.table, 64, num_heads=H,
+                                                                        num_kv_heads=H, head_dim=wide, scale=la.scale, window=la.window,
+                                                                        sinks=sinks, value_dim=la.vdim, tiles=plan.tiles, slots=plan.entries),
+                   n * H * (2.0 * qd + 2.0 * la.vdim) * 2.0, fl)
+        del pool, proj
 
 
 def run_roluzen(args, peaks, timer) -> None:

@@ -344,9 +344,10 @@ def head_product(x, w, out, *, transposed: bool = False, x_rows=None, out_rows=N
 
 
 def latent_splits(tokens: int, heads: int, tiles: int) -> int:
-    """Tiles of 64 keys per CTA of `latent_decode`: whole waves of one CTA per SM, each with a fixed cost of about two tiles."""
+    """Tiles of 64 keys per CTA of `latent_decode`: whole waves of one CTA per SM, each with a fixed cost of about two tiles, and about
+    three for merging splits."""
     groups = -(-heads // (32 if heads > 16 else 16))
-    cost = lambda per: -(-tokens * groups * -(-tiles // per) // 148) * (per + 2)  # noqa: E731
+    cost = lambda per: -(-tokens * groups * -(-tiles // per) // 148) * (per + 2) + (3 if per < tiles else 0)  # noqa: E731
     return min(range(1, tiles + 1), key=lambda per: (cost(per), -per))
 
 
