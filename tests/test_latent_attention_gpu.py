@@ -23,7 +23,8 @@ def rot_dict(sp):
     return {"dims": sp.rot_dims, "base": sp.rot_base, "scaling": {"factor": s.factor, "original": s.original, "fast": s.fast, "slow": s.slow}}
 
 
-SIZES = [(3, 16, 8, 24, 40), (3, 7, 6, 5, 13), (20, 96, 64, 128, 136), (2, 48, 16, 40, 264), (17, 104, 24, 64, 512), (1, 128, 128, 64, 72)]
+SIZES = [(3, 16, 8, 24, 40), (3, 7, 6, 5, 13), (20, 96, 64, 128, 136), (2, 48, 16, 40, 264), (17, 104, 24, 64, 512), (1, 128, 128, 64, 72), (3, 64, 16, 56, 88),
+         (2, 128, 64, 128, 320)]
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, BF])
@@ -149,12 +150,13 @@ def expanded(c, q, parts, uk, uv, sink):
     rb = batch(parts)
     plan = rb.latent_plan(sp.window)
     assert plan.blocks is not None
-    kv = K.gemm(SK.latent_gather(c.pool, *plan.blocks, c.table, c.page), m.expansion(c.W, wide, wide_v))
+    rows, w = SK.latent_gather(c.pool, *plan.blocks, c.table, c.page), m.expansion(c.W)
+    kv, keys = K.gemm(rows[:, :w.shape[1]], w), sp.heads * (sp.dim if sp.split_keys else wide)
     qd = sp.dim + sp.rot_dim
     row = torch.cat([q.reshape(q.shape[0], -1), torch.full((q.shape[0], wide + 8), 2.0, dtype=BF, device="cuda")], 1)
-    out = K.attn_fwd_paged(row.as_strided((q.shape[0], sp.heads, wide), (row.stride(0), qd, 1)), kv[:, :sp.heads * wide], kv[:, sp.heads * wide:], rb,
+    out = K.attn_fwd_paged(row.as_strided((q.shape[0], sp.heads, wide), (row.stride(0), qd, 1)), kv[:, :keys], kv[:, keys:], rb,
                            plan.table, 64, num_heads=sp.heads, num_kv_heads=sp.heads, head_dim=wide, scale=sp.scale, window=sp.window, sinks=sink,
-                           value_dim=sp.vdim, tiles=plan.tiles, slots=plan.entries)
+                           value_dim=sp.vdim, tiles=plan.tiles, slots=plan.entries, shared_keys=(rows, sp.kv_rank) if sp.split_keys else None)
     return out.view(q.shape[0], sp.heads, sp.vdim), plan
 
 
@@ -211,7 +213,7 @@ def test_expanded_portions(sizes, window):
 
 @pytest.mark.parametrize("window", [20, 64, 70, 129, 128])
 @pytest.mark.parametrize("form", ["absorbed", "expanded"])
-@pytest.mark.parametrize("sizes", [(3, 16, 16, 24, 64), (20, 64, 64, 128, 136)])
+@pytest.mark.parametrize("sizes", [(3, 16, 16, 24, 64), (20, 96, 64, 128, 136), (4, 128, 64, 104, 200)])
 def test_one_key_at_a_window_edge(sizes, form, window):
     """The rotated part singles out one key: seen, the output is its value; just outside, it is something else."""
     sp = spec(*sizes, window=window, scale=0.5)

@@ -495,6 +495,7 @@ def test_rows_of_both_sublayers_are_one_product():
     assert torch.equal(ex.w[1]["o"][:, n:], mlp.down_proj.weight) and torch.equal(ex.w[1]["o"][:, :n], lat.o_proj.weight)
     sp, e = lat.spec, ex.w[1]["expand"]
     wide, wide_v = sp.tile_heads()
+    assert not sp.split_keys
     row = torch.randn(sp.stored(torch.bfloat16)[0])
     row[sp.width:] = 0
     kv = e.float() @ row
@@ -504,6 +505,15 @@ def test_rows_of_both_sublayers_are_one_product():
     assert torch.allclose(v[:, :sp.vdim].flatten(), lat.uv_proj.weight.float() @ c, atol=1e-5)
     assert torch.equal(k[:, sp.dim:sp.dim + sp.rot_dim], row[sp.kv_rank:sp.width].expand(sp.heads, -1))
     assert k[:, sp.dim + sp.rot_dim:].eq(0).all() and v[:, sp.vdim:].eq(0).all() and ex.w[1]["sinks"].eq(3).all()
+    import dataclasses
+
+    from tunix_b200.models.mixers import create_mixer
+    whole = create_mixer(dataclasses.replace(sp, dim=64), 96, 1e-5, torch.bfloat16)      # keys of whole slabs: the rotated part stays behind
+    whole.uk_proj.weight.data.normal_()
+    whole.uv_proj.weight.data.normal_()
+    e, n = whole.expansion(64), 64 * sp.heads
+    assert e.shape == (n + 64 * sp.heads, sp.kv_rank) and torch.equal(e[:n], whole.uk_proj.weight)
+    assert torch.equal(e[n:].view(sp.heads, 64, -1)[:, :sp.vdim].flatten(0, 1), whole.uv_proj.weight) and e[n:].view(sp.heads, 64, -1)[:, sp.vdim:].eq(0).all()
     want = -0.25 * torch.log1p(model.layers[0].mixer.r2.double()[:, None] * torch.arange(32).double())
     assert torch.allclose(ex._far[(0, 32)].double(), want, atol=1e-6)
     assert set(ex.pack_sources()[1]) == {"proj", "gu", "o"}

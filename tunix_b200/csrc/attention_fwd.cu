@@ -53,6 +53,8 @@ struct AttnArgs {
   const __nv_bfloat16* gate; // paged: rows ldg apart, or null: head n's output is multiplied by sigmoid(gate[row, n])
   long long ldg;
   int q_heads;               // paged: columns from one query head to the next
+  int k_own, k_col;          // paged: 64-column slabs of a key that every head has of its own; the others are columns k_col ..
+                             // of rows that all heads share
   float out_scale;           // paged: factor of the output
 };
 
@@ -79,10 +81,11 @@ struct FwdCfg {
   static constexpr int TMEM_COLS = (128 + HV) <= 256 ? 256 : 512;
 };
 
+// five warps of two CTAs leave a scheduler three warps: at most 168 registers a thread
 template <int H, int HV, bool PAGED>
-__global__ void __launch_bounds__(160, 1)
+__global__ void __launch_bounds__(160, FwdCfg<H, HV>::SMEM_BYTES <= 113 * 1024 ? 2 : 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-                const __grid_constant__ CUtensorMap tmV, const AttnArgs a) {
+                const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmR, const AttnArgs a) {
   using C_ = FwdCfg<H, HV>;
   constexpr int NV = C_::NV;
   extern __shared__ uint8_t smem_raw[];
@@ -162,8 +165,11 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         mbar_expect_tx(barK, C_::K_BYTES);
         const int row = block_row(j);
 #pragma unroll
-        for (int c = 0; c < C_::HS; ++c)
-          tma_load_2d(sK + c * (BKV * 128), &tmK, barK, kvh * H + 64 * c, row);
+        for (int c = 0; c < C_::HS; ++c) {
+          if (!PAGED) tma_load_2d(sK + c * (BKV * 128), &tmK, barK, kvh * H + 64 * c, row);
+          else if (c < a.k_own) tma_load_2d(sK + c * (BKV * 128), &tmK, barK, (kvh * a.k_own + c) * 64, row);
+          else tma_load_2d(sK + c * (BKV * 128), &tmR, barK, a.k_col + (c - a.k_own) * 64, row);
+        }
       };
       auto load_v = [&](int j) {
         const int buf = j % NV;
@@ -422,7 +428,7 @@ int launch_fwd(const void* q, const void* k, const void* v, const AttnArgs& a, l
       cudaFuncSetAttribute(attn_fwd_kernel<H, H, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, C_::SMEM_BYTES) != cudaSuccess)
     return -5;
   dim3 grid((a.Tq + BQ - 1) / BQ, a.N, a.B);
-  attn_fwd_kernel<H, H, false><<<grid, 160, C_::SMEM_BYTES, stream>>>(tq, tk, tv, a);
+  attn_fwd_kernel<H, H, false><<<grid, 160, C_::SMEM_BYTES, stream>>>(tq, tk, tv, tk, a);
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
 }
 
@@ -852,20 +858,22 @@ TB_API int tb_attn_fwd(const void* q, const void* k, const void* v, void* o, flo
 }
 
 template <int H, int HV>
-static int launch_fwd_paged(const void* q, long long ldq, int q_cols, const void* k, long long ldk, const void* v, long long ldv, const AttnArgs& a,
-                            long long rows, long long pool_rows, int tiles, cudaStream_t stream) {
+static int launch_fwd_paged(const void* q, long long ldq, int q_cols, const void* k, long long ldk, const void* v, long long ldv, const void* shared,
+                            long long lds, const AttnArgs& a, long long rows, long long pool_rows, int tiles, cudaStream_t stream) {
   using C_ = FwdCfg<H, HV>;
-  CUtensorMap tq, tk, tv;
+  CUtensorMap tq, tk, tv, tr;
   // heads that lie closer than H columns: the columns behind a head meet the zeros behind the stored key
   if (tb_make_tmap_2d_bf16(&tq, q, (uint64_t)rows, (uint64_t)q_cols, (uint64_t)ldq, BQ, 64, 1) ||
-      tb_make_tmap_2d_bf16(&tk, k, (uint64_t)pool_rows, (uint64_t)a.KH * H, (uint64_t)ldk, BKV, 64, 1) ||
+      tb_make_tmap_2d_bf16(&tk, k, (uint64_t)pool_rows, (uint64_t)a.KH * a.k_own * 64, (uint64_t)ldk, BKV, 64, 1) ||
       tb_make_tmap_2d_bf16(&tv, v, (uint64_t)pool_rows, (uint64_t)a.KH * HV, (uint64_t)ldv, BKV, 64, 1))
     return -3;
   static DeviceOnce once;
   if (once.first() &&
       cudaFuncSetAttribute(attn_fwd_kernel<H, HV, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, C_::SMEM_BYTES) != cudaSuccess)
     return -5;
-  attn_fwd_kernel<H, HV, true><<<dim3(tiles, a.N), 160, C_::SMEM_BYTES, stream>>>(tq, tk, tv, a);
+  tr = tk;
+  if (shared && tb_make_tmap_2d_bf16(&tr, shared, (uint64_t)pool_rows, (uint64_t)lds, (uint64_t)lds, BKV, 64, 1)) return -3;
+  attn_fwd_kernel<H, HV, true><<<dim3(tiles, a.N), 160, C_::SMEM_BYTES, stream>>>(tq, tk, tv, tr, a);
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
 }
 
@@ -875,10 +883,12 @@ static int launch_fwd_paged(const void* q, long long ldq, int q_cols, const void
 // tokens lies in one page and is fetched by TMA through the page table. window, chunk <= 0: none; softcap <= 0: none. The unused
 // tail of a page must hold finite values. sink: one more score without a value in the sum of the weights (-inf: none), or sinks
 // fp32 [N], one per head. gate bf16, rows ldg apart, or null: head h's output is multiplied by sigmoid(gate[row, h]). out [n, ldo],
-// 16-byte aligned, head h at columns h * vd (the first vd <= HV value columns, a multiple of 8), times out_scale.
+// 16-byte aligned, head h at columns h * vd (the first vd <= HV value columns, a multiple of 8), times out_scale. shared bf16 [pool_rows,
+// lds] or null: what lies behind the first k_own columns (a multiple of 64) of a key is the same for all heads, columns k_col .. of
+// these rows (zeros behind the last one).
 // (H, HV): (64, 64), (128, 64), (128, 128), (192, 128), (256, 256).
 TB_API int tb_attn_fwd_paged(const void* q, long long ldq, int q_cols, int q_heads, const void* k_pool, long long ldk, const void* v_pool,
-                             long long ldv, void* out, long long ldo, int n, long long pool_rows, int N, int KH, int H, int HV, int vd,
+                             long long ldv, const void* shared, long long lds, int k_own, int k_col, void* out, long long ldo, int n, long long pool_rows, int N, int KH, int H, int HV, int vd,
                              float scale, float softcap, int window, int chunk, int keep, float sink, const float* sinks,
                              const void* gate, long long ldg, float out_scale, const float* bias, int far, const int* cu,
                              const int* slot, const int* pos0, const int* tile_t0, const int* tile_ent, int tiles,
@@ -886,7 +896,9 @@ TB_API int tb_attn_fwd_paged(const void* q, long long ldq, int q_cols, int q_hea
   if (n <= 0 || tiles <= 0) return 0;
   if (KH <= 0 || N % KH || page_size % BKV || N > 65535 || vd <= 0 || vd > HV || vd % 8 || ldo % 8 || ((uintptr_t)out & 15)) return -2;
   if (q_heads % 8 || ldq % 8 || ldk % 8 || ldv % 8 || ((uintptr_t)q & 15) || ((uintptr_t)k_pool & 15) || ((uintptr_t)v_pool & 15)) return -2;
+  if (k_own <= 0 || k_own % 64 || k_own > H || (!shared && k_own != H) || (shared && (lds % 8 || k_col % 8 || ((uintptr_t)shared & 15)))) return -2;
   AttnArgs a = {};
+  a.k_own = k_own / 64; a.k_col = k_col;
   a.vd = vd; a.sink2 = sink * LOG2E; a.sinks = sinks; a.out_scale = out_scale;
   a.gate = reinterpret_cast<const __nv_bfloat16*>(gate); a.ldg = ldg; a.q_heads = q_heads;
   a.N = N; a.KH = KH; a.scale = scale; a.causal = 1; a.window = window > 0 ? window : 0;
@@ -896,7 +908,7 @@ TB_API int tb_attn_fwd_paged(const void* q, long long ldq, int q_cols, int q_hea
   a.cu = cu; a.slot = slot; a.pos0 = pos0; a.tile_t0 = tile_t0; a.tile_ent = tile_ent; a.table = table;
   a.max_pages = max_pages; a.page_size = page_size;
 #define PAIR(K, V) \
-  if (H == K && HV == V) return launch_fwd_paged<K, V>(q, ldq, q_cols, k_pool, ldk, v_pool, ldv, a, n, pool_rows, tiles, stream)
+  if (H == K && HV == V) return launch_fwd_paged<K, V>(q, ldq, q_cols, k_pool, ldk, v_pool, ldv, shared, lds, a, n, pool_rows, tiles, stream)
   PAIR(64, 64);
   PAIR(128, 64);
   PAIR(128, 128);

@@ -280,6 +280,11 @@ class LatentAttentionSpec:
         """Widths of the key and value heads that portions of prompts expand the latents to."""
         return next((p for p in TILE_PAIRS if p[0] >= self.dim + self.rot_dim and p[1] >= self.vdim), None)
 
+    @property
+    def split_keys(self) -> bool:
+        """Whether the unrotated part of a key fills whole slabs of the tensor-core kernel for portions."""
+        return self.dim % 64 == 0
+
     def stored(self, dtype):
         """Width of a cached row as key and as value: the latent, the rotated part, and zeros up to a multiple of 64."""
         w = -(-self.width // 64) * 64 if self.tiled(dtype) else self.width
@@ -555,10 +560,18 @@ class LatentAttention(nn.Module):
         self.sink = _param(H, dtype=dtype, device=device)
 
     @torch.no_grad()
-    def expansion(self, stored: int, wide: int, wide_v: int) -> torch.Tensor:
-        """[heads * (wide + wide_v), stored]: takes a cached row to the heads' keys (made from the latent, then the shared rotated
-        part, then zeros) and behind all of them to their values."""
+    def expansion(self, stored: int) -> torch.Tensor:
+        """What takes a cached row to the heads' keys and behind all of them to their values, as the attention kernel of portions
+        reads them. Keys of whole slabs of 64 are made from the latent alone, [heads * (dim + value width), rank]: the kernel reads the
+        shared rotated part from the cached rows themselves. Otherwise [heads * (key width + value width), stored]: a key is made
+        from the latent, then the rotated part, then zeros."""
         sp, H = self.spec, self.spec.heads
+        wide, wide_v = sp.tile_heads()
+        if sp.split_keys:
+            w = self.uk_proj.weight.new_zeros(H * (sp.dim + wide_v), sp.kv_rank)
+            w[:H * sp.dim] = self.uk_proj.weight
+            w[H * sp.dim:].view(H, wide_v, sp.kv_rank)[:, :sp.vdim] = self.uv_proj.weight.view(H, sp.vdim, sp.kv_rank)
+            return w
         w = self.uk_proj.weight.new_zeros(H * (wide + wide_v), stored)
         k, v = w[:H * wide].view(H, wide, stored), w[H * wide:].view(H, wide_v, stored)
         k[:, :sp.dim, :sp.kv_rank] = self.uk_proj.weight.view(H, sp.dim, sp.kv_rank)

@@ -190,7 +190,7 @@ class StackExecutor:
                 sp, w = layer.mixer.spec, layer.mixer.uk_proj.weight
                 _plain([layer.mixer.uk_proj, layer.mixer.uv_proj])
                 if sp.tiled(w.dtype):
-                    d["expand"] = layer.mixer.expansion(sp.stored(w.dtype)[0], *sp.tile_heads())
+                    d["expand"] = layer.mixer.expansion(sp.stored(w.dtype)[0])
             if isinstance(layer.mlp, PlainMLP):
                 d["up"], _ = joint_weight([layer.mlp.up_proj])
             elif isinstance(layer.mlp, ExpertsMLP):
@@ -319,12 +319,14 @@ class StackExecutor:
         plan = rb.latent_plan(sp.window)
         if plan.blocks is not None:
             wide, wide_v = sp.tile_heads()
-            kv = linear(SK.latent_gather(lat, *plan.blocks, pool.table, pool.page_size), d["expand"])
+            rows = SK.latent_gather(lat, *plan.blocks, pool.table, pool.page_size)
+            kv = linear(rows[:, :d["expand"].shape[1]], d["expand"])
+            keys = H * (sp.dim if sp.split_keys else wide)
             qw = proj.as_strided((n, H, wide), (proj.stride(0), qd, 1)) if (H - 1) * qd + wide <= proj.shape[1] else \
                 torch.nn.functional.pad(q, (0, wide - qd))
-            K.attn_fwd_paged(qw, kv[:, :H * wide], kv[:, H * wide:], rb, plan.table, 64, num_heads=H, num_kv_heads=H, head_dim=wide,
+            K.attn_fwd_paged(qw, kv[:, :keys], kv[:, keys:], rb, plan.table, 64, num_heads=H, num_kv_heads=H, head_dim=wide,
                              scale=sp.scale, window=sp.window, sinks=d["sinks"], out=to, value_dim=sp.vdim, tiles=plan.tiles,
-                             slots=plan.entries)
+                             slots=plan.entries, shared_keys=(rows, R) if sp.split_keys else None)
         count = n if plan.rows is None else plan.rows.shape[0]
         if count:
             q1 = SK.head_product(q, uk, torch.empty((count, H, W), dtype=h.dtype, device=h.device), x_rows=plan.rows, rows=count,

@@ -342,18 +342,20 @@ def run_zigipel(args, peaks, timer) -> None:
             wk = rand(H * la.dim, D)
             report("like_narrow_gemm_decode", lambda: K.gemm(h, wk), n * D * 2.0 + n * H * la.dim * 2 + wk.numel() * 2, note="a projection")
         else:
-            plan, expand = rb.latent_plan(la.window), m.expansion(W, wide, wide_v)
+            plan, expand = rb.latent_plan(la.window), m.expansion(W)
             rows = plan.blocks[0].shape[0] * 64
             report("latent_gather_prefill", lambda: SK.latent_gather(pool, *plan.blocks, pt, 64), rows * W * 4.0)
             g = SK.latent_gather(pool, *plan.blocks, pt, 64)
-            report("latent_expand_prefill", lambda: K.gemm(g, expand), rows * (W + H * (la.dim + la.rot_dim + la.vdim)) * 2.0,
+            gk, keys = g[:, :expand.shape[1]], H * (la.dim if la.split_keys else wide)
+            report("latent_expand_prefill", lambda: K.gemm(gk, expand), rows * (R + H * (la.dim + la.vdim)) * 2.0,
                    2.0 * rows * R * H * (la.dim + la.vdim))
-            kv = K.gemm(g, expand)
+            kv = K.gemm(gk, expand)
             q3 = proj.as_strided((n, H, wide), (proj.stride(0), qd, 1))
             fl = sum(min(i + 1, la.window) for i in range(args.seq)) * float(B) * H * (qd + la.vdim) * 2.0
-            report("latent_attention_prefill", lambda: K.attn_fwd_paged(q3, kv[:, :H * wide], kv[:, H * wide:], rb, plan.table, 64, num_heads=H,
+            report("latent_attention_prefill", lambda: K.attn_fwd_paged(q3, kv[:, :keys], kv[:, keys:], rb, plan.table, 64, num_heads=H,
                                                                         num_kv_heads=H, head_dim=wide, scale=la.scale, window=la.window,
-                                                                        sinks=sinks, value_dim=la.vdim, tiles=plan.tiles, slots=plan.entries),
+                                                                        sinks=sinks, value_dim=la.vdim, tiles=plan.tiles, slots=plan.entries,
+                                                                        shared_keys=(g, R) if la.split_keys else None),
                    n * H * (2.0 * qd + 2.0 * la.vdim) * 2.0, fl)
         del pool, proj
 

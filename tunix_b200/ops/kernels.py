@@ -284,7 +284,7 @@ _lib.register_cuda_sigs({
     "tb_attn_fwd": [_lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.I, _lib.I, _lib.I, _lib.I, _lib.I, _lib.I,
                     _lib.LL, _lib.LL, _lib.LL, _lib.LL, _lib.F, _lib.F, _lib.I, _lib.I, _lib.I, _lib.P, _lib.P,
                     _lib.P, _lib.P],
-    "tb_attn_fwd_paged": [_lib.P, _lib.LL, _lib.I, _lib.I, _lib.P, _lib.LL, _lib.P, _lib.LL, _lib.P, _lib.LL, _lib.I, _lib.LL, _lib.I,
+    "tb_attn_fwd_paged": [_lib.P, _lib.LL, _lib.I, _lib.I, _lib.P, _lib.LL, _lib.P, _lib.LL, _lib.P, _lib.LL, _lib.I, _lib.I, _lib.P, _lib.LL, _lib.I, _lib.LL, _lib.I,
                           _lib.I, _lib.I, _lib.I, _lib.I, _lib.F, _lib.F, _lib.I, _lib.I, _lib.I, _lib.F, _lib.P, _lib.P, _lib.LL,
                           _lib.F, _lib.P, _lib.I, _lib.P, _lib.P, _lib.P, _lib.P, _lib.P, _lib.I, _lib.P, _lib.I, _lib.I, _lib.P,
                           _lib.P],
@@ -328,28 +328,31 @@ def attn_fwd(q, k, v, *, scale: float, causal: bool = True, window: int = 0, sof
 
 def attn_fwd_paged(q, k_pool, v_pool, rb, table, page_size: int, *, num_heads: int, num_kv_heads: int, head_dim: int, scale: float,
                    softcap: float = 0.0, window: int = 0, chunk: int = 0, keep_first: int = 0, sink: float = NO_SINK, sinks=None,
-                   gate=None, bias=None, out=None, value_dim: int = 0, out_scale: float = 1.0, tiles=None, slots=None) -> torch.Tensor:
+                   gate=None, bias=None, out=None, value_dim: int = 0, out_scale: float = 1.0, tiles=None, slots=None,
+                   shared_keys: tuple | None = None) -> torch.Tensor:
     """Flash attention of the entries of a `ops.ragged.RaggedBatch` (prompt portions) over the paged cache that already
     holds their keys and values. q [n, N * H] bf16, or a view [n, N, H] (heads may overlap where the stored keys have zeros behind
     their own columns) -> [n, N * value_dim]; pools [pages, page_size, KH * H] (or [rows, KH * H], rows may lie apart), page_size a
     multiple of 64; values may have heads of another size. `softcap` / `window` / `chunk` / `keep_first` / `sink` / `sinks` / `gate` /
     `bias` / `out_scale` as in `paged_decode`. `value_dim` (0: as stored): the heads' values stand in the first columns of the stored
     ones. `out`: columns of wider rows. `tiles`, `slots`: other query tiles (first row, entry, number) and page-table rows of the
-    entries than the batch's."""
+    entries than the batch's. `shared_keys` = (rows [as many as the pools', W], column): the pool has only the first columns of the
+    heads' keys (a multiple of 64), the rest of a key is the same for all heads and stands in these rows from that column on."""
     rows = lambda p: p.shape[0] * (page_size if p.dim() == 3 else 1)  # noqa: E731
     HV = v_pool.shape[-1] // num_kv_heads
     n, vd = q.shape[0], value_dim or HV
     q3 = q if q.dim() == 3 else q.view(n, num_heads, head_dim)
     assert q3.shape == (n, num_heads, head_dim) and q3.stride(2) == 1 and page_size % 64 == 0
-    assert k_pool.shape[-1] == num_kv_heads * head_dim and rows(k_pool) == rows(v_pool) and k_pool.stride(-1) == v_pool.stride(-1) == 1
+    own, (shared, col) = k_pool.shape[-1] // num_kv_heads, shared_keys or (None, 0)
+    assert k_pool.shape[-1] == num_kv_heads * own and (own == head_dim or shared is not None) and rows(k_pool) == rows(v_pool) and k_pool.stride(-1) == v_pool.stride(-1) == 1
     assert all(p.dim() == 2 or p.is_contiguous() for p in (k_pool, v_pool))
     if out is None:
         out = torch.empty((n, num_heads * vd), dtype=q.dtype, device=q.device)
     assert out.shape == (n, num_heads * vd) and out.stride(1) == 1
     t0, ent, n_tiles = tiles if tiles is not None else (lambda t: (t[0], t[1], t[3]))(rb.tiles(128))
     rc = _lib.cuda().tb_attn_fwd_paged(q3.data_ptr(), q3.stride(0), (num_heads - 1) * q3.stride(1) + head_dim, q3.stride(1),
-                                       k_pool.data_ptr(), k_pool.stride(-2), v_pool.data_ptr(), v_pool.stride(-2), out.data_ptr(),
-                                       out.stride(0), n, rows(k_pool), num_heads, num_kv_heads, head_dim, HV, vd, float(scale),
+                                       k_pool.data_ptr(), k_pool.stride(-2), v_pool.data_ptr(), v_pool.stride(-2), _lib.ptr(shared),
+                                       0 if shared is None else shared.shape[-1], own, col, out.data_ptr(), out.stride(0), n, rows(k_pool), num_heads, num_kv_heads, head_dim, HV, vd, float(scale),
                                        float(softcap), int(window), int(chunk), int(keep_first), float(sink), _lib.ptr(sinks),
                                        _lib.ptr(gate), 0 if gate is None else gate.stride(0), float(out_scale), _lib.ptr(bias),
                                        0 if bias is None else bias.shape[1] - 1, rb.cu.data_ptr(),
