@@ -24,7 +24,7 @@ def rot_dict(sp):
 
 
 SIZES = [(3, 16, 8, 24, 40), (3, 7, 6, 5, 13), (20, 96, 64, 128, 136), (2, 48, 16, 40, 264), (17, 104, 24, 64, 512), (1, 128, 128, 64, 72), (3, 64, 16, 56, 88),
-         (2, 128, 64, 128, 320)]
+         (2, 128, 64, 128, 320), (40, 32, 16, 48, 64)]
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, BF])

@@ -377,7 +377,7 @@ def test_stream_step_token_pairs_and_rows_beside_it(D, dtype):
     rb.pos0[3] = -1
     n, toks = 8, [3, 0, 49, 7, 7, 1, 2, 30]
     rb.tokens.copy_(torch.tensor(toks))
-    rule = (13, 31, 5)
+    rule = (13, 17, 5)
     last = torch.tensor([11, 22, 33, 44, 55, 66], device="cuda")
     embed, pairs, nw, y = (rand(*s, dtype=dtype, seed=80 + i) for i, s in enumerate([(50, D), (14, D), (D,), (n, D)]))
     one = torch.ones(1, device="cuda", dtype=dtype)

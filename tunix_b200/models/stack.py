@@ -80,7 +80,7 @@ class StackConfig(ModelConfig):
             raise ValueError("this layer form takes distance or latent attention and gated feed-forwards")
         if self.parallel_ff != self.token_shift:
             raise ValueError("shifted mixers and side by side sublayers come together")
-        if self.logit_scale != 1.0 and (self.final_logit_softcap or self.logit_scale <= 0):
+        if self.logit_scale == 0.0 or (self.logit_scale != 1.0 and self.final_logit_softcap):
             raise ValueError(f"a logit scale of {self.logit_scale}" + (" beside a score cap" if self.final_logit_softcap else ""))
         if self.embed_dim % self.norm_groups:
             raise ValueError(f"a width of {self.embed_dim} does not split into {self.norm_groups} norm groups")
@@ -234,7 +234,7 @@ class StackConfig(ModelConfig):
                                   window=lwindow, rot_dims=rot, rot_base=500000.0, rot_scaling=YarnScaling(4.0, 4096.0, 32.0, 1.0))
         specs = tuple(LayerSpec(lat if i % 2 else att, ff) for i in range(n))
         return cls(family="zigipel", vocab_size=vocab, embed_dim=D, layer_specs=specs, loop=loop, loop_input=True,
-                   bigram=(buckets, 31, 7), parallel_ff=True, token_shift=True, ff_bias=True, activation="gelu", logit_scale=0.5)
+                   bigram=(buckets, 4099, 257), parallel_ff=True, token_shift=True, ff_bias=True, activation="gelu", logit_scale=0.5)
 
     @classmethod
     def zigipel_tiny(cls) -> "StackConfig":
